@@ -48,14 +48,9 @@ class _Context:
         self.m = m
         self._rope_changed = _rope_overrides(m.model, rope)
         hp = m.model.hp
-        dtype = m.model.dtype
         self.block_size = block_size
         self.presample = presample
-        if getattr(m.model, "split", False):
-            from .runtime.engine import SplitCache
-            self.cache = SplitCache(m.model.layer_dev, n_blocks * block_size, hp.kv_row, dtype, block_size)
-        else:
-            self.cache = torch.zeros(hp.n_layer, n_blocks * block_size, hp.kv_row, dtype=dtype, device=m.device)
+        self.cache = m.model.make_cache(n_blocks * block_size, 0)
         if n_ctx > m.model.max_positions or self._rope_changed:
             lo, hi = hp.yarn_corr_dims()
             m.model.max_positions = max(n_ctx, m.model.max_positions)

@@ -125,14 +125,21 @@ __global__ void __launch_bounds__(NT) rmsnorm_kernel(const bf16 * __restrict__ x
     JIB_KS(4, 9);
 }
 
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ void put(bf16 * p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void put(float * p, float v) { *p = v; }
+
 // One block per token: c = rmsnorm(ckv[:r]) * w -> cache[slot][:r]; k_pe = rope(ckv[r:]) -> cache[slot][r:];
 // q_pe = rope(q[h][dn:]) -> q_out[t][h][r:].  rope_table [max_pos][dr/2][2] holds (cos, sin) * magnitude.
+// HALF: element i is paired with element i + dr/2 ("rotate half"), else with its neighbour (2i, 2i + 1).
+// ckv == nullptr: the layer reads rows another layer has written; only the query part runs.
 // dry: the same instructions without stores or status reports.
-template <int NT>
-__device__ __noinline__ void mla_qkv_post_row(const bf16 * __restrict__ q, long long q_stride, const bf16 * __restrict__ ckv,
+template <int NT, typename T, bool HALF>
+__device__ __noinline__ void mla_qkv_post_row(const T * __restrict__ q, long long q_stride, const T * __restrict__ ckv,
                                               long long ckv_stride, const float * __restrict__ kv_norm_w, float eps,
                                               const float * __restrict__ rope_table, const int * __restrict__ positions,
-                                              const int * __restrict__ slot_mapping, bf16 * __restrict__ cache, bf16 * __restrict__ q_out,
+                                              const int * __restrict__ slot_mapping, T * __restrict__ cache, T * __restrict__ q_out,
                                               long long qo_row, long long qo_head, int H, int dn, int dr, int r, int max_pos,
                                               long long n_slots, int * status, float * red, bool dry) {
     const int t = blockIdx.x;
@@ -143,61 +150,79 @@ __device__ __noinline__ void mla_qkv_post_row(const bf16 * __restrict__ q, long 
         pos = pos < 0 ? 0 : max_pos - 1;
     }
     const float * cs = rope_table + (size_t) pos * dr;       // dr/2 pairs * 2
-    const bf16 * crow = ckv + (size_t) t * ckv_stride;
-    // latent RMSNorm
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < r; i += NT) {
-        const float v = __bfloat162float(crow[i]);
-        ss += v * v;
-    }
-    ss = block_sum<NT>(ss, red);
-    const float inv = rsqrtf(ss / (float) r + eps);
-    const bool write_kv = slot >= 0 && slot < n_slots;
-    if (slot >= n_slots && !dry) jib_report(status, JIB_ERR_BOUNDS, 11, slot);
-    if (write_kv) {
-        bf16 * dst = cache + (size_t) slot * (r + dr);
+    const int half = dr / 2;
+    if (ckv != nullptr) {
+        const T * crow = ckv + (size_t) t * ckv_stride;
+        // latent RMSNorm
+        float ss = 0.f;
         for (int i = threadIdx.x; i < r; i += NT) {
-            const bf16 v = __float2bfloat16(__bfloat162float(crow[i]) * inv * kv_norm_w[i]);
-            if (!dry) dst[i] = v;
+            const float v = to_f(crow[i]);
+            ss += v * v;
         }
-        for (int i = threadIdx.x; i < dr / 2; i += NT) {
-            const float x0 = __bfloat162float(crow[r + 2 * i]), x1 = __bfloat162float(crow[r + 2 * i + 1]);
-            const float c = cs[2 * i], s = cs[2 * i + 1];
-            const __nv_bfloat162 v = __floats2bfloat162_rn(x0 * c - x1 * s, x0 * s + x1 * c);
-            if (!dry) *(__nv_bfloat162 *) (dst + r + 2 * i) = v;
+        ss = block_sum<NT>(ss, red);
+        const float inv = rsqrtf(ss / (float) r + eps);
+        const bool write_kv = slot >= 0 && slot < n_slots;
+        if (slot >= n_slots && !dry) jib_report(status, JIB_ERR_BOUNDS, 11, slot);
+        if (write_kv) {
+            T * dst = cache + (size_t) slot * (r + dr);
+            for (int i = threadIdx.x; i < r; i += NT) {
+                T v;
+                put(&v, to_f(crow[i]) * inv * kv_norm_w[i]);
+                if (!dry) dst[i] = v;
+            }
+            for (int i = threadIdx.x; i < half; i += NT) {
+                const int i0 = HALF ? i : 2 * i, i1 = HALF ? i + half : 2 * i + 1;
+                const float x0 = to_f(crow[r + i0]), x1 = to_f(crow[r + i1]);
+                const float c = cs[2 * i], s = cs[2 * i + 1];
+                T v0, v1;
+                put(&v0, x0 * c - x1 * s);
+                put(&v1, x0 * s + x1 * c);
+                if (!dry) { dst[r + i0] = v0; dst[r + i1] = v1; }
+            }
         }
     }
     // q rope: H * dr/2 pairs
-    const int half = dr / 2;
-    const bf16 * qrow = q + (size_t) t * q_stride;
-    bf16 * qo = q_out + (size_t) t * qo_row;      // q_out points at the first RoPE element of token 0, head 0
+    const T * qrow = q + (size_t) t * q_stride;
+    T * qo = q_out + (size_t) t * qo_row;      // q_out points at the first RoPE element of token 0, head 0
     for (int i = threadIdx.x; i < H * half; i += NT) {
         const int h = i / half, p = i - h * half;
-        const __nv_bfloat162 xx = *(const __nv_bfloat162 *) (qrow + (size_t) h * (dn + dr) + dn + 2 * p);
-        const float2 f = __bfloat1622float2(xx);
         const float c = cs[2 * p], s = cs[2 * p + 1];
-        const __nv_bfloat162 v = __floats2bfloat162_rn(f.x * c - f.y * s, f.x * s + f.y * c);
-        if (!dry) *(__nv_bfloat162 *) (qo + (size_t) h * qo_head + 2 * p) = v;
+        const T * src = qrow + (size_t) h * (dn + dr) + dn;
+        if constexpr (!HALF && sizeof(T) == 2) {
+            const float2 f = __bfloat1622float2(*(const __nv_bfloat162 *) (src + 2 * p));
+            const __nv_bfloat162 v = __floats2bfloat162_rn(f.x * c - f.y * s, f.x * s + f.y * c);
+            if (!dry) *(__nv_bfloat162 *) (qo + (size_t) h * qo_head + 2 * p) = v;
+        } else {
+            const int i0 = HALF ? p : 2 * p, i1 = HALF ? p + half : 2 * p + 1;
+            const float x0 = to_f(src[i0]), x1 = to_f(src[i1]);
+            T v0, v1;
+            put(&v0, x0 * c - x1 * s);
+            put(&v1, x0 * s + x1 * c);
+            if (!dry) {
+                qo[(size_t) h * qo_head + i0] = v0;
+                qo[(size_t) h * qo_head + i1] = v1;
+            }
+        }
     }
 }
 
-template <int NT>
-__global__ void __launch_bounds__(NT) mla_qkv_post_kernel(const bf16 * __restrict__ q, long long q_stride, const bf16 * __restrict__ ckv,
+template <int NT, typename T, bool HALF>
+__global__ void __launch_bounds__(NT) mla_qkv_post_kernel(const T * __restrict__ q, long long q_stride, const T * __restrict__ ckv,
                                                           long long ckv_stride, const float * __restrict__ kv_norm_w, float eps,
                                                           const float * __restrict__ rope_table, const int * __restrict__ positions,
-                                                          const int * __restrict__ slot_mapping, bf16 * __restrict__ cache,
-                                                          bf16 * __restrict__ q_out, long long qo_row, long long qo_head, int H, int dn,
+                                                          const int * __restrict__ slot_mapping, T * __restrict__ cache,
+                                                          T * __restrict__ q_out, long long qo_row, long long qo_head, int H, int dn,
                                                           int dr, int r, int max_pos, long long n_slots, int * status, int warm) {
     JIB_KS(5, 0);
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
     // positions / slot_mapping are step inputs, uploaded before the first kernel of the step: valid during the dry pass
-    if (warm) mla_qkv_post_row<NT>(q, q_stride, ckv, ckv_stride, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, qo_row,
-                                   qo_head, H, dn, dr, r, max_pos, n_slots, status, red, true);
+    if (warm) mla_qkv_post_row<NT, T, HALF>(q, q_stride, ckv, ckv_stride, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out,
+                                            qo_row, qo_head, H, dn, dr, r, max_pos, n_slots, status, red, true);
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     JIB_KS(5, 1);
-    mla_qkv_post_row<NT>(q, q_stride, ckv, ckv_stride, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, qo_row, qo_head, H,
-                         dn, dr, r, max_pos, n_slots, status, red, false);
+    mla_qkv_post_row<NT, T, HALF>(q, q_stride, ckv, ckv_stride, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, qo_row,
+                                  qo_head, H, dn, dr, r, max_pos, n_slots, status, red, false);
     JIB_KS(5, 9);
 }
 
@@ -399,14 +424,23 @@ int jib_rmsnorm(const void * x, const void * residual, const float * w, void * o
 
 int jib_mla_qkv_post(const void * q, long long q_stride, const void * ckv, long long ckv_stride, const float * kv_norm_w, float eps,
                      const float * rope_table, const int * positions, const int * slot_mapping, void * cache, void * q_out,
-                     long long qo_row, long long qo_head, int T, int H, int dn, int dr, int r, int max_pos, long long n_slots, int * status,
-                     void * stream) {
+                     long long qo_row, long long qo_head, int T, int H, int dn, int dr, int r, int max_pos, long long n_slots, int rot_half,
+                     int f32, int * status, void * stream) {
     if (T <= 0) return 0;
-    if ((dr & 1) || (dn & 1) || (r & 1) || (q_stride & 1) || (qo_row & 1) || (qo_head & 1) || ((uintptr_t) q_out & 3)) return JIB_E_ARG;
-    JIB_LAUNCH((mla_qkv_post_kernel<256>), T, 256, 0, (cudaStream_t) stream, (const bf16 *) q, q_stride, (const bf16 *) ckv, ckv_stride, kv_norm_w,
-                                                                    eps, rope_table, positions, slot_mapping, (bf16 *) cache,
-                                                                    (bf16 *) q_out, qo_row, qo_head, H, dn, dr, r, max_pos, n_slots, status,
-                                                                    jib::warm_for(T));
+    if (dr & 1) return JIB_E_ARG;
+    if (!f32 && !rot_half && ((dn & 1) || (q_stride & 1) || (qo_row & 1) || (qo_head & 1) || ((uintptr_t) q_out & 3))) return JIB_E_ARG;
+#define JIB_POST(TT, HALF)                                                                                                               \
+    JIB_LAUNCH((mla_qkv_post_kernel<256, TT, HALF>), T, 256, 0, (cudaStream_t) stream, (const TT *) q, q_stride, (const TT *) ckv, ckv_stride, \
+               kv_norm_w, eps, rope_table, positions, slot_mapping, (TT *) cache, (TT *) q_out, qo_row, qo_head, H, dn, dr, r, max_pos,       \
+               n_slots, status, jib::warm_for(T))
+    if (f32) {
+        if (rot_half) JIB_POST(float, true);
+        else JIB_POST(float, false);
+    } else {
+        if (rot_half) JIB_POST(bf16, true);
+        else JIB_POST(bf16, false);
+    }
+#undef JIB_POST
     return launched();
 }
 

@@ -66,6 +66,8 @@ typedef struct jib_gemm_desc {
 } jib_gemm_desc;
 
 JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream);
+// The same product on CUDA cores (gemm_simt.cu): fp32 operands (f32 = 1, result fp32), or bf16 operands TMA cannot address.
+JIB_EXPORT int jib_gemm_simt(const jib_gemm_desc * d, int f32, void * stream);
 
 // ---- sampling (sampling.cu) ---------------------------------------------------------------------
 // One id per row from the row's top-k candidates (vals / ids [n][k], sorted by value, descending; k <= 128).
@@ -80,11 +82,12 @@ JIB_EXPORT int jib_embed_gather(const void * table, const int * ids, void * out,
 JIB_EXPORT int jib_rmsnorm(const void * x, const void * residual, const float * w, void * out_norm, void * out_sum, int T, int d,
                            long long x_stride, float eps, void * stream);
 // q_out: where the rotated RoPE part of token 0, head 0 goes; token t, head h at q_out + t * qo_row + h * qo_head (elements):
-// into the absorbed-query buffer [T][H][r + dr] at offset r, or in place into q at offset dn.
+// into the absorbed-query buffer [T][H][r + dr] at offset r, or in place into q at offset dn.  ckv NULL: queries only (the
+// layer reads another layer's latent rows).  rot_half: pairs (i, i + dr/2) instead of (2i, 2i + 1).  f32: fp32 activations and cache.
 JIB_EXPORT int jib_mla_qkv_post(const void * q, long long q_stride, const void * ckv, long long ckv_stride, const float * kv_norm_w,
                                 float eps, const float * rope_table, const int * positions, const int * slot_mapping, void * cache,
                                 void * q_out, long long qo_row, long long qo_head, int T, int H, int dn, int dr, int r, int max_pos,
-                                long long n_slots, int * status, void * stream);
+                                long long n_slots, int rot_half, int f32, int * status, void * stream);
 JIB_EXPORT int jib_argmax(const float * logits, int * out, int n, int V, void * stream);
 JIB_EXPORT int jib_topk(const float * logits, float * vals, int * ids, int n, int V, int k, void * stream);
 JIB_EXPORT int jib_kv_block_copy(void * cache, long long layer_stride_elems, int n_layers, const int * src, const int * dst, int n,
@@ -94,9 +97,11 @@ JIB_EXPORT int jib_gather_rows(const void * x, const int * src_row, void * out, 
 // ---- MoE routing (moe.cu) ---------------------------------------------------------------------
 // logits: fp32 scratch [T][E] (router outputs, kept for inspection).  ids / wts have k + n_shared columns: the last
 // n_shared columns name the shared experts (ids E, E+1, ...; weight 1) so that they run in the grouped GEMMs.
-JIB_EXPORT int jib_moe_gate(const void * g, const float * w_router, const float * bias, float * logits, int * ids, float * wts, int T,
-                            int d, int E, int k, int n_group, int topk_group, float scale, int norm, int sigmoid, int n_shared,
-                            int group_top2, void * stream);
+// bias: added to the scores for the choice only (DeepSeek-V3); logit_bias: added to the router logits before anything else.
+// g NULL: logits already holds the router outputs (fp32 activations).
+JIB_EXPORT int jib_moe_gate(const void * g, const float * w_router, const float * bias, const float * logit_bias, float * logits, int * ids,
+                            float * wts, int T, int d, int E, int k, int n_group, int topk_group, float scale, int norm, int sigmoid,
+                            int n_shared, int group_top2, void * stream);
 // jib_moe_gate + jib_moe_permute (over the k + n_shared id columns) in one launch, for T <= 64.  counter: one device int that is
 // zero between launches.  norm_w != NULL: the rows of g are RMS-normalised first (as jib_rmsnorm would) and stored to g_out.
 JIB_EXPORT int jib_moe_route_fused(const void * g, const float * w_router, const float * bias, float * logits, int * ids, float * wts,
@@ -121,27 +126,64 @@ JIB_EXPORT int jib_moe_combine_norm(const void * y, const int * dest, const floa
                                     const float * norm_w, void * out, void * out_norm, int T, int k, int d, float eps, void * stream);
 
 // ---- attention (mla_attention.cu) -------------------------------------------------------------
-// Split-KV absorbed MLA over the paged latent cache. q [T][H][r+dr] bf16; o_lat [T][H][r] bf16.
+// Split-KV absorbed MLA over the paged latent cache. q [T][H][r+dr], o_lat [T][H][r], cache rows: bf16, or fp32 with f32.
+// window > 0: position i sees j with 0 <= i - j < window.  r <= 1024.
 // part_o [T][n_splits][H][r] fp32 and part_ml [T][n_splits][H][2] fp32 are scratch.
 JIB_EXPORT int jib_mla_attention(const void * q, const void * cache, const int * block_tables, int max_blocks, const int * seq_lens,
                                  const int * q_start, int n_seqs, int T, int H, int r, int dr, int block_size, float scale,
-                                 int n_splits, float * part_o, float * part_ml, void * o_lat, void * stream);
+                                 int window, int n_splits, int f32, float * part_o, float * part_ml, void * o_lat, void * stream);
 
 JIB_EXPORT int jib_mla_combine(const float * part_o, const float * part_ml, int n_splits, int T, int H, int r, void * o_lat,
                                void * stream);
 // tcgen05 flash MLA (mla_flash_tcgen05.cu): r = 512, dr = 64, block size 64 only; qt = query tokens per CTA (1 or 2).
 JIB_EXPORT int jib_mla_flash(const void * q, const void * cache, long long n_slots, const int * block_tables, int max_blocks,
-                             const int * seq_lens, const int * q_start, int n_seqs, int T, int H, float scale, int n_splits, int qt,
+                             const int * seq_lens, const int * q_start, int n_seqs, int T, int H, float scale, int window, int n_splits, int qt,
                              float * part_o, float * part_ml, void * o_lat, int * status, void * stream);
 
 // ---- prefill attention in the per-head form (mha_prefill_tcgen05.cu): head dims 128 + 64 (keys), 128 (values) ---------------
 // jib_kv_gather: lat [total_cap][row_elems] <- the cached latent rows of every sequence, in sequence order; kv_start [n_seqs].
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, void * lat, int * kv_start, int total_cap, void * stream);
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, void * lat, int * kv_start,
+                             int total_cap, void * stream);
 // q [T][H][192] (RoPE applied), kv [total][H][256] = k_nope | v, kpe [total][64] (row stride kpe_stride), out [T][H * 128].
 JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * kv, const void * kpe, long long kpe_stride, long long total,
                                const int * q_start, const int * seq_lens, const int * kv_start, int n_seqs, int T, int H, float scale,
-                               int n_q_tiles, void * out, long long ldo, int * status, void * stream);
+                               int window, int n_q_tiles, void * out, long long ldo, int * status, void * stream);
+
+// ---- parallel blocks over an fp32 residual (parallel_block.cu), per-sequence state (recurrent.cu) ---------------------------
+// What happens to a token's row once its residual value is known: x_out [T][d] fp32; with norm_w, h_out = row / rms * norm_w; with
+// conv_w ([taps][d] fp32, one token per sequence only), hc_out = h + causal convolution of h, whose last taps - 1 inputs live in
+// conv_state [n_state][taps - 1][d] at row seq_slots[t] (negative: none) and are advanced.  positions[t] == 0 starts from zeros.
+typedef struct jib_row_tail {
+    void * x_out;
+    const float * norm_w;
+    void * h_out;
+    const float * conv_w;
+    void * hc_out;
+    void * conv_state;
+    const int * seq_slots;
+    const int * positions;
+    int * status;
+    float eps;
+    int taps, n_state;
+} jib_row_tail;
+JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, int T, int d, int n_vocab, int f32,
+                              const jib_row_tail * tail, void * stream);
+// x_out = x + mult * (sigmoid(gates[:, :d] + b1) * o + sigmoid(gates[:, d:2d] + b2) * sum_j wts[t][j] * y[dest[t][j]]); y NULL: no second
+// sublayer.  x_out may be x.
+JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, const void * gates, long long gate_stride, const float * b1,
+                                const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
+                                const jib_row_tail * tail, void * stream);
+JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
+                            void * stream);
+// out = h + causal convolution over time of h (w [taps][d] fp32); sequence b continues from, and advances, its stored rows.
+JIB_EXPORT int jib_causal_conv(const void * h, const float * w, int taps, void * state, int n_state, const int * seq_slots,
+                               const int * positions, const int * q_start, int n_seqs, int T, int d, int f32, void * out, int * status,
+                               void * stream);
+// Gated recurrence over zxg [T][>= 3W]; state [n_state][W] fp32; single: one token per sequence (row t = sequence t).
+JIB_EXPORT int jib_mingru(const void * zxg, long long ld, const float * zb, const float * xb, float * state, int n_state,
+                          const int * seq_slots, const int * positions, const int * q_start, int n_seqs, int T, int W, int single, int f32,
+                          void * y, int * status, void * stream);
 
 // ---- expert-parallel all-to-all over peer memory (ep_alltoall.cu); ctx is a JibEpCtx (ep_alltoall.h) ---------
 JIB_EXPORT int jib_ep_plan(const int * ids, int T, int k, const struct JibEpCtx * ctx, int site, int * seg, int * pair_dst, void * stream);

@@ -17,7 +17,9 @@
 // the running maximum grew by more than 2^8 since the last rescale (the exponent base stays behind the true maximum by
 // at most that factor, which fp32 / bf16 absorb), so the correction pass is rare.
 // Warp 0: TMA producer.  Warp 1: MMA issuer, owns TMEM.  Warps 2..5: softmax, P, correction, epilogue.
-// Causality and sequence boundaries come from q_start / seq_lens; KV tiles below the diagonal skip the mask.
+// Causality and sequence boundaries come from q_start / seq_lens; KV tiles below the diagonal skip the mask.  With a sliding
+// window (position i sees j with 0 <= i - j < window) only the rows some query of the chunk can see are gathered and
+// expanded, and a CTA starts at the KV tile that holds the first row its first query sees.
 // All waits are bounded (sm100.cuh); no multicast.
 #include "sm100.cuh"
 
@@ -52,8 +54,16 @@ struct MhaArgs {
     int * status;
     long long ldo;
     int n_seqs, T, H;
+    int window;               // 0: none
     float scale_log2e;
 };
+
+// Rows of a sequence with S cached tokens that its last q_len tokens can see: the last min(S, q_len + window - 1).
+__host__ __device__ __forceinline__ int visible_rows(int S, int q_len, int window) {
+    if (window <= 0 || S <= 0) return S;
+    const long long need = (long long) q_len + window - 1;
+    return need < S ? (int) need : S;
+}
 
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
@@ -120,14 +130,16 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             x -= nt;
         }
     }
-    int n_tiles = 0, ctx0 = 0, kv0 = 0, rows = 0;
+    // n_tiles KV tiles from tile kt0 on, in gathered coordinates (row 0 = the first row the chunk can see)
+    int n_tiles = 0, kt0 = 0, ctx0 = 0, kv0 = 0, rows = 0;
     if (b >= 0) {
-        const int S = a.seq_lens[b];
-        ctx0 = S - q_len;                             // tokens cached before this chunk
+        const int S = visible_rows(a.seq_lens[b], q_len, a.window);
+        ctx0 = S - q_len;                             // gathered rows before this chunk
         kv0 = a.kv_start[b];
         rows = min(QT, q_len - tile * QT);            // valid query rows of the tile
         const int last_lim = ctx0 + tile * QT + rows; // kv rows visible to the last valid query row
-        n_tiles = rows > 0 && S > 0 ? (last_lim + KT - 1) / KT : 0;
+        kt0 = a.window > 0 ? max(0, ctx0 + tile * QT + 1 - a.window) / KT : 0;
+        n_tiles = rows > 0 && S > 0 ? (last_lim + KT - 1) / KT - kt0 : 0;
     }
     const int row0 = q0 + tile * QT;                  // first query row (global)
 
@@ -138,7 +150,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             for (int c = 0; c < 3; ++c) tma_load_2d(q_s + c * CHUNK, &tmQ, q_full, h * DQK + c * 64, row0);
             for (int kt = 0; kt < n_tiles; ++kt) {
                 const int s = kt & 1;
-                const int krow = kv0 + kt * KT;
+                const int krow = kv0 + (kt0 + kt) * KT;
                 if (!mbar_wait(&k_empty[s], ((kt >> 1) & 1) ^ 1)) { jib_report(a.status, JIB_ERR_WAIT_TIMEOUT, 31, kt); break; }
                 uint8_t * kd = k_s + s * K_BYTES;
                 mbar_expect_tx(&k_full[s], K_BYTES);
@@ -213,8 +225,11 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             if (!ok) break;
             tc_fence_after();
             const uint32_t ts = tm_S + lane_addr + s * KT;
-            const bool need_mask = (kt + 1) * KT > lim_first;          // the tile reaches the diagonal (or the sequence end)
-            const int vis = lim - kt * KT;            // columns [0, vis) of this tile are visible to this row
+            const int col0 = (kt0 + kt) * KT;
+            // the tile reaches the diagonal (or the sequence end), or begins before the last row's window does
+            const bool need_mask = col0 + KT > lim_first || (a.window > 0 && col0 < lim_first + QT - 1 - a.window);
+            const int vis = lim - col0;               // columns [inv, vis) of this tile are visible to this row
+            const int inv = a.window > 0 ? vis - a.window : 0;
             // The row's 128 scores come out of tensor memory once, all loads in flight before one wait; the S buffer is
             // handed back to the tensor core right away (Q.K^T of the tile after the next may start).
             float x[KT];
@@ -227,7 +242,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             float mt = -INFINITY;
             if (need_mask) {
 #pragma unroll
-                for (int c = 0; c < KT; ++c) { x[c] = c < vis ? x[c] * a.scale_log2e : -INFINITY; mt = fmaxf(mt, x[c]); }
+                for (int c = 0; c < KT; ++c) { x[c] = (c < vis && c >= inv) ? x[c] * a.scale_log2e : -INFINITY; mt = fmaxf(mt, x[c]); }
             } else {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) { x[c] *= a.scale_log2e; mt = fmaxf(mt, x[c]); }
@@ -320,21 +335,22 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 }
 
 // ---- latent rows of the sequences of a batch, gathered from the paged cache into one contiguous buffer ---------------------
-// lat [total][row] <- cache[block_tables[b][s / bs] * bs + s % bs][row] for s < seq_lens[b]; kv_start[b] = first row of
-// sequence b (exclusive prefix of seq_lens).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
+// lat [total][row] <- cache[block_tables[b][s / bs] * bs + s % bs][row] for s < seq_lens[b] (with a window: for the rows the
+// sequence's last q_len tokens can see); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
 __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict__ cache, const int * __restrict__ block_tables, int max_blocks,
                                                         const int * __restrict__ seq_lens, int n_seqs, int block_size, int row_elems,
-                                                        long long n_slots, bf16 * __restrict__ lat, int * __restrict__ kv_start, int total_cap) {
+                                                        long long n_slots, const int * __restrict__ q_start, int window,
+                                                        bf16 * __restrict__ lat, int * __restrict__ kv_start, int total_cap) {
     PDL_TRIGGER_TOP();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = blockIdx.x * 8 + warp;              // global row of the gathered buffer this warp copies
     int b = -1, s = 0, acc = 0;
     for (int i = 0; i < n_seqs; ++i) {
-        const int S = seq_lens[i];
+        const int S = seq_lens[i], n = window > 0 ? visible_rows(S, q_start[i + 1] - q_start[i], window) : S;
         if (blockIdx.x == 0 && threadIdx.x == 0) kv_start[i] = acc;
-        if (b < 0 && g < acc + S) { b = i; s = g - acc; }
-        acc += S;
+        if (b < 0 && g < acc + n) { b = i; s = S - n + g - acc; }
+        acc += n;
     }
     if (b < 0 || g >= total_cap) return;
     const int blk = block_tables[(size_t) b * max_blocks + s / block_size];
@@ -380,14 +396,15 @@ int map_2d(CUtensorMap * out, const void * ptr, long long rows, long long cols, 
 
 extern "C" {
 
-// Gathers the latent rows of all sequences of the batch (seq_lens[b] rows each, in sequence order) from the paged cache
-// layer into lat [total_cap][row_elems] and writes the first row of every sequence to kv_start [n_seqs].
+// Gathers the latent rows of all sequences of the batch (seq_lens[b] rows each, or with window > 0 the last
+// min(seq_lens[b], q_len[b] + window - 1), in sequence order) from the paged cache layer into lat [total_cap][row_elems] and writes the first row of every sequence to kv_start [n_seqs].
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, void * lat, int * kv_start, int total_cap, void * stream) {
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, void * lat, int * kv_start,
+                             int total_cap, void * stream) {
     if (n_seqs <= 0 || total_cap <= 0) return 0;
-    if (row_elems % 8 || block_size <= 0) return JIB_E_ARG;
+    if (row_elems % 8 || block_size <= 0 || (window > 0 && q_start == nullptr)) return JIB_E_ARG;
     JIB_LAUNCH((kv_gather_kernel), (total_cap + 7) / 8, 256, 0, (cudaStream_t) stream, (const bf16 *) cache, block_tables, max_blocks, seq_lens,
-               n_seqs, block_size, row_elems, n_slots, (bf16 *) lat, kv_start, total_cap);
+               n_seqs, block_size, row_elems, n_slots, q_start, window, (bf16 *) lat, kv_start, total_cap);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 
@@ -397,7 +414,7 @@ JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * 
 // of its seq_lens[b] cached tokens) and K/V rows kv_start[b].. ; n_q_tiles >= sum_b ceil(q_len_b / 128).
 JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * kv, const void * kpe, long long kpe_stride, long long total,
                                const int * q_start, const int * seq_lens, const int * kv_start, int n_seqs, int T, int H, float scale,
-                               int n_q_tiles, void * out, long long ldo, int * status, void * stream_) {
+                               int window, int n_q_tiles, void * out, long long ldo, int * status, void * stream_) {
     cudaStream_t stream = (cudaStream_t) stream_;
     if (T <= 0 || n_seqs <= 0 || n_q_tiles <= 0) return 0;
     if (ldo % 8 || ((uintptr_t) out & 15) || total <= 0) return JIB_E_ALIGN;
@@ -410,7 +427,7 @@ JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * 
     if (rc) return rc;
     MhaArgs a;
     a.q_start = q_start; a.seq_lens = seq_lens; a.kv_start = kv_start; a.out = (bf16 *) out; a.status = status; a.ldo = ldo;
-    a.n_seqs = n_seqs; a.T = T; a.H = H;
+    a.n_seqs = n_seqs; a.T = T; a.H = H; a.window = window;
     a.scale_log2e = scale * 1.4426950408889634f;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(mha_prefill_kernel, SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;

@@ -61,6 +61,7 @@ struct FlashArgs {
     bf16 * o_lat;         // [T][H][R]
     int * status;
     int max_blocks, n_seqs, T, H, n_splits, n_blocks;
+    int window;           // > 0: position i sees j with 0 <= i - j < window
     float scale_log2e;
 };
 
@@ -125,13 +126,17 @@ mla_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             lim[n_pass - 1][j] = n_kv;
         }
         for (int p = 0; p < n_pass; ++p) {
-            int mx = 0;
+            int mx = 0, mn = 0x7fffffff;          // last visible position + 1, first visible position over the pass's tokens
 #pragma unroll
-            for (int jj = 0; jj < QT; ++jj) mx = max(mx, lim[p][jj]);
-            int chunk = (mx + a.n_splits - 1) / a.n_splits;
+            for (int jj = 0; jj < QT; ++jj) {
+                mx = max(mx, lim[p][jj]);
+                if (lim[p][jj] > 0) mn = min(mn, a.window > 0 ? max(0, lim[p][jj] - a.window) : 0);
+            }
+            mn = min(mn, mx) / BLK * BLK;         // a tile starts on a cache block
+            int chunk = (mx - mn + a.n_splits - 1) / a.n_splits;
             chunk = (chunk + KV_TILE - 1) / KV_TILE * KV_TILE;
             if (chunk < KV_TILE) chunk = KV_TILE;
-            pass_k0[p] = sp * chunk;
+            pass_k0[p] = mn + sp * chunk;
             pass_k1[p] = min(mx, pass_k0[p] + chunk);
         }
     }
@@ -308,7 +313,8 @@ mla_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
                 // tile max per column over the 128 kv lanes
 #pragma unroll
                 for (int c = 0; c < NQ; ++c) {
-                    const bool vis = pos < lim[p][c >> 4];
+                    const int up = lim[p][c >> 4];
+                    const bool vis = pos < up && (a.window <= 0 || pos >= up - a.window);
                     float v = vis ? s[c] : -INFINITY;
                     s[c] = v;
 #pragma unroll
@@ -451,8 +457,8 @@ JIB_TL_DEFINE_SETTER(flash)
 // qt: query tokens per CTA (1 for decode batches, 2 for prompt chunks).  n_splits > 1 writes partials that
 // jib_mla_combine merges.  Only block_size 64, r 512, dr 64.
 extern "C" JIB_EXPORT int jib_mla_flash(const void * q, const void * cache, long long n_slots, const int * block_tables, int max_blocks,
-                                        const int * seq_lens, const int * q_start, int n_seqs, int T, int H, float scale, int n_splits,
-                                        int qt, float * part_o, float * part_ml, void * o_lat, int * status, void * stream_) {
+                                        const int * seq_lens, const int * q_start, int n_seqs, int T, int H, float scale, int window,
+                                        int n_splits, int qt, float * part_o, float * part_ml, void * o_lat, int * status, void * stream_) {
     cudaStream_t stream = (cudaStream_t) stream_;
     if (T <= 0) return 0;
     if (n_splits < 1 || (qt != 1 && qt != 2) || n_slots % BLK) return JIB_E_ARG;
@@ -482,7 +488,7 @@ extern "C" JIB_EXPORT int jib_mla_flash(const void * q, const void * cache, long
     FlashArgs a;
     a.block_tables = block_tables; a.seq_lens = seq_lens; a.q_start = q_start; a.part_o = part_o; a.part_ml = part_ml;
     a.o_lat = (bf16 *) o_lat; a.status = status; a.max_blocks = max_blocks; a.n_seqs = n_seqs; a.T = T; a.H = H;
-    a.n_splits = n_splits; a.n_blocks = (int) (n_slots / BLK);
+    a.n_splits = n_splits; a.n_blocks = (int) (n_slots / BLK); a.window = window;
     a.scale_log2e = scale * 1.4426950408889634f;
     dim3 grid((T + qt - 1) / qt, n_splits, (H + 15) / 16);
     return qt == 1 ? launch_flash<1>(mq, mkv, a, grid, stream) : launch_flash<2>(mq, mkv, a, grid, stream);

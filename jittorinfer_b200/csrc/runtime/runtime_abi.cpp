@@ -99,6 +99,17 @@ JIB_API int jib_sched_step(jib_sched * s, StepArrays * arrays, int32_t * info_ou
     info_out[4] = i.max_q_len; info_out[5] = i.n_preempted; info_out[6] = i.n_copies;
     return i.n_tokens;
 }
+JIB_API int jib_sched_fed_open(jib_sched * s) { return s->sched.fed_open(); }
+JIB_API int jib_sched_fed_close(jib_sched * s, int slot) { return s->sched.fed_close(slot) ? 1 : 0; }
+// One batch of caller-supplied tokens; info_out as in jib_sched_step.  Returns the token count, 0 if an entry does not fit.
+JIB_API int jib_sched_step_fed(jib_sched * s, StepArrays * arrays, const int32_t * slots, const int32_t * lens, int n, const int32_t * tokens,
+                               int32_t * info_out) {
+    StepInfo i = s->sched.step_fed(*arrays, slots, lens, n, tokens);
+    info_out[0] = i.n_tokens; info_out[1] = i.n_seqs; info_out[2] = i.n_out; info_out[3] = i.n_decode_seqs;
+    info_out[4] = i.max_q_len; info_out[5] = i.n_preempted; info_out[6] = i.n_copies;
+    return i.n_tokens;
+}
+JIB_API void jib_sched_set_recurrent(jib_sched * s, int on) { s->sched.set_recurrent(on != 0); }
 JIB_API void jib_sched_commit(jib_sched * s, const int32_t * sampled, int n_out) { s->sched.commit(sampled, n_out, &s->events); }
 JIB_API int jib_sched_can_run_ahead(jib_sched * s) { return s->sched.can_run_ahead() ? 1 : 0; }
 JIB_API void jib_sched_commit_deferred(jib_sched * s, int n_out) { s->sched.commit_deferred(n_out); }

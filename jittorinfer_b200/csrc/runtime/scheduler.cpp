@@ -14,7 +14,7 @@ Scheduler::Scheduler(PagedKv * kv, int n_slots, int n_batch, int n_ctx_slot, int
 bool Scheduler::idle() const {
     if (!waiting_.empty()) return false;
     for (const auto & s : slots_)
-        if (s.state != SLOT_IDLE) return false;
+        if (s.state != SLOT_IDLE && s.state != SLOT_FED) return false;
     return true;
 }
 
@@ -80,6 +80,7 @@ void Scheduler::launch(Slot & s, const Request & r, int lcp) {
     // at least one prompt token must be evaluated to obtain logits
     int n_past = std::min(lcp, s.n_prompt - 1);
     if (n_past < 0) n_past = 0;
+    if (recurrent_ && n_past != kv_->seq_len(s.id)) n_past = 0;      // the state belongs to the end of what the slot holds
     kv_->seq_rm(s.id, n_past, -1);
     if (n_past > 0) ++stats_.prefix_hits;
     s.tokens.swap(prompt);
@@ -137,7 +138,7 @@ bool Scheduler::ensure_blocks(int slot, int n_tokens, int protect_slot) {
         }
         int64_t newest = -1;
         for (auto & s : slots_)
-            if (s.state != SLOT_IDLE && s.id != slot && s.id != protect_slot && !s.in_batch && s.t_started > newest) {
+            if (s.state != SLOT_IDLE && s.state != SLOT_FED && s.id != slot && s.id != protect_slot && !s.in_batch && s.t_started > newest) {
                 newest = s.t_started;
                 victim = s.id;
             }
@@ -155,12 +156,111 @@ bool Scheduler::cancel(int64_t req_id, std::vector<StepEvent> * events) {
             return true;
         }
     for (auto & s : slots_)
-        if (s.state != SLOT_IDLE && s.req_id == req_id) {
+        if (s.state != SLOT_IDLE && s.state != SLOT_FED && s.req_id == req_id) {
             if (events) events->push_back({req_id, s.id, -1, FINISH_CANCELLED, s.n_prompt_orig, s.n_decoded});
             release(s, true);
             return true;
         }
     return false;
+}
+
+// Tokens s.tokens[n_past .. n_past + n_new) enter the cache and the batch now.
+void Scheduler::emit(StepArrays & out, StepInfo & info, Slot & s, int n_new, bool want_logits) {
+    const int n_tok = info.n_tokens, n_seq = info.n_seqs;
+    out.q_start[n_seq] = n_tok;
+    for (int i = 0; i < n_new; ++i) {
+        out.tokens[n_tok + i] = s.tokens[s.n_past + i];
+        out.positions[n_tok + i] = s.n_past + i;
+    }
+    kv_->append(s.id, n_new, out.slot_mapping + n_tok);
+    info.n_tokens += n_new;
+    s.n_past += n_new;
+    out.seq_lens[n_seq] = s.n_past;
+    out.seq_slots[n_seq] = s.id;
+    const auto & bl = kv_->seq_blocks(s.id);
+    int32_t * row = out.block_tables + (size_t) n_seq * out.max_blocks_per_seq;
+    int nb = std::min<int>((int) bl.size(), out.max_blocks_per_seq);
+    std::memcpy(row, bl.data(), nb * sizeof(int32_t));
+    for (int i = nb; i < out.max_blocks_per_seq; ++i) row[i] = 0;
+    if (want_logits) {
+        out.out_rows[info.n_out] = info.n_tokens - 1;
+        out.out_slots[info.n_out] = s.id;
+        s.out_row = info.n_out;
+        last_out_slots_.push_back(s.id);
+        ++info.n_out;
+    }
+    info.max_q_len = std::max(info.max_q_len, n_new);
+    ++info.n_seqs;
+    s.in_batch = true;
+    s.t_last_used = ++clock_;
+}
+
+int Scheduler::fed_open() {
+    int sid = -1;
+    int64_t t = INT64_MAX;
+    for (const auto & s : slots_)
+        if (s.state == SLOT_IDLE && s.t_last_used < t) { t = s.t_last_used; sid = s.id; }
+    if (sid < 0) return -1;
+    Slot & s = slots_[sid];
+    kv_->seq_rm(sid, 0, -1);
+    s.tokens.clear();
+    s.n_past = s.n_cached = s.n_prompt = s.n_prompt_orig = s.n_decoded = 0;
+    s.req_id = -1;
+    s.pending_token = -1;
+    s.out_row = -1;
+    s.state = SLOT_FED;
+    s.t_started = s.t_last_used = ++clock_;
+    return sid;
+}
+
+bool Scheduler::fed_close(int slot) {
+    if (slot < 0 || slot >= (int) slots_.size() || slots_[slot].state != SLOT_FED) return false;
+    release(slots_[slot], false);
+    return true;
+}
+
+StepInfo Scheduler::step_fed(StepArrays & out, const int32_t * slots, const int32_t * lens, int n, const int32_t * tokens) {
+    StepInfo info;
+    int total = 0, blocks = 0;
+    for (int i = 0; i < n; ++i) {
+        if (slots[i] < 0 || slots[i] >= (int) slots_.size() || lens[i] <= 0) return info;
+        const Slot & s = slots_[slots[i]];
+        if (s.state != SLOT_FED || s.n_past + lens[i] > n_ctx_slot_) return info;
+        for (int j = 0; j < i; ++j)
+            if (slots[j] == slots[i]) return info;
+        total += lens[i];
+        blocks += kv_->blocks_needed(slots[i], lens[i]);
+    }
+    if (n > out.cap_seqs || total > out.cap_tokens) return info;
+    // room for everybody: cached blocks of idle slots go first (least recently used), then running generations
+    while (blocks > kv_->free_blocks()) {
+        int victim = -1;
+        int64_t t = INT64_MAX;
+        for (const auto & s : slots_)
+            if (s.state == SLOT_IDLE && kv_->seq_len(s.id) > 0 && s.t_last_used < t) { t = s.t_last_used; victim = s.id; }
+        if (victim >= 0) {
+            kv_->seq_rm(victim, 0, -1);
+            slots_[victim].tokens.clear();
+            continue;
+        }
+        int64_t newest = -1;
+        for (const auto & s : slots_)
+            if (s.state != SLOT_IDLE && s.state != SLOT_FED && s.t_started > newest) { newest = s.t_started; victim = s.id; }
+        if (victim < 0) return info;
+        preempt(slots_[victim]);
+    }
+    for (auto & s : slots_) { s.out_row = -1; s.in_batch = false; }
+    last_out_slots_.clear();
+    for (int i = 0; i < n; ++i) {
+        Slot & s = slots_[slots[i]];
+        s.tokens.insert(s.tokens.end(), tokens, tokens + lens[i]);
+        tokens += lens[i];
+        emit(out, info, s, lens[i], false);
+    }
+    out.q_start[info.n_seqs] = info.n_tokens;
+    info.n_copies = (int) kv_->pending_copies().size();
+    if (info.n_tokens > 0) ++stats_.steps;
+    return info;
 }
 
 StepInfo Scheduler::step(StepArrays & out) {
@@ -172,10 +272,10 @@ StepInfo Scheduler::step(StepArrays & out) {
         if (sid < 0) break;
         Request r = std::move(waiting_.front());
         waiting_.pop_front();
-        if (r.prompt.empty()) r.prompt.push_back(eos_id_);
+        if (r.prompt.empty()) r.prompt.push_back(std::max(eos_id_, 0));
         // A longer prefix may sit in another slot's sequence (idle or running): share its full blocks by reference.
         // Whole blocks only, so that neither sequence ever has to copy one on its next write.
-        {
+        if (!recurrent_) {
             const int bs = kv_->block_size();
             int donor = -1, best = lcp;
             for (const auto & o : slots_) {
@@ -196,38 +296,9 @@ StepInfo Scheduler::step(StepArrays & out) {
     for (auto & s : slots_) { s.out_row = -1; s.in_batch = false; }
     last_out_slots_.clear();
 
-    int n_tok = 0, n_seq = 0, n_outp = 0;
     const int budget = std::min(n_batch_, out.cap_tokens);
-    auto emit_seq = [&](Slot & s, int n_new, bool want_logits) {
-        // tokens s.tokens[n_past .. n_past+n_new) enter the cache now
-        out.q_start[n_seq] = n_tok;
-        for (int i = 0; i < n_new; ++i) {
-            out.tokens[n_tok + i] = s.tokens[s.n_past + i];
-            out.positions[n_tok + i] = s.n_past + i;
-        }
-        kv_->append(s.id, n_new, out.slot_mapping + n_tok);
-        n_tok += n_new;
-        s.n_past += n_new;
-        out.seq_lens[n_seq] = s.n_past;
-        out.seq_slots[n_seq] = s.id;
-        const auto & bl = kv_->seq_blocks(s.id);
-        int32_t * row = out.block_tables + (size_t) n_seq * out.max_blocks_per_seq;
-        int nb = std::min<int>((int) bl.size(), out.max_blocks_per_seq);
-        std::memcpy(row, bl.data(), nb * sizeof(int32_t));
-        for (int i = nb; i < out.max_blocks_per_seq; ++i) row[i] = 0;
-        if (want_logits) {
-            out.out_rows[n_outp] = n_tok - 1;
-            out.out_slots[n_outp] = s.id;
-            s.out_row = n_outp;
-            last_out_slots_.push_back(s.id);
-            ++n_outp;
-        }
-        info.max_q_len = std::max(info.max_q_len, n_new);
-        ++n_seq;
-        s.in_batch = true;
-        s.t_last_used = ++clock_;
-    };
-
+    int & n_tok = info.n_tokens;
+    int & n_seq = info.n_seqs;
     // 2. one token per generating slot (oldest first so that preemption hits the youngest)
     std::vector<int> order;
     for (auto & s : slots_)
@@ -245,7 +316,7 @@ StepInfo Scheduler::step(StepArrays & out) {
         }
         if ((int) s.tokens.size() == s.n_past) s.tokens.push_back(s.pending_token);
         s.pending_token = -1;
-        emit_seq(s, 1, true);
+        emit(out, info, s, 1, true);
         ++info.n_decode_seqs;
     }
     // 3. prompt chunks until the token budget is used (a smaller budget while sequences are generating, if configured)
@@ -271,15 +342,12 @@ StepInfo Scheduler::step(StepArrays & out) {
             }
             s.state = SLOT_PROCESSING_PROMPT;
             bool last = chunk == remaining;
-            emit_seq(s, chunk, last);
+            emit(out, info, s, chunk, last);
             stats_.prompt_tokens += chunk;
             if (last) s.state = SLOT_DONE_PROMPT;
         }
     }
     out.q_start[n_seq] = n_tok;
-    info.n_tokens = n_tok;
-    info.n_seqs = n_seq;
-    info.n_out = n_outp;
     info.n_copies = (int) kv_->pending_copies().size();
     info.n_preempted += 0;
     if (n_tok > 0) ++stats_.steps;
@@ -312,7 +380,7 @@ bool Scheduler::can_run_ahead() const {
     if (!waiting_.empty() || !deferred_.empty()) return false;
     int active = 0, new_blocks = 0;
     for (const auto & s : slots_) {
-        if (s.state == SLOT_IDLE) continue;
+        if (s.state == SLOT_IDLE || s.state == SLOT_FED) continue;
         if (s.out_row < 0) return false;                   // still inside its prompt: the next step is not a pure decode step
         ++active;
         new_blocks += kv_->blocks_needed(s.id, 1);         // incl. a copy-on-write block

@@ -18,7 +18,8 @@
 
 namespace jib {
 
-enum SlotState : int32_t { SLOT_IDLE = 0, SLOT_STARTED, SLOT_PROCESSING_PROMPT, SLOT_DONE_PROMPT, SLOT_GENERATING };
+// SLOT_FED: the slot belongs to a caller that supplies every token itself (fed_open / step_fed / fed_close).
+enum SlotState : int32_t { SLOT_IDLE = 0, SLOT_STARTED, SLOT_PROCESSING_PROMPT, SLOT_DONE_PROMPT, SLOT_GENERATING, SLOT_FED };
 
 enum FinishReason : int32_t { FINISH_NONE = 0, FINISH_STOP = 1, FINISH_LENGTH = 2, FINISH_CANCELLED = 3, FINISH_ERROR = 4 };
 
@@ -115,6 +116,19 @@ class Scheduler {
     void resolve(const int32_t * sampled, int n_out, std::vector<StepEvent> * events);
     int n_deferred() const { return (int) deferred_.size(); }
 
+    // ---- sequences whose tokens come from outside (replay, teacher forcing) --------------------------------------------
+    // fed_open() takes an idle slot (least recently used; what it still caches is dropped) and returns its id, -1 if none is
+    // idle.  step_fed() assembles one batch: entry i appends lens[i] tokens (read from `tokens`, entry after entry) to slot
+    // slots[i]; no output rows are named.  n_tokens == 0: an entry does not fit (its slot is not fed, the slot limit, the
+    // batch arrays or the blocks that can be freed) and no token has been taken.  fed_close() returns the slot and its blocks.
+    int fed_open();
+    StepInfo step_fed(StepArrays & out, const int32_t * slots, const int32_t * lens, int n, const int32_t * tokens);
+    bool fed_close(int slot);
+
+    // Models that carry a recurrent state beside the cache: the state of a sequence exists only at its end, so a cached prefix
+    // can be continued but not cut, and blocks cannot be shared with another slot.
+    void set_recurrent(bool on) { recurrent_ = on; }
+
     bool idle() const;
     int n_waiting() const { return (int) waiting_.size(); }
     int n_running() const;
@@ -134,6 +148,7 @@ class Scheduler {
     bool ensure_blocks(int slot, int n_tokens, int protect_slot);
     void release(Slot & s, bool keep_cache);
     void preempt(Slot & s);
+    void emit(StepArrays & out, StepInfo & info, Slot & s, int n_new, bool want_logits);
 
     PagedKv * kv_;
     std::vector<Slot> slots_;
@@ -141,6 +156,7 @@ class Scheduler {
     int n_batch_, n_ctx_slot_, eos_id_, n_keep_;
     int mixed_prompt_budget_ = 0;
     bool cont_batching_;
+    bool recurrent_ = false;
     int64_t clock_ = 0;
     std::vector<int32_t> last_out_slots_;
     SchedStats stats_;

@@ -16,7 +16,9 @@ import time
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="jittorinfer_b200.generate")
     ap.add_argument("--config", "-c", default=None)
-    ap.add_argument("--random-init", default=None, help="tiny | tiny-v2 | lite | v2: random weights instead of a GGUF file")
+    ap.add_argument("--model", "-m", default=None, help="GGUF file, or a folder with config.json and safetensors files")
+    ap.add_argument("--random-init", default=None,
+                    help="tiny | tiny-v2 | lite | v2 | nibalix-tiny | nibalix-lite: random weights instead of a model file")
     ap.add_argument("--prompt", "-p", action="append", default=[], help="text prompt (repeatable)")
     ap.add_argument("--tokens", action="append", default=[], help="prompt as comma-separated token ids (repeatable)")
     ap.add_argument("--chat", action="store_true", help="wrap each text prompt in the chat template as a user turn")
@@ -35,6 +37,8 @@ def main(argv=None) -> int:
     from .server.chat import ChatTemplate
     from .server.launch import build_from_config
     cfg = load_yaml(a.config)
+    if a.model:
+        cfg.model = a.model
     if a.random_init:
         cfg.random_init = a.random_init
     if not cfg.model and not cfg.random_init:

@@ -40,7 +40,8 @@ class ForwardBatch:
     ``tokens/positions/slot_mapping`` have one entry per query token; tokens of one sequence are
     contiguous.  Sequence ``b`` owns rows ``q_start[b]:q_start[b+1]`` and, after this step, has
     ``seq_lens[b]`` cached tokens.  ``slot_mapping[i] < 0`` marks a padding row.
-    ``out_rows`` selects the rows whose logits are wanted.
+    ``out_rows`` selects the rows whose logits are wanted.  ``seq_slots[b]`` is the engine's slot of sequence ``b`` (the row of
+    whatever state the model keeps per sequence; negative for a padding sequence).
     """
     tokens: torch.Tensor
     positions: torch.Tensor
@@ -51,12 +52,13 @@ class ForwardBatch:
     out_rows: torch.Tensor
     max_q_len: int = 1
     attn_meta: Optional[object] = None
+    seq_slots: Optional[torch.Tensor] = None
 
 
 def _batch_to(b: ForwardBatch, dev: torch.device) -> ForwardBatch:
     mv = lambda t: None if t is None else t.to(dev, non_blocking=True)
     return ForwardBatch(mv(b.tokens), mv(b.positions), mv(b.slot_mapping), mv(b.block_tables), mv(b.seq_lens), mv(b.q_start),
-                        mv(b.out_rows), b.max_q_len, None)
+                        mv(b.out_rows), b.max_q_len, None, mv(b.seq_slots))
 
 
 def assign_layers(n_layer: int, devices, tensor_split=None):
@@ -89,6 +91,8 @@ class _Layer:
 
 
 class DeepSeek2Model:
+    recurrent = False                 # the cached rows are all that a sequence leaves behind
+
     def __init__(self, hp: DeepSeek2HParams, weights: Iterable[Tuple[str, torch.Tensor]],
                  dtype: torch.dtype = torch.bfloat16, device="cpu", spec: ShardSpec = ShardSpec(),
                  comm=None, max_positions: int = 8192, block_size: int = 64, ep=None, layer_devices=None):
@@ -258,6 +262,16 @@ class DeepSeek2Model:
             missing = [n for n in need if getattr(L, n) is None]
             if missing:
                 raise ValueError(f"layer {il}: missing tensors {missing}")
+
+    def cache_bytes_per_token(self) -> int:
+        return self.hp.n_layer * self.hp.kv_row * torch.empty(0, dtype=self.dtype).element_size()
+
+    def make_cache(self, n_slots: int, n_seqs: int):
+        """Latent rows of ``n_slots`` tokens in every layer; nothing is kept per sequence."""
+        if self.split:
+            from ..runtime.cache import SplitCache
+            return SplitCache(self.layer_dev, n_slots, self.hp.kv_row, self.dtype, self.block_size)
+        return torch.zeros(self.hp.n_layer, n_slots, self.hp.kv_row, dtype=self.dtype, device=self.device)
 
     def weight_bytes(self) -> int:
         n = 0

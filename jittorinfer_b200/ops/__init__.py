@@ -68,9 +68,9 @@ def gateup_silu(x, wg, wu):
     return ref.gateup_silu(x, wg, wu)
 
 
-def mla_qkv_post(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r):
+def mla_qkv_post(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r, rot_half=False):
     f = nat().mla_qkv_post if use_native(q) else ref.mla_qkv_post
-    return f(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r)
+    return f(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r, rot_half)
 
 
 def q_absorb(q_nope, w_uk, q_out, r):
@@ -81,22 +81,29 @@ def v_up(o_lat, w_uv):
     return (nat().v_up if use_native(o_lat) else ref.v_up)(o_lat, w_uv)
 
 
-def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len=None, meta=None):
+def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len=None, meta=None, window=0):
     if use_native(q):
-        return nat().mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len, meta)
-    return ref.mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size)
+        return nat().mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len, meta, window)
+    return ref.mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, window)
 
 
-def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None, pre_norm=None):
+def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None, pre_norm=None,
+             logit_bias=None):
     """``route=(expert_base, E_local)`` tells the CUDA path which local expert sort follows (see ``native.moe_gate``).
     ``pre_norm=(weight, eps)``: ``g`` is the un-normalised block input; returns (ids, wts, rmsnorm(g) * weight) -- on the CUDA
     path the router launch of a decode batch normalises the rows itself."""
     if use_native(g):
-        return nat().moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, route, pre_norm)
+        return nat().moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, route, pre_norm,
+                              logit_bias)
     if pre_norm is not None:
         g, _ = ref.rmsnorm(g, pre_norm[0], pre_norm[1])
         return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2) + (g,)
-    return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2)
+    return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, logit_bias)
+
+
+def moe_routed(x, ids, wts, wg, wu, wd):
+    """(expert outputs of the (token, choice) pairs, row of each pair); the weighted sum is the caller's (``block_update``)."""
+    return (nat() if use_native(x) else ref).moe_routed(x, ids, wts, wg, wu, wd)
 
 
 def moe_experts(x, ids, wts, wg, wu, wd, expert_base=0):
@@ -118,6 +125,31 @@ def fused_combine_norm() -> bool:
     """Whether the model should ask ``moe_ffn`` for the next block's norm as well (one launch on the CUDA path;
     JIB_FUSED_COMBINE_NORM=0 keeps the two launches for A/B measurements)."""
     return os.environ.get("JIB_FUSED_COMBINE_NORM", "1") == "1"
+
+
+# ---- parallel blocks over an fp32 residual stream, per-sequence state -------------------------------------------------------------
+# ``nxt`` = (norm weight, eps, conv): the norm the next block reads, computed in the same pass; conv = None, or -- one token per
+# sequence only -- (weights [taps, d], state, seq_slots, positions) of that block's input convolution.
+def embed_norm(table, ids, w, eps, nxt=None):
+    """(x fp32 = norm of the embedding rows, h, h + convolution)."""
+    return (nat() if use_native(table) else ref).embed_norm(table, ids, w, eps, nxt)
+
+
+def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
+    """(x + mult * (sigmoid(g1 + b1) * o + sigmoid(g2 + b2) * combine(moe)), h, h + convolution); x may be overwritten."""
+    return (nat() if use_native(x) else ref).block_update(x, mult, o, gates, b1, b2, moe, nxt)
+
+
+def rms_rows(x, rows, w, eps, dtype):
+    return (nat() if use_native(x) else ref).rms_rows(x, rows, w, eps, dtype)
+
+
+def causal_conv(h, w, state, seq_slots, positions, q_start):
+    return (nat() if use_native(h) else ref).causal_conv(h, w, state, seq_slots, positions, q_start)
+
+
+def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
+    return (nat() if use_native(zxg) else ref).mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single)
 
 
 def argmax(logits):

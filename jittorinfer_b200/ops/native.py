@@ -61,6 +61,11 @@ class GemmDesc(C.Structure):
                                                                              ("n_slots", C.c_int), ("list_tiles", C.c_int), ("pdl_flags", C.c_int)]
 
 
+class RowTail(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x_out", "norm_w", "h_out", "conv_w", "hc_out", "conv_state", "seq_slots", "positions", "status")] + \
+               [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int)]
+
+
 def load():
     global _lib
     if _lib is not None:
@@ -78,26 +83,32 @@ def load():
         fn.argtypes = list(args)
 
     sig("jib_gemm_bf16", C.POINTER(GemmDesc), vp)
+    sig("jib_gemm_simt", C.POINTER(GemmDesc), i, vp)
+    sig("jib_embed_norm", vp, ip, fp, f, i, i, i, i, C.POINTER(RowTail), vp)
+    sig("jib_block_update", fp, f, vp, vp, ll, fp, fp, vp, ip, fp, i, i, i, i, C.POINTER(RowTail), vp)
+    sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, vp, vp)
+    sig("jib_causal_conv", vp, fp, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
+    sig("jib_mingru", vp, ll, fp, fp, fp, i, ip, ip, ip, i, i, i, i, i, vp, ip, vp)
     sig("jib_embed_gather", vp, ip, vp, i, i, i, vp)
     sig("jib_rmsnorm", vp, vp, fp, vp, vp, i, i, ll, f, vp)
-    sig("jib_mla_qkv_post", vp, ll, vp, ll, fp, f, fp, ip, ip, vp, vp, ll, ll, i, i, i, i, i, i, ll, ip, vp)
-    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, vp, ip, i, vp)
-    sig("jib_mha_prefill", vp, ll, vp, vp, ll, ll, ip, ip, ip, i, i, i, f, i, vp, ll, ip, vp)
+    sig("jib_mla_qkv_post", vp, ll, vp, ll, fp, f, fp, ip, ip, vp, vp, ll, ll, i, i, i, i, i, i, ll, i, i, ip, vp)
+    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, ip, i, vp, ip, i, vp)
+    sig("jib_mha_prefill", vp, ll, vp, vp, ll, ll, ip, ip, ip, i, i, i, f, i, i, vp, ll, ip, vp)
     sig("jib_argmax", fp, ip, i, i, vp)
     sig("jib_topk", fp, fp, ip, i, i, i, vp)
     sig("jib_sample_topk", fp, ip, fp, ip, i, i, vp)
     sig("jib_kv_block_copy", vp, ll, i, ip, ip, i, i, vp)
     sig("jib_gather_rows", vp, ip, vp, i, i, i, vp)
-    sig("jib_moe_gate", vp, fp, fp, fp, ip, fp, i, i, i, i, i, i, f, i, i, i, i, vp)
+    sig("jib_moe_gate", vp, fp, fp, fp, fp, ip, fp, i, i, i, i, i, i, f, i, i, i, i, vp)
     sig("jib_moe_permute", ip, i, i, i, i, ip, ip, ip, vp)
     sig("jib_moe_route_fused", vp, fp, fp, fp, ip, fp, ip, ip, ip, ip, i, i, i, i, i, i, f, i, i, i, i, i, i, fp, f, vp, vp)
     sig("jib_moe_permute_multi", ip, i, i, i, i, ip, ip, ip, ip, vp)
     sig("jib_moe_tile_list", ip, i, i, ip, i, vp)
     sig("jib_moe_combine", vp, ip, fp, vp, vp, vp, i, i, i, vp)
     sig("jib_moe_combine_norm", vp, ip, fp, vp, vp, fp, vp, vp, i, i, i, f, vp)
-    sig("jib_mla_attention", vp, vp, ip, i, ip, ip, i, i, i, i, i, i, f, i, fp, fp, vp, vp)
+    sig("jib_mla_attention", vp, vp, ip, i, ip, ip, i, i, i, i, i, i, f, i, i, i, fp, fp, vp, vp)
     sig("jib_mla_combine", fp, fp, i, i, i, i, vp, vp)
-    sig("jib_mla_flash", vp, vp, ll, ip, i, ip, ip, i, i, i, f, i, i, fp, fp, vp, ip, vp)
+    sig("jib_mla_flash", vp, vp, ll, ip, i, ip, ip, i, i, i, f, i, i, i, fp, fp, vp, ip, vp)
     _lib = L
     return L
 
@@ -178,14 +189,24 @@ def _p(t: Optional[torch.Tensor]) -> Optional[int]:
 
 
 # ---- GEMM family ---------------------------------------------------------------------------------
+def _tma_ok(*vals: int) -> bool:
+    """Whether pointers (bytes) and element strides given in bytes can be addressed by TMA."""
+    return all(v % 16 == 0 for v in vals)
+
+
+def _gemm_simt(d: GemmDesc, f32: bool, what: str) -> None:
+    d.expert_list, d.n_slots, d.list_tiles = None, 0, 0
+    _ck(load().jib_gemm_simt(C.byref(d), int(f32), _stream()), what)
+
+
 def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *, out: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, splits: int = 0, bn: int = 0,
          ar=None, ar_site: int = 0, ar_rs_rows: int = 0, ag=None) -> torch.Tensor:
     """out[T,N] = x[T,K] @ w[N,K]^T  (w2: silu(x w^T) * (x w2^T)) (+ residual)."""
-    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.stride(-1) == 1 and w.is_contiguous()
+    assert x.dtype == w.dtype and x.dtype in (torch.bfloat16, torch.float32) and x.stride(-1) == 1 and w.is_contiguous()
     T, K = x.shape
     N = w.shape[0]
-    od = out_dtype or torch.bfloat16
+    od = out_dtype or x.dtype
     if out is None:
         out = torch.empty(T, N, dtype=od, device=x.device)
     ws = workspace(x.device)
@@ -204,13 +225,17 @@ def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *,
         d.ar, d.ar_site, d.ar_rs_rows = C.addressof(ar), ar_site, ar_rs_rows
     if ag is not None:          # x is a gather buffer other ranks are still filling: (flags ptr, epoch ptr, rows per rank, world)
         d.ag_flags, d.ag_epoch, d.ag_rows, d.ag_world = ag
+    f32 = x.dtype == torch.float32
+    if f32 or not _tma_ok(d.x, d.w, d.w2 or 0, x.stride(0) * 2, K * 2):
+        _gemm_simt(d, f32, "gemm")
+        return out
     _ck(load().jib_gemm_bf16(C.byref(d), _stream()), "gemm")
     return out
 
 
 def gemm_batched(x_ptr: int, x_row_stride: int, x_batch_stride: int, w: torch.Tensor, out_ptr: int, ldo: int,
                  out_batch_stride: int, T: int, device, splits: int = 0) -> None:
-    """Per-batch (per-head) GEMM with arbitrary element strides: out[b][t][:N] = x[b][t][:K] @ w[b]^T."""
+    """Per-batch (per-head) GEMM with arbitrary element strides: out[b][t][:N] = x[b][t][:K] @ w[b]^T, all in w's dtype."""
     B, N, K = w.shape
     ws = workspace(device)
     d = GemmDesc()
@@ -220,7 +245,11 @@ def gemm_batched(x_ptr: int, x_row_stride: int, x_batch_stride: int, w: torch.Te
     d.ldo, d.out_batch_stride, d.ldr, d.res_batch_stride = ldo, out_batch_stride, 0, 0
     d.x_rows_total, d.scratch_bytes, d.n_counters = T, ws.SCRATCH_BYTES, ws.N_COUNTERS
     d.T, d.N, d.K, d.batch, d.max_rows, d.active_hint = T, N, K, B, 0, 0
-    d.out_f32, d.res_f32, d.splits, d.bn, d.sm_count = 0, 0, splits, 0, ws.sm_count
+    f32 = w.dtype == torch.float32
+    d.out_f32, d.res_f32, d.splits, d.bn, d.sm_count = int(f32), 0, splits, 0, ws.sm_count
+    if f32 or not _tma_ok(x_ptr, d.w, x_row_stride * 2, x_batch_stride * 2 if B > 1 else 0, K * 2):
+        _gemm_simt(d, f32, "gemm_batched")
+        return
     _ck(load().jib_gemm_bf16(C.byref(d), _stream()), "gemm_batched")
 
 
@@ -241,7 +270,7 @@ def gemm_grouped_raw(x_ptr: int, x_rows_total: int, K: int, seg: torch.Tensor, w
     E, N, K2 = w.shape
     assert K2 == K
     device = device or w.device
-    out = None if out_row_ptr else torch.empty(x_rows_total, N, dtype=torch.bfloat16, device=device)
+    out = None if out_row_ptr else torch.empty(x_rows_total, N, dtype=w.dtype, device=device)
     ws = workspace(device)
     d = GemmDesc()
     d.x, d.w, d.w2, d.residual = x_ptr, w.data_ptr(), _p(w2), None
@@ -256,6 +285,11 @@ def gemm_grouped_raw(x_ptr: int, x_rows_total: int, K: int, seg: torch.Tensor, w
     if src_token is not None:
         d.src_token, d.src_rows = src_token.data_ptr(), src_rows
     d.pdl_flags = pdl_flags
+    f32 = w.dtype == torch.float32
+    if f32 or not _tma_ok(x_ptr, d.w, d.w2 or 0, K * 2, N * K * 2):
+        d.out_f32 = int(f32)
+        _gemm_simt(d, f32, "gemm_grouped")
+        return out
     if tile_list is not None:    # (expert, token tile) pairs built for this bn (moe_tile_list): large batches
         assert bn > 0
         d.expert_list, d.n_slots, d.list_tiles = tile_list.data_ptr(), tile_list.numel(), 1
@@ -277,6 +311,11 @@ def gemm_grouped(xp: torch.Tensor, seg: torch.Tensor, w: torch.Tensor, w2: Optio
 
 def linear(x, w, residual=None, out_dtype=None):
     return gemm(x, w, residual=residual, out_dtype=out_dtype)
+
+
+def grouped_tma_ok(x: torch.Tensor, wg: torch.Tensor) -> bool:
+    """Whether the grouped expert products of these shapes run on the tensor cores."""
+    return x.dtype == torch.bfloat16 and wg.shape[1] % 8 == 0 and wg.shape[2] % 8 == 0
 
 
 def gateup_silu(x, wg, wu):
@@ -301,18 +340,21 @@ def rmsnorm(x, w, eps, residual=None):
     return out, (summed if residual is not None else x)
 
 
-def mla_qkv_post(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r):
-    """``q_out`` None: the rotated RoPE part of q is written back into q (the per-head prefill form reads q as it is)."""
+def mla_qkv_post(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r, rot_half=False):
+    """``q_out`` None: the rotated RoPE part of q is written back into q (the per-head prefill form reads q as it is).
+    ``ckv`` None: queries only.  ``rot_half``: pairs (i, i + dr/2)."""
     T = q.shape[0]
     ws = workspace(q.device)
+    assert q.dtype == cache.dtype and q.dtype in (torch.bfloat16, torch.float32) and q.stride(-1) == 1 and cache.is_contiguous()
+    el = q.element_size()
     if q_out is None:
-        qo_ptr, qo_row, qo_head = q.data_ptr() + dn * 2, q.stride(0), dn + dr
+        qo_ptr, qo_row, qo_head = q.data_ptr() + dn * el, q.stride(0), dn + dr
     else:
-        qo_ptr, qo_row, qo_head = q_out.data_ptr() + r * 2, n_head * (r + dr), r + dr
-    _ck(load().jib_mla_qkv_post(q.data_ptr(), q.stride(0), ckv.data_ptr(), ckv.stride(0), kv_norm_w.data_ptr(), float(eps),
+        qo_ptr, qo_row, qo_head = q_out.data_ptr() + r * el, n_head * (r + dr), r + dr
+    _ck(load().jib_mla_qkv_post(q.data_ptr(), q.stride(0), _p(ckv), ckv.stride(0) if ckv is not None else 0, _p(kv_norm_w), float(eps),
                                 rope_table.data_ptr(), positions.data_ptr(), slot_mapping.data_ptr(), cache.data_ptr(),
-                                qo_ptr, qo_row, qo_head, T, n_head, dn, dr, r, rope_table.shape[0], cache.shape[0],
-                                ws.status.data_ptr(), _stream()), "mla_qkv_post")
+                                qo_ptr, qo_row, qo_head, T, n_head, dn, dr, r, rope_table.shape[0], cache.shape[0], int(rot_half),
+                                int(q.dtype == torch.float32), ws.status.data_ptr(), _stream()), "mla_qkv_post")
     return q.view(T, n_head, dn + dr)[..., :dn] if q.is_contiguous() else q.as_strided((T, n_head, dn), (q.stride(0), dn + dr, 1))
 
 
@@ -341,27 +383,33 @@ def attn_splits(T: int, H: int, sm_count: int = 148) -> int:
 ATTN_IMPL = os.environ.get("JITTORINFER_ATTN", "flash")      # "flash" (tcgen05) | "simt" (CUDA-core kernel)
 
 
-def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len=None, meta=None):
+def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_size, max_q_len=None, meta=None, window=0):
+    """``window`` > 0: position i sees j with 0 <= i - j < window."""
     T, H, D = q.shape
     n_seqs = seq_lens.shape[0]
     prefill = (max_q_len or 1) > 1
+    assert q.dtype == cache.dtype and q.is_contiguous() and cache.is_contiguous()
     o = torch.empty(T, H, r, dtype=q.dtype, device=q.device)
-    if ATTN_IMPL == "flash" and r == 512 and D == 576 and block_size == 64 and cache.shape[0] % 64 == 0:
+    if ATTN_IMPL == "flash" and q.dtype == torch.bfloat16 and r == 512 and D == 576 and block_size == 64 and cache.shape[0] % 64 == 0:
         qt = 2 if prefill else 1
         n_splits = 1 if prefill else attn_splits(T, H)
+        if window > 0:
+            n_splits = min(n_splits, (window + 63 + 127) // 128)      # a window covers this many 128-row tiles at most
         part_o = part_ml = None
         if n_splits > 1:
             part_o = torch.empty(T, n_splits, H, r, dtype=torch.float32, device=q.device)
             part_ml = torch.empty(T, n_splits, H, 2, dtype=torch.float32, device=q.device)
         ws = workspace(q.device)
         _ck(load().jib_mla_flash(q.data_ptr(), cache.data_ptr(), cache.shape[0], block_tables.data_ptr(), block_tables.stride(0),
-                                 seq_lens.data_ptr(), q_start.data_ptr(), n_seqs, T, H, float(scale), n_splits, qt, _p(part_o),
+                                 seq_lens.data_ptr(), q_start.data_ptr(), n_seqs, T, H, float(scale), window, n_splits, qt, _p(part_o),
                                  _p(part_ml), o.data_ptr(), ws.status.data_ptr(), _stream()), "mla_flash")
         if n_splits > 1:
             _ck(load().jib_mla_combine(part_o.data_ptr(), part_ml.data_ptr(), n_splits, T, H, r, o.data_ptr(), _stream()),
                 "mla_combine")
         return o
     n_splits = 1 if prefill and T > 64 else attn_splits(T, H)
+    if window > 0:
+        n_splits = min(n_splits, (window + 63) // 64)                 # a split of this kernel holds at least 64 rows
     if n_splits > 1:
         part_o = torch.empty(T, n_splits, H, r, dtype=torch.float32, device=q.device)
         part_ml = torch.empty(T, n_splits, H, 2, dtype=torch.float32, device=q.device)
@@ -369,7 +417,7 @@ def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_siz
         part_o = part_ml = None
     _ck(load().jib_mla_attention(q.data_ptr(), cache.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
                                  seq_lens.data_ptr(), q_start.data_ptr(), n_seqs, T, H, r, D - r, block_size, float(scale),
-                                 n_splits, _p(part_o), _p(part_ml), o.data_ptr(), _stream()), "mla_attention")
+                                 window, n_splits, int(q.dtype == torch.float32), _p(part_o), _p(part_ml), o.data_ptr(), _stream()), "mla_attention")
     return o
 
 
@@ -377,59 +425,71 @@ MHA_PREFILL = os.environ.get("JIB_MHA_PREFILL", "1") == "1"      # "0": prompt c
 MHA_PREFILL_MIN_TOKENS = 64
 
 
-def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, meta) -> bool:
+def visible_total(meta, window: int) -> int:
+    """Cached rows the queries of a step can see, over its sequences (what ``kv_gather`` writes)."""
+    if window <= 0:
+        return int(meta["total_kv"])
+    return sum(min(int(s), int(q) + window - 1) for q, s in zip(meta["q_lens"], meta["s_lens"]))
+
+
+def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, meta, window: int = 0) -> bool:
     """Whether a chunk of T query tokens takes the per-head prefill attention (needs the host-side totals in ``meta``)."""
     if not (MHA_PREFILL and meta is not None and T >= MHA_PREFILL_MIN_TOKENS and dn == 128 and dr == 64 and dv == 128 and r == 512):
         return False
     total, dec = meta.get("total_kv", 0), meta.get("kv_decode", 0)
+    if window > 0:
+        if "q_lens" not in meta:
+            return False
+        total = visible_total(meta, window)
+        dec = sum(min(int(s), window) for q, s in zip(meta["q_lens"], meta["s_lens"]) if q <= 1)
     # Expanding K / V costs ~4 MFLOP per cached row and pays for itself over the many query rows of a prompt; a sequence that
     # only decodes brings one query row and its whole context.  A mixed step whose gathered rows are mostly such contexts
     # stays with the absorbed form, which reads the latent rows as they are.
     return total > 0 and dec <= total - dec
 
 
-def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int):
-    """The cached latent rows of every sequence of the batch, in sequence order: ([total, row] bf16, first row of each
-    sequence [n_seqs] int32)."""
+def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int, q_start=None, window: int = 0):
+    """The cached latent rows of every sequence of the batch (with a window: those its query tokens can see), in sequence
+    order: ([total, row] bf16, first row of each sequence [n_seqs] int32)."""
     n_seqs = seq_lens.shape[0]
     row = cache.shape[1]
     lat = torch.empty(total, row, dtype=torch.bfloat16, device=cache.device)
     kv_start = torch.empty(n_seqs, dtype=torch.int32, device=cache.device)
     _ck(load().jib_kv_gather(cache.data_ptr(), cache.shape[0], block_tables.data_ptr(), block_tables.stride(0), seq_lens.data_ptr(),
-                             n_seqs, block_size, row, lat.data_ptr(), kv_start.data_ptr(), total, _stream()), "kv_gather")
+                             n_seqs, block_size, row, _p(q_start), window, lat.data_ptr(), kv_start.data_ptr(), total, _stream()), "kv_gather")
     return lat, kv_start
 
 
-def mha_prefill_core(q, kv, lat, kv_start, seq_lens, q_start, scale, n_head, n_q_tiles: int):
+def mha_prefill_core(q, kv, lat, kv_start, seq_lens, q_start, scale, n_head, n_q_tiles: int, window: int = 0):
     """The attention kernel itself: q [T, H*192], kv [total, H*256] = k_nope | v per head, lat [total, 576] (its last 64
     columns are the RoPE part of the keys, shared by the heads).  Returns [T, H*128] bf16."""
     T, total = q.shape[0], lat.shape[0]
     out = torch.empty(T, n_head * 128, dtype=torch.bfloat16, device=q.device)
     ws = workspace(q.device)
     _ck(load().jib_mha_prefill(q.data_ptr(), q.stride(0), kv.data_ptr(), lat.data_ptr() + 512 * 2, lat.shape[1], total,
-                               q_start.data_ptr(), seq_lens.data_ptr(), kv_start.data_ptr(), seq_lens.shape[0], T, n_head, float(scale),
+                               q_start.data_ptr(), seq_lens.data_ptr(), kv_start.data_ptr(), seq_lens.shape[0], T, n_head, float(scale), window,
                                int(n_q_tiles), out.data_ptr(), out.stride(0), ws.status.data_ptr(), _stream()), "mha_prefill")
     return out
 
 
-def mha_prefill(q, cache, w_kv_b, block_tables, seq_lens, q_start, scale, n_head, block_size, meta):
+def mha_prefill(q, cache, w_kv_b, block_tables, seq_lens, q_start, scale, n_head, block_size, meta, window: int = 0):
     """Causal multi-head attention of a prompt chunk in the per-head form.  q [T, H*192] (RoPE already applied in place; may
     be a strided view), cache [n_slots, 576] one layer's latent rows, w_kv_b [H*256, 512].  ``meta``: host-side totals of the
     batch, {"total_kv": sum of seq_lens, "n_q_tiles": upper bound of sum ceil(q_len / 128)}.  Returns [T, H*128] bf16."""
-    lat, kv_start = kv_gather(cache, block_tables, seq_lens, int(meta["total_kv"]), block_size)
+    lat, kv_start = kv_gather(cache, block_tables, seq_lens, visible_total(meta, window), block_size, q_start, window)
     kv = gemm(lat[:, :512], w_kv_b)                     # [total, H*256]: k_nope | v per head
-    return mha_prefill_core(q, kv, lat, kv_start, seq_lens, q_start, scale, n_head, int(meta["n_q_tiles"]))
+    return mha_prefill_core(q, kv, lat, kv_start, seq_lens, q_start, scale, n_head, int(meta["n_q_tiles"]), window)
 
 
 # ---- MoE -----------------------------------------------------------------------------------------
 def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None,
-             pre_norm=None):
+             pre_norm=None, logit_bias=None):
     """``route=(expert_base, E_local)``: the caller will sort these ids by local expert next (``moe_permute``); for decode
     batches both steps then run as one launch and ``moe_permute`` picks the result up.
     ``pre_norm=(weight, eps)``: ``g`` holds un-normalised rows; returns (ids, wts, rmsnorm(g) * weight), the norm done by
     the router launch itself for decode batches."""
     T, d = g.shape
-    fused = FUSED_ROUTE and route is not None and T <= FUSED_ROUTE_MAX_T
+    fused = FUSED_ROUTE and route is not None and T <= FUSED_ROUTE_MAX_T and logit_bias is None and g.dtype == torch.bfloat16
     g_in = g
     g_pre = None
     if pre_norm is not None and not (fused and ROUTE_NORM):
@@ -457,7 +517,9 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
         _route_stash.clear()                       # at most one pending result: the sort that follows this gate
         _route_stash[(ids.data_ptr(), expert_base, E_local)] = (seg, src, dest, ids)
         return (ids, wts, g_out if g_out is not None else g_pre) if pre_norm is not None else (ids, wts)
-    _ck(load().jib_moe_gate(g.data_ptr(), w_router.data_ptr(), _p(bias), logits.data_ptr(), ids.data_ptr(), wts.data_ptr(), T, d,
+    if g.dtype == torch.float32:
+        torch.matmul(g, w_router.T, out=logits)
+    _ck(load().jib_moe_gate(g.data_ptr() if g.dtype == torch.bfloat16 else None, w_router.data_ptr(), _p(bias), _p(logit_bias), logits.data_ptr(), ids.data_ptr(), wts.data_ptr(), T, d,
                             E, k, n_group, topk_group, float(scale), int(norm), int(sigmoid), n_shared, int(group_top2), _stream()), "moe_gate")
     return (ids, wts, g) if pre_norm is not None else (ids, wts)
 
@@ -492,6 +554,8 @@ def moe_tile_list(seg, E_local: int, bn: int, n_pairs: int) -> torch.Tensor:
 
 
 def gather_rows(x, src_row):
+    if x.dtype == torch.float32:                   # the kernel moves 16-byte vectors: an fp32 row is a bf16 row of twice the width
+        return gather_rows(x.view(torch.bfloat16), src_row).view(torch.float32)
     R, d = src_row.shape[0], x.shape[1]
     out = torch.empty(R, d, dtype=x.dtype, device=x.device)
     _ck(load().jib_gather_rows(x.data_ptr(), src_row.data_ptr(), out.data_ptr(), R, d, x.shape[0], _stream()), "gather_rows")
@@ -529,6 +593,9 @@ def moe_routed(x, ids, wts, wg, wu, wd, expert_base=0, n_expert=None):
     T, k = ids.shape
     E_local = wg.shape[0]
     seg, src, dest = moe_permute(ids, expert_base, E_local)
+    if not grouped_tma_ok(x, wg):                  # fp32 operands, or rows TMA cannot address
+        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, 0)
+        return gemm_grouped(h, seg, wd, None, T, 0), dest
     # the two grouped launches run back to back over one segment table: the second may start on its weights early
     pair = (1, 2) if GROUPED_PAIR else (0, 0)
     # few pairs, many experts: the grouped launches cover the list of experts that have rows instead of all of them
@@ -567,6 +634,73 @@ def moe_ffn(x, residual, ids, wts, wg, wu, wd, wgs, wus, wds, expert_base=0, n_e
     if wgs is not None:
         shared = gemm(gemm(x, wgs, wus), wds)
     return moe_combine(y, dest, wts, shared, residual, norm)
+
+
+# ---- parallel blocks over an fp32 residual (parallel_block.cu), per-sequence state (recurrent.cu) ------------------------------
+def _row_tail(x_out, nxt, dtype):
+    """(RowTail, h, hc) for ``nxt`` = (norm weight, eps, conv), see ``ops.embed_norm``."""
+    t, h, hc = RowTail(), None, None
+    t.x_out, t.status = x_out.data_ptr(), workspace(x_out.device).status.data_ptr()
+    if nxt is not None:
+        w, eps, conv = nxt
+        h = torch.empty(x_out.shape, dtype=dtype, device=x_out.device)
+        t.norm_w, t.eps, t.h_out = w.data_ptr(), float(eps), h.data_ptr()
+        if conv is not None:
+            cw, state, slots, positions = conv
+            assert cw.dtype == torch.float32 and cw.is_contiguous() and state.dtype == dtype and state.is_contiguous()
+            hc = torch.empty_like(h)
+            t.conv_w, t.hc_out, t.conv_state = cw.data_ptr(), hc.data_ptr(), state.data_ptr()
+            t.seq_slots, t.positions, t.taps, t.n_state = slots.data_ptr(), positions.data_ptr(), cw.shape[0], state.shape[0]
+    return t, h, hc
+
+
+def embed_norm(table, ids, w, eps, nxt=None):
+    T, d = ids.shape[0], table.shape[1]
+    x = torch.empty(T, d, dtype=torch.float32, device=table.device)
+    tail, h, hc = _row_tail(x, nxt, table.dtype)
+    _ck(load().jib_embed_norm(table.data_ptr(), ids.data_ptr(), w.data_ptr(), float(eps), T, d, table.shape[0],
+                              int(table.dtype == torch.float32), C.byref(tail), _stream()), "embed_norm")
+    return x, h, hc
+
+
+def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
+    T, d = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and o.is_contiguous() and gates.dtype == o.dtype and gates.stride(-1) == 1
+    y, dest, wts = moe if moe is not None else (None, None, None)
+    tail, h, hc = _row_tail(x, nxt, o.dtype)
+    _ck(load().jib_block_update(x.data_ptr(), float(mult), o.data_ptr(), gates.data_ptr(), gates.stride(0), b1.data_ptr(), _p(b2), _p(y), _p(dest),
+                                _p(wts), dest.shape[1] if dest is not None else 0, T, d, int(o.dtype == torch.float32), C.byref(tail),
+                                _stream()), "block_update")
+    return x, h, hc
+
+
+def rms_rows(x, rows, w, eps, dtype):
+    n, d = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
+    out = torch.empty(n, d, dtype=dtype, device=x.device)
+    _ck(load().jib_rms_rows(x.data_ptr(), _p(rows), w.data_ptr(), float(eps), n, d, x.shape[0], int(dtype == torch.float32), out.data_ptr(),
+                            _stream()), "rms_rows")
+    return out
+
+
+def causal_conv(h, w, state, seq_slots, positions, q_start):
+    T, d = h.shape
+    assert w.dtype == torch.float32 and w.is_contiguous() and h.is_contiguous() and state.dtype == h.dtype and state.is_contiguous()
+    out = torch.empty_like(h)
+    _ck(load().jib_causal_conv(h.data_ptr(), w.data_ptr(), w.shape[0], state.data_ptr(), state.shape[0], seq_slots.data_ptr(),
+                               positions.data_ptr(), q_start.data_ptr(), q_start.shape[0] - 1, T, d, int(h.dtype == torch.float32),
+                               out.data_ptr(), workspace(h.device).status.data_ptr(), _stream()), "causal_conv")
+    return out
+
+
+def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
+    """``single``: one token per sequence (row t belongs to sequence t)."""
+    T, W = zxg.shape[0], zb.shape[0]
+    assert state.dtype == torch.float32 and state.is_contiguous() and zxg.stride(-1) == 1
+    y = torch.empty(T, W, dtype=zxg.dtype, device=zxg.device)
+    _ck(load().jib_mingru(zxg.data_ptr(), zxg.stride(0), zb.data_ptr(), xb.data_ptr(), state.data_ptr(), state.shape[0], seq_slots.data_ptr(),
+                          positions.data_ptr(), q_start.data_ptr(), q_start.shape[0] - 1, T, W, int(single),
+                          int(zxg.dtype == torch.float32), y.data_ptr(), workspace(zxg.device).status.data_ptr(), _stream()), "mingru")
+    return y
 
 
 # ---- sampling / cache ----------------------------------------------------------------------------
@@ -609,6 +743,8 @@ def dequantize_bf16(raw, ggml_type: int, n_elements: int):
 
 
 def kv_block_copy(cache, src_blocks, dst_blocks, block_size):
+    if cache.dtype == torch.float32:
+        cache = cache.view(torch.bfloat16)
     L, n_slots, row = cache.shape
     _ck(load().jib_kv_block_copy(cache.data_ptr(), n_slots * row, L, src_blocks.data_ptr(), dst_blocks.data_ptr(),
                                  src_blocks.shape[0], block_size * row, _stream()), "kv_block_copy")

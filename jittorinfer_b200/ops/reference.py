@@ -65,36 +65,41 @@ def yarn_table(n_pos: int, dr: int, freq_base: float, freq_scale: float, ext_fac
     return torch.stack([torch.cos(theta) * m, torch.sin(theta) * m], dim=-1).float().to(device)
 
 
-def _rope(x: torch.Tensor, cs: torch.Tensor) -> torch.Tensor:
-    # x [T, ..., dr]; cs [T, dr/2, 2]
+def _rope(x: torch.Tensor, cs: torch.Tensor, half: bool = False) -> torch.Tensor:
+    """x [T, ..., dr]; cs [T, dr/2, 2].  Pairs are neighbours (2i, 2i + 1), or with ``half`` (i, i + dr/2)."""
     shp = x.shape
-    xp = x.float().reshape(*shp[:-1], shp[-1] // 2, 2)
     c, s = cs[..., 0], cs[..., 1]
-    while c.dim() < xp.dim() - 1:
+    while c.dim() < x.dim():
         c, s = c.unsqueeze(1), s.unsqueeze(1)
+    if half:
+        x0, x1 = x.float().chunk(2, dim=-1)
+        return torch.cat([x0 * c - x1 * s, x0 * s + x1 * c], dim=-1)
+    xp = x.float().reshape(*shp[:-1], shp[-1] // 2, 2)
     x0, x1 = xp[..., 0], xp[..., 1]
     return torch.stack([x0 * c - x1 * s, x0 * s + x1 * c], dim=-1).reshape(shp)
 
 
 def mla_qkv_post(q: torch.Tensor, ckv: torch.Tensor, kv_norm_w: torch.Tensor, eps: float, rope_table: torch.Tensor,
                  positions: torch.Tensor, slot_mapping: torch.Tensor, cache: torch.Tensor,
-                 q_out: torch.Tensor, n_head: int, dn: int, dr: int, r: int) -> torch.Tensor:
+                 q_out: torch.Tensor, n_head: int, dn: int, dr: int, r: int, rot_half: bool = False) -> torch.Tensor:
     """RMSNorm(c) + RoPE(k_pe) + latent-cache write + RoPE(q_pe)  (src/llama-graph-deepseek2.cpp:197-240).
 
     q [T, H*(dn+dr)], ckv [T, r+dr]; cache [n_slots, r+dr]; q_out [T, H, r+dr]: only the rope tail
     ``q_out[..., r:]`` is written here (the nope part is absorbed by :func:`q_absorb`).
-    Rows with ``slot_mapping < 0`` are padding and are skipped.  Returns q_nope [T,H,dn] (a view).
+    Rows with ``slot_mapping < 0`` are padding and are skipped.  ``ckv`` None: another layer has written the rows, only the
+    queries are rotated.  Returns q_nope [T,H,dn] (a view).
     """
     T = q.shape[0]
     cs = rope_table[positions.long()]
-    c = ckv[:, :r].float()
-    c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * kv_norm_w.float()
-    kpe = _rope(ckv[:, r:], cs)
-    row = torch.cat([c, kpe], dim=-1).to(cache.dtype)
-    valid = slot_mapping >= 0
-    cache[slot_mapping[valid].long()] = row[valid]
-    qv = q.view(T, n_head, dn + dr)
-    q_out[..., r:] = _rope(qv[..., dn:], cs).to(q_out.dtype)
+    if ckv is not None:
+        c = ckv[:, :r].float()
+        c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * kv_norm_w.float()
+        kpe = _rope(ckv[:, r:], cs, rot_half)
+        row = torch.cat([c, kpe], dim=-1).to(cache.dtype)
+        valid = slot_mapping >= 0
+        cache[slot_mapping[valid].long()] = row[valid]
+    qv = q.reshape(T, n_head, dn + dr)
+    q_out[..., r:] = _rope(qv[..., dn:], cs, rot_half).to(q_out.dtype)
     return qv[..., :dn]
 
 
@@ -110,11 +115,12 @@ def v_up(o_lat: torch.Tensor, w_uv: torch.Tensor) -> torch.Tensor:
 
 
 def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, seq_lens: torch.Tensor,
-                  q_start: torch.Tensor, scale: float, r: int, block_size: int) -> torch.Tensor:
+                  q_start: torch.Tensor, scale: float, r: int, block_size: int, window: int = 0) -> torch.Tensor:
     """Weight-absorbed MLA over the paged latent cache (src/llama-graph-attn.cpp:219-342).
 
     q [T,H,r+dr]; cache [n_blocks*block_size, r+dr]; sequence b owns query rows
-    q_start[b]:q_start[b+1] (its *last* tokens) and kv length seq_lens[b].  Returns o_lat [T,H,r].
+    q_start[b]:q_start[b+1] (its *last* tokens) and kv length seq_lens[b].  ``window`` > 0: position i sees j with
+    0 <= i - j < window.  Returns o_lat [T,H,r].
     """
     T, H, _ = q.shape
     out = torch.zeros(T, H, r, dtype=q.dtype, device=q.device)
@@ -133,6 +139,8 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
         Tq = q1 - q0
         pos = S - Tq + torch.arange(Tq, device=q.device)
         vis = torch.arange(S, device=q.device)[None, :] <= pos[:, None]
+        if window > 0:
+            vis &= torch.arange(S, device=q.device)[None, :] > pos[:, None] - window
         s = s.masked_fill(~vis[None], float("-inf"))
         p = torch.softmax(s, dim=-1)
         out[q0:q1] = torch.einsum("hts,sr->thr", p, lat[:, :r]).to(q.dtype)
@@ -141,10 +149,13 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
 
 def moe_gate(g: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], k: int, n_group: int,
              topk_group: int, scale: float, norm: bool, sigmoid: bool, n_shared: int = 0,
-             group_top2: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
+             group_top2: bool = False, logit_bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """Router matmul (fp32) + softmax/sigmoid + [group-limited] top-k + renorm/scale
-    (src/llama-graph-ffn.cpp:145-197).  Returns ids [T,k] int32, weights [T,k] fp32."""
+    (src/llama-graph-ffn.cpp:145-197).  ``bias`` takes part in the choice only, ``logit_bias`` is part of the logits (with
+    softmax and ``norm`` the weights are then a softmax over the chosen logits).  Returns ids [T,k] int32, weights [T,k] fp32."""
     logits = g.float() @ w_router.float().T
+    if logit_bias is not None:
+        logits = logits + logit_bias.float()
     probs = torch.sigmoid(logits) if sigmoid else torch.softmax(logits, dim=-1)
     sel = probs if bias is None else probs + bias.float()
     T, E = sel.shape
@@ -239,3 +250,96 @@ def kv_block_copy(cache: torch.Tensor, src_blocks: torch.Tensor, dst_blocks: tor
     L = cache.shape[0]
     c = cache.view(L, -1, block_size, cache.shape[-1])
     c[:, dst_blocks.long()] = c[:, src_blocks.long()]
+
+
+def moe_routed(x, ids, wts, wg, wu, wd):
+    """Expert outputs of every (token, choice) pair: (y [T*k, d], dest [T, k] row of each pair); here in pair order."""
+    T, k = ids.shape
+    y = torch.zeros(T * k, x.shape[1], dtype=x.dtype, device=x.device)
+    flat = ids.reshape(-1).long()
+    for e in range(wg.shape[0]):
+        rows = torch.nonzero(flat == e).reshape(-1)
+        if rows.numel():
+            y[rows] = linear(gateup_silu(x[rows // k], wg[e], wu[e]), wd[e])
+    return y, torch.arange(T * k, dtype=torch.int32, device=x.device).view(T, k)
+
+
+# ---- blocks over an fp32 residual stream whose sublayers read one norm (csrc/kernels/parallel_block.cu) ------------------------
+def _finish_row(x, nxt, dtype):
+    """x fp32 -> (x, h, hc) for ``nxt`` = (norm weight, eps, conv) with conv = None or (w [taps, d], state, seq_slots, positions)."""
+    if nxt is None:
+        return x, None, None
+    w, eps, conv = nxt
+    h = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
+    if conv is None:
+        return x, h, None
+    cw, state, slots, positions = conv
+    n = torch.arange(x.shape[0] + 1, dtype=torch.int32)
+    return x, h, causal_conv(h, cw, state, slots, positions, n)
+
+
+def embed_norm(table, ids, w, eps, nxt=None):
+    v = table[ids.long()].float()
+    return _finish_row(v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w, nxt, table.dtype)
+
+
+def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
+    """x + mult * (sigmoid(g1 + b1) * o + sigmoid(g2 + b2) * combine(moe)), ``moe`` = (y, dest, wts) or None."""
+    d = x.shape[1]
+    s = torch.sigmoid(gates[:, :d].float() + b1) * o.float()
+    if moe is not None:
+        y, dest, wts = moe
+        f = (y.float()[dest.long()] * wts[..., None]).sum(1)
+        s = s + torch.sigmoid(gates[:, d:2 * d].float() + b2) * f
+    return _finish_row(x + mult * s, nxt, o.dtype)
+
+
+def rms_rows(x, rows, w, eps, dtype):
+    v = x if rows is None else x[rows.long()]
+    return (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
+
+
+def causal_conv(h, w, state, seq_slots, positions, q_start):
+    """h + causal convolution over time, w [taps, d]; ``state`` [n, taps - 1, d] holds each sequence's last inputs."""
+    out = torch.empty_like(h)
+    taps = w.shape[0]
+    qs = q_start.tolist()
+    for b in range(len(qs) - 1):
+        q0, q1 = qs[b], qs[b + 1]
+        if q1 <= q0:
+            continue
+        slot = int(seq_slots[b])
+        old = torch.zeros(taps - 1, h.shape[1], dtype=h.dtype, device=h.device)
+        if slot >= 0 and taps > 1 and int(positions[q0]) > 0:
+            old = state[slot]
+        ext = torch.cat([old, h[q0:q1]], 0)
+        acc = h[q0:q1].float()
+        for j in range(taps):
+            acc = acc + w[j].float() * ext[j:j + q1 - q0].float()
+        out[q0:q1] = acc.to(h.dtype)
+        if slot >= 0 and taps > 1:
+            state[slot] = ext[q1 - q0:].clone()
+    return out
+
+
+def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
+    """S_t = (1 - z) S_(t-1) + z c, y = S silu(g) over zxg = [z | x | gate] pre-activations; ``state`` [n, W] fp32."""
+    W = zb.shape[0]
+    z = torch.sigmoid(zxg[:, :W].float() + zb)
+    u = zxg[:, W:2 * W].float() + xb
+    c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    g = F.silu(zxg[:, 2 * W:3 * W].float())
+    y = torch.empty(zxg.shape[0], W, dtype=zxg.dtype, device=zxg.device)
+    qs = q_start.tolist()
+    for b in range(len(qs) - 1):
+        q0, q1 = qs[b], qs[b + 1]
+        if q1 <= q0:
+            continue
+        slot = int(seq_slots[b])
+        s = state[slot].clone() if slot >= 0 and int(positions[q0]) > 0 else torch.zeros(W, device=zxg.device)
+        for t in range(q0, q1):
+            s = (1 - z[t]) * s + z[t] * c[t]
+            y[t] = (s * g[t]).to(y.dtype)
+        if slot >= 0:
+            state[slot] = s
+    return y

@@ -26,8 +26,8 @@ import torch
 from .. import ops
 from ..utils import fault
 from ..utils.trace import PhaseTimer, Tracer
-from ..models.deepseek2 import DeepSeek2Model, ForwardBatch
-from ..models.hparams import DeepSeek2HParams
+from ..models.deepseek2 import ForwardBatch
+from .cache import SplitCache                                          # noqa: F401  (re-exported)
 from .native_rt import PagedKV, Scheduler, StepArrays, i32p
 from .sampling import DeviceSampler, SamplingParams, device_samplable, make_sampler
 
@@ -97,8 +97,8 @@ class _StepIO:
             self.off[name] = (off, n)
             off = (off + n + 3) // 4 * 4           # keep every section 16-byte aligned
         self.total = off
-        # seq_slots / out_slots are host-only: the device copy stops before them
-        self.dev_len = self.off["seq_slots"][0]
+        # out_slots is host-only: the device copy stops before it
+        self.dev_len = self.off["out_slots"][0]
         pin = device.type == "cuda"
         self._pin = pin
         self.dev = torch.zeros(self.dev_len, dtype=torch.int32, device=device)
@@ -132,41 +132,12 @@ class _StepIO:
         return self.dev_len * 4
 
 
-class SplitCache:
-    """Latent cache of a layer-split model: one [layers-on-device, n_slots, row] tensor per device; ``cache[il]`` is the
-    layer's slice on its own device."""
-
-    def __init__(self, layer_dev, n_slots: int, row: int, dtype, block_size: int):
-        self.block_size = block_size
-        self.by_dev: Dict[torch.device, torch.Tensor] = {}
-        self.index: List[Tuple[torch.device, int]] = []
-        counts: Dict[torch.device, int] = {}
-        for d in layer_dev:
-            self.index.append((d, counts.get(d, 0)))
-            counts[d] = counts.get(d, 0) + 1
-        for d, n in counts.items():
-            self.by_dev[d] = torch.zeros(n, n_slots, row, dtype=dtype, device=d)
-
-    def __getitem__(self, il: int) -> torch.Tensor:
-        d, i = self.index[il]
-        return self.by_dev[d][i]
-
-    def copy_blocks(self, src: np.ndarray, dst: np.ndarray) -> None:
-        for d, t in self.by_dev.items():
-            s = torch.from_numpy(np.ascontiguousarray(src)).to(d)
-            e = torch.from_numpy(np.ascontiguousarray(dst)).to(d)
-            if d.type == "cuda":
-                with torch.cuda.device(d):
-                    ops.kv_block_copy(t, s, e, self.block_size)
-            else:
-                ops.kv_block_copy(t, s, e, self.block_size)
-
-
 class LLMEngine:
-    def __init__(self, model: DeepSeek2Model, cfg: EngineConfig = EngineConfig()):
+    def __init__(self, model, cfg: EngineConfig = EngineConfig()):
+        """``model``: an instance of one of the registry's model classes (``models/registry.py``)."""
         self.model = model
         self.cfg = cfg
-        self.hp: DeepSeek2HParams = model.hp
+        self.hp = model.hp
         self.device = model.device
         bs = cfg.block_size
         self.n_ctx_slot = cfg.n_ctx_slot or max(bs, cfg.n_ctx // cfg.n_parallel)
@@ -175,20 +146,14 @@ class LLMEngine:
         if self.n_ctx_slot > model.max_positions:
             raise ValueError(f"n_ctx_slot {self.n_ctx_slot} exceeds the model's RoPE table ({model.max_positions})")
         self.kv = PagedKV(self.n_blocks, bs, cfg.n_parallel)
-        self.sched = Scheduler(self.kv, cfg.n_parallel, cfg.n_batch, self.n_ctx_slot, self.hp.eos_id, cfg.n_keep,
-                               cfg.cont_batching)
-        if cfg.mixed_prompt_budget > 0:
-            self.sched.set_mixed_prompt_budget(cfg.mixed_prompt_budget)
-        if getattr(model, "split", False):
-            self.kv_cache = SplitCache(model.layer_dev, self.n_blocks * bs, self.hp.kv_row, model.dtype, bs)
-        else:
-            self.kv_cache = torch.zeros(self.hp.n_layer, self.n_blocks * bs, self.hp.kv_row, dtype=model.dtype,
-                                        device=self.device)
+        self.sched = self._new_scheduler()
+        self.kv_cache = model.make_cache(self.n_blocks * bs, cfg.n_parallel)
         cap_tokens = max(cfg.n_batch, max(cfg.graph_buckets))
         cap_seqs = max(cfg.n_parallel, max(cfg.graph_buckets))
         self.io = _StepIO(cap_tokens, cap_seqs, self.max_blocks, self.device)
         self.requests: Dict[int, RequestState] = {}
         self._next_id = 1
+        self._streams: Dict[object, int] = {}      # sequences fed by the caller (feed): key -> scheduler slot
         self._graphs: Dict[Tuple[int, str], Tuple[torch.cuda.CUDAGraph, torch.Tensor]] = {}
         self._use_graphs = cfg.cuda_graphs and self.device.type == "cuda" and not getattr(model, "split", False)
         self._out_host = torch.zeros(cap_seqs * (1 + 2 * max(1, cfg.presample_count)), dtype=torch.int32,
@@ -241,6 +206,14 @@ class LLMEngine:
         if getattr(model, "comm", None) is not None or getattr(self, "dp", False):
             self._host_barrier()
 
+    def _new_scheduler(self) -> Scheduler:
+        cfg = self.cfg
+        sched = Scheduler(self.kv, cfg.n_parallel, cfg.n_batch, self.n_ctx_slot, self.hp.eos_id, cfg.n_keep, cfg.cont_batching)
+        if cfg.mixed_prompt_budget > 0:
+            sched.set_mixed_prompt_budget(cfg.mixed_prompt_budget)
+        sched.set_recurrent(self.model.recurrent)
+        return sched
+
     # ------------------------------------------------------------------------------------------
     def add_request(self, prompt: Sequence[int], params: Optional[SamplingParams] = None) -> int:
         params = params or SamplingParams()
@@ -284,15 +257,18 @@ class LLMEngine:
             q_len, s_len = np.diff(qs), h["seq_lens"][:n_seqs]
             # kv_decode: cached rows of the sequences that only decode in this step (the per-head form would expand them all)
             meta = {"total_kv": int(s_len.sum()), "n_q_tiles": int(((q_len + 127) // 128).sum()),
-                    "kv_decode": int(s_len[q_len <= 1].sum())}
+                    "kv_decode": int(s_len[q_len <= 1].sum()), "q_lens": q_len.tolist(), "s_lens": s_len.tolist()}
         return ForwardBatch(tokens=d["tokens"][:n_tokens], positions=d["positions"][:n_tokens],
                             slot_mapping=d["slot_mapping"][:n_tokens],
                             block_tables=d["block_tables"].view(self.io.cap_seqs, self.max_blocks)[:n_seqs],
                             seq_lens=d["seq_lens"][:n_seqs], q_start=d["q_start"][:n_seqs + 1],
-                            out_rows=d["out_rows"][:n_out], max_q_len=max_q_len, attn_meta=meta)
+                            out_rows=d["out_rows"][:n_out], max_q_len=max_q_len, attn_meta=meta, seq_slots=d["seq_slots"][:n_seqs])
 
     def _sample_device(self, logits: torch.Tensor, mode: str) -> torch.Tensor:
-        """Returns an int32 tensor: [n] token ids (greedy) or [n, 2k] (k float bit patterns + k ids)."""
+        """Returns an int32 tensor: [n] token ids (greedy) or [n, 2k] (k float bit patterns + k ids); mode "logits": the fp32
+        logits themselves."""
+        if mode == "logits":
+            return logits
         if mode == "greedy":
             return ops.argmax(logits)
         k = min(self.cfg.presample_count, logits.shape[-1])
@@ -345,6 +321,8 @@ class LLMEngine:
         bs = self.cfg.block_size
         for il in range(self.hp.n_layer):
             layer = self.kv_cache[il]
+            if layer is None:            # a layer without paged rows
+                continue
             rows = (torch.from_numpy(blocks.astype(np.int64)).to(layer.device)[:, None] * bs +
                     torch.arange(bs, device=layer.device)[None, :]).reshape(-1)
             layer[rows] = float("nan")
@@ -355,13 +333,18 @@ class LLMEngine:
         if key in self._graphs:
             return self._graphs[key]
         batch = self._batch_views(bucket, bucket, bucket, 1)
-        # warm-up on a side stream (allocations, lazy init), then capture
+        # warm-up on a side stream (allocations, lazy init), then capture.  The warm-up passes must not advance any sequence's
+        # state: they run with every row marked as belonging to no slot (rewriting cached rows with the same values is harmless).
+        slots = self.io.d["seq_slots"][:bucket]
+        kept = slots.clone()
+        slots.fill_(-1)
         s = torch.cuda.Stream(device=self.device)
         s.wait_stream(torch.cuda.current_stream(self.device))
         with torch.cuda.stream(s):
             for _ in range(2):
                 self._forward_sample(batch, mode)
         torch.cuda.current_stream(self.device).wait_stream(s)
+        slots.copy_(kept)
         torch.cuda.synchronize(self.device)
         g = torch.cuda.CUDAGraph()
         n0 = ops.nat().launch_count if not ops.force_torch() else 0
@@ -395,11 +378,9 @@ class LLMEngine:
         between planning and commit).  Weights, cache memory and captured graphs stay."""
         cfg = self.cfg
         self.kv = PagedKV(self.n_blocks, cfg.block_size, cfg.n_parallel)
-        self.sched = Scheduler(self.kv, cfg.n_parallel, cfg.n_batch, self.n_ctx_slot, self.hp.eos_id, cfg.n_keep,
-                               cfg.cont_batching)
-        if cfg.mixed_prompt_budget > 0:
-            self.sched.set_mixed_prompt_budget(cfg.mixed_prompt_budget)
+        self.sched = self._new_scheduler()
         self.requests.clear()
+        self._streams.clear()
         self._pressure = False
         self._inflight = None
         if self._poison:
@@ -428,6 +409,7 @@ class LLMEngine:
         h["samp"][:] = 0
         h["slot_mapping"][:] = -1
         h["seq_lens"][:] = 0
+        h["seq_slots"][:] = -1
         h["q_start"][:] = np.arange(len(h["q_start"]))
         h["out_rows"][:] = np.arange(len(h["out_rows"]))
         self.io.upload()
@@ -464,7 +446,7 @@ class LLMEngine:
         return len(src)
 
     def _copy_blocks(self, src: np.ndarray, dst: np.ndarray):
-        if isinstance(self.kv_cache, SplitCache):
+        if not isinstance(self.kv_cache, torch.Tensor):
             self.kv_cache.copy_blocks(src, dst)
             return
         s = torch.from_numpy(np.ascontiguousarray(src)).to(self.device)
@@ -542,6 +524,110 @@ class LLMEngine:
         self.stats["d2h_bytes"] += infl.n_out * 4 + (16 if infl.status is not None else 0)
         return infl.host[:infl.n_out].numpy().astype(np.int32, copy=True)
 
+    def _dispatch(self, n_tokens: int, n_seqs: int, n_out: int, max_q: int, mode: str, after_upload=None,
+                  out_rows: Optional[torch.Tensor] = None):
+        """Uploads the assembled step and runs the model on it: a graph replay for decode-only batches, eagerly otherwise.
+        ``out_rows`` (device): rows whose logits an eager step returns, instead of the ones the scheduler named.  Returns
+        (result of ``_sample_device`` or None, whether a graph ran)."""
+        io = self.io
+        use_graph = self._use_graphs and max_q == 1 and n_seqs == n_tokens and n_seqs <= max(self.cfg.graph_buckets) \
+            and getattr(self.model, "tensor_hook", None) is None
+        bucket = next(b for b in self.cfg.graph_buckets if b >= n_seqs) if use_graph else 0
+        if use_graph and self.dp:
+            # ranks capture in lockstep during warmup() only: a capture on first use would run collectives alone
+            use_graph = (bucket, mode) in self._graphs
+        if use_graph and bucket > n_seqs:
+            h = io.h
+            h["tokens"][n_seqs:bucket] = 0
+            h["positions"][n_seqs:bucket] = 0
+            h["slot_mapping"][n_seqs:bucket] = -1
+            h["seq_lens"][n_seqs:bucket] = 0
+            h["seq_slots"][n_seqs:bucket] = -1
+            h["q_start"][n_seqs:bucket + 1] = np.arange(n_seqs, bucket + 1)
+            h["out_rows"][n_out:bucket] = np.arange(n_out, bucket)
+            h["block_tables"][n_seqs * self.max_blocks: bucket * self.max_blocks] = 0
+        io.upload()                          # before a first-use capture too: its warm-up runs read these buffers
+        if after_upload is not None:
+            after_upload()
+        if use_graph:
+            g, out = self._graph_for(bucket, mode)
+            g.replay()
+            self.launches += self.graph_launches.get((bucket, mode), 0)
+            self.stats["graph_steps"] += 1
+        else:
+            batch = self._batch_views(n_tokens, n_seqs, n_out, max_q)
+            if out_rows is not None:
+                batch.out_rows = out_rows
+            count = self.device.type == "cuda" and not ops.force_torch()
+            n0 = ops.nat().launch_count if count else 0
+            out = self._forward_sample(batch, mode) if batch.out_rows.shape[0] else None
+            if out is None:
+                self.model.forward(batch, self.kv_cache)
+            if count:
+                self.launches += ops.nat().launch_count - n0
+            self.stats["eager_steps"] += 1
+        self.stats["steps"] += 1
+        self.stats["tokens_in"] += n_tokens
+        self.stats["h2d_bytes"] += io.h2d_bytes
+        return out, use_graph
+
+    # ---- sequences whose tokens the caller supplies --------------------------------------------------------------------------
+    @torch.no_grad()
+    def feed(self, entries: Sequence[Tuple[object, Sequence[int], Sequence[int]]]) -> torch.Tensor:
+        """One engine step over given tokens (replaying a trace, scoring text): every entry is (key, next tokens, places among
+        them whose logits are wanted).  A key is admitted to a slot at its first entry, may be left out of later steps, and
+        holds its slot and cache blocks until ``end_feed``.  Batching, cache, state and kernels are those of ``step``.
+        Returns the fp32 logits [wanted, n_vocab] on the CPU, in the order of the entries and their places."""
+        if self._inflight is not None:
+            self.sched.commit(self._collect(self._inflight), self._inflight.n_out)
+            self._inflight = None
+        entries = [e for e in entries if len(e[1])]
+        keys = [e[0] for e in entries]
+        if len(set(keys)) != len(keys):
+            raise ValueError("a sequence can take part in a step once")
+        for _, toks, want in entries:
+            if min(toks) < 0 or max(toks) >= self.hp.n_vocab:
+                raise ValueError(f"token ids must be in [0, {self.hp.n_vocab})")
+            if len(want) and (min(want) < 0 or max(want) >= len(toks)):
+                raise ValueError("a wanted place lies outside the entry's tokens")
+        if not entries:
+            return torch.empty(0, self.hp.n_vocab)
+        for k in keys:
+            if k not in self._streams:
+                slot = self.sched.fed_open()
+                if slot < 0:
+                    raise RuntimeError("no free sequence slot")
+                self._streams[k] = slot
+        lens = [len(e[1]) for e in entries]
+        flat = [t for e in entries for t in e[1]]
+        info = self.sched.step_fed(self.io.arrays, [self._streams[k] for k in keys], lens, flat)
+        n_tokens, n_seqs, _, _, max_q, _, n_copies = (int(x) for x in info[:7])
+        if n_tokens == 0:
+            raise RuntimeError("the step does not fit: cache blocks, batch size or a sequence's length limit")
+        if n_copies:
+            src, dst = self.kv.take_copies()
+            self._copy_blocks(src, dst)
+        if self._poison:
+            self._poison_freed()
+        starts = np.concatenate([[0], np.cumsum(lens)])
+        rows = [int(s) + int(p) for s, (_, _, want) in zip(starts, entries) for p in want]
+        rows_dev = torch.tensor(rows, dtype=torch.int32).to(self.device)
+        # a graph computes every row's logits (row t is sequence t); an eager step computes the wanted ones
+        self.io.h["out_rows"][:n_seqs] = np.arange(n_seqs)
+        out, graph = self._dispatch(n_tokens, n_seqs, n_seqs if max_q == 1 else 0, max_q, "logits", out_rows=rows_dev)
+        self.stats["tokens_out"] += len(rows)
+        if graph and rows:
+            out = out.index_select(0, rows_dev.long())
+        res = out.float().cpu() if rows else torch.empty(0, self.hp.n_vocab)
+        if self._status_hosts is not None:
+            self._status_hosts[0].copy_(self._status_dev)
+            self._check_device_status(self._status_hosts[0])
+        return res
+
+    def end_feed(self, key: object) -> None:
+        """Gives back the slot and the cache blocks of a fed sequence."""
+        self.sched.fed_close(self._streams.pop(key))
+
     def _launch_greedy(self, n_tokens: int, n_seqs: int, n_out: int, max_q: int, feedback: Optional[_InFlight]) -> _InFlight:
         """Launches a step whose ids are chosen on the device (arg-max, or the device sampler for requests that use it)."""
         io = self.io
@@ -549,20 +635,7 @@ class LLMEngine:
         mode = self._step_mode(states)
         if mode == "sample":
             self._fill_sampling_rows(states, io.cap_seqs)
-        use_graph = self._use_graphs and max_q == 1 and n_seqs == n_tokens and n_seqs <= max(self.cfg.graph_buckets) \
-            and getattr(self.model, "tensor_hook", None) is None
-        bucket = next(b for b in self.cfg.graph_buckets if b >= n_seqs) if use_graph else 0
-        if use_graph and bucket > n_seqs:
-            h = io.h
-            h["tokens"][n_seqs:bucket] = 0
-            h["positions"][n_seqs:bucket] = 0
-            h["slot_mapping"][n_seqs:bucket] = -1
-            h["seq_lens"][n_seqs:bucket] = 0
-            h["q_start"][n_seqs:bucket + 1] = np.arange(n_seqs, bucket + 1)
-            h["out_rows"][n_out:bucket] = np.arange(n_out, bucket)
-            h["block_tables"][n_seqs * self.max_blocks: bucket * self.max_blocks] = 0
-        io.upload()
-        if feedback is not None:
+        def feed_back():
             # this step's tokens are the ids the step in flight sampled: a device-to-device copy, in output-row order
             row_of = {int(sl): i for i, sl in enumerate(feedback.out_slots)}
             src = np.fromiter((row_of[int(sl)] for sl in io.h["seq_slots"][:n_seqs]), dtype=np.int64, count=n_seqs)
@@ -571,18 +644,7 @@ class LLMEngine:
                 io.d["tokens"][:n_seqs].copy_(prev[:n_seqs])
             else:
                 io.d["tokens"][:n_seqs].copy_(prev.index_select(0, torch.from_numpy(src).to(prev.device)))
-        if use_graph:
-            g, out = self._graph_for(bucket, mode)
-            g.replay()
-            self.launches += self.graph_launches.get((bucket, mode), 0)
-            self.stats["graph_steps"] += 1
-        else:
-            batch = self._batch_views(n_tokens, n_seqs, n_out, max_q)
-            n0 = ops.nat().launch_count if self.device.type == "cuda" and not ops.force_torch() else 0
-            out = self._forward_sample(batch, mode)
-            if self.device.type == "cuda" and not ops.force_torch():
-                self.launches += ops.nat().launch_count - n0
-            self.stats["eager_steps"] += 1
+        out, _ = self._dispatch(n_tokens, n_seqs, n_out, max_q, mode, after_upload=feed_back if feedback is not None else None)
         host = self._out_hosts[self._flip]
         self._flip ^= 1
         host[:n_out].copy_(out.reshape(-1)[:n_out], non_blocking=True)
@@ -594,10 +656,7 @@ class LLMEngine:
         if self.device.type == "cuda":
             event = torch.cuda.Event()
             event.record()
-        self.stats["steps"] += 1
-        self.stats["tokens_in"] += n_tokens
         self.stats["tokens_out"] += n_out
-        self.stats["h2d_bytes"] += io.h2d_bytes
         return _InFlight(out, host, event, n_out, io.h["out_slots"][:n_out].copy(), status)
 
     def _trace_ahead(self, pt, ev, launched, n_tokens=0, n_seqs=0, n_out=0, max_q=0) -> None:
@@ -717,42 +776,9 @@ class LLMEngine:
         states = [self.requests[int(r)] for r in self.sched.out_reqs(n_out)] if n_out else []
         mode = self._step_mode(states)
         samp_rows = self._fill_sampling_rows(states, io.cap_seqs) if mode != "greedy" else None
-        use_graph = self._use_graphs and max_q == 1 and n_seqs == n_tokens and n_seqs <= max(self.cfg.graph_buckets) \
-            and getattr(self.model, "tensor_hook", None) is None
-        if use_graph and self.dp:
-            # ranks capture in lockstep during warmup() only: a capture on first use would run collectives alone
-            use_graph = (next(b for b in self.cfg.graph_buckets if b >= n_seqs), mode) in self._graphs
-        if use_graph:
-            bucket = next(b for b in self.cfg.graph_buckets if b >= n_seqs)
-            h = io.h
-            if bucket > n_seqs:
-                h["tokens"][n_seqs:bucket] = 0
-                h["positions"][n_seqs:bucket] = 0
-                h["slot_mapping"][n_seqs:bucket] = -1
-                h["seq_lens"][n_seqs:bucket] = 0
-                h["q_start"][n_seqs:bucket + 1] = np.arange(n_seqs, bucket + 1)
-                h["out_rows"][n_out:bucket] = np.arange(n_out, bucket)
-                h["block_tables"][n_seqs * self.max_blocks: bucket * self.max_blocks] = 0
-            io.upload()                      # before a first-use capture too: its warm-up runs read these buffers
-            g, out = self._graph_for(bucket, mode)
-            g.replay()
-            self.launches += self.graph_launches.get((bucket, mode), 0)
-            self.stats["graph_steps"] += 1
-        else:
-            io.upload()
-            batch = self._batch_views(n_tokens, n_seqs, n_out, max_q)
-            n0 = ops.nat().launch_count if self.device.type == "cuda" and not ops.force_torch() else 0
-            out = self._forward_sample(batch, mode) if n_out else None
-            if n_out == 0:
-                self.model.forward(batch, self.kv_cache)
-            if self.device.type == "cuda" and not ops.force_torch():
-                self.launches += ops.nat().launch_count - n0
-            self.stats["eager_steps"] += 1
+        out, use_graph = self._dispatch(n_tokens, n_seqs, n_out, max_q, mode)
         if pt:
             pt.mark("launch")
-        self.stats["steps"] += 1
-        self.stats["tokens_in"] += n_tokens
-        self.stats["h2d_bytes"] += io.h2d_bytes
         if n_out:
             flat = out.reshape(-1)
             n_el = flat.numel()

@@ -9,19 +9,40 @@ from typing import Optional, Sequence
 
 import torch
 
+from ..models import registry
 from ..models.deepseek2 import DeepSeek2Model
 from ..models.hparams import DeepSeek2HParams
 from ..models.weights import ShardSpec, iter_gguf, iter_random
 from .engine import EngineConfig, LLMEngine
 
 
+def _build_folder_arch(arch: registry.Architecture, hp, path: Optional[str], device, dtype: torch.dtype, world: int, seed: int,
+                       max_positions: int, check_tensors: bool, layer_devices):
+    """Models of architectures that come as a folder (or, with ``path`` None, with random weights): one GPU."""
+    if world > 1 or layer_devices is not None:
+        raise ValueError(f"{arch.name} runs on one GPU: no tensor, expert or layer parallelism")
+    dev = torch.device(device)
+    if path is not None:
+        hp = arch.load_config(path)
+        weights = arch.iter_checkpoint(path, hp)
+        if check_tensors:
+            from ..models.weights import checked
+            weights = checked(weights)
+    else:
+        weights = arch.iter_random(hp, seed=seed, dtype=dtype if dev.type == "cuda" else torch.float32, device=dev)
+    return arch.model(hp, weights, dtype=dtype, device=dev, max_positions=max_positions)
+
+
 def build_model(hp: Optional[DeepSeek2HParams] = None, gguf_path: Optional[str] = None, device="cuda",
                 dtype: torch.dtype = torch.bfloat16, world: int = 1, rank: int = 0, expert_parallel: bool = True,
                 comm=None, seed: int = 0, std: float = 0.02, max_positions: int = 8192, fast_random: bool = True,
                 dp_attention: bool = False, ep_max_tokens: int = 256, layer_devices=None,
-                tensor_split=None, kv_overrides=None, check_tensors: bool = False) -> DeepSeek2Model:
-    """``dp_attention``: attention data-parallel (every rank serves its own requests), routed experts sharded over the
+                tensor_split=None, kv_overrides=None, check_tensors: bool = False):
+    """``gguf_path``: a GGUF file, or the folder of an architecture that comes as config.json + safetensors.  ``dp_attention``: attention data-parallel (every rank serves its own requests), routed experts sharded over the
     ranks and reached through the all-to-all dispatcher; ``ep_max_tokens`` bounds the tokens of one rank per step."""
+    arch = registry.for_path(gguf_path) if gguf_path is not None else registry.for_hparams(hp)
+    if arch.load_config is not None:
+        return _build_folder_arch(arch, hp, gguf_path, device, dtype, world, seed, max_positions, check_tensors, layer_devices)
     dp_attention = dp_attention and world > 1
     spec = ShardSpec(rank, world, (expert_parallel or dp_attention) and world > 1, dp_attention)
     if gguf_path is not None:
@@ -93,8 +114,7 @@ def build_engine(hp: Optional[DeepSeek2HParams] = None, gguf_path: Optional[str]
     dev = torch.device(device)
     if not n_ctx and gpu_memory_utilization and dev.type == "cuda":
         free, total = torch.cuda.mem_get_info(dev)
-        elem = torch.empty(0, dtype=dtype).element_size()
-        fit = kv_tokens_for_budget(total, free, gpu_memory_utilization, model.hp.n_layer, model.hp.kv_row, elem)
+        fit = kv_tokens_for_budget(total, free, gpu_memory_utilization, 1, model.cache_bytes_per_token(), 1)
         if fit < n_ctx_slot:
             raise RuntimeError(f"only {fit} cache tokens fit at gpu_memory_utilization={gpu_memory_utilization}; "
                                f"one sequence needs {n_ctx_slot}")

@@ -75,6 +75,10 @@ def lib():
         sig("jib_sched_add_keep", None, vp, C.c_int64, i32p, C.c_int, C.c_int, C.c_int, C.c_int)
         sig("jib_sched_cancel", C.c_int, vp, C.c_int64)
         sig("jib_sched_step", C.c_int, vp, C.POINTER(StepArrays), i32p)
+        sig("jib_sched_fed_open", C.c_int, vp)
+        sig("jib_sched_fed_close", C.c_int, vp, C.c_int)
+        sig("jib_sched_step_fed", C.c_int, vp, C.POINTER(StepArrays), i32p, i32p, C.c_int, i32p, i32p)
+        sig("jib_sched_set_recurrent", None, vp, C.c_int)
         sig("jib_sched_commit", None, vp, i32p, C.c_int)
         sig("jib_sched_can_run_ahead", C.c_int, vp)
         sig("jib_sched_commit_deferred", None, vp, C.c_int)
@@ -161,7 +165,7 @@ class PagedKV:
 
 
 FINISH_NAMES = {0: None, 1: "stop", 2: "length", 3: "cancelled", 4: "error"}
-SLOT_STATES = ("IDLE", "STARTED", "PROCESSING_PROMPT", "DONE_PROMPT", "GENERATING")
+SLOT_STATES = ("IDLE", "STARTED", "PROCESSING_PROMPT", "DONE_PROMPT", "GENERATING", "FED")
 
 
 class Scheduler:
@@ -199,6 +203,19 @@ class Scheduler:
         """Returns int32 info: n_tokens, n_seqs, n_out, n_decode_seqs, max_q_len, n_preempted, n_copies."""
         self._L.jib_sched_step(self._h, C.byref(arrays), _p32(self._info))
         return self._info
+
+    # sequences whose tokens the caller supplies (csrc/runtime/scheduler.h)
+    def fed_open(self) -> int: return int(self._L.jib_sched_fed_open(self._h))
+    def fed_close(self, slot: int) -> bool: return bool(self._L.jib_sched_fed_close(self._h, slot))
+
+    def step_fed(self, arrays: StepArrays, slots, lens, tokens) -> np.ndarray:
+        """Assembles a batch that appends ``lens[i]`` of ``tokens`` to each slot; the info of ``step`` (n_tokens 0: no room)."""
+        sl, ln, tk = (np.ascontiguousarray(a, dtype=np.int32) for a in (slots, lens, tokens))
+        self._info[:] = 0
+        self._L.jib_sched_step_fed(self._h, C.byref(arrays), _p32(sl), _p32(ln), len(sl), _p32(tk), _p32(self._info))
+        return self._info
+
+    def set_recurrent(self, on: bool) -> None: self._L.jib_sched_set_recurrent(self._h, int(on))
 
     def commit(self, sampled: np.ndarray, n_out: int):
         self._L.jib_sched_commit(self._h, _p32(sampled), n_out)

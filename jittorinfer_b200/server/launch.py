@@ -11,7 +11,7 @@ log = logging.getLogger("jittorinfer_b200.server")
 
 def build_from_config(cfg, device=None, world: int = 1, rank: int = 0):
     import torch
-    from ..models.hparams import preset
+    from ..models.registry import is_folder_model, preset
     from ..runtime.factory import build_engine
     from ..tokenizer import Tokenizer
     from ..utils.toy_vocab import toy_vocab_kv
@@ -30,7 +30,8 @@ def build_from_config(cfg, device=None, world: int = 1, rank: int = 0):
                   mixed_prompt_budget=int(getattr(cfg, "mixed_prompt_budget", 0)),
                   check_tensors=bool(getattr(cfg, "check_tensors", False)))
     hp_known = preset(cfg.random_init) if cfg.random_init else None
-    if world == 1 and device.type == "cuda" and cfg.split_mode == "LLAMA_SPLIT_MODE_LAYER":
+    folder = is_folder_model(cfg.model) and not cfg.random_init
+    if world == 1 and device.type == "cuda" and not folder and (hp_known is None or hasattr(hp_known, "kv_row")) and cfg.split_mode == "LLAMA_SPLIT_MODE_LAYER":
         n = int(getattr(cfg, "layer_split_gpus", 1))
         if n <= 0:          # automatic, as the reference spreads layers over all devices by free memory (src/llama-model.cpp:495-540)
             if hp_known is None:
@@ -44,11 +45,14 @@ def build_from_config(cfg, device=None, world: int = 1, rank: int = 0):
         if n > 1:
             common.update(layer_devices=[torch.device("cuda", (cfg.main_gpu + i) % torch.cuda.device_count()) for i in range(n)],
                           tensor_split=list(cfg.tensor_split) or None)
-    if cfg.random_init:
-        hp = hp_known
-        eng = build_engine(hp, **common)
+    if cfg.random_init or folder:
+        # no vocabulary comes with the model: byte-level toy tokens (architectures without special tokens add none)
+        eng = build_engine(None, gguf_path=cfg.model, **common) if folder else build_engine(hp_known, **common)
+        hp = eng.hp
         kv = {k: (v[1] if isinstance(v, tuple) else v) for k, v in toy_vocab_kv(hp.n_vocab, hp.bos_id, hp.eos_id).items()}
         kv["tokenizer.ggml.bos_token_id"], kv["tokenizer.ggml.eos_token_id"] = hp.bos_id, hp.eos_id
+        if hp.bos_id < 0:
+            kv["tokenizer.ggml.add_bos_token"] = False
         tok = Tokenizer.from_gguf_kv(kv)
         template_src = ""
     else:
@@ -89,7 +93,7 @@ def main(argv=None, world: int = 1, rank: int = 0, control_group=None) -> int:
     ap.add_argument("--config", "-c", default=None, help="YAML file with the reference's keys (configs/*.yaml)")
     ap.add_argument("--port", type=int, default=None)
     ap.add_argument("--host", default=None)
-    ap.add_argument("--random-init", default=None, help="serve a random-init preset (tiny | lite | v2) instead of a GGUF file")
+    ap.add_argument("--random-init", default=None, help="serve a random-init preset (tiny | lite | v2 | nibalix-tiny | nibalix-lite) instead of a model file")
     args = ap.parse_args(argv)
     logging.basicConfig(level=os.environ.get("JITTORINFER_LOG", "INFO"), format="%(asctime)s %(levelname)s %(name)s: %(message)s")
     from ..config import load_yaml
