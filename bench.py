@@ -123,9 +123,15 @@ def main():
     ap.add_argument("--timeline", action="store_true",
                     help="diagnostic (needs JITTORINFER_KERNELS_SO = the timeline build): report how long the fused all-reduces "
                          "wait for their peers during the timed steps; the stamps cost time, so the tokens/s of such a run is not a result")
+    ap.add_argument("--design", default=None,
+                    help="instead of the headline: prefill and decode throughput of this design (nibalix) at real layer sizes beside the "
+                         "closest other model at equal sizes (1 GPU)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.design:
+        from jittorinfer_b200.utils import design_bench
+        return design_bench.run(args, ClockSampler(0).start())
     if args.warmup < 3:
         args.warmup = 3
 

@@ -38,46 +38,50 @@ __device__ __forceinline__ float block_sum(float v, float * red) {
     return t;
 }
 
-__device__ __forceinline__ void load4(const float * p, float (&v)[4]) {
-    const float4 a = *(const float4 *) p;
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-}
-__device__ __forceinline__ void load4(const bf16 * p, float (&v)[4]) {
-    const uint2 raw = *(const uint2 *) p;
-    const float2 a = __bfloat1622float2(*(const __nv_bfloat162 *) &raw.x), b = __bfloat1622float2(*(const __nv_bfloat162 *) &raw.y);
-    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-}
-__device__ __forceinline__ void store4(float * p, const float (&v)[4]) { *(float4 *) p = make_float4(v[0], v[1], v[2], v[3]); }
-__device__ __forceinline__ void store4(bf16 * p, const float (&v)[4]) {
-    uint2 o;
-    *(__nv_bfloat162 *) &o.x = __floats2bfloat162_rn(v[0], v[1]);
-    *(__nv_bfloat162 *) &o.y = __floats2bfloat162_rn(v[2], v[3]);
-    *(uint2 *) p = o;
-}
-__device__ __forceinline__ void round4(float (&)[4], const float *) {}
-__device__ __forceinline__ void round4(float (&v)[4], const bf16 *) {
+// 8 adjacent elements of a row: one 16-byte access of bf16, two of fp32.
+template <typename T> struct Pack8;
+template <> struct Pack8<bf16> {
+    uint4 r;
+    __device__ __forceinline__ void load(const bf16 * p) { r = *(const uint4 *) p; }
+    __device__ __forceinline__ void zero() { r = make_uint4(0, 0, 0, 0); }
+    __device__ __forceinline__ void store(bf16 * p) const { *(uint4 *) p = r; }
+    __device__ __forceinline__ void get(float (&v)[8]) const {
+        const __nv_bfloat162 * h = (const __nv_bfloat162 *) &r;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) v[e] = __bfloat162float(__float2bfloat16(v[e]));
+        for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+    }
+    __device__ __forceinline__ void set(const float (&v)[8]) {
+        __nv_bfloat162 * h = (__nv_bfloat162 *) &r;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    }
+};
+template <> struct Pack8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float * p) { a = ((const float4 *) p)[0]; b = ((const float4 *) p)[1]; }
+    __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+    __device__ __forceinline__ void store(float * p) const { ((float4 *) p)[0] = a; ((float4 *) p)[1] = b; }
+    __device__ __forceinline__ void get(float (&v)[8]) const {
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    }
+    __device__ __forceinline__ void set(const float (&v)[8]) { a = make_float4(v[0], v[1], v[2], v[3]); b = make_float4(v[4], v[5], v[6], v[7]); }
+};
+template <typename T> __device__ __forceinline__ void load8(const T * p, float (&v)[8]) {
+    Pack8<T> k;
+    k.load(p);
+    k.get(v);
 }
-__device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
+// bf16 activations: fast exponential and division (a few ulp of fp32); fp32 ones: the accurate forms.
+template <typename T> __device__ __forceinline__ float sigmoid(float v);
+template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
+
+constexpr int FAST_TAPS = 4;         // up to this many taps the stored rows are requested before the row's reductions
 
 // x row -> residual store, norm, and (decode) the next block's input convolution.
 template <typename T, int NT, int MAXV>
-__device__ __forceinline__ void finish_row(float (&v)[MAXV][4], int t, int d, const jib_row_tail & a, float * red, bool dry) {
-    const int nv = d / 4;
-    float ss = 0.f;
-#pragma unroll
-    for (int it = 0; it < MAXV; ++it) {
-        const int i = threadIdx.x + it * NT;
-        if (i < nv) {
-            if (!dry) store4((float *) a.x_out + (size_t) t * d + 4 * i, v[it]);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) ss += v[it][e] * v[it][e];
-        }
-    }
-    if (a.norm_w == nullptr) return;
-    ss = block_sum<NT>(ss, red);
-    const float inv = rsqrtf(ss / (float) d + a.eps);
+__device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, const jib_row_tail & a, float * red, bool dry) {
+    const int nv = d / 8;
     const bool conv = a.conv_w != nullptr;
     int slot = -1;
     bool past = false;
@@ -89,34 +93,80 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][4], int t, int d, co
         }
         past = slot >= 0 && a.positions[t] > 0;      // a sequence's first token starts from zeros, whatever the slot held
     }
+    const int n_old = a.taps - 1;
+    T * const state = (T *) a.conv_state + (size_t) (slot < 0 ? 0 : slot) * n_old * d;
+    Pack8<T> old[MAXV == 1 ? FAST_TAPS - 1 : 1];
+    const bool early = MAXV == 1 && conv && a.taps <= FAST_TAPS;
+    if (early) {
+#pragma unroll
+        for (int j = 0; j < (MAXV == 1 ? FAST_TAPS - 1 : 0); ++j) {
+            old[j].zero();
+            if (past && j < n_old && threadIdx.x < nv) old[j].load(state + (size_t) j * d + 8 * threadIdx.x);
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it) {
+        const int i = threadIdx.x + it * NT;
+        if (i < nv) {
+            Pack8<float> k;
+            k.set(v[it]);
+            if (!dry) k.store((float *) a.x_out + (size_t) t * d + 8 * i);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+        }
+    }
+    if (a.norm_w == nullptr) return;
+    ss = block_sum<NT>(ss, red);
+    const float inv = rsqrtf(ss / (float) d + a.eps);
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i >= nv) continue;
-        float w[4], h[4];
-        load4(a.norm_w + 4 * i, w);
+        float w[8], h[8];
+        load8(a.norm_w + 8 * i, w);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) h[e] = v[it][e] * inv * w[e];
-        if (!dry) store4((T *) a.h_out + (size_t) t * d + 4 * i, h);
+        for (int e = 0; e < 8; ++e) h[e] = v[it][e] * inv * w[e];
+        Pack8<T> hp;
+        hp.set(h);
+        if (!dry) hp.store((T *) a.h_out + (size_t) t * d + 8 * i);
         if (conv) {
-            round4(h, (const T *) nullptr);          // the convolution reads what a later step will read back from the state
-            float c[4], k[4];
-            load4(a.conv_w + (size_t) (a.taps - 1) * d + 4 * i, k);
+            hp.get(h);                               // the convolution reads what a later step will read back from the state
+            float c[8], k[8], s[8];
+            load8(a.conv_w + (size_t) n_old * d + 8 * i, k);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) c[e] = h[e] + k[e] * h[e];
-            T * st = (T *) a.conv_state + ((size_t) (slot < 0 ? 0 : slot) * (a.taps - 1)) * d + 4 * i;
-            for (int j = 0; j < a.taps - 1; ++j) {
-                float s[4] = {0.f, 0.f, 0.f, 0.f};
-                if (past) {
-                    load4(st + (size_t) j * d, s);
-                    load4(a.conv_w + (size_t) j * d + 4 * i, k);
+            for (int e = 0; e < 8; ++e) c[e] = h[e] + k[e] * h[e];
+            T * st = state + 8 * i;
+            if (early) {
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) c[e] += k[e] * s[e];
+                for (int j = 0; j < (MAXV == 1 ? FAST_TAPS - 1 : 0); ++j) {
+                    if (j >= n_old) continue;
+                    if (past) {
+                        load8(a.conv_w + (size_t) j * d + 8 * i, k);
+                        old[j].get(s);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) c[e] += k[e] * s[e];
+                    }
+                    if (slot >= 0 && !dry && j > 0) old[j].store(st + (size_t) (j - 1) * d);
                 }
-                if (slot >= 0 && !dry && j > 0) store4(st + (size_t) (j - 1) * d, s);
+            } else {
+                for (int j = 0; j < n_old; ++j) {
+                    Pack8<T> o;
+                    o.zero();
+                    if (past) {
+                        o.load(st + (size_t) j * d);
+                        load8(a.conv_w + (size_t) j * d + 8 * i, k);
+                        o.get(s);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) c[e] += k[e] * s[e];
+                    }
+                    if (slot >= 0 && !dry && j > 0) o.store(st + (size_t) (j - 1) * d);
+                }
             }
-            if (slot >= 0 && !dry && a.taps > 1) store4(st + (size_t) (a.taps - 2) * d, h);
-            if (!dry) store4((T *) a.hc_out + (size_t) t * d + 4 * i, c);
+            if (slot >= 0 && !dry && n_old > 0) hp.store(st + (size_t) (n_old - 1) * d);
+            Pack8<T> cp;
+            cp.set(c);
+            if (!dry) cp.store((T *) a.hc_out + (size_t) t * d + 8 * i);
         }
     }
 }
@@ -133,16 +183,16 @@ __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ t
         if (threadIdx.x == 0) jib_report(tail.status, JIB_ERR_BOUNDS, 40, id);
         id = id < 0 ? 0 : n_vocab - 1;
     }
-    const int nv = d / 4;
-    float v[MAXV][4];
+    const int nv = d / 8;
+    float v[MAXV][8];
     float ss = 0.f;
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i < nv) {
-            load4(table + (size_t) id * d + 4 * i, v[it]);
+            load8(table + (size_t) id * d + 8 * i, v[it]);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) ss += v[it][e] * v[it][e];
+            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
         }
     }
     ss = block_sum<NT>(ss, red);
@@ -151,10 +201,10 @@ __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ t
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i < nv) {
-            float k[4];
-            load4(w + 4 * i, k);
+            float k[8];
+            load8(w + 8 * i, k);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) v[it][e] *= inv * k[e];
+            for (int e = 0; e < 8; ++e) v[it][e] *= inv * k[e];
         }
     }
     finish_row<T, NT, MAXV>(v, t, d, tail, red, false);
@@ -173,51 +223,84 @@ struct UpdateArgs {
     float mult;
 };
 
+constexpr int MAX_TOP = 32;
+
 template <typename T, int NT, int MAXV>
-__device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_row_tail & tail, float * red, bool dry) {
-    const int t = blockIdx.x, d = a.d, nv = d / 4;
-    float v[MAXV][4];
+__device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, bool dry) {
+    const int t = blockIdx.x, d = a.d, nv = d / 8;
+    if (a.y != nullptr) {
+        if (threadIdx.x < a.k) {
+            const int r = dry ? 0 : a.dest[(size_t) t * a.k + threadIdx.x];
+            rows[threadIdx.x] = r < 0 ? 0 : r;
+            wts[threadIdx.x] = r < 0 ? 0.f : a.wts[(size_t) t * a.k + threadIdx.x];
+        }
+        __syncthreads();
+    }
+    float v[MAXV][8];
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i >= nv) continue;
-        float o[4], g[4], b[4], sum[4];
-        load4((const T *) a.o + (size_t) t * d + 4 * i, o);
-        load4((const T *) a.gates + (size_t) t * a.gate_stride + 4 * i, g);
-        load4(a.b1 + 4 * i, b);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) sum[e] = sigmoid(g[e] + b[e]) * o[e];
+        Pack8<float> xp, b1p, b2p;
+        Pack8<T> op, g1p, g2p;
+        xp.load(a.x + (size_t) t * d + 8 * i);       // everything the row needs is requested before any of it is used
+        op.load((const T *) a.o + (size_t) t * d + 8 * i);
+        g1p.load((const T *) a.gates + (size_t) t * a.gate_stride + 8 * i);
+        b1p.load(a.b1 + 8 * i);
+        float f[8], sum[8];
         if (a.y != nullptr) {
-            float f[4] = {0.f, 0.f, 0.f, 0.f};
-            for (int j = 0; j < a.k; ++j) {
-                const int row = dry ? 0 : a.dest[(size_t) t * a.k + j];
-                if (row < 0) continue;
-                const float w = a.wts[(size_t) t * a.k + j];
-                float y[4];
-                load4((const T *) a.y + (size_t) row * d + 4 * i, y);
+            g2p.load((const T *) a.gates + (size_t) t * a.gate_stride + d + 8 * i);
+            b2p.load(a.b2 + 8 * i);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) f[e] += w * y[e];
+            for (int e = 0; e < 8; ++e) f[e] = 0.f;
+            const T * y = (const T *) a.y + 8 * i;
+            int j = 0;
+            for (; j + 4 <= a.k; j += 4) {
+                Pack8<T> p[4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) p[u].load(y + (size_t) rows[j + u] * d);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    float q[8];
+                    p[u].get(q);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) f[e] += wts[j + u] * q[e];
+                }
             }
-            load4((const T *) a.gates + (size_t) t * a.gate_stride + d + 4 * i, g);
-            load4(a.b2 + 4 * i, b);
+            for (; j < a.k; ++j) {
+                float q[8];
+                load8(y + (size_t) rows[j] * d, q);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) sum[e] += sigmoid(g[e] + b[e]) * f[e];
+                for (int e = 0; e < 8; ++e) f[e] += wts[j] * q[e];
+            }
         }
-        float x[4];
-        load4(a.x + (size_t) t * d + 4 * i, x);
+        float o[8], g[8], b[8], x[8];
+        op.get(o); g1p.get(g); b1p.get(b); xp.get(x);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) v[it][e] = x[e] + a.mult * sum[e];
+        for (int e = 0; e < 8; ++e) sum[e] = sigmoid<T>(g[e] + b[e]) * o[e];
+        if (a.y != nullptr) {
+            g2p.get(g); b2p.get(b);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) sum[e] += sigmoid<T>(g[e] + b[e]) * f[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[it][e] = x[e] + a.mult * sum[e];
     }
     finish_row<T, NT, MAXV>(v, t, d, tail, red, dry);
 }
 
 template <typename T, int NT, int MAXV>
-__global__ void __launch_bounds__(NT) block_update_kernel(const UpdateArgs a, const jib_row_tail tail, int warm) {
+__global__ void __launch_bounds__(NT) block_update_kernel(const __grid_constant__ UpdateArgs a, const __grid_constant__ jib_row_tail tail, int warm) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
-    if (warm) block_update_row<T, NT, MAXV>(a, tail, red, true);
+    __shared__ int rows[MAX_TOP];
+    __shared__ float wts[MAX_TOP];
+    if (warm) {
+        block_update_row<T, NT, MAXV>(a, tail, red, rows, wts, true);
+        __syncthreads();
+    }
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    block_update_row<T, NT, MAXV>(a, tail, red, false);
+    block_update_row<T, NT, MAXV>(a, tail, red, rows, wts, false);
 }
 
 // out[i] = x[rows[i]] / rms * w
@@ -229,16 +312,16 @@ __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     int r = rows != nullptr ? rows[blockIdx.x] : (int) blockIdx.x;
     r = r < 0 ? 0 : (r >= n_src ? n_src - 1 : r);
-    const int nv = d / 4;
-    float v[MAXV][4];
+    const int nv = d / 8;
+    float v[MAXV][8];
     float ss = 0.f;
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i < nv) {
-            load4(x + (size_t) r * d + 4 * i, v[it]);
+            load8(x + (size_t) r * d + 8 * i, v[it]);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) ss += v[it][e] * v[it][e];
+            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
         }
     }
     ss = block_sum<NT>(ss, red);
@@ -247,11 +330,13 @@ __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i < nv) {
-            float k[4];
-            load4(w + 4 * i, k);
+            float k[8];
+            load8(w + 8 * i, k);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) v[it][e] *= inv * k[e];
-            store4(out + (size_t) blockIdx.x * d + 4 * i, v[it]);
+            for (int e = 0; e < 8; ++e) v[it][e] *= inv * k[e];
+            Pack8<T> o;
+            o.set(v[it]);
+            o.store(out + (size_t) blockIdx.x * d + 8 * i);
         }
     }
 }
@@ -259,7 +344,7 @@ __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
 inline bool tail_ok(const jib_row_tail * t, int d) {
-    if (t == nullptr || t->x_out == nullptr || d % 4 || d > 16384) return false;
+    if (t == nullptr || t->x_out == nullptr || d % 8 || d > 16384) return false;
     if (t->norm_w != nullptr && t->h_out == nullptr) return false;
     if (t->conv_w != nullptr)
         return t->norm_w != nullptr && t->hc_out != nullptr && t->taps >= 1 && (t->taps == 1 || t->conv_state != nullptr) &&
@@ -269,12 +354,14 @@ inline bool tail_ok(const jib_row_tail * t, int d) {
 
 }  // namespace
 
-// (threads, 4-element vectors per thread) by row width
+// (threads, 8-element vectors per thread) by row width
 #define JIB_ROW_DISPATCH(d, CALL)            \
-    if ((d) <= 1024) CALL(256, 1);           \
-    else if ((d) <= 2048) CALL(256, 2);      \
-    else if ((d) <= 8192) CALL(512, 4);      \
-    else CALL(512, 8)
+    if ((d) <= 1024) CALL(128, 1);           \
+    else if ((d) <= 2048) CALL(256, 1);      \
+    else if ((d) <= 4096) CALL(512, 1);      \
+    else if ((d) <= 5120) CALL(640, 1);      \
+    else if ((d) <= 8192) CALL(512, 2);      \
+    else CALL(512, 4)
 
 extern "C" {
 
@@ -297,7 +384,7 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
                                 const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
                                 const jib_row_tail * tail, void * stream) {
     if (T <= 0) return 0;
-    if (!tail_ok(tail, d) || gate_stride % 4 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1))) return JIB_E_ARG;
+    if (!tail_ok(tail, d) || gate_stride % 8 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1 || k > MAX_TOP))) return JIB_E_ARG;
     UpdateArgs a;
     a.x = x; a.o = o; a.gates = gates; a.b1 = b1; a.b2 = b2; a.y = y; a.dest = dest; a.wts = wts; a.gate_stride = gate_stride;
     a.k = k; a.d = d; a.mult = mult;
@@ -316,7 +403,7 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
 JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
                             void * stream) {
     if (n <= 0) return 0;
-    if (d % 4 || d > 16384 || n_src <= 0) return JIB_E_ARG;
+    if (d % 8 || d > 16384 || n_src <= 0) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
 #define CALL(NT, MAXV)                                                                                                       \
     do {                                                                                                                     \

@@ -45,16 +45,62 @@ __device__ __forceinline__ int find_seq(const int * q_start, int n_seqs, int t) 
 }
 
 // ---- out[t] = h[t] + sum_j w[j] * h[t - taps + 1 + j] --------------------------------------------------------------------
-// grid (T): one CTA per token.  The first taps - 1 tokens of a sequence's range read the stored rows, so one CTA (the first
-// token's) computes all of them and then, as the only reader, writes the stored rows of the range's end.
+// grid (ceil(T / CONV_RUN)): a CTA takes a run of tokens.  A run inside one sequence and past its first taps - 1 tokens loads every
+// row once and slides over them in registers.  The first taps - 1 tokens of a sequence's range read the stored rows, so one CTA
+// (the first token's) computes all of them and then, as the only reader, writes the stored rows of the range's end.
+constexpr int CONV_RUN = 4, CONV_TAPS = 4;
+
+template <typename T>
+__device__ __forceinline__ void causal_conv_token(const T * __restrict__ h, const float * __restrict__ w, int taps, T * __restrict__ state,
+                                                  int n_state, const int * __restrict__ seq_slots, const int * __restrict__ positions,
+                                                  const int * __restrict__ q_start, int n_seqs, int d, T * __restrict__ out, int * status,
+                                                  int t);
+
 template <typename T>
 __global__ void __launch_bounds__(256) causal_conv_kernel(const T * __restrict__ h, const float * __restrict__ w, int taps,
                                                           T * __restrict__ state, int n_state, const int * __restrict__ seq_slots,
                                                           const int * __restrict__ positions, const int * __restrict__ q_start, int n_seqs,
-                                                          int d, T * __restrict__ out, int * status) {
+                                                          int n_tok, int d, T * __restrict__ out, int * status) {
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int t = blockIdx.x;
+    const int t0 = blockIdx.x * CONV_RUN, t1 = min(n_tok, t0 + CONV_RUN);
+    const int b = find_seq(q_start, n_seqs, t0);
+    const bool inner = taps <= CONV_TAPS && t0 - q_start[b] >= taps - 1 && t0 + CONV_RUN <= q_start[b + 1];
+    if (!inner) {
+        for (int t = t0; t < t1; ++t)
+            causal_conv_token(h, w, taps, state, n_state, seq_slots, positions, q_start, n_seqs, d, out, status, t);
+        return;
+    }
+    const int n_old = taps - 1;
+    for (int v = threadIdx.x; v < d / 4; v += blockDim.x) {
+        const int ch = 4 * v;
+        float x[CONV_RUN + CONV_TAPS - 1][4], k[CONV_TAPS][4];        // rows t0 - CONV_TAPS + 1 .. ; taps, the last one in k[CONV_TAPS - 1]
+#pragma unroll
+        for (int r = 0; r < CONV_RUN + CONV_TAPS - 1; ++r)
+            if (r >= CONV_TAPS - 1 - n_old) load4(h + (size_t) (t0 + r - (CONV_TAPS - 1)) * d + ch, x[r]);
+#pragma unroll
+        for (int j = 0; j < CONV_TAPS; ++j)
+            if (j >= CONV_TAPS - taps) load4(w + (size_t) (j - (CONV_TAPS - taps)) * d + ch, k[j]);
+#pragma unroll
+        for (int r = 0; r < CONV_RUN; ++r) {
+            float c[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) c[e] = x[r + CONV_TAPS - 1][e] + k[CONV_TAPS - 1][e] * x[r + CONV_TAPS - 1][e];
+#pragma unroll
+            for (int j = 0; j < CONV_TAPS - 1; ++j)
+                if (j >= CONV_TAPS - taps)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) c[e] += k[j][e] * x[r + j][e];
+            store4(out + (size_t) (t0 + r) * d + ch, c);
+        }
+    }
+}
+
+template <typename T>
+__device__ __forceinline__ void causal_conv_token(const T * __restrict__ h, const float * __restrict__ w, int taps, T * __restrict__ state,
+                                                  int n_state, const int * __restrict__ seq_slots, const int * __restrict__ positions,
+                                                  const int * __restrict__ q_start, int n_seqs, int d, T * __restrict__ out, int * status,
+                                                  int t) {
     const int b = find_seq(q_start, n_seqs, t);
     const int q0 = q_start[b], n = q_start[b + 1] - q0, i = t - q0;
     if (i < 0 || i >= n || (i > 0 && i < taps - 1)) return;
@@ -104,13 +150,33 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const T * __restrict__
 
 // ---- minGRU: S_t = (1 - z_t) S_(t-1) + z_t c_t,  y_t = S_t * silu(g_t) -------------------------------------------------------
 // zxg [T][ld]: pre-activations of z, of the candidate and of the output gate, W columns each.  All arithmetic fp32.
-__device__ __forceinline__ void gru_terms(float az, float au, float & a, float & b) {
-    const float z = 1.f / (1.f + expf(-az));
-    const float c = au >= 0.f ? au + 0.5f : 1.f / (1.f + expf(-au));
+// (bf16 activations: fast exponential and division, a few ulp of fp32; fp32 ones: the accurate forms)
+template <typename T> __device__ __forceinline__ float sigmoid(float v);
+template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
+template <typename T> __device__ __forceinline__ void gru_terms(float az, float au, float & a, float & b) {
+    const float z = sigmoid<T>(az), c = sigmoid<T>(au);
     a = 1.f - z;
-    b = z * c;
+    b = z * (au >= 0.f ? au + 0.5f : c);
 }
-__device__ __forceinline__ float silu(float g) { return g / (1.f + expf(-g)); }
+template <typename T> __device__ __forceinline__ float silu(float g) { return g * sigmoid<T>(g); }
+// Two adjacent elements; pair: the address is a multiple of their size (else, or past the last channel, one by one).
+__device__ __forceinline__ float2 load2(const bf16 * p, bool pair, bool second) {
+    if (pair) return __bfloat1622float2(*(const __nv_bfloat162 *) p);
+    return make_float2(__bfloat162float(p[0]), second ? __bfloat162float(p[1]) : 0.f);
+}
+__device__ __forceinline__ float2 load2(const float * p, bool pair, bool second) {
+    if (pair) return *(const float2 *) p;
+    return make_float2(p[0], second ? p[1] : 0.f);
+}
+__device__ __forceinline__ void store2(bf16 * p, float a, float b, bool pair, bool second) {
+    if (pair) *(__nv_bfloat162 *) p = __floats2bfloat162_rn(a, b);
+    else { put(p, a); if (second) put(p + 1, b); }
+}
+__device__ __forceinline__ void store2(float * p, float a, float b, bool pair, bool second) {
+    if (pair) *(float2 *) p = make_float2(a, b);
+    else { put(p, a); if (second) put(p + 1, b); }
+}
 
 // One token per sequence (decode): grid (ceil(W / 256), T), row t belongs to sequence t.
 template <typename T>
@@ -130,10 +196,10 @@ __global__ void __launch_bounds__(256) mingru_step_kernel(const T * __restrict__
     const T * row = zxg + (size_t) t * ld;
     float * st = state + (size_t) (slot < 0 ? 0 : slot) * W + ch;
     float a, b;
-    gru_terms(to_f(row[ch]) + zb[ch], to_f(row[W + ch]) + xb[ch], a, b);
+    gru_terms<T>(to_f(row[ch]) + zb[ch], to_f(row[W + ch]) + xb[ch], a, b);
     const float s = (slot >= 0 && positions[t] > 0) ? a * *st + b : b;
     if (slot >= 0) *st = s;
-    put(y + (size_t) t * W + ch, s * silu(to_f(row[2 * W + ch])));
+    put(y + (size_t) t * W + ch, s * silu<T>(to_f(row[2 * W + ch])));
 }
 
 // Ranges of any length: grid (ceil(W / 16), n_seqs), 1024 threads = 8 channel pairs x 128 runs of SCAN_L tokens.  Every thread
@@ -164,23 +230,36 @@ __global__ void __launch_bounds__(1024) mingru_scan_kernel(const T * __restrict_
         carry[threadIdx.x] = (slot >= 0 && positions[q0] > 0 && c < W) ? state[(size_t) slot * W + c] : 0.f;
     }
     const bool in[2] = {ch < W, ch + 1 < W};
+    const bool pair = (W & 1) == 0 && (ld & 1) == 0 && (((uintptr_t) zxg | (uintptr_t) y) & (2 * sizeof(T) - 1)) == 0;
     const float bz[2] = {in[0] ? zb[ch] : 0.f, in[1] ? zb[ch + 1] : 0.f};
     const float bx[2] = {in[0] ? xb[ch] : 0.f, in[1] ? xb[ch + 1] : 0.f};
     __syncthreads();
     for (int t0 = 0; t0 < n; t0 += SCAN_L * SCAN_RUNS) {
-        float a[SCAN_L][2], v[SCAN_L][2], g[SCAN_L][2];
+        float a[SCAN_L][2], v[SCAN_L][2];
+        float2 g[SCAN_L];
         float A[2] = {1.f, 1.f}, B[2] = {0.f, 0.f};
 #pragma unroll
-        for (int l = 0; l < SCAN_L; ++l) {
+        for (int l = 0; l < SCAN_L; ++l) {                             // every load of the round first
             const int t = t0 + run * SCAN_L + l;
             const T * row = zxg + (size_t) (q0 + t) * ld + ch;
+            float2 az = make_float2(0.f, 0.f), au = az;
+            g[l] = az;
+            if (t < n && in[0]) {
+                az = load2(row, pair, in[1]);
+                au = load2(row + W, pair, in[1]);
+                g[l] = load2(row + 2 * W, pair, in[1]);
+            }
+            a[l][0] = az.x; a[l][1] = az.y; v[l][0] = au.x; v[l][1] = au.y;
+        }
+#pragma unroll
+        for (int l = 0; l < SCAN_L; ++l) {
+            const bool live = t0 + run * SCAN_L + l < n;
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                a[l][e] = 1.f; v[l][e] = 0.f; g[l][e] = 0.f;           // past the end: S passes through
-                if (t < n && in[e]) {
-                    gru_terms(to_f(row[e]) + bz[e], to_f(row[W + e]) + bx[e], a[l][e], v[l][e]);
-                    g[l][e] = to_f(row[2 * W + e]);
-                }
+                float ta, tv;
+                gru_terms<T>(a[l][e] + bz[e], v[l][e] + bx[e], ta, tv);
+                a[l][e] = live ? ta : 1.f;                              // past the end: S passes through
+                v[l][e] = live ? tv : 0.f;
                 B[e] = a[l][e] * B[e] + v[l][e];
                 A[e] *= a[l][e];
             }
@@ -217,14 +296,15 @@ __global__ void __launch_bounds__(1024) mingru_scan_kernel(const T * __restrict_
             if (lane == 31) carry[warp] = s_end;
         }
         __syncthreads();
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            float s = xa[e] * wa[2 * cp + e][warp] + xv[e];
+        {
+            float s0 = xa[0] * wa[2 * cp][warp] + xv[0], s1 = xa[1] * wa[2 * cp + 1][warp] + xv[1];
 #pragma unroll
             for (int l = 0; l < SCAN_L; ++l) {
                 const int t = t0 + run * SCAN_L + l;
-                s = a[l][e] * s + v[l][e];
-                if (t < n && in[e]) put(y + (size_t) (q0 + t) * W + ch + e, s * silu(g[l][e]));
+                s0 = a[l][0] * s0 + v[l][0];
+                s1 = a[l][1] * s1 + v[l][1];
+                if (t < n && in[0])
+                    store2(y + (size_t) (q0 + t) * W + ch, s0 * silu<T>(g[l].x), s1 * silu<T>(g[l].y), pair, in[1]);
             }
         }
         __syncthreads();                                                // wa / wb are rewritten in the next round
@@ -247,12 +327,13 @@ JIB_EXPORT int jib_causal_conv(const void * h, const float * w, int taps, void *
     if (T <= 0 || n_seqs <= 0) return 0;
     if (d % 4 || taps < 1 || (taps > 1 && state == nullptr)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
+    const int grid = (T + CONV_RUN - 1) / CONV_RUN;
     if (f32)
-        JIB_LAUNCH((causal_conv_kernel<float>), T, 256, 0, s, (const float *) h, w, taps, (float *) state, n_state, seq_slots, positions, q_start,
-                   n_seqs, d, (float *) out, status);
+        JIB_LAUNCH((causal_conv_kernel<float>), grid, 256, 0, s, (const float *) h, w, taps, (float *) state, n_state, seq_slots, positions,
+                   q_start, n_seqs, T, d, (float *) out, status);
     else
-        JIB_LAUNCH((causal_conv_kernel<bf16>), T, 256, 0, s, (const bf16 *) h, w, taps, (bf16 *) state, n_state, seq_slots, positions, q_start,
-                   n_seqs, d, (bf16 *) out, status);
+        JIB_LAUNCH((causal_conv_kernel<bf16>), grid, 256, 0, s, (const bf16 *) h, w, taps, (bf16 *) state, n_state, seq_slots, positions,
+                   q_start, n_seqs, T, d, (bf16 *) out, status);
     return launched();
 }
 

@@ -122,7 +122,7 @@ def test_padding_rows_leave_every_state_alone(dev, dtype):
 
 # ---- residual update, norms ------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dev,dtype", WHERE)
-@pytest.mark.parametrize("d", [24, 1028, 2056, 5128])
+@pytest.mark.parametrize("d", [24, 1032, 2056, 5128, 8200])
 @pytest.mark.parametrize("with_ff", [True, False])
 def test_block_update_gates_sum_and_norm(dev, dtype, d, with_ff):
     T, k = 5, 3
