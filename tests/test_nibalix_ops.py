@@ -83,15 +83,15 @@ def _gru_ref(zxg, zb, xb, s0=None):
 @pytest.mark.parametrize("dev,dtype", WHERE)
 @pytest.mark.parametrize("W", [16, 33, 200])
 def test_mingru_in_portions_equals_one_pass(dev, dtype, W):
-    """Portions around the scan's run and round lengths (4, 512), single tokens, two sequences, slots with old states; the state
+    """Portions around the scan's run, chunk and round lengths (4, 128, 1024), single tokens, two sequences, slots with old states; the state
     is slow to forget (gates near 0), so an error in the carry would stay."""
-    lens = (700, 61)
+    lens = (1300, 61)
     zxg = [rnd(n, 3 * W, seed=10 + i) for i, n in enumerate(lens)]
     zb, xb = rnd(W, seed=4) - 5.0, rnd(W, seed=5)
     want = [_gru_ref(x, zb, xb) for x in zxg]
     state = torch.full((4, W), -3.0, device=dev)
     at = [0, 0]
-    for cut in [(1, 3), (2, 0), (513, 4), (1, 1), (3, 50), (180, 3)]:
+    for cut in [(1, 3), (2, 0), (1027, 4), (1, 1), (129, 50), (128, 3), (12, 0)]:
         part = [(s, at[s], n) for s, n in enumerate(cut) if n]
         x = torch.cat([zxg[s][p:p + n] for s, p, n in part]).to(dev, dtype)
         pos = i32([p + k for _, p, n in part for k in range(n)], dev)
