@@ -79,10 +79,11 @@ template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.
 constexpr int FAST_TAPS = 4;         // up to this many taps the stored rows are requested before the row's reductions
 
 // x row -> residual store, norm, and (decode) the next block's input convolution.
-template <typename T, int NT, int MAXV>
+// CONV: the tail has the convolution (decode: registers for latency); else (prompts) occupancy matters.
+template <typename T, int NT, int MAXV, bool CONV>
 __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, const jib_row_tail & a, float * red, bool dry) {
     const int nv = d / 8;
-    const bool conv = a.conv_w != nullptr;
+    constexpr bool conv = CONV;
     int slot = -1;
     bool past = false;
     if (conv) {
@@ -95,11 +96,11 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
     }
     const int n_old = a.taps - 1;
     T * const state = (T *) a.conv_state + (size_t) (slot < 0 ? 0 : slot) * n_old * d;
-    Pack8<T> old[MAXV == 1 ? FAST_TAPS - 1 : 1];
+    Pack8<T> old[MAXV == 1 && CONV ? FAST_TAPS - 1 : 1];
     const bool early = MAXV == 1 && conv && a.taps <= FAST_TAPS;
     if (early) {
 #pragma unroll
-        for (int j = 0; j < (MAXV == 1 ? FAST_TAPS - 1 : 0); ++j) {
+        for (int j = 0; j < (MAXV == 1 && CONV ? FAST_TAPS - 1 : 0); ++j) {
             old[j].zero();
             if (past && j < n_old && threadIdx.x < nv) old[j].load(state + (size_t) j * d + 8 * threadIdx.x);
         }
@@ -139,7 +140,7 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
             T * st = state + 8 * i;
             if (early) {
 #pragma unroll
-                for (int j = 0; j < (MAXV == 1 ? FAST_TAPS - 1 : 0); ++j) {
+                for (int j = 0; j < (MAXV == 1 && CONV ? FAST_TAPS - 1 : 0); ++j) {
                     if (j >= n_old) continue;
                     if (past) {
                         load8(a.conv_w + (size_t) j * d + 8 * i, k);
@@ -171,7 +172,7 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
     }
 }
 
-template <typename T, int NT, int MAXV>
+template <typename T, int NT, int MAXV, bool CONV>
 __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ table, const int * __restrict__ ids, const float * __restrict__ w,
                                                         float eps, int d, int n_vocab, const jib_row_tail tail) {
     PDL_TRIGGER_TOP();
@@ -207,7 +208,7 @@ __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ t
             for (int e = 0; e < 8; ++e) v[it][e] *= inv * k[e];
         }
     }
-    finish_row<T, NT, MAXV>(v, t, d, tail, red, false);
+    finish_row<T, NT, MAXV, CONV>(v, t, d, tail, red, false);
 }
 
 struct UpdateArgs {
@@ -225,7 +226,7 @@ struct UpdateArgs {
 
 constexpr int MAX_TOP = 32;
 
-template <typename T, int NT, int MAXV>
+template <typename T, int NT, int MAXV, bool CONV>
 __device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, bool dry) {
     const int t = blockIdx.x, d = a.d, nv = d / 8;
     if (a.y != nullptr) {
@@ -286,21 +287,21 @@ __device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_ro
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[it][e] = x[e] + a.mult * sum[e];
     }
-    finish_row<T, NT, MAXV>(v, t, d, tail, red, dry);
+    finish_row<T, NT, MAXV, CONV>(v, t, d, tail, red, dry);
 }
 
-template <typename T, int NT, int MAXV>
-__global__ void __launch_bounds__(NT) block_update_kernel(const __grid_constant__ UpdateArgs a, const __grid_constant__ jib_row_tail tail, int warm) {
+template <typename T, int NT, int MAXV, bool CONV>
+__global__ void __launch_bounds__(NT, CONV || MAXV > 1 || sizeof(T) > 2 ? 1 : (1024 / NT > 1 ? 1024 / NT : 1)) block_update_kernel(const __grid_constant__ UpdateArgs a, const __grid_constant__ jib_row_tail tail, int warm) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
     __shared__ int rows[MAX_TOP];
     __shared__ float wts[MAX_TOP];
     if (warm) {
-        block_update_row<T, NT, MAXV>(a, tail, red, rows, wts, true);
+        block_update_row<T, NT, MAXV, CONV>(a, tail, red, rows, wts, true);
         __syncthreads();
     }
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    block_update_row<T, NT, MAXV>(a, tail, red, rows, wts, false);
+    block_update_row<T, NT, MAXV, CONV>(a, tail, red, rows, wts, false);
 }
 
 // out[i] = x[rows[i]] / rms * w
@@ -370,13 +371,21 @@ JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float *
     if (T <= 0) return 0;
     if (!tail_ok(tail, d)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
-#define CALL(NT, MAXV)                                                                                                             \
-    do {                                                                                                                           \
-        if (f32) JIB_LAUNCH((embed_norm_kernel<float, NT, MAXV>), T, NT, 0, s, (const float *) table, ids, w, eps, d, n_vocab, *tail); \
-        else JIB_LAUNCH((embed_norm_kernel<bf16, NT, MAXV>), T, NT, 0, s, (const bf16 *) table, ids, w, eps, d, n_vocab, *tail);       \
+#define EMBED(TT, NT, MAXV, CONV) \
+    JIB_LAUNCH((embed_norm_kernel<TT, NT, MAXV, CONV>), T, NT, 0, s, (const TT *) table, ids, w, eps, d, n_vocab, *tail)
+#define CALL(NT, MAXV)                                                    \
+    do {                                                                  \
+        if (tail->conv_w != nullptr) {                                    \
+            if (f32) EMBED(float, NT, MAXV, true);                        \
+            else EMBED(bf16, NT, MAXV, true);                             \
+        } else {                                                          \
+            if (f32) EMBED(float, NT, MAXV, false);                       \
+            else EMBED(bf16, NT, MAXV, false);                            \
+        }                                                                 \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
 #undef CALL
+#undef EMBED
     return launched();
 }
 
@@ -390,13 +399,20 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
     a.k = k; a.d = d; a.mult = mult;
     cudaStream_t s = (cudaStream_t) stream;
     const int warm = jib::warm_for(T);
-#define CALL(NT, MAXV)                                                                              \
-    do {                                                                                            \
-        if (f32) JIB_LAUNCH((block_update_kernel<float, NT, MAXV>), T, NT, 0, s, a, *tail, warm);   \
-        else JIB_LAUNCH((block_update_kernel<bf16, NT, MAXV>), T, NT, 0, s, a, *tail, warm);        \
+#define UPDATE(TT, NT, MAXV, CONV) JIB_LAUNCH((block_update_kernel<TT, NT, MAXV, CONV>), T, NT, 0, s, a, *tail, warm)
+#define CALL(NT, MAXV)                                                    \
+    do {                                                                  \
+        if (tail->conv_w != nullptr) {                                    \
+            if (f32) UPDATE(float, NT, MAXV, true);                       \
+            else UPDATE(bf16, NT, MAXV, true);                            \
+        } else {                                                          \
+            if (f32) UPDATE(float, NT, MAXV, false);                      \
+            else UPDATE(bf16, NT, MAXV, false);                           \
+        }                                                                 \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
 #undef CALL
+#undef UPDATE
     return launched();
 }
 
