@@ -64,7 +64,8 @@ def test_every_entry_point_is_exported():
                  "jib_moe_permute", "jib_moe_combine", "jib_rmsnorm", "jib_mla_qkv_post", "jib_embed_gather", "jib_argmax", "jib_topk",
                  "jib_kv_block_copy", "jib_gather_rows", "jib_allreduce_oneshot", "jib_allreduce_twoshot", "jib_ar_epoch_bump",
                  "jib_ep_plan", "jib_ep_push", "jib_ep_combine", "jib_symm_alloc", "jib_symm_open", "jib_allgather_rows",
-                 "jib_moe_permute_multi", "jib_moe_route_fused", "jib_moe_combine_norm", "jib_moe_combine_allreduce", "jib_sample_topk"):
+                 "jib_moe_permute_multi", "jib_moe_route_fused", "jib_moe_combine_norm", "jib_moe_combine_allreduce", "jib_sample_topk",
+                 "jib_gemm_simt", "jib_embed_norm", "jib_block_update", "jib_rms_rows", "jib_causal_conv", "jib_mingru"):
         assert hasattr(L, name), name
 
 
@@ -88,6 +89,8 @@ int main() {
     F(jib_gemm_desc, n_counters); F(jib_gemm_desc, T); F(jib_gemm_desc, splits); F(jib_gemm_desc, ar_site); F(jib_gemm_desc, ar);
     F(jib_gemm_desc, out_row_ptr); F(jib_gemm_desc, ag_flags); F(jib_gemm_desc, ag_epoch); F(jib_gemm_desc, ag_rows);
     F(jib_gemm_desc, ag_world); F(jib_gemm_desc, ar_rs_rows);
+    printf("jib_row_tail %zu\n", sizeof(jib_row_tail));
+    F(jib_row_tail, conv_w); F(jib_row_tail, status); F(jib_row_tail, eps); F(jib_row_tail, n_state);
     return 0;
 }
 """
@@ -98,7 +101,7 @@ def test_ctypes_structs_match_the_c_layouts(tmp_path):
     program prints the C sizes and offsets and they must equal the ctypes ones."""
     import os
     import subprocess
-    from jittorinfer_b200.ops.native import GemmDesc
+    from jittorinfer_b200.ops.native import GemmDesc, RowTail
     from jittorinfer_b200.parallel.comm import ArCtx
     from jittorinfer_b200.parallel.ep import EpCtx
     src = tmp_path / "abi.cu"
@@ -107,7 +110,7 @@ def test_ctypes_structs_match_the_c_layouts(tmp_path):
     subprocess.run([build.nvcc_path(), "-std=c++17", "-gencode", "arch=compute_100a,code=sm_100a", "-I", os.path.join(build.CSRC, "kernels"),
                     str(src), "-o", exe], check=True, capture_output=True)
     lines = subprocess.run([exe], check=True, capture_output=True, text=True).stdout.split("\n")
-    py = {"JibArCtx": ArCtx, "JibEpCtx": EpCtx, "jib_gemm_desc": GemmDesc}
+    py = {"JibArCtx": ArCtx, "JibEpCtx": EpCtx, "jib_gemm_desc": GemmDesc, "jib_row_tail": RowTail}
     checked = 0
     for line in filter(None, lines):
         name, val = line.split()

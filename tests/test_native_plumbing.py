@@ -22,19 +22,21 @@ def _stand_in(calls, fused_norm):
     def make(name):
         nsig = inspect.signature(getattr(native, name))
         rfn = getattr(ref, name)
-        n_ref = len(inspect.signature(rfn).parameters)
+        ref_params = list(inspect.signature(rfn).parameters)
 
         def f(*a, **k):
             ba = nsig.bind(*a, **k)                     # TypeError here = the front-end does not fit the native signature
             ba.apply_defaults()
             calls.append(name)
             vals = list(ba.arguments.values())
+            # by name where both sides use it (optional arguments differ in order), else by position
+            vals = [ba.arguments[p] if p in ba.arguments else vals[i] for i, p in enumerate(ref_params)]
             if name == "moe_gate" and ba.arguments.get("pre_norm") is not None:
                 w, eps = ba.arguments["pre_norm"]             # the router launch normalises its input rows itself
                 gn = ref.rmsnorm(vals[0], w, eps)[0]
-                ids, wts = rfn(gn, *vals[1:n_ref])
+                ids, wts = rfn(gn, *vals[1:])
                 return ids, wts, gn
-            out = rfn(*vals[:n_ref])
+            out = rfn(*vals)
             if name == "moe_ffn" and ba.arguments.get("norm") is not None:
                 w, eps = ba.arguments["norm"]
                 return out, ref.rmsnorm(out, w, eps)[0]
@@ -82,6 +84,27 @@ def test_model_calls_fit_the_native_signatures(monkeypatch, name, fused_norm):
             "sample_topk", "embed_gather"} <= used, sorted(used)
 
 
+def test_nibalix_calls_fit_the_native_signatures(monkeypatch):
+    from jittorinfer_b200.models import nibalix
+    hp = nibalix.preset("nibalix-tiny")
+    w = dict(nibalix.iter_random(hp, seed=0))
+    g = torch.Generator().manual_seed(1)
+    prompts = [torch.randint(0, hp.n_vocab, (n,), generator=g).tolist() for n in (9, 90)]
+
+    def run():
+        eng = LLMEngine(nibalix.NibalixModel(hp, w.items(), dtype=torch.bfloat16), EngineConfig(n_ctx=512, n_batch=32, n_parallel=2, n_ctx_slot=128))
+        return eng.generate(prompts, SamplingParams(temperature=0.0, ignore_eos=True), max_new_tokens=4)
+
+    want = run()
+    calls = []
+    fake, _ = _stand_in(calls, True)
+    monkeypatch.setattr(ops, "_native", fake)
+    monkeypatch.setattr(ops, "use_native", lambda t: True)
+    assert run() == want
+    assert {"embed_norm", "block_update", "rms_rows", "causal_conv", "mingru", "moe_gate", "moe_routed", "mla_qkv_post", "mla_attention",
+            "linear", "argmax"} <= set(calls), sorted(set(calls))
+
+
 def test_prompt_attention_form_is_chosen_by_what_would_be_expanded():
     """The per-head prompt attention expands the cached rows of every sequence of the step: it is taken for prompt chunks, not
     for small batches, other head sizes, or mixed steps whose rows are mostly the contexts of sequences that only decode."""
@@ -94,3 +117,7 @@ def test_prompt_attention_form_is_chosen_by_what_would_be_expanded():
     assert not ok(32, *dims, {"total_kv": 32, "n_q_tiles": 1})                                    # below the size that pays
     assert not ok(2048, 32, 16, 32, 64, 64, {"total_kv": 2048, "n_q_tiles": 16})                  # not the DeepSeek head sizes
     assert not ok(2048, *dims, None)
+    # with a window only the visible rows count: a chunk deep into a long prompt, decoding neighbours with long contexts
+    meta = {"total_kv": 64000 + 64 * 4000, "n_q_tiles": 80, "kv_decode": 64 * 4000, "q_lens": [2048] + [1] * 64, "s_lens": [64000] + [4000] * 64}
+    assert not ok(2112, *dims, meta, 4000) and ok(2112, *dims, meta, 30)
+    assert native.visible_total(meta, 30) == 2048 + 29 + 64 * 30 and native.visible_total(meta, 0) == meta["total_kv"]
