@@ -43,7 +43,7 @@ class ServerConfig:
     n_batch: int = 2048
     n_keep: int = 0
     n_parallel: int = 8
-    model: str = ""
+    model: str = ""                    # GGUF file, or a folder with config.json and safetensors (models/registry.py)
     model_alias: str = ""
     special: bool = False
     cont_batching: bool = True
