@@ -1,5 +1,5 @@
 // CUDA-core GEMM behind the same descriptor as gemm_tcgen05.cu: Y[b][t][n] = sum_k X[b][t][k] * W[b][n][k], optional second
-// weight (silu(X W^T) * (X W2^T)), optional residual, optional expert segments.
+// weight (act(X W^T) * (X W2^T)), optional residual, optional expert segments.
 //
 // Two uses: fp32 operands in true 32-bit arithmetic (the tensor cores have no such mode), and bf16 operands whose rows are
 // not 16-byte multiples, which TMA cannot address.  A plain 64 x 64 tile with 4 x 4 results per thread.
@@ -17,6 +17,10 @@ constexpr int TM = 64, TN = 64, TK = 16, NT = 256, PAD = 4;
 
 __device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float to_f(float v) { return v; }
+// act(z) = z * sigmoid(gate_arg(z)): 0.5 (1 + tanh(u)) is sigmoid(2 u)
+__device__ __forceinline__ float gate_arg(float z, int act) {
+    return act == JIB_ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+}
 
 template <typename T, bool DUAL>
 __global__ void __launch_bounds__(NT) gemm_simt_kernel(const jib_gemm_desc d) {
@@ -76,7 +80,7 @@ __global__ void __launch_bounds__(NT) gemm_simt_kernel(const jib_gemm_desc d) {
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             if (n >= d.N) continue;
-            float y = DUAL ? acc[i][j] / (1.f + expf(-acc[i][j])) * acu[i][j] : acc[i][j];
+            float y = DUAL ? acc[i][j] / (1.f + expf(-gate_arg(acc[i][j], d.act))) * acu[i][j] : acc[i][j];
             if (d.residual != nullptr) {
                 const long long ri = (long long) batch * d.res_batch_stride + row * d.ldr + n;
                 y += d.res_f32 ? ((const float *) d.residual)[ri] : to_f(((const bf16 *) d.residual)[ri]);

@@ -15,7 +15,7 @@
 //    fp32 partials to a scratch buffer; the last CTA to arrive (per-tile counter) reduces them and runs
 //    the epilogue, then resets the counter so the buffers need no clearing between launches;
 //  * DUAL mode keeps two accumulators (gate and up projections of the same tile) and stores
-//    silu(gate) * up — the gated-FFN epilogue — so the 2x wider intermediate never reaches HBM;
+//    act(gate) * up — the gated-FFN epilogue — so the 2x wider intermediate never reaches HBM;
 //  * grouped mode: blockIdx.z selects an expert; the token rows of that expert are a segment
 //    [seg[e], seg[e+1]) of an expert-sorted activation matrix; segment bounds are read on the device
 //    (no host sync, unlike aclnn_ops.cpp:2136-2146).
@@ -68,6 +68,7 @@ struct GemmArgs {
     int list_tiles;           // the list holds (token tile << 16 | expert) entries and gridDim.y is 1
     int pdl_flags;            // grouped pairs: bit 0 = release dependents after the own wait, bit 1 = segment table valid at start
     int w_evict_first;        // weight tiles are loaded with the L2 evict_first policy (each is read once: small batches)
+    int act;                  // of a gated pair (JIB_ACT_*)
     int vec_store;            // bf16 result rows are written as 16-byte vectors through a shared-memory transpose
     const int * src_token;    // grouped, decode batches: x holds the T token rows unsorted, every expert multiplies all of
                               // them (one token tile) and sorted row i of the result is accumulator column src_token[i]
@@ -144,7 +145,11 @@ __device__ __forceinline__ uint2 pack_bf16x4(float4 v) {
     return o;
 }
 
-__device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
+// act(z) = z * sigmoid(z), or for the tanh form of gelu z * sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)): 0.5 (1 + tanh(u)) = sigmoid(2 u)
+__device__ __forceinline__ float gated(float x, int act) {
+    const float z = act == JIB_ACT_GELU_TANH ? 1.5957691216057308f * (x + 0.044715f * x * x * x) : x;
+    return x / (1.0f + __expf(-z));
+}
 
 // Cluster-wide barrier (all threads of all CTAs of the cluster) and a load from a peer CTA's shared memory.
 __device__ __forceinline__ void cluster_sync_all() {
@@ -380,7 +385,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         }
         // One finished element: feature n of row (row_base + t_rel); gv / uv are the summed accumulators.
         auto finish = [&](int t_rel, float gv, float uv) {
-            float y = DUAL ? silu(gv) * uv : gv;
+            float y = DUAL ? gated(gv, args.act) * uv : gv;
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
@@ -557,7 +562,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     const int ltid = (int) threadIdx.x - 64;
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? silu(g[j]) * u[j] : g[j];
+                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : g[j];
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -846,7 +851,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
-                    sb[k * BM + r] = DUAL ? silu(g) * __uint_as_float(uv[k]) : g;
+                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : g;
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
@@ -1139,6 +1144,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream_)
     if (a.ag_flags != nullptr && (a.ag_epoch == nullptr || a.ag_rows <= 0 || a.ag_world <= 0 || grouped || batch != 1)) return JIB_E_ARG;
     if (a.ar_rs_rows < 0) return JIB_E_ARG;
     if (a.row_ptr != nullptr && (dual || d->out_f32 || d->residual != nullptr || d->ar != nullptr)) return JIB_E_ARG;
+    a.act = d->act;
     memset(&a.ar, 0, sizeof(a.ar));
     if (d->ar != nullptr) {
         const JibArCtx * ar = (const JibArCtx *) d->ar;
@@ -1312,6 +1318,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16_noalloc(const void * x, const void * w, 
     a.expert_list = nullptr;
     a.list_tiles = 0;
     a.ag_flags = nullptr; a.ag_epoch = nullptr; a.ag_rows = 0; a.ag_world = 0; a.ar_rs_rows = 0; a.ag_spin_limit = 0;
+    a.act = JIB_ACT_SILU;
     memset(&a.ar, 0, sizeof(a.ar));
     dim3 grid(p.n_tiles, 1, p.splits);
     switch (p.bn) {

@@ -15,12 +15,15 @@ enum {
     JIB_E_SCRATCH = -6,     // scratch / counter buffer too small for the requested split
 };
 
+// Activation of a gated pair: z * sigmoid(z), or 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
+enum { JIB_ACT_SILU = 0, JIB_ACT_GELU_TANH = 1 };
+
 #ifdef __cplusplus
 extern "C" {
 #endif
 
 // Y[b][t][n] = sum_k X[b][t][k] * W[b][n][k]  (bf16 in, fp32 accumulate), optional second weight
-// (w2: out = silu(X W^T) * (X W2^T)), optional residual add, optional expert-grouped rows.
+// (w2: out = act(X W^T) * (X W2^T), act = silu or the tanh form of gelu), optional residual add, optional expert-grouped rows.
 typedef struct jib_gemm_desc {
     const void * x;            // bf16 activations
     const void * w;            // bf16 weights [batch][N][K]
@@ -63,6 +66,7 @@ typedef struct jib_gemm_desc {
     int pdl_flags;             // grouped, two launches back to back over one segment table: 1 on the first (it lets its dependents
                                //   start only once the table is known to be complete), 2 on the second (it may read the table and
                                //   request weights before the first launch has finished); 0 otherwise
+    int act;                   // with w2: JIB_ACT_*
 } jib_gemm_desc;
 
 JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream);
@@ -167,8 +171,12 @@ typedef struct jib_row_tail {
     float eps;
     int taps, n_state;
 } jib_row_tail;
-JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, int T, int d, int n_vocab, int f32,
+// x_out = scale * table[ids[t]], RMS-normed and times w unless w is null.
+JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, float scale, int T, int d, int n_vocab, int f32,
                               const jib_row_tail * tail, void * stream);
+// x_out = x + y / rms(y) * w (y [T][d] in the activation type); x_out may be x.
+JIB_EXPORT int jib_post_norm(const float * x, const void * y, const float * w, float eps, int T, int d, int f32, const jib_row_tail * tail,
+                             void * stream);
 // x_out = x + mult * (sigmoid(gates[:, :d] + b1) * o + sigmoid(gates[:, d:2d] + b2) * sum_j wts[t][j] * y[dest[t][j]]); y NULL: no second
 // sublayer.  x_out may be x.
 JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, const void * gates, long long gate_stride, const float * b1,
@@ -184,6 +192,53 @@ JIB_EXPORT int jib_causal_conv(const void * h, const float * w, int taps, void *
 JIB_EXPORT int jib_mingru(const void * zxg, long long ld, const float * zb, const float * xb, float * state, int n_state,
                           const int * seq_slots, const int * positions, const int * q_start, int n_seqs, int T, int W, int single, int f32,
                           void * y, int * status, void * stream);
+
+// ---- grouped-query attention over paged key / value rows (gqa_attention.cu) ------------------------------------------------
+typedef struct jib_gqa {
+    void * cache;              // [n_slots][row]: G * D key columns, then G * V value columns (activation type)
+    const int * block_tables;  // [n_seqs][max_blocks]
+    const int * seq_lens, * q_start, * positions;
+    int * status;
+    long long n_slots, row;
+    int H, G, D, V, rot, block_size, max_blocks, n_seqs, T, max_pos;
+    int window, chunk;         // position i sees j <= i with i - j < window (0: no window) and j / chunk == i / chunk (0: no chunks)
+    int sink;                  // 1: the softmax' denominator also holds exp(0)
+    float scale, softcap;      // softcap 0: none
+    float eps, out_scale;
+} jib_gqa;
+// q, k, v: columns of the projection (row stride ld).  rope [max_pos][rot / 2] pairs (cos, sin); pairs are (i, i + rot / 2).
+JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * k, const void * v, long long ld, const float * q_norm,
+                                const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int f32, void * stream);
+// q [T][H][D]; gate null or [T][ld_gate] pre-activations of one sigmoid per head; out [T][ldo].  single: one token per sequence.
+// splits (<= 8): CTAs that share a row's keys.
+JIB_EXPORT int jib_gqa_attention(const jib_gqa * m, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single,
+                                 int splits, int f32, void * stream);
+
+// ---- mixers with a matrix state per head (state_mix.cu) ----------------------------------------------------------------------
+enum { JIB_STATE_DELTA = 0, JIB_STATE_LINEAR = 1, JIB_STATE_SSD = 2 };
+typedef struct jib_state_mix {
+    // activations (bf16 or fp32): proj [T][ld] holds q (H / rep heads x K), k, v (H x V) and the pre-activation of the per-head
+    // factor (s_off; H columns; not LINEAR) at these columns; dec_in [T][ld_dec] the decays' (H x K; not SSD); gate [T][ld_gate] H x V
+    const void * proj, * dec_in, * gate;
+    void * y;                  // [T][ldy] result, H x V columns
+    // per-sequence state: [n_state][taps][n_conv] ring of convolution inputs (activation type), [n_state][H][K][V] fp32
+    void * conv_state;
+    float * state;
+    const float * conv_w;      // [taps][n_conv]: columns conv0 .. conv0 + n_conv of proj are convolved (taps 0: none), last tap = current
+    const float * conv_b;      // [n_conv] or null
+    const float * bias;        // decays' (H x K) or SSD's factor's (H)
+    const float * neg_a;       // [H], not LINEAR
+    const float * skip;        // [H], SSD
+    const float * norm_w;      // [V], SSD [H x V]
+    const int * seq_slots, * positions, * q_start;
+    int * status;
+    float * qk, * v, * dec, * s, * o;      // scratch: [T][2][H / rep][K], [T][H][V], [T][H][K] (SSD [T][H]), [T][H], [T][H][V]
+    long long ld, ld_dec, ld_gate, ldy;
+    int kind, H, K, V, rep, taps, conv0, n_conv, q_off, k_off, v_off, s_off, norm_groups, n_state, n_seqs, T;
+    float q_scale, inv_tau, eps, out_scale;
+} jib_state_mix;
+// single: one token per sequence (row t = sequence t; scratch only for SSD: o).  K <= 512.
+JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, void * stream);
 
 // ---- expert-parallel all-to-all over peer memory (ep_alltoall.cu); ctx is a JibEpCtx (ep_alltoall.h) ---------
 JIB_EXPORT int jib_ep_plan(const int * ids, int T, int k, const struct JibEpCtx * ctx, int site, int * seg, int * pair_dst, void * stream);

@@ -1,9 +1,11 @@
-// Row kernels of blocks with an fp32 residual stream whose sublayers run side by side on one norm:
+// Row kernels of blocks with an fp32 residual stream.
 //
-//   h = norm(x);   x <- x + m * (sigmoid(g1) * mixer(h) + sigmoid(g2) * ff(h))
+// Sublayers side by side on one norm:        h = norm(x);   x <- x + m * (sigmoid(g1) * mixer(h) + sigmoid(g2) * ff(h))
+// Sublayers in turn between two norms each:  x <- x + norm'(f(norm(x)))
 //
-//   embed_norm     x = norm(embedding row), then the first block's norm
-//   block_update   the sum above -- the expert-weighted combine of the feed-forward included -- then the next block's norm
+//   embed_norm     x = scale * embedding row, normed or not, then the first block's norm
+//   block_update   the first form's sum -- the expert-weighted combine of the feed-forward included -- then the next block's norm
+//   post_norm      the second form's sum with the norm of the sublayer's output, then the next sublayer's norm
 //   rms_rows       norm of selected rows (before the output head)
 //
 // One CTA owns one token's row and keeps it in registers, so the sum, the residual store and the norm that follows are one
@@ -174,7 +176,7 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
 
 template <typename T, int NT, int MAXV, bool CONV>
 __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ table, const int * __restrict__ ids, const float * __restrict__ w,
-                                                        float eps, int d, int n_vocab, const jib_row_tail tail) {
+                                                        float eps, float scale, int d, int n_vocab, const jib_row_tail tail) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
@@ -193,19 +195,24 @@ __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ t
         if (i < nv) {
             load8(table + (size_t) id * d + 8 * i, v[it]);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+            for (int e = 0; e < 8; ++e) {
+                v[it][e] *= scale;
+                ss += v[it][e] * v[it][e];
+            }
         }
     }
-    ss = block_sum<NT>(ss, red);
-    const float inv = rsqrtf(ss / (float) d + eps);
+    if (w != nullptr) {
+        ss = block_sum<NT>(ss, red);
+        const float inv = rsqrtf(ss / (float) d + eps);
 #pragma unroll
-    for (int it = 0; it < MAXV; ++it) {
-        const int i = threadIdx.x + it * NT;
-        if (i < nv) {
-            float k[8];
-            load8(w + 8 * i, k);
+        for (int it = 0; it < MAXV; ++it) {
+            const int i = threadIdx.x + it * NT;
+            if (i < nv) {
+                float k[8];
+                load8(w + 8 * i, k);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v[it][e] *= inv * k[e];
+                for (int e = 0; e < 8; ++e) v[it][e] *= inv * k[e];
+            }
         }
     }
     finish_row<T, NT, MAXV, CONV>(v, t, d, tail, red, false);
@@ -304,6 +311,122 @@ __global__ void __launch_bounds__(NT, CONV || MAXV > 1 || sizeof(T) > 2 ? 1 : (1
     block_update_row<T, NT, MAXV, CONV>(a, tail, red, rows, wts, false);
 }
 
+// x_out = x + y / rms(y) * w, then the tail's norm of it
+template <typename T, int NT, int MAXV>
+__device__ __noinline__ void post_norm_row(const float * x, const T * y, const float * w, float eps, int d, const jib_row_tail & tail, float * red,
+                                           bool dry) {
+    const int t = blockIdx.x, nv = d / 8;
+    float v[MAXV][8];
+    Pack8<float> xp[MAXV], wp[MAXV];
+    float ss = 0.f;
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it) {
+        const int i = threadIdx.x + it * NT;
+        if (i >= nv) continue;
+        Pack8<T> yp;
+        yp.load(y + (size_t) t * d + 8 * i);             // everything the row needs is requested before any of it is used
+        xp[it].load(x + (size_t) t * d + 8 * i);
+        wp[it].load(w + 8 * i);
+        yp.get(v[it]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+    }
+    ss = block_sum<NT>(ss, red);
+    const float inv = rsqrtf(ss / (float) d + eps);
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it) {
+        if (threadIdx.x + it * NT >= nv) continue;
+        float k[8], r[8];
+        xp[it].get(r);
+        wp[it].get(k);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[it][e] = r[e] + v[it][e] * inv * k[e];
+    }
+    finish_row<T, NT, MAXV, false>(v, t, d, tail, red, dry);
+}
+
+template <typename T, int NT, int MAXV>
+__global__ void __launch_bounds__(NT) post_norm_kernel(const float * x, const T * __restrict__ y, const float * __restrict__ w, float eps, int d,
+                                                       const __grid_constant__ jib_row_tail tail, int warm) {
+    PDL_TRIGGER_TOP();
+    __shared__ float red[32];
+    if (warm) {
+        post_norm_row<T, NT, MAXV>(x, y, w, eps, d, tail, red, true);
+        __syncthreads();
+    }
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    post_norm_row<T, NT, MAXV>(x, y, w, eps, d, tail, red, false);
+}
+
+// The three row kernels for widths that 8-element vectors do not divide: element by element, the row re-read from memory.
+//   ids:  v = scale * src[ids[t]], normed by w if given         (src: T table of n_src rows)
+//   y:    v = x[t] + y / rms(y) * w
+//   else: v = x[rows[t]] (rows null: x[t])                      (x has n_src rows)
+struct AnyRow {
+    const void * src;
+    const int * ids;
+    const float * x;
+    const void * y;
+    const int * rows;
+    const float * w;
+    float eps, scale;
+    int d, n_src;
+};
+template <typename T> __device__ __forceinline__ float as_f(const void * p, size_t i);
+template <> __device__ __forceinline__ float as_f<bf16>(const void * p, size_t i) { return __bfloat162float(((const bf16 *) p)[i]); }
+template <> __device__ __forceinline__ float as_f<float>(const void * p, size_t i) { return ((const float *) p)[i]; }
+__device__ __forceinline__ void put_f(bf16 * p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void put_f(float * p, float v) { *p = v; }
+
+template <typename T>
+__global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_row_tail tail) {
+    PDL_TRIGGER_TOP();
+    __shared__ float red[32];
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int t = blockIdx.x, d = a.d;
+    size_t row = t;
+    if (a.ids != nullptr || a.rows != nullptr) {
+        int r = a.ids != nullptr ? a.ids[t] : a.rows[t];
+        if (r < 0 || r >= a.n_src) {
+            if (threadIdx.x == 0 && a.ids != nullptr) jib_report(tail.status, JIB_ERR_BOUNDS, 40, r);
+            r = r < 0 ? 0 : a.n_src - 1;
+        }
+        row = r;
+    }
+    const void * normed = a.ids != nullptr ? a.src : a.y;        // the operand that w belongs to
+    float inv = 1.f;
+    if (normed != nullptr && a.w != nullptr) {
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < d; i += 256) {
+            const float v = a.scale * as_f<T>(normed, row * d + i);
+            ss += v * v;
+        }
+        inv = rsqrtf(block_sum<256>(ss, red) / (float) d + a.eps);
+    }
+    auto value = [&](int i) {
+        float v = 0.f;
+        if (normed != nullptr) {
+            v = a.scale * as_f<T>(normed, row * d + i);
+            if (a.w != nullptr) v *= inv * a.w[i];
+        }
+        return a.x != nullptr ? v + a.x[row * d + i] : v;
+    };
+    float * xo = (float *) tail.x_out;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += 256) {
+        const float v = value(i);
+        ss += v * v;
+        if (tail.norm_w == nullptr && xo != nullptr) xo[(size_t) t * d + i] = v;
+    }
+    if (tail.norm_w == nullptr) return;
+    const float ni = rsqrtf(block_sum<256>(ss, red) / (float) d + tail.eps);
+    for (int i = threadIdx.x; i < d; i += 256) {
+        const float v = value(i);
+        put_f((T *) tail.h_out + (size_t) t * d + i, v * ni * tail.norm_w[i]);
+        if (xo != nullptr) xo[(size_t) t * d + i] = v;            // last: x_out may be x
+    }
+}
+
 // out[i] = x[rows[i]] / rms * w
 template <typename T, int NT, int MAXV>
 __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__ x, const int * __restrict__ rows, const float * __restrict__ w,
@@ -345,7 +468,8 @@ __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
 inline bool tail_ok(const jib_row_tail * t, int d) {
-    if (t == nullptr || t->x_out == nullptr || d % 8 || d > 16384) return false;
+    if (t == nullptr || t->x_out == nullptr || d > 16384) return false;
+    if (d % 8) return t->conv_w == nullptr && (t->norm_w == nullptr || t->h_out != nullptr);      // the element-wise kernel
     if (t->norm_w != nullptr && t->h_out == nullptr) return false;
     if (t->conv_w != nullptr)
         return t->norm_w != nullptr && t->hc_out != nullptr && t->taps >= 1 && (t->taps == 1 || t->conv_state != nullptr) &&
@@ -366,13 +490,24 @@ inline bool tail_ok(const jib_row_tail * t, int d) {
 
 extern "C" {
 
-JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, int T, int d, int n_vocab, int f32,
+static int launch_any(const AnyRow & a, const jib_row_tail & tail, int n, int f32, cudaStream_t s) {
+    if (f32) JIB_LAUNCH((any_row_kernel<float>), n, 256, 0, s, a, tail);
+    else JIB_LAUNCH((any_row_kernel<bf16>), n, 256, 0, s, a, tail);
+    return launched();
+}
+
+JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, float scale, int T, int d, int n_vocab, int f32,
                               const jib_row_tail * tail, void * stream) {
     if (T <= 0) return 0;
     if (!tail_ok(tail, d)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
+    if (d % 8) {
+        AnyRow a = {};
+        a.src = table; a.ids = ids; a.w = w; a.eps = eps; a.scale = scale; a.d = d; a.n_src = n_vocab;
+        return launch_any(a, *tail, T, f32, s);
+    }
 #define EMBED(TT, NT, MAXV, CONV) \
-    JIB_LAUNCH((embed_norm_kernel<TT, NT, MAXV, CONV>), T, NT, 0, s, (const TT *) table, ids, w, eps, d, n_vocab, *tail)
+    JIB_LAUNCH((embed_norm_kernel<TT, NT, MAXV, CONV>), T, NT, 0, s, (const TT *) table, ids, w, eps, scale, d, n_vocab, *tail)
 #define CALL(NT, MAXV)                                                    \
     do {                                                                  \
         if (tail->conv_w != nullptr) {                                    \
@@ -393,7 +528,7 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
                                 const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
                                 const jib_row_tail * tail, void * stream) {
     if (T <= 0) return 0;
-    if (!tail_ok(tail, d) || gate_stride % 8 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1 || k > MAX_TOP))) return JIB_E_ARG;
+    if (!tail_ok(tail, d) || d % 8 || gate_stride % 8 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1 || k > MAX_TOP))) return JIB_E_ARG;
     UpdateArgs a;
     a.x = x; a.o = o; a.gates = gates; a.b1 = b1; a.b2 = b2; a.y = y; a.dest = dest; a.wts = wts; a.gate_stride = gate_stride;
     a.k = k; a.d = d; a.mult = mult;
@@ -416,11 +551,39 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
     return launched();
 }
 
+JIB_EXPORT int jib_post_norm(const float * x, const void * y, const float * w, float eps, int T, int d, int f32, const jib_row_tail * tail,
+                             void * stream) {
+    if (T <= 0) return 0;
+    if (!tail_ok(tail, d) || tail->conv_w != nullptr || w == nullptr) return JIB_E_ARG;
+    cudaStream_t s = (cudaStream_t) stream;
+    if (d % 8) {
+        AnyRow a = {};
+        a.x = x; a.y = y; a.w = w; a.eps = eps; a.scale = 1.f; a.d = d; a.n_src = T;
+        return launch_any(a, *tail, T, f32, s);
+    }
+    const int warm = jib::warm_for(T);
+#define CALL(NT, MAXV)                                                                                                          \
+    do {                                                                                                                        \
+        if (f32) JIB_LAUNCH((post_norm_kernel<float, NT, MAXV>), T, NT, 0, s, x, (const float *) y, w, eps, d, *tail, warm);    \
+        else JIB_LAUNCH((post_norm_kernel<bf16, NT, MAXV>), T, NT, 0, s, x, (const bf16 *) y, w, eps, d, *tail, warm);          \
+    } while (0)
+    JIB_ROW_DISPATCH(d, CALL);
+#undef CALL
+    return launched();
+}
+
 JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
                             void * stream) {
     if (n <= 0) return 0;
-    if (d % 8 || d > 16384 || n_src <= 0) return JIB_E_ARG;
+    if (d > 16384 || n_src <= 0) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
+    if (d % 8) {
+        AnyRow a = {};
+        jib_row_tail t = {};
+        a.x = x; a.rows = rows; a.d = d; a.n_src = n_src; a.scale = 1.f;
+        t.norm_w = w; t.eps = eps; t.h_out = out;
+        return launch_any(a, t, n, f32, s);
+    }
 #define CALL(NT, MAXV)                                                                                                       \
     do {                                                                                                                     \
         if (f32) JIB_LAUNCH((rms_rows_kernel<float, NT, MAXV>), n, NT, 0, s, x, rows, w, eps, d, n_src, (float *) out);      \

@@ -1,0 +1,586 @@
+// Token mixers with a matrix state per head: S [K key channels][V value channels], fp32, one per sequence slot and head.
+//
+//   S <- diag(decay_t) S;   u = s_t (v_t - [delta] S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t + D v_t
+//
+// in three kinds that differ in where q, k, v, the decay and the factor s come from:
+//   DELTA   q, k unit vectors, one decay per (head, key channel) = exp(-a_h softplus(. + bias)), s = sigmoid(.), the delta term
+//   LINEAR  one decay per (head, key channel) = sigmoid(. + bias)^(1/tau), s = 1
+//   SSD     one decay per head = exp(-a_h s), s = softplus(. + bias); q and k shared by a group of heads
+// A window of the projection's columns may pass a short causal convolution and silu first (DELTA: q, k, v; SSD: v, k, q).
+// What follows the read-out: DELTA / LINEAR a norm over each head's V channels times a gate; SSD a gate, then a norm over
+// parts of the row.
+//
+// Single tokens (decode): state_step does all of it in one launch per layer (SSD: plus the gated norm of whole rows).
+// Portions: state_prep (convolution, unit norm, decays -> fp32), state_scan (the recurrence), state_finish (gate and norm).
+//
+// A sequence's state lives in row seq_slots[b] of [n_state][H][K][V]; its last convolution inputs in a ring [n_state][taps][channels]
+// whose row p % taps holds position p's.  A range that starts at position 0 starts from zeros whatever the rows hold, so slots are
+// handed on without clearing.  Sequence b owns token rows q_start[b] .. q_start[b + 1].  Activations bf16 or fp32, the rest fp32.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "jib_kernels.h"
+#include "pdl.cuh"
+#include "sm100.cuh"
+
+namespace {
+
+typedef __nv_bfloat16 bf16;
+enum { DELTA = JIB_STATE_DELTA, LINEAR = JIB_STATE_LINEAR, SSD = JIB_STATE_SSD };
+
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ void put(bf16 * p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void put(float * p, float v) { *p = v; }
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+// bf16 activations: fast exponential and division for gates and silu (a few ulp of fp32); fp32 ones: the accurate forms.
+template <typename T> __device__ __forceinline__ float sigmoid(float v);
+template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
+template <typename T> __device__ __forceinline__ float silu(float v) { return v * sigmoid<T>(v); }
+__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+template <int KIND> __device__ __forceinline__ float channel_decay(const jib_state_mix & a, float z, int h) {
+    return KIND == DELTA ? expf(a.neg_a[h] * softplus(z)) : expf(-a.inv_tau * softplus(-z));
+}
+template <int KIND> __device__ __forceinline__ float head_factor(const jib_state_mix & a, float z, int h) {
+    return KIND == DELTA ? 1.f / (1.f + expf(-z)) : softplus(z + a.bias[h]);
+}
+
+__device__ __forceinline__ int seq_of(const int * q_start, int n_seqs, int t) {
+    int b = 0, hi = n_seqs;
+    while (hi - b > 1) {
+        const int mid = (b + hi) >> 1;
+        if (q_start[mid] <= t) b = mid; else hi = mid;
+    }
+    return b;
+}
+__device__ __forceinline__ int checked_slot(const jib_state_mix & a, int b, int site) {
+    const int slot = a.seq_slots[b];
+    if (slot >= a.n_state) {
+        if (threadIdx.x == 0) jib_report(a.status, JIB_ERR_BOUNDS, site, slot);
+        return -1;
+    }
+    return slot;
+}
+
+// Column c of token row t (position p, back rows of its range precede it in the batch): convolved and silu'd if c lies in the window.
+template <typename T>
+__device__ __forceinline__ float column(const jib_state_mix & a, int t, int c, int p, int back, int slot) {
+    const T * x = (const T *) a.proj + (size_t) t * a.ld + c;
+    if (a.taps == 0) return to_f(*x);
+    const int w = c - a.conv0;
+    float acc = a.conv_b != nullptr ? a.conv_b[w] : 0.f;
+    for (int j = 0; j < a.taps; ++j) {
+        const int d = a.taps - 1 - j;                        // tokens back
+        if (d > p) continue;
+        float v;
+        if (d <= back) v = to_f(x[-(long long) d * a.ld]);
+        else if (slot >= 0) v = to_f(((const T *) a.conv_state)[((size_t) slot * a.taps + (p - d) % a.taps) * a.n_conv + w]);
+        else continue;
+        acc += a.conv_w[(size_t) j * a.n_conv + w] * v;
+    }
+    return silu<T>(acc);
+}
+
+// ---- portions: inputs of the recurrence in fp32 ------------------------------------------------------------------------------
+// qk [T][2][Hk][K], v [T][H][V], dec [T][H][K] (SSD: [T][H]), s [T][H].  One warp per (token, item); items: q heads, k heads,
+// value heads, then one for the per-head factors and (DELTA, LINEAR) one per head's decays.
+constexpr int PREP_C = 16;                                   // channels of a q / k head per lane: K <= 32 * PREP_C
+
+template <typename T, int KIND>
+__global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__ jib_state_mix a) {
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int lane = threadIdx.x & 31, t = blockIdx.y;
+    const int Hk = a.H / a.rep;
+    int item = blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int b = seq_of(a.q_start, a.n_seqs, t), back = t - a.q_start[b], p = a.positions[t];
+    const int slot = a.taps > 0 ? checked_slot(a, b, 45) : -1;
+    if (item < 2 * Hk) {
+        const bool is_q = item < Hk;
+        const int c0 = (is_q ? a.q_off : a.k_off) + (is_q ? item : item - Hk) * a.K;
+        float v[PREP_C], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < PREP_C; ++i) {
+            const int c = lane + 32 * i;
+            v[i] = 0.f;
+            if (c < a.K) v[i] = column<T>(a, t, c0 + c, p, back, slot);
+            if (KIND == DELTA) ss += v[i] * v[i];
+        }
+        float scale = is_q ? a.q_scale : 1.f;
+        if (KIND == DELTA) scale /= sqrtf(warp_sum(ss) + 1e-6f);
+        float * out = a.qk + ((size_t) t * 2 * Hk + item) * a.K;
+#pragma unroll
+        for (int i = 0; i < PREP_C; ++i)
+            if (lane + 32 * i < a.K) out[lane + 32 * i] = v[i] * scale;
+        return;
+    }
+    item -= 2 * Hk;
+    if (item < a.H) {
+        for (int c = lane; c < a.V; c += 32)
+            a.v[((size_t) t * a.H + item) * a.V + c] = column<T>(a, t, a.v_off + item * a.V + c, p, back, slot);
+        return;
+    }
+    item -= a.H;
+    if (KIND != LINEAR && item == 0) {
+        for (int h = lane; h < a.H; h += 32) {
+            const float s = head_factor<KIND>(a, to_f(((const T *) a.proj)[(size_t) t * a.ld + a.s_off + h]), h);
+            a.s[(size_t) t * a.H + h] = s;
+            if (KIND == SSD) a.dec[(size_t) t * a.H + h] = expf(a.neg_a[h] * s);
+        }
+        return;
+    }
+    if (KIND != LINEAR) --item;
+    if (KIND != SSD && item < a.H)
+        for (int c = lane; c < a.K; c += 32) {
+            const int i = item * a.K + c;
+            a.dec[(size_t) t * a.H * a.K + i] = channel_decay<KIND>(a, to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + i]) + a.bias[i], item);
+        }
+}
+
+// ---- portions: the recurrence --------------------------------------------------------------------------------------------------
+// grid (H * ceil(V / VB), n_seqs), 128 threads = VB columns of one head's state x LK lanes; a lane keeps 16 of the K channels of its
+// column in registers, channels (j * LK + lane) * 4 + e.  Tokens are staged through shared memory SCAN_TT at a time, one tile
+// ahead.  Also stores the range's last convolution inputs (their old values were read by state_prep).
+constexpr int SCAN_NT = 128, SCAN_TT = 8;
+
+__device__ __forceinline__ void cp16(float * dst, const float * src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t) __cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp4(float * dst, const float * src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t) __cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+template <typename T>
+__device__ void store_conv_tail(const jib_state_mix & a, int slot, int q0, int n, int part, int parts) {
+    if (a.taps < 2 || slot < 0) return;
+    const int keep = min(n, a.taps - 1), p_end = a.positions[q0] + n;
+    for (int i = part * SCAN_NT + threadIdx.x; i < keep * a.n_conv; i += parts * SCAN_NT) {
+        const int d = i / a.n_conv + 1, w = i % a.n_conv;    // d tokens before the end of the range
+        ((T *) a.conv_state)[((size_t) slot * a.taps + (p_end - d) % a.taps) * a.n_conv + w] =
+            ((const T *) a.proj)[(size_t) (q0 + n - d) * a.ld + a.conv0 + w];
+    }
+}
+
+template <typename T, int KIND, int LK>
+__global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_constant__ jib_state_mix a, int splits, int aligned) {
+    constexpr int KP = LK * 16, VB = SCAN_NT / LK;
+    constexpr int ROW = (KIND == SSD ? 2 : 3) * KP;          // k | q | decay
+    constexpr int TILE = SCAN_TT * (ROW + VB + 2);
+    extern __shared__ float smem[];
+    PDL_TRIGGER_TOP();
+    const int h = blockIdx.x / splits, v0 = (blockIdx.x % splits) * VB;
+    const int b = blockIdx.y, lane = threadIdx.x % LK, col = threadIdx.x / LK;
+    const int K = a.K, V = a.V, H = a.H, Hk = H / a.rep, nv = min(VB, V - v0);
+    for (int i = threadIdx.x; i < 2 * TILE; i += SCAN_NT) smem[i] = 0.f;       // channels past K stay zero
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
+    if (n <= 0) return;
+    const int slot = checked_slot(a, b, 46);
+    store_conv_tail<T>(a, slot, q0, n, blockIdx.x, gridDim.x);
+    const bool mine = col < nv;
+    float * st = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K) * V + v0 + col;
+    float s[16];
+    const bool past = slot >= 0 && a.positions[q0] > 0;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        const int c = ((i >> 2) * LK + lane) * 4 + (i & 3);
+        s[i] = past && mine && c < K ? st[(size_t) c * V] : 0.f;
+    }
+    const float * kp = a.qk + ((size_t) q0 * 2 * Hk + Hk + h / a.rep) * K;
+    const float * qp = a.qk + ((size_t) q0 * 2 * Hk + h / a.rep) * K;
+    const float * vp = a.v + ((size_t) q0 * H + h) * V + v0;
+    const float * dp = a.dec + (KIND == SSD ? (size_t) q0 * H + h : ((size_t) q0 * H + h) * K);
+    const float * sp = a.s + (size_t) q0 * H + h;
+    auto stage = [&](int t0, float * d) {
+        const int m = min(SCAN_TT, n - t0);
+        constexpr int NR = KIND == SSD ? 2 : 3;
+        if (aligned) {
+            const int k4 = K / 4;
+            for (int i = threadIdx.x; i < m * NR * k4; i += SCAN_NT) {
+                const int c = i % k4, r = i / k4, tok = r / NR, w = r - tok * NR;
+                const size_t row = t0 + tok;
+                const float * src = w == 0 ? kp + row * 2 * Hk * K : w == 1 ? qp + row * 2 * Hk * K : dp + row * H * K;
+                cp16(d + tok * ROW + w * KP + 4 * c, src + 4 * c);
+            }
+        } else {
+            for (int i = threadIdx.x; i < m * NR * K; i += SCAN_NT) {
+                const int c = i % K, r = i / K, tok = r / NR, w = r - tok * NR;
+                const size_t row = t0 + tok;
+                const float * src = w == 0 ? kp + row * 2 * Hk * K : w == 1 ? qp + row * 2 * Hk * K : dp + row * H * K;
+                cp4(d + tok * ROW + w * KP + c, src + c);
+            }
+        }
+        float * dv = d + SCAN_TT * ROW;
+        for (int i = threadIdx.x; i < m * nv; i += SCAN_NT) cp4(dv + (i / nv) * VB + i % nv, vp + (size_t) (t0 + i / nv) * H * V + i % nv);
+        float * ds = dv + SCAN_TT * VB;
+        if (threadIdx.x < m) {
+            if (KIND != LINEAR) cp4(ds + threadIdx.x, sp + (size_t) (t0 + threadIdx.x) * H);
+            if (KIND == SSD) cp4(ds + SCAN_TT + threadIdx.x, dp + (size_t) (t0 + threadIdx.x) * H);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    __syncthreads();
+    stage(0, smem);
+    const float skip = KIND == SSD ? a.skip[h] : 0.f;
+    float * op = a.o + ((size_t) q0 * H + h) * V + v0 + col;
+    int buf = 0;
+    for (int t0 = 0; t0 < n; t0 += SCAN_TT, buf ^= 1) {
+        if (t0 + SCAN_TT < n) {
+            stage(t0 + SCAN_TT, smem + (buf ^ 1) * TILE);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float * d = smem + buf * TILE;
+        const float * dv = d + SCAN_TT * ROW, * ds = dv + SCAN_TT * VB;
+        const int m = min(SCAN_TT, n - t0);
+        for (int i = 0; i < m; ++i) {
+            float k[16], q[16];
+            const float * row = d + i * ROW + 4 * lane;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float4 x = *(const float4 *) (row + 4 * LK * j), y = *(const float4 *) (row + KP + 4 * LK * j);
+                k[4 * j] = x.x; k[4 * j + 1] = x.y; k[4 * j + 2] = x.z; k[4 * j + 3] = x.w;
+                q[4 * j] = y.x; q[4 * j + 1] = y.y; q[4 * j + 2] = y.z; q[4 * j + 3] = y.w;
+            }
+            if (KIND == SSD) {
+                const float g = ds[SCAN_TT + i];
+#pragma unroll
+                for (int c = 0; c < 16; ++c) s[c] *= g;
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float4 g = *(const float4 *) (row + 2 * KP + 4 * LK * j);
+                    s[4 * j] *= g.x; s[4 * j + 1] *= g.y; s[4 * j + 2] *= g.z; s[4 * j + 3] *= g.w;
+                }
+            }
+            const float v = dv[i * VB + col];
+            float u = v;
+            if (KIND == DELTA) {
+                float e[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int c = 0; c < 16; ++c) e[c & 3] += s[c] * k[c];
+                float r = (e[0] + e[1]) + (e[2] + e[3]);
+#pragma unroll
+                for (int o = LK / 2; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+                u = v - r;
+            }
+            if (KIND != LINEAR) u *= ds[i];
+            float e[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int c = 0; c < 16; ++c) {
+                s[c] += k[c] * u;
+                e[c & 3] += s[c] * q[c];
+            }
+            float r = (e[0] + e[1]) + (e[2] + e[3]);
+#pragma unroll
+            for (int o = LK / 2; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+            if (lane == 0 && mine) op[(size_t) (t0 + i) * H * V] = KIND == SSD ? r + skip * v : r;
+        }
+        __syncthreads();
+    }
+    if (slot >= 0 && mine) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            const int c = ((i >> 2) * LK + lane) * 4 + (i & 3);
+            if (c < K) st[(size_t) c * V] = s[i];
+        }
+    }
+}
+
+// ---- gate and norm of the read-out ---------------------------------------------------------------------------------------------
+// DELTA / LINEAR: one warp per (token, head): o / rms(o) * norm_w * gate.
+template <typename T, int KIND>
+__global__ void __launch_bounds__(256) state_finish_kernel(const __grid_constant__ jib_state_mix a) {
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int lane = threadIdx.x & 31, t = blockIdx.y, h = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (h >= a.H) return;
+    const float * o = a.o + ((size_t) t * a.H + h) * a.V;
+    float ss = 0.f;
+    for (int c = lane; c < a.V; c += 32) ss += o[c] * o[c];
+    const float inv = a.out_scale * rsqrtf(warp_sum(ss) / (float) a.V + a.eps);
+    const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * a.V;
+    T * y = (T *) a.y + (size_t) t * a.ldy + h * a.V;
+    for (int c = lane; c < a.V; c += 32) {
+        const float g = to_f(gate[c]);
+        put(y + c, o[c] * inv * a.norm_w[c] * (KIND == DELTA ? sigmoid<T>(g) : silu<T>(g)));
+    }
+}
+
+// SSD: one CTA per (token, part of the row): y = o * silu(gate), then y / rms(y) * norm_w over the part.
+template <typename T>
+__global__ void __launch_bounds__(256) state_gate_norm_kernel(const __grid_constant__ jib_state_mix a) {
+    PDL_TRIGGER_TOP();
+    __shared__ float red[8];
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int t = blockIdx.y, inner = a.H * a.V, m = inner / a.norm_groups, c0 = blockIdx.x * m;
+    const float * o = a.o + (size_t) t * inner + c0;
+    const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + c0;
+    T * y = (T *) a.y + (size_t) t * a.ldy + c0;
+    constexpr int KEEP = 16;                                 // values a thread holds; longer parts are computed twice
+    float v[KEEP], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        v[i] = c < m ? o[c] * silu<T>(to_f(gate[c])) : 0.f;
+        ss += v[i] * v[i];
+    }
+    for (int c = threadIdx.x + 256 * KEEP; c < m; c += 256) {
+        const float x = o[c] * silu<T>(to_f(gate[c]));
+        ss += x * x;
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += red[i];
+    const float inv = a.out_scale * rsqrtf(ss / (float) m + a.eps);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        if (c < m) put(y + c, v[i] * inv * a.norm_w[c0 + c]);
+    }
+    for (int c = threadIdx.x + 256 * KEEP; c < m; c += 256) put(y + c, o[c] * silu<T>(to_f(gate[c])) * inv * a.norm_w[c0 + c]);
+}
+
+// ---- single tokens -------------------------------------------------------------------------------------------------------------
+// grid (H, n_seqs): one CTA per head and sequence; thread = VEC adjacent columns x every NRG-th row of S, up to STEP_R rows in
+// registers (KEEP: all of them, the state is read once).
+constexpr int STEP_R = 16;
+
+template <int VEC> struct Cols { float v[VEC]; };
+template <int VEC> __device__ __forceinline__ Cols<VEC> ld_cols(const float * p) {
+    Cols<VEC> r;
+    if (VEC == 4) *(float4 *) r.v = *(const float4 *) p;
+    else r.v[0] = *p;
+    return r;
+}
+template <int VEC> __device__ __forceinline__ void st_cols(float * p, const Cols<VEC> & c) {
+    if (VEC == 4) *(float4 *) p = *(const float4 *) c.v;
+    else *p = c.v[0];
+}
+
+template <typename T, int KIND, int VEC, bool KEEP>
+__global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
+    extern __shared__ float smem[];
+    PDL_TRIGGER_TOP();
+    const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, NT = blockDim.x;
+    const int K = a.K, V = a.V, H = a.H;
+    const int ncg = (V + VEC - 1) / VEC, nrg = NT / ncg, cg = tid % ncg, rg = tid / ncg;
+    const bool live = rg < nrg;
+    float * sq = smem, * sk = sq + K, * sd = sk + K, * sv = sd + K, * red = sv + (V + 3) / 4 * 4, * sums = red + nrg * ncg * VEC;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    int slot = a.seq_slots[t];
+    if (slot >= a.n_state) {
+        if (h == 0 && tid == 0) jib_report(a.status, JIB_ERR_BOUNDS, 47, slot);
+        slot = -1;
+    }
+    const int p = a.positions[t];
+    const bool past = slot >= 0 && p > 0;
+    float * st = a.state + ((size_t) (slot < 0 ? 0 : slot) * H + h) * K * V + cg * VEC;
+    Cols<VEC> s[STEP_R];
+    auto load = [&](int r0) {
+#pragma unroll
+        for (int i = 0; i < STEP_R; ++i) {
+            const int r = r0 + rg + i * nrg;
+            if (past && live && r < K) {
+                s[i] = ld_cols<VEC>(st + (size_t) r * V);
+            } else {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) s[i].v[e] = 0.f;
+            }
+        }
+    };
+    if (KEEP) load(0);                                       // in flight while the inputs are prepared
+    const int hk = h / a.rep;
+    for (int i = tid; i < (KIND == SSD ? 2 : 3) * K + V; i += NT) {
+        if (i < K) sq[i] = column<T>(a, t, a.q_off + hk * K + i, p, 0, slot);
+        else if (i < 2 * K) sk[i - K] = column<T>(a, t, a.k_off + hk * K + i - K, p, 0, slot);
+        else if (i < 2 * K + V) sv[i - 2 * K] = column<T>(a, t, a.v_off + h * V + i - 2 * K, p, 0, slot);
+        else {
+            const int c = i - 2 * K - V, g = h * K + c;
+            sd[c] = channel_decay<KIND>(a, to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + g]) + a.bias[g], h);
+        }
+    }
+    float factor = 1.f, decay = 1.f;
+    if (KIND != LINEAR) factor = head_factor<KIND>(a, to_f(((const T *) a.proj)[(size_t) t * a.ld + a.s_off + h]), h);
+    if (KIND == SSD) decay = expf(a.neg_a[h] * factor);
+    __syncthreads();
+    if (a.taps > 1 && slot >= 0) {                           // this position's convolution inputs; no reader of this launch needs the row
+        T * ring = (T *) a.conv_state + ((size_t) slot * a.taps + p % a.taps) * a.n_conv;
+        const T * x = (const T *) a.proj + (size_t) t * a.ld;
+        const bool owner = h % a.rep == 0;
+        for (int i = tid; i < (owner ? 2 * K : 0) + V; i += NT) {
+            const int c = i < V ? a.v_off + h * V + i : (i < V + K ? a.q_off + hk * K + i - V : a.k_off + hk * K + i - V - K);
+            ring[c - a.conv0] = x[c];
+        }
+    }
+    float qn = a.q_scale, kn = 1.f;
+    if (KIND == DELTA) {
+        if (tid < 64) {
+            const float * x = tid < 32 ? sq : sk;
+            float ss = 0.f;
+            for (int c = tid & 31; c < K; c += 32) ss += x[c] * x[c];
+            ss = warp_sum(ss);
+            if ((tid & 31) == 0) sums[tid >> 5] = 1.f / sqrtf(ss + 1e-6f);
+        }
+        __syncthreads();
+        qn *= sums[0];
+        kn = sums[1];
+        // S^T k after the decay
+        Cols<VEC> d;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) d.v[e] = 0.f;
+        for (int r0 = 0; r0 < K; r0 += nrg * STEP_R) {
+            if (!KEEP) load(r0);
+#pragma unroll
+            for (int i = 0; i < STEP_R; ++i) {
+                const int r = r0 + rg + i * nrg;
+                if (r >= K) continue;
+                const float g = sd[r], kk = sk[r] * kn;
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) d.v[e] += s[i].v[e] * g * kk;
+            }
+        }
+        if (live) st_cols<VEC>(red + (rg * ncg + cg) * VEC, d);
+        __syncthreads();
+    }
+    Cols<VEC> u, o;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+        o.v[e] = 0.f;
+        u.v[e] = live && cg * VEC + e < V ? sv[cg * VEC + e] : 0.f;
+    }
+    if (KIND == DELTA && live)
+        for (int g = 0; g < nrg; ++g) {
+            const Cols<VEC> d = ld_cols<VEC>(red + (g * ncg + cg) * VEC);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) u.v[e] -= d.v[e];
+        }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u.v[e] *= factor * kn;
+    for (int r0 = 0; r0 < K; r0 += nrg * STEP_R) {
+        if (!KEEP) load(r0);
+#pragma unroll
+        for (int i = 0; i < STEP_R; ++i) {
+            const int r = r0 + rg + i * nrg;
+            if (r >= K || !live) continue;
+            const float g = KIND == SSD ? decay : sd[r], kk = sk[r], qq = sq[r];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                s[i].v[e] = s[i].v[e] * g + kk * u.v[e];
+                o.v[e] += s[i].v[e] * qq;
+            }
+            if (slot >= 0) st_cols<VEC>(st + (size_t) r * V, s[i]);
+        }
+    }
+    if (KIND == DELTA) __syncthreads();                      // red is read above
+    if (live) st_cols<VEC>(red + (rg * ncg + cg) * VEC, o);
+    __syncthreads();
+    // columns back to one thread each: sum over the row groups, then norm and gate
+    float ss = 0.f;
+    for (int c = tid; c < V; c += NT) {
+        float v = 0.f;
+        for (int g = 0; g < nrg; ++g) v += red[g * ncg * VEC + c];
+        v *= qn;
+        if (KIND == SSD) a.o[((size_t) t * H + h) * V + c] = v + a.skip[h] * sv[c];
+        else sv[c] = v;
+        ss += v * v;
+    }
+    if (KIND == SSD) return;
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) sums[2 + (tid >> 5)] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < NT / 32; ++i) ss += sums[2 + i];
+    const float inv = a.out_scale * rsqrtf(ss / (float) V + a.eps);
+    const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * V;
+    T * y = (T *) a.y + (size_t) t * a.ldy + h * V;
+    for (int c = tid; c < V; c += NT) {
+        const float g = to_f(gate[c]);
+        put(y + c, sv[c] * inv * a.norm_w[c] * (KIND == DELTA ? sigmoid<T>(g) : silu<T>(g)));
+    }
+}
+
+inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
+
+template <typename T, int KIND, int LK>
+int launch_scan(const jib_state_mix & a, cudaStream_t s) {
+    constexpr int VB = SCAN_NT / LK, SMEM = 2 * SCAN_TT * ((KIND == SSD ? 2 : 3) * LK * 16 + VB + 2) * 4;
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (!jib::ensure_dyn_smem(state_scan_kernel<T, KIND, LK>, SMEM, done)) return JIB_E_LAUNCH;
+    const int splits = (a.V + VB - 1) / VB;
+    JIB_LAUNCH((state_scan_kernel<T, KIND, LK>), dim3(a.H * splits, a.n_seqs), SCAN_NT, SMEM, s, a, splits, a.K % 4 == 0);
+    return launched();
+}
+
+template <typename T, int KIND>
+int launch_finish(const jib_state_mix & a, cudaStream_t s) {
+    if (KIND == SSD) JIB_LAUNCH((state_gate_norm_kernel<T>), dim3(a.norm_groups, a.T), 256, 0, s, a);
+    else JIB_LAUNCH((state_finish_kernel<T, KIND>), dim3((a.H + 7) / 8, a.T), 256, 0, s, a);
+    return launched();
+}
+
+template <typename T, int KIND, int VEC, bool KEEP>
+int launch_step(const jib_state_mix & a, int nt, cudaStream_t s) {
+    const int ncg = (a.V + VEC - 1) / VEC, nrg = nt / ncg;
+    const int smem = (3 * a.K + (a.V + 3) / 4 * 4 + nrg * ncg * VEC + 2 + 32) * 4;
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (smem > 100 * 1024 || !jib::ensure_dyn_smem(state_step_kernel<T, KIND, VEC, KEEP>, 100 * 1024, done)) return JIB_E_ARG;
+    JIB_LAUNCH((state_step_kernel<T, KIND, VEC, KEEP>), dim3(a.H, a.n_seqs), nt, smem, s, a);
+    return KIND == SSD ? launch_finish<T, SSD>(a, s) : launched();
+}
+
+template <typename T, int KIND>
+int run(const jib_state_mix & a, int single, cudaStream_t s) {
+    if (single) {
+        const int vec = a.V % 4 == 0 && a.K % 4 == 0 ? 4 : 1;
+        const int ncg = (a.V + vec - 1) / vec;
+        if (ncg > 512) return JIB_E_ARG;
+        int nt = 256;
+        while (nt < 512 && ((nt / ncg) * STEP_R < a.K)) nt *= 2;
+        const bool keep = (nt / ncg) * STEP_R >= a.K;
+        if (vec == 4) return keep ? launch_step<T, KIND, 4, true>(a, nt, s) : launch_step<T, KIND, 4, false>(a, nt, s);
+        return keep ? launch_step<T, KIND, 1, true>(a, nt, s) : launch_step<T, KIND, 1, false>(a, nt, s);
+    }
+    const int items = 2 * (a.H / a.rep) + a.H + (KIND == LINEAR ? 0 : 1) + (KIND == SSD ? 0 : a.H);
+    JIB_LAUNCH((state_prep_kernel<T, KIND>), dim3((items + 7) / 8, a.T), 256, 0, s, a);
+    int rc = launched();
+    if (rc) return rc;
+    if (a.K <= 16) rc = launch_scan<T, KIND, 1>(a, s);
+    else if (a.K <= 32) rc = launch_scan<T, KIND, 2>(a, s);
+    else if (a.K <= 64) rc = launch_scan<T, KIND, 4>(a, s);
+    else if (a.K <= 128) rc = launch_scan<T, KIND, 8>(a, s);
+    else if (a.K <= 256) rc = launch_scan<T, KIND, 16>(a, s);
+    else rc = launch_scan<T, KIND, 32>(a, s);
+    return rc ? rc : launch_finish<T, KIND>(a, s);
+}
+
+}  // namespace
+
+extern "C" JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, void * stream) {
+    const jib_state_mix & a = *m;
+    if (a.T <= 0 || a.n_seqs <= 0) return 0;
+    if (a.H < 1 || a.K < 1 || a.V < 1 || a.K > 32 * PREP_C || a.rep < 1 || a.H % a.rep || a.T > 65535 || a.n_seqs > 65535 ||
+        (a.taps > 0 && (a.conv_state == nullptr || a.conv_w == nullptr)) || (a.kind == SSD && (a.norm_groups < 1 || (a.H * a.V) % a.norm_groups)) ||
+        (single && a.n_seqs != a.T) || (!single && (a.qk == nullptr || a.v == nullptr || a.dec == nullptr)) || (a.kind != LINEAR && !single && a.s == nullptr) ||
+        ((a.kind == SSD || !single) && a.o == nullptr))
+        return JIB_E_ARG;
+    cudaStream_t s = (cudaStream_t) stream;
+    switch (a.kind) {
+        case DELTA: return f32 ? run<float, DELTA>(a, single, s) : run<bf16, DELTA>(a, single, s);
+        case LINEAR: return f32 ? run<float, LINEAR>(a, single, s) : run<bf16, LINEAR>(a, single, s);
+        case SSD: return f32 ? run<float, SSD>(a, single, s) : run<bf16, SSD>(a, single, s);
+    }
+    return JIB_E_ARG;
+}

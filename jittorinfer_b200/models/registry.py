@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Any, Callable, Dict, Optional
 
-from . import nibalix
+from . import lugovik, nibalix
 from .deepseek2 import DeepSeek2Model
 from .hparams import ARCH as DEEPSEEK2, DeepSeek2HParams
 from .hparams import preset as _deepseek2_preset
@@ -33,6 +33,8 @@ ARCHITECTURES: Dict[str, Architecture] = {
     DEEPSEEK2: Architecture(DEEPSEEK2, DeepSeek2HParams, DeepSeek2Model, _deepseek2_preset, sharded=True),
     nibalix.ARCH: Architecture(nibalix.ARCH, nibalix.NibalixHParams, nibalix.NibalixModel, nibalix.preset, nibalix.load_config,
                                nibalix.iter_checkpoint, nibalix.iter_random),
+    lugovik.ARCH: Architecture(lugovik.ARCH, lugovik.LugovikHParams, lugovik.LugovikModel, lugovik.preset, lugovik.load_config,
+                               lugovik.iter_checkpoint, lugovik.iter_random),
 }
 
 

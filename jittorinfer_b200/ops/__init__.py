@@ -68,6 +68,13 @@ def gateup_silu(x, wg, wu):
     return ref.gateup_silu(x, wg, wu)
 
 
+def gateup(x, wg, wu, act):
+    """act(x wg^T) * (x wu^T), ``act`` "silu" or "gelu_tanh"; fp32 operands take the library's products."""
+    if use_native(x) and x.dtype == torch.bfloat16:
+        return nat().gateup(x, wg, wu, act)
+    return ref.gateup(x, wg, wu, act)
+
+
 def mla_qkv_post(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r, rot_half=False):
     f = nat().mla_qkv_post if use_native(q) else ref.mla_qkv_post
     return f(q, ckv, kv_norm_w, eps, rope_table, positions, slot_mapping, cache, q_out, n_head, dn, dr, r, rot_half)
@@ -130,9 +137,14 @@ def fused_combine_norm() -> bool:
 # ---- parallel blocks over an fp32 residual stream, per-sequence state -------------------------------------------------------------
 # ``nxt`` = (norm weight, eps, conv): the norm the next block reads, computed in the same pass; conv = None, or -- one token per
 # sequence only -- (weights [taps, d], state, seq_slots, positions) of that block's input convolution.
-def embed_norm(table, ids, w, eps, nxt=None):
-    """(x fp32 = norm of the embedding rows, h, h + convolution)."""
-    return (nat() if use_native(table) else ref).embed_norm(table, ids, w, eps, nxt)
+def embed_norm(table, ids, w, eps, nxt=None, scale=1.0):
+    """(x fp32 = norm of the scaled embedding rows (``w`` None: the rows themselves), h, h + convolution)."""
+    return (nat() if use_native(table) else ref).embed_norm(table, ids, w, eps, nxt, scale)
+
+
+def post_norm(x, y, w, eps, nxt=None):
+    """(x + norm(y) * w, h) with ``nxt`` = (norm weight, eps, None) of the sublayer that follows; x may be overwritten."""
+    return (nat() if use_native(x) else ref).post_norm(x, y, w, eps, nxt)
 
 
 def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
@@ -150,6 +162,21 @@ def causal_conv(h, w, state, seq_slots, positions, q_start):
 
 def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
     return (nat() if use_native(zxg) else ref).mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single)
+
+
+# ---- mixers described by a spec (ops/specs.py) ------------------------------------------------------------------------------------
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
+    """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view)."""
+    return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out)
+
+
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
+    return (nat() if use_native(q) else ref).gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache)
+
+
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
+    """Result columns go to ``out`` (a view)."""
+    return (nat() if use_native(q) else ref).gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out)
 
 
 def argmax(logits):

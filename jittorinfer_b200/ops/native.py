@@ -48,6 +48,9 @@ ERRORS = {-1: "unsupported shape/argument", -2: "pointer or stride not 16-byte a
           -4: "tensor map encode failed", -5: "kernel launch failed", -6: "scratch too small for requested split"}
 
 
+ACTS = {"silu": 0, "gelu_tanh": 1}     # activation of a gated pair (JIB_ACT_*)
+
+
 class GemmDesc(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x", "w", "w2", "out", "residual", "seg", "scratch", "counters", "status")] + \
                [(n, C.c_longlong) for n in ("x_row_stride", "x_batch_stride", "w_row_stride", "w_batch_stride", "ldo",
@@ -58,12 +61,29 @@ class GemmDesc(C.Structure):
                                                                              ("ag_epoch", C.c_void_p), ("ag_rows", C.c_int),
                                                                              ("ag_world", C.c_int), ("ar_rs_rows", C.c_int),
                                                                              ("src_token", C.c_void_p), ("src_rows", C.c_int), ("expert_list", C.c_void_p),
-                                                                             ("n_slots", C.c_int), ("list_tiles", C.c_int), ("pdl_flags", C.c_int)]
+                                                                             ("n_slots", C.c_int), ("list_tiles", C.c_int), ("pdl_flags", C.c_int),
+                                                                             ("act", C.c_int)]
 
 
 class RowTail(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x_out", "norm_w", "h_out", "conv_w", "hc_out", "conv_state", "seq_slots", "positions", "status")] + \
                [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int)]
+
+
+class StateMixDesc(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "dec_in", "gate", "y", "conv_state", "state", "conv_w", "conv_b", "bias", "neg_a", "skip", "norm_w",
+                                          "seq_slots", "positions", "q_start", "status", "qk", "v", "dec", "s", "o")] + \
+               [(n, C.c_longlong) for n in ("ld", "ld_dec", "ld_gate", "ldy")] + \
+               [(n, C.c_int) for n in ("kind", "H", "K", "V", "rep", "taps", "conv0", "n_conv", "q_off", "k_off", "v_off", "s_off", "norm_groups",
+                                       "n_state", "n_seqs", "T")] + \
+               [(n, C.c_float) for n in ("q_scale", "inv_tau", "eps", "out_scale")]
+
+
+class GqaDesc(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("cache", "block_tables", "seq_lens", "q_start", "positions", "status")] + \
+               [(n, C.c_longlong) for n in ("n_slots", "row")] + \
+               [(n, C.c_int) for n in ("H", "G", "D", "V", "rot", "block_size", "max_blocks", "n_seqs", "T", "max_pos", "window", "chunk", "sink")] + \
+               [(n, C.c_float) for n in ("scale", "softcap", "eps", "out_scale")]
 
 
 def load():
@@ -84,11 +104,15 @@ def load():
 
     sig("jib_gemm_bf16", C.POINTER(GemmDesc), vp)
     sig("jib_gemm_simt", C.POINTER(GemmDesc), i, vp)
-    sig("jib_embed_norm", vp, ip, fp, f, i, i, i, i, C.POINTER(RowTail), vp)
+    sig("jib_embed_norm", vp, ip, fp, f, f, i, i, i, i, C.POINTER(RowTail), vp)
+    sig("jib_post_norm", fp, vp, fp, f, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_block_update", fp, f, vp, vp, ll, fp, fp, vp, ip, fp, i, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, vp, vp)
     sig("jib_causal_conv", vp, fp, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
     sig("jib_mingru", vp, ll, fp, fp, fp, i, ip, ip, ip, i, i, i, i, i, vp, ip, vp)
+    sig("jib_state_mix_run", C.POINTER(StateMixDesc), i, i, vp)
+    sig("jib_gqa_qkv_post", C.POINTER(GqaDesc), vp, vp, vp, ll, fp, fp, fp, ip, vp, i, vp)
+    sig("jib_gqa_attention", C.POINTER(GqaDesc), vp, vp, ll, vp, ll, i, i, i, vp)
     sig("jib_embed_gather", vp, ip, vp, i, i, i, vp)
     sig("jib_rmsnorm", vp, vp, fp, vp, vp, i, i, ll, f, vp)
     sig("jib_mla_qkv_post", vp, ll, vp, ll, fp, f, fp, ip, ip, vp, vp, ll, ll, i, i, i, i, i, i, ll, i, i, ip, vp)
@@ -201,8 +225,8 @@ def _gemm_simt(d: GemmDesc, f32: bool, what: str) -> None:
 
 def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *, out: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, splits: int = 0, bn: int = 0,
-         ar=None, ar_site: int = 0, ar_rs_rows: int = 0, ag=None) -> torch.Tensor:
-    """out[T,N] = x[T,K] @ w[N,K]^T  (w2: silu(x w^T) * (x w2^T)) (+ residual)."""
+         ar=None, ar_site: int = 0, ar_rs_rows: int = 0, ag=None, act: str = "silu") -> torch.Tensor:
+    """out[T,N] = x[T,K] @ w[N,K]^T  (w2: act(x w^T) * (x w2^T)) (+ residual)."""
     assert x.dtype == w.dtype and x.dtype in (torch.bfloat16, torch.float32) and x.stride(-1) == 1 and w.is_contiguous()
     T, K = x.shape
     N = w.shape[0]
@@ -220,7 +244,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *,
     d.T, d.N, d.K, d.batch, d.max_rows, d.active_hint = T, N, K, 1, 0, 0
     d.out_f32 = int(out.dtype == torch.float32)
     d.res_f32 = int(residual is not None and residual.dtype == torch.float32)
-    d.splits, d.bn, d.sm_count = splits, bn, ws.sm_count
+    d.splits, d.bn, d.sm_count, d.act = splits, bn, ws.sm_count, ACTS[act]
     if ar is not None:          # fused all-reduce (or, with ar_rs_rows, reduce-scatter by rows) over peer memory in the epilogue
         d.ar, d.ar_site, d.ar_rs_rows = C.addressof(ar), ar_site, ar_rs_rows
     if ag is not None:          # x is a gather buffer other ranks are still filling: (flags ptr, epoch ptr, rows per rank, world)
@@ -320,6 +344,10 @@ def grouped_tma_ok(x: torch.Tensor, wg: torch.Tensor) -> bool:
 
 def gateup_silu(x, wg, wu):
     return gemm(x, wg, wu)
+
+
+def gateup(x, wg, wu, act):
+    return gemm(x, wg, wu, act=act)
 
 
 # ---- memory-bound kernels ------------------------------------------------------------------------
@@ -654,11 +682,11 @@ def _row_tail(x_out, nxt, dtype):
     return t, h, hc
 
 
-def embed_norm(table, ids, w, eps, nxt=None):
+def embed_norm(table, ids, w, eps, nxt=None, scale=1.0):
     T, d = ids.shape[0], table.shape[1]
     x = torch.empty(T, d, dtype=torch.float32, device=table.device)
     tail, h, hc = _row_tail(x, nxt, table.dtype)
-    _ck(load().jib_embed_norm(table.data_ptr(), ids.data_ptr(), w.data_ptr(), float(eps), T, d, table.shape[0],
+    _ck(load().jib_embed_norm(table.data_ptr(), ids.data_ptr(), _p(w), float(eps), float(scale), T, d, table.shape[0],
                               int(table.dtype == torch.float32), C.byref(tail), _stream()), "embed_norm")
     return x, h, hc
 
@@ -672,6 +700,15 @@ def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
                                 _p(wts), dest.shape[1] if dest is not None else 0, T, d, int(o.dtype == torch.float32), C.byref(tail),
                                 _stream()), "block_update")
     return x, h, hc
+
+
+def post_norm(x, y, w, eps, nxt=None):
+    T, d = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous()
+    tail, h, _ = _row_tail(x, nxt, y.dtype)
+    _ck(load().jib_post_norm(x.data_ptr(), y.data_ptr(), w.data_ptr(), float(eps), T, d, int(y.dtype == torch.float32), C.byref(tail), _stream()),
+        "post_norm")
+    return x, h
 
 
 def rms_rows(x, rows, w, eps, dtype):
@@ -701,6 +738,82 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
                           positions.data_ptr(), q_start.data_ptr(), q_start.shape[0] - 1, T, W, int(single),
                           int(zxg.dtype == torch.float32), y.data_ptr(), workspace(zxg.device).status.data_ptr(), _stream()), "mingru")
     return y
+
+
+# ---- mixers described by a spec: matrix state per head (state_mix.cu), grouped-query attention (gqa_attention.cu) ----------------
+STATE_KINDS = {"delta": 0, "linear": 1, "ssd": 2}
+
+
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
+    T, H, K, V = proj.shape[0], m.heads, m.dim, m.vdim
+    assert proj.stride(1) == 1 and gate.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype == gate.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and (m.taps == 0 or (conv_state.is_contiguous() and conv_state.dtype == proj.dtype))
+    f32 = lambda *s: torch.empty(*s, dtype=torch.float32, device=proj.device)        # noqa: E731
+    d = StateMixDesc()
+    d.proj, d.ld, d.gate, d.ld_gate, d.y, d.ldy = proj.data_ptr(), proj.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
+    if dec_in is not None:
+        assert dec_in.stride(1) == 1 and dec_in.dtype == proj.dtype
+        d.dec_in, d.ld_dec = dec_in.data_ptr(), dec_in.stride(0)
+    d.conv_state, d.state, d.n_state = _p(conv_state), state.data_ptr(), state.shape[0]
+    d.conv_w, d.conv_b, d.bias, d.neg_a, d.skip, d.norm_w = _p(m.conv_w), _p(m.conv_b), _p(m.bias), _p(m.neg_a), _p(m.skip), _p(m.norm_w)
+    d.seq_slots, d.positions, d.q_start = seq_slots.data_ptr(), positions.data_ptr(), q_start.data_ptr()
+    d.status = workspace(proj.device).status.data_ptr()
+    d.kind, d.H, d.K, d.V, d.rep, d.taps, d.conv0 = STATE_KINDS[m.kind], H, K, V, m.rep, m.taps, m.conv0
+    d.n_conv = m.conv_w.shape[1] if m.conv_w is not None else 0
+    d.q_off, d.k_off, d.v_off, d.s_off, d.norm_groups = m.q_off, m.k_off, m.v_off, m.s_off, m.norm_groups
+    d.n_seqs, d.T = q_start.shape[0] - 1, T
+    d.q_scale, d.inv_tau, d.eps, d.out_scale = m.q_scale, m.inv_tau, m.eps, m.out_scale
+    scratch = []
+    if not single:
+        scratch = [f32(T, 2 * (H // m.rep) * K), f32(T, H * V), f32(T, H * (1 if m.kind == "ssd" else K)), f32(T, H)]
+        d.qk, d.v, d.dec, d.s = (x.data_ptr() for x in scratch)
+    if not single or m.kind == "ssd":
+        scratch.append(f32(T, H * V))
+        d.o = scratch[-1].data_ptr()
+    _ck(load().jib_state_mix_run(C.byref(d), int(single), int(proj.dtype == torch.float32), _stream()), "state_mix")
+    return out
+
+
+def _gqa_desc(m, cache, T, n_seqs):
+    assert cache.is_contiguous()
+    d = GqaDesc()
+    d.cache, d.n_slots, d.row, d.status = cache.data_ptr(), cache.shape[0], cache.shape[1], workspace(cache.device).status.data_ptr()
+    d.H, d.G, d.D, d.V, d.rot, d.T, d.n_seqs, d.block_size = m.heads, m.kv_heads, m.dim, m.vdim, m.rot, T, n_seqs, 64
+    d.window, d.chunk, d.sink = m.window, m.chunk, int(m.sink)
+    d.scale, d.softcap, d.eps, d.out_scale = m.scale, m.softcap, m.eps, m.out_scale
+    return d
+
+
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
+    T = q.shape[0]
+    assert q.dtype == cache.dtype and q.stride(1) == 1 and k.stride(0) == q.stride(0) == v.stride(0) and rope_table.is_contiguous()
+    out = torch.empty(T, m.heads, m.dim, dtype=q.dtype, device=q.device)
+    d = _gqa_desc(m, cache, T, 1)
+    d.positions, d.max_pos = positions.data_ptr(), rope_table.shape[0]
+    _ck(load().jib_gqa_qkv_post(C.byref(d), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), m.q_norm.data_ptr(), m.k_norm.data_ptr(),
+                                rope_table.data_ptr(), slot_mapping.data_ptr(), out.data_ptr(), int(q.dtype == torch.float32), _stream()), "gqa_qkv_post")
+    return out
+
+
+def gqa_splits(m, T, max_keys, sm_count=148):
+    """CTAs that share one row's keys in a batch of single tokens: as many as fill the machine, at most one per 64 visible keys."""
+    keys = min([x for x in (m.window, m.chunk, max_keys) if x > 0])
+    fill = max(1, 2 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
+    n = min(8, fill, (keys + 63) // 64)
+    return 1 << (n.bit_length() - 1)
+
+
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
+    T, H, D = q.shape
+    assert q.dtype == cache.dtype == out.dtype and q.is_contiguous() and out.stride(1) == 1
+    single = max_q_len == 1 and seq_lens.shape[0] == T
+    d = _gqa_desc(m, cache, T, seq_lens.shape[0])
+    d.block_tables, d.max_blocks, d.block_size = block_tables.data_ptr(), block_tables.stride(0), block_size
+    d.seq_lens, d.q_start = seq_lens.data_ptr(), q_start.data_ptr()
+    splits = gqa_splits(m, T, block_tables.shape[1] * block_size, workspace(q.device).sm_count) if single else 1
+    _ck(load().jib_gqa_attention(C.byref(d), q.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), int(single),
+                                 splits, int(q.dtype == torch.float32), _stream()), "gqa_attention")
+    return out
 
 
 # ---- sampling / cache ----------------------------------------------------------------------------

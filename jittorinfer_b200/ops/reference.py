@@ -47,6 +47,13 @@ def gateup_silu(x: torch.Tensor, wg: torch.Tensor, wu: torch.Tensor) -> torch.Te
     return (F.silu(g) * u).to(x.dtype)
 
 
+def gateup(x: torch.Tensor, wg: torch.Tensor, wu: torch.Tensor, act: str) -> torch.Tensor:
+    """act(x wg^T) * (x wu^T), ``act`` "silu" or "gelu_tanh"."""
+    g = linear(x, wg, out_dtype=torch.float32)
+    u = linear(x, wu, out_dtype=torch.float32)
+    return ((F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh")) * u).to(x.dtype)
+
+
 def yarn_table(n_pos: int, dr: int, freq_base: float, freq_scale: float, ext_factor: float, attn_factor: float,
                corr_lo: float, corr_hi: float, device="cpu") -> torch.Tensor:
     """[n_pos, dr/2, 2] fp32 (cos, sin) incl. magnitude factor — the GE path's RopeCache
@@ -278,8 +285,10 @@ def _finish_row(x, nxt, dtype):
     return x, h, causal_conv(h, cw, state, slots, positions, n)
 
 
-def embed_norm(table, ids, w, eps, nxt=None):
-    v = table[ids.long()].float()
+def embed_norm(table, ids, w, eps, nxt=None, scale=1.0):
+    v = table[ids.long()].float() * scale
+    if w is None:
+        return _finish_row(v, nxt, table.dtype)
     return _finish_row(v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w, nxt, table.dtype)
 
 
@@ -292,6 +301,11 @@ def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
         f = (y.float()[dest.long()] * wts[..., None]).sum(1)
         s = s + torch.sigmoid(gates[:, d:2 * d].float() + b2) * f
     return _finish_row(x + mult * s, nxt, o.dtype)
+
+
+def post_norm(x, y, w, eps, nxt=None):
+    v = y.float()
+    return _finish_row(x + v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w, nxt, y.dtype)[:2]
 
 
 def rms_rows(x, rows, w, eps, dtype):
@@ -343,3 +357,117 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
         if slot >= 0:
             state[slot] = s
     return y
+
+
+# ---- mixers with a matrix state per head (csrc/kernels/state_mix.cu) ------------------------------------------------------------------
+def _softplus(x):
+    return F.softplus(x, threshold=1e9)
+
+
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
+    """Runs the mixer described by ``m`` (``ops.specs.StateMix``) over a batch; result columns go to ``out`` [T, H * V]."""
+    H, K, V, Hk = m.heads, m.dim, m.vdim, m.heads // m.rep
+    qs = q_start.tolist()
+    for b in range(len(qs) - 1):
+        q0, q1 = qs[b], qs[b + 1]
+        if q1 <= q0:
+            continue
+        slot, n, p0 = int(seq_slots[b]), q1 - q0, int(positions[q0])
+        x = proj[q0:q1].float().clone()
+        if m.taps:
+            c0, nc = m.conv0, m.conv_w.shape[1]
+            old = torch.zeros(m.taps - 1, nc, device=proj.device)
+            for d in range(1, m.taps):                            # ring row p % taps holds position p's inputs
+                if slot >= 0 and p0 - d >= 0:
+                    old[m.taps - 1 - d] = conv_state[slot, (p0 - d) % m.taps].float()
+            ext = torch.cat([old, x[:, c0:c0 + nc]], 0)
+            acc = torch.zeros(n, nc, device=proj.device) if m.conv_b is None else m.conv_b.expand(n, nc).clone()
+            for j in range(m.taps):
+                acc += m.conv_w[j] * ext[j:j + n]
+            if slot >= 0:
+                for d in range(1, min(n, m.taps - 1) + 1):
+                    conv_state[slot, (p0 + n - d) % m.taps] = proj[q1 - d, c0:c0 + nc]
+            x[:, c0:c0 + nc] = F.silu(acc)
+        cols = lambda off, h, w: x[:, off:off + h * w].view(n, h, w)          # noqa: B023,E731
+        q, k, v = cols(m.q_off, Hk, K), cols(m.k_off, Hk, K), cols(m.v_off, H, V)
+        s = torch.ones(n, H, device=proj.device)
+        if m.kind == "delta":
+            q, k = (y / torch.sqrt(y.pow(2).sum(-1, keepdim=True) + 1e-6) for y in (q, k))
+            s = torch.sigmoid(x[:, m.s_off:m.s_off + H])
+        if m.kind == "ssd":
+            s = _softplus(x[:, m.s_off:m.s_off + H] + m.bias)
+            dec = torch.exp(m.neg_a * s)[..., None]
+        else:
+            z = dec_in[q0:q1].float() + m.bias
+            dec = torch.exp(m.neg_a[:, None] * _softplus(z).view(n, H, K)) if m.kind == "delta" else \
+                torch.exp(-m.inv_tau * _softplus(-z)).view(n, H, K)
+        q, k = (q * m.q_scale).repeat_interleave(m.rep, 1), k.repeat_interleave(m.rep, 1)
+        S = state[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, K, V, device=proj.device)
+        o = torch.empty(n, H, V, device=proj.device)
+        for t in range(n):
+            S = S * dec[t][..., None]
+            u = v[t] - torch.einsum("hkv,hk->hv", S, k[t]) if m.kind == "delta" else v[t]
+            S = S + k[t][..., None] * (s[t][:, None] * u)[:, None, :]
+            o[t] = torch.einsum("hkv,hk->hv", S, q[t])
+        if slot >= 0:
+            state[slot] = S
+        g = gate[q0:q1, :H * V].float()
+        if m.kind == "ssd":
+            y = (o + m.skip[:, None] * v).reshape(n, H * V) * F.silu(g)
+            y = y.view(n, m.norm_groups, -1)
+            y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + m.eps)).reshape(n, H * V) * m.norm_w
+        else:
+            y = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + m.eps) * m.norm_w).reshape(n, H * V)
+            y = y * (torch.sigmoid(g) if m.kind == "delta" else F.silu(g))
+        out[q0:q1, :H * V] = (y * m.out_scale).to(out.dtype)
+    return out
+
+
+# ---- grouped-query attention over paged rows (csrc/kernels/gqa_attention.cu) ------------------------------------------------------------
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
+    """Norms and rotates q and k, stores the rows of the cache; returns q [T, H, D].  ``m``: ``ops.specs.Gqa``."""
+    T, H, G, D, V = q.shape[0], m.heads, m.kv_heads, m.dim, m.vdim
+    cs = rope_table[positions.long()]
+
+    def post(x, n, w):
+        x = x.float().reshape(T, n, D)
+        x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + m.eps) * w
+        return torch.cat([_rope(x[..., :m.rot], cs, True), x[..., m.rot:]], -1)
+    qo = post(q, H, m.q_norm).to(q.dtype)
+    rows = torch.cat([post(k, G, m.k_norm).reshape(T, G * D), v.float()], 1).to(cache.dtype)
+    ok = slot_mapping >= 0
+    cache[slot_mapping[ok].long()] = rows[ok]
+    return qo
+
+
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
+    """Result columns go to ``out`` [T, H * V]; ``gate`` [T, H] pre-activations."""
+    T, H, D = q.shape
+    G, V = m.kv_heads, m.vdim
+    qs, sl = q_start.tolist(), seq_lens.tolist()
+    for b in range(len(qs) - 1):
+        q0, q1, S = qs[b], qs[b + 1], sl[b]
+        if q1 <= q0 or S <= 0:
+            continue
+        pos = torch.arange(S, device=q.device)
+        rows = cache[block_tables[b].long()[pos // block_size] * block_size + pos % block_size].float()
+        k = rows[:, :G * D].view(S, G, D).repeat_interleave(H // G, 1)
+        v = rows[:, G * D:].view(S, G, V).repeat_interleave(H // G, 1)
+        i, j = torch.arange(S - (q1 - q0), S, device=q.device)[:, None], pos[None]
+        see = j <= i
+        if m.window:
+            see = see & (i - j < m.window)
+        if m.chunk:
+            see = see & (i // m.chunk == j // m.chunk)
+        s = torch.einsum("ihd,jhd->hij", q[q0:q1].float(), k) * m.scale
+        if m.softcap:
+            s = m.softcap * torch.tanh(s / m.softcap)
+        s = s.masked_fill(~see, float("-inf"))
+        if m.sink:                                                # a key of score 0 without a value
+            s = torch.cat([s, torch.zeros_like(s[..., :1])], -1)
+        p = torch.softmax(s, -1)[..., :S]
+        o = torch.einsum("hij,jhv->ihv", p, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].float())[..., None]
+        out[q0:q1, :H * V] = (o * m.out_scale).reshape(q1 - q0, H * V).to(out.dtype)
+    return out

@@ -1,0 +1,63 @@
+"""What one layer's token mixer computes: sizes, constants and small parameter tensors, shared by the kernels and the reference ops."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+
+@dataclass
+class StateMix:
+    """A mixer with a matrix state per head: S <- diag(decay) S; u = s (v - [delta] S^T k); S <- S + k u^T; o = S^T q + skip v.
+
+    ``kind``  "delta": q, k unit vectors, decay exp(neg_a softplus(. + bias)) per key channel, s = sigmoid(.), norm per head, sigmoid gate;
+    "linear": decay sigmoid(. + bias)^inv_tau per key channel, s = 1, norm per head, silu gate;
+    "ssd": s = softplus(. + bias), decay exp(neg_a s) per head, silu gate, then a norm over ``norm_groups`` parts of the row.
+    ``*_off``: columns of the projection.  Columns conv0 .. conv0 + n of it pass a causal convolution of ``taps`` taps (0: none) and silu."""
+    kind: str
+    heads: int
+    dim: int                                    # key channels
+    vdim: int
+    rep: int = 1                                # heads that share a q / k head
+    q_off: int = 0
+    k_off: int = 0
+    v_off: int = 0
+    s_off: int = 0
+    taps: int = 0
+    conv0: int = 0
+    conv_w: Optional[torch.Tensor] = None       # [taps, n] fp32, last tap = current token
+    conv_b: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    neg_a: Optional[torch.Tensor] = None        # [heads]
+    skip: Optional[torch.Tensor] = None         # [heads]
+    norm_w: Optional[torch.Tensor] = None
+    norm_groups: int = 1
+    q_scale: float = 1.0
+    inv_tau: float = 1.0
+    eps: float = 1e-6
+    out_scale: float = 1.0
+
+
+@dataclass
+class Gqa:
+    """Grouped-query attention with normed q and k, rotate-half RoPE on the first ``rot`` dimensions, scores * scale, softcap (0: none), a
+    causal mask with a sliding window and / or chunks (0: none), and with ``sink`` one more key of score 0 without a value."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot: int
+    scale: float
+    q_norm: Optional[torch.Tensor] = None
+    k_norm: Optional[torch.Tensor] = None
+    softcap: float = 0.0
+    window: int = 0
+    chunk: int = 0
+    sink: bool = False
+    eps: float = 1e-6
+    out_scale: float = 1.0
+
+    @property
+    def kv_row(self) -> int:
+        return self.kv_heads * (self.dim + self.vdim)
