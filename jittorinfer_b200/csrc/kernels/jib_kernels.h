@@ -233,12 +233,14 @@ typedef struct jib_state_mix {
     const int * seq_slots, * positions, * q_start;
     int * status;
     float * qk, * v, * dec, * s, * o;      // scratch: [T][2][H / rep][K], [T][H][V], [T][H][K] (SSD [T][H]), [T][H], [T][H][V]
-    long long ld, ld_dec, ld_gate, ldy;
+    void * chunk;              // null, or chunk_bytes >= jib_state_chunk_bytes: portions of bf16 go through the tensor cores (then qk, dec unused)
+    long long ld, ld_dec, ld_gate, ldy, chunk_bytes;
     int kind, H, K, V, rep, taps, conv0, n_conv, q_off, k_off, v_off, s_off, norm_groups, n_state, n_seqs, T;
     float q_scale, inv_tau, eps, out_scale;
 } jib_state_mix;
 // single: one token per sequence (row t = sequence t; scratch only for SSD: o).  K <= 512.
 JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, void * stream);
+JIB_EXPORT long long jib_state_chunk_bytes(const jib_state_mix * m);
 
 // ---- expert-parallel all-to-all over peer memory (ep_alltoall.cu); ctx is a JibEpCtx (ep_alltoall.h) ---------
 JIB_EXPORT int jib_ep_plan(const int * ids, int T, int k, const struct JibEpCtx * ctx, int site, int * seg, int * pair_dst, void * stream);

@@ -1,0 +1,681 @@
+// Portions through the matrix-state mixers on tensor cores (bf16 activations, K of 64 or 128, V a multiple of 16).
+//
+// Within a chunk of 32 tokens, with G_t the running sum of the log decays (G_t <= 0) and S the state before the chunk:
+//
+//   o_t = S^T (q_t e^{G_t}) + sum_{s <= t} A_ts u_s         A_ts = sum_c q_tc k_sc e^{G_tc - G_sc}
+//   S'  = e^{G_C} S + sum_s (k_s e^{G_C - G_s}) u_s^T
+//   DELTA: u = b (v - .) is the solution of a triangular system, (1 + b B) u = b (v - S^T (k e^{G})) with B_ts = sum_c k_tc k_sc e^{G_tc - G_sc},
+//   s < t:  u = U0 - W S with W = (1 + b B)^-1 b (k e^{G}), U0 = (1 + b B)^-1 b v.
+//
+// Every exponent that occurs is a difference G_t - G_s with s <= t and so at most 0, however fast the decay: nothing overflows and no
+// quotient of vanishing products is formed.
+//   prepare (one CTA per chunk and head; SSD: per chunk and group): convolution, unit norm, decays, A, W, U0.  Independent of S.
+//   pass    (one CTA per head and 16 value columns): walks the chunks, S in registers, everything else a product of small matrices.
+// State, decays, A, W, U0 are fp32; the tensor cores see each as a sum of two bf16 numbers and the products hi * hi + hi * lo + lo * hi
+// (about 16 bits of mantissa); q and k of SSD are bf16 to begin with.  Accumulation is fp32.
+#include "pdl.cuh"
+#include "state_mix.cuh"
+
+namespace {
+
+using namespace state_mix;
+
+constexpr int C = 32, VB = 16, NT = 256, STAGES = 3;
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int QK_LD = 40;                                    // row stride of SSD's q . k table (fp32)
+
+// A chunk's record: bf16 tiles of 32 rows x K columns in 16-byte units u of row r stored at u ^ (r & 7); A: 32 x 32, unit u ^ (r / 2 & 3).
+template <int KIND, int K> struct Rec {
+    static constexpr int TILE = C * K * 2, ATILE = C * C * 2;
+    static constexpr int Q = 0, D = KIND == SSD ? TILE : 2 * TILE;                        // q e^G, k e^{G_C - G} (SSD: q, k)
+    static constexpr int A = KIND == SSD ? 2 * TILE : 4 * TILE;                           // hi, lo (SSD: q . k fp32)
+    static constexpr int W = A + 2 * ATILE;                                               // DELTA
+    static constexpr int E = W + (KIND == DELTA ? 2 * TILE : 0);                          // e^{G_C}
+    static constexpr int BYTES = KIND == SSD ? A + C * QK_LD * 4 : E + K * 4;
+};
+
+// run index: sequence b's chunks start at q_start[b] / C + b; indices in the gaps have no tokens
+__device__ __forceinline__ int chunk_key(const int * q_start, int b) { return q_start[b] / C + b; }
+__device__ __forceinline__ int chunk_seq(const jib_state_mix & a, int ci) {
+    int b = 0, hi = a.n_seqs;
+    while (hi - b > 1) {
+        const int mid = (b + hi) >> 1;
+        if (chunk_key(a.q_start, mid) <= ci) b = mid; else hi = mid;
+    }
+    return b;
+}
+
+__device__ __forceinline__ void load4(const bf16 * p, float (&v)[4]) {
+    const uint2 r = *(const uint2 *) p;
+    const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &r.x), y = __bfloat1622float2(*(const __nv_bfloat162 *) &r.y);
+    v[0] = x.x; v[1] = x.y; v[2] = y.x; v[3] = y.y;
+}
+// 4 columns from column c on of tokens i0 .. i0 + 7 of a range (its first token: row q0, position p0; n tokens): convolved and silu'd.
+// Up to 4 taps; every row is loaded once, all loads in flight together.  Rows past the range are zero.
+__device__ __forceinline__ void conv_run(const jib_state_mix & a, int q0, int p0, int n, int i0, int c, int slot, float (&out)[8][4]) {
+    const bf16 * x = (const bf16 *) a.proj + (size_t) q0 * a.ld + c;
+    float v[11][4];
+#pragma unroll
+    for (int r = 0; r < 11; ++r) {
+        const int i = i0 + r - 3;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[r][e] = 0.f;
+        if (r < 3 && 3 - r >= a.taps) continue;              // further back than the filter reaches
+        if (i >= 0 && i < n) load4(x + (long long) i * a.ld, v[r]);
+        else if (i < 0 && slot >= 0 && p0 + i >= 0)
+            load4((const bf16 *) a.conv_state + ((size_t) slot * a.taps + (p0 + i) % a.taps) * a.n_conv + c - a.conv0, v[r]);
+    }
+    if (a.taps == 0) {
+#pragma unroll
+        for (int r = 0; r < 8; ++r)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) out[r][e] = v[r + 3][e];
+        return;
+    }
+    float4 w[4], b = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        w[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j >= 4 - a.taps) w[j] = *(const float4 *) (a.conv_w + (size_t) (j - (4 - a.taps)) * a.n_conv + c - a.conv0);
+    }
+    if (a.conv_b != nullptr) b = *(const float4 *) (a.conv_b + c - a.conv0);
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+        float acc[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            acc[0] += w[j].x * v[r + j][0];
+            acc[1] += w[j].y * v[r + j][1];
+            acc[2] += w[j].z * v[r + j][2];
+            acc[3] += w[j].w * v[r + j][3];
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) out[r][e] = i0 + r < n ? silu<bf16>(acc[e]) : 0.f;
+    }
+}
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// x = hi + lo, both bf16; two numbers packed
+__device__ __forceinline__ void split2(float x, float y, uint32_t & hi, uint32_t & lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const float2 f = __bfloat1622float2(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
+    hi = *(const uint32_t *) &h;
+    lo = *(const uint32_t *) &l;
+}
+template <int K> __device__ __forceinline__ int tile_off(int r, int c) { return r * (K * 2) + (((c >> 3) ^ (r & 7)) << 4) + (c & 7) * 2; }
+__device__ __forceinline__ int a_off(int r, int c) { return r * 64 + (((c >> 3) ^ ((r >> 1) & 3)) << 4) + (c & 7) * 2; }
+template <int K> __device__ __forceinline__ void put_tile4(uint8_t * hi, int r, int c, float4 v) {
+    uint2 h, l;
+    split2(v.x, v.y, h.x, l.x);
+    split2(v.z, v.w, h.y, l.y);
+    *(uint2 *) (hi + tile_off<K>(r, c)) = h;
+    *(uint2 *) (hi + C * K * 2 + tile_off<K>(r, c)) = l;
+}
+
+// ---- prepare: DELTA, LINEAR ------------------------------------------------------------------------------------------------------
+template <int K> constexpr int prep_smem(int V) { return 4 * (3 * C * (K + 4) + C * (V + 4) + C * 36 + 3 * C); }
+
+template <int KIND, int K>
+__global__ void __launch_bounds__(NT) chunk_prepare_kernel(const __grid_constant__ jib_state_mix a) {
+    using R = Rec<KIND, K>;
+    constexpr int KS = K + 4;
+    extern __shared__ __align__(16) float sm[];
+    PDL_TRIGGER_TOP();
+    const int V = a.V, VS = V + 4, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    float * q = sm, * k = q + C * KS, * G = k + C * KS, * v = G + C * KS, * B = v + C * VS, * beta = B + C * 36, * norm = beta + C;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int ci = blockIdx.x, h = blockIdx.y, b = chunk_seq(a, ci);
+    const int r0 = a.q_start[b], nr = a.q_start[b + 1] - r0, t0 = (ci - chunk_key(a.q_start, b)) * C;
+    if (t0 < 0 || t0 >= nr) return;
+    const int p0 = a.positions[r0], n = min(C, nr - t0);
+    const int slot = a.taps > 0 ? checked_slot(a, b, 45) : -1;
+    // inputs: 8 tokens x 4 columns per job
+    const int jk = K / 4 * (C / 8), jv = V / 4 * (C / 8);
+    for (int j = tid; j < 3 * jk + jv; j += NT) {
+        float x[8][4];
+        float * dst;
+        int ld, col, run;
+        if (j < 2 * jk + jv) {
+            const int jj = j < jk ? j : j < 2 * jk ? j - jk : j - 2 * jk, w = j < 2 * jk ? K / 4 : V / 4;
+            col = jj % w * 4;
+            run = jj / w * 8;
+            ld = j < 2 * jk ? KS : VS;
+            dst = j < jk ? q : j < 2 * jk ? k : v;
+            conv_run(a, r0, p0, nr, t0 + run, (j < jk ? a.q_off + h / a.rep * K : j < 2 * jk ? a.k_off + h / a.rep * K : a.v_off + h * V) + col, slot, x);
+        } else {
+            const int jj = j - 2 * jk - jv;
+            col = jj % (K / 4) * 4;
+            run = jj / (K / 4) * 8;
+            ld = KS;
+            dst = G;
+            const bf16 * z = (const bf16 *) a.dec_in + (size_t) (r0 + t0) * a.ld_dec + h * K + col;
+            const float4 bias = *(const float4 *) (a.bias + h * K + col);
+            const float f = LOG2E * (KIND == DELTA ? a.neg_a[h] : -a.inv_tau);
+#pragma unroll
+            for (int r = 0; r < 8; ++r) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) x[r][e] = 0.f;
+                if (run + r < n) load4(z + (size_t) (run + r) * a.ld_dec, x[r]);
+            }
+#pragma unroll
+            for (int r = 0; r < 8; ++r) {
+                const float s = KIND == DELTA ? 1.f : -1.f;
+                x[r][0] = run + r < n ? f * softplus(s * (x[r][0] + bias.x)) : 0.f;
+                x[r][1] = run + r < n ? f * softplus(s * (x[r][1] + bias.y)) : 0.f;
+                x[r][2] = run + r < n ? f * softplus(s * (x[r][2] + bias.z)) : 0.f;
+                x[r][3] = run + r < n ? f * softplus(s * (x[r][3] + bias.w)) : 0.f;
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < 8; ++r) *(float4 *) (dst + (run + r) * ld + col) = make_float4(x[r][0], x[r][1], x[r][2], x[r][3]);
+    }
+    if (KIND == DELTA && tid < C)
+        beta[tid] = tid < n ? head_factor<DELTA>(a, to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + tid) * a.ld + a.s_off + h]), h) : 0.f;
+    __syncthreads();
+    // unit norms (folded into q and k) and running sums of the log decays
+    if (KIND == DELTA) {
+        for (int r = warp; r < 2 * C; r += NT / 32) {
+            const float * x = (r < C ? q : k) + (r & (C - 1)) * KS;
+            float ss = 0.f;
+            for (int c = lane; c < K; c += 32) ss += x[c] * x[c];
+            ss = warp_sum(ss);
+            if (lane == 0) norm[r] = rsqrtf(ss + 1e-6f) * (r < C ? a.q_scale : 1.f);
+        }
+    } else if (tid < 2 * C) {
+        norm[tid] = tid < C ? a.q_scale : 1.f;
+    }
+    for (int c = tid; c < K; c += NT) {
+        float g[C], s = 0.f;
+#pragma unroll
+        for (int t = 0; t < C; ++t) g[t] = G[t * KS + c];
+#pragma unroll
+        for (int t = 0; t < C; ++t) {
+            s += g[t];
+            G[t * KS + c] = s;
+        }
+    }
+    __syncthreads();
+    for (int i = tid; i < 2 * C * (K / 4); i += NT) {
+        const int r = i / (K / 4), c = i % (K / 4) * 4;
+        float4 * x = (float4 *) ((r < C ? q : k) + (r & (C - 1)) * KS + c);
+        const float s = norm[r];
+        float4 y = *x;
+        y.x *= s; y.y *= s; y.z *= s; y.w *= s;
+        *x = y;
+    }
+    __syncthreads();
+    uint8_t * rec = (uint8_t *) a.chunk + ((size_t) ci * a.H + h) * (R::BYTES + C * 4 * V);
+    // A and B: one thread per pair s < t (rows i and C - 1 - i together have C - 1 of them)
+    for (int i = tid; i < C * (C - 1) / 2; i += NT) {
+        const int i1 = i / (C - 1), j = i % (C - 1);
+        const int t = j < i1 ? i1 : C - 1 - i1, s = j < i1 ? j : j - i1;
+        const float * qt = q + t * KS, * kt = k + t * KS, * gt = G + t * KS, * ks = k + s * KS, * gs = G + s * KS;
+        float aq = 0.f, ak = 0.f;
+#pragma unroll 4
+        for (int c = 0; c < K; c += 4) {
+            const float4 x = *(const float4 *) (gt + c), y = *(const float4 *) (gs + c), z = *(const float4 *) (ks + c), u = *(const float4 *) (qt + c);
+            const float e0 = z.x * ex2(x.x - y.x), e1 = z.y * ex2(x.y - y.y), e2 = z.z * ex2(x.z - y.z), e3 = z.w * ex2(x.w - y.w);
+            aq += u.x * e0 + u.y * e1 + u.z * e2 + u.w * e3;
+            if (KIND == DELTA) {
+                const float4 w = *(const float4 *) (kt + c);
+                ak += w.x * e0 + w.y * e1 + w.z * e2 + w.w * e3;
+            }
+        }
+        if (KIND == DELTA) B[t * 36 + s] = ak * beta[t];
+        const bf16 hi = __float2bfloat16(aq);
+        *(bf16 *) (rec + R::A + a_off(t, s)) = hi;
+        *(bf16 *) (rec + R::A + R::ATILE + a_off(t, s)) = __float2bfloat16(aq - to_f(hi));
+        *(bf16 *) (rec + R::A + a_off(s, t)) = __float2bfloat16(0.f);
+        *(bf16 *) (rec + R::A + R::ATILE + a_off(s, t)) = __float2bfloat16(0.f);
+    }
+    for (int t = warp; t < C; t += NT / 32) {                // the diagonal
+        float d = 0.f;
+        for (int c = lane; c < K; c += 32) d += q[t * KS + c] * k[t * KS + c];
+        d = warp_sum(d);
+        if (lane == 0) {
+            const bf16 hi = __float2bfloat16(d);
+            *(bf16 *) (rec + R::A + a_off(t, t)) = hi;
+            *(bf16 *) (rec + R::A + R::ATILE + a_off(t, t)) = __float2bfloat16(d - to_f(hi));
+        }
+    }
+    for (int i = tid; i < C * (K / 4); i += NT) {            // q e^G, k e^{G_C - G}
+        const int t = i / (K / 4), c = i % (K / 4) * 4;
+        const float4 g = *(const float4 *) (G + t * KS + c), e = *(const float4 *) (G + (C - 1) * KS + c);
+        const float4 x = *(const float4 *) (q + t * KS + c), y = *(const float4 *) (k + t * KS + c);
+        put_tile4<K>(rec + R::Q, t, c, make_float4(x.x * ex2(g.x), x.y * ex2(g.y), x.z * ex2(g.z), x.w * ex2(g.w)));
+        put_tile4<K>(rec + R::D, t, c, make_float4(y.x * ex2(e.x - g.x), y.y * ex2(e.y - g.y), y.z * ex2(e.z - g.z), y.w * ex2(e.w - g.w)));
+    }
+    for (int c = tid; c < K; c += NT) ((float *) (rec + R::E))[c] = ex2(G[(C - 1) * KS + c]);
+    float * U = (float *) (rec + R::BYTES);
+    if (KIND == LINEAR) {
+        for (int i = tid; i < C * V; i += NT) {
+            const int t = i / V, c = i % V;
+            U[(c >> 4) * (C * VB) + t * VB + (c & 15)] = v[t * VS + c];
+        }
+        return;
+    }
+    __syncthreads();
+    // forward substitution, one right-hand side per thread: columns of k e^G, then of v
+    for (int c = tid; c < K + V; c += NT) {
+        float x[C];
+#pragma unroll
+        for (int t = 0; t < C; ++t) x[t] = beta[t] * (c < K ? k[t * KS + c] * ex2(G[t * KS + c]) : v[t * VS + c - K]);
+#pragma unroll
+        for (int t = 1; t < C; ++t) {
+            float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+            for (int s = 0; s < t; s += 4) {
+                const float4 w = *(const float4 *) (B + t * 36 + s);
+                s0 += w.x * x[s];
+                if (s + 1 < t) s1 += w.y * x[s + 1];
+                if (s + 2 < t) s0 += w.z * x[s + 2];
+                if (s + 3 < t) s1 += w.w * x[s + 3];
+            }
+            x[t] -= s0 + s1;
+        }
+        if (c < K) {
+#pragma unroll
+            for (int t = 0; t < C; ++t) {
+                const bf16 hi = __float2bfloat16(x[t]);
+                *(bf16 *) (rec + R::W + tile_off<K>(t, c)) = hi;
+                *(bf16 *) (rec + R::W + R::TILE + tile_off<K>(t, c)) = __float2bfloat16(x[t] - to_f(hi));
+            }
+        } else {
+            const int cc = c - K;
+#pragma unroll
+            for (int t = 0; t < C; ++t) U[(cc >> 4) * (C * VB) + t * VB + (cc & 15)] = x[t];
+        }
+    }
+}
+
+// ---- prepare: SSD ------------------------------------------------------------------------------------------------------------------
+// blockIdx.y < groups: q and k tiles of a group and their products; then runs of 256 value columns (bf16 into a.v), then the factors.
+template <int K>
+__global__ void __launch_bounds__(NT) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
+    using R = Rec<SSD, K>;
+    constexpr int KS = K + 4;
+    extern __shared__ __align__(16) float sm[];
+    PDL_TRIGGER_TOP();
+    const int tid = threadIdx.x, groups = a.H / a.rep, inner = a.H * a.V;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int ci = blockIdx.x, b = chunk_seq(a, ci);
+    const int r0 = a.q_start[b], nr = a.q_start[b + 1] - r0, t0 = (ci - chunk_key(a.q_start, b)) * C;
+    if (t0 < 0 || t0 >= nr) return;
+    const int p0 = a.positions[r0], n = min(C, nr - t0);
+    const int slot = a.taps > 0 ? checked_slot(a, b, 45) : -1;
+    int y = blockIdx.y;
+    if (y < groups) {
+        float * q = sm, * k = sm + C * KS;
+        uint8_t * rec = (uint8_t *) a.chunk + ((size_t) ci * groups + y) * R::BYTES;
+        const int jk = K / 4 * (C / 8);
+        for (int j = tid; j < 2 * jk; j += NT) {
+            float x[8][4];
+            const int jj = j < jk ? j : j - jk, col = jj % (K / 4) * 4, run = jj / (K / 4) * 8;
+            conv_run(a, r0, p0, nr, t0 + run, (j < jk ? a.q_off : a.k_off) + y * K + col, slot, x);
+#pragma unroll
+            for (int r = 0; r < 8; ++r) {
+                __nv_bfloat162 v[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
+                *(uint2 *) (rec + (j < jk ? R::Q : R::D) + tile_off<K>(run + r, col)) = *(const uint2 *) v;
+                const float2 f0 = __bfloat1622float2(v[0]), f1 = __bfloat1622float2(v[1]);
+                *(float4 *) ((j < jk ? q : k) + (run + r) * KS + col) = make_float4(f0.x, f0.y, f1.x, f1.y);
+            }
+        }
+        __syncthreads();
+        for (int i = tid; i < C * C; i += NT) {
+            const int t = i / C, s = i % C;
+            if (s > t) continue;
+            float d = 0.f;
+#pragma unroll 4
+            for (int c = 0; c < K; c += 4) {
+                const float4 x = *(const float4 *) (q + t * KS + c), z = *(const float4 *) (k + s * KS + c);
+                d += x.x * z.x + x.y * z.y + x.z * z.z + x.w * z.w;
+            }
+            ((float *) (rec + R::A))[t * QK_LD + s] = d;
+        }
+        return;
+    }
+    y -= groups;
+    const int vblocks = (inner + 255) / 256;
+    if (y < vblocks) {
+        const int col = y * 256 + (tid & 63) * 4, run = (tid >> 6) * 8;
+        if (col >= inner) return;
+        float x[8][4];
+        conv_run(a, r0, p0, nr, t0 + run, a.v_off + col, slot, x);
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+            if (run + r >= n) break;
+            __nv_bfloat162 v[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
+            *(uint2 *) ((bf16 *) a.v + (size_t) (r0 + t0 + run + r) * inner + col) = *(const uint2 *) v;
+        }
+        return;
+    }
+    for (int i = tid; i < n * a.H; i += NT) {
+        const size_t row = r0 + t0 + i / a.H;
+        const int h = i % a.H;
+        a.s[row * a.H + h] = head_factor<SSD>(a, to_f(((const bf16 *) a.proj)[row * a.ld + a.s_off + h]), h);
+    }
+}
+
+// ---- pass --------------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&x)[4], uint32_t y0, uint32_t y1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(x[0]), "r"(x[1]), "r"(x[2]), "r"(x[3]), "r"(y0), "r"(y1));
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
+constexpr int BS = 24;                                       // row stride of the [.][VB] bf16 operands (48 bytes: rows hit different banks)
+
+template <int KIND, int K> struct Pass {
+    using R = Rec<KIND, K>;
+    static constexpr int X = (R::BYTES + 15) / 16 * 16;      // U0 fp32 [C][VB] (SSD: x bf16 [C][VB]), then SSD's factors fp32 [C]
+    static constexpr int STAGE = X + (KIND == SSD ? C * VB * 2 + C * 4 : C * VB * 4);
+    static constexpr int S = STAGES * STAGE;                 // S hi, lo [K][BS]
+    static constexpr int U = S + 2 * K * BS * 2;             // U hi, lo [C][BS] (SSD: then the decayed ones)
+    static constexpr int SMEM = U + (KIND == SSD ? 4 : 2) * C * BS * 2;
+};
+
+template <int KIND, int K>
+__global__ void __launch_bounds__(NT) chunk_pass_kernel(const __grid_constant__ jib_state_mix a) {
+    using R = Rec<KIND, K>;
+    using P = Pass<KIND, K>;
+    constexpr int TPW = K / 64;                              // 16 x 8 tiles of S per warp: K / 16 x 2 tiles over 8 warps
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int splits = a.V / VB, h = blockIdx.x / splits, vs = blockIdx.x % splits, b = blockIdx.y, V = a.V, H = a.H;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
+    if (n <= 0) return;
+    const int slot = checked_slot(a, b, 46);
+    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
+    const int chunks = (n + C - 1) / C, c0 = chunk_key(a.q_start, b);
+    auto stage = [&](int i) {
+        if (i < chunks) {
+            uint8_t * dst = smem + i % STAGES * P::STAGE;
+            if (KIND == SSD) {
+                const int groups = H / a.rep, m = min(C, n - i * C);
+                const uint8_t * src = (const uint8_t *) a.chunk + ((size_t) (c0 + i) * groups + h / a.rep) * R::BYTES;
+                for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
+                const size_t row = r0 + i * C;
+                if (tid < 2 * m) cp16(dst + P::X + tid * 16, (const bf16 *) a.v + (row + (tid >> 1)) * H * V + h * V + vs * VB + (tid & 1) * 8);
+                if (tid < m) cp4(dst + P::X + C * VB * 2 + tid * 4, a.s + (row + tid) * H + h);
+            } else {
+                const uint8_t * src = (const uint8_t *) a.chunk + ((size_t) (c0 + i) * H + h) * (R::BYTES + C * 4 * V);
+                for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
+                if (tid < C * VB / 4) cp16(dst + P::X + tid * 16, src + R::BYTES + vs * (C * VB * 4) + tid * 16);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int i = 0; i < STAGES - 1; ++i) stage(i);
+
+    bf16 * Sh = (bf16 *) (smem + P::S), * Uh = (bf16 *) (smem + P::U);
+    const uint32_t S_addr = sm100::smem_u32(Sh), U_addr = sm100::smem_u32(Uh);
+    constexpr uint32_t S_LO = K * BS * 2, U_LO = C * BS * 2;
+    const int fr = lane >> 2, fc = (lane & 3) * 2;           // accumulator element: rows fr, fr + 8, columns fc, fc + 1
+    // ldmatrix lane addresses: operand rows (x4: 16 rows x 2 units), transposed ones
+    const int lr = lane & 15, lu = lane >> 4;
+    const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;         // k^T tiles: rows = tokens
+    const int br = lane & 31;                                // [k][n] operands: 32 rows of one 8-column unit
+    float st[TPW][4];
+    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K) * V + vs * VB;
+    const bool past = slot >= 0 && a.positions[r0] > 0;
+#pragma unroll
+    for (int i = 0; i < TPW; ++i) {
+        const int m = (warp * TPW + i) >> 1, nt = (warp * TPW + i) & 1;
+        const float * p = state + (size_t) (m * 16 + fr) * V + nt * 8 + fc;
+        const float2 x = past ? *(const float2 *) p : make_float2(0.f, 0.f), y = past ? *(const float2 *) (p + (size_t) 8 * V) : make_float2(0.f, 0.f);
+        st[i][0] = x.x; st[i][1] = x.y; st[i][2] = y.x; st[i][3] = y.y;
+    }
+    auto publish_state = [&]() {
+#pragma unroll
+        for (int i = 0; i < TPW; ++i) {
+            const int m = (warp * TPW + i) >> 1, nt = (warp * TPW + i) & 1;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                uint32_t hi, lo;
+                split2(st[i][2 * e], st[i][2 * e + 1], hi, lo);
+                bf16 * p = Sh + (m * 16 + fr + 8 * e) * BS + nt * 8 + fc;
+                *(uint32_t *) p = hi;
+                *(uint32_t *) (p + K * BS) = lo;
+            }
+        }
+    };
+    publish_state();
+    const int mt = (warp >> 1) & 1, nt = warp & 1;           // this warp's 16 x 8 tile of o (warps 0 - 3) or u (4 - 7)
+    const bool is_o = warp < 4;
+    const float na = KIND == SSD ? a.neg_a[h] * LOG2E : 0.f, skip = KIND == SSD ? a.skip[h] : 0.f;
+
+    for (int ch = 0; ch < chunks; ++ch) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+        __syncthreads();                                     // this chunk's record and S are there; the buffer before it is free
+        stage(ch + STAGES - 1);
+        const uint8_t * rec = smem + ch % STAGES * P::STAGE;
+        const uint32_t rec_addr = sm100::smem_u32(rec);
+        const int m = min(C, n - ch * C);
+        float g = 0.f;                                       // SSD: lane t holds G_t
+        if (KIND == SSD) {
+            g = lane < m ? na * ((const float *) (rec + P::X + C * VB * 2))[lane] : 0.f;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float x = __shfl_up_sync(0xffffffffu, g, o);
+                if (lane >= o) g += x;
+            }
+        }
+        float acc[3][4];
+#pragma unroll
+        for (int i = 0; i < 3; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+        if (is_o || KIND == DELTA) {
+            const uint32_t base = rec_addr + (is_o ? R::Q : R::W);
+#pragma unroll
+            for (int kk = 0; kk < K / 32; ++kk) {            // 32 channels at a time
+                uint32_t bh[4], bl[4];
+                const uint32_t off = ((kk * 32 + br) * BS + nt * 8) * 2;
+                ldm4t(bh, S_addr + off);
+                ldm4t(bl, S_addr + S_LO + off);
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int r = mt * 16 + lr, u = kk * 4 + e * 2 + lu;
+                    uint32_t x[4];
+                    ldm4(x, base + r * (K * 2) + ((u ^ (r & 7)) << 4));
+                    mma(acc[0], x, bh[2 * e], bh[2 * e + 1]);
+                    mma(acc[1], x, bl[2 * e], bl[2 * e + 1]);
+                    if (KIND != SSD) {
+                        ldm4(x, base + R::TILE + r * (K * 2) + ((u ^ (r & 7)) << 4));
+                        mma(acc[2], x, bh[2 * e], bh[2 * e + 1]);
+                    }
+                }
+            }
+        }
+        float o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] = acc[0][e] + (acc[1][e] + acc[2][e]);
+        if (!is_o) {                                         // u of this chunk as an operand
+            const int t = mt * 16 + fr, c = nt * 8 + fc;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int row = t + 8 * e;
+                uint32_t hi, lo;
+                bf16 * p = Uh + row * BS + c;
+                if (KIND == SSD) {
+                    float2 x = make_float2(0.f, 0.f);
+                    float f = 0.f;
+                    if (row < m) {
+                        x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (row * VB + c) * 2));
+                        f = ((const float *) (rec + P::X + C * VB * 2))[row];
+                    }
+                    const float w = f * ex2(__shfl_sync(0xffffffffu, g, 31) - __shfl_sync(0xffffffffu, g, row));
+                    split2(x.x * f, x.y * f, hi, lo);
+                    *(uint32_t *) p = hi;
+                    *(uint32_t *) (p + C * BS) = lo;
+                    split2(x.x * w, x.y * w, hi, lo);
+                    *(uint32_t *) (p + 2 * C * BS) = hi;
+                    *(uint32_t *) (p + 3 * C * BS) = lo;
+                } else {
+                    const float2 x = *(const float2 *) (rec + P::X + (row * VB + c) * 4);
+                    split2(x.x - o[2 * e], x.y - o[2 * e + 1], hi, lo);
+                    *(uint32_t *) p = hi;
+                    *(uint32_t *) (p + C * BS) = lo;
+                }
+            }
+        }
+        __syncthreads();
+        if (is_o) {
+            float p[3][4];
+#pragma unroll
+            for (int i = 0; i < 3; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) p[i][e] = 0.f;
+            uint32_t bh[4], bl[4];
+            const uint32_t off = (br * BS + nt * 8) * 2;
+            ldm4t(bh, U_addr + off);
+            ldm4t(bl, U_addr + U_LO + off);
+            const float g0 = __shfl_sync(0xffffffffu, g, mt * 16 + fr), g1 = __shfl_sync(0xffffffffu, g, mt * 16 + fr + 8);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                uint32_t xh[4], xl[4];
+                if (KIND == SSD) {                           // A = q . k times the decay between the two tokens
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {            // rows fr + 8 (j & 1), columns 16 e + 8 (j >> 1) + fc
+                        const int t = mt * 16 + fr + 8 * (j & 1), s = e * 16 + 8 * (j >> 1) + fc;
+                        const float gt = (j & 1) ? g1 : g0, s0 = __shfl_sync(0xffffffffu, g, s), s1 = __shfl_sync(0xffffffffu, g, s + 1);
+                        const float2 x = *(const float2 *) (rec + R::A + (t * QK_LD + s) * 4);
+                        split2(s <= t ? x.x * ex2(gt - s0) : 0.f, s + 1 <= t ? x.y * ex2(gt - s1) : 0.f, xh[j], xl[j]);
+                    }
+                } else {
+                    const int r = mt * 16 + lr, u = e * 2 + lu;
+                    ldm4(xh, rec_addr + R::A + r * 64 + ((u ^ ((r >> 1) & 3)) << 4));
+                    ldm4(xl, rec_addr + R::A + R::ATILE + r * 64 + ((u ^ ((r >> 1) & 3)) << 4));
+                }
+                mma(p[0], xh, bh[2 * e], bh[2 * e + 1]);
+                mma(p[1], xh, bl[2 * e], bl[2 * e + 1]);
+                mma(p[2], xl, bh[2 * e], bh[2 * e + 1]);
+            }
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int t = mt * 16 + fr + 8 * e, c = nt * 8 + fc;
+                if (t >= m) continue;
+                float2 y = make_float2(p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]), p[0][2 * e + 1] + (p[1][2 * e + 1] + p[2][2 * e + 1]));
+                if (KIND == SSD) {
+                    const float w = ex2(e ? g1 : g0);
+                    const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (t * VB + c) * 2));
+                    y.x += w * o[2 * e] + skip * x.x;
+                    y.y += w * o[2 * e + 1] + skip * x.y;
+                } else {
+                    y.x += o[2 * e];
+                    y.y += o[2 * e + 1];
+                }
+                *(float2 *) (a.o + ((size_t) (r0 + ch * C + t) * H + h) * V + vs * VB + c) = y;
+            }
+        }
+        // S' = decay S + k^T u
+        const float gC = __shfl_sync(0xffffffffu, g, 31);
+#pragma unroll
+        for (int i = 0; i < TPW; ++i) {
+            const int sm_ = (warp * TPW + i) >> 1, sn = (warp * TPW + i) & 1;
+            uint32_t bh[4], bl[4];
+            const uint32_t off = (br * BS + sn * 8) * 2 + (KIND == SSD ? 2 * U_LO : 0);
+            ldm4t(bh, U_addr + off);
+            ldm4t(bl, U_addr + U_LO + off);
+            float e0, e1;
+            if (KIND == SSD) {
+                e0 = e1 = ex2(gC);
+            } else {
+                const float * E = (const float *) (rec + R::E) + sm_ * 16 + fr;
+                e0 = E[0];
+                e1 = E[8];
+            }
+            st[i][0] *= e0; st[i][1] *= e0; st[i][2] *= e1; st[i][3] *= e1;
+            float p1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int r = e * 16 + tr, u = sm_ * 2 + tu;
+                uint32_t x[4];
+                ldm4t(x, rec_addr + R::D + r * (K * 2) + ((u ^ (r & 7)) << 4));
+                mma(st[i], x, bh[2 * e], bh[2 * e + 1]);
+                mma(p1, x, bl[2 * e], bl[2 * e + 1]);
+                if (KIND != SSD) {
+                    ldm4t(x, rec_addr + R::D + R::TILE + r * (K * 2) + ((u ^ (r & 7)) << 4));
+                    mma(p1, x, bh[2 * e], bh[2 * e + 1]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[i][e] += p1[e];
+        }
+        publish_state();                                     // its readers of this chunk are behind the barrier above
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    PDL_TRIGGER_LATE();
+    if (slot >= 0) {
+#pragma unroll
+        for (int i = 0; i < TPW; ++i) {
+            const int m = (warp * TPW + i) >> 1, nt2 = (warp * TPW + i) & 1;
+            float * p = state + (size_t) (m * 16 + fr) * V + nt2 * 8 + fc;
+            *(float2 *) p = make_float2(st[i][0], st[i][1]);
+            *(float2 *) (p + (size_t) 8 * V) = make_float2(st[i][2], st[i][3]);
+        }
+    }
+}
+
+inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
+
+template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t s) {
+    const int nch = a.T / C + a.n_seqs;
+    static std::atomic<unsigned char> done1[jib::MAX_DEVICES], done2[jib::MAX_DEVICES];
+    if (KIND == SSD) {
+        constexpr int smem = 2 * C * (K + 4) * 4;
+        if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done1)) return JIB_E_LAUNCH;
+        JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(nch, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
+    } else {
+        const int smem = prep_smem<K>(a.V);
+        if (!jib::ensure_dyn_smem(chunk_prepare_kernel<KIND == SSD ? LINEAR : KIND, K>, prep_smem<K>(256), done1)) return JIB_E_LAUNCH;
+        JIB_LAUNCH((chunk_prepare_kernel<KIND == SSD ? LINEAR : KIND, K>), dim3(nch, a.H), NT, smem, s, a);
+    }
+    const int rc = launched();
+    if (rc) return rc;
+    if (!jib::ensure_dyn_smem(chunk_pass_kernel<KIND, K>, Pass<KIND, K>::SMEM, done2)) return JIB_E_LAUNCH;
+    // a plain launch: as a programmatic dependent its CTAs would settle wherever the last CTAs of prepare leave room, several to an SM
+    chunk_pass_kernel<KIND, K><<<dim3(a.H * (a.V / VB), a.n_seqs), NT, Pass<KIND, K>::SMEM, s>>>(a);
+    return launched();
+}
+
+long long rec_bytes(const jib_state_mix & a) {
+#define REC(KIND) (a.K == 64 ? Rec<KIND, 64>::BYTES : Rec<KIND, 128>::BYTES)
+    const long long nch = a.T / C + a.n_seqs;
+    if (a.kind == SSD) return nch * (a.H / a.rep) * REC(SSD);
+    return nch * a.H * ((a.kind == DELTA ? REC(DELTA) : REC(LINEAR)) + C * 4 * a.V);
+#undef REC
+}
+
+}  // namespace
+
+bool jib_state_chunk_ok(const jib_state_mix & a) {
+    const long long cols = a.ld | a.q_off | a.k_off | a.v_off | a.conv0 | a.n_conv | (a.kind == SSD ? 0 : a.ld_dec);
+    return (a.K == 64 || a.K == 128) && a.V % VB == 0 && a.V <= 256 && a.taps <= 4 && cols % 4 == 0 && ((uintptr_t) a.proj & 7) == 0 &&
+           (a.kind == SSD || ((uintptr_t) a.dec_in & 7) == 0) && a.H % a.rep == 0;
+}
+
+int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s) {
+    if (rec_bytes(a) > a.chunk_bytes) return JIB_E_SCRATCH;
+    switch (a.kind) {
+        case DELTA: return a.K == 64 ? run_chunks<DELTA, 64>(a, s) : run_chunks<DELTA, 128>(a, s);
+        case LINEAR: return a.K == 64 ? run_chunks<LINEAR, 64>(a, s) : run_chunks<LINEAR, 128>(a, s);
+        default: return a.K == 64 ? run_chunks<SSD, 64>(a, s) : run_chunks<SSD, 128>(a, s);
+    }
+}
+
+// Bytes of scratch (m->chunk) with which jib_state_mix_run takes a batch of portions through the tensor cores; 0: not these sizes.
+extern "C" JIB_EXPORT long long jib_state_chunk_bytes(const jib_state_mix * m) { return jib_state_chunk_ok(*m) ? rec_bytes(*m) : 0; }

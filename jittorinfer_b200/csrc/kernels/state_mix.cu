@@ -11,7 +11,8 @@
 // parts of the row.
 //
 // Single tokens (decode): state_step does all of it in one launch per layer (SSD: plus the gated norm of whole rows).
-// Portions: state_prep (convolution, unit norm, decays -> fp32), state_scan (the recurrence), state_finish (gate and norm).
+// Portions: state_prep (convolution, unit norm, decays -> fp32), state_scan (the recurrence, token by token), state_finish (gate and
+// norm); bf16 portions of the head sizes it is built for take state_chunk.cu in place of the first two.
 //
 // A sequence's state lives in row seq_slots[b] of [n_state][H][K][V]; its last convolution inputs in a ring [n_state][taps][channels]
 // whose row p % taps holds position p's.  A range that starts at position 0 starts from zeros whatever the rows hold, so slots are
@@ -23,70 +24,11 @@
 #include "jib_kernels.h"
 #include "pdl.cuh"
 #include "sm100.cuh"
+#include "state_mix.cuh"
 
 namespace {
 
-typedef __nv_bfloat16 bf16;
-enum { DELTA = JIB_STATE_DELTA, LINEAR = JIB_STATE_LINEAR, SSD = JIB_STATE_SSD };
-
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ void put(bf16 * p, float v) { *p = __float2bfloat16(v); }
-__device__ __forceinline__ void put(float * p, float v) { *p = v; }
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-// bf16 activations: fast exponential and division for gates and silu (a few ulp of fp32); fp32 ones: the accurate forms.
-template <typename T> __device__ __forceinline__ float sigmoid(float v);
-template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
-template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
-template <typename T> __device__ __forceinline__ float silu(float v) { return v * sigmoid<T>(v); }
-__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
-
-template <int KIND> __device__ __forceinline__ float channel_decay(const jib_state_mix & a, float z, int h) {
-    return KIND == DELTA ? expf(a.neg_a[h] * softplus(z)) : expf(-a.inv_tau * softplus(-z));
-}
-template <int KIND> __device__ __forceinline__ float head_factor(const jib_state_mix & a, float z, int h) {
-    return KIND == DELTA ? 1.f / (1.f + expf(-z)) : softplus(z + a.bias[h]);
-}
-
-__device__ __forceinline__ int seq_of(const int * q_start, int n_seqs, int t) {
-    int b = 0, hi = n_seqs;
-    while (hi - b > 1) {
-        const int mid = (b + hi) >> 1;
-        if (q_start[mid] <= t) b = mid; else hi = mid;
-    }
-    return b;
-}
-__device__ __forceinline__ int checked_slot(const jib_state_mix & a, int b, int site) {
-    const int slot = a.seq_slots[b];
-    if (slot >= a.n_state) {
-        if (threadIdx.x == 0) jib_report(a.status, JIB_ERR_BOUNDS, site, slot);
-        return -1;
-    }
-    return slot;
-}
-
-// Column c of token row t (position p, back rows of its range precede it in the batch): convolved and silu'd if c lies in the window.
-template <typename T>
-__device__ __forceinline__ float column(const jib_state_mix & a, int t, int c, int p, int back, int slot) {
-    const T * x = (const T *) a.proj + (size_t) t * a.ld + c;
-    if (a.taps == 0) return to_f(*x);
-    const int w = c - a.conv0;
-    float acc = a.conv_b != nullptr ? a.conv_b[w] : 0.f;
-    for (int j = 0; j < a.taps; ++j) {
-        const int d = a.taps - 1 - j;                        // tokens back
-        if (d > p) continue;
-        float v;
-        if (d <= back) v = to_f(x[-(long long) d * a.ld]);
-        else if (slot >= 0) v = to_f(((const T *) a.conv_state)[((size_t) slot * a.taps + (p - d) % a.taps) * a.n_conv + w]);
-        else continue;
-        acc += a.conv_w[(size_t) j * a.n_conv + w] * v;
-    }
-    return silu<T>(acc);
-}
+using namespace state_mix;
 
 // ---- portions: inputs of the recurrence in fp32 ------------------------------------------------------------------------------
 // qk [T][2][Hk][K], v [T][H][V], dec [T][H][K] (SSD: [T][H]), s [T][H].  One warp per (token, item); items: q heads, k heads,
@@ -150,24 +92,6 @@ __global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__
 // ahead.  Also stores the range's last convolution inputs (their old values were read by state_prep).
 constexpr int SCAN_NT = 128, SCAN_TT = 8;
 
-__device__ __forceinline__ void cp16(float * dst, const float * src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t) __cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp4(float * dst, const float * src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t) __cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-
-template <typename T>
-__device__ void store_conv_tail(const jib_state_mix & a, int slot, int q0, int n, int part, int parts) {
-    if (a.taps < 2 || slot < 0) return;
-    const int keep = min(n, a.taps - 1), p_end = a.positions[q0] + n;
-    for (int i = part * SCAN_NT + threadIdx.x; i < keep * a.n_conv; i += parts * SCAN_NT) {
-        const int d = i / a.n_conv + 1, w = i % a.n_conv;    // d tokens before the end of the range
-        ((T *) a.conv_state)[((size_t) slot * a.taps + (p_end - d) % a.taps) * a.n_conv + w] =
-            ((const T *) a.proj)[(size_t) (q0 + n - d) * a.ld + a.conv0 + w];
-    }
-}
-
 template <typename T, int KIND, int LK>
 __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_constant__ jib_state_mix a, int splits, int aligned) {
     constexpr int KP = LK * 16, VB = SCAN_NT / LK;
@@ -183,7 +107,7 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
     const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
     if (n <= 0) return;
     const int slot = checked_slot(a, b, 46);
-    store_conv_tail<T>(a, slot, q0, n, blockIdx.x, gridDim.x);
+    store_conv_tail<T>(a, slot, q0, n, blockIdx.x * SCAN_NT + threadIdx.x, gridDim.x * SCAN_NT);
     const bool mine = col < nv;
     float * st = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K) * V + v0 + col;
     float s[16];
@@ -520,7 +444,8 @@ int launch_scan(const jib_state_mix & a, cudaStream_t s) {
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(state_scan_kernel<T, KIND, LK>, SMEM, done)) return JIB_E_LAUNCH;
     const int splits = (a.V + VB - 1) / VB;
-    JIB_LAUNCH((state_scan_kernel<T, KIND, LK>), dim3(a.H * splits, a.n_seqs), SCAN_NT, SMEM, s, a, splits, a.K % 4 == 0);
+    // a plain launch: as a programmatic dependent its CTAs would settle wherever the last CTAs of state_prep leave room, several to an SM
+    state_scan_kernel<T, KIND, LK><<<dim3(a.H * splits, a.n_seqs), SCAN_NT, SMEM, s>>>(a, splits, a.K % 4 == 0);
     return launched();
 }
 
@@ -553,6 +478,10 @@ int run(const jib_state_mix & a, int single, cudaStream_t s) {
         if (vec == 4) return keep ? launch_step<T, KIND, 4, true>(a, nt, s) : launch_step<T, KIND, 4, false>(a, nt, s);
         return keep ? launch_step<T, KIND, 1, true>(a, nt, s) : launch_step<T, KIND, 1, false>(a, nt, s);
     }
+    if (sizeof(T) == 2 && a.chunk != nullptr && jib_state_chunk_ok(a)) {
+        const int rc = jib_state_chunk_run(a, s);
+        return rc ? rc : launch_finish<T, KIND>(a, s);
+    }
     const int items = 2 * (a.H / a.rep) + a.H + (KIND == LINEAR ? 0 : 1) + (KIND == SSD ? 0 : a.H);
     JIB_LAUNCH((state_prep_kernel<T, KIND>), dim3((items + 7) / 8, a.T), 256, 0, s, a);
     int rc = launched();
@@ -573,7 +502,7 @@ extern "C" JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single,
     if (a.T <= 0 || a.n_seqs <= 0) return 0;
     if (a.H < 1 || a.K < 1 || a.V < 1 || a.K > 32 * PREP_C || a.rep < 1 || a.H % a.rep || a.T > 65535 || a.n_seqs > 65535 ||
         (a.taps > 0 && (a.conv_state == nullptr || a.conv_w == nullptr)) || (a.kind == SSD && (a.norm_groups < 1 || (a.H * a.V) % a.norm_groups)) ||
-        (single && a.n_seqs != a.T) || (!single && (a.qk == nullptr || a.v == nullptr || a.dec == nullptr)) || (a.kind != LINEAR && !single && a.s == nullptr) ||
+        (single && a.n_seqs != a.T) || (!single && a.chunk == nullptr && (a.qk == nullptr || a.v == nullptr || a.dec == nullptr)) || (a.kind != LINEAR && !single && a.chunk == nullptr && a.s == nullptr) ||
         ((a.kind == SSD || !single) && a.o == nullptr))
         return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;

@@ -72,8 +72,8 @@ class RowTail(C.Structure):
 
 class StateMixDesc(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("proj", "dec_in", "gate", "y", "conv_state", "state", "conv_w", "conv_b", "bias", "neg_a", "skip", "norm_w",
-                                          "seq_slots", "positions", "q_start", "status", "qk", "v", "dec", "s", "o")] + \
-               [(n, C.c_longlong) for n in ("ld", "ld_dec", "ld_gate", "ldy")] + \
+                                          "seq_slots", "positions", "q_start", "status", "qk", "v", "dec", "s", "o", "chunk")] + \
+               [(n, C.c_longlong) for n in ("ld", "ld_dec", "ld_gate", "ldy", "chunk_bytes")] + \
                [(n, C.c_int) for n in ("kind", "H", "K", "V", "rep", "taps", "conv0", "n_conv", "q_off", "k_off", "v_off", "s_off", "norm_groups",
                                        "n_state", "n_seqs", "T")] + \
                [(n, C.c_float) for n in ("q_scale", "inv_tau", "eps", "out_scale")]
@@ -110,6 +110,7 @@ def load():
     sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, vp, vp)
     sig("jib_causal_conv", vp, fp, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
     sig("jib_mingru", vp, ll, fp, fp, fp, i, ip, ip, ip, i, i, i, i, i, vp, ip, vp)
+    L.jib_state_chunk_bytes.restype, L.jib_state_chunk_bytes.argtypes = C.c_longlong, [C.POINTER(StateMixDesc)]
     sig("jib_state_mix_run", C.POINTER(StateMixDesc), i, i, vp)
     sig("jib_gqa_qkv_post", C.POINTER(GqaDesc), vp, vp, vp, ll, fp, fp, fp, ip, vp, i, vp)
     sig("jib_gqa_attention", C.POINTER(GqaDesc), vp, vp, ll, vp, ll, i, i, i, vp)
@@ -741,6 +742,7 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 
 
 # ---- mixers described by a spec: matrix state per head (state_mix.cu), grouped-query attention (gqa_attention.cu) ----------------
+STATE_CHUNKS = os.environ.get("JIB_STATE_CHUNKS", "1") == "1"      # "0": portions token by token on CUDA cores (A/B)
 STATE_KINDS = {"delta": 0, "linear": 1, "ssd": 2}
 
 
@@ -749,48 +751,55 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     assert proj.stride(1) == 1 and gate.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype == gate.dtype
     assert state.dtype == torch.float32 and state.is_contiguous() and (m.taps == 0 or (conv_state.is_contiguous() and conv_state.dtype == proj.dtype))
     f32 = lambda *s: torch.empty(*s, dtype=torch.float32, device=proj.device)        # noqa: E731
-    d = StateMixDesc()
-    d.proj, d.ld, d.gate, d.ld_gate, d.y, d.ldy = proj.data_ptr(), proj.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
+    sd = StateMixDesc()
+    sd.proj, sd.ld, sd.gate, sd.ld_gate, sd.y, sd.ldy = proj.data_ptr(), proj.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
     if dec_in is not None:
         assert dec_in.stride(1) == 1 and dec_in.dtype == proj.dtype
-        d.dec_in, d.ld_dec = dec_in.data_ptr(), dec_in.stride(0)
-    d.conv_state, d.state, d.n_state = _p(conv_state), state.data_ptr(), state.shape[0]
-    d.conv_w, d.conv_b, d.bias, d.neg_a, d.skip, d.norm_w = _p(m.conv_w), _p(m.conv_b), _p(m.bias), _p(m.neg_a), _p(m.skip), _p(m.norm_w)
-    d.seq_slots, d.positions, d.q_start = seq_slots.data_ptr(), positions.data_ptr(), q_start.data_ptr()
-    d.status = workspace(proj.device).status.data_ptr()
-    d.kind, d.H, d.K, d.V, d.rep, d.taps, d.conv0 = STATE_KINDS[m.kind], H, K, V, m.rep, m.taps, m.conv0
-    d.n_conv = m.conv_w.shape[1] if m.conv_w is not None else 0
-    d.q_off, d.k_off, d.v_off, d.s_off, d.norm_groups = m.q_off, m.k_off, m.v_off, m.s_off, m.norm_groups
-    d.n_seqs, d.T = q_start.shape[0] - 1, T
-    d.q_scale, d.inv_tau, d.eps, d.out_scale = m.q_scale, m.inv_tau, m.eps, m.out_scale
+        sd.dec_in, sd.ld_dec = dec_in.data_ptr(), dec_in.stride(0)
+    sd.conv_state, sd.state, sd.n_state = _p(conv_state), state.data_ptr(), state.shape[0]
+    sd.conv_w, sd.conv_b, sd.bias, sd.neg_a, sd.skip, sd.norm_w = _p(m.conv_w), _p(m.conv_b), _p(m.bias), _p(m.neg_a), _p(m.skip), _p(m.norm_w)
+    sd.seq_slots, sd.positions, sd.q_start = seq_slots.data_ptr(), positions.data_ptr(), q_start.data_ptr()
+    sd.status = workspace(proj.device).status.data_ptr()
+    sd.kind, sd.H, sd.K, sd.V, sd.rep, sd.taps, sd.conv0 = STATE_KINDS[m.kind], H, K, V, m.rep, m.taps, m.conv0
+    sd.n_conv = m.conv_w.shape[1] if m.conv_w is not None else 0
+    sd.q_off, sd.k_off, sd.v_off, sd.s_off, sd.norm_groups = m.q_off, m.k_off, m.v_off, m.s_off, m.norm_groups
+    sd.n_seqs, sd.T = q_start.shape[0] - 1, T
+    sd.q_scale, sd.inv_tau, sd.eps, sd.out_scale = m.q_scale, m.inv_tau, m.eps, m.out_scale
     scratch = []
-    if not single:
+    n = 0 if single or proj.dtype == torch.float32 or not STATE_CHUNKS else load().jib_state_chunk_bytes(C.byref(sd))
+    if n > 0:                         # portions through the tensor cores
+        scratch = [torch.empty(n, dtype=torch.uint8, device=proj.device)]
+        sd.chunk, sd.chunk_bytes = scratch[0].data_ptr(), n
+        if m.kind == "ssd":
+            scratch += [torch.empty(T, H * V, dtype=proj.dtype, device=proj.device), f32(T, H)]
+            sd.v, sd.s = scratch[1].data_ptr(), scratch[2].data_ptr()
+    elif not single:
         scratch = [f32(T, 2 * (H // m.rep) * K), f32(T, H * V), f32(T, H * (1 if m.kind == "ssd" else K)), f32(T, H)]
-        d.qk, d.v, d.dec, d.s = (x.data_ptr() for x in scratch)
+        sd.qk, sd.v, sd.dec, sd.s = (x.data_ptr() for x in scratch)
     if not single or m.kind == "ssd":
         scratch.append(f32(T, H * V))
-        d.o = scratch[-1].data_ptr()
-    _ck(load().jib_state_mix_run(C.byref(d), int(single), int(proj.dtype == torch.float32), _stream()), "state_mix")
+        sd.o = scratch[-1].data_ptr()
+    _ck(load().jib_state_mix_run(C.byref(sd), int(single), int(proj.dtype == torch.float32), _stream()), "state_chunk" if n > 0 else "state_mix")
     return out
 
 
 def _gqa_desc(m, cache, T, n_seqs):
     assert cache.is_contiguous()
-    d = GqaDesc()
-    d.cache, d.n_slots, d.row, d.status = cache.data_ptr(), cache.shape[0], cache.shape[1], workspace(cache.device).status.data_ptr()
-    d.H, d.G, d.D, d.V, d.rot, d.T, d.n_seqs, d.block_size = m.heads, m.kv_heads, m.dim, m.vdim, m.rot, T, n_seqs, 64
-    d.window, d.chunk, d.sink = m.window, m.chunk, int(m.sink)
-    d.scale, d.softcap, d.eps, d.out_scale = m.scale, m.softcap, m.eps, m.out_scale
-    return d
+    gd = GqaDesc()
+    gd.cache, gd.n_slots, gd.row, gd.status = cache.data_ptr(), cache.shape[0], cache.shape[1], workspace(cache.device).status.data_ptr()
+    gd.H, gd.G, gd.D, gd.V, gd.rot, gd.T, gd.n_seqs, gd.block_size = m.heads, m.kv_heads, m.dim, m.vdim, m.rot, T, n_seqs, 64
+    gd.window, gd.chunk, gd.sink = m.window, m.chunk, int(m.sink)
+    gd.scale, gd.softcap, gd.eps, gd.out_scale = m.scale, m.softcap, m.eps, m.out_scale
+    return gd
 
 
 def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
     T = q.shape[0]
     assert q.dtype == cache.dtype and q.stride(1) == 1 and k.stride(0) == q.stride(0) == v.stride(0) and rope_table.is_contiguous()
     out = torch.empty(T, m.heads, m.dim, dtype=q.dtype, device=q.device)
-    d = _gqa_desc(m, cache, T, 1)
-    d.positions, d.max_pos = positions.data_ptr(), rope_table.shape[0]
-    _ck(load().jib_gqa_qkv_post(C.byref(d), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), m.q_norm.data_ptr(), m.k_norm.data_ptr(),
+    gd = _gqa_desc(m, cache, T, 1)
+    gd.positions, gd.max_pos = positions.data_ptr(), rope_table.shape[0]
+    _ck(load().jib_gqa_qkv_post(C.byref(gd), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), m.q_norm.data_ptr(), m.k_norm.data_ptr(),
                                 rope_table.data_ptr(), slot_mapping.data_ptr(), out.data_ptr(), int(q.dtype == torch.float32), _stream()), "gqa_qkv_post")
     return out
 
@@ -807,11 +816,11 @@ def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size
     T, H, D = q.shape
     assert q.dtype == cache.dtype == out.dtype and q.is_contiguous() and out.stride(1) == 1
     single = max_q_len == 1 and seq_lens.shape[0] == T
-    d = _gqa_desc(m, cache, T, seq_lens.shape[0])
-    d.block_tables, d.max_blocks, d.block_size = block_tables.data_ptr(), block_tables.stride(0), block_size
-    d.seq_lens, d.q_start = seq_lens.data_ptr(), q_start.data_ptr()
+    gd = _gqa_desc(m, cache, T, seq_lens.shape[0])
+    gd.block_tables, gd.max_blocks, gd.block_size = block_tables.data_ptr(), block_tables.stride(0), block_size
+    gd.seq_lens, gd.q_start = seq_lens.data_ptr(), q_start.data_ptr()
     splits = gqa_splits(m, T, block_tables.shape[1] * block_size, workspace(q.device).sm_count) if single else 1
-    _ck(load().jib_gqa_attention(C.byref(d), q.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), int(single),
+    _ck(load().jib_gqa_attention(C.byref(gd), q.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), int(single),
                                  splits, int(q.dtype == torch.float32), _stream()), "gqa_attention")
     return out
 
