@@ -119,25 +119,40 @@ __device__ __forceinline__ float ld_peer(const float * p, int rank) {
     return v;
 }
 
-// 4 elements c .. c + 3 of a row of n, zero past its end
-template <typename T> __device__ __forceinline__ float4 load4(const T * p, int c, int n, bool vec);
-template <> __device__ __forceinline__ float4 load4<float>(const float * p, int c, int n, bool vec) {
-    if (vec) return *(const float4 *) (p + c);
-    return make_float4(p[c], c + 1 < n ? p[c + 1] : 0.f, c + 2 < n ? p[c + 2] : 0.f, c + 3 < n ? p[c + 3] : 0.f);
-}
-template <> __device__ __forceinline__ float4 load4<bf16>(const bf16 * p, int c, int n, bool vec) {
-    if (vec) {
-        const uint2 r = *(const uint2 *) (p + c);
+// 4 elements c .. c + 3 of a row of n, zero past its end; kept as stored until they are needed (many loads in flight)
+template <typename T> struct Quad;
+template <> struct Quad<float> {
+    float4 r;
+    __device__ __forceinline__ void zero() { r = make_float4(0.f, 0.f, 0.f, 0.f); }
+    __device__ __forceinline__ void load(const float * p, int c, int n, bool vec) {
+        if (vec) r = *(const float4 *) (p + c);
+        else r = make_float4(p[c], c + 1 < n ? p[c + 1] : 0.f, c + 2 < n ? p[c + 2] : 0.f, c + 3 < n ? p[c + 3] : 0.f);
+    }
+    __device__ __forceinline__ float4 get() const { return r; }
+};
+template <> struct Quad<bf16> {
+    uint2 r;
+    __device__ __forceinline__ void zero() { r = make_uint2(0, 0); }
+    __device__ __forceinline__ void load(const bf16 * p, int c, int n, bool vec) {
+        if (vec) {
+            r = *(const uint2 *) (p + c);
+        } else {
+            const unsigned short * q = (const unsigned short *) p;
+            r.x = q[c] | (c + 1 < n ? (unsigned) q[c + 1] << 16 : 0u);
+            r.y = (c + 2 < n ? q[c + 2] : 0u) | (c + 3 < n ? (unsigned) q[c + 3] << 16 : 0u);
+        }
+    }
+    __device__ __forceinline__ float4 get() const {
         const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &r.x), y = __bfloat1622float2(*(const __nv_bfloat162 *) &r.y);
         return make_float4(x.x, x.y, y.x, y.y);
     }
-    return make_float4(to_f(p[c]), c + 1 < n ? to_f(p[c + 1]) : 0.f, c + 2 < n ? to_f(p[c + 2]) : 0.f, c + 3 < n ? to_f(p[c + 3]) : 0.f);
-}
+};
 
 template <typename T, int NVC>
 __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ gate,
                                                            long long ld_gate, T * __restrict__ out, long long ldo, int run, int heads, int KT) {
     extern __shared__ float smem[];
+    __shared__ int rows_s[64];
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int tid = threadIdx.x, D = a.D, V = a.V, rep = a.H / a.G;
@@ -165,7 +180,11 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
     for (int i = tid; i < ROWS * (DP / 4); i += NT) {
         const int r = i / (DP / 4), c = i % (DP / 4) * 4;
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < rows && c < D) x = load4<T>(q + ((size_t) (q0 + i0 + r / nh) * a.H + h0 + r % nh) * D, c, D, vec);
+        if (r < rows && c < D) {
+            Quad<T> k;
+            k.load(q + ((size_t) (q0 + i0 + r / nh) * a.H + h0 + r % nh) * D, c, D, vec);
+            x = k.get();
+        }
         x.x *= a.scale; x.y *= a.scale; x.z *= a.scale; x.w *= a.scale;
         *(float4 *) (qs + r * DP + c) = x;
     }
@@ -179,17 +198,30 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
     const int key = tid % KT, rg = tid / KT, rpt = ROWS * KT / NT;       // scores: this thread's key and its rpt rows
     for (int kt = k_lo; kt < k_hi; ++kt) {
         __syncthreads();
-        const int w4 = DP / 4 - 1 + VP / 4;
-        for (int i = tid; i < KT * w4; i += NT) {
-            const int j = i / w4, c = i % w4 * 4, p = kt * KT + j;
-            const bool is_k = c < DP - 4;
-            const int cc = is_k ? c : c - (DP - 4);
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (p < end && p >= lo) {
-                const T * row = (const T *) a.cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row;
-                x = load4<T>(is_k ? row + g * D : row + a.G * D + g * V, cc, is_k ? D : V, vec);
+        if (tid < KT) {                                      // where this tile's rows are
+            const int p = kt * KT + tid;
+            rows_s[tid] = p < end && p >= lo ? bt[p / a.block_size] * a.block_size + p % a.block_size : -1;
+        }
+        __syncthreads();
+        const int k4 = DP / 4 - 1, w4 = k4 + VP / 4;
+        constexpr int FLY = 8;
+        for (int i = tid; i < KT * w4; i += NT * FLY) {
+            Quad<T> x[FLY];
+#pragma unroll
+            for (int u = 0; u < FLY; ++u) {
+                const int e = i + u * NT, j = e / w4, c = e - j * w4;
+                x[u].zero();
+                const int slot = e < KT * w4 ? rows_s[j] : -1;
+                if (slot < 0) continue;
+                const T * row = (const T *) a.cache + (size_t) slot * a.row;
+                if (c < k4) x[u].load(row + g * D, 4 * c, D, vec);
+                else x[u].load(row + a.G * D + g * V, 4 * (c - k4), V, vec);
             }
-            *(float4 *) ((is_k ? ks + j * DP : vs + j * VP) + cc) = x;
+#pragma unroll
+            for (int u = 0; u < FLY; ++u) {
+                const int e = i + u * NT, j = e / w4, c = e - j * w4;
+                if (e < KT * w4) *(float4 *) (c < k4 ? ks + j * DP + 4 * c : vs + j * VP + 4 * (c - k4)) = x[u].get();
+            }
         }
         __syncthreads();
         float s[8];

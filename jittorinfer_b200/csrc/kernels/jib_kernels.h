@@ -147,7 +147,7 @@ JIB_EXPORT int jib_mla_flash(const void * q, const void * cache, long long n_slo
 // ---- prefill attention in the per-head form (mha_prefill_tcgen05.cu): head dims 128 + 64 (keys), 128 (values) ---------------
 // jib_kv_gather: lat [total_cap][row_elems] <- the cached latent rows of every sequence, in sequence order; kv_start [n_seqs].
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, void * lat, int * kv_start,
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, void * lat, int * kv_start,
                              int total_cap, void * stream);
 // q [T][H][192] (RoPE applied), kv [total][H][256] = k_nope | v, kpe [total][64] (row stride kpe_stride), out [T][H * 128].
 JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * kv, const void * kpe, long long kpe_stride, long long total,
@@ -213,6 +213,11 @@ JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * 
 // splits (<= 8): CTAs that share a row's keys.
 JIB_EXPORT int jib_gqa_attention(const jib_gqa * m, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single,
                                  int splits, int f32, void * stream);
+
+// The same for prompt chunks on tcgen05 tensor cores (mha_prefill_tcgen05.cu): bf16, D = V = 128.  kv [total][row]: the rows jib_kv_gather
+// copied; kv_start [n_seqs] the first of each sequence; n_q_tiles >= sum_b ceil(q_len_b / 128).
+JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * kv, long long total, const int * kv_start, const void * gate,
+                               long long ld_gate, int n_q_tiles, void * out, long long ldo, void * stream);
 
 // ---- mixers with a matrix state per head (state_mix.cu) ----------------------------------------------------------------------
 enum { JIB_STATE_DELTA = 0, JIB_STATE_LINEAR = 1, JIB_STATE_SSD = 2 };

@@ -20,12 +20,16 @@
 // Causality and sequence boundaries come from q_start / seq_lens; KV tiles below the diagonal skip the mask.  With a sliding
 // window (position i sees j with 0 <= i - j < window) only the rows some query of the chunk can see are gathered and
 // expanded, and a CTA starts at the KV tile that holds the first row its first query sees.
+// A second form of the same kernel (GQA) serves grouped-query attention: keys of 128 dims and values of 128 per key / value head, shared
+// by H / G query heads and gathered as they are cached (no expansion, no RoPE part of their own), with softcap, a sink, chunks counted
+// from position 0 and a gate per head.
 // All waits are bounded (sm100.cuh); no multicast.
 #include "sm100.cuh"
 
 #include <mutex>
 #include <string.h>
 
+#include "gqa_mask.cuh"
 #include "jib_kernels.h"
 #include "pdl.cuh"
 #include "timeline.cuh"
@@ -40,8 +44,12 @@ constexpr int DN = 128, DR = 64, DQK = DN + DR, DV = 128;
 constexpr int QT = 128;                       // query rows per CTA
 constexpr int KT = 128;                       // kv rows per tile
 constexpr int CHUNK = QT * 128;               // [128 rows][64 cols] bf16 with 128-byte rows
-constexpr int Q_BYTES = 3 * CHUNK, K_BYTES = 3 * CHUNK, V_BYTES = 2 * CHUNK, P_BYTES = 2 * CHUNK;
-constexpr int SMEM_BYTES = 1024 + Q_BYTES + 2 * K_BYTES + V_BYTES + P_BYTES + 256;
+constexpr int V_BYTES = 2 * CHUNK, P_BYTES = 2 * CHUNK;
+template <bool GQA> struct Form {
+    static constexpr int NC = GQA ? 2 : 3;    // 64-dim chunks of a query / key head
+    static constexpr int Q_BYTES = NC * CHUNK, K_BYTES = NC * CHUNK;
+    static constexpr int SMEM_BYTES = 1024 + Q_BYTES + 2 * K_BYTES + V_BYTES + P_BYTES + 256;
+};
 constexpr int TMEM_COLS = 512;                // S x2 (256) + O (128), rounded to a power of two
 constexpr int NUM_THREADS = 192;
 constexpr float RESCALE_LAG = 8.0f;           // log2 units the exponent base may lag behind the running maximum
@@ -56,21 +64,34 @@ struct MhaArgs {
     int n_seqs, T, H;
     int window;               // 0: none
     float scale_log2e;
+    // GQA
+    const bf16 * gate;        // null, or [T][ld_gate] pre-activations of a sigmoid per head
+    long long ld_gate;
+    int G, chunk, sink;
+    float cap_log2e, inv_cap2, out_scale;     // softcap * log2 e (0: none), 2 * scale * log2 e / softcap
 };
 
-// Rows of a sequence with S cached tokens that its last q_len tokens can see: the last min(S, q_len + window - 1).
-__host__ __device__ __forceinline__ int visible_rows(int S, int q_len, int window) {
-    if (window <= 0 || S <= 0) return S;
-    const long long need = (long long) q_len + window - 1;
-    return need < S ? (int) need : S;
+// Rows of a sequence with S cached tokens that its last q_len tokens can see: the last ...
+__host__ __device__ __forceinline__ int visible_rows(int S, int q_len, int window, int chunk) {
+    return S <= 0 ? S : S - gqa_first_key(S > q_len ? S - q_len : 0, window, chunk);
 }
 
+// softcap * tanh(score * scale / softcap) * log2 e from the raw product
+__device__ __forceinline__ float capped_log2(float s, const MhaArgs & a) {
+    return a.cap_log2e * (1.f - __fdividef(2.f, 1.f + exp2f(fminf(s * a.inv_cap2, 120.f))));
+}
+
+template <bool GQA>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                    const __grid_constant__ CUtensorMap tmPE, const MhaArgs a) {
+    using F = Form<GQA>;
+    constexpr int NC = F::NC, Q_BYTES = F::Q_BYTES, K_BYTES = F::K_BYTES;
     extern __shared__ uint8_t smem_raw[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y;
+    // columns of this head's keys and values in the gathered rows, and of its queries
+    const int kcol = GQA ? h / (a.H / a.G) * DN : h * (DN + DV), vcol = GQA ? a.G * DN + h / (a.H / a.G) * DV : h * (DN + DV) + DN, qcol = h * NC * 64;
 
     uint8_t * base = (uint8_t *) (((uintptr_t) smem_raw + 1023) & ~(uintptr_t) 1023);
     uint8_t * q_s = base;
@@ -101,7 +122,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         fence_barrier_init();
         prefetch_tmap(&tmQ);
         prefetch_tmap(&tmKV);
-        prefetch_tmap(&tmPE);
+        if (!GQA) prefetch_tmap(&tmPE);
     }
     // This kernel takes ALL tensor-memory columns of its SM, and tcgen05.alloc blocks until they are free.  So it asks for them
     // only after the grid before it has completed (a CTA of that grid that still had to start on this SM could never get
@@ -131,14 +152,15 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         }
     }
     // n_tiles KV tiles from tile kt0 on, in gathered coordinates (row 0 = the first row the chunk can see)
-    int n_tiles = 0, kt0 = 0, ctx0 = 0, kv0 = 0, rows = 0;
+    int n_tiles = 0, kt0 = 0, ctx0 = 0, kv0 = 0, rows = 0, base_pos = 0;      // base_pos: position of gathered row 0
     if (b >= 0) {
-        const int S = visible_rows(a.seq_lens[b], q_len, a.window);
+        const int S = visible_rows(a.seq_lens[b], q_len, a.window, a.chunk);
+        base_pos = a.seq_lens[b] - S;
         ctx0 = S - q_len;                             // gathered rows before this chunk
         kv0 = a.kv_start[b];
         rows = min(QT, q_len - tile * QT);            // valid query rows of the tile
         const int last_lim = ctx0 + tile * QT + rows; // kv rows visible to the last valid query row
-        kt0 = a.window > 0 ? max(0, ctx0 + tile * QT + 1 - a.window) / KT : 0;
+        kt0 = max(0, gqa_first_key(base_pos + ctx0 + tile * QT, a.window, a.chunk) - base_pos) / KT;
         n_tiles = rows > 0 && S > 0 ? (last_lim + KT - 1) / KT - kt0 : 0;
     }
     const int row0 = q0 + tile * QT;                  // first query row (global)
@@ -147,20 +169,20 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         // ================= TMA producer =================
         if (elect_one()) {
             mbar_expect_tx(q_full, Q_BYTES);
-            for (int c = 0; c < 3; ++c) tma_load_2d(q_s + c * CHUNK, &tmQ, q_full, h * DQK + c * 64, row0);
+            for (int c = 0; c < NC; ++c) tma_load_2d(q_s + c * CHUNK, &tmQ, q_full, qcol + c * 64, row0);
             for (int kt = 0; kt < n_tiles; ++kt) {
                 const int s = kt & 1;
                 const int krow = kv0 + (kt0 + kt) * KT;
                 if (!mbar_wait(&k_empty[s], ((kt >> 1) & 1) ^ 1)) { jib_report(a.status, JIB_ERR_WAIT_TIMEOUT, 31, kt); break; }
                 uint8_t * kd = k_s + s * K_BYTES;
                 mbar_expect_tx(&k_full[s], K_BYTES);
-                tma_load_2d(kd, &tmKV, &k_full[s], h * (DN + DV), krow);
-                tma_load_2d(kd + CHUNK, &tmKV, &k_full[s], h * (DN + DV) + 64, krow);
-                tma_load_2d(kd + 2 * CHUNK, &tmPE, &k_full[s], 0, krow);
+                tma_load_2d(kd, &tmKV, &k_full[s], kcol, krow);
+                tma_load_2d(kd + CHUNK, &tmKV, &k_full[s], kcol + 64, krow);
+                if (!GQA) tma_load_2d(kd + 2 * CHUNK, &tmPE, &k_full[s], 0, krow);
                 if (!mbar_wait(v_empty, (kt & 1) ^ 1)) { jib_report(a.status, JIB_ERR_WAIT_TIMEOUT, 32, kt); break; }
                 mbar_expect_tx(v_full, V_BYTES);
-                tma_load_2d(v_s, &tmKV, v_full, h * (DN + DV) + DN, krow);
-                tma_load_2d(v_s + CHUNK, &tmKV, v_full, h * (DN + DV) + DN + 64, krow);
+                tma_load_2d(v_s, &tmKV, v_full, vcol, krow);
+                tma_load_2d(v_s + CHUNK, &tmKV, v_full, vcol + 64, krow);
             }
         }
     } else if (n_tiles > 0 && warp == 1) {
@@ -191,7 +213,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
                 tc_fence_after();
                 const uint32_t k_addr = smem_u32(k_s + s * K_BYTES);
 #pragma unroll
-                for (int c = 0; c < 3; ++c)
+                for (int c = 0; c < NC; ++c)
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk)
                         mma_bf16(tm_S + s * KT, desc_k_sw128(q_addr + c * CHUNK + kk * 32), desc_k_sw128(k_addr + c * CHUNK + kk * 32), idesc_qk,
@@ -215,6 +237,9 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const uint32_t lane_addr = (uint32_t) (qd * 32) << 16;
         const int lim = r < rows ? ctx0 + tile * QT + r + 1 : 0;      // visible kv rows of this query row
         const int lim_first = ctx0 + tile * QT + 1;                   // ... of the tile's first row
+        // first visible gathered row of this query row, and of the tile's last one
+        const int first = gqa_first_key(base_pos + ctx0 + tile * QT + r, a.window, a.chunk) - base_pos;
+        const int first_last = gqa_first_key(base_pos + ctx0 + tile * QT + QT - 1, a.window, a.chunk) - base_pos;
         float m_ref = -INFINITY;                      // exponent base, log2 domain (score * scale * log2 e)
         float l_sum = 0.f;
         bool ok = true;
@@ -226,10 +251,10 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             tc_fence_after();
             const uint32_t ts = tm_S + lane_addr + s * KT;
             const int col0 = (kt0 + kt) * KT;
-            // the tile reaches the diagonal (or the sequence end), or begins before the last row's window does
-            const bool need_mask = col0 + KT > lim_first || (a.window > 0 && col0 < lim_first + QT - 1 - a.window);
+            // the tile reaches the diagonal (or the sequence end), or begins before what the last row sees does
+            const bool need_mask = col0 + KT > lim_first || col0 < first_last;
             const int vis = lim - col0;               // columns [inv, vis) of this tile are visible to this row
-            const int inv = a.window > 0 ? vis - a.window : 0;
+            const int inv = first - col0;
             // The row's 128 scores come out of tensor memory once, all loads in flight before one wait; the S buffer is
             // handed back to the tensor core right away (Q.K^T of the tile after the next may start).
             float x[KT];
@@ -240,7 +265,13 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_empty[s]);
             float mt = -INFINITY;
-            if (need_mask) {
+            if (GQA && a.cap_log2e > 0.f) {
+#pragma unroll
+                for (int c = 0; c < KT; ++c) {
+                    x[c] = !need_mask || (c < vis && c >= inv) ? capped_log2(x[c], a) : -INFINITY;
+                    mt = fmaxf(mt, x[c]);
+                }
+            } else if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) { x[c] = (c < vis && c >= inv) ? x[c] * a.scale_log2e : -INFINITY; mt = fmaxf(mt, x[c]); }
             } else {
@@ -308,7 +339,13 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             // rows end inside this warp; only the stores are predicated per row.  (Executed under a per-lane condition it
             // never completes.)
             const bool valid = r < rows;
-            const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+            if (GQA && a.sink && l_sum > 0.f) l_sum += exp2f(-m_ref);     // a key of score 0 without a value
+            float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+            if (GQA) {
+                inv *= a.out_scale;
+                if (a.gate != nullptr && valid)
+                    inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(a.gate[(size_t) (row0 + r) * a.ld_gate + h])));
+            }
             bf16 * dst = a.out + (size_t) (row0 + (valid ? r : 0)) * a.ldo + (size_t) h * DV;
 #pragma unroll 1
             for (int c = 0; c < DV; c += 16) {
@@ -339,7 +376,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 // sequence's last q_len tokens can see); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
 __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict__ cache, const int * __restrict__ block_tables, int max_blocks,
                                                         const int * __restrict__ seq_lens, int n_seqs, int block_size, int row_elems,
-                                                        long long n_slots, const int * __restrict__ q_start, int window,
+                                                        long long n_slots, const int * __restrict__ q_start, int window, int chunk,
                                                         bf16 * __restrict__ lat, int * __restrict__ kv_start, int total_cap) {
     PDL_TRIGGER_TOP();
     pdl_wait();
@@ -347,7 +384,7 @@ __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict_
     const int g = blockIdx.x * 8 + warp;              // global row of the gathered buffer this warp copies
     int b = -1, s = 0, acc = 0;
     for (int i = 0; i < n_seqs; ++i) {
-        const int S = seq_lens[i], n = window > 0 ? visible_rows(S, q_start[i + 1] - q_start[i], window) : S;
+        const int S = seq_lens[i], n = window > 0 || chunk > 0 ? visible_rows(S, q_start[i + 1] - q_start[i], window, chunk) : S;
         if (blockIdx.x == 0 && threadIdx.x == 0) kv_start[i] = acc;
         if (b < 0 && g < acc + n) { b = i; s = S - n + g - acc; }
         acc += n;
@@ -396,15 +433,15 @@ int map_2d(CUtensorMap * out, const void * ptr, long long rows, long long cols, 
 
 extern "C" {
 
-// Gathers the latent rows of all sequences of the batch (seq_lens[b] rows each, or with window > 0 the last
-// min(seq_lens[b], q_len[b] + window - 1), in sequence order) from the paged cache layer into lat [total_cap][row_elems] and writes the first row of every sequence to kv_start [n_seqs].
+// Gathers the cached rows of all sequences of the batch (seq_lens[b] rows each, or with a window or chunks those the sequence's last
+// q_len[b] tokens can see, in sequence order) from the paged cache layer into lat [total_cap][row_elems] and writes the first row of every sequence to kv_start [n_seqs].
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, void * lat, int * kv_start,
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, void * lat, int * kv_start,
                              int total_cap, void * stream) {
     if (n_seqs <= 0 || total_cap <= 0) return 0;
-    if (row_elems % 8 || block_size <= 0 || (window > 0 && q_start == nullptr)) return JIB_E_ARG;
+    if (row_elems % 8 || block_size <= 0 || ((window > 0 || chunk > 0) && q_start == nullptr)) return JIB_E_ARG;
     JIB_LAUNCH((kv_gather_kernel), (total_cap + 7) / 8, 256, 0, (cudaStream_t) stream, (const bf16 *) cache, block_tables, max_blocks, seq_lens,
-               n_seqs, block_size, row_elems, n_slots, q_start, window, (bf16 *) lat, kv_start, total_cap);
+               n_seqs, block_size, row_elems, n_slots, q_start, window, chunk, (bf16 *) lat, kv_start, total_cap);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 
@@ -425,13 +462,40 @@ JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * 
     if (rc) return rc;
     rc = map_2d(&mpe, kpe, total, DR, kpe_stride);
     if (rc) return rc;
-    MhaArgs a;
+    MhaArgs a = {};
     a.q_start = q_start; a.seq_lens = seq_lens; a.kv_start = kv_start; a.out = (bf16 *) out; a.status = status; a.ldo = ldo;
     a.n_seqs = n_seqs; a.T = T; a.H = H; a.window = window;
     a.scale_log2e = scale * 1.4426950408889634f;
+    constexpr int SMEM = Form<false>::SMEM_BYTES;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(mha_prefill_kernel, SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((mha_prefill_kernel), dim3(n_q_tiles, H), NUM_THREADS, SMEM_BYTES, stream, mq, mkv, mpe, a);
+    if (!jib::ensure_dyn_smem(mha_prefill_kernel<false>, SMEM, attr_done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((mha_prefill_kernel<false>), dim3(n_q_tiles, H), NUM_THREADS, SMEM, stream, mq, mkv, mpe, a);
+    return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
+}
+
+// Grouped-query attention of a prompt chunk: D = V = 128.  q [T][H][128]; kv [total][row]: the gathered cache rows (keys, then values).
+JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * kv, long long total, const int * kv_start, const void * gate,
+                               long long ld_gate, int n_q_tiles, void * out, long long ldo, void * stream_) {
+    cudaStream_t stream = (cudaStream_t) stream_;
+    if (m->T <= 0 || m->n_seqs <= 0 || n_q_tiles <= 0) return 0;
+    if (m->D != DN || m->V != DV || m->H < 1 || m->G < 1 || m->H % m->G || m->row < (long long) m->G * (DN + DV)) return JIB_E_ARG;
+    if (ldo % 8 || ((uintptr_t) out & 15) || total <= 0) return JIB_E_ALIGN;
+    CUtensorMap mq, mkv;
+    int rc = map_2d(&mq, q, m->T, (long long) m->H * DN, (long long) m->H * DN);
+    if (rc) return rc;
+    rc = map_2d(&mkv, kv, total, m->row, m->row);
+    if (rc) return rc;
+    MhaArgs a = {};
+    a.q_start = m->q_start; a.seq_lens = m->seq_lens; a.kv_start = kv_start; a.out = (bf16 *) out; a.status = m->status; a.ldo = ldo;
+    a.n_seqs = m->n_seqs; a.T = m->T; a.H = m->H; a.G = m->G; a.window = m->window; a.chunk = m->chunk; a.sink = m->sink;
+    a.scale_log2e = m->scale * 1.4426950408889634f;
+    a.cap_log2e = m->softcap * 1.4426950408889634f;
+    a.inv_cap2 = m->softcap > 0.f ? 2.f * a.scale_log2e / m->softcap : 0.f;
+    a.gate = (const bf16 *) gate; a.ld_gate = ld_gate; a.out_scale = m->out_scale;
+    constexpr int SMEM = Form<true>::SMEM_BYTES;
+    static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
+    if (!jib::ensure_dyn_smem(mha_prefill_kernel<true>, SMEM, attr_done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((mha_prefill_kernel<true>), dim3(n_q_tiles, m->H), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 

@@ -113,11 +113,12 @@ def load():
     L.jib_state_chunk_bytes.restype, L.jib_state_chunk_bytes.argtypes = C.c_longlong, [C.POINTER(StateMixDesc)]
     sig("jib_state_mix_run", C.POINTER(StateMixDesc), i, i, vp)
     sig("jib_gqa_qkv_post", C.POINTER(GqaDesc), vp, vp, vp, ll, fp, fp, fp, ip, vp, i, vp)
+    sig("jib_gqa_prefill", C.POINTER(GqaDesc), vp, vp, ll, ip, vp, ll, i, vp, ll, vp)
     sig("jib_gqa_attention", C.POINTER(GqaDesc), vp, vp, ll, vp, ll, i, i, i, vp)
     sig("jib_embed_gather", vp, ip, vp, i, i, i, vp)
     sig("jib_rmsnorm", vp, vp, fp, vp, vp, i, i, ll, f, vp)
     sig("jib_mla_qkv_post", vp, ll, vp, ll, fp, f, fp, ip, ip, vp, vp, ll, ll, i, i, i, i, i, i, ll, i, i, ip, vp)
-    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, ip, i, vp, ip, i, vp)
+    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, ip, i, i, vp, ip, i, vp)
     sig("jib_mha_prefill", vp, ll, vp, vp, ll, ll, ip, ip, ip, i, i, i, f, i, i, vp, ll, ip, vp)
     sig("jib_argmax", fp, ip, i, i, vp)
     sig("jib_topk", fp, fp, ip, i, i, i, vp)
@@ -454,11 +455,17 @@ MHA_PREFILL = os.environ.get("JIB_MHA_PREFILL", "1") == "1"      # "0": prompt c
 MHA_PREFILL_MIN_TOKENS = 64
 
 
-def visible_total(meta, window: int) -> int:
+def visible_rows(q_len: int, s_len: int, window: int = 0, chunk: int = 0) -> int:
+    """Cached rows of a sequence that its last ``q_len`` of ``s_len`` tokens can see."""
+    p = max(0, s_len - q_len)
+    return s_len - max(0, p - window + 1 if window > 0 else 0, p // chunk * chunk if chunk > 0 else 0)
+
+
+def visible_total(meta, window: int, chunk: int = 0) -> int:
     """Cached rows the queries of a step can see, over its sequences (what ``kv_gather`` writes)."""
-    if window <= 0:
+    if window <= 0 and chunk <= 0:
         return int(meta["total_kv"])
-    return sum(min(int(s), int(q) + window - 1) for q, s in zip(meta["q_lens"], meta["s_lens"]))
+    return sum(visible_rows(int(q), int(s), window, chunk) for q, s in zip(meta["q_lens"], meta["s_lens"]))
 
 
 def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, meta, window: int = 0) -> bool:
@@ -477,15 +484,15 @@ def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, m
     return total > 0 and dec <= total - dec
 
 
-def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int, q_start=None, window: int = 0):
-    """The cached latent rows of every sequence of the batch (with a window: those its query tokens can see), in sequence
+def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int, q_start=None, window: int = 0, chunk: int = 0):
+    """The cached rows of every sequence of the batch (with a window or chunks: those its query tokens can see), in sequence
     order: ([total, row] bf16, first row of each sequence [n_seqs] int32)."""
     n_seqs = seq_lens.shape[0]
     row = cache.shape[1]
     lat = torch.empty(total, row, dtype=torch.bfloat16, device=cache.device)
     kv_start = torch.empty(n_seqs, dtype=torch.int32, device=cache.device)
     _ck(load().jib_kv_gather(cache.data_ptr(), cache.shape[0], block_tables.data_ptr(), block_tables.stride(0), seq_lens.data_ptr(),
-                             n_seqs, block_size, row, _p(q_start), window, lat.data_ptr(), kv_start.data_ptr(), total, _stream()), "kv_gather")
+                             n_seqs, block_size, row, _p(q_start), window, chunk, lat.data_ptr(), kv_start.data_ptr(), total, _stream()), "kv_gather")
     return lat, kv_start
 
 
@@ -807,9 +814,15 @@ def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
 def gqa_splits(m, T, max_keys, sm_count=148):
     """CTAs that share one row's keys in a batch of single tokens: as many as fill the machine, at most one per 64 visible keys."""
     keys = min([x for x in (m.window, m.chunk, max_keys) if x > 0])
-    fill = max(1, 2 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
+    fill = max(1, 4 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
     n = min(8, fill, (keys + 63) // 64)
     return 1 << (n.bit_length() - 1)
+
+
+def gqa_prefill_ok(m, q, cache, out, block_size: int, single: bool, meta) -> bool:
+    """Whether a batch of portions takes the tensor-core kernel (needs the host-side totals in ``meta``)."""
+    return not single and MHA_PREFILL and meta is not None and "q_lens" in meta and q.dtype == torch.bfloat16 and q.shape[0] >= MHA_PREFILL_MIN_TOKENS and \
+        m.dim == 128 and m.vdim == 128 and cache.shape[1] % 8 == 0 and block_size == 64 and _tma_ok(q.data_ptr(), out.data_ptr(), out.stride(0) * 2)
 
 
 def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
@@ -819,6 +832,12 @@ def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size
     gd = _gqa_desc(m, cache, T, seq_lens.shape[0])
     gd.block_tables, gd.max_blocks, gd.block_size = block_tables.data_ptr(), block_tables.stride(0), block_size
     gd.seq_lens, gd.q_start = seq_lens.data_ptr(), q_start.data_ptr()
+    if gqa_prefill_ok(m, q, cache, out, block_size, single, meta):
+        total = visible_total(meta, m.window, m.chunk)
+        kv, kv_start = kv_gather(cache, block_tables, seq_lens, total, block_size, q_start, m.window, m.chunk)
+        _ck(load().jib_gqa_prefill(C.byref(gd), q.data_ptr(), kv.data_ptr(), total, kv_start.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0,
+                                   int(meta["n_q_tiles"]), out.data_ptr(), out.stride(0), _stream()), "gqa_prefill")
+        return out
     splits = gqa_splits(m, T, block_tables.shape[1] * block_size, workspace(q.device).sm_count) if single else 1
     _ck(load().jib_gqa_attention(C.byref(gd), q.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), int(single),
                                  splits, int(q.dtype == torch.float32), _stream()), "gqa_attention")

@@ -219,6 +219,7 @@ def run_attention(m, dev, dtype, cuts, lens, rot, seed=0, hot=()):
     sc = rot.get("scaling")
     table = lugovik.rope_table(max(lens), lugovik.Rotation(rot["dims"], rot["base"], None if sc is None else lugovik.Yarn(**sc)), dev)
     at, got = [0] * len(lens), [[] for _ in lens]
+    prefills = ops.nat().launches_by_name.get("gqa_prefill", 0) if dev == "cuda" else 0
     for cut in cuts:
         part = [(j, at[j], n) for j, n in enumerate(cut) if n]
         proj = torch.cat([torch.cat([x[p:p + n] for x in seqs[j]], 1) for j, p, n in part]).to(dev, dtype)
@@ -241,6 +242,9 @@ def run_attention(m, dev, dtype, cuts, lens, rot, seed=0, hot=()):
     assert tuple(at) == tuple(lens)
     for j in range(len(lens)):
         close(torch.cat(got[j]), want[j], dtype, f"sequence {j}")
+    if dev == "cuda":                                                # the tensor-core kernel ran where it should
+        assert (ops.nat().launches_by_name.get("gqa_prefill", 0) > prefills) == (dtype == BF16 and D == V == 128 and max(map(sum, cuts)) >= 64)
+        ops.nat().check_status()
     return want
 
 
