@@ -3,8 +3,10 @@
 //
 //   gqa_qkv_post    per-head RMS norm of q and k, rotate-half RoPE on the first rot dimensions, rows into the cache
 //   gqa_attention   scores * scale, softcap, causal mask with a sliding window and / or chunks counted from position 0, softmax
-//                   with or without a sink (a key of score 0 without a value), a gate per head: any sizes, any mix of portions
-//                   and single tokens, keys split over a thread-block cluster
+//                   with or without a sink (a key of score 0 without a value), a gate per head: any mix of portions and single
+//                   tokens, keys split over a thread-block cluster.  bf16 heads whose sizes are multiples of 16: products on the
+//                   tensor cores (gqa_mma); fp32 and other sizes: CUDA cores (gqa_attention).  Prompts with heads of 128 have a
+//                   kernel of their own (mha_prefill_tcgen05.cu).
 //
 // Activations and cache rows bf16 or fp32; norms, angles, scores and softmax fp32.
 #include <cuda_bf16.h>
@@ -39,9 +41,9 @@ template <> __device__ __forceinline__ float capped<bf16>(float s, float cap) {
 template <> __device__ __forceinline__ float capped<float>(float s, float cap) { return cap * tanhf(s / cap); }
 
 // ---- norm, rotation, cache rows: one warp per (token, head of q / k / v) ------------------------------------------------------
-constexpr int POST_D = 16;                                   // elements of a head per lane: D <= 32 * POST_D
+constexpr int POST_D = 16;                                   // elements of a head per lane (N): D <= 32 * POST_D
 
-template <typename T>
+template <typename T, int N>
 __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ k,
                                                            const T * __restrict__ v, long long ld, const float * __restrict__ q_norm,
                                                            const float * __restrict__ k_norm, const float * __restrict__ rope,
@@ -74,32 +76,44 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
     const T * src = (is_q ? q : k) + (size_t) t * ld + head * D;
     const float * w = is_q ? q_norm : k_norm;
     float * x = heads + warp * D;
-    float e[POST_D], ss = 0.f;
+    float e[N], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < POST_D; ++i) {
+    for (int i = 0; i < N; ++i) {
         const int c = lane + 32 * i;
         e[i] = c < D ? to_f(src[c]) : 0.f;
         ss += e[i] * e[i];
     }
-    const float inv = rsqrtf(warp_sum(ss) / (float) D + a.eps);
-#pragma unroll
-    for (int i = 0; i < POST_D; ++i) {
-        const int c = lane + 32 * i;
-        if (c < D) x[c] = e[i] * inv * w[c];
-    }
-    __syncwarp();
     int pos = a.positions[t];
     if (pos < 0 || pos >= a.max_pos) {
         if (lane == 0) jib_report(a.status, JIB_ERR_BOUNDS, 49, pos);
         pos = 0;
     }
-    const float2 * cs = (const float2 *) rope + (size_t) pos * (a.rot / 2);
-    T * dst = is_q ? q_out + ((size_t) t * H + head) * D : row + head * D;
     const int half = a.rot / 2;
-    for (int c = lane; c < D; c += 32) {
-        float y = x[c];
-        if (c < half) y = y * cs[c].x - x[c + half] * cs[c].y;
-        else if (c < a.rot) y = y * cs[c - half].x + x[c - half] * cs[c - half].y;
+    const float2 * cs = (const float2 *) rope + (size_t) pos * half;
+    float wt[N];
+    float2 r[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {                            // requested before the reduction
+        const int c = lane + 32 * i;
+        wt[i] = c < D ? w[c] : 0.f;
+        r[i] = c < a.rot ? cs[c < half ? c : c - half] : make_float2(1.f, 0.f);
+    }
+    const float inv = rsqrtf(warp_sum(ss) / (float) D + a.eps);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const int c = lane + 32 * i;
+        e[i] *= inv * wt[i];
+        if (c < D) x[c] = e[i];
+    }
+    __syncwarp();
+    T * dst = is_q ? q_out + ((size_t) t * H + head) * D : row + head * D;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const int c = lane + 32 * i;
+        if (c >= D) continue;
+        float y = e[i];
+        if (c < half) y = y * r[i].x - x[c + half] * r[i].y;
+        else if (c < a.rot) y = y * r[i].x + x[c - half] * r[i].y;
         put(dst + c, y);
     }
 }
@@ -148,17 +162,12 @@ template <> struct Quad<bf16> {
     }
 };
 
-template <typename T, int NVC>
-__global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ gate,
-                                                           long long ld_gate, T * __restrict__ out, long long ldo, int run, int heads, int KT) {
-    extern __shared__ float smem[];
-    __shared__ int rows_s[64];
-    PDL_TRIGGER_TOP();
-    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int tid = threadIdx.x, D = a.D, V = a.V, rep = a.H / a.G;
-    const int DP = (D + 3) / 4 * 4 + 4, VP = (V + 3) / 4 * 4;
-    float * qs = smem, * m_s = qs + ROWS * DP, * l_s = m_s + ROWS, * c_s = l_s + ROWS;
-    float * ks = c_s + ROWS, * vs = ks + KT * DP, * ps = vs + KT * VP;                           // ps [KT][ROWS]
+// What a CTA works on: rows (token i0 + r / nh of sequence b, head h0 + r % nh), r < rows, against the key tiles k_lo .. k_hi.
+struct Work {
+    int b, q0, i0, g, h0, nh, rows, p0, lo, end, k_lo, k_hi;
+};
+// false: no work for this CTA nor for the others of its cluster
+__device__ __forceinline__ bool find_work(const jib_gqa & a, int run, int heads, int KT, Work & w) {
     // which (sequence, run of tokens)?  Sequence b's runs start at index q_start[b] / run + b; indices in the gaps have no tokens.
     // (run 0: one token per sequence)
     int b = run == 0 ? (int) blockIdx.x : 0, hi = run == 0 ? 0 : a.n_seqs;
@@ -166,16 +175,79 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
         const int mid = (b + hi) >> 1;
         if (a.q_start[mid] / run + mid <= (int) blockIdx.x) b = mid; else hi = mid;
     }
-    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0, i0 = run == 0 ? 0 : ((int) blockIdx.x - (q0 / run + b)) * run;
+    w.b = b;
+    w.q0 = a.q_start[b];
+    const int n = a.q_start[b + 1] - w.q0;
+    w.i0 = run == 0 ? 0 : ((int) blockIdx.x - (w.q0 / run + b)) * run;
     if (run == 0) run = 1;
-    if (i0 < 0 || i0 >= n) return;                           // the same for the whole cluster
-    const int groups = (rep + heads - 1) / heads, g = blockIdx.y / groups, h0 = g * rep + (blockIdx.y % groups) * heads;
-    const int nh = min(heads, (g + 1) * rep - h0), nt = min(run, n - i0), rows = nt * nh;       // row r: token i0 + r / nh, head h0 + r % nh
-    const int S = a.seq_lens[b], p0 = S - n + i0;            // position of the first token
-    const int lo = max(0, gqa_first_key(p0, a.window, a.chunk)), end = S > 0 ? p0 + nt : 0;
-    const int t_lo = lo / KT, tiles = end > lo ? (end - 1) / KT + 1 - t_lo : 0;
-    const int split = blockIdx.z, n_splits = gridDim.z, per = (tiles + n_splits - 1) / n_splits;
-    const int k_lo = t_lo + split * per, k_hi = min(t_lo + tiles, k_lo + per);
+    if (w.i0 < 0 || w.i0 >= n) return false;
+    const int rep = a.H / a.G, groups = (rep + heads - 1) / heads;
+    w.g = blockIdx.y / groups;
+    w.h0 = w.g * rep + (blockIdx.y % groups) * heads;
+    w.nh = min(heads, (w.g + 1) * rep - w.h0);
+    const int nt = min(run, n - w.i0);
+    w.rows = nt * w.nh;
+    const int S = a.seq_lens[b];
+    w.p0 = S - n + w.i0;                                     // position of the first token
+    w.lo = max(0, gqa_first_key(w.p0, a.window, a.chunk));
+    w.end = S > 0 ? w.p0 + nt : 0;
+    const int t_lo = w.lo / KT, tiles = w.end > w.lo ? (w.end - 1) / KT + 1 - t_lo : 0;
+    const int per = (tiles + (int) gridDim.z - 1) / (int) gridDim.z;
+    w.k_lo = t_lo + (int) blockIdx.z * per;
+    w.k_hi = min(t_lo + tiles, w.k_lo + per);
+    return true;
+}
+
+// part [ROWS][V], m_s and l_s [ROWS] of this CTA, complete behind a barrier -> this CTA's share of the results
+template <typename T>
+__device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, const float * part, const float * m_s, const float * l_s,
+                                            const T * gate, long long ld_gate, T * out, long long ldo) {
+    const int n_splits = gridDim.z, V = a.V;
+    if (n_splits > 1) cluster_sync(); else __syncthreads();
+    for (int i = threadIdx.x + (int) blockIdx.z * NT; i < w.rows * V; i += NT * n_splits) {
+        const int r = i / V, col = i % V;
+        float ms[8], ls[8], os[8], m = a.sink ? 0.f : -INFINITY;
+#pragma unroll
+        for (int s = 0; s < 8; ++s) {                        // every peer's value requested before any is used
+            ms[s] = -INFINITY;
+            ls[s] = os[s] = 0.f;
+            if (s >= n_splits) continue;
+            ms[s] = n_splits > 1 ? ld_peer(m_s + r, s) : m_s[r];
+            ls[s] = n_splits > 1 ? ld_peer(l_s + r, s) : l_s[r];
+            os[s] = n_splits > 1 ? ld_peer(part + r * V + col, s) : part[r * V + col];
+        }
+        const int t = w.q0 + w.i0 + r / w.nh, h = w.h0 + r % w.nh;
+        const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + h]) : 0.f;
+#pragma unroll
+        for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
+        float l = a.sink ? exp_t<T>(-m) : 0.f, o = 0.f;
+#pragma unroll
+        for (int s = 0; s < 8; ++s) {
+            const float e = ms[s] == -INFINITY ? 0.f : exp_t<T>(ms[s] - m);
+            l += e * ls[s];
+            o += e * os[s];
+        }
+        float y = l > 0.f ? o / l * a.out_scale : 0.f;
+        if (gate != nullptr) y /= 1.f + exp_t<T>(-gt);
+        put(out + (size_t) t * ldo + h * V + col, y);
+    }
+    if (n_splits > 1) cluster_sync();                        // a CTA that leaves takes its shared memory with it
+}
+
+template <typename T, int NVC>
+__global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ gate,
+                                                           long long ld_gate, T * __restrict__ out, long long ldo, int run, int heads, int KT) {
+    extern __shared__ float smem[];
+    __shared__ int rows_s[64];
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int tid = threadIdx.x, D = a.D, V = a.V;
+    const int DP = (D + 3) / 4 * 4 + 4, VP = (V + 3) / 4 * 4;
+    float * qs = smem, * m_s = qs + ROWS * DP, * l_s = m_s + ROWS, * c_s = l_s + ROWS;
+    float * ks = c_s + ROWS, * vs = ks + KT * DP, * ps = vs + KT * VP;                           // ps [KT][ROWS]
+    Work w;
+    if (!find_work(a, run, heads, KT, w)) return;
+    const int q0 = w.q0, i0 = w.i0, g = w.g, h0 = w.h0, nh = w.nh, rows = w.rows, p0 = w.p0, lo = w.lo, end = w.end;
     const bool vec = ((D | V | a.row) & 3) == 0;
     for (int i = tid; i < ROWS * (DP / 4); i += NT) {
         const int r = i / (DP / 4), c = i % (DP / 4) * 4;
@@ -194,9 +266,9 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
     for (int c = 0; c < NVC; ++c)
 #pragma unroll
         for (int r = 0; r < ROWS; ++r) acc[c][r] = 0.f;
-    const int * bt = a.block_tables + (size_t) b * a.max_blocks;
+    const int * bt = a.block_tables + (size_t) w.b * a.max_blocks;
     const int key = tid % KT, rg = tid / KT, rpt = ROWS * KT / NT;       // scores: this thread's key and its rpt rows
-    for (int kt = k_lo; kt < k_hi; ++kt) {
+    for (int kt = w.k_lo; kt < w.k_hi; ++kt) {
         __syncthreads();
         if (tid < KT) {                                      // where this tile's rows are
             const int p = kt * KT + tid;
@@ -305,25 +377,195 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
         if (col < V)
             for (int r = 0; r < ROWS; ++r) part[r * V + col] = acc[c][r];
     }
-    if (n_splits > 1) cluster_sync(); else __syncthreads();
-    for (int i = tid + split * NT; i < rows * V; i += NT * n_splits) {
-        const int r = i / V, col = i % V;
-        float m = a.sink ? 0.f : -INFINITY;
-        for (int s = 0; s < n_splits; ++s) m = fmaxf(m, n_splits > 1 ? ld_peer(m_s + r, s) : m_s[r]);
-        float l = a.sink ? exp_t<T>(-m) : 0.f, o = 0.f;
-        for (int s = 0; s < n_splits; ++s) {
-            const float ms = n_splits > 1 ? ld_peer(m_s + r, s) : m_s[r];
-            if (ms == -INFINITY) continue;
-            const float w = exp_t<T>(ms - m);
-            l += w * (n_splits > 1 ? ld_peer(l_s + r, s) : l_s[r]);
-            o += w * (n_splits > 1 ? ld_peer(part + r * V + col, s) : part[r * V + col]);
+    finish_rows<T>(a, w, part, m_s, l_s, gate, ld_gate, out, ldo);
+}
+
+// ---- attention on tensor cores: bf16, D and V multiples of 16 ---------------------------------------------------------------------
+// The same decomposition; the 16 rows are the M of m16n8k16 products.  Tiles of 64 keys arrive by asynchronous copies, one ahead; each
+// of the 4 warps takes 16 keys of a tile and keeps its own running maximum, sum and output (NV x 8 columns), which meet at the end.
+constexpr int MK = 64, PADC = 8;                             // keys per tile; padding of the shared rows (16 bytes: rows hit different banks)
+
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&x)[4], uint32_t y0, uint32_t y1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(x[0]), "r"(x[1]), "r"(x[2]), "r"(x[3]), "r"(y0), "r"(y1));
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void * src, bool valid) {       // zeros if not valid (src is not read)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+
+template <int NV>                                            // columns of V per 16: V <= 16 NV
+__global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib_gqa a, const bf16 * __restrict__ q, const bf16 * __restrict__ gate,
+                                                     long long ld_gate, bf16 * __restrict__ out, long long ldo, int run, int heads) {
+    extern __shared__ __align__(16) uint8_t smem_mma[];
+    __shared__ float m_s[ROWS], l_s[ROWS], wm[4][ROWS], wl[4][ROWS];
+    PDL_TRIGGER_TOP();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, D = a.D, V = a.V;
+    const int LD = D + PADC, LV = V + PADC;                  // row strides (elements)
+    const uint32_t q_addr = (uint32_t) __cvta_generic_to_shared(smem_mma), kv_addr = q_addr + ROWS * LD * 2;
+    const uint32_t tile_bytes = MK * (LD + LV) * 2;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    Work w;
+    if (!find_work(a, run, heads, MK, w)) return;
+    const int * bt = a.block_tables + (size_t) w.b * a.max_blocks;
+    const bf16 * cache = (const bf16 *) a.cache;
+    const int d8 = D / 8, v8 = V / 8;
+    // a thread copies half of one key's row: 2 threads per key
+    auto stage = [&](int kt, int buf) {
+        if (kt < w.k_hi) {
+            const int j = tid >> 1, p = kt * MK + j;
+            const bool in = p >= w.lo && p < w.end;
+            const bf16 * row = in ? cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row : cache;
+            const uint32_t kd = kv_addr + buf * tile_bytes + j * LD * 2, vd = kv_addr + buf * tile_bytes + (MK * LD + j * LV) * 2;
+            for (int c = tid & 1; c < d8; c += 2) cp16(kd + c * 16, row + w.g * D + c * 8, in);
+            for (int c = tid & 1; c < v8; c += 2) cp16(vd + c * 16, row + a.G * D + w.g * V + c * 8, in);
         }
-        const int t = q0 + i0 + r / nh, h = h0 + r % nh;
-        float y = l > 0.f ? o / l * a.out_scale : 0.f;
-        if (gate != nullptr) y /= 1.f + exp_t<T>(-to_f(gate[(size_t) t * ld_gate + h]));
-        put(out + (size_t) t * ldo + h * V + col, y);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    for (int i = tid; i < ROWS * d8; i += NT) {
+        const int r = i / d8, c = i % d8;
+        cp16(q_addr + (r * LD + c * 8) * 2, q + (r < w.rows ? ((size_t) (w.q0 + w.i0 + r / w.nh) * a.H + w.h0 + r % w.nh) * D + c * 8 : 0), r < w.rows);
     }
-    if (n_splits > 1) cluster_sync();                        // a CTA that leaves takes its shared memory with it
+    stage(w.k_lo, 0);
+    const int fr = lane >> 2, fc = (lane & 3) * 2;
+    // positions and first keys of this thread's two rows
+    int pos[2], first[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int r = fr + 8 * e;
+        pos[e] = r < w.rows ? w.p0 + r / w.nh : -1;
+        first[e] = r < w.rows ? gqa_first_key(pos[e], a.window, a.chunk) : 0;
+    }
+    float o[2 * NV][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+    for (int n = 0; n < 2 * NV; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float sc = a.softcap > 0.f ? 2.f * LOG2E * a.scale / a.softcap : a.scale * LOG2E, cap = a.softcap * LOG2E;
+    for (int kt = w.k_lo; kt < w.k_hi; ++kt) {
+        const int buf = (kt - w.k_lo) & 1;
+        stage(kt + 1, buf ^ 1);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const uint32_t k_addr = kv_addr + buf * tile_bytes + warp * 16 * LD * 2, v_addr = kv_addr + buf * tile_bytes + (MK * LD + warp * 16 * LV) * 2;
+        float s[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
+#pragma unroll 4
+        for (int kk = 0; kk < D; kk += 16) {
+            uint32_t x[4], y[4];
+            ldm4(x, q_addr + ((lane & 15) * LD + kk + (lane >> 4) * 8) * 2);
+            ldm4(y, k_addr + (((lane & 7) + ((lane >> 4) << 3)) * LD + kk + ((lane >> 3) & 1) * 8) * 2);      // keys 0-7 | 8-15
+            mma(s[0], x, y[0], y[1]);
+            mma(s[1], x, y[2], y[3]);
+        }
+        const int key = kt * MK + warp * 16 + fc;            // this thread's keys: key, key + 1, key + 8, key + 9
+        float mt[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float y = s[n][e] * sc;
+                if (a.softcap > 0.f) {
+                    float x, r;
+                    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(x) : "f"(fminf(y, 120.f)));
+                    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + x));
+                    y = cap - 2.f * cap * r;                 // 1 - 2 / (1 + e^{2 y}) = tanh(y)
+                }
+                const int p = key + n * 8 + (e & 1);
+                s[n][e] = p <= pos[e >> 1] && p >= first[e >> 1] ? y : -INFINITY;
+                mt[e >> 1] = fmaxf(mt[e >> 1], s[n][e]);
+            }
+        float cf[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            mt[e] = fmaxf(mt[e], __shfl_xor_sync(0xffffffffu, mt[e], 1));
+            mt[e] = fmaxf(mt[e], __shfl_xor_sync(0xffffffffu, mt[e], 2));
+            const float mn = fmaxf(m[e], mt[e]);
+            cf[e] = mn == -INFINITY ? 1.f : exp2f(m[e] - mn);
+            m[e] = mn;
+            l[e] *= cf[e];
+        }
+        uint32_t x[4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float p0 = s[n][2 * e] == -INFINITY ? 0.f : exp2f(s[n][2 * e] - m[e]), p1 = s[n][2 * e + 1] == -INFINITY ? 0.f : exp2f(s[n][2 * e + 1] - m[e]);
+                l[e] += p0 + p1;
+                const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
+                x[n * 2 + e] = *(const uint32_t *) &pk;
+            }
+#pragma unroll
+        for (int n = 0; n < 2 * NV; n += 2) {
+            if (n * 8 >= V) break;
+            uint32_t y[4];
+            ldm4t(y, v_addr + ((lane & 15) * LV + n * 8 + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                o[n][e] *= cf[e >> 1];
+                o[n + 1][e] *= cf[e >> 1];
+            }
+            mma(o[n], x, y[0], y[1]);
+            mma(o[n + 1], x, y[2], y[3]);
+        }
+        __syncthreads();                                     // the buffer is free
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+        if ((lane & 3) == 0) {
+            wm[warp][fr + 8 * e] = m[e];
+            wl[warp][fr + 8 * e] = l[e];
+        }
+    }
+    __syncthreads();
+    // the four warps' outputs, brought to a common maximum, summed in shared memory one warp after the other
+    float * part = (float *) (smem_mma + ROWS * LD * 2);
+    float f[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int r = fr + 8 * e;
+        const float mx = fmaxf(fmaxf(wm[0][r], wm[1][r]), fmaxf(wm[2][r], wm[3][r]));
+        f[e] = m[e] == -INFINITY ? 0.f : exp2f(m[e] - mx);
+    }
+    for (int k = 0; k < 4; ++k) {
+        if (warp == k) {
+#pragma unroll
+            for (int n = 0; n < 2 * NV; ++n) {
+                if (n * 8 >= V) break;
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    float2 * p = (float2 *) (part + (fr + 8 * e) * V + n * 8 + fc);
+                    float2 y = k == 0 ? make_float2(0.f, 0.f) : *p;
+                    y.x += o[n][2 * e] * f[e];
+                    y.y += o[n][2 * e + 1] * f[e];
+                    *p = y;
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (tid < ROWS) {
+        const float mx = fmaxf(fmaxf(wm[0][tid], wm[1][tid]), fmaxf(wm[2][tid], wm[3][tid]));
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) s += wm[k][tid] == -INFINITY ? 0.f : wl[k][tid] * exp2f(wm[k][tid] - mx);
+        m_s[tid] = mx == -INFINITY ? mx : mx / LOG2E;        // natural units
+        l_s[tid] = s;
+    }
+    finish_rows<bf16>(a, w, part, m_s, l_s, gate, ld_gate, out, ldo);
 }
 
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
@@ -351,6 +593,26 @@ int launch_attention(const jib_gqa & a, const void * q, const void * gate, long 
     return launched();
 }
 
+// bf16 rows that 16-byte copies can address
+bool mma_ok(const jib_gqa & a, const void * q) {
+    return a.D % 16 == 0 && a.V % 16 == 0 && a.V <= 256 && a.row % 8 == 0 && (((uintptr_t) a.cache | (uintptr_t) q) & 15) == 0;
+}
+
+template <int NV>
+int launch_mma(const jib_gqa & a, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single, int splits,
+               cudaStream_t s) {
+    const int tile = MK * (a.D + a.V + 2 * PADC) * 2, smem = ROWS * (a.D + PADC) * 2 + 2 * tile;       // >= the [ROWS][V] partial results
+    constexpr int CAP = 220 * 1024;
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (smem > CAP || !jib::ensure_dyn_smem(gqa_mma_kernel<NV>, CAP, done)) return JIB_E_ARG;
+    const int rep = a.H / a.G, heads = rep < ROWS ? rep : ROWS, run = single ? 0 : ROWS / heads;
+    const dim3 grid(single ? a.T : a.T / run + a.n_seqs, a.G * ((rep + heads - 1) / heads), splits);
+    const cudaError_t e = jib::launch_pdl_cluster(gqa_mma_kernel<NV>, grid, dim3(NT), (size_t) smem, s, splits, a, (const bf16 *) q, (const bf16 *) gate,
+                                                  ld_gate, (bf16 *) out, ldo, run, heads);
+    if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
+    return launched();
+}
+
 bool ok(const jib_gqa & a) {
     return a.H >= 1 && a.G >= 1 && a.H % a.G == 0 && a.D >= 1 && a.D <= 32 * POST_D && a.V >= 1 && a.V <= 4 * NT && a.rot >= 0 && a.rot % 2 == 0 && a.rot <= a.D &&
            a.row >= (long long) a.G * (a.D + a.V) && a.T <= 65535 && a.block_size > 0;
@@ -368,12 +630,19 @@ JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * 
     cudaStream_t s = (cudaStream_t) stream;
     const dim3 grid((a.H + 2 * a.G + 7) / 8, a.T);
     const int smem = 8 * a.D * 4;
-    if (f32)
-        JIB_LAUNCH((gqa_qkv_post_kernel<float>), grid, 256, smem, s, a, (const float *) q, (const float *) k, (const float *) v, ld, q_norm, k_norm,
-                   rope, slot_mapping, (float *) q_out);
-    else
-        JIB_LAUNCH((gqa_qkv_post_kernel<bf16>), grid, 256, smem, s, a, (const bf16 *) q, (const bf16 *) k, (const bf16 *) v, ld, q_norm, k_norm, rope,
-                   slot_mapping, (bf16 *) q_out);
+#define POST(TT, N)                                                                                                                        \
+    JIB_LAUNCH((gqa_qkv_post_kernel<TT, N>), grid, 256, smem, s, a, (const TT *) q, (const TT *) k, (const TT *) v, ld, q_norm, k_norm, rope, \
+               slot_mapping, (TT *) q_out)
+#define CALL(N)                     \
+    do {                            \
+        if (f32) POST(float, N);    \
+        else POST(bf16, N);         \
+    } while (0)
+    if (a.D <= 64) CALL(2);
+    else if (a.D <= 128) CALL(4);
+    else CALL(POST_D);
+#undef CALL
+#undef POST
     return launched();
 }
 
@@ -383,6 +652,11 @@ JIB_EXPORT int jib_gqa_attention(const jib_gqa * m, const void * q, const void *
     if (a.T <= 0 || a.n_seqs <= 0) return 0;
     if (!ok(a) || splits < 1 || splits > 8 || (single && a.T != a.n_seqs)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
+    if (!f32 && mma_ok(a, q)) {
+        if (a.V <= 64) return launch_mma<4>(a, q, gate, ld_gate, out, ldo, single, splits, s);
+        if (a.V <= 128) return launch_mma<8>(a, q, gate, ld_gate, out, ldo, single, splits, s);
+        return launch_mma<16>(a, q, gate, ld_gate, out, ldo, single, splits, s);
+    }
 #define CALL(NVC) (f32 ? launch_attention<float, NVC>(a, q, gate, ld_gate, out, ldo, single, splits, s)     \
                        : launch_attention<bf16, NVC>(a, q, gate, ld_gate, out, ldo, single, splits, s))
     if (a.V <= NT) return CALL(1);

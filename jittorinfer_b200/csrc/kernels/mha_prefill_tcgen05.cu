@@ -78,7 +78,10 @@ __host__ __device__ __forceinline__ int visible_rows(int S, int q_len, int windo
 
 // softcap * tanh(score * scale / softcap) * log2 e from the raw product
 __device__ __forceinline__ float capped_log2(float s, const MhaArgs & a) {
-    return a.cap_log2e * (1.f - __fdividef(2.f, 1.f + exp2f(fminf(s * a.inv_cap2, 120.f))));
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(s * a.inv_cap2, 120.f)));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+    return a.cap_log2e - 2.f * a.cap_log2e * r;               // 1 - 2 / (1 + e^{2 y}) = tanh(y), absolute error of a few 1e-7
 }
 
 template <bool GQA>
@@ -267,10 +270,13 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             float mt = -INFINITY;
             if (GQA && a.cap_log2e > 0.f) {
 #pragma unroll
-                for (int c = 0; c < KT; ++c) {
-                    x[c] = !need_mask || (c < vis && c >= inv) ? capped_log2(x[c], a) : -INFINITY;
-                    mt = fmaxf(mt, x[c]);
+                for (int c = 0; c < KT; ++c) x[c] = capped_log2(x[c], a);       // no branch around it: the 128 chains overlap
+                if (need_mask) {
+#pragma unroll
+                    for (int c = 0; c < KT; ++c) x[c] = (c < vis && c >= inv) ? x[c] : -INFINITY;
                 }
+#pragma unroll
+                for (int c = 0; c < KT; ++c) mt = fmaxf(mt, x[c]);
             } else if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) { x[c] = (c < vis && c >= inv) ? x[c] * a.scale_log2e : -INFINITY; mt = fmaxf(mt, x[c]); }

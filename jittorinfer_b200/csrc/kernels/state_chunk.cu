@@ -99,6 +99,20 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// log(1 + e^x) to a few ulp: max(x, 0) + log(1 + y) with y = e^-|x|, and log(1 + y) = 2 atanh(t), t = y / (2 + y) <= 1 / 3, by its
+// power series.
+__device__ __forceinline__ float softplus_series(float x) {
+    const float y = ex2(-fabsf(x) * LOG2E), t = __fdividef(y, 2.f + y), z = t * t;
+    float s = 1.f / 15.f;
+    s = s * z + 1.f / 13.f;
+    s = s * z + 1.f / 11.f;
+    s = s * z + 1.f / 9.f;
+    s = s * z + 1.f / 7.f;
+    s = s * z + 1.f / 5.f;
+    s = s * z + 1.f / 3.f;
+    s = s * z + 1.f;
+    return fmaxf(x, 0.f) + 2.f * t * s;
+}
 // x = hi + lo, both bf16; two numbers packed
 __device__ __forceinline__ void split2(float x, float y, uint32_t & hi, uint32_t & lo) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
@@ -121,7 +135,7 @@ template <int K> __device__ __forceinline__ void put_tile4(uint8_t * hi, int r, 
 template <int K> constexpr int prep_smem(int V) { return 4 * (3 * C * (K + 4) + C * (V + 4) + C * 36 + 3 * C); }
 
 template <int KIND, int K>
-__global__ void __launch_bounds__(NT) chunk_prepare_kernel(const __grid_constant__ jib_state_mix a) {
+__global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<KIND, K>;
     constexpr int KS = K + 4;
     extern __shared__ __align__(16) float sm[];
@@ -165,10 +179,10 @@ __global__ void __launch_bounds__(NT) chunk_prepare_kernel(const __grid_constant
 #pragma unroll
             for (int r = 0; r < 8; ++r) {
                 const float s = KIND == DELTA ? 1.f : -1.f;
-                x[r][0] = run + r < n ? f * softplus(s * (x[r][0] + bias.x)) : 0.f;
-                x[r][1] = run + r < n ? f * softplus(s * (x[r][1] + bias.y)) : 0.f;
-                x[r][2] = run + r < n ? f * softplus(s * (x[r][2] + bias.z)) : 0.f;
-                x[r][3] = run + r < n ? f * softplus(s * (x[r][3] + bias.w)) : 0.f;
+                x[r][0] = run + r < n ? f * softplus_series(s * (x[r][0] + bias.x)) : 0.f;
+                x[r][1] = run + r < n ? f * softplus_series(s * (x[r][1] + bias.y)) : 0.f;
+                x[r][2] = run + r < n ? f * softplus_series(s * (x[r][2] + bias.z)) : 0.f;
+                x[r][3] = run + r < n ? f * softplus_series(s * (x[r][3] + bias.w)) : 0.f;
             }
         }
 #pragma unroll

@@ -221,47 +221,110 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
 }
 
 // ---- gate and norm of the read-out ---------------------------------------------------------------------------------------------
-// DELTA / LINEAR: one warp per (token, head): o / rms(o) * norm_w * gate.
-template <typename T, int KIND>
+// Vectors of E adjacent values (E 4 or 1: rows of any size and alignment).
+template <int E> struct Vals { float v[E]; };
+template <int E> __device__ __forceinline__ Vals<E> load_vals(const float * p) {
+    Vals<E> r;
+    if (E == 4) *(float4 *) r.v = *(const float4 *) p;
+    else r.v[0] = *p;
+    return r;
+}
+template <int E> __device__ __forceinline__ Vals<E> load_vals(const bf16 * p) {
+    Vals<E> r;
+    if (E == 4) {
+        const uint2 x = *(const uint2 *) p;
+        const float2 a = __bfloat1622float2(*(const __nv_bfloat162 *) &x.x), b = __bfloat1622float2(*(const __nv_bfloat162 *) &x.y);
+        r.v[0] = a.x; r.v[1 % E] = a.y; r.v[2 % E] = b.x; r.v[3 % E] = b.y;
+    } else {
+        r.v[0] = to_f(*p);
+    }
+    return r;
+}
+template <int E> __device__ __forceinline__ void store_vals(float * p, const Vals<E> & r) {
+    if (E == 4) *(float4 *) p = *(const float4 *) r.v;
+    else *p = r.v[0];
+}
+template <int E> __device__ __forceinline__ void store_vals(bf16 * p, const Vals<E> & r) {
+    if (E == 4) {
+        uint2 x;
+        *(__nv_bfloat162 *) &x.x = __floats2bfloat162_rn(r.v[0], r.v[1 % E]);
+        *(__nv_bfloat162 *) &x.y = __floats2bfloat162_rn(r.v[2 % E], r.v[3 % E]);
+        *(uint2 *) p = x;
+    } else {
+        put(p, r.v[0]);
+    }
+}
+
+// DELTA / LINEAR: one warp per (token, head): o / rms(o) * norm_w * gate.  V <= 32 * N * E.
+template <typename T, int KIND, int E, int N>
 __global__ void __launch_bounds__(256) state_finish_kernel(const __grid_constant__ jib_state_mix a) {
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int lane = threadIdx.x & 31, t = blockIdx.y, h = blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (h >= a.H) return;
-    const float * o = a.o + ((size_t) t * a.H + h) * a.V;
+    const int lane = threadIdx.x & 31, i = blockIdx.x * 8 + (threadIdx.x >> 5), t = i / a.H, h = i % a.H, V = a.V;
+    if (t >= a.T) return;
+    const float * o = a.o + (size_t) i * V;
+    const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * V;
+    T * y = (T *) a.y + (size_t) t * a.ldy + h * V;
+    Vals<E> x[N], g[N], w[N];
     float ss = 0.f;
-    for (int c = lane; c < a.V; c += 32) ss += o[c] * o[c];
-    const float inv = a.out_scale * rsqrtf(warp_sum(ss) / (float) a.V + a.eps);
-    const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * a.V;
-    T * y = (T *) a.y + (size_t) t * a.ldy + h * a.V;
-    for (int c = lane; c < a.V; c += 32) {
-        const float g = to_f(gate[c]);
-        put(y + c, o[c] * inv * a.norm_w[c] * (KIND == DELTA ? sigmoid<T>(g) : silu<T>(g)));
+#pragma unroll
+    for (int k = 0; k < N; ++k) {                            // everything the row needs is requested before any of it is used
+        const int c = (lane + 32 * k) * E;
+        if (c >= V) continue;
+        x[k] = load_vals<E>(o + c);
+        g[k] = load_vals<E>(gate + c);
+        w[k] = load_vals<E>(a.norm_w + c);
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+        if ((lane + 32 * k) * E < V)
+#pragma unroll
+            for (int e = 0; e < E; ++e) ss += x[k].v[e] * x[k].v[e];
+    const float inv = a.out_scale * rsqrtf(warp_sum(ss) / (float) V + a.eps);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+        const int c = (lane + 32 * k) * E;
+        if (c >= V) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) x[k].v[e] *= inv * w[k].v[e] * (KIND == DELTA ? sigmoid<T>(g[k].v[e]) : silu<T>(g[k].v[e]));
+        store_vals<E>(y + c, x[k]);
     }
 }
 
 // SSD: one CTA per (token, part of the row): y = o * silu(gate), then y / rms(y) * norm_w over the part.
-template <typename T>
+template <typename T, int E>
 __global__ void __launch_bounds__(256) state_gate_norm_kernel(const __grid_constant__ jib_state_mix a) {
     PDL_TRIGGER_TOP();
     __shared__ float red[8];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int t = blockIdx.y, inner = a.H * a.V, m = inner / a.norm_groups, c0 = blockIdx.x * m;
-    const float * o = a.o + (size_t) t * inner + c0;
+    const float * o = a.o + (size_t) t * inner + c0, * w = a.norm_w + c0;
     const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + c0;
     T * y = (T *) a.y + (size_t) t * a.ldy + c0;
-    constexpr int KEEP = 16;                                 // values a thread holds; longer parts are computed twice
-    float v[KEEP], ss = 0.f;
+    constexpr int KEEP = 4;                                  // vectors a thread holds; longer parts are computed twice
+    Vals<E> v[KEEP], g[KEEP];
+    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
-        const int c = threadIdx.x + 256 * i;
-        v[i] = c < m ? o[c] * silu<T>(to_f(gate[c])) : 0.f;
-        ss += v[i] * v[i];
+        const int c = (threadIdx.x + 256 * i) * E;
+        if (c >= m) continue;
+        v[i] = load_vals<E>(o + c);
+        g[i] = load_vals<E>(gate + c);
     }
-    for (int c = threadIdx.x + 256 * KEEP; c < m; c += 256) {
-        const float x = o[c] * silu<T>(to_f(gate[c]));
-        ss += x * x;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+        if ((threadIdx.x + 256 * i) * E >= m) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            v[i].v[e] *= silu<T>(g[i].v[e]);
+            ss += v[i].v[e] * v[i].v[e];
+        }
     }
+    for (int c = (threadIdx.x + 256 * KEEP) * E; c < m; c += 256 * E)
+        for (int e = 0; e < E; ++e) {
+            const float x = o[c + e] * silu<T>(to_f(gate[c + e]));
+            ss += x * x;
+        }
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
@@ -271,16 +334,20 @@ __global__ void __launch_bounds__(256) state_gate_norm_kernel(const __grid_const
     const float inv = a.out_scale * rsqrtf(ss / (float) m + a.eps);
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
-        const int c = threadIdx.x + 256 * i;
-        if (c < m) put(y + c, v[i] * inv * a.norm_w[c0 + c]);
+        const int c = (threadIdx.x + 256 * i) * E;
+        if (c >= m) continue;
+        const Vals<E> n = load_vals<E>(w + c);
+#pragma unroll
+        for (int e = 0; e < E; ++e) v[i].v[e] *= inv * n.v[e];
+        store_vals<E>(y + c, v[i]);
     }
-    for (int c = threadIdx.x + 256 * KEEP; c < m; c += 256) put(y + c, o[c] * silu<T>(to_f(gate[c])) * inv * a.norm_w[c0 + c]);
+    for (int c = (threadIdx.x + 256 * KEEP) * E; c < m; c += 256 * E)
+        for (int e = 0; e < E; ++e) put(y + c + e, o[c + e] * silu<T>(to_f(gate[c + e])) * inv * w[c + e]);
 }
 
 // ---- single tokens -------------------------------------------------------------------------------------------------------------
-// grid (H, n_seqs): one CTA per head and sequence; thread = VEC adjacent columns x every NRG-th row of S, up to STEP_R rows in
-// registers (KEEP: all of them, the state is read once).
-constexpr int STEP_R = 16;
+// grid (H, n_seqs): one CTA per head and sequence; thread = VEC adjacent columns x every NRG-th row of S, up to R rows in registers
+// (KEEP: all of them, the state is read once).
 
 template <int VEC> struct Cols { float v[VEC]; };
 template <int VEC> __device__ __forceinline__ Cols<VEC> ld_cols(const float * p) {
@@ -294,8 +361,8 @@ template <int VEC> __device__ __forceinline__ void st_cols(float * p, const Cols
     else *p = c.v[0];
 }
 
-template <typename T, int KIND, int VEC, bool KEEP>
-__global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
+template <typename T, int KIND, int VEC, int R, bool KEEP>
+__global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const __grid_constant__ jib_state_mix a) {
     extern __shared__ float smem[];
     PDL_TRIGGER_TOP();
     const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, NT = blockDim.x;
@@ -312,10 +379,10 @@ __global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
     const int p = a.positions[t];
     const bool past = slot >= 0 && p > 0;
     float * st = a.state + ((size_t) (slot < 0 ? 0 : slot) * H + h) * K * V + cg * VEC;
-    Cols<VEC> s[STEP_R];
+    Cols<VEC> s[R];                                          // R rows
     auto load = [&](int r0) {
 #pragma unroll
-        for (int i = 0; i < STEP_R; ++i) {
+        for (int i = 0; i < R; ++i) {
             const int r = r0 + rg + i * nrg;
             if (past && live && r < K) {
                 s[i] = ld_cols<VEC>(st + (size_t) r * V);
@@ -328,9 +395,9 @@ __global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
     if (KEEP) load(0);                                       // in flight while the inputs are prepared
     const int hk = h / a.rep;
     for (int i = tid; i < (KIND == SSD ? 2 : 3) * K + V; i += NT) {
-        if (i < K) sq[i] = column<T>(a, t, a.q_off + hk * K + i, p, 0, slot);
-        else if (i < 2 * K) sk[i - K] = column<T>(a, t, a.k_off + hk * K + i - K, p, 0, slot);
-        else if (i < 2 * K + V) sv[i - 2 * K] = column<T>(a, t, a.v_off + h * V + i - 2 * K, p, 0, slot);
+        if (i < K) sq[i] = column_single<T>(a, t, a.q_off + hk * K + i, p, slot);
+        else if (i < 2 * K) sk[i - K] = column_single<T>(a, t, a.k_off + hk * K + i - K, p, slot);
+        else if (i < 2 * K + V) sv[i - 2 * K] = column_single<T>(a, t, a.v_off + h * V + i - 2 * K, p, slot);
         else {
             const int c = i - 2 * K - V, g = h * K + c;
             sd[c] = channel_decay<KIND>(a, to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + g]) + a.bias[g], h);
@@ -365,10 +432,10 @@ __global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
         Cols<VEC> d;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) d.v[e] = 0.f;
-        for (int r0 = 0; r0 < K; r0 += nrg * STEP_R) {
+        for (int r0 = 0; r0 < K; r0 += nrg * R) {
             if (!KEEP) load(r0);
 #pragma unroll
-            for (int i = 0; i < STEP_R; ++i) {
+            for (int i = 0; i < R; ++i) {
                 const int r = r0 + rg + i * nrg;
                 if (r >= K) continue;
                 const float g = sd[r], kk = sk[r] * kn;
@@ -393,10 +460,10 @@ __global__ void state_step_kernel(const __grid_constant__ jib_state_mix a) {
         }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) u.v[e] *= factor * kn;
-    for (int r0 = 0; r0 < K; r0 += nrg * STEP_R) {
+    for (int r0 = 0; r0 < K; r0 += nrg * R) {
         if (!KEEP) load(r0);
 #pragma unroll
-        for (int i = 0; i < STEP_R; ++i) {
+        for (int i = 0; i < R; ++i) {
             const int r = r0 + rg + i * nrg;
             if (r >= K || !live) continue;
             const float g = KIND == SSD ? decay : sd[r], kk = sk[r], qq = sq[r];
@@ -451,32 +518,46 @@ int launch_scan(const jib_state_mix & a, cudaStream_t s) {
 
 template <typename T, int KIND>
 int launch_finish(const jib_state_mix & a, cudaStream_t s) {
-    if (KIND == SSD) JIB_LAUNCH((state_gate_norm_kernel<T>), dim3(a.norm_groups, a.T), 256, 0, s, a);
-    else JIB_LAUNCH((state_finish_kernel<T, KIND>), dim3((a.H + 7) / 8, a.T), 256, 0, s, a);
+    const int part = KIND == SSD ? a.H * a.V / a.norm_groups : a.V;
+    const bool vec = part % 4 == 0 && a.ld_gate % 4 == 0 && a.ldy % 4 == 0 && (((uintptr_t) a.gate | (uintptr_t) a.y) & (4 * sizeof(T) - 1)) == 0;
+    if (KIND == SSD) {
+        if (vec) JIB_LAUNCH((state_gate_norm_kernel<T, 4>), dim3(a.norm_groups, a.T), 256, 0, s, a);
+        else JIB_LAUNCH((state_gate_norm_kernel<T, 1>), dim3(a.norm_groups, a.T), 256, 0, s, a);
+    } else {
+        const long long items = (long long) a.H * a.T;
+        const dim3 grid((unsigned) ((items + 7) / 8));
+        if (vec && a.V <= 128) JIB_LAUNCH((state_finish_kernel<T, KIND, 4, 1>), grid, 256, 0, s, a);
+        else if (vec && a.V <= 512) JIB_LAUNCH((state_finish_kernel<T, KIND, 4, 4>), grid, 256, 0, s, a);
+        else if (a.V <= 512) JIB_LAUNCH((state_finish_kernel<T, KIND, 1, 16>), grid, 256, 0, s, a);
+        else return JIB_E_ARG;
+    }
     return launched();
 }
 
-template <typename T, int KIND, int VEC, bool KEEP>
+template <typename T, int KIND, int VEC, int R, bool KEEP>
 int launch_step(const jib_state_mix & a, int nt, cudaStream_t s) {
     const int ncg = (a.V + VEC - 1) / VEC, nrg = nt / ncg;
     const int smem = (3 * a.K + (a.V + 3) / 4 * 4 + nrg * ncg * VEC + 2 + 32) * 4;
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
-    if (smem > 100 * 1024 || !jib::ensure_dyn_smem(state_step_kernel<T, KIND, VEC, KEEP>, 100 * 1024, done)) return JIB_E_ARG;
-    JIB_LAUNCH((state_step_kernel<T, KIND, VEC, KEEP>), dim3(a.H, a.n_seqs), nt, smem, s, a);
+    if (smem > 100 * 1024 || !jib::ensure_dyn_smem(state_step_kernel<T, KIND, VEC, R, KEEP>, 100 * 1024, done)) return JIB_E_ARG;
+    JIB_LAUNCH((state_step_kernel<T, KIND, VEC, R, KEEP>), dim3(a.H, a.n_seqs), nt, smem, s, a);
     return KIND == SSD ? launch_finish<T, SSD>(a, s) : launched();
+}
+template <typename T, int KIND, int VEC>
+int step(const jib_state_mix & a, cudaStream_t s) {
+    const int ncg = (a.V + VEC - 1) / VEC;
+    if (ncg > 512) return JIB_E_ARG;
+    const int nt = ncg > 256 || (long long) a.K * a.V >= 16384 ? 512 : 256, rows = nt / ncg;
+    if (rows * 4 >= a.K) return launch_step<T, KIND, VEC, 4, true>(a, nt, s);
+    if (rows * 8 >= a.K) return launch_step<T, KIND, VEC, 8, true>(a, nt, s);
+    if (rows * 16 >= a.K) return launch_step<T, KIND, VEC, 16, true>(a, nt, s);
+    return launch_step<T, KIND, VEC, 8, false>(a, nt, s);
 }
 
 template <typename T, int KIND>
 int run(const jib_state_mix & a, int single, cudaStream_t s) {
     if (single) {
-        const int vec = a.V % 4 == 0 && a.K % 4 == 0 ? 4 : 1;
-        const int ncg = (a.V + vec - 1) / vec;
-        if (ncg > 512) return JIB_E_ARG;
-        int nt = 256;
-        while (nt < 512 && ((nt / ncg) * STEP_R < a.K)) nt *= 2;
-        const bool keep = (nt / ncg) * STEP_R >= a.K;
-        if (vec == 4) return keep ? launch_step<T, KIND, 4, true>(a, nt, s) : launch_step<T, KIND, 4, false>(a, nt, s);
-        return keep ? launch_step<T, KIND, 1, true>(a, nt, s) : launch_step<T, KIND, 1, false>(a, nt, s);
+        return a.V % 4 == 0 && a.K % 4 == 0 ? step<T, KIND, 4>(a, s) : step<T, KIND, 1>(a, s);
     }
     if (sizeof(T) == 2 && a.chunk != nullptr && jib_state_chunk_ok(a)) {
         const int rc = jib_state_chunk_run(a, s);

@@ -75,6 +75,28 @@ __device__ __forceinline__ float column(const jib_state_mix & a, int t, int c, i
     return silu<T>(acc);
 }
 
+// The same for a single token (nothing of its sequence precedes it in the batch): up to 4 taps all loads are in flight together.
+template <typename T>
+__device__ __forceinline__ float column_single(const jib_state_mix & a, int t, int c, int p, int slot) {
+    if (a.taps > 4) return column<T>(a, t, c, p, 0, slot);
+    const float x = to_f(((const T *) a.proj)[(size_t) t * a.ld + c]);
+    if (a.taps == 0) return x;
+    const int w = c - a.conv0;
+    const T * ring = (const T *) a.conv_state + (size_t) (slot < 0 ? 0 : slot) * a.taps * a.n_conv + w;
+    float v[3], k[4];
+    int row = p % a.taps;
+#pragma unroll
+    for (int d = 1; d < 4; ++d) {                            // d tokens back
+        row = row == 0 ? a.taps - 1 : row - 1;
+        const bool in = d < a.taps && d <= p && slot >= 0;
+        v[d - 1] = in ? to_f(ring[(size_t) row * a.n_conv]) : 0.f;
+        k[d] = d < a.taps ? a.conv_w[(size_t) (a.taps - 1 - d) * a.n_conv + w] : 0.f;
+    }
+    k[0] = a.conv_w[(size_t) (a.taps - 1) * a.n_conv + w];
+    const float b = a.conv_b != nullptr ? a.conv_b[w] : 0.f;
+    return silu<T>(b + k[0] * x + k[1] * v[0] + k[2] * v[1] + k[3] * v[2]);
+}
+
 __device__ __forceinline__ void cp16(void * dst, const void * src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t) __cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
