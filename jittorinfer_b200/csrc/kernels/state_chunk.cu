@@ -10,7 +10,7 @@
 // Every exponent that occurs is a difference G_t - G_s with s <= t and so at most 0, however fast the decay: nothing overflows and no
 // quotient of vanishing products is formed.
 //   prepare (one CTA per chunk and head; SSD: per chunk and group): convolution, unit norm, decays, A, W, U0.  Independent of S.
-//   pass    (one CTA per head and 16 value columns): walks the chunks, S in registers, everything else a product of small matrices.
+//   pass    (one CTA per head and 16 value columns, SSD 32): walks the chunks, S in registers, everything else a product of small matrices.
 // State, decays, A, W, U0 are fp32; the tensor cores see each as a sum of two bf16 numbers and the products hi * hi + hi * lo + lo * hi
 // (about 16 bits of mantissa); q and k of SSD are bf16 to begin with.  Accumulation is fp32.
 #include "pdl.cuh"
@@ -22,7 +22,7 @@ using namespace state_mix;
 
 constexpr int C = 32, VB = 16, NT = 256, STAGES = 3;
 constexpr float LOG2E = 1.4426950408889634f;
-constexpr int QK_LD = 40;                                    // row stride of SSD's q . k table (fp32)
+constexpr int QK_LD = 32;                                    // row stride of SSD's q . k table (fp32)
 
 // A chunk's record: bf16 tiles of 32 rows x K columns in 16-byte units u of row r stored at u ^ (r & 7); A: 32 x 32, unit u ^ (r / 2 & 3).
 template <int KIND, int K> struct Rec {
@@ -388,22 +388,24 @@ __device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-constexpr int BS = 24;                                       // row stride of the [.][VB] bf16 operands (48 bytes: rows hit different banks)
+constexpr int BS = VB + 8;                                   // row stride of the [.][VB] bf16 operands (48 bytes: rows hit different banks)
 
 template <int KIND, int K> struct Pass {
     using R = Rec<KIND, K>;
-    static constexpr int X = (R::BYTES + 15) / 16 * 16;      // U0 fp32 [C][VB] (SSD: x bf16 [C][VB]), then SSD's factors fp32 [C]
-    static constexpr int STAGE = X + (KIND == SSD ? C * VB * 2 + C * 4 : C * VB * 4);
+    static constexpr int X = R::BYTES;                       // U0 fp32 [C][VB]
+    static constexpr int STAGE = X + C * VB * 4;
     static constexpr int S = STAGES * STAGE;                 // S hi, lo [K][BS]
-    static constexpr int U = S + 2 * K * BS * 2;             // U hi, lo [C][BS] (SSD: then the decayed ones)
-    static constexpr int SMEM = U + (KIND == SSD ? 4 : 2) * C * BS * 2;
+    static constexpr int U = S + 2 * K * BS * 2;             // U hi, lo [C][BS]
+    static constexpr int SMEM = U + 2 * C * BS * 2;
 };
 
+// DELTA, LINEAR.  Warps 0 - 3 own a 16 x 8 tile of o each, warps 4 - 7 one of u; all warps own tiles of S.  Two barriers per chunk: u is
+// there (and so is the next chunk's record), S is there.  Operands that depend on neither are in registers by then.
 template <int KIND, int K>
-__global__ void __launch_bounds__(NT) chunk_pass_kernel(const __grid_constant__ jib_state_mix a) {
+__global__ void __launch_bounds__(NT, 1) chunk_pass_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<KIND, K>;
     using P = Pass<KIND, K>;
-    constexpr int TPW = K / 64;                              // 16 x 8 tiles of S per warp: K / 16 x 2 tiles over 8 warps
+    constexpr int TPW = K / 64;                              // 16 x 8 tiles of S per warp (K / 16 x 2 over 8 warps), side by side
     extern __shared__ __align__(16) uint8_t smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int splits = a.V / VB, h = blockIdx.x / splits, vs = blockIdx.x % splits, b = blockIdx.y, V = a.V, H = a.H;
@@ -411,169 +413,368 @@ __global__ void __launch_bounds__(NT) chunk_pass_kernel(const __grid_constant__ 
     const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
     if (n <= 0) return;
     const int slot = checked_slot(a, b, 46);
-    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
-    const int chunks = (n + C - 1) / C, c0 = chunk_key(a.q_start, b);
+    const int chunks = (n + C - 1) / C;
+    const uint8_t * rec0 = (const uint8_t *) a.chunk + ((size_t) chunk_key(a.q_start, b) * H + h) * (R::BYTES + C * 4 * V);
+    const size_t rec_step = (size_t) H * (R::BYTES + C * 4 * V);
     auto stage = [&](int i) {
         if (i < chunks) {
             uint8_t * dst = smem + i % STAGES * P::STAGE;
-            if (KIND == SSD) {
-                const int groups = H / a.rep, m = min(C, n - i * C);
-                const uint8_t * src = (const uint8_t *) a.chunk + ((size_t) (c0 + i) * groups + h / a.rep) * R::BYTES;
-                for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
-                const size_t row = r0 + i * C;
-                if (tid < 2 * m) cp16(dst + P::X + tid * 16, (const bf16 *) a.v + (row + (tid >> 1)) * H * V + h * V + vs * VB + (tid & 1) * 8);
-                if (tid < m) cp4(dst + P::X + C * VB * 2 + tid * 4, a.s + (row + tid) * H + h);
-            } else {
-                const uint8_t * src = (const uint8_t *) a.chunk + ((size_t) (c0 + i) * H + h) * (R::BYTES + C * 4 * V);
-                for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
-                if (tid < C * VB / 4) cp16(dst + P::X + tid * 16, src + R::BYTES + vs * (C * VB * 4) + tid * 16);
-            }
+            const uint8_t * src = rec0 + i * rec_step;
+            for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
+            if (tid < C * VB / 4) cp16(dst + P::X + tid * 16, src + R::BYTES + vs * (C * VB * 4) + tid * 16);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-#pragma unroll
-    for (int i = 0; i < STAGES - 1; ++i) stage(i);
+    stage(0);
+    stage(1);
+    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
 
     bf16 * Sh = (bf16 *) (smem + P::S), * Uh = (bf16 *) (smem + P::U);
     const uint32_t S_addr = sm100::smem_u32(Sh), U_addr = sm100::smem_u32(Uh);
     constexpr uint32_t S_LO = K * BS * 2, U_LO = C * BS * 2;
     const int fr = lane >> 2, fc = (lane & 3) * 2;           // accumulator element: rows fr, fr + 8, columns fc, fc + 1
-    // ldmatrix lane addresses: operand rows (x4: 16 rows x 2 units), transposed ones
-    const int lr = lane & 15, lu = lane >> 4;
-    const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;         // k^T tiles: rows = tokens
-    const int br = lane & 31;                                // [k][n] operands: 32 rows of one 8-column unit
+    const int lr = lane & 15, lu = lane >> 4;                // ldmatrix lane addresses: operand rows (16 rows x 2 units) ...
+    const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;         // ... and k^T tiles (rows = tokens)
+    const int mt = (warp >> 1) & 1, nt = warp & 1;           // this warp's tile of o or u
+    const bool is_o = warp < 4;
+    const int sm_ = warp * TPW >> 1, sn0 = TPW == 2 ? 0 : warp & 1;               // tiles of S: rows 16 sm_, columns 8 (sn0 + i)
     float st[TPW][4];
-    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K) * V + vs * VB;
+    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + sm_ * 16 + fr) * V + vs * VB + fc;
     const bool past = slot >= 0 && a.positions[r0] > 0;
 #pragma unroll
-    for (int i = 0; i < TPW; ++i) {
-        const int m = (warp * TPW + i) >> 1, nt = (warp * TPW + i) & 1;
-        const float * p = state + (size_t) (m * 16 + fr) * V + nt * 8 + fc;
-        const float2 x = past ? *(const float2 *) p : make_float2(0.f, 0.f), y = past ? *(const float2 *) (p + (size_t) 8 * V) : make_float2(0.f, 0.f);
-        st[i][0] = x.x; st[i][1] = x.y; st[i][2] = y.x; st[i][3] = y.y;
-    }
+    for (int i = 0; i < TPW; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const float2 x = past ? *(const float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) : make_float2(0.f, 0.f);
+            st[i][2 * e] = x.x;
+            st[i][2 * e + 1] = x.y;
+        }
     auto publish_state = [&]() {
 #pragma unroll
-        for (int i = 0; i < TPW; ++i) {
-            const int m = (warp * TPW + i) >> 1, nt = (warp * TPW + i) & 1;
+        for (int i = 0; i < TPW; ++i)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 uint32_t hi, lo;
                 split2(st[i][2 * e], st[i][2 * e + 1], hi, lo);
-                bf16 * p = Sh + (m * 16 + fr + 8 * e) * BS + nt * 8 + fc;
+                bf16 * p = Sh + (sm_ * 16 + fr + 8 * e) * BS + (sn0 + i) * 8 + fc;
                 *(uint32_t *) p = hi;
                 *(uint32_t *) (p + K * BS) = lo;
             }
+    };
+    uint32_t xh[K / 16][4], xl[K / 16][4];                   // q e^G or W rows of this warp's tile
+    auto load_rows = [&](int ch) {
+        if (!is_o && KIND == LINEAR) return;
+        const int r = mt * 16 + lr;
+        const uint32_t base = sm100::smem_u32(smem + ch % STAGES * P::STAGE) + (is_o ? R::Q : R::W) + r * (K * 2);
+#pragma unroll
+        for (int kk = 0; kk < K / 16; ++kk) {
+            ldm4(xh[kk], base + (((kk * 2 + lu) ^ (r & 7)) << 4));
+            ldm4(xl[kk], base + R::TILE + (((kk * 2 + lu) ^ (r & 7)) << 4));
         }
     };
     publish_state();
-    const int mt = (warp >> 1) & 1, nt = warp & 1;           // this warp's 16 x 8 tile of o (warps 0 - 3) or u (4 - 7)
-    const bool is_o = warp < 4;
-    const float na = KIND == SSD ? a.neg_a[h] * LOG2E : 0.f, skip = KIND == SSD ? a.skip[h] : 0.f;
-
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    load_rows(0);
     for (int ch = 0; ch < chunks; ++ch) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
-        __syncthreads();                                     // this chunk's record and S are there; the buffer before it is free
-        stage(ch + STAGES - 1);
+        stage(ch + 2);                                       // into the buffer of chunk ch - 1
         const uint8_t * rec = smem + ch % STAGES * P::STAGE;
         const uint32_t rec_addr = sm100::smem_u32(rec);
-        const int m = min(C, n - ch * C);
-        float g = 0.f;                                       // SSD: lane t holds G_t
-        if (KIND == SSD) {
-            g = lane < m ? na * ((const float *) (rec + P::X + C * VB * 2))[lane] : 0.f;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float x = __shfl_up_sync(0xffffffffu, g, o);
-                if (lane >= o) g += x;
-            }
-        }
-        float acc[3][4];
-#pragma unroll
-        for (int i = 0; i < 3; ++i)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
         if (is_o || KIND == DELTA) {
-            const uint32_t base = rec_addr + (is_o ? R::Q : R::W);
+            float acc[4][4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
 #pragma unroll
             for (int kk = 0; kk < K / 32; ++kk) {            // 32 channels at a time
                 uint32_t bh[4], bl[4];
-                const uint32_t off = ((kk * 32 + br) * BS + nt * 8) * 2;
+                const uint32_t off = ((kk * 32 + lane) * BS + nt * 8) * 2;
                 ldm4t(bh, S_addr + off);
                 ldm4t(bl, S_addr + S_LO + off);
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    const int r = mt * 16 + lr, u = kk * 4 + e * 2 + lu;
-                    uint32_t x[4];
-                    ldm4(x, base + r * (K * 2) + ((u ^ (r & 7)) << 4));
-                    mma(acc[0], x, bh[2 * e], bh[2 * e + 1]);
-                    mma(acc[1], x, bl[2 * e], bl[2 * e + 1]);
-                    if (KIND != SSD) {
-                        ldm4(x, base + R::TILE + r * (K * 2) + ((u ^ (r & 7)) << 4));
-                        mma(acc[2], x, bh[2 * e], bh[2 * e + 1]);
-                    }
+                    mma(acc[e], xh[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
+                    mma(acc[2], xh[2 * kk + e], bl[2 * e], bl[2 * e + 1]);
+                    mma(acc[3], xl[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
                 }
             }
-        }
-        float o[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[e] = acc[0][e] + (acc[1][e] + acc[2][e]);
+            for (int e = 0; e < 4; ++e) o[e] = (acc[0][e] + acc[1][e]) + (acc[2][e] + acc[3][e]);
+        }
         if (!is_o) {                                         // u of this chunk as an operand
-            const int t = mt * 16 + fr, c = nt * 8 + fc;
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const int row = t + 8 * e;
+                const int row = mt * 16 + fr + 8 * e, c = nt * 8 + fc;
+                const float2 x = *(const float2 *) (rec + P::X + (row * VB + c) * 4);
                 uint32_t hi, lo;
+                split2(x.x - o[2 * e], x.y - o[2 * e + 1], hi, lo);
                 bf16 * p = Uh + row * BS + c;
-                if (KIND == SSD) {
-                    float2 x = make_float2(0.f, 0.f);
-                    float f = 0.f;
-                    if (row < m) {
-                        x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (row * VB + c) * 2));
-                        f = ((const float *) (rec + P::X + C * VB * 2))[row];
-                    }
-                    const float w = f * ex2(__shfl_sync(0xffffffffu, g, 31) - __shfl_sync(0xffffffffu, g, row));
-                    split2(x.x * f, x.y * f, hi, lo);
-                    *(uint32_t *) p = hi;
-                    *(uint32_t *) (p + C * BS) = lo;
-                    split2(x.x * w, x.y * w, hi, lo);
-                    *(uint32_t *) (p + 2 * C * BS) = hi;
-                    *(uint32_t *) (p + 3 * C * BS) = lo;
-                } else {
-                    const float2 x = *(const float2 *) (rec + P::X + (row * VB + c) * 4);
-                    split2(x.x - o[2 * e], x.y - o[2 * e + 1], hi, lo);
-                    *(uint32_t *) p = hi;
-                    *(uint32_t *) (p + C * BS) = lo;
-                }
+                *(uint32_t *) p = hi;
+                *(uint32_t *) (p + C * BS) = lo;
             }
         }
-        __syncthreads();
+        // what the second half needs of the record
+        uint32_t dh[2][4], dl[2][4], ah[2][4], al[2][4];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int r = e * 16 + tr;
+            const uint32_t d = rec_addr + R::D + r * (K * 2) + (((sm_ * 2 + tu) ^ (r & 7)) << 4);
+            ldm4t(dh[e], d);
+            ldm4t(dl[e], d + R::TILE);
+            if (is_o) {
+                const int q = mt * 16 + lr;
+                const uint32_t p = rec_addr + R::A + q * 64 + (((e * 2 + lu) ^ ((q >> 1) & 3)) << 4);
+                ldm4(ah[e], p);
+                ldm4(al[e], p + R::ATILE);
+            }
+        }
+        const float * E = (const float *) (rec + R::E) + sm_ * 16 + fr;
+        const float e0 = E[0], e1 = E[8];
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();                                     // u, and the next chunk's record
+        uint32_t uh[2][4], ul[2][4];                         // both 8-column units of u
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            ldm4t(uh[i], U_addr + (lane * BS + i * 8) * 2);
+            ldm4t(ul[i], U_addr + U_LO + (lane * BS + i * 8) * 2);
+        }
+        // S' = e^{G_C} S + (k e^{G_C - G})^T u
+#pragma unroll
+        for (int i = 0; i < TPW; ++i) {
+            const int c = TPW == 2 ? i : sn0;
+            float p1[4] = {0.f, 0.f, 0.f, 0.f}, p2[4] = {0.f, 0.f, 0.f, 0.f};
+            st[i][0] *= e0; st[i][1] *= e0; st[i][2] *= e1; st[i][3] *= e1;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const uint32_t h0 = c ? uh[1][2 * e] : uh[0][2 * e], h1 = c ? uh[1][2 * e + 1] : uh[0][2 * e + 1];
+                const uint32_t l0 = c ? ul[1][2 * e] : ul[0][2 * e], l1 = c ? ul[1][2 * e + 1] : ul[0][2 * e + 1];
+                mma(st[i], dh[e], h0, h1);
+                mma(p1, dh[e], l0, l1);
+                mma(p2, dl[e], h0, h1);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[i][e] += p1[e] + p2[e];
+        }
+        publish_state();                                     // its readers of this chunk are behind the barrier above
         if (is_o) {
             float p[3][4];
 #pragma unroll
             for (int i = 0; i < 3; ++i)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) p[i][e] = 0.f;
-            uint32_t bh[4], bl[4];
-            const uint32_t off = (br * BS + nt * 8) * 2;
-            ldm4t(bh, U_addr + off);
-            ldm4t(bl, U_addr + U_LO + off);
-            const float g0 = __shfl_sync(0xffffffffu, g, mt * 16 + fr), g1 = __shfl_sync(0xffffffffu, g, mt * 16 + fr + 8);
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                uint32_t xh[4], xl[4];
-                if (KIND == SSD) {                           // A = q . k times the decay between the two tokens
+                const uint32_t h0 = nt ? uh[1][2 * e] : uh[0][2 * e], h1 = nt ? uh[1][2 * e + 1] : uh[0][2 * e + 1];
+                const uint32_t l0 = nt ? ul[1][2 * e] : ul[0][2 * e], l1 = nt ? ul[1][2 * e + 1] : ul[0][2 * e + 1];
+                mma(p[0], ah[e], h0, h1);
+                mma(p[1], ah[e], l0, l1);
+                mma(p[2], al[e], h0, h1);
+            }
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {            // rows fr + 8 (j & 1), columns 16 e + 8 (j >> 1) + fc
-                        const int t = mt * 16 + fr + 8 * (j & 1), s = e * 16 + 8 * (j >> 1) + fc;
-                        const float gt = (j & 1) ? g1 : g0, s0 = __shfl_sync(0xffffffffu, g, s), s1 = __shfl_sync(0xffffffffu, g, s + 1);
-                        const float2 x = *(const float2 *) (rec + R::A + (t * QK_LD + s) * 4);
-                        split2(s <= t ? x.x * ex2(gt - s0) : 0.f, s + 1 <= t ? x.y * ex2(gt - s1) : 0.f, xh[j], xl[j]);
-                    }
-                } else {
-                    const int r = mt * 16 + lr, u = e * 2 + lu;
-                    ldm4(xh, rec_addr + R::A + r * 64 + ((u ^ ((r >> 1) & 3)) << 4));
-                    ldm4(xl, rec_addr + R::A + R::ATILE + r * 64 + ((u ^ ((r >> 1) & 3)) << 4));
-                }
+            for (int e = 0; e < 2; ++e) {
+                const int t = ch * C + mt * 16 + fr + 8 * e;
+                if (t < n)
+                    *(float2 *) (a.o + ((size_t) (r0 + t) * H + h) * V + vs * VB + nt * 8 + fc) =
+                        make_float2(o[2 * e] + p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]), o[2 * e + 1] + p[0][2 * e + 1] + (p[1][2 * e + 1] + p[2][2 * e + 1]));
+            }
+        }
+        if (ch + 1 < chunks) load_rows(ch + 1);
+        __syncthreads();                                     // S; this chunk's record is free
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (slot >= 0) {
+#pragma unroll
+        for (int i = 0; i < TPW; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) *(float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) = make_float2(st[i][2 * e], st[i][2 * e + 1]);
+    }
+}
+
+// SSD: 32 value columns per CTA; every warp owns a 16 x 8 tile of o and K / 32 tiles of S.  q and k are bf16, so only A, u and S are split.
+constexpr int SV = 32, SB = SV + 8;                          // 80-byte rows hit different banks
+template <int K> struct PassSsd {
+    using R = Rec<SSD, K>;
+    static constexpr int X = R::BYTES;                       // x bf16 [C][SV], factors fp32 [C]
+    static constexpr int STAGE = X + C * SV * 2 + C * 4;
+    static constexpr int S = STAGES * STAGE;                 // S hi, lo [K][SB]
+    static constexpr int U = S + 2 * K * SB * 2;             // s x and its decayed form: hi, lo, hi, lo [C][SB]
+    static constexpr int A = U + 4 * C * SB * 2;             // A hi, lo
+    static constexpr int SMEM = A + 2 * R::ATILE;
+};
+
+template <int K>
+__global__ void __launch_bounds__(NT, 1) chunk_pass_ssd_kernel(const __grid_constant__ jib_state_mix a) {
+    using R = Rec<SSD, K>;
+    using P = PassSsd<K>;
+    constexpr int TPW = K / 32;
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int V = a.V, H = a.H, splits = (V + SV - 1) / SV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * SV, b = blockIdx.y;
+    const int units = min(SV, V - v0) / 8;                   // 8-column units that exist
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
+    if (n <= 0) return;
+    const int slot = checked_slot(a, b, 46), groups = H / a.rep;
+    const int chunks = (n + C - 1) / C;
+    const uint8_t * rec0 = (const uint8_t *) a.chunk + ((size_t) chunk_key(a.q_start, b) * groups + h / a.rep) * R::BYTES;
+    auto stage = [&](int i) {
+        if (i < chunks) {
+            uint8_t * dst = smem + i % STAGES * P::STAGE;
+            const uint8_t * src = rec0 + (size_t) i * groups * R::BYTES;
+            for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
+            const int m = min(C, n - i * C), row = tid >> 2, u = tid & 3;
+            if (row < m && u < units) cp16(dst + P::X + tid * 16, (const bf16 *) a.v + (size_t) (r0 + i * C + row) * H * V + h * V + v0 + u * 8);
+            if (tid < m) cp4(dst + P::X + C * SV * 2 + tid * 4, a.s + (size_t) (r0 + i * C + tid) * H + h);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(0);
+    stage(1);
+    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
+
+    bf16 * Sh = (bf16 *) (smem + P::S), * Uh = (bf16 *) (smem + P::U);
+    const uint32_t S_addr = sm100::smem_u32(Sh), U_addr = sm100::smem_u32(Uh), A_addr = sm100::smem_u32(smem + P::A);
+    constexpr uint32_t S_LO = K * SB * 2, U_LO = C * SB * 2;
+    const int fr = lane >> 2, fc = (lane & 3) * 2, lr = lane & 15, lu = lane >> 4;
+    const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;
+    const int mt = warp >> 2, nt = warp & 3;
+    const int sm_ = warp * TPW >> 2, sn0 = TPW == 4 ? 0 : (warp & 1) * 2;
+    float st[TPW][4];
+    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + sm_ * 16 + fr) * V + v0 + fc;
+    const bool past = slot >= 0 && a.positions[r0] > 0;
+#pragma unroll
+    for (int i = 0; i < TPW; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const float2 x = past && sn0 + i < units ? *(const float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) : make_float2(0.f, 0.f);
+            st[i][2 * e] = x.x;
+            st[i][2 * e + 1] = x.y;
+        }
+    auto publish_state = [&]() {
+#pragma unroll
+        for (int i = 0; i < TPW; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                uint32_t hi, lo;
+                split2(st[i][2 * e], st[i][2 * e + 1], hi, lo);
+                bf16 * p = Sh + (sm_ * 16 + fr + 8 * e) * SB + (sn0 + i) * 8 + fc;
+                *(uint32_t *) p = hi;
+                *(uint32_t *) (p + K * SB) = lo;
+            }
+    };
+    uint32_t xq[K / 16][4], xk[2][4];                        // rows of q of this warp's tile; k^T of its tiles of S
+    auto load_rows = [&](int ch) {
+        const uint32_t rec = sm100::smem_u32(smem + ch % STAGES * P::STAGE);
+        const int r = mt * 16 + lr;
+#pragma unroll
+        for (int kk = 0; kk < K / 16; ++kk) ldm4(xq[kk], rec + R::Q + r * (K * 2) + (((kk * 2 + lu) ^ (r & 7)) << 4));
+    };
+    const float na = a.neg_a[h] * LOG2E, skip = a.skip[h];
+    publish_state();
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    load_rows(0);
+    for (int ch = 0; ch < chunks; ++ch) {
+        stage(ch + 2);                                       // into the buffer of chunk ch - 1
+        const uint8_t * rec = smem + ch % STAGES * P::STAGE;
+        const uint32_t rec_addr = sm100::smem_u32(rec);
+        const int m = min(C, n - ch * C);
+        const float * factor = (const float *) (rec + P::X + C * SV * 2);
+        float acc[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < K / 32; ++kk) {
+            uint32_t bh[4], bl[4];
+            const uint32_t off = ((kk * 32 + lane) * SB + nt * 8) * 2;
+            ldm4t(bh, S_addr + off);
+            ldm4t(bl, S_addr + S_LO + off);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                mma(acc[e], xq[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
+                mma(acc[2 + e], xq[2 * kk + e], bl[2 * e], bl[2 * e + 1]);
+            }
+        }
+        // lane t: G_t
+        float g = lane < m ? na * factor[lane] : 0.f;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float x = __shfl_up_sync(0xffffffffu, g, o);
+            if (lane >= o) g += x;
+        }
+        const float gC = __shfl_sync(0xffffffffu, g, 31);
+        {   // s x and s x e^{G_C - G}: 4 columns of a row per thread
+            const int row = tid >> 3, c = (tid & 7) * 4;
+            const float f = row < m ? factor[row] : 0.f, w = f * ex2(gC - __shfl_sync(0xffffffffu, g, row));
+            float x[4] = {0.f, 0.f, 0.f, 0.f};
+            if (row < m) load4((const bf16 *) (rec + P::X) + row * SV + c, x);
+            uint2 hi, lo;
+            bf16 * p = Uh + row * SB + c;
+            split2(x[0] * f, x[1] * f, hi.x, lo.x);
+            split2(x[2] * f, x[3] * f, hi.y, lo.y);
+            *(uint2 *) p = hi;
+            *(uint2 *) (p + C * SB) = lo;
+            split2(x[0] * w, x[1] * w, hi.x, lo.x);
+            split2(x[2] * w, x[3] * w, hi.y, lo.y);
+            *(uint2 *) (p + 2 * C * SB) = hi;
+            *(uint2 *) (p + 3 * C * SB) = lo;
+        }
+#pragma unroll
+        for (int k = 0; k < C / 8; ++k) {                    // A = q . k times the decay between the two tokens: 4 rows per warp
+            const int t = warp * (C / 8) + k;
+            const float gt = __shfl_sync(0xffffffffu, g, t);                         // by all lanes, outside the condition
+            const float x = lane <= t ? ((const float *) (rec + R::A))[t * QK_LD + lane] * ex2(gt - g) : 0.f;
+            const bf16 hi = __float2bfloat16(x);
+            *(bf16 *) (smem + P::A + a_off(t, lane)) = hi;
+            *(bf16 *) (smem + P::A + R::ATILE + a_off(t, lane)) = __float2bfloat16(x - to_f(hi));
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int r = e * 16 + tr;
+            ldm4t(xk[e], rec_addr + R::D + r * (K * 2) + (((sm_ * 2 + tu) ^ (r & 7)) << 4));
+        }
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();                                     // u, A, and the next chunk's record
+        const float decay = ex2(gC);
+#pragma unroll
+        for (int i = 0; i < TPW; ++i) {
+            uint32_t bh[4], bl[4];
+            const uint32_t off = (lane * SB + (sn0 + i) * 8) * 2;
+            ldm4t(bh, U_addr + 2 * U_LO + off);
+            ldm4t(bl, U_addr + 3 * U_LO + off);
+            float p1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[i][e] *= decay;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                mma(st[i], xk[e], bh[2 * e], bh[2 * e + 1]);
+                mma(p1, xk[e], bl[2 * e], bl[2 * e + 1]);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) st[i][e] += p1[e];
+        }
+        publish_state();                                     // its readers of this chunk are behind the barrier above
+        {
+            float p[3][4];
+#pragma unroll
+            for (int i = 0; i < 3; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) p[i][e] = 0.f;
+            uint32_t bh[4], bl[4], xh[4], xl[4];
+            const float w0 = ex2(__shfl_sync(0xffffffffu, g, mt * 16 + fr)), w1 = ex2(__shfl_sync(0xffffffffu, g, mt * 16 + fr + 8));
+            const uint32_t off = (lane * SB + nt * 8) * 2;
+            ldm4t(bh, U_addr + off);
+            ldm4t(bl, U_addr + U_LO + off);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int r = mt * 16 + lr;
+                const uint32_t q = A_addr + r * 64 + (((e * 2 + lu) ^ ((r >> 1) & 3)) << 4);
+                ldm4(xh, q);
+                ldm4(xl, q + R::ATILE);
                 mma(p[0], xh, bh[2 * e], bh[2 * e + 1]);
                 mma(p[1], xh, bl[2 * e], bl[2 * e + 1]);
                 mma(p[2], xl, bh[2 * e], bh[2 * e + 1]);
@@ -581,88 +782,54 @@ __global__ void __launch_bounds__(NT) chunk_pass_kernel(const __grid_constant__ 
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int t = mt * 16 + fr + 8 * e, c = nt * 8 + fc;
-                if (t >= m) continue;
-                float2 y = make_float2(p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]), p[0][2 * e + 1] + (p[1][2 * e + 1] + p[2][2 * e + 1]));
-                if (KIND == SSD) {
-                    const float w = ex2(e ? g1 : g0);
-                    const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (t * VB + c) * 2));
-                    y.x += w * o[2 * e] + skip * x.x;
-                    y.y += w * o[2 * e + 1] + skip * x.y;
-                } else {
-                    y.x += o[2 * e];
-                    y.y += o[2 * e + 1];
-                }
-                *(float2 *) (a.o + ((size_t) (r0 + ch * C + t) * H + h) * V + vs * VB + c) = y;
+                const float w = e ? w1 : w0;
+                if (t >= m || nt >= units) continue;
+                const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (t * SV + c) * 2));
+                float2 y;
+                y.x = w * ((acc[0][2 * e] + acc[1][2 * e]) + (acc[2][2 * e] + acc[3][2 * e])) + p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]) + skip * x.x;
+                y.y = w * ((acc[0][2 * e + 1] + acc[1][2 * e + 1]) + (acc[2][2 * e + 1] + acc[3][2 * e + 1])) + p[0][2 * e + 1] +
+                      (p[1][2 * e + 1] + p[2][2 * e + 1]) + skip * x.y;
+                *(float2 *) (a.o + ((size_t) (r0 + ch * C + t) * H + h) * V + v0 + c) = y;
             }
         }
-        // S' = decay S + k^T u
-        const float gC = __shfl_sync(0xffffffffu, g, 31);
-#pragma unroll
-        for (int i = 0; i < TPW; ++i) {
-            const int sm_ = (warp * TPW + i) >> 1, sn = (warp * TPW + i) & 1;
-            uint32_t bh[4], bl[4];
-            const uint32_t off = (br * BS + sn * 8) * 2 + (KIND == SSD ? 2 * U_LO : 0);
-            ldm4t(bh, U_addr + off);
-            ldm4t(bl, U_addr + U_LO + off);
-            float e0, e1;
-            if (KIND == SSD) {
-                e0 = e1 = ex2(gC);
-            } else {
-                const float * E = (const float *) (rec + R::E) + sm_ * 16 + fr;
-                e0 = E[0];
-                e1 = E[8];
-            }
-            st[i][0] *= e0; st[i][1] *= e0; st[i][2] *= e1; st[i][3] *= e1;
-            float p1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = e * 16 + tr, u = sm_ * 2 + tu;
-                uint32_t x[4];
-                ldm4t(x, rec_addr + R::D + r * (K * 2) + ((u ^ (r & 7)) << 4));
-                mma(st[i], x, bh[2 * e], bh[2 * e + 1]);
-                mma(p1, x, bl[2 * e], bl[2 * e + 1]);
-                if (KIND != SSD) {
-                    ldm4t(x, rec_addr + R::D + R::TILE + r * (K * 2) + ((u ^ (r & 7)) << 4));
-                    mma(p1, x, bh[2 * e], bh[2 * e + 1]);
-                }
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) st[i][e] += p1[e];
-        }
-        publish_state();                                     // its readers of this chunk are behind the barrier above
+        if (ch + 1 < chunks) load_rows(ch + 1);
+        __syncthreads();                                     // S; this chunk's record is free
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    PDL_TRIGGER_LATE();
     if (slot >= 0) {
 #pragma unroll
-        for (int i = 0; i < TPW; ++i) {
-            const int m = (warp * TPW + i) >> 1, nt2 = (warp * TPW + i) & 1;
-            float * p = state + (size_t) (m * 16 + fr) * V + nt2 * 8 + fc;
-            *(float2 *) p = make_float2(st[i][0], st[i][1]);
-            *(float2 *) (p + (size_t) 8 * V) = make_float2(st[i][2], st[i][3]);
-        }
+        for (int i = 0; i < TPW; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+                if (sn0 + i < units) *(float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) = make_float2(st[i][2 * e], st[i][2 * e + 1]);
     }
 }
 
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
+// The passes are plain launches: as programmatic dependents their CTAs would settle wherever the last CTAs of prepare leave room,
+// several to an SM.
 template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t s) {
     const int nch = a.T / C + a.n_seqs;
     static std::atomic<unsigned char> done1[jib::MAX_DEVICES], done2[jib::MAX_DEVICES];
-    if (KIND == SSD) {
-        constexpr int smem = 2 * C * (K + 4) * 4;
-        if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done1)) return JIB_E_LAUNCH;
-        JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(nch, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
-    } else {
-        const int smem = prep_smem<K>(a.V);
-        if (!jib::ensure_dyn_smem(chunk_prepare_kernel<KIND == SSD ? LINEAR : KIND, K>, prep_smem<K>(256), done1)) return JIB_E_LAUNCH;
-        JIB_LAUNCH((chunk_prepare_kernel<KIND == SSD ? LINEAR : KIND, K>), dim3(nch, a.H), NT, smem, s, a);
-    }
+    if (!jib::ensure_dyn_smem(chunk_prepare_kernel<KIND, K>, prep_smem<K>(256), done1)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((chunk_prepare_kernel<KIND, K>), dim3(nch, a.H), NT, prep_smem<K>(a.V), s, a);
     const int rc = launched();
     if (rc) return rc;
     if (!jib::ensure_dyn_smem(chunk_pass_kernel<KIND, K>, Pass<KIND, K>::SMEM, done2)) return JIB_E_LAUNCH;
-    // a plain launch: as a programmatic dependent its CTAs would settle wherever the last CTAs of prepare leave room, several to an SM
     chunk_pass_kernel<KIND, K><<<dim3(a.H * (a.V / VB), a.n_seqs), NT, Pass<KIND, K>::SMEM, s>>>(a);
+    return launched();
+}
+template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
+    const int nch = a.T / C + a.n_seqs;
+    static std::atomic<unsigned char> done1[jib::MAX_DEVICES], done2[jib::MAX_DEVICES];
+    constexpr int smem = 2 * C * (K + 4) * 4;
+    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done1)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(nch, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
+    const int rc = launched();
+    if (rc) return rc;
+    if (!jib::ensure_dyn_smem(chunk_pass_ssd_kernel<K>, PassSsd<K>::SMEM, done2)) return JIB_E_LAUNCH;
+    chunk_pass_ssd_kernel<K><<<dim3(a.H * ((a.V + SV - 1) / SV), a.n_seqs), NT, PassSsd<K>::SMEM, s>>>(a);
     return launched();
 }
 
@@ -687,7 +854,7 @@ int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s) {
     switch (a.kind) {
         case DELTA: return a.K == 64 ? run_chunks<DELTA, 64>(a, s) : run_chunks<DELTA, 128>(a, s);
         case LINEAR: return a.K == 64 ? run_chunks<LINEAR, 64>(a, s) : run_chunks<LINEAR, 128>(a, s);
-        default: return a.K == 64 ? run_chunks<SSD, 64>(a, s) : run_chunks<SSD, 128>(a, s);
+        default: return a.K == 64 ? run_chunks_ssd<64>(a, s) : run_chunks_ssd<128>(a, s);
     }
 }
 
