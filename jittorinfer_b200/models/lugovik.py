@@ -213,9 +213,9 @@ def preset(name: str) -> LugovikHParams:
                             LinearPart(3, 24, 40, 12.0), 0.8, 1.1)
         return LugovikHParams(n_vocab=640, n_embd=160, eps=1e-5, embed_scale=4.0,
                               layers=stack(4, Mamba2Mixer(6, 24, 16, 2, 3, 4), DeltaMixer(4, 2, 24, 40, 4), par, 208), random_rank=12)
-    if name in ("lugovik-lite", "lugovik-v2"):
-        # the widths of the two DeepSeek-V2 models: 2048 with 16 attention heads, 5120 with 40; heads of 128
-        w, n, ff = (2048, 12, 5632) if name == "lugovik-lite" else (5120, 4, 12288)
+    if name in ("lugovik-lite", "lugovik-wide"):
+        # heads of 128: 16 of them at width 2048, 32 at width 4096
+        w, n, ff = (2048, 12, 5632) if name == "lugovik-lite" else (4096, 8, 11008)
         h = w // 128
         par = ParallelMixer(attention(h, h // 4, 128, 512, 500000.0), LinearPart(h, 128, 128, 16.0), 0.7, 0.7)
         return LugovikHParams(n_vocab=102400, n_embd=w, eps=1e-6, embed_scale=w ** 0.5,
