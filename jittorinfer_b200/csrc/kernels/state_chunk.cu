@@ -50,6 +50,32 @@ __device__ __forceinline__ void load4(const bf16 * p, float (&v)[4]) {
     const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &r.x), y = __bfloat1622float2(*(const __nv_bfloat162 *) &r.y);
     v[0] = x.x; v[1] = x.y; v[2] = y.x; v[3] = y.y;
 }
+// Two fp32 operations per instruction.
+struct F2 { unsigned long long v; };
+__device__ __forceinline__ F2 f2(float x, float y) {
+    F2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(x), "f"(y));
+    return r;
+}
+__device__ __forceinline__ float2 unpack(F2 a) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+    return r;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+    F2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+    return r;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+    F2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+    return r;
+}
+__device__ __forceinline__ float sum2(F2 a) {
+    const float2 x = unpack(a);
+    return x.x + x.y;
+}
 // 4 columns from column c on of tokens i0 .. i0 + 7 of a range (its first token: row q0, position p0; n tokens): convolved and silu'd.
 // Up to 4 taps; every row is loaded once, all loads in flight together.  Rows past the range are zero.
 __device__ __forceinline__ void conv_run(const jib_state_mix & a, int q0, int p0, int n, int i0, int c, int slot, float (&out)[8][4]) {
@@ -81,14 +107,14 @@ __device__ __forceinline__ void conv_run(const jib_state_mix & a, int q0, int p0
     if (a.conv_b != nullptr) b = *(const float4 *) (a.conv_b + c - a.conv0);
 #pragma unroll
     for (int r = 0; r < 8; ++r) {
-        float acc[4] = {b.x, b.y, b.z, b.w};
+        F2 s0 = f2(b.x, b.y), s1 = f2(b.z, b.w);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            acc[0] += w[j].x * v[r + j][0];
-            acc[1] += w[j].y * v[r + j][1];
-            acc[2] += w[j].z * v[r + j][2];
-            acc[3] += w[j].w * v[r + j][3];
+            s0 = fma2(f2(w[j].x, w[j].y), f2(v[r + j][0], v[r + j][1]), s0);
+            s1 = fma2(f2(w[j].z, w[j].w), f2(v[r + j][2], v[r + j][3]), s1);
         }
+        const float2 a0 = unpack(s0), a1 = unpack(s1);
+        const float acc[4] = {a0.x, a0.y, a1.x, a1.y};
 #pragma unroll
         for (int e = 0; e < 4; ++e) out[r][e] = i0 + r < n ? silu<bf16>(acc[e]) : 0.f;
     }
@@ -229,18 +255,26 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         const int i1 = i / (C - 1), j = i % (C - 1);
         const int t = j < i1 ? i1 : C - 1 - i1, s = j < i1 ? j : j - i1;
         const float * qt = q + t * KS, * kt = k + t * KS, * gt = G + t * KS, * ks = k + s * KS, * gs = G + s * KS;
-        float aq = 0.f, ak = 0.f;
+        F2 q0 = f2(0.f, 0.f), q1 = q0, k0 = q0, k1 = q0;
+        const F2 minus = f2(-1.f, -1.f);
 #pragma unroll 4
         for (int c = 0; c < K; c += 4) {
             const float4 x = *(const float4 *) (gt + c), y = *(const float4 *) (gs + c), z = *(const float4 *) (ks + c), u = *(const float4 *) (qt + c);
-            const float e0 = z.x * ex2(x.x - y.x), e1 = z.y * ex2(x.y - y.y), e2 = z.z * ex2(x.z - y.z), e3 = z.w * ex2(x.w - y.w);
-            aq += u.x * e0 + u.y * e1 + u.z * e2 + u.w * e3;
+            const float2 d0 = unpack(fma2(f2(y.x, y.y), minus, f2(x.x, x.y))), d1 = unpack(fma2(f2(y.z, y.w), minus, f2(x.z, x.w)));
+            const F2 e0 = mul2(f2(z.x, z.y), f2(ex2(d0.x), ex2(d0.y))), e1 = mul2(f2(z.z, z.w), f2(ex2(d1.x), ex2(d1.y)));
+            q0 = fma2(f2(u.x, u.y), e0, q0);
+            q1 = fma2(f2(u.z, u.w), e1, q1);
             if (KIND == DELTA) {
                 const float4 w = *(const float4 *) (kt + c);
-                ak += w.x * e0 + w.y * e1 + w.z * e2 + w.w * e3;
+                k0 = fma2(f2(w.x, w.y), e0, k0);
+                k1 = fma2(f2(w.z, w.w), e1, k1);
             }
         }
-        if (KIND == DELTA) B[t * 36 + s] = ak * beta[t];
+        const float aq = sum2(q0) + sum2(q1), ak = sum2(k0) + sum2(k1);
+        if (KIND == DELTA) {
+            B[t * 36 + s] = ak * beta[t];
+            B[s * 36 + t] = 0.f;
+        }
         const bf16 hi = __float2bfloat16(aq);
         *(bf16 *) (rec + R::A + a_off(t, s)) = hi;
         *(bf16 *) (rec + R::A + R::ATILE + a_off(t, s)) = __float2bfloat16(aq - to_f(hi));
@@ -255,6 +289,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
             const bf16 hi = __float2bfloat16(d);
             *(bf16 *) (rec + R::A + a_off(t, t)) = hi;
             *(bf16 *) (rec + R::A + R::ATILE + a_off(t, t)) = __float2bfloat16(d - to_f(hi));
+            if (KIND == DELTA) B[t * 36 + t] = 0.f;
         }
     }
     for (int i = tid; i < C * (K / 4); i += NT) {            // q e^G, k e^{G_C - G}
@@ -280,17 +315,15 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
 #pragma unroll
         for (int t = 0; t < C; ++t) x[t] = beta[t] * (c < K ? k[t * KS + c] * ex2(G[t * KS + c]) : v[t * VS + c - K]);
 #pragma unroll
-        for (int t = 1; t < C; ++t) {
-            float s0 = 0.f, s1 = 0.f;
+        for (int t = 1; t < C; ++t) {                        // B is 0 from its diagonal on: whole vectors of 4
+            F2 s0 = f2(0.f, 0.f), s1 = s0;
 #pragma unroll
             for (int s = 0; s < t; s += 4) {
                 const float4 w = *(const float4 *) (B + t * 36 + s);
-                s0 += w.x * x[s];
-                if (s + 1 < t) s1 += w.y * x[s + 1];
-                if (s + 2 < t) s0 += w.z * x[s + 2];
-                if (s + 3 < t) s1 += w.w * x[s + 3];
+                s0 = fma2(f2(w.x, w.y), f2(x[s], x[s + 1]), s0);
+                if (s + 2 < t) s1 = fma2(f2(w.z, w.w), f2(x[s + 2], x[s + 3]), s1);
             }
-            x[t] -= s0 + s1;
+            x[t] -= sum2(s0) + sum2(s1);
         }
         if (c < K) {
 #pragma unroll
@@ -310,7 +343,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
 // ---- prepare: SSD ------------------------------------------------------------------------------------------------------------------
 // blockIdx.y < groups: q and k tiles of a group and their products; then runs of 256 value columns (bf16 into a.v), then the factors.
 template <int K>
-__global__ void __launch_bounds__(NT) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
+__global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<SSD, K>;
     constexpr int KS = K + 4;
     extern __shared__ __align__(16) float sm[];
