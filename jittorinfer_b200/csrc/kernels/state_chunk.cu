@@ -10,7 +10,7 @@
 // Every exponent that occurs is a difference G_t - G_s with s <= t and so at most 0, however fast the decay: nothing overflows and no
 // quotient of vanishing products is formed.
 //   prepare (one CTA per chunk and head; SSD: per chunk and group): convolution, unit norm, decays, A, W, U0.  Independent of S.
-//   pass    (one CTA per head and 16 value columns, SSD 32): walks the chunks, S in registers, everything else a product of small matrices.
+//   pass    (K / 32 warps per head and 16 value columns): walks the chunks, S in registers, everything else a product of small matrices.
 // State, decays, A, W, U0 are fp32; the tensor cores see each as a sum of two bf16 numbers and the products hi * hi + hi * lo + lo * hi
 // (about 16 bits of mantissa); q and k of SSD are bf16 to begin with.  Accumulation is fp32.
 #include "pdl.cuh"
@@ -20,7 +20,7 @@ namespace {
 
 using namespace state_mix;
 
-constexpr int C = 32, VB = 16, NT = 256, STAGES = 3;
+constexpr int C = 32, NT = 256;                              // tokens of a chunk; threads of prepare
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int QK_LD = 32;                                    // row stride of SSD's q . k table (fp32)
 
@@ -187,6 +187,15 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
             ld = j < 2 * jk ? KS : VS;
             dst = j < jk ? q : j < 2 * jk ? k : v;
             conv_run(a, r0, p0, nr, t0 + run, (j < jk ? a.q_off + h / a.rep * K : j < 2 * jk ? a.k_off + h / a.rep * K : a.v_off + h * V) + col, slot, x);
+            if (KIND == LINEAR && j >= 2 * jk) {             // values as they are
+#pragma unroll
+                for (int r = 0; r < 8; ++r) {
+                    if (run + r >= n) break;
+                    __nv_bfloat162 y[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
+                    *(uint2 *) ((bf16 *) a.v + ((size_t) (r0 + t0 + run + r) * a.H + h) * V + col) = *(const uint2 *) y;
+                }
+                continue;
+            }
         } else {
             const int jj = j - 2 * jk - jv;
             col = jj % (K / 4) * 4;
@@ -249,7 +258,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         *x = y;
     }
     __syncthreads();
-    uint8_t * rec = (uint8_t *) a.chunk + ((size_t) ci * a.H + h) * (R::BYTES + C * 4 * V);
+    uint8_t * rec = (uint8_t *) a.chunk + ((size_t) ci * a.H + h) * (R::BYTES + (KIND == DELTA ? C * 4 * V : 0));
     // A and B: one thread per pair s < t (rows i and C - 1 - i together have C - 1 of them)
     for (int i = tid; i < C * (C - 1) / 2; i += NT) {
         const int i1 = i / (C - 1), j = i % (C - 1);
@@ -300,14 +309,8 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         put_tile4<K>(rec + R::D, t, c, make_float4(y.x * ex2(e.x - g.x), y.y * ex2(e.y - g.y), y.z * ex2(e.z - g.z), y.w * ex2(e.w - g.w)));
     }
     for (int c = tid; c < K; c += NT) ((float *) (rec + R::E))[c] = ex2(G[(C - 1) * KS + c]);
+    if (KIND == LINEAR) return;
     float * U = (float *) (rec + R::BYTES);
-    if (KIND == LINEAR) {
-        for (int i = tid; i < C * V; i += NT) {
-            const int t = i / V, c = i % V;
-            U[(c >> 4) * (C * VB) + t * VB + (c & 15)] = v[t * VS + c];
-        }
-        return;
-    }
     __syncthreads();
     // forward substitution, one right-hand side per thread: columns of k e^G, then of v
     for (int c = tid; c < K + V; c += NT) {
@@ -335,7 +338,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         } else {
             const int cc = c - K;
 #pragma unroll
-            for (int t = 0; t < C; ++t) U[(cc >> 4) * (C * VB) + t * VB + (cc & 15)] = x[t];
+            for (int t = 0; t < C; ++t) U[(cc >> 4) * (C * 16) + t * 16 + (cc & 15)] = x[t];
         }
     }
 }
@@ -421,456 +424,308 @@ __device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-constexpr int BS = VB + 8;                                   // row stride of the [.][VB] bf16 operands (48 bytes: rows hit different banks)
-
 template <int KIND, int K> struct Pass {
     using R = Rec<KIND, K>;
-    static constexpr int X = R::BYTES;                       // U0 fp32 [C][VB]
-    static constexpr int STAGE = X + C * VB * 4;
-    static constexpr int S = STAGES * STAGE;                 // S hi, lo [K][BS]
-    static constexpr int U = S + 2 * K * BS * 2;             // U hi, lo [C][BS]
-    static constexpr int SMEM = U + 2 * C * BS * 2;
+    static constexpr int KS = K / 32;                        // warps that share a head's 16 value columns, 32 key channels each
+    static constexpr int NG = (KIND == SSD ? 8 : 4) / KS;    // groups of 16 columns
+    static constexpr int WARPS = KS * NG, PT = WARPS * 32, PV = NG * 16;
+    static constexpr int STAGES = KIND == DELTA ? 3 : 4;
+    static constexpr int XS = PV * 2 + 16;                   // bytes of a row of v: rows hit different banks
+    static constexpr int X = R::BYTES;                       // v bf16 [C][PV] in rows of XS; DELTA: U0 fp32 [NG][C][16]
+    static constexpr int F = X + (KIND == DELTA ? NG * C * 16 * 4 : C * XS);              // SSD: factors fp32 [C]
+    static constexpr int STAGE = F + (KIND == SSD ? C * 4 : 0);
+    static constexpr int A = STAGES * STAGE;                 // SSD: A hi, lo, two buffers
+    static constexpr int O = A + (KIND == SSD ? 4 * R::ATILE : 0);       // partial o^T [WARPS][4][32] float4, then (DELTA) of W S
+    static constexpr int SMEM = O + WARPS * 2048 * (KIND == DELTA ? 2 : 1);
 };
 
-// DELTA, LINEAR.  Warps 0 - 3 own a 16 x 8 tile of o each, warps 4 - 7 one of u; all warps own tiles of S.  Two barriers per chunk: u is
-// there (and so is the next chunk's record), S is there.  Operands that depend on neither are in registers by then.
+// 16 value columns of a head belong to K / 32 warps; each keeps its channels of S^T (16 x 32) in registers as the accumulators of
+// S^T += u^T k.  In the products o^T = S^T q^T and S^T W^T those accumulators are the left operand as they stand (two m16n8 results are
+// an m16k16 operand), and u^T, the result of one product, is the left operand of the next two.  Only the partial sums over the channels
+// pass through shared memory.  Two barriers per chunk: the record is there; the partial sums are there.
 template <int KIND, int K>
-__global__ void __launch_bounds__(NT, 1) chunk_pass_kernel(const __grid_constant__ jib_state_mix a) {
+__global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<KIND, K>;
     using P = Pass<KIND, K>;
-    constexpr int TPW = K / 64;                              // 16 x 8 tiles of S per warp (K / 16 x 2 over 8 warps), side by side
+    constexpr int ST = P::STAGES, KS = P::KS, PT = P::PT, PV = P::PV;
     extern __shared__ __align__(16) uint8_t smem[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int splits = a.V / VB, h = blockIdx.x / splits, vs = blockIdx.x % splits, b = blockIdx.y, V = a.V, H = a.H;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, V = a.V, H = a.H, groups = H / a.rep;
+    const int splits = (V + PV - 1) / PV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * PV, b = blockIdx.y;
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
     if (n <= 0) return;
-    const int slot = checked_slot(a, b, 46);
-    const int chunks = (n + C - 1) / C;
-    const uint8_t * rec0 = (const uint8_t *) a.chunk + ((size_t) chunk_key(a.q_start, b) * H + h) * (R::BYTES + C * 4 * V);
-    const size_t rec_step = (size_t) H * (R::BYTES + C * 4 * V);
+    const int slot = checked_slot(a, b, 46), chunks = (n + C - 1) / C;
+    const int units = min(PV, V - v0) / 8;                   // 8-column units that exist
+    const int grp = warp / KS, ks = warp % KS;               // this warp's columns and channels
+    const bool active = grp * 2 < units;
+    const size_t rec_bytes = KIND == SSD ? R::BYTES : R::BYTES + (KIND == DELTA ? C * 4 * V : 0);
+    const size_t rec_step = rec_bytes * (KIND == SSD ? groups : H);
+    const uint8_t * rec0 = (const uint8_t *) a.chunk + chunk_key(a.q_start, b) * rec_step + (KIND == SSD ? h / a.rep : h) * rec_bytes;
     auto stage = [&](int i) {
         if (i < chunks) {
-            uint8_t * dst = smem + i % STAGES * P::STAGE;
+            uint8_t * dst = smem + i % ST * P::STAGE;
             const uint8_t * src = rec0 + i * rec_step;
-            for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
-            if (tid < C * VB / 4) cp16(dst + P::X + tid * 16, src + R::BYTES + vs * (C * VB * 4) + tid * 16);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    stage(0);
-    stage(1);
-    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
-
-    bf16 * Sh = (bf16 *) (smem + P::S), * Uh = (bf16 *) (smem + P::U);
-    const uint32_t S_addr = sm100::smem_u32(Sh), U_addr = sm100::smem_u32(Uh);
-    constexpr uint32_t S_LO = K * BS * 2, U_LO = C * BS * 2;
-    const int fr = lane >> 2, fc = (lane & 3) * 2;           // accumulator element: rows fr, fr + 8, columns fc, fc + 1
-    const int lr = lane & 15, lu = lane >> 4;                // ldmatrix lane addresses: operand rows (16 rows x 2 units) ...
-    const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;         // ... and k^T tiles (rows = tokens)
-    const int mt = (warp >> 1) & 1, nt = warp & 1;           // this warp's tile of o or u
-    const bool is_o = warp < 4;
-    const int sm_ = warp * TPW >> 1, sn0 = TPW == 2 ? 0 : warp & 1;               // tiles of S: rows 16 sm_, columns 8 (sn0 + i)
-    float st[TPW][4];
-    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + sm_ * 16 + fr) * V + vs * VB + fc;
-    const bool past = slot >= 0 && a.positions[r0] > 0;
-#pragma unroll
-    for (int i = 0; i < TPW; ++i)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const float2 x = past ? *(const float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) : make_float2(0.f, 0.f);
-            st[i][2 * e] = x.x;
-            st[i][2 * e + 1] = x.y;
-        }
-    auto publish_state = [&]() {
-#pragma unroll
-        for (int i = 0; i < TPW; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                uint32_t hi, lo;
-                split2(st[i][2 * e], st[i][2 * e + 1], hi, lo);
-                bf16 * p = Sh + (sm_ * 16 + fr + 8 * e) * BS + (sn0 + i) * 8 + fc;
-                *(uint32_t *) p = hi;
-                *(uint32_t *) (p + K * BS) = lo;
-            }
-    };
-    uint32_t xh[K / 16][4], xl[K / 16][4];                   // q e^G or W rows of this warp's tile
-    auto load_rows = [&](int ch) {
-        if (!is_o && KIND == LINEAR) return;
-        const int r = mt * 16 + lr;
-        const uint32_t base = sm100::smem_u32(smem + ch % STAGES * P::STAGE) + (is_o ? R::Q : R::W) + r * (K * 2);
-#pragma unroll
-        for (int kk = 0; kk < K / 16; ++kk) {
-            ldm4(xh[kk], base + (((kk * 2 + lu) ^ (r & 7)) << 4));
-            ldm4(xl[kk], base + R::TILE + (((kk * 2 + lu) ^ (r & 7)) << 4));
-        }
-    };
-    publish_state();
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    load_rows(0);
-    for (int ch = 0; ch < chunks; ++ch) {
-        stage(ch + 2);                                       // into the buffer of chunk ch - 1
-        const uint8_t * rec = smem + ch % STAGES * P::STAGE;
-        const uint32_t rec_addr = sm100::smem_u32(rec);
-        float o[4] = {0.f, 0.f, 0.f, 0.f};
-        if (is_o || KIND == DELTA) {
-            float acc[4][4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-#pragma unroll
-            for (int kk = 0; kk < K / 32; ++kk) {            // 32 channels at a time
-                uint32_t bh[4], bl[4];
-                const uint32_t off = ((kk * 32 + lane) * BS + nt * 8) * 2;
-                ldm4t(bh, S_addr + off);
-                ldm4t(bl, S_addr + S_LO + off);
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    mma(acc[e], xh[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
-                    mma(acc[2], xh[2 * kk + e], bl[2 * e], bl[2 * e + 1]);
-                    mma(acc[3], xl[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
+#pragma unroll 4
+            for (int o = tid * 16; o < R::BYTES; o += PT * 16) cp16(dst + o, src + o);
+            if (KIND == DELTA) {
+                for (int o = tid * 16; o < units / 2 * (C * 64); o += PT * 16) cp16(dst + P::X + o, src + R::BYTES + v0 / 16 * (C * 64) + o);
+            } else {
+                const int m = min(C, n - i * C);
+                for (int j = tid; j < C * (PV / 8); j += PT) {
+                    const int row = j / (PV / 8), u = j % (PV / 8);
+                    if (row >= m) *(uint4 *) (dst + P::X + row * P::XS + (u << 4)) = make_uint4(0, 0, 0, 0);
+                    else if (u < units)
+                        cp16(dst + P::X + row * P::XS + (u << 4), (const bf16 *) a.v + (size_t) (r0 + i * C + row) * H * V + h * V + v0 + u * 8);
                 }
+                if (KIND == SSD && tid < m) cp4(dst + P::F + tid * 4, a.s + (size_t) (r0 + i * C + tid) * H + h);
             }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) o[e] = (acc[0][e] + acc[1][e]) + (acc[2][e] + acc[3][e]);
-        }
-        if (!is_o) {                                         // u of this chunk as an operand
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int row = mt * 16 + fr + 8 * e, c = nt * 8 + fc;
-                const float2 x = *(const float2 *) (rec + P::X + (row * VB + c) * 4);
-                uint32_t hi, lo;
-                split2(x.x - o[2 * e], x.y - o[2 * e + 1], hi, lo);
-                bf16 * p = Uh + row * BS + c;
-                *(uint32_t *) p = hi;
-                *(uint32_t *) (p + C * BS) = lo;
-            }
-        }
-        // what the second half needs of the record
-        uint32_t dh[2][4], dl[2][4], ah[2][4], al[2][4];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int r = e * 16 + tr;
-            const uint32_t d = rec_addr + R::D + r * (K * 2) + (((sm_ * 2 + tu) ^ (r & 7)) << 4);
-            ldm4t(dh[e], d);
-            ldm4t(dl[e], d + R::TILE);
-            if (is_o) {
-                const int q = mt * 16 + lr;
-                const uint32_t p = rec_addr + R::A + q * 64 + (((e * 2 + lu) ^ ((q >> 1) & 3)) << 4);
-                ldm4(ah[e], p);
-                ldm4(al[e], p + R::ATILE);
-            }
-        }
-        const float * E = (const float *) (rec + R::E) + sm_ * 16 + fr;
-        const float e0 = E[0], e1 = E[8];
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();                                     // u, and the next chunk's record
-        uint32_t uh[2][4], ul[2][4];                         // both 8-column units of u
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            ldm4t(uh[i], U_addr + (lane * BS + i * 8) * 2);
-            ldm4t(ul[i], U_addr + U_LO + (lane * BS + i * 8) * 2);
-        }
-        // S' = e^{G_C} S + (k e^{G_C - G})^T u
-#pragma unroll
-        for (int i = 0; i < TPW; ++i) {
-            const int c = TPW == 2 ? i : sn0;
-            float p1[4] = {0.f, 0.f, 0.f, 0.f}, p2[4] = {0.f, 0.f, 0.f, 0.f};
-            st[i][0] *= e0; st[i][1] *= e0; st[i][2] *= e1; st[i][3] *= e1;
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const uint32_t h0 = c ? uh[1][2 * e] : uh[0][2 * e], h1 = c ? uh[1][2 * e + 1] : uh[0][2 * e + 1];
-                const uint32_t l0 = c ? ul[1][2 * e] : ul[0][2 * e], l1 = c ? ul[1][2 * e + 1] : ul[0][2 * e + 1];
-                mma(st[i], dh[e], h0, h1);
-                mma(p1, dh[e], l0, l1);
-                mma(p2, dl[e], h0, h1);
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) st[i][e] += p1[e] + p2[e];
-        }
-        publish_state();                                     // its readers of this chunk are behind the barrier above
-        if (is_o) {
-            float p[3][4];
-#pragma unroll
-            for (int i = 0; i < 3; ++i)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) p[i][e] = 0.f;
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const uint32_t h0 = nt ? uh[1][2 * e] : uh[0][2 * e], h1 = nt ? uh[1][2 * e + 1] : uh[0][2 * e + 1];
-                const uint32_t l0 = nt ? ul[1][2 * e] : ul[0][2 * e], l1 = nt ? ul[1][2 * e + 1] : ul[0][2 * e + 1];
-                mma(p[0], ah[e], h0, h1);
-                mma(p[1], ah[e], l0, l1);
-                mma(p[2], al[e], h0, h1);
-            }
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int t = ch * C + mt * 16 + fr + 8 * e;
-                if (t < n)
-                    *(float2 *) (a.o + ((size_t) (r0 + t) * H + h) * V + vs * VB + nt * 8 + fc) =
-                        make_float2(o[2 * e] + p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]), o[2 * e + 1] + p[0][2 * e + 1] + (p[1][2 * e + 1] + p[2][2 * e + 1]));
-            }
-        }
-        if (ch + 1 < chunks) load_rows(ch + 1);
-        __syncthreads();                                     // S; this chunk's record is free
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    if (slot >= 0) {
-#pragma unroll
-        for (int i = 0; i < TPW; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) *(float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) = make_float2(st[i][2 * e], st[i][2 * e + 1]);
-    }
-}
-
-// SSD: 32 value columns per CTA; every warp owns a 16 x 8 tile of o and K / 32 tiles of S.  q and k are bf16, so only A, u and S are split.
-constexpr int SV = 32, SB = SV + 8;                          // 80-byte rows hit different banks
-template <int K> struct PassSsd {
-    using R = Rec<SSD, K>;
-    static constexpr int X = R::BYTES;                       // x bf16 [C][SV], factors fp32 [C]
-    static constexpr int STAGE = X + C * SV * 2 + C * 4;
-    static constexpr int S = STAGES * STAGE;                 // S hi, lo [K][SB]
-    static constexpr int U = S + 2 * K * SB * 2;             // s x and its decayed form: hi, lo, hi, lo [C][SB]
-    static constexpr int A = U + 4 * C * SB * 2;             // A hi, lo
-    static constexpr int SMEM = A + 2 * R::ATILE;
-};
-
-template <int K>
-__global__ void __launch_bounds__(NT, 1) chunk_pass_ssd_kernel(const __grid_constant__ jib_state_mix a) {
-    using R = Rec<SSD, K>;
-    using P = PassSsd<K>;
-    constexpr int TPW = K / 32;
-    extern __shared__ __align__(16) uint8_t smem[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int V = a.V, H = a.H, splits = (V + SV - 1) / SV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * SV, b = blockIdx.y;
-    const int units = min(SV, V - v0) / 8;                   // 8-column units that exist
-    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
-    if (n <= 0) return;
-    const int slot = checked_slot(a, b, 46), groups = H / a.rep;
-    const int chunks = (n + C - 1) / C;
-    const uint8_t * rec0 = (const uint8_t *) a.chunk + ((size_t) chunk_key(a.q_start, b) * groups + h / a.rep) * R::BYTES;
-    auto stage = [&](int i) {
-        if (i < chunks) {
-            uint8_t * dst = smem + i % STAGES * P::STAGE;
-            const uint8_t * src = rec0 + (size_t) i * groups * R::BYTES;
-            for (int o = tid * 16; o < R::BYTES; o += NT * 16) cp16(dst + o, src + o);
-            const int m = min(C, n - i * C), row = tid >> 2, u = tid & 3;
-            if (row < m && u < units) cp16(dst + P::X + tid * 16, (const bf16 *) a.v + (size_t) (r0 + i * C + row) * H * V + h * V + v0 + u * 8);
-            if (tid < m) cp4(dst + P::X + C * SV * 2 + tid * 4, a.s + (size_t) (r0 + i * C + tid) * H + h);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    stage(0);
-    stage(1);
-    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * NT + tid, gridDim.x * NT);
+#pragma unroll
+    for (int i = 0; i < ST - 1; ++i) stage(i);
+    store_conv_tail<bf16>(a, slot, r0, n, blockIdx.x * PT + tid, gridDim.x * PT);
 
-    bf16 * Sh = (bf16 *) (smem + P::S), * Uh = (bf16 *) (smem + P::U);
-    const uint32_t S_addr = sm100::smem_u32(Sh), U_addr = sm100::smem_u32(Uh), A_addr = sm100::smem_u32(smem + P::A);
-    constexpr uint32_t S_LO = K * SB * 2, U_LO = C * SB * 2;
-    const int fr = lane >> 2, fc = (lane & 3) * 2, lr = lane & 15, lu = lane >> 4;
+    const int fr = lane >> 2, fc = (lane & 3) * 2;           // accumulator element: rows fr, fr + 8 (values), columns fc, fc + 1
     const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;
-    const int mt = warp >> 2, nt = warp & 3;
-    const int sm_ = warp * TPW >> 2, sn0 = TPW == 4 ? 0 : (warp & 1) * 2;
-    float st[TPW][4];
-    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + sm_ * 16 + fr) * V + v0 + fc;
-    const bool past = slot >= 0 && a.positions[r0] > 0;
+    float st[4][4];                                          // 4 tiles of 8 channels
+    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + ks * 32) * V + v0 + grp * 16 + fr;
+    const bool past = slot >= 0 && a.positions[r0] > 0 && active;
 #pragma unroll
-    for (int i = 0; i < TPW; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const float2 x = past && sn0 + i < units ? *(const float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) : make_float2(0.f, 0.f);
-            st[i][2 * e] = x.x;
-            st[i][2 * e + 1] = x.y;
-        }
-    auto publish_state = [&]() {
-#pragma unroll
-        for (int i = 0; i < TPW; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                uint32_t hi, lo;
-                split2(st[i][2 * e], st[i][2 * e + 1], hi, lo);
-                bf16 * p = Sh + (sm_ * 16 + fr + 8 * e) * SB + (sn0 + i) * 8 + fc;
-                *(uint32_t *) p = hi;
-                *(uint32_t *) (p + K * SB) = lo;
-            }
-    };
-    uint32_t xq[K / 16][4], xk[2][4];                        // rows of q of this warp's tile; k^T of its tiles of S
-    auto load_rows = [&](int ch) {
-        const uint32_t rec = sm100::smem_u32(smem + ch % STAGES * P::STAGE);
-        const int r = mt * 16 + lr;
-#pragma unroll
-        for (int kk = 0; kk < K / 16; ++kk) ldm4(xq[kk], rec + R::Q + r * (K * 2) + (((kk * 2 + lu) ^ (r & 7)) << 4));
-    };
-    const float na = a.neg_a[h] * LOG2E, skip = a.skip[h];
-    publish_state();
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    load_rows(0);
-    for (int ch = 0; ch < chunks; ++ch) {
-        stage(ch + 2);                                       // into the buffer of chunk ch - 1
-        const uint8_t * rec = smem + ch % STAGES * P::STAGE;
-        const uint32_t rec_addr = sm100::smem_u32(rec);
-        const int m = min(C, n - ch * C);
-        const float * factor = (const float *) (rec + P::X + C * SV * 2);
-        float acc[4][4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-#pragma unroll
-        for (int kk = 0; kk < K / 32; ++kk) {
-            uint32_t bh[4], bl[4];
-            const uint32_t off = ((kk * 32 + lane) * SB + nt * 8) * 2;
-            ldm4t(bh, S_addr + off);
-            ldm4t(bl, S_addr + S_LO + off);
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                mma(acc[e], xq[2 * kk + e], bh[2 * e], bh[2 * e + 1]);
-                mma(acc[2 + e], xq[2 * kk + e], bl[2 * e], bl[2 * e + 1]);
-            }
-        }
-        // lane t: G_t
-        float g = lane < m ? na * factor[lane] : 0.f;
+        for (int e = 0; e < 4; ++e) st[i][e] = past ? state[(size_t) (i * 8 + fc + (e & 1)) * V + 8 * (e >> 1)] : 0.f;
+    const float na = KIND == SSD ? a.neg_a[h] * LOG2E : 0.f, skip = KIND == SSD ? a.skip[h] : 0.f;
+    float g = 0.f, f = 0.f;                                  // SSD: lane t holds G_t and the factor of the chunk at hand
+    // SSD: the chunk's G and factors, and its A (C / WARPS rows by this warp): q . k, the decay between the two tokens, the
+    // factor of the earlier one, and D on the diagonal
+    auto decays = [&](int ch) {
+        const uint8_t * rec = smem + ch % ST * P::STAGE;
+        f = lane < n - ch * C ? ((const float *) (rec + P::F))[lane] : 0.f;
+        g = na * f;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float x = __shfl_up_sync(0xffffffffu, g, o);
             if (lane >= o) g += x;
         }
-        const float gC = __shfl_sync(0xffffffffu, g, 31);
-        {   // s x and s x e^{G_C - G}: 4 columns of a row per thread
-            const int row = tid >> 3, c = (tid & 7) * 4;
-            const float f = row < m ? factor[row] : 0.f, w = f * ex2(gC - __shfl_sync(0xffffffffu, g, row));
-            float x[4] = {0.f, 0.f, 0.f, 0.f};
-            if (row < m) load4((const bf16 *) (rec + P::X) + row * SV + c, x);
-            uint2 hi, lo;
-            bf16 * p = Uh + row * SB + c;
-            split2(x[0] * f, x[1] * f, hi.x, lo.x);
-            split2(x[2] * f, x[3] * f, hi.y, lo.y);
-            *(uint2 *) p = hi;
-            *(uint2 *) (p + C * SB) = lo;
-            split2(x[0] * w, x[1] * w, hi.x, lo.x);
-            split2(x[2] * w, x[3] * w, hi.y, lo.y);
-            *(uint2 *) (p + 2 * C * SB) = hi;
-            *(uint2 *) (p + 3 * C * SB) = lo;
-        }
+        uint8_t * A = smem + P::A + (ch & 1) * 2 * R::ATILE;
 #pragma unroll
-        for (int k = 0; k < C / 8; ++k) {                    // A = q . k times the decay between the two tokens: 4 rows per warp
-            const int t = warp * (C / 8) + k;
-            const float gt = __shfl_sync(0xffffffffu, g, t);                         // by all lanes, outside the condition
-            const float x = lane <= t ? ((const float *) (rec + R::A))[t * QK_LD + lane] * ex2(gt - g) : 0.f;
+        for (int i = 0; i < C / P::WARPS; ++i) {
+            const int t = warp * (C / P::WARPS) + i;
+            const float gt = __shfl_sync(0xffffffffu, g, t);
+            float x = lane <= t ? ((const float *) (rec + R::A))[t * QK_LD + lane] * (ex2(gt - g) * f) : 0.f;
+            if (lane == t) x += skip;
             const bf16 hi = __float2bfloat16(x);
-            *(bf16 *) (smem + P::A + a_off(t, lane)) = hi;
-            *(bf16 *) (smem + P::A + R::ATILE + a_off(t, lane)) = __float2bfloat16(x - to_f(hi));
+            *(bf16 *) (A + a_off(t, lane)) = hi;
+            *(bf16 *) (A + R::ATILE + a_off(t, lane)) = __float2bfloat16(x - to_f(hi));
         }
+    };
+    if (KIND == SSD) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+        __syncthreads();
+        decays(0);
+    }
+    for (int ch = 0; ch < chunks; ++ch) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(KIND == SSD ? ST - 3 : ST - 2) : "memory");
+        __syncthreads();                                     // this chunk's record (SSD: the next one's and this chunk's A); the oldest is free
+        stage(ch + ST - 1);
+        const uint8_t * rec = smem + ch % ST * P::STAGE;
+        const uint32_t rec_addr = sm100::smem_u32(rec);
+        const uint32_t A_addr = KIND == SSD ? sm100::smem_u32(smem + P::A + (ch & 1) * 2 * R::ATILE) : rec_addr + R::A;
+        float4 * part = (float4 *) (smem + P::O) + warp * 128 + lane;          // this warp's partial sums: [4 token tiles][32 lanes]
+        uint32_t xh[2][4], xl[2][4], yh[2][4], yl[2][4];     // u^T, hi and lo, 16 tokens at a time (x: of the read-out, y: of the update)
+        const float gC = KIND == SSD ? __shfl_sync(0xffffffffu, g, 31) : 0.f, dC = KIND == SSD ? ex2(gC) : 0.f;
+        if (active) {
+            float o[4][4], w[4][4];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int r = e * 16 + tr;
-            ldm4t(xk[e], rec_addr + R::D + r * (K * 2) + (((sm_ * 2 + tu) ^ (r & 7)) << 4));
-        }
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();                                     // u, A, and the next chunk's record
-        const float decay = ex2(gC);
+            for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int i = 0; i < TPW; ++i) {
-            uint32_t bh[4], bl[4];
-            const uint32_t off = (lane * SB + (sn0 + i) * 8) * 2;
-            ldm4t(bh, U_addr + 2 * U_LO + off);
-            ldm4t(bl, U_addr + 3 * U_LO + off);
-            float p1[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int e = 0; e < 4; ++e) o[i][e] = w[i][e] = 0.f;
+            uint32_t sh[2][4], sl[2][4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) st[i][e] *= decay;
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                mma(st[i], xk[e], bh[2 * e], bh[2 * e + 1]);
-                mma(p1, xk[e], bl[2 * e], bl[2 * e + 1]);
+                for (int i = 0; i < 4; ++i) split2(st[2 * j + (i >> 1)][2 * (i & 1)], st[2 * j + (i >> 1)][2 * (i & 1) + 1], sh[j][i], sl[j][i]);
+            uint32_t y[4][4], z[4][4];
+            auto rows = [&](uint32_t (&t)[4][4], uint32_t tile) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int r = i * 8 + (lane & 7);
+                    ldm4(t[i], rec_addr + tile + r * (K * 2) + (((ks * 4 + (lane >> 3)) ^ (r & 7)) << 4));
+                }
+            };
+            if (KIND == DELTA) rows(z, R::W);
+            rows(y, R::Q);
+            // in an order that keeps four (DELTA: eight) accumulators in flight
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (KIND == DELTA) mma(w[i], sh[j], z[i][2 * j], z[i][2 * j + 1]);
+                    mma(o[i], sh[j], y[i][2 * j], y[i][2 * j + 1]);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (KIND == DELTA) mma(w[i], sl[j], z[i][2 * j], z[i][2 * j + 1]);
+                    mma(o[i], sl[j], y[i][2 * j], y[i][2 * j + 1]);
+                }
+            }
+            if (KIND != SSD) {
+                if (KIND == DELTA) rows(z, R::W + R::TILE);
+                rows(y, R::Q + R::TILE);
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        if (KIND == DELTA) mma(w[i], sh[j], z[i][2 * j], z[i][2 * j + 1]);
+                        mma(o[i], sh[j], y[i][2 * j], y[i][2 * j + 1]);
+                    }
             }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) st[i][e] += p1[e];
+            for (int i = 0; i < 4; ++i) {
+                part[i * 32] = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+                if (KIND == DELTA) part[P::WARPS * 128 + i * 32] = make_float4(w[i][0], w[i][1], w[i][2], w[i][3]);
+            }
         }
-        publish_state();                                     // its readers of this chunk are behind the barrier above
-        {
-            float p[3][4];
+        if (KIND == DELTA) __syncthreads();
+        if (active) {
+            if (KIND == DELTA) {                             // u^T = U0^T - S^T W^T
+                const float4 * all = (const float4 *) (smem + P::O) + (P::WARPS + grp * KS) * 128 + lane;
+                const float * u0 = (const float *) (rec + P::X) + grp * (C * 16) + fr;
+                float u[4][4];
 #pragma unroll
-            for (int i = 0; i < 3; ++i)
+                for (int i = 0; i < 4; ++i) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) p[i][e] = 0.f;
-            uint32_t bh[4], bl[4], xh[4], xl[4];
-            const float w0 = ex2(__shfl_sync(0xffffffffu, g, mt * 16 + fr)), w1 = ex2(__shfl_sync(0xffffffffu, g, mt * 16 + fr + 8));
-            const uint32_t off = (lane * SB + nt * 8) * 2;
-            ldm4t(bh, U_addr + off);
-            ldm4t(bl, U_addr + U_LO + off);
+                    for (int e = 0; e < 4; ++e) u[i][e] = u0[(i * 8 + fc + (e & 1)) * 16 + 8 * (e >> 1)];
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = mt * 16 + lr;
-                const uint32_t q = A_addr + r * 64 + (((e * 2 + lu) ^ ((r >> 1) & 3)) << 4);
-                ldm4(xh, q);
-                ldm4(xl, q + R::ATILE);
-                mma(p[0], xh, bh[2 * e], bh[2 * e + 1]);
-                mma(p[1], xh, bl[2 * e], bl[2 * e + 1]);
-                mma(p[2], xl, bh[2 * e], bh[2 * e + 1]);
+                    for (int k = 0; k < KS; ++k) {
+                        const float4 p = all[k * 128 + i * 32];
+                        u[i][0] -= p.x; u[i][1] -= p.y; u[i][2] -= p.z; u[i][3] -= p.w;
+                    }
+                }
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) split2(u[2 * e + (i >> 1)][2 * (i & 1)], u[2 * e + (i >> 1)][2 * (i & 1) + 1], xh[e][i], xl[e][i]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) ldm4t(xh[e], rec_addr + P::X + (e * 16 + tr) * P::XS + ((grp * 2 + tu) << 4));
+            }
+            if (KIND == SSD) {
+                const float wt = f * ex2(gC - g);
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {            // tokens 16 e + 8 j + fc, + 1
+                        const float w0 = __shfl_sync(0xffffffffu, wt, e * 16 + j * 8 + fc), w1 = __shfl_sync(0xffffffffu, wt, e * 16 + j * 8 + fc + 1);
+#pragma unroll
+                        for (int i = 2 * j; i < 2 * j + 2; ++i) {
+                            const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &xh[e][i]);
+                            split2(x.x * w0, x.y * w1, yh[e][i], yl[e][i]);
+                        }
+                    }
+            }
+            // S^T <- decay S^T + u^T k
+            uint32_t y[4][4], z[4][4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const uint32_t off = lane * (K * 2) + (((ks * 4 + i) ^ (lane & 7)) << 4);
+                ldm4t(y[i], rec_addr + R::D + off);
+                if (KIND != SSD) ldm4t(z[i], rec_addr + R::D + R::TILE + off);
+                float2 d = make_float2(dC, dC);
+                if (KIND != SSD) d = *(const float2 *) (rec + R::E + (ks * 32 + i * 8 + fc) * 4);
+                st[i][0] *= d.x; st[i][1] *= d.y; st[i][2] *= d.x; st[i][3] *= d.y;
             }
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const int t = mt * 16 + fr + 8 * e, c = nt * 8 + fc;
-                const float w = e ? w1 : w0;
-                if (t >= m || nt >= units) continue;
-                const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) (rec + P::X + (t * SV + c) * 2));
-                float2 y;
-                y.x = w * ((acc[0][2 * e] + acc[1][2 * e]) + (acc[2][2 * e] + acc[3][2 * e])) + p[0][2 * e] + (p[1][2 * e] + p[2][2 * e]) + skip * x.x;
-                y.y = w * ((acc[0][2 * e + 1] + acc[1][2 * e + 1]) + (acc[2][2 * e + 1] + acc[3][2 * e + 1])) + p[0][2 * e + 1] +
-                      (p[1][2 * e + 1] + p[2][2 * e + 1]) + skip * x.y;
-                *(float2 *) (a.o + ((size_t) (r0 + ch * C + t) * H + h) * V + v0 + c) = y;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) mma(st[i], KIND == SSD ? yh[e] : xh[e], y[i][2 * e], y[i][2 * e + 1]);
+                if (KIND != LINEAR) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) mma(st[i], KIND == SSD ? yl[e] : xl[e], y[i][2 * e], y[i][2 * e + 1]);
+                }
+                if (KIND != SSD) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) mma(st[i], xh[e], z[i][2 * e], z[i][2 * e + 1]);
+                }
             }
         }
-        if (ch + 1 < chunks) load_rows(ch + 1);
-        __syncthreads();                                     // S; this chunk's record is free
+        if (KIND != DELTA) __syncthreads();
+        const float eg = KIND == SSD ? ex2(g) : 0.f;
+        if (active) {                                        // o^T of 4 / KS token tiles: the partial sums, then += u^T A^T
+#pragma unroll
+            for (int k = 0; k < 4 / KS; ++k) {
+                const int i = ks * (4 / KS) + k, r = i * 8 + (lane & 7);
+                const float4 * all = (const float4 *) (smem + P::O) + grp * KS * 128 + i * 32 + lane;
+                float o[4] = {0.f, 0.f, 0.f, 0.f}, q[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int p = 0; p < KS; ++p) {
+                    const float4 x = all[p * 128];
+                    o[0] += x.x; o[1] += x.y; o[2] += x.z; o[3] += x.w;
+                }
+                if (KIND == SSD) {
+                    const float e0 = __shfl_sync(0xffffffffu, eg, i * 8 + fc), e1 = __shfl_sync(0xffffffffu, eg, i * 8 + fc + 1);
+                    o[0] *= e0; o[1] *= e1; o[2] *= e0; o[3] *= e1;
+                }
+                const uint32_t off = r * 64 + (((lane >> 3) ^ ((r >> 1) & 3)) << 4);
+                uint32_t y[4], z[4];
+                ldm4(y, A_addr + off);
+                ldm4(z, A_addr + R::ATILE + off);
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    mma(o, xh[e], y[2 * e], y[2 * e + 1]);
+                    mma(q, xh[e], z[2 * e], z[2 * e + 1]);
+                    if (KIND == DELTA) mma(q, xl[e], y[2 * e], y[2 * e + 1]);
+                }
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = ch * C + i * 8 + fc + (e & 1);
+                    if (t < n) a.o[((size_t) (r0 + t) * H + h) * V + v0 + grp * 16 + fr + 8 * (e >> 1)] = o[e] + q[e];
+                }
+            }
+        }
+        if (KIND == SSD && ch + 1 < chunks) decays(ch + 1);
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    if (slot >= 0) {
+    if (slot >= 0 && active) {
 #pragma unroll
-        for (int i = 0; i < TPW; ++i)
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int e = 0; e < 2; ++e)
-                if (sn0 + i < units) *(float2 *) (state + (size_t) (8 * e) * V + (sn0 + i) * 8) = make_float2(st[i][2 * e], st[i][2 * e + 1]);
+            for (int e = 0; e < 4; ++e) state[(size_t) (i * 8 + fc + (e & 1)) * V + 8 * (e >> 1)] = st[i][e];
     }
 }
 
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
-// The passes are plain launches: as programmatic dependents their CTAs would settle wherever the last CTAs of prepare leave room,
-// several to an SM.
-template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t s) {
-    const int nch = a.T / C + a.n_seqs;
-    static std::atomic<unsigned char> done1[jib::MAX_DEVICES], done2[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(chunk_prepare_kernel<KIND, K>, prep_smem<K>(256), done1)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((chunk_prepare_kernel<KIND, K>), dim3(nch, a.H), NT, prep_smem<K>(a.V), s, a);
-    const int rc = launched();
-    if (rc) return rc;
-    if (!jib::ensure_dyn_smem(chunk_pass_kernel<KIND, K>, Pass<KIND, K>::SMEM, done2)) return JIB_E_LAUNCH;
-    chunk_pass_kernel<KIND, K><<<dim3(a.H * (a.V / VB), a.n_seqs), NT, Pass<KIND, K>::SMEM, s>>>(a);
+// The pass is a plain launch: as a programmatic dependent its CTAs would settle wherever the last CTAs of prepare leave room, several
+// to an SM.
+template <int KIND, int K> int launch_pass(const jib_state_mix & a, cudaStream_t s) {
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (!jib::ensure_dyn_smem(chunk_pass_kernel<KIND, K>, Pass<KIND, K>::SMEM, done)) return JIB_E_LAUNCH;
+    chunk_pass_kernel<KIND, K><<<dim3(a.H * ((a.V + Pass<KIND, K>::PV - 1) / Pass<KIND, K>::PV), a.n_seqs), Pass<KIND, K>::PT, Pass<KIND, K>::SMEM, s>>>(a);
     return launched();
 }
-template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
-    const int nch = a.T / C + a.n_seqs;
-    static std::atomic<unsigned char> done1[jib::MAX_DEVICES], done2[jib::MAX_DEVICES];
-    constexpr int smem = 2 * C * (K + 4) * 4;
-    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done1)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(nch, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
+template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t s) {
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (!jib::ensure_dyn_smem(chunk_prepare_kernel<KIND, K>, prep_smem<K>(256), done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((chunk_prepare_kernel<KIND, K>), dim3(a.T / C + a.n_seqs, a.H), NT, prep_smem<K>(a.V), s, a);
     const int rc = launched();
-    if (rc) return rc;
-    if (!jib::ensure_dyn_smem(chunk_pass_ssd_kernel<K>, PassSsd<K>::SMEM, done2)) return JIB_E_LAUNCH;
-    chunk_pass_ssd_kernel<K><<<dim3(a.H * ((a.V + SV - 1) / SV), a.n_seqs), NT, PassSsd<K>::SMEM, s>>>(a);
-    return launched();
+    return rc ? rc : launch_pass<KIND, K>(a, s);
+}
+template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    constexpr int smem = 2 * C * (K + 4) * 4;
+    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(a.T / C + a.n_seqs, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
+    const int rc = launched();
+    return rc ? rc : launch_pass<SSD, K>(a, s);
 }
 
 long long rec_bytes(const jib_state_mix & a) {
 #define REC(KIND) (a.K == 64 ? Rec<KIND, 64>::BYTES : Rec<KIND, 128>::BYTES)
     const long long nch = a.T / C + a.n_seqs;
     if (a.kind == SSD) return nch * (a.H / a.rep) * REC(SSD);
-    return nch * a.H * ((a.kind == DELTA ? REC(DELTA) : REC(LINEAR)) + C * 4 * a.V);
+    return nch * a.H * (a.kind == DELTA ? REC(DELTA) + C * 4 * a.V : REC(LINEAR));
 #undef REC
 }
 
@@ -878,7 +733,7 @@ long long rec_bytes(const jib_state_mix & a) {
 
 bool jib_state_chunk_ok(const jib_state_mix & a) {
     const long long cols = a.ld | a.q_off | a.k_off | a.v_off | a.conv0 | a.n_conv | (a.kind == SSD ? 0 : a.ld_dec);
-    return (a.K == 64 || a.K == 128) && a.V % VB == 0 && a.V <= 256 && a.taps <= 4 && cols % 4 == 0 && ((uintptr_t) a.proj & 7) == 0 &&
+    return (a.K == 64 || a.K == 128) && a.V % 16 == 0 && a.V <= 256 && a.taps <= 4 && cols % 4 == 0 && ((uintptr_t) a.proj & 7) == 0 &&
            (a.kind == SSD || ((uintptr_t) a.dec_in & 7) == 0) && a.H % a.rep == 0;
 }
 

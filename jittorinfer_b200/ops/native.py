@@ -777,7 +777,7 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     if n > 0:                         # portions through the tensor cores
         scratch = [torch.empty(n, dtype=torch.uint8, device=proj.device)]
         sd.chunk, sd.chunk_bytes = scratch[0].data_ptr(), n
-        if m.kind == "ssd":
+        if m.kind != "delta":
             scratch += [torch.empty(T, H * V, dtype=proj.dtype, device=proj.device), f32(T, H)]
             sd.v, sd.s = scratch[1].data_ptr(), scratch[2].data_ptr()
     elif not single:
