@@ -22,17 +22,24 @@ using namespace state_mix;
 
 constexpr int C = 32, NT = 256;                              // tokens of a chunk; threads of prepare
 constexpr float LOG2E = 1.4426950408889634f;
-constexpr int QK_LD = 32;                                    // row stride of SSD's q . k table (fp32)
 
 // A chunk's record: bf16 tiles of 32 rows x K columns in 16-byte units u of row r stored at u ^ (r & 7); A: 32 x 32, unit u ^ (r / 2 & 3).
 template <int KIND, int K> struct Rec {
     static constexpr int TILE = C * K * 2, ATILE = C * C * 2;
     static constexpr int Q = 0, D = KIND == SSD ? TILE : 2 * TILE;                        // q e^G, k e^{G_C - G} (SSD: q, k)
-    static constexpr int A = KIND == SSD ? 2 * TILE : 4 * TILE;                           // hi, lo (SSD: q . k fp32)
+    static constexpr int A = KIND == SSD ? 2 * TILE : 4 * TILE;                           // hi, lo
     static constexpr int W = A + 2 * ATILE;                                               // DELTA
-    static constexpr int E = W + (KIND == DELTA ? 2 * TILE : 0);                          // e^{G_C}
-    static constexpr int BYTES = KIND == SSD ? A + C * QK_LD * 4 : E + K * 4;
+    static constexpr int E = W + (KIND == DELTA ? 2 * TILE : 0);                          // e^{G_C}; SSD: e^{G_t}, then s_t e^{G_C - G_t}
+    static constexpr int BYTES = E + (KIND == SSD ? 2 * C : K) * 4;
 };
+// SSD: q and k (the first A bytes) are shared by a group; the rest is per head and lies behind all groups' parts.
+template <int K> __device__ __forceinline__ uint8_t * ssd_group_part(const jib_state_mix & a, int ci, int group) {
+    return (uint8_t *) a.chunk + ((size_t) ci * (a.H / a.rep) + group) * Rec<SSD, K>::A;
+}
+template <int K> __device__ __forceinline__ uint8_t * ssd_head_part(const jib_state_mix & a, int ci, int h) {
+    using R = Rec<SSD, K>;
+    return (uint8_t *) a.chunk + (size_t) (a.T / C + a.n_seqs) * (a.H / a.rep) * R::A + ((size_t) ci * a.H + h) * (R::BYTES - R::A);
+}
 
 // run index: sequence b's chunks start at q_start[b] / C + b; indices in the gaps have no tokens
 __device__ __forceinline__ int chunk_key(const int * q_start, int b) { return q_start[b] / C + b; }
@@ -344,7 +351,10 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
 }
 
 // ---- prepare: SSD ------------------------------------------------------------------------------------------------------------------
-// blockIdx.y < groups: q and k tiles of a group and their products; then runs of 256 value columns (bf16 into a.v), then the factors.
+// blockIdx.y < groups * blocks of 16 heads: q and k tiles of a group and their products, then A and the decays of 16 heads of the group
+// (A_ts also holds the factor s_s of the earlier token, and D on the diagonal).  Then runs of 256 value columns (bf16 into a.v).
+constexpr int HB = 16;
+
 template <int K>
 __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<SSD, K>;
@@ -358,10 +368,13 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
     if (t0 < 0 || t0 >= nr) return;
     const int p0 = a.positions[r0], n = min(C, nr - t0);
     const int slot = a.taps > 0 ? checked_slot(a, b, 45) : -1;
+    const int blocks = (a.rep + HB - 1) / HB;
     int y = blockIdx.y;
-    if (y < groups) {
-        float * q = sm, * k = sm + C * KS;
-        uint8_t * rec = (uint8_t *) a.chunk + ((size_t) ci * groups + y) * R::BYTES;
+    if (y < groups * blocks) {
+        float * q = sm, * k = sm + C * KS, * qk = k + C * KS;             // qk [C][C + 1]
+        const int block = y % blocks;
+        y /= blocks;
+        uint8_t * rec = ssd_group_part<K>(a, ci, y);
         const int jk = K / 4 * (C / 8);
         for (int j = tid; j < 2 * jk; j += NT) {
             float x[8][4];
@@ -370,7 +383,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
 #pragma unroll
             for (int r = 0; r < 8; ++r) {
                 __nv_bfloat162 v[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
-                *(uint2 *) (rec + (j < jk ? R::Q : R::D) + tile_off<K>(run + r, col)) = *(const uint2 *) v;
+                if (block == 0) *(uint2 *) (rec + (j < jk ? R::Q : R::D) + tile_off<K>(run + r, col)) = *(const uint2 *) v;
                 const float2 f0 = __bfloat1622float2(v[0]), f1 = __bfloat1622float2(v[1]);
                 *(float4 *) ((j < jk ? q : k) + (run + r) * KS + col) = make_float4(f0.x, f0.y, f1.x, f1.y);
             }
@@ -385,29 +398,46 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
                 const float4 x = *(const float4 *) (q + t * KS + c), z = *(const float4 *) (k + s * KS + c);
                 d += x.x * z.x + x.y * z.y + x.z * z.z + x.w * z.w;
             }
-            ((float *) (rec + R::A))[t * QK_LD + s] = d;
+            qk[t * (C + 1) + s] = d;
         }
-        return;
-    }
-    y -= groups;
-    const int vblocks = (inner + 255) / 256;
-    if (y < vblocks) {
-        const int col = y * 256 + (tid & 63) * 4, run = (tid >> 6) * 8;
-        if (col >= inner) return;
-        float x[8][4];
-        conv_run(a, r0, p0, nr, t0 + run, a.v_off + col, slot, x);
+        __syncthreads();
+        const int lane = tid & 31;
+        for (int i = tid >> 5; i < HB && block * HB + i < a.rep; i += NT / 32) {
+            const int h = y * a.rep + block * HB + i;
+            uint8_t * hr = ssd_head_part<K>(a, ci, h);
+            const float f = lane < n ? softplus_series(to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + lane) * a.ld + a.s_off + h]) + a.bias[h]) : 0.f;
+            float g = a.neg_a[h] * LOG2E * f;                // lane t: G_t
 #pragma unroll
-        for (int r = 0; r < 8; ++r) {
-            if (run + r >= n) break;
-            __nv_bfloat162 v[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
-            *(uint2 *) ((bf16 *) a.v + (size_t) (r0 + t0 + run + r) * inner + col) = *(const uint2 *) v;
+            for (int o = 1; o < 32; o <<= 1) {
+                const float x = __shfl_up_sync(0xffffffffu, g, o);
+                if (lane >= o) g += x;
+            }
+            const float gC = __shfl_sync(0xffffffffu, g, 31), skip = a.skip[h];
+            float * e = (float *) (hr + R::E - R::A);
+            e[lane] = ex2(g);
+            e[C + lane] = f * ex2(gC - g);
+#pragma unroll 4
+            for (int t = 0; t < C; ++t) {
+                const float gt = __shfl_sync(0xffffffffu, g, t);
+                float x = lane <= t ? qk[t * (C + 1) + lane] * (ex2(gt - g) * f) : 0.f;
+                if (lane == t) x += skip;
+                const bf16 hi = __float2bfloat16(x);
+                *(bf16 *) (hr + a_off(t, lane)) = hi;
+                *(bf16 *) (hr + R::ATILE + a_off(t, lane)) = __float2bfloat16(x - to_f(hi));
+            }
         }
         return;
     }
-    for (int i = tid; i < n * a.H; i += NT) {
-        const size_t row = r0 + t0 + i / a.H;
-        const int h = i % a.H;
-        a.s[row * a.H + h] = head_factor<SSD>(a, to_f(((const bf16 *) a.proj)[row * a.ld + a.s_off + h]), h);
+    y -= groups * blocks;
+    const int col = y * 256 + (tid & 63) * 4, run = (tid >> 6) * 8;
+    if (col >= inner) return;
+    float x[8][4];
+    conv_run(a, r0, p0, nr, t0 + run, a.v_off + col, slot, x);
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+        if (run + r >= n) break;
+        __nv_bfloat162 v[2] = {__floats2bfloat162_rn(x[r][0], x[r][1]), __floats2bfloat162_rn(x[r][2], x[r][3])};
+        *(uint2 *) ((bf16 *) a.v + (size_t) (r0 + t0 + run + r) * inner + col) = *(const uint2 *) v;
     }
 }
 
@@ -432,10 +462,8 @@ template <int KIND, int K> struct Pass {
     static constexpr int STAGES = KIND == DELTA ? 3 : 4;
     static constexpr int XS = PV * 2 + 16;                   // bytes of a row of v: rows hit different banks
     static constexpr int X = R::BYTES;                       // v bf16 [C][PV] in rows of XS; DELTA: U0 fp32 [NG][C][16]
-    static constexpr int F = X + (KIND == DELTA ? NG * C * 16 * 4 : C * XS);              // SSD: factors fp32 [C]
-    static constexpr int STAGE = F + (KIND == SSD ? C * 4 : 0);
-    static constexpr int A = STAGES * STAGE;                 // SSD: A hi, lo, two buffers
-    static constexpr int O = A + (KIND == SSD ? 4 * R::ATILE : 0);       // partial o^T [WARPS][4][32] float4, then (DELTA) of W S
+    static constexpr int STAGE = X + (KIND == DELTA ? NG * C * 16 * 4 : C * XS);
+    static constexpr int O = STAGES * STAGE;                 // partial o^T [WARPS][4][32] float4, then (DELTA) of W S
     static constexpr int SMEM = O + WARPS * 2048 * (KIND == DELTA ? 2 : 1);
 };
 
@@ -449,7 +477,7 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     using P = Pass<KIND, K>;
     constexpr int ST = P::STAGES, KS = P::KS, PT = P::PT, PV = P::PV;
     extern __shared__ __align__(16) uint8_t smem[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, V = a.V, H = a.H, groups = H / a.rep;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, V = a.V, H = a.H;
     const int splits = (V + PV - 1) / PV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * PV, b = blockIdx.y;
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
@@ -458,15 +486,18 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     const int units = min(PV, V - v0) / 8;                   // 8-column units that exist
     const int grp = warp / KS, ks = warp % KS;               // this warp's columns and channels
     const bool active = grp * 2 < units;
-    const size_t rec_bytes = KIND == SSD ? R::BYTES : R::BYTES + (KIND == DELTA ? C * 4 * V : 0);
-    const size_t rec_step = rec_bytes * (KIND == SSD ? groups : H);
-    const uint8_t * rec0 = (const uint8_t *) a.chunk + chunk_key(a.q_start, b) * rec_step + (KIND == SSD ? h / a.rep : h) * rec_bytes;
+    const size_t rec_bytes = R::BYTES + (KIND == DELTA ? C * 4 * V : 0);
+    const int c0 = chunk_key(a.q_start, b);
     auto stage = [&](int i) {
         if (i < chunks) {
             uint8_t * dst = smem + i % ST * P::STAGE;
-            const uint8_t * src = rec0 + i * rec_step;
+            const uint8_t * src = KIND == SSD ? ssd_group_part<K>(a, c0 + i, h / a.rep) : (const uint8_t *) a.chunk + ((size_t) (c0 + i) * H + h) * rec_bytes;
 #pragma unroll 4
-            for (int o = tid * 16; o < R::BYTES; o += PT * 16) cp16(dst + o, src + o);
+            for (int o = tid * 16; o < (KIND == SSD ? R::A : R::BYTES); o += PT * 16) cp16(dst + o, src + o);
+            if (KIND == SSD) {
+                const uint8_t * hr = ssd_head_part<K>(a, c0 + i, h);
+                for (int o = tid * 16; o < R::BYTES - R::A; o += PT * 16) cp16(dst + R::A + o, hr + o);
+            }
             if (KIND == DELTA) {
                 for (int o = tid * 16; o < units / 2 * (C * 64); o += PT * 16) cp16(dst + P::X + o, src + R::BYTES + v0 / 16 * (C * 64) + o);
             } else {
@@ -477,7 +508,6 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                     else if (u < units)
                         cp16(dst + P::X + row * P::XS + (u << 4), (const bf16 *) a.v + (size_t) (r0 + i * C + row) * H * V + h * V + v0 + u * 8);
                 }
-                if (KIND == SSD && tid < m) cp4(dst + P::F + tid * 4, a.s + (size_t) (r0 + i * C + tid) * H + h);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -495,46 +525,17 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[i][e] = past ? state[(size_t) (i * 8 + fc + (e & 1)) * V + 8 * (e >> 1)] : 0.f;
-    const float na = KIND == SSD ? a.neg_a[h] * LOG2E : 0.f, skip = KIND == SSD ? a.skip[h] : 0.f;
-    float g = 0.f, f = 0.f;                                  // SSD: lane t holds G_t and the factor of the chunk at hand
-    // SSD: the chunk's G and factors, and its A (C / WARPS rows by this warp): q . k, the decay between the two tokens, the
-    // factor of the earlier one, and D on the diagonal
-    auto decays = [&](int ch) {
-        const uint8_t * rec = smem + ch % ST * P::STAGE;
-        f = lane < n - ch * C ? ((const float *) (rec + P::F))[lane] : 0.f;
-        g = na * f;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const float x = __shfl_up_sync(0xffffffffu, g, o);
-            if (lane >= o) g += x;
-        }
-        uint8_t * A = smem + P::A + (ch & 1) * 2 * R::ATILE;
-#pragma unroll
-        for (int i = 0; i < C / P::WARPS; ++i) {
-            const int t = warp * (C / P::WARPS) + i;
-            const float gt = __shfl_sync(0xffffffffu, g, t);
-            float x = lane <= t ? ((const float *) (rec + R::A))[t * QK_LD + lane] * (ex2(gt - g) * f) : 0.f;
-            if (lane == t) x += skip;
-            const bf16 hi = __float2bfloat16(x);
-            *(bf16 *) (A + a_off(t, lane)) = hi;
-            *(bf16 *) (A + R::ATILE + a_off(t, lane)) = __float2bfloat16(x - to_f(hi));
-        }
-    };
-    if (KIND == SSD) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
-        __syncthreads();
-        decays(0);
-    }
     for (int ch = 0; ch < chunks; ++ch) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(KIND == SSD ? ST - 3 : ST - 2) : "memory");
-        __syncthreads();                                     // this chunk's record (SSD: the next one's and this chunk's A); the oldest is free
+        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+        __syncthreads();                                     // this chunk's record is there; the oldest is free
         stage(ch + ST - 1);
         const uint8_t * rec = smem + ch % ST * P::STAGE;
         const uint32_t rec_addr = sm100::smem_u32(rec);
-        const uint32_t A_addr = KIND == SSD ? sm100::smem_u32(smem + P::A + (ch & 1) * 2 * R::ATILE) : rec_addr + R::A;
+        const uint32_t A_addr = rec_addr + R::A;
         float4 * part = (float4 *) (smem + P::O) + warp * 128 + lane;          // this warp's partial sums: [4 token tiles][32 lanes]
         uint32_t xh[2][4], xl[2][4], yh[2][4], yl[2][4];     // u^T, hi and lo, 16 tokens at a time (x: of the read-out, y: of the update)
-        const float gC = KIND == SSD ? __shfl_sync(0xffffffffu, g, 31) : 0.f, dC = KIND == SSD ? ex2(gC) : 0.f;
+        const float * eg = (const float *) (rec + R::E), * wt = eg + C;        // SSD
+        const float dC = KIND == SSD ? eg[C - 1] : 0.f;
         if (active) {
             float o[4][4], w[4][4];
 #pragma unroll
@@ -612,16 +613,15 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                 for (int e = 0; e < 2; ++e) ldm4t(xh[e], rec_addr + P::X + (e * 16 + tr) * P::XS + ((grp * 2 + tu) << 4));
             }
             if (KIND == SSD) {
-                const float wt = f * ex2(gC - g);
 #pragma unroll
                 for (int e = 0; e < 2; ++e)
 #pragma unroll
                     for (int j = 0; j < 2; ++j) {            // tokens 16 e + 8 j + fc, + 1
-                        const float w0 = __shfl_sync(0xffffffffu, wt, e * 16 + j * 8 + fc), w1 = __shfl_sync(0xffffffffu, wt, e * 16 + j * 8 + fc + 1);
+                        const float2 wj = *(const float2 *) (wt + e * 16 + j * 8 + fc);
 #pragma unroll
                         for (int i = 2 * j; i < 2 * j + 2; ++i) {
                             const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &xh[e][i]);
-                            split2(x.x * w0, x.y * w1, yh[e][i], yl[e][i]);
+                            split2(x.x * wj.x, x.y * wj.y, yh[e][i], yl[e][i]);
                         }
                     }
             }
@@ -651,7 +651,6 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
             }
         }
         if (KIND != DELTA) __syncthreads();
-        const float eg = KIND == SSD ? ex2(g) : 0.f;
         if (active) {                                        // o^T of 4 / KS token tiles: the partial sums, then += u^T A^T
 #pragma unroll
             for (int k = 0; k < 4 / KS; ++k) {
@@ -664,8 +663,8 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                     o[0] += x.x; o[1] += x.y; o[2] += x.z; o[3] += x.w;
                 }
                 if (KIND == SSD) {
-                    const float e0 = __shfl_sync(0xffffffffu, eg, i * 8 + fc), e1 = __shfl_sync(0xffffffffu, eg, i * 8 + fc + 1);
-                    o[0] *= e0; o[1] *= e1; o[2] *= e0; o[3] *= e1;
+                    const float2 e = *(const float2 *) (eg + i * 8 + fc);
+                    o[0] *= e.x; o[1] *= e.y; o[2] *= e.x; o[3] *= e.y;
                 }
                 const uint32_t off = r * 64 + (((lane >> 3) ^ ((r >> 1) & 3)) << 4);
                 uint32_t y[4], z[4];
@@ -684,7 +683,6 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                 }
             }
         }
-        if (KIND == SSD && ch + 1 < chunks) decays(ch + 1);
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     if (slot >= 0 && active) {
@@ -714,18 +712,18 @@ template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t 
 }
 template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
-    constexpr int smem = 2 * C * (K + 4) * 4;
+    constexpr int smem = (2 * C * (K + 4) + C * (C + 1)) * 4;
     if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(a.T / C + a.n_seqs, a.H / a.rep + (a.H * a.V + 255) / 256 + 1), NT, smem, s, a);
+    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(a.T / C + a.n_seqs, a.H / a.rep * ((a.rep + HB - 1) / HB) + (a.H * a.V + 255) / 256), NT, smem, s, a);
     const int rc = launched();
     return rc ? rc : launch_pass<SSD, K>(a, s);
 }
 
 long long rec_bytes(const jib_state_mix & a) {
-#define REC(KIND) (a.K == 64 ? Rec<KIND, 64>::BYTES : Rec<KIND, 128>::BYTES)
+#define REC(KIND, FIELD) (a.K == 64 ? Rec<KIND, 64>::FIELD : Rec<KIND, 128>::FIELD)
     const long long nch = a.T / C + a.n_seqs;
-    if (a.kind == SSD) return nch * (a.H / a.rep) * REC(SSD);
-    return nch * a.H * (a.kind == DELTA ? REC(DELTA) + C * 4 * a.V : REC(LINEAR));
+    if (a.kind == SSD) return nch * (a.H / a.rep * REC(SSD, A) + a.H * (REC(SSD, BYTES) - REC(SSD, A)));
+    return nch * a.H * (a.kind == DELTA ? REC(DELTA, BYTES) + C * 4 * a.V : REC(LINEAR, BYTES));
 #undef REC
 }
 

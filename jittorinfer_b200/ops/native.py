@@ -778,8 +778,8 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
         scratch = [torch.empty(n, dtype=torch.uint8, device=proj.device)]
         sd.chunk, sd.chunk_bytes = scratch[0].data_ptr(), n
         if m.kind != "delta":
-            scratch += [torch.empty(T, H * V, dtype=proj.dtype, device=proj.device), f32(T, H)]
-            sd.v, sd.s = scratch[1].data_ptr(), scratch[2].data_ptr()
+            scratch.append(torch.empty(T, H * V, dtype=proj.dtype, device=proj.device))
+            sd.v = scratch[1].data_ptr()
     elif not single:
         scratch = [f32(T, 2 * (H // m.rep) * K), f32(T, H * V), f32(T, H * (1 if m.kind == "ssd" else K)), f32(T, H)]
         sd.qk, sd.v, sd.dec, sd.s = (x.data_ptr() for x in scratch)
