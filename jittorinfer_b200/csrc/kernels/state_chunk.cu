@@ -235,13 +235,23 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
     __syncthreads();
     // unit norms (folded into q and k) and running sums of the log decays
     if (KIND == DELTA) {
-        for (int r = warp; r < 2 * C; r += NT / 32) {
+        float ss[2 * C / (NT / 32)];                         // 8 rows per warp, their reductions side by side
+#pragma unroll
+        for (int i = 0; i < 2 * C / (NT / 32); ++i) {
+            const int r = warp + i * (NT / 32);
             const float * x = (r < C ? q : k) + (r & (C - 1)) * KS;
-            float ss = 0.f;
-            for (int c = lane; c < K; c += 32) ss += x[c] * x[c];
-            ss = warp_sum(ss);
-            if (lane == 0) norm[r] = rsqrtf(ss + 1e-6f) * (r < C ? a.q_scale : 1.f);
+            ss[i] = 0.f;
+#pragma unroll
+            for (int c = lane; c < K; c += 32) ss[i] += x[c] * x[c];
         }
+#pragma unroll
+        for (int i = 0; i < 2 * C / (NT / 32); ++i) ss[i] = warp_sum(ss[i]);
+        if (lane == 0)
+#pragma unroll
+            for (int i = 0; i < 2 * C / (NT / 32); ++i) {
+                const int r = warp + i * (NT / 32);
+                norm[r] = rsqrtf(ss[i] + 1e-6f) * (r < C ? a.q_scale : 1.f);
+            }
     } else if (tid < 2 * C) {
         norm[tid] = tid < C ? a.q_scale : 1.f;
     }
@@ -297,10 +307,18 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         *(bf16 *) (rec + R::A + a_off(s, t)) = __float2bfloat16(0.f);
         *(bf16 *) (rec + R::A + R::ATILE + a_off(s, t)) = __float2bfloat16(0.f);
     }
-    for (int t = warp; t < C; t += NT / 32) {                // the diagonal
-        float d = 0.f;
-        for (int c = lane; c < K; c += 32) d += q[t * KS + c] * k[t * KS + c];
-        d = warp_sum(d);
+    float dg[C / (NT / 32)];                                 // the diagonal
+#pragma unroll
+    for (int i = 0; i < C / (NT / 32); ++i) {
+        const int t = warp + i * (NT / 32);
+        dg[i] = 0.f;
+#pragma unroll
+        for (int c = lane; c < K; c += 32) dg[i] += q[t * KS + c] * k[t * KS + c];
+    }
+#pragma unroll
+    for (int i = 0; i < C / (NT / 32); ++i) {
+        const int t = warp + i * (NT / 32);
+        const float d = warp_sum(dg[i]);
         if (lane == 0) {
             const bf16 hi = __float2bfloat16(d);
             *(bf16 *) (rec + R::A + a_off(t, t)) = hi;
