@@ -235,6 +235,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *,
     od = out_dtype or x.dtype
     if out is None:
         out = torch.empty(T, N, dtype=od, device=x.device)
+    if T == 0:                  # e.g. the output head of a prompt portion nobody wants logits of
+        return out
     ws = workspace(x.device)
     d = GemmDesc()
     d.x, d.w, d.w2, d.out, d.residual = x.data_ptr(), w.data_ptr(), _p(w2), out.data_ptr(), _p(residual)

@@ -181,3 +181,23 @@ def test_quantised_file_expanded_on_the_device_serves_the_same_tokens(tmp_path, 
         outs.append(eng.generate(prompts, SamplingParams(ignore_eos=True), max_new_tokens=8))
         del eng
     assert outs[0] == outs[1], outs
+
+
+def test_prompt_longer_than_the_step_budget():
+    """Portions of a long prompt produce no output row: the output head then multiplies nothing."""
+    hp = preset("tiny")
+    w = random_weights(hp, seed=0, std=0.05)
+    prompt = torch.randint(0, hp.n_vocab, (150,), generator=torch.Generator().manual_seed(4)).tolist()
+
+    def first(n_batch):
+        m = DeepSeek2Model(hp, w.items(), dtype=torch.bfloat16, device="cuda")
+        eng = LLMEngine(m, EngineConfig(n_ctx=512, n_batch=n_batch, n_parallel=2, graph_buckets=(1, 2)))
+        out = eng.generate([prompt], SamplingParams(ignore_eos=True), max_new_tokens=3)[0]
+        eng.feed([("s", prompt[:100], [])])
+        logits = eng.feed([("s", prompt[100:], [49])])
+        return out, logits
+    out, l_cut = first(100)
+    whole, l_whole = first(256)
+    assert len(out) == len(whole) == 3
+    rows_close(l_cut, l_whole, l_whole.abs().max().item())
+    ops.nat().check_status()
