@@ -1,5 +1,5 @@
 // CUDA-core GEMM behind the same descriptor as gemm_tcgen05.cu: Y[b][t][n] = sum_k X[b][t][k] * W[b][n][k], optional second
-// weight (act(X W^T) * (X W2^T)), optional residual, optional expert segments.
+// weight (act(X W^T) * (X W2^T)) or a function of the single product, optional residual, optional expert segments.
 //
 // Two uses: fp32 operands in true 32-bit arithmetic (the tensor cores have no such mode), and bf16 operands whose rows are
 // not 16-byte multiples, which TMA cannot address.  A plain 64 x 64 tile with 4 x 4 results per thread.
@@ -20,6 +20,13 @@ __device__ __forceinline__ float to_f(float v) { return v; }
 // act(z) = z * sigmoid(gate_arg(z)): 0.5 (1 + tanh(u)) is sigmoid(2 u)
 __device__ __forceinline__ float gate_arg(float z, int act) {
     return act == JIB_ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+}
+
+__device__ __forceinline__ float unary(float v, const jib_gemm_desc & d) {
+    if (d.unary == JIB_UNARY_NONE) return v;
+    if (d.unary == JIB_UNARY_RELU2) return v > 0.f ? v * v : 0.f;
+    v *= d.scale;
+    return d.softcap > 0.f ? d.softcap * tanhf(v / d.softcap) : v;
 }
 
 template <typename T, bool DUAL>
@@ -80,7 +87,7 @@ __global__ void __launch_bounds__(NT) gemm_simt_kernel(const jib_gemm_desc d) {
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             if (n >= d.N) continue;
-            float y = DUAL ? acc[i][j] / (1.f + expf(-gate_arg(acc[i][j], d.act))) * acu[i][j] : acc[i][j];
+            float y = DUAL ? acc[i][j] / (1.f + expf(-gate_arg(acc[i][j], d.act))) * acu[i][j] : unary(acc[i][j], d);
             if (d.residual != nullptr) {
                 const long long ri = (long long) batch * d.res_batch_stride + row * d.ldr + n;
                 y += d.res_f32 ? ((const float *) d.residual)[ri] : to_f(((const bf16 *) d.residual)[ri]);

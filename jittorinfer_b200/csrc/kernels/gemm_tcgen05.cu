@@ -69,6 +69,8 @@ struct GemmArgs {
     int pdl_flags;            // grouped pairs: bit 0 = release dependents after the own wait, bit 1 = segment table valid at start
     int w_evict_first;        // weight tiles are loaded with the L2 evict_first policy (each is read once: small batches)
     int act;                  // of a gated pair (JIB_ACT_*)
+    int unary;                // of a single product (JIB_UNARY_*)
+    float scale, softcap;
     int vec_store;            // bf16 result rows are written as 16-byte vectors through a shared-memory transpose
     const int * src_token;    // grouped, decode batches: x holds the T token rows unsorted, every expert multiplies all of
                               // them (one token tile) and sorted row i of the result is accumulator column src_token[i]
@@ -149,6 +151,14 @@ __device__ __forceinline__ uint2 pack_bf16x4(float4 v) {
 __device__ __forceinline__ float gated(float x, int act) {
     const float z = act == JIB_ACT_GELU_TANH ? 1.5957691216057308f * (x + 0.044715f * x * x * x) : x;
     return x / (1.0f + __expf(-z));
+}
+
+// JIB_UNARY_* of a single product; softcap y = c tanh(s v / c) with tanh(u) = 1 - 2 / (1 + e^{2u})
+__device__ __forceinline__ float unary(float v, const GemmArgs & a) {
+    if (a.unary == JIB_UNARY_NONE) return v;
+    if (a.unary == JIB_UNARY_RELU2) return v > 0.f ? v * v : 0.f;
+    v *= a.scale;
+    return a.softcap > 0.f ? a.softcap * (1.f - 2.f / (1.f + __expf(2.f * fminf(v / a.softcap, 40.f)))) : v;
 }
 
 // Cluster-wide barrier (all threads of all CTAs of the cluster) and a load from a peer CTA's shared memory.
@@ -385,7 +395,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         }
         // One finished element: feature n of row (row_base + t_rel); gv / uv are the summed accumulators.
         auto finish = [&](int t_rel, float gv, float uv) {
-            float y = DUAL ? gated(gv, args.act) * uv : gv;
+            float y = DUAL ? gated(gv, args.act) * uv : unary(gv, args);
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
@@ -562,7 +572,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     const int ltid = (int) threadIdx.x - 64;
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : g[j];
+                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : unary(g[j], args);
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -851,7 +861,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
-                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : g;
+                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : unary(g, args);
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
@@ -1144,7 +1154,8 @@ extern "C" JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream_)
     if (a.ag_flags != nullptr && (a.ag_epoch == nullptr || a.ag_rows <= 0 || a.ag_world <= 0 || grouped || batch != 1)) return JIB_E_ARG;
     if (a.ar_rs_rows < 0) return JIB_E_ARG;
     if (a.row_ptr != nullptr && (dual || d->out_f32 || d->residual != nullptr || d->ar != nullptr)) return JIB_E_ARG;
-    a.act = d->act;
+    a.act = d->act; a.unary = dual ? JIB_UNARY_NONE : d->unary; a.scale = d->scale; a.softcap = d->softcap;
+    if (a.unary != JIB_UNARY_NONE && d->ar != nullptr) return JIB_E_ARG;
     memset(&a.ar, 0, sizeof(a.ar));
     if (d->ar != nullptr) {
         const JibArCtx * ar = (const JibArCtx *) d->ar;
@@ -1318,7 +1329,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16_noalloc(const void * x, const void * w, 
     a.expert_list = nullptr;
     a.list_tiles = 0;
     a.ag_flags = nullptr; a.ag_epoch = nullptr; a.ag_rows = 0; a.ag_world = 0; a.ar_rs_rows = 0; a.ag_spin_limit = 0;
-    a.act = JIB_ACT_SILU;
+    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = 0.f;
     memset(&a.ar, 0, sizeof(a.ar));
     dim3 grid(p.n_tiles, 1, p.splits);
     switch (p.bn) {

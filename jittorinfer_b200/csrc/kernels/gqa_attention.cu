@@ -1,9 +1,9 @@
 // Grouped-query attention over paged key / value rows: H query heads share G key / value heads (head h reads h / (H / G)).
 // A cached row holds the normed and rotated keys of a token (G * D columns), then its values (G * V columns).
 //
-//   gqa_qkv_post    per-head RMS norm of q and k, rotate-half RoPE on the first rot dimensions, rows into the cache
+//   gqa_qkv_post    per-head RMS norm of q and k (or none), rotate-half RoPE on the first rot dimensions, rows into the cache
 //   gqa_attention   scores * scale, softcap, causal mask with a sliding window and / or chunks counted from position 0, softmax
-//                   with or without a sink (a key of score 0 without a value), a gate per head: any mix of portions and single
+//                   with or without a sink (a key without a value, of score 0 or of a number per head), a gate per head: any mix of portions and single
 //                   tokens, keys split over a thread-block cluster.  bf16 heads whose sizes are multiples of 16: products on the
 //                   tensor cores (gqa_mma); fp32 and other sizes: CUDA cores (gqa_attention).  Prompts with heads of 128 have a
 //                   kernel of their own (mha_prefill_tcgen05.cu).
@@ -95,16 +95,17 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
 #pragma unroll
     for (int i = 0; i < N; ++i) {                            // requested before the reduction
         const int c = lane + 32 * i;
-        wt[i] = c < D ? w[c] : 0.f;
+        wt[i] = w != nullptr && c < D ? w[c] : 0.f;
         r[i] = c < a.rot ? cs[c < half ? c : c - half] : make_float2(1.f, 0.f);
     }
-    const float inv = rsqrtf(warp_sum(ss) / (float) D + a.eps);
+    if (w != nullptr) {
+        const float inv = rsqrtf(warp_sum(ss) / (float) D + a.eps);
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        const int c = lane + 32 * i;
-        e[i] *= inv * wt[i];
-        if (c < D) x[c] = e[i];
+        for (int i = 0; i < N; ++i) e[i] *= inv * wt[i];
     }
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+        if (lane + 32 * i < D) x[lane + 32 * i] = e[i];
     __syncwarp();
     T * dst = is_q ? q_out + ((size_t) t * H + head) * D : row + head * D;
 #pragma unroll
@@ -206,7 +207,9 @@ __device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, c
     if (n_splits > 1) cluster_sync(); else __syncthreads();
     for (int i = threadIdx.x + (int) blockIdx.z * NT; i < w.rows * V; i += NT * n_splits) {
         const int r = i / V, col = i % V;
-        float ms[8], ls[8], os[8], m = a.sink ? 0.f : -INFINITY;
+        const int t = w.q0 + w.i0 + r / w.nh, h = w.h0 + r % w.nh;
+        const float sink = !a.sink ? -INFINITY : a.sink_w != nullptr ? a.sink_w[h] : 0.f;
+        float ms[8], ls[8], os[8], m = sink;
 #pragma unroll
         for (int s = 0; s < 8; ++s) {                        // every peer's value requested before any is used
             ms[s] = -INFINITY;
@@ -216,11 +219,10 @@ __device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, c
             ls[s] = n_splits > 1 ? ld_peer(l_s + r, s) : l_s[r];
             os[s] = n_splits > 1 ? ld_peer(part + r * V + col, s) : part[r * V + col];
         }
-        const int t = w.q0 + w.i0 + r / w.nh, h = w.h0 + r % w.nh;
         const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + h]) : 0.f;
 #pragma unroll
         for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
-        float l = a.sink ? exp_t<T>(-m) : 0.f, o = 0.f;
+        float l = a.sink ? exp_t<T>(sink - m) : 0.f, o = 0.f;
 #pragma unroll
         for (int s = 0; s < 8; ++s) {
             const float e = ms[s] == -INFINITY ? 0.f : exp_t<T>(ms[s] - m);

@@ -17,13 +17,16 @@ enum {
 
 // Activation of a gated pair: z * sigmoid(z), or 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
 enum { JIB_ACT_SILU = 0, JIB_ACT_GELU_TANH = 1 };
+// Function of a single product (no w2): none, max(y, 0)^2, or s y with s = scale, capped to softcap tanh(s y / softcap) unless softcap is 0.
+enum { JIB_UNARY_NONE = 0, JIB_UNARY_RELU2 = 1, JIB_UNARY_CAP = 2 };
 
 #ifdef __cplusplus
 extern "C" {
 #endif
 
 // Y[b][t][n] = sum_k X[b][t][k] * W[b][n][k]  (bf16 in, fp32 accumulate), optional second weight
-// (w2: out = act(X W^T) * (X W2^T), act = silu or the tanh form of gelu), optional residual add, optional expert-grouped rows.
+// (w2: out = act(X W^T) * (X W2^T), act = silu or the tanh form of gelu) or a function of the single product, optional residual add
+// (row stride 0: one row for all tokens, i.e. a bias), optional expert-grouped rows.
 typedef struct jib_gemm_desc {
     const void * x;            // bf16 activations
     const void * w;            // bf16 weights [batch][N][K]
@@ -67,6 +70,8 @@ typedef struct jib_gemm_desc {
                                //   start only once the table is known to be complete), 2 on the second (it may read the table and
                                //   request weights before the first launch has finished); 0 otherwise
     int act;                   // with w2: JIB_ACT_*
+    int unary;                // without w2: JIB_UNARY_*, applied before the residual (not with ar)
+    float scale, softcap;     // of JIB_UNARY_CAP
 } jib_gemm_desc;
 
 JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream);
@@ -103,9 +108,10 @@ JIB_EXPORT int jib_gather_rows(const void * x, const int * src_row, void * out, 
 // n_shared columns name the shared experts (ids E, E+1, ...; weight 1) so that they run in the grouped GEMMs.
 // bias: added to the scores for the choice only (DeepSeek-V3); logit_bias: added to the router logits before anything else.
 // g NULL: logits already holds the router outputs (fp32 activations).
+// shared_gate: w_router and logits have a row / column more, E, and the shared experts' weight is sigmoid(logits[t][E]) instead of 1.
 JIB_EXPORT int jib_moe_gate(const void * g, const float * w_router, const float * bias, const float * logit_bias, float * logits, int * ids,
                             float * wts, int T, int d, int E, int k, int n_group, int topk_group, float scale, int norm, int sigmoid,
-                            int n_shared, int group_top2, void * stream);
+                            int n_shared, int group_top2, int shared_gate, void * stream);
 // jib_moe_gate + jib_moe_permute (over the k + n_shared id columns) in one launch, for T <= 64.  counter: one device int that is
 // zero between launches.  norm_w != NULL: the rows of g are RMS-normalised first (as jib_rmsnorm would) and stored to g_out.
 JIB_EXPORT int jib_moe_route_fused(const void * g, const float * w_router, const float * bias, float * logits, int * ids, float * wts,
@@ -155,7 +161,8 @@ JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * 
                                int window, int n_q_tiles, void * out, long long ldo, int * status, void * stream);
 
 // ---- parallel blocks over an fp32 residual (parallel_block.cu), per-sequence state (recurrent.cu) ---------------------------
-// What happens to a token's row once its residual value is known: x_out [T][d] fp32; with norm_w, h_out = row / rms * norm_w; with
+// What happens to a token's row once its residual value is known: x_out [T][d] fp32; with norm_w, h_out = row / rms * norm_w (with
+// norm2_w too, h2_out = row / rms * norm2_w); with h_out but no norm_w, h_out = the row itself in the activation type; with
 // conv_w ([taps][d] fp32, one token per sequence only), hc_out = h + causal convolution of h, whose last taps - 1 inputs live in
 // conv_state [n_state][taps - 1][d] at row seq_slots[t] (negative: none) and are advanced.  positions[t] == 0 starts from zeros.
 typedef struct jib_row_tail {
@@ -170,6 +177,8 @@ typedef struct jib_row_tail {
     int * status;
     float eps;
     int taps, n_state;
+    const float * norm2_w;     // null, or a second norm of the same row (not with conv_w)
+    void * h2_out;
 } jib_row_tail;
 // x_out = scale * table[ids[t]], RMS-normed and times w unless w is null.
 JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, float scale, int T, int d, int n_vocab, int f32,
@@ -182,12 +191,18 @@ JIB_EXPORT int jib_post_norm(const float * x, const void * y, const float * w, f
 JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, const void * gates, long long gate_stride, const float * b1,
                                 const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
                                 const jib_row_tail * tail, void * stream);
+// x_out = x + s1 * o + s2 * (sum_j wts[t][j] * y[dest[t][j]] + g * f), s1, s2 [d]; any of o, y, f may be null (absent).  f [T][d]: a dense
+// sublayer; g = sigmoid(f_gate[t * ld_gate]), 1 with f_gate null.  x_out may be x, or null: only the tail's norms.
+JIB_EXPORT int jib_scaled_update(const float * x, const void * o, const float * s1, const void * y, const int * dest, const float * wts, int k,
+                                 const void * f, const float * f_gate, long long ld_gate, const float * s2, int T, int d, int f32,
+                                 const jib_row_tail * tail, void * stream);
 JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
                             void * stream);
-// out = h + causal convolution over time of h (w [taps][d] fp32); sequence b continues from, and advances, its stored rows.
-JIB_EXPORT int jib_causal_conv(const void * h, const float * w, int taps, void * state, int n_state, const int * seq_slots,
-                               const int * positions, const int * q_start, int n_seqs, int T, int d, int f32, void * out, int * status,
-                               void * stream);
+// out = h + causal convolution over time of h (w [taps][d] fp32), or with silu != 0 out = silu(bias + convolution); h [T][ldh], out
+// [T][d]; sequence b continues from, and advances, its stored rows (state [n_state][taps - 1][d]).
+JIB_EXPORT int jib_causal_conv(const void * h, long long ldh, const float * w, const float * bias, int silu, int taps, void * state, int n_state,
+                               const int * seq_slots, const int * positions, const int * q_start, int n_seqs, int T, int d, int f32, void * out,
+                               int * status, void * stream);
 // Gated recurrence over zxg [T][>= 3W]; state [n_state][W] fp32; single: one token per sequence (row t = sequence t).
 JIB_EXPORT int jib_mingru(const void * zxg, long long ld, const float * zb, const float * xb, float * state, int n_state,
                           const int * seq_slots, const int * positions, const int * q_start, int n_seqs, int T, int W, int single, int f32,
@@ -202,11 +217,12 @@ typedef struct jib_gqa {
     long long n_slots, row;
     int H, G, D, V, rot, block_size, max_blocks, n_seqs, T, max_pos;
     int window, chunk;         // position i sees j <= i with i - j < window (0: no window) and j / chunk == i / chunk (0: no chunks)
-    int sink;                  // 1: the softmax' denominator also holds exp(0)
+    int sink;                  // 1: the softmax' denominator also holds exp(0), or exp(sink_w[h])
     float scale, softcap;      // softcap 0: none
     float eps, out_scale;
+    const float * sink_w;      // [H] or null
 } jib_gqa;
-// q, k, v: columns of the projection (row stride ld).  rope [max_pos][rot / 2] pairs (cos, sin); pairs are (i, i + rot / 2).
+// q, k, v: columns of the projection (row stride ld); q_norm, k_norm [D], or null: no norm.  rope [max_pos][rot / 2] pairs (cos, sin); pairs are (i, i + rot / 2).
 JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * k, const void * v, long long ld, const float * q_norm,
                                 const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int f32, void * stream);
 // q [T][H][D]; gate null or [T][ld_gate] pre-activations of one sigmoid per head; out [T][ldo].  single: one token per sequence.
@@ -246,6 +262,25 @@ typedef struct jib_state_mix {
 // single: one token per sequence (row t = sequence t; scratch only for SSD: o).  K <= 512.
 JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, void * stream);
 JIB_EXPORT long long jib_state_chunk_bytes(const jib_state_mix * m);
+
+// ---- selective scan: a diagonal state per channel (selective_scan.cu) -------------------------------------------------------------
+//   S[c][n] <- exp(dt_c a[c][n]) S[c][n] + dt_c x_c B_n;   y_c = (sum_n S[c][n] C_n + skip_c x_c) * silu(z_c) * out_scale,   dt = softplus(dt_c)
+// over ch channels (a multiple of 8) with N states each (a multiple of 8, at most 256).
+typedef struct jib_scan {
+    const void * x, * z, * bc; // activations: [T][ldx], [T][ldz], and [T][ldbc] = B | C
+    const float * dt;          // [T][lddt] pre-activations of the step sizes, bias included
+    void * y;                  // [T][ldy]
+    const float * neg_a;       // [ch][N]
+    const float * skip;        // [ch]
+    float * state;             // [n_state][ch][N]
+    const int * seq_slots, * positions, * q_start;
+    int * status;
+    long long ldx, ldz, ldbc, lddt, ldy;
+    int ch, N, n_state, n_seqs, T;
+    float out_scale;
+} jib_scan;
+// single: one token per sequence (row t = sequence t).
+JIB_EXPORT int jib_selective_scan(const jib_scan * m, int single, int f32, void * stream);
 
 // ---- expert-parallel all-to-all over peer memory (ep_alltoall.cu); ctx is a JibEpCtx (ep_alltoall.h) ---------
 JIB_EXPORT int jib_ep_plan(const int * ids, int T, int k, const struct JibEpCtx * ctx, int site, int * seg, int * pair_dst, void * stream);

@@ -68,6 +68,7 @@ struct MhaArgs {
     const bf16 * gate;        // null, or [T][ld_gate] pre-activations of a sigmoid per head
     long long ld_gate;
     int G, chunk, sink;
+    const float * sink_w;     // null: the sink's score is 0
     float cap_log2e, inv_cap2, out_scale;     // softcap * log2 e (0: none), 2 * scale * log2 e / softcap
 };
 
@@ -345,7 +346,8 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             // rows end inside this warp; only the stores are predicated per row.  (Executed under a per-lane condition it
             // never completes.)
             const bool valid = r < rows;
-            if (GQA && a.sink && l_sum > 0.f) l_sum += exp2f(-m_ref);     // a key of score 0 without a value
+            if (GQA && a.sink && l_sum > 0.f)                             // a key of its own score without a value
+                l_sum += exp2f((a.sink_w != nullptr ? a.sink_w[h] * 1.4426950408889634f : 0.f) - m_ref);
             float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
             if (GQA) {
                 inv *= a.out_scale;
@@ -493,7 +495,7 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
     if (rc) return rc;
     MhaArgs a = {};
     a.q_start = m->q_start; a.seq_lens = m->seq_lens; a.kv_start = kv_start; a.out = (bf16 *) out; a.status = m->status; a.ldo = ldo;
-    a.n_seqs = m->n_seqs; a.T = m->T; a.H = m->H; a.G = m->G; a.window = m->window; a.chunk = m->chunk; a.sink = m->sink;
+    a.n_seqs = m->n_seqs; a.T = m->T; a.H = m->H; a.G = m->G; a.window = m->window; a.chunk = m->chunk; a.sink = m->sink; a.sink_w = m->sink_w;
     a.scale_log2e = m->scale * 1.4426950408889634f;
     a.cap_log2e = m->softcap * 1.4426950408889634f;
     a.inv_cap2 = m->softcap > 0.f ? 2.f * a.scale_log2e / m->softcap : 0.f;

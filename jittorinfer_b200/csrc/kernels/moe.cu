@@ -161,7 +161,7 @@ __device__ __noinline__ void gate_token(const float * __restrict__ logits_row, c
                                            float * __restrict__ wts, int t, int E, int k, int n_group, int topk_group, float scale,
                                            int norm, int sigmoid, int n_shared, int group_top2, float * prob, float * sel,
                                            float * gscore, int * ids_copy = nullptr, bool dry = false,
-                                           const float * __restrict__ logit_bias = nullptr) {
+                                           const float * __restrict__ logit_bias = nullptr, int shared_gate = 0) {
     // dry: runs the same instructions on whatever `prob` holds and stores nothing -- a caller that is still waiting for its
     // inputs uses it to pull this code into the SM's instruction cache ahead of the real call
     const int lane = threadIdx.x & 31;
@@ -242,10 +242,10 @@ __device__ __noinline__ void gate_token(const float * __restrict__ logits_row, c
         }
         if (ids_copy != nullptr) ids_copy[t * ld + lane] = my_id;
     } else if (lane < ld) {
-        // shared experts ride along as always-selected experts E, E+1, ... with weight 1
+        // shared experts ride along as always-selected experts E, E+1, ... with weight 1, or that of their gate
         if (!dry) {
             ids[(size_t) t * ld + lane] = E + (lane - k);
-            wts[(size_t) t * ld + lane] = 1.f;
+            wts[(size_t) t * ld + lane] = shared_gate ? 1.f / (1.f + expf(-__ldcg(logits_row + E))) : 1.f;
         }
         if (ids_copy != nullptr) ids_copy[t * ld + lane] = E + (lane - k);
     }
@@ -255,7 +255,7 @@ __device__ __noinline__ void gate_token(const float * __restrict__ logits_row, c
 __global__ void __launch_bounds__(32) moe_gate_kernel(const float * __restrict__ logits, const float * __restrict__ bias,
                                                       int * __restrict__ ids, float * __restrict__ wts, int E, int k, int n_group,
                                                       int topk_group, float scale, int norm, int sigmoid, int n_shared,
-                                                      int group_top2, const float * __restrict__ logit_bias, int warm) {
+                                                      int group_top2, const float * __restrict__ logit_bias, int shared_gate, int warm) {
     JIB_KS(10, 0);
     PDL_TRIGGER_TOP();
     __shared__ float prob[MAX_E];
@@ -271,8 +271,8 @@ __global__ void __launch_bounds__(32) moe_gate_kernel(const float * __restrict__
     }
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     JIB_KS(10, 1);
-    gate_token(logits + (size_t) t * E, bias, ids, wts, t, E, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, prob,
-               sel, gscore, nullptr, false, logit_bias);
+    gate_token(logits + (size_t) t * (E + shared_gate), bias, ids, wts, t, E, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2,
+               prob, sel, gscore, nullptr, false, logit_bias, shared_gate);
     JIB_KS(10, 9);
 }
 
@@ -752,17 +752,18 @@ extern "C" {
 
 int jib_moe_gate(const void * g, const float * w_router, const float * bias, const float * logit_bias, float * logits, int * ids, float * wts,
                  int T, int d, int E, int k, int n_group, int topk_group, float scale, int norm, int sigmoid, int n_shared, int group_top2,
-                 void * stream) {
+                 int shared_gate, void * stream) {
     if (T <= 0) return 0;
+    shared_gate = shared_gate ? 1 : 0;
     if (E > MAX_E || k + n_shared > 32 || n_shared < 0 || k > E || n_group > 32 || (n_group > 1 && E % n_group)) return JIB_E_ARG;
     if (g != nullptr) {
         if (d % 8 || d > GATE_MAXC * GATE_NT * 8) return JIB_E_ARG;
-        JIB_LAUNCH((router_logits_kernel), dim3(E, (T + 63) / 64), GATE_NT, 0, (cudaStream_t) stream, (const bf16 *) g, w_router, logits, T, d, E,
-                   jib::warm_for(T));
+        JIB_LAUNCH((router_logits_kernel), dim3(E + shared_gate, (T + 63) / 64), GATE_NT, 0, (cudaStream_t) stream, (const bf16 *) g, w_router, logits, T, d,
+                   E + shared_gate, jib::warm_for(T));
         if (cudaGetLastError() != cudaSuccess) return JIB_E_LAUNCH;
     }
     JIB_LAUNCH((moe_gate_kernel), T, 32, 0, (cudaStream_t) stream, logits, bias, ids, wts, E, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2,
-               logit_bias, jib::warm_for(T));
+               logit_bias, shared_gate, jib::warm_for(T));
     return launched();
 }
 

@@ -2,10 +2,12 @@
 //
 // Sublayers side by side on one norm:        h = norm(x);   x <- x + m * (sigmoid(g1) * mixer(h) + sigmoid(g2) * ff(h))
 // Sublayers in turn between two norms each:  x <- x + norm'(f(norm(x)))
+// Sublayers side by side, a norm and a scale each:  x <- x + s1 mixer(norm1(x)) + s2 ff(norm2(x))
 //
 //   embed_norm     x = scale * embedding row, normed or not, then the first block's norm
 //   block_update   the first form's sum -- the expert-weighted combine of the feed-forward included -- then the next block's norm
 //   post_norm      the second form's sum with the norm of the sublayer's output, then the next sublayer's norm
+//   scaled_update  the third form's sum, the experts' combine and a gated shared expert included, then one or two norms of the row
 //   rms_rows       norm of selected rows (before the output head)
 //
 // One CTA owns one token's row and keeps it in registers, so the sum, the residual store and the norm that follows are one
@@ -114,9 +116,14 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
         if (i < nv) {
             Pack8<float> k;
             k.set(v[it]);
-            if (!dry) k.store((float *) a.x_out + (size_t) t * d + 8 * i);
+            if (!dry && a.x_out != nullptr) k.store((float *) a.x_out + (size_t) t * d + 8 * i);
 #pragma unroll
             for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+            if (a.norm_w == nullptr && a.h_out != nullptr && !dry) {
+                Pack8<T> hp;
+                hp.set(v[it]);
+                hp.store((T *) a.h_out + (size_t) t * d + 8 * i);
+            }
         }
     }
     if (a.norm_w == nullptr) return;
@@ -133,6 +140,14 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
         Pack8<T> hp;
         hp.set(h);
         if (!dry) hp.store((T *) a.h_out + (size_t) t * d + 8 * i);
+        if (!conv && a.norm2_w != nullptr) {
+            float h2[8];
+            load8(a.norm2_w + 8 * i, w);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) h2[e] = v[it][e] * inv * w[e];
+            hp.set(h2);
+            if (!dry) hp.store((T *) a.h2_out + (size_t) t * d + 8 * i);
+        }
         if (conv) {
             hp.get(h);                               // the convolution reads what a later step will read back from the state
             float c[8], k[8], s[8];
@@ -233,17 +248,45 @@ struct UpdateArgs {
 
 constexpr int MAX_TOP = 32;
 
+// f = sum_j wts[j] * y[rows[j]] over 8 adjacent columns
+template <typename T>
+__device__ __forceinline__ void expert_sum(const T * y, const int * rows, const float * wts, int k, int d, float (&f)[8]) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = 0.f;
+    int j = 0;
+    for (; j + 4 <= k; j += 4) {
+        Pack8<T> p[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) p[u].load(y + (size_t) rows[j + u] * d);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            float q[8];
+            p[u].get(q);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] += wts[j + u] * q[e];
+        }
+    }
+    for (; j < k; ++j) {
+        float q[8];
+        load8(y + (size_t) rows[j] * d, q);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] += wts[j] * q[e];
+    }
+}
+// a token's expert rows and weights into shared memory; all threads of the CTA
+__device__ __forceinline__ void stage_pairs(const int * dest, const float * w, int k, int t, bool dry, int * rows, float * wts) {
+    if (threadIdx.x < k) {
+        const int r = dry ? 0 : dest[(size_t) t * k + threadIdx.x];
+        rows[threadIdx.x] = r < 0 ? 0 : r;
+        wts[threadIdx.x] = r < 0 ? 0.f : w[(size_t) t * k + threadIdx.x];
+    }
+    __syncthreads();
+}
+
 template <typename T, int NT, int MAXV, bool CONV>
 __device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, bool dry) {
     const int t = blockIdx.x, d = a.d, nv = d / 8;
-    if (a.y != nullptr) {
-        if (threadIdx.x < a.k) {
-            const int r = dry ? 0 : a.dest[(size_t) t * a.k + threadIdx.x];
-            rows[threadIdx.x] = r < 0 ? 0 : r;
-            wts[threadIdx.x] = r < 0 ? 0.f : a.wts[(size_t) t * a.k + threadIdx.x];
-        }
-        __syncthreads();
-    }
+    if (a.y != nullptr) stage_pairs(a.dest, a.wts, a.k, t, dry, rows, wts);
     float v[MAXV][8];
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
@@ -259,28 +302,7 @@ __device__ __noinline__ void block_update_row(const UpdateArgs & a, const jib_ro
         if (a.y != nullptr) {
             g2p.load((const T *) a.gates + (size_t) t * a.gate_stride + d + 8 * i);
             b2p.load(a.b2 + 8 * i);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = 0.f;
-            const T * y = (const T *) a.y + 8 * i;
-            int j = 0;
-            for (; j + 4 <= a.k; j += 4) {
-                Pack8<T> p[4];
-#pragma unroll
-                for (int u = 0; u < 4; ++u) p[u].load(y + (size_t) rows[j + u] * d);
-#pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    float q[8];
-                    p[u].get(q);
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) f[e] += wts[j + u] * q[e];
-                }
-            }
-            for (; j < a.k; ++j) {
-                float q[8];
-                load8(y + (size_t) rows[j] * d, q);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) f[e] += wts[j] * q[e];
-            }
+            expert_sum<T>((const T *) a.y + 8 * i, rows, wts, a.k, d, f);
         }
         float o[8], g[8], b[8], x[8];
         op.get(o); g1p.get(g); b1p.get(b); xp.get(x);
@@ -358,9 +380,74 @@ __global__ void __launch_bounds__(NT) post_norm_kernel(const float * x, const T 
     post_norm_row<T, NT, MAXV>(x, y, w, eps, d, tail, red, false);
 }
 
-// The three row kernels for widths that 8-element vectors do not divide: element by element, the row re-read from memory.
+struct ScaledArgs {
+    const float * x;
+    const void * o, * y, * f;
+    const float * s1, * s2;
+    const int * dest;
+    const float * wts, * f_gate;
+    long long ld_gate;
+    int k, d;
+};
+
+template <typename T, int NT, int MAXV>
+__device__ __noinline__ void scaled_update_row(const ScaledArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, bool dry) {
+    const int t = blockIdx.x, d = a.d, nv = d / 8;
+    if (a.y != nullptr) stage_pairs(a.dest, a.wts, a.k, t, dry, rows, wts);
+    const float g = a.f_gate != nullptr ? sigmoid<T>(a.f_gate[(size_t) t * a.ld_gate]) : 1.f;
+    float v[MAXV][8];
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it) {
+        const int i = threadIdx.x + it * NT;
+        if (i >= nv) continue;
+        Pack8<float> xp, s1p, s2p;
+        Pack8<T> op, fp;
+        xp.load(a.x + (size_t) t * d + 8 * i);       // everything the row needs is requested before any of it is used
+        op.zero(); fp.zero(); s1p.zero(); s2p.zero();
+        if (a.o != nullptr) {
+            op.load((const T *) a.o + (size_t) t * d + 8 * i);
+            s1p.load(a.s1 + 8 * i);
+        }
+        if (a.y != nullptr || a.f != nullptr) s2p.load(a.s2 + 8 * i);
+        if (a.f != nullptr) fp.load((const T *) a.f + (size_t) t * d + 8 * i);
+        float sum[8], p[8], q[8];
+        if (a.y != nullptr) {
+            expert_sum<T>((const T *) a.y + 8 * i, rows, wts, a.k, d, sum);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) sum[e] = 0.f;
+        }
+        fp.get(p); s2p.get(q);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] = (sum[e] + g * p[e]) * q[e];
+        op.get(p); s1p.get(q);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] += p[e] * q[e];
+        xp.get(p);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[it][e] = p[e] + sum[e];
+    }
+    finish_row<T, NT, MAXV, false>(v, t, d, tail, red, dry);
+}
+
+template <typename T, int NT, int MAXV>
+__global__ void __launch_bounds__(NT) scaled_update_kernel(const __grid_constant__ ScaledArgs a, const __grid_constant__ jib_row_tail tail, int warm) {
+    PDL_TRIGGER_TOP();
+    __shared__ float red[32];
+    __shared__ int rows[MAX_TOP];
+    __shared__ float wts[MAX_TOP];
+    if (warm) {
+        scaled_update_row<T, NT, MAXV>(a, tail, red, rows, wts, true);
+        __syncthreads();
+    }
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    scaled_update_row<T, NT, MAXV>(a, tail, red, rows, wts, false);
+}
+
+// The row kernels for widths that 8-element vectors do not divide: element by element, the row re-read from memory.
 //   ids:  v = scale * src[ids[t]], normed by w if given         (src: T table of n_src rows)
 //   y:    v = x[t] + y / rms(y) * w
+//   o..:  v = x[t] + the scaled sublayers of jib_scaled_update
 //   else: v = x[rows[t]] (rows null: x[t])                      (x has n_src rows)
 struct AnyRow {
     const void * src;
@@ -371,6 +458,7 @@ struct AnyRow {
     const float * w;
     float eps, scale;
     int d, n_src;
+    ScaledArgs u;
 };
 template <typename T> __device__ __forceinline__ float as_f(const void * p, size_t i);
 template <> __device__ __forceinline__ float as_f<bf16>(const void * p, size_t i) { return __bfloat162float(((const bf16 *) p)[i]); }
@@ -382,8 +470,13 @@ template <typename T>
 __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_row_tail tail) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
+    __shared__ int pair_rows[MAX_TOP];
+    __shared__ float pair_wts[MAX_TOP];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int t = blockIdx.x, d = a.d;
+    const ScaledArgs & u = a.u;
+    if (u.y != nullptr) stage_pairs(u.dest, u.wts, u.k, t, false, pair_rows, pair_wts);
+    const float gate = u.f_gate != nullptr ? sigmoid<T>(u.f_gate[(size_t) t * u.ld_gate]) : 1.f;
     size_t row = t;
     if (a.ids != nullptr || a.rows != nullptr) {
         int r = a.ids != nullptr ? a.ids[t] : a.rows[t];
@@ -409,6 +502,13 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
             v = a.scale * as_f<T>(normed, row * d + i);
             if (a.w != nullptr) v *= inv * a.w[i];
         }
+        if (u.y != nullptr || u.f != nullptr) {
+            float f = u.f != nullptr ? gate * as_f<T>(u.f, row * d + i) : 0.f;
+            if (u.y != nullptr)
+                for (int j = 0; j < u.k; ++j) f += pair_wts[j] * as_f<T>(u.y, (size_t) pair_rows[j] * d + i);
+            v += u.s2[i] * f;
+        }
+        if (u.o != nullptr) v += u.s1[i] * as_f<T>(u.o, row * d + i);
         return a.x != nullptr ? v + a.x[row * d + i] : v;
     };
     float * xo = (float *) tail.x_out;
@@ -416,6 +516,7 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
     for (int i = threadIdx.x; i < d; i += 256) {
         const float v = value(i);
         ss += v * v;
+        if (tail.norm_w == nullptr && tail.h_out != nullptr) put_f((T *) tail.h_out + (size_t) t * d + i, v);
         if (tail.norm_w == nullptr && xo != nullptr) xo[(size_t) t * d + i] = v;
     }
     if (tail.norm_w == nullptr) return;
@@ -423,6 +524,7 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
     for (int i = threadIdx.x; i < d; i += 256) {
         const float v = value(i);
         put_f((T *) tail.h_out + (size_t) t * d + i, v * ni * tail.norm_w[i]);
+        if (tail.norm2_w != nullptr) put_f((T *) tail.h2_out + (size_t) t * d + i, v * ni * tail.norm2_w[i]);
         if (xo != nullptr) xo[(size_t) t * d + i] = v;            // last: x_out may be x
     }
 }
@@ -469,6 +571,7 @@ inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAU
 
 inline bool tail_ok(const jib_row_tail * t, int d) {
     if (t == nullptr || t->x_out == nullptr || d > 16384) return false;
+    if (t->norm2_w != nullptr && (t->norm_w == nullptr || t->h2_out == nullptr || t->conv_w != nullptr)) return false;
     if (d % 8) return t->conv_w == nullptr && (t->norm_w == nullptr || t->h_out != nullptr);      // the element-wise kernel
     if (t->norm_w != nullptr && t->h_out == nullptr) return false;
     if (t->conv_w != nullptr)
@@ -566,6 +669,35 @@ JIB_EXPORT int jib_post_norm(const float * x, const void * y, const float * w, f
     do {                                                                                                                        \
         if (f32) JIB_LAUNCH((post_norm_kernel<float, NT, MAXV>), T, NT, 0, s, x, (const float *) y, w, eps, d, *tail, warm);    \
         else JIB_LAUNCH((post_norm_kernel<bf16, NT, MAXV>), T, NT, 0, s, x, (const bf16 *) y, w, eps, d, *tail, warm);          \
+    } while (0)
+    JIB_ROW_DISPATCH(d, CALL);
+#undef CALL
+    return launched();
+}
+
+JIB_EXPORT int jib_scaled_update(const float * x, const void * o, const float * s1, const void * y, const int * dest, const float * wts, int k,
+                                 const void * f, const float * f_gate, long long ld_gate, const float * s2, int T, int d, int f32,
+                                 const jib_row_tail * tail, void * stream) {
+    if (T <= 0) return 0;
+    jib_row_tail chk = *tail;
+    if (chk.x_out == nullptr) chk.x_out = (void *) x;
+    if (!tail_ok(&chk, d) || tail->conv_w != nullptr || (o != nullptr && s1 == nullptr) || ((y != nullptr || f != nullptr) && s2 == nullptr) ||
+        (y != nullptr && (dest == nullptr || wts == nullptr || k < 1 || k > MAX_TOP)))
+        return JIB_E_ARG;
+    ScaledArgs a;
+    a.x = x; a.o = o; a.y = y; a.f = f; a.s1 = s1; a.s2 = s2; a.dest = dest; a.wts = wts; a.f_gate = f_gate; a.ld_gate = ld_gate;
+    a.k = k; a.d = d;
+    cudaStream_t s = (cudaStream_t) stream;
+    if (d % 8) {
+        AnyRow r = {};
+        r.x = x; r.d = d; r.n_src = T; r.scale = 1.f; r.u = a;
+        return launch_any(r, *tail, T, f32, s);
+    }
+    const int warm = jib::warm_for(T);
+#define CALL(NT, MAXV)                                                                                    \
+    do {                                                                                                  \
+        if (f32) JIB_LAUNCH((scaled_update_kernel<float, NT, MAXV>), T, NT, 0, s, a, *tail, warm);        \
+        else JIB_LAUNCH((scaled_update_kernel<bf16, NT, MAXV>), T, NT, 0, s, a, *tail, warm);             \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
 #undef CALL

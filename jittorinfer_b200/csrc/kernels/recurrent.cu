@@ -35,7 +35,13 @@ __device__ __forceinline__ void store4(bf16 * p, const float (&v)[4]) {
     *(uint2 *) p = o;
 }
 
-// ---- out[t] = h[t] + sum_j w[j] * h[t - taps + 1 + j] --------------------------------------------------------------------
+// bf16 activations: fast exponential and division, a few ulp of fp32; fp32 ones: the accurate forms.
+template <typename T> __device__ __forceinline__ float sigmoid(float v);
+template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
+template <typename T> __device__ __forceinline__ float silu(float g) { return g * sigmoid<T>(g); }
+
+// ---- out[t] = h[t] + sum_j w[j] * h[t - taps + 1 + j], or silu(bias + sum_j w[j] * h[t - taps + 1 + j]) (ACT) ------------------
 // A CTA takes a run of CONV_RUN tokens of one sequence (runs are counted from the sequence's first token in the batch) and a slice
 // of the channels.  Up to CONV_TAPS taps only a sequence's first run reaches back to the stored rows: it loads every row once,
 // slides over them in registers and then, as their only reader, replaces the stored rows by the range's last ones.  Longer
@@ -47,34 +53,46 @@ static_assert(CONV_RUN >= CONV_TAPS - 1, "only the first run may reach back to t
 // every partial run before it; indices in the gaps have no tokens.
 __device__ __forceinline__ int run_key(const int * q_start, int b) { return q_start[b] / CONV_RUN + b; }
 
-template <typename T>
-__device__ __noinline__ void conv_run_long(const T * h, const float * w, int taps, T * st, bool past, bool keep, int q0, int n, int i0, int d,
-                                           int ch, T * out) {
+// what the filter's sum starts from, and what becomes of it
+template <bool ACT> __device__ __forceinline__ void conv_begin(const float (&x)[4], const float (&k)[4], const float (&b)[4], float (&c)[4]) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) c[e] = (ACT ? b[e] : x[e]) + k[e] * x[e];
+}
+template <typename T, bool ACT> __device__ __forceinline__ void conv_store(T * p, float (&c)[4]) {
+    if (ACT) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) c[e] = silu<T>(c[e]);
+    }
+    store4(p, c);
+}
+
+template <typename T, bool ACT>
+__device__ __noinline__ void conv_run_long(const T * h, long long ldh, const float * w, const float (&b)[4], int taps, T * st, bool past, bool keep,
+                                           int q0, int n, int i0, int d, int ch, T * out) {
     const int n_old = taps - 1;
     for (int i = i0; i < min(n, i0 + CONV_RUN); ++i) {
         if (i > 0 && i < n_old) continue;
         for (int r = i; r < (i == 0 ? min(n, max(n_old, 1)) : i + 1); ++r) {
             float x[4], k[4], c[4];
-            load4(h + (size_t) (q0 + r) * d + ch, x);
+            load4(h + (size_t) (q0 + r) * ldh + ch, x);
             load4(w + (size_t) n_old * d + ch, k);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) c[e] = x[e] + k[e] * x[e];
+            conv_begin<ACT>(x, k, b, c);
             for (int j = 0; j < n_old; ++j) {
                 const int src = r - n_old + j;
-                if (src >= 0) load4(h + (size_t) (q0 + src) * d + ch, x);
+                if (src >= 0) load4(h + (size_t) (q0 + src) * ldh + ch, x);
                 else if (past) load4(st + (size_t) (src + n_old) * d, x);
                 else continue;
                 load4(w + (size_t) j * d + ch, k);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) c[e] += k[e] * x[e];
             }
-            store4(out + (size_t) (q0 + r) * d + ch, c);
+            conv_store<T, ACT>(out + (size_t) (q0 + r) * d + ch, c);
         }
         if (i == 0 && keep) {
             for (int j = 0; j < n_old; ++j) {              // ascending: entry j only needs old entries behind it
                 const int src = n - n_old + j;
                 float x[4] = {0.f, 0.f, 0.f, 0.f};
-                if (src >= 0) load4(h + (size_t) (q0 + src) * d + ch, x);
+                if (src >= 0) load4(h + (size_t) (q0 + src) * ldh + ch, x);
                 else if (past) load4(st + (size_t) (src + n_old) * d, x);
                 store4(st + (size_t) j * d, x);
             }
@@ -82,9 +100,9 @@ __device__ __noinline__ void conv_run_long(const T * h, const float * w, int tap
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restrict__ h, const float * __restrict__ w, int taps,
-                                                              T * __restrict__ state, int n_state, const int * __restrict__ seq_slots,
+template <typename T, bool ACT>
+__global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restrict__ h, long long ldh, const float * __restrict__ w,
+                                                              const float * __restrict__ bias, int taps, T * __restrict__ state, int n_state, const int * __restrict__ seq_slots,
                                                               const int * __restrict__ positions, const int * __restrict__ q_start,
                                                               int n_seqs, int d, T * __restrict__ out, int * status) {
     PDL_TRIGGER_TOP();
@@ -109,20 +127,22 @@ __global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restri
         past = slot >= 0 && positions[q0] > 0;
     }
     T * st = state + (size_t) (slot < 0 ? 0 : slot) * n_old * d + ch;
+    float b4[4] = {0.f, 0.f, 0.f, 0.f};
+    if (ACT) load4(bias + ch, b4);
     if (taps > CONV_TAPS) {
-        conv_run_long(h, w, taps, st, past, slot >= 0, q0, n, i0, d, ch, out);
+        conv_run_long<T, ACT>(h, ldh, w, b4, taps, st, past, slot >= 0, q0, n, i0, d, ch, out);
         return;
     }
     // rows i0 - (CONV_TAPS - 1) .. i0 + CONV_RUN - 1 in x; taps right-aligned in k; the range's last rows for the stored ones in z
     float x[CONV_RUN + CONV_TAPS - 1][4], k[CONV_TAPS][4], z[CONV_TAPS - 1][4];
-    const T * hb = h + (size_t) q0 * d + ch;
+    const T * hb = h + (size_t) q0 * ldh + ch;
 #pragma unroll
     for (int r = 0; r < CONV_RUN + CONV_TAPS - 1; ++r) {
         const int i = i0 + r - (CONV_TAPS - 1);
 #pragma unroll
         for (int e = 0; e < 4; ++e) x[r][e] = 0.f;
         if (r >= CONV_TAPS - taps && i < n) {
-            if (i >= 0) load4(hb + (size_t) i * d, x[r]);
+            if (i >= 0) load4(hb + (size_t) i * ldh, x[r]);
             else if (past) load4(st + (size_t) (i + n_old) * d, x[r]);
         }
     }
@@ -136,7 +156,7 @@ __global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restri
 #pragma unroll
             for (int e = 0; e < 4; ++e) z[j][e] = 0.f;
             if (j < n_old) {
-                if (i >= 0) load4(hb + (size_t) i * d, z[j]);
+                if (i >= 0) load4(hb + (size_t) i * ldh, z[j]);
                 else if (past) load4(st + (size_t) (i + n_old) * d, z[j]);
             }
         }
@@ -145,14 +165,13 @@ __global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restri
     for (int r = 0; r < CONV_RUN; ++r) {
         if (i0 + r >= n) break;
         float c[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) c[e] = x[r + CONV_TAPS - 1][e] + k[CONV_TAPS - 1][e] * x[r + CONV_TAPS - 1][e];
+        conv_begin<ACT>(x[r + CONV_TAPS - 1], k[CONV_TAPS - 1], b4, c);
 #pragma unroll
         for (int j = 0; j < CONV_TAPS - 1; ++j)
             if (j >= CONV_TAPS - taps)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) c[e] += k[j][e] * x[r + j][e];
-        store4(out + (size_t) (q0 + i0 + r) * d + ch, c);
+        conv_store<T, ACT>(out + (size_t) (q0 + i0 + r) * d + ch, c);
     }
     if (slot >= 0) {
 #pragma unroll
@@ -163,16 +182,11 @@ __global__ void __launch_bounds__(CONV_NT) causal_conv_kernel(const T * __restri
 
 // ---- minGRU: S_t = (1 - z_t) S_(t-1) + z_t c_t,  y_t = S_t * silu(g_t) -------------------------------------------------------
 // zxg [T][ld]: pre-activations of z, of the candidate and of the output gate, W columns each.  All arithmetic fp32.
-// (bf16 activations: fast exponential and division, a few ulp of fp32; fp32 ones: the accurate forms)
-template <typename T> __device__ __forceinline__ float sigmoid(float v);
-template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
-template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
 template <typename T> __device__ __forceinline__ void gru_terms(float az, float au, float & a, float & b) {
     const float z = sigmoid<T>(az), c = sigmoid<T>(au);
     a = 1.f - z;
     b = z * (au >= 0.f ? au + 0.5f : c);
 }
-template <typename T> __device__ __forceinline__ float silu(float g) { return g * sigmoid<T>(g); }
 // Two adjacent elements at p.  PAIR: one access; else two, the second at p + step (0 at the last channel: no branch around a load,
 // so that a round's loads are all in flight together).
 template <bool PAIR> __device__ __forceinline__ float2 load2(const bf16 * p, int step) {
@@ -376,19 +390,24 @@ inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAU
 
 extern "C" {
 
-JIB_EXPORT int jib_causal_conv(const void * h, const float * w, int taps, void * state, int n_state, const int * seq_slots,
-                               const int * positions, const int * q_start, int n_seqs, int T, int d, int f32, void * out, int * status,
-                               void * stream) {
+JIB_EXPORT int jib_causal_conv(const void * h, long long ldh, const float * w, const float * bias, int silu, int taps, void * state, int n_state,
+                               const int * seq_slots, const int * positions, const int * q_start, int n_seqs, int T, int d, int f32, void * out,
+                               int * status, void * stream) {
     if (T <= 0 || n_seqs <= 0) return 0;
-    if (d % 4 || taps < 1 || (taps > 1 && state == nullptr)) return JIB_E_ARG;
+    if (d % 4 || ldh % 4 || taps < 1 || (taps > 1 && state == nullptr) || (silu && bias == nullptr)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
     const dim3 grid(T / CONV_RUN + n_seqs, (d / 4 + CONV_NT - 1) / CONV_NT);
-    if (f32)
-        JIB_LAUNCH((causal_conv_kernel<float>), grid, CONV_NT, 0, s, (const float *) h, w, taps, (float *) state, n_state, seq_slots, positions,
-                   q_start, n_seqs, d, (float *) out, status);
-    else
-        JIB_LAUNCH((causal_conv_kernel<bf16>), grid, CONV_NT, 0, s, (const bf16 *) h, w, taps, (bf16 *) state, n_state, seq_slots, positions,
-                   q_start, n_seqs, d, (bf16 *) out, status);
+#define CALL(TT, ACT)                                                                                                                       \
+    JIB_LAUNCH((causal_conv_kernel<TT, ACT>), grid, CONV_NT, 0, s, (const TT *) h, ldh, w, bias, taps, (TT *) state, n_state, seq_slots, positions, \
+               q_start, n_seqs, d, (TT *) out, status)
+    if (f32) {
+        if (silu) CALL(float, true);
+        else CALL(float, false);
+    } else {
+        if (silu) CALL(bf16, true);
+        else CALL(bf16, false);
+    }
+#undef CALL
     return launched();
 }
 

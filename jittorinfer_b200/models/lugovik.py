@@ -32,28 +32,13 @@ from .. import ops
 from ..ops.specs import Gqa, StateMix
 from ..utils import trace as _trace
 from .deepseek2 import ForwardBatch
+from .folder import Rotation, Yarn, block_diagonal, checked_tensors, fits, rope_table, stack_rows, up
 from .weights import ShardSpec, _stream_seed
 
 ARCH = "Lugovik"
-ALIGN = 8                          # columns: 16 bytes of bf16
 
 
 # ---- configuration -----------------------------------------------------------------------------------------------------------
-@dataclass(frozen=True)
-class Yarn:
-    factor: float
-    original: float
-    fast: float
-    slow: float
-
-
-@dataclass(frozen=True)
-class Rotation:
-    dims: int
-    base: float
-    yarn: Optional[Yarn] = None
-
-
 @dataclass(frozen=True)
 class Mamba2Mixer:
     heads: int
@@ -264,10 +249,6 @@ def _concrete(hp: LugovikHParams) -> Dict[str, Tuple[int, ...]]:
     return {k: tuple(hp.random_rank if n is None else n for n in s) for k, s in tensor_table(hp).items()}
 
 
-def _fits(shape: Sequence[int], want: Sequence[Optional[int]]) -> bool:
-    return len(shape) == len(want) and all(w is None or s == w for s, w in zip(shape, want))
-
-
 def _unused(hp: LugovikHParams, name: str) -> bool:
     """Norms of a feed-forward the layer does not have."""
     layer, _, k = name.partition(".")
@@ -276,24 +257,7 @@ def _unused(hp: LugovikHParams, name: str) -> bool:
 
 def iter_checkpoint(directory: str, hp: LugovikHParams) -> Iterator[Tuple[str, torch.Tensor]]:
     """(name, CPU tensor) of every tensor of the model from the folder's safetensors file(s); checks names and shapes."""
-    from ..gguf.convert_hf import Checkpoint
-    ck = Checkpoint(directory)
-    try:
-        table = tensor_table(hp)
-        have = set(ck.names())
-        missing = [n for n in table if n not in have]
-        if missing:
-            raise KeyError(f"checkpoint is missing {len(missing)} tensors, e.g. {missing[:3]}")
-        extra = sorted(n for n in have - set(table) if not _unused(hp, n))
-        if extra:
-            raise ValueError(f"checkpoint has {len(extra)} tensors the model does not use, e.g. {extra[:3]}")
-        for name, shape in table.items():
-            t = ck.get(name)
-            if not _fits(t.shape, shape):
-                raise ValueError(f"{name}: shape {tuple(t.shape)} != expected {shape}")
-            yield name, t
-    finally:
-        ck.close()
+    return checked_tensors(directory, tensor_table(hp), lambda n: _unused(hp, n))
 
 
 def iter_random(hp: LugovikHParams, seed: int = 0, dtype: torch.dtype = torch.float32, device="cpu") -> Iterator[Tuple[str, torch.Tensor]]:
@@ -311,48 +275,6 @@ def iter_random(hp: LugovikHParams, seed: int = 0, dtype: torch.dtype = torch.fl
 def load_config(directory: str) -> LugovikHParams:
     with open(os.path.join(directory, "config.json")) as f:
         return LugovikHParams.from_config(json.load(f))
-
-
-def rope_table(n_pos: int, rot: Rotation, device) -> torch.Tensor:
-    """[n_pos, dims / 2, 2] fp32 (cos, sin), with YaRN's blend of stretched and plain frequencies and its magnitude factor."""
-    i = torch.arange(rot.dims // 2, dtype=torch.float64)
-    f, mult = rot.base ** (-2.0 * i / rot.dims), 1.0
-    if rot.yarn is not None:
-        y = rot.yarn
-        at = lambda turns: rot.dims * math.log(y.original / (2 * math.pi * turns)) / (2 * math.log(rot.base))       # noqa: E731
-        lo, hi = max(math.floor(at(y.fast)), 0), min(math.ceil(at(y.slow)), rot.dims - 1)
-        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-        f, mult = f / y.factor * ramp + f * (1 - ramp), 0.1 * math.log(y.factor) + 1
-    a = torch.arange(n_pos, dtype=torch.float64)[:, None] * f
-    return torch.stack([torch.cos(a) * mult, torch.sin(a) * mult], -1).float().contiguous().to(device)
-
-
-def _up(n: int) -> int:
-    return (n + ALIGN - 1) // ALIGN * ALIGN
-
-
-def stack_rows(parts: Sequence[Tuple[str, torch.Tensor]]) -> Tuple[torch.Tensor, Dict[str, int]]:
-    """Matrices of equal width over one another, each starting at a multiple of 8 rows (zero rows between); (matrix, first row of each)."""
-    off, n = {}, 0
-    for k, w in parts:
-        off[k] = n
-        n += _up(w.shape[0])
-    out = torch.zeros(n, parts[0][1].shape[1], dtype=parts[0][1].dtype, device=parts[0][1].device)
-    for k, w in parts:
-        out[off[k]:off[k] + w.shape[0]] = w
-    return out, off
-
-
-def block_diagonal(parts: Sequence[torch.Tensor]) -> Tuple[torch.Tensor, List[int]]:
-    """Matrices along the diagonal of one, rows and columns of each starting at multiples of 8; (matrix, first row of each)."""
-    rows, cols = [0], [0]
-    for w in parts:
-        rows.append(rows[-1] + _up(w.shape[0]))
-        cols.append(cols[-1] + _up(w.shape[1]))
-    out = torch.zeros(rows[-1], cols[-1], dtype=parts[0].dtype, device=parts[0].device)
-    for w, r, c in zip(parts, rows, cols):
-        out[r:r + w.shape[0], c:c + w.shape[1]] = w
-    return out, rows[:-1]
 
 
 class _Layer:
@@ -398,7 +320,7 @@ class LugovikModel:
                 if _unused(hp, name):
                     continue
                 raise KeyError(f"unknown tensor {name}")
-            if not _fits(t.shape, table[name]):
+            if not fits(t.shape, table[name]):
                 raise ValueError(f"{name}: shape {tuple(t.shape)} != expected {table[name]}")
             seen.add(name)
             small = t.dim() == 1 or name.endswith(".conv")
@@ -450,7 +372,7 @@ class LugovikModel:
                                    [("r" + k, take("mix.right." + k)) for k in ("q", "k", "v", "g")] + [("a1", a1)])
             L.w_low, _ = block_diagonal([a2])
             wl, wr = take("mix.left.o"), take("mix.right.o")
-            nl = _up(wl.shape[1])                             # the right half's first column
+            nl = up(wl.shape[1])                             # the right half's first column
             L.w_o = torch.zeros(wl.shape[0], nl + wr.shape[1], dtype=wl.dtype, device=wl.device)
             L.w_o[:, :wl.shape[1]], L.w_o[:, nl:] = wl, wr
             c["y"] = nl

@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Any, Callable, Dict, Optional
 
-from . import lugovik, nibalix
+from . import lugovik, nibalix, zomavik
 from .deepseek2 import DeepSeek2Model
 from .hparams import ARCH as DEEPSEEK2, DeepSeek2HParams
 from .hparams import preset as _deepseek2_preset
@@ -35,6 +35,8 @@ ARCHITECTURES: Dict[str, Architecture] = {
                                nibalix.iter_checkpoint, nibalix.iter_random),
     lugovik.ARCH: Architecture(lugovik.ARCH, lugovik.LugovikHParams, lugovik.LugovikModel, lugovik.preset, lugovik.load_config,
                                lugovik.iter_checkpoint, lugovik.iter_random),
+    zomavik.ARCH: Architecture(zomavik.ARCH, zomavik.ZomavikHParams, zomavik.ZomavikModel, zomavik.preset, zomavik.load_config,
+                               zomavik.iter_checkpoint, zomavik.iter_random),
 }
 
 

@@ -56,10 +56,11 @@ def rmsnorm(x, w, eps, residual=None):
     return nat().rmsnorm(x, w, eps, residual) if use_native(x) else ref.rmsnorm(x, w, eps, residual)
 
 
-def linear(x, w, residual=None, out_dtype=None):
+def linear(x, w, residual=None, out_dtype=None, unary=None):
+    """f(x w^T) + residual (a bias: one row expanded over the tokens); ``unary``: None, ("relu2",) or ("cap", scale, softcap)."""
     if use_native(x) and x.dtype == torch.bfloat16:
-        return nat().linear(x, w, residual, out_dtype)
-    return ref.linear(x, w, residual, out_dtype)
+        return nat().linear(x, w, residual, out_dtype, unary)
+    return ref.linear(x, w, residual, out_dtype, unary)
 
 
 def gateup_silu(x, wg, wu):
@@ -95,17 +96,19 @@ def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_siz
 
 
 def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None, pre_norm=None,
-             logit_bias=None):
-    """``route=(expert_base, E_local)`` tells the CUDA path which local expert sort follows (see ``native.moe_gate``).
+             logit_bias=None, shared_gate=False):
+    """``shared_gate``: the last row of ``w_router`` is the shared experts' gate, not an expert: their weight is its sigmoid (``n_shared``
+    columns), and the router outputs' last column is returned as well.
+    ``route=(expert_base, E_local)`` tells the CUDA path which local expert sort follows (see ``native.moe_gate``).
     ``pre_norm=(weight, eps)``: ``g`` is the un-normalised block input; returns (ids, wts, rmsnorm(g) * weight) -- on the CUDA
     path the router launch of a decode batch normalises the rows itself."""
     if use_native(g):
         return nat().moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, route, pre_norm,
-                              logit_bias)
+                              logit_bias, shared_gate)
     if pre_norm is not None:
         g, _ = ref.rmsnorm(g, pre_norm[0], pre_norm[1])
         return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2) + (g,)
-    return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, logit_bias)
+    return ref.moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared, group_top2, logit_bias, shared_gate)
 
 
 def moe_routed(x, ids, wts, wg, wu, wd):
@@ -136,7 +139,8 @@ def fused_combine_norm() -> bool:
 
 # ---- parallel blocks over an fp32 residual stream, per-sequence state -------------------------------------------------------------
 # ``nxt`` = (norm weight, eps, conv): the norm the next block reads, computed in the same pass; conv = None, or -- one token per
-# sequence only -- (weights [taps, d], state, seq_slots, positions) of that block's input convolution.
+# sequence only -- (weights [taps, d], state, seq_slots, positions) of that block's input convolution.  Or a ``specs.RowNorms``: one or
+# two norms of the row, or the row in the activation type; the second comes back in the place of h + convolution.
 def embed_norm(table, ids, w, eps, nxt=None, scale=1.0):
     """(x fp32 = norm of the scaled embedding rows (``w`` None: the rows themselves), h, h + convolution)."""
     return (nat() if use_native(table) else ref).embed_norm(table, ids, w, eps, nxt, scale)
@@ -152,12 +156,20 @@ def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
     return (nat() if use_native(x) else ref).block_update(x, mult, o, gates, b1, b2, moe, nxt)
 
 
+def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=None, dtype=None):
+    """(x + s1 * o + s2 * (combine(moe) + sigmoid(dense_gate) * dense), h, h2); ``o``, ``moe`` = (rows, row of each pair, weights) and
+    ``dense`` may be None, ``dense_gate`` [T] None is a factor of one; ``dtype``: activation type (default: that of the sublayers' rows); x may be
+    overwritten."""
+    return (nat() if use_native(x) else ref).scaled_update(x, o, s1, s2, moe, dense, dense_gate, nxt, dtype)
+
+
 def rms_rows(x, rows, w, eps, dtype):
     return (nat() if use_native(x) else ref).rms_rows(x, rows, w, eps, dtype)
 
 
-def causal_conv(h, w, state, seq_slots, positions, q_start):
-    return (nat() if use_native(h) else ref).causal_conv(h, w, state, seq_slots, positions, q_start)
+def causal_conv(h, w, state, seq_slots, positions, q_start, bias=None):
+    """h + convolution, or with ``bias`` silu(convolution + bias); h may be a slice of columns."""
+    return (nat() if use_native(h) else ref).causal_conv(h, w, state, seq_slots, positions, q_start, bias)
 
 
 def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
@@ -168,6 +180,11 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
     """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view)."""
     return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out)
+
+
+def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
+    """``m``: ``specs.SelectiveScan``; ``bc`` = B | C, ``dt`` fp32 pre-activations of the step sizes; result columns go to ``out`` (a view)."""
+    return (nat() if use_native(x) else ref).selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out)
 
 
 def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):

@@ -12,6 +12,8 @@ from typing import Dict, Optional
 
 import torch
 
+from .specs import RowNorms
+
 _lib = None
 _ws: Dict[int, "Workspace"] = {}
 launch_count = 0            # kernels launched through this module (bench.py reports it)
@@ -49,6 +51,7 @@ ERRORS = {-1: "unsupported shape/argument", -2: "pointer or stride not 16-byte a
 
 
 ACTS = {"silu": 0, "gelu_tanh": 1}     # activation of a gated pair (JIB_ACT_*)
+UNARIES = {"relu2": 1, "cap": 2}       # function of a single product (JIB_UNARY_*)
 
 
 class GemmDesc(C.Structure):
@@ -62,12 +65,13 @@ class GemmDesc(C.Structure):
                                                                              ("ag_world", C.c_int), ("ar_rs_rows", C.c_int),
                                                                              ("src_token", C.c_void_p), ("src_rows", C.c_int), ("expert_list", C.c_void_p),
                                                                              ("n_slots", C.c_int), ("list_tiles", C.c_int), ("pdl_flags", C.c_int),
-                                                                             ("act", C.c_int)]
+                                                                             ("act", C.c_int), ("unary", C.c_int), ("scale", C.c_float),
+                                                                             ("softcap", C.c_float)]
 
 
 class RowTail(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x_out", "norm_w", "h_out", "conv_w", "hc_out", "conv_state", "seq_slots", "positions", "status")] + \
-               [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int)]
+               [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int), ("norm2_w", C.c_void_p), ("h2_out", C.c_void_p)]
 
 
 class StateMixDesc(C.Structure):
@@ -83,7 +87,13 @@ class GqaDesc(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("cache", "block_tables", "seq_lens", "q_start", "positions", "status")] + \
                [(n, C.c_longlong) for n in ("n_slots", "row")] + \
                [(n, C.c_int) for n in ("H", "G", "D", "V", "rot", "block_size", "max_blocks", "n_seqs", "T", "max_pos", "window", "chunk", "sink")] + \
-               [(n, C.c_float) for n in ("scale", "softcap", "eps", "out_scale")]
+               [(n, C.c_float) for n in ("scale", "softcap", "eps", "out_scale")] + [("sink_w", C.c_void_p)]
+
+
+class ScanDesc(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("x", "z", "bc", "dt", "y", "neg_a", "skip", "state", "seq_slots", "positions", "q_start", "status")] + \
+               [(n, C.c_longlong) for n in ("ldx", "ldz", "ldbc", "lddt", "ldy")] + \
+               [(n, C.c_int) for n in ("ch", "N", "n_state", "n_seqs", "T")] + [("out_scale", C.c_float)]
 
 
 def load():
@@ -108,7 +118,9 @@ def load():
     sig("jib_post_norm", fp, vp, fp, f, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_block_update", fp, f, vp, vp, ll, fp, fp, vp, ip, fp, i, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, vp, vp)
-    sig("jib_causal_conv", vp, fp, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
+    sig("jib_scaled_update", fp, vp, fp, vp, ip, fp, i, vp, fp, ll, fp, i, i, i, C.POINTER(RowTail), vp)
+    sig("jib_causal_conv", vp, ll, fp, fp, i, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
+    sig("jib_selective_scan", C.POINTER(ScanDesc), i, i, vp)
     sig("jib_mingru", vp, ll, fp, fp, fp, i, ip, ip, ip, i, i, i, i, i, vp, ip, vp)
     L.jib_state_chunk_bytes.restype, L.jib_state_chunk_bytes.argtypes = C.c_longlong, [C.POINTER(StateMixDesc)]
     sig("jib_state_mix_run", C.POINTER(StateMixDesc), i, i, vp)
@@ -125,7 +137,7 @@ def load():
     sig("jib_sample_topk", fp, ip, fp, ip, i, i, vp)
     sig("jib_kv_block_copy", vp, ll, i, ip, ip, i, i, vp)
     sig("jib_gather_rows", vp, ip, vp, i, i, i, vp)
-    sig("jib_moe_gate", vp, fp, fp, fp, fp, ip, fp, i, i, i, i, i, i, f, i, i, i, i, vp)
+    sig("jib_moe_gate", vp, fp, fp, fp, fp, ip, fp, i, i, i, i, i, i, f, i, i, i, i, i, vp)
     sig("jib_moe_permute", ip, i, i, i, i, ip, ip, ip, vp)
     sig("jib_moe_route_fused", vp, fp, fp, fp, ip, fp, ip, ip, ip, ip, i, i, i, i, i, i, f, i, i, i, i, i, i, fp, f, vp, vp)
     sig("jib_moe_permute_multi", ip, i, i, i, i, ip, ip, ip, ip, vp)
@@ -227,8 +239,8 @@ def _gemm_simt(d: GemmDesc, f32: bool, what: str) -> None:
 
 def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *, out: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, splits: int = 0, bn: int = 0,
-         ar=None, ar_site: int = 0, ar_rs_rows: int = 0, ag=None, act: str = "silu") -> torch.Tensor:
-    """out[T,N] = x[T,K] @ w[N,K]^T  (w2: act(x w^T) * (x w2^T)) (+ residual)."""
+         ar=None, ar_site: int = 0, ar_rs_rows: int = 0, ag=None, act: str = "silu", unary=None) -> torch.Tensor:
+    """out[T,N] = f(x[T,K] @ w[N,K]^T)  (w2: act(x w^T) * (x w2^T)) (+ residual; row stride 0: a bias); ``unary``: see ``ops.linear``."""
     assert x.dtype == w.dtype and x.dtype in (torch.bfloat16, torch.float32) and x.stride(-1) == 1 and w.is_contiguous()
     T, K = x.shape
     N = w.shape[0]
@@ -249,6 +261,9 @@ def gemm(x: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor] = None, *,
     d.out_f32 = int(out.dtype == torch.float32)
     d.res_f32 = int(residual is not None and residual.dtype == torch.float32)
     d.splits, d.bn, d.sm_count, d.act = splits, bn, ws.sm_count, ACTS[act]
+    if unary is not None:
+        d.unary = UNARIES[unary[0]]
+        d.scale, d.softcap = (float(unary[1]), float(unary[2])) if unary[0] == "cap" else (1.0, 0.0)
     if ar is not None:          # fused all-reduce (or, with ar_rs_rows, reduce-scatter by rows) over peer memory in the epilogue
         d.ar, d.ar_site, d.ar_rs_rows = C.addressof(ar), ar_site, ar_rs_rows
     if ag is not None:          # x is a gather buffer other ranks are still filling: (flags ptr, epoch ptr, rows per rank, world)
@@ -337,8 +352,8 @@ def gemm_grouped(xp: torch.Tensor, seg: torch.Tensor, w: torch.Tensor, w2: Optio
                             pdl_flags=pdl_flags, n_slots=n_slots, tile_list=tile_list)
 
 
-def linear(x, w, residual=None, out_dtype=None):
-    return gemm(x, w, residual=residual, out_dtype=out_dtype)
+def linear(x, w, residual=None, out_dtype=None, unary=None):
+    return gemm(x, w, residual=residual, out_dtype=out_dtype, unary=unary)
 
 
 def grouped_tma_ok(x: torch.Tensor, wg: torch.Tensor) -> bool:
@@ -521,13 +536,13 @@ def mha_prefill(q, cache, w_kv_b, block_tables, seq_lens, q_start, scale, n_head
 
 # ---- MoE -----------------------------------------------------------------------------------------
 def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None,
-             pre_norm=None, logit_bias=None):
+             pre_norm=None, logit_bias=None, shared_gate=False):
     """``route=(expert_base, E_local)``: the caller will sort these ids by local expert next (``moe_permute``); for decode
     batches both steps then run as one launch and ``moe_permute`` picks the result up.
     ``pre_norm=(weight, eps)``: ``g`` holds un-normalised rows; returns (ids, wts, rmsnorm(g) * weight), the norm done by
     the router launch itself for decode batches."""
     T, d = g.shape
-    fused = FUSED_ROUTE and route is not None and T <= FUSED_ROUTE_MAX_T and logit_bias is None and g.dtype == torch.bfloat16
+    fused = FUSED_ROUTE and route is not None and T <= FUSED_ROUTE_MAX_T and logit_bias is None and not shared_gate and g.dtype == torch.bfloat16
     g_in = g
     g_pre = None
     if pre_norm is not None and not (fused and ROUTE_NORM):
@@ -539,6 +554,7 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
     ids = torch.empty(T, k + n_shared, dtype=torch.int32, device=g.device)
     wts = torch.empty(T, k + n_shared, dtype=torch.float32, device=g.device)
     logits = torch.empty(T, E, dtype=torch.float32, device=g.device)
+    E -= int(shared_gate)
     if fused:
         expert_base, E_local = route
         n = T * (k + n_shared)
@@ -555,11 +571,13 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
         _route_stash.clear()                       # at most one pending result: the sort that follows this gate
         _route_stash[(ids.data_ptr(), expert_base, E_local)] = (seg, src, dest, ids)
         return (ids, wts, g_out if g_out is not None else g_pre) if pre_norm is not None else (ids, wts)
-    if g.dtype == torch.float32:
-        torch.matmul(g, w_router.T, out=logits)
-    _ck(load().jib_moe_gate(g.data_ptr() if g.dtype == torch.bfloat16 else None, w_router.data_ptr(), _p(bias), _p(logit_bias), logits.data_ptr(), ids.data_ptr(), wts.data_ptr(), T, d,
-                            E, k, n_group, topk_group, float(scale), int(norm), int(sigmoid), n_shared, int(group_top2), _stream()), "moe_gate")
-    return (ids, wts, g) if pre_norm is not None else (ids, wts)
+    own = g.dtype == torch.bfloat16 and d % 8 == 0 and d <= 8192          # the router kernel; else fp32 products of the library
+    if not own:
+        torch.matmul(g.float(), w_router.T, out=logits)
+    _ck(load().jib_moe_gate(g.data_ptr() if own else None, w_router.data_ptr(), _p(bias), _p(logit_bias), logits.data_ptr(), ids.data_ptr(), wts.data_ptr(), T, d,
+                            E, k, n_group, topk_group, float(scale), int(norm), int(sigmoid), n_shared, int(group_top2), int(shared_gate), _stream()),
+        "moe_gate")
+    return (ids, wts) + ((g,) if pre_norm is not None else ()) + ((logits[:, E],) if shared_gate else ())
 
 
 def moe_permute(ids, expert_base, E_local):
@@ -676,10 +694,16 @@ def moe_ffn(x, residual, ids, wts, wg, wu, wd, wgs, wus, wds, expert_base=0, n_e
 
 # ---- parallel blocks over an fp32 residual (parallel_block.cu), per-sequence state (recurrent.cu) ------------------------------
 def _row_tail(x_out, nxt, dtype):
-    """(RowTail, h, hc) for ``nxt`` = (norm weight, eps, conv), see ``ops.embed_norm``."""
+    """(RowTail, h, hc) for ``nxt`` = (norm weight, eps, conv) or a ``RowNorms``, see ``ops.embed_norm``."""
     t, h, hc = RowTail(), None, None
     t.x_out, t.status = x_out.data_ptr(), workspace(x_out.device).status.data_ptr()
-    if nxt is not None:
+    if isinstance(nxt, RowNorms):
+        h = torch.empty(x_out.shape, dtype=dtype, device=x_out.device)
+        t.h_out, t.norm_w, t.eps = h.data_ptr(), _p(nxt.w1), float(nxt.eps)
+        if nxt.w2 is not None:
+            hc = torch.empty_like(h)
+            t.norm2_w, t.h2_out = nxt.w2.data_ptr(), hc.data_ptr()
+    elif nxt is not None:
         w, eps, conv = nxt
         h = torch.empty(x_out.shape, dtype=dtype, device=x_out.device)
         t.norm_w, t.eps, t.h_out = w.data_ptr(), float(eps), h.data_ptr()
@@ -721,6 +745,20 @@ def post_norm(x, y, w, eps, nxt=None):
     return x, h
 
 
+def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=None, dtype=None):
+    T, d = x.shape
+    y, dest, wts = moe if moe is not None else (None, None, None)
+    dtype = dtype or next((t.dtype for t in (o, dense, y) if t is not None), x.dtype)
+    for t in (o, y, dense):
+        assert t is None or (t.dtype == dtype and t.is_contiguous())
+    assert x.dtype == torch.float32 and x.is_contiguous() and (dense_gate is None or dense_gate.dtype == torch.float32)
+    tail, h, h2 = _row_tail(x, nxt, dtype)
+    _ck(load().jib_scaled_update(x.data_ptr(), _p(o), _p(s1), _p(y), _p(dest), _p(wts), dest.shape[1] if dest is not None else 0, _p(dense),
+                                 _p(dense_gate), dense_gate.stride(0) if dense_gate is not None else 0, _p(s2), T, d, int(dtype == torch.float32),
+                                 C.byref(tail), _stream()), "scaled_update")
+    return x, h, h2
+
+
 def rms_rows(x, rows, w, eps, dtype):
     n, d = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
     out = torch.empty(n, d, dtype=dtype, device=x.device)
@@ -729,11 +767,11 @@ def rms_rows(x, rows, w, eps, dtype):
     return out
 
 
-def causal_conv(h, w, state, seq_slots, positions, q_start):
+def causal_conv(h, w, state, seq_slots, positions, q_start, bias=None):
     T, d = h.shape
-    assert w.dtype == torch.float32 and w.is_contiguous() and h.is_contiguous() and state.dtype == h.dtype and state.is_contiguous()
-    out = torch.empty_like(h)
-    _ck(load().jib_causal_conv(h.data_ptr(), w.data_ptr(), w.shape[0], state.data_ptr(), state.shape[0], seq_slots.data_ptr(),
+    assert w.dtype == torch.float32 and w.is_contiguous() and h.stride(1) == 1 and state.dtype == h.dtype and state.is_contiguous()
+    out = torch.empty(T, d, dtype=h.dtype, device=h.device)
+    _ck(load().jib_causal_conv(h.data_ptr(), h.stride(0), w.data_ptr(), _p(bias), int(bias is not None), w.shape[0], state.data_ptr(), state.shape[0], seq_slots.data_ptr(),
                                positions.data_ptr(), q_start.data_ptr(), q_start.shape[0] - 1, T, d, int(h.dtype == torch.float32),
                                out.data_ptr(), workspace(h.device).status.data_ptr(), _stream()), "causal_conv")
     return out
@@ -792,6 +830,21 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     return out
 
 
+def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
+    T = x.shape[0]
+    assert x.dtype == z.dtype == bc.dtype == out.dtype and dt.dtype == state.dtype == torch.float32 and state.is_contiguous()
+    assert x.stride(1) == z.stride(1) == bc.stride(1) == dt.stride(1) == out.stride(1) == 1 and m.neg_a.is_contiguous()
+    cd = ScanDesc()
+    for name, t in (("x", x), ("z", z), ("bc", bc), ("dt", dt), ("y", out)):
+        setattr(cd, name, t.data_ptr())
+        setattr(cd, "ld" + name, t.stride(0))
+    cd.neg_a, cd.skip, cd.state, cd.status = m.neg_a.data_ptr(), m.skip.data_ptr(), state.data_ptr(), workspace(x.device).status.data_ptr()
+    cd.seq_slots, cd.positions, cd.q_start = seq_slots.data_ptr(), positions.data_ptr(), q_start.data_ptr()
+    cd.ch, cd.N, cd.n_state, cd.n_seqs, cd.T, cd.out_scale = m.channels, m.state, state.shape[0], q_start.shape[0] - 1, T, m.out_scale
+    _ck(load().jib_selective_scan(C.byref(cd), int(single), int(x.dtype == torch.float32), _stream()), "selective_scan")
+    return out
+
+
 def _gqa_desc(m, cache, T, n_seqs):
     assert cache.is_contiguous()
     gd = GqaDesc()
@@ -799,6 +852,7 @@ def _gqa_desc(m, cache, T, n_seqs):
     gd.H, gd.G, gd.D, gd.V, gd.rot, gd.T, gd.n_seqs, gd.block_size = m.heads, m.kv_heads, m.dim, m.vdim, m.rot, T, n_seqs, 64
     gd.window, gd.chunk, gd.sink = m.window, m.chunk, int(m.sink)
     gd.scale, gd.softcap, gd.eps, gd.out_scale = m.scale, m.softcap, m.eps, m.out_scale
+    gd.sink_w = _p(m.sink_w)
     return gd
 
 
@@ -808,7 +862,7 @@ def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
     out = torch.empty(T, m.heads, m.dim, dtype=q.dtype, device=q.device)
     gd = _gqa_desc(m, cache, T, 1)
     gd.positions, gd.max_pos = positions.data_ptr(), rope_table.shape[0]
-    _ck(load().jib_gqa_qkv_post(C.byref(gd), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), m.q_norm.data_ptr(), m.k_norm.data_ptr(),
+    _ck(load().jib_gqa_qkv_post(C.byref(gd), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _p(m.q_norm), _p(m.k_norm),
                                 rope_table.data_ptr(), slot_mapping.data_ptr(), out.data_ptr(), int(q.dtype == torch.float32), _stream()), "gqa_qkv_post")
     return out
 

@@ -13,6 +13,8 @@ from typing import Optional, Tuple
 import torch
 import torch.nn.functional as F
 
+from .specs import RowNorms
+
 
 def embed_gather(table: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
     """ggml get_rows on the token embedding (src/llama-graph-utils.cpp:7-40)."""
@@ -28,13 +30,24 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, residual: Optional[tor
     return n.to(x.dtype), s
 
 
+def unary_of(y: torch.Tensor, unary) -> torch.Tensor:
+    """None, ("relu2",): max(y, 0)^2, or ("cap", s, c): c tanh(s y / c), s y with c = 0."""
+    if unary is None:
+        return y
+    if unary[0] == "relu2":
+        return torch.relu(y).square()
+    y = y.float() * unary[1]
+    return unary[2] * torch.tanh(y / unary[2]) if unary[2] else y
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor] = None,
-           out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """y = x @ w.T (+ residual); fp32 accumulate."""
+           out_dtype: Optional[torch.dtype] = None, unary=None) -> torch.Tensor:
+    """y = f(x @ w.T) (+ residual); fp32 accumulate."""
     if x.dtype == torch.float32 or x.is_cuda:
         y = x @ w.T if out_dtype in (None, x.dtype) else (x.float() @ w.float().T)
     else:
         y = (x.float() @ w.float().T)
+    y = unary_of(y, unary)
     if residual is not None:
         y = y.float() + residual.float()
     return y.to(out_dtype or x.dtype)
@@ -156,11 +169,15 @@ def mla_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tens
 
 def moe_gate(g: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], k: int, n_group: int,
              topk_group: int, scale: float, norm: bool, sigmoid: bool, n_shared: int = 0,
-             group_top2: bool = False, logit_bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+             group_top2: bool = False, logit_bias: Optional[torch.Tensor] = None, shared_gate: bool = False):
     """Router matmul (fp32) + softmax/sigmoid + [group-limited] top-k + renorm/scale
     (src/llama-graph-ffn.cpp:145-197).  ``bias`` takes part in the choice only, ``logit_bias`` is part of the logits (with
-    softmax and ``norm`` the weights are then a softmax over the chosen logits).  Returns ids [T,k] int32, weights [T,k] fp32."""
+    softmax and ``norm`` the weights are then a softmax over the chosen logits).  Returns ids [T,k] int32, weights [T,k] fp32; with
+    ``shared_gate`` also the outputs of the router's last row, whose sigmoid is then the shared experts' weight."""
     logits = g.float() @ w_router.float().T
+    gate = None
+    if shared_gate:
+        logits, gate = logits[:, :-1], logits[:, -1]
     if logit_bias is not None:
         logits = logits + logit_bias.float()
     probs = torch.sigmoid(logits) if sigmoid else torch.softmax(logits, dim=-1)
@@ -180,8 +197,9 @@ def moe_gate(g: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tenso
     if n_shared:        # shared experts as always-selected experts E, E+1, ... with weight 1
         sh = torch.arange(E, E + n_shared, dtype=torch.int32, device=ids.device)[None].expand(T, n_shared)
         ids = torch.cat([ids, sh], dim=1)
-        w = torch.cat([w, torch.ones(T, n_shared, dtype=w.dtype, device=w.device)], dim=1)
-    return ids.contiguous(), w.contiguous()
+        one = torch.ones(T, 1, dtype=w.dtype, device=w.device) if gate is None else torch.sigmoid(gate)[:, None]
+        w = torch.cat([w, one.expand(T, n_shared)], dim=1)
+    return (ids.contiguous(), w.contiguous()) + ((gate,) if shared_gate else ())
 
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, wg: torch.Tensor, wu: torch.Tensor,
@@ -273,9 +291,15 @@ def moe_routed(x, ids, wts, wg, wu, wd):
 
 # ---- blocks over an fp32 residual stream whose sublayers read one norm (csrc/kernels/parallel_block.cu) ------------------------
 def _finish_row(x, nxt, dtype):
-    """x fp32 -> (x, h, hc) for ``nxt`` = (norm weight, eps, conv) with conv = None or (w [taps, d], state, seq_slots, positions)."""
+    """x fp32 -> (x, h, hc) for ``nxt`` = (norm weight, eps, conv) with conv = None or (w [taps, d], state, seq_slots, positions), or a
+    ``RowNorms``."""
     if nxt is None:
         return x, None, None
+    if isinstance(nxt, RowNorms):
+        if nxt.w1 is None:
+            return x, x.to(dtype, copy=True), None
+        n = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + nxt.eps)
+        return x, (n * nxt.w1).to(dtype), None if nxt.w2 is None else (n * nxt.w2).to(dtype)
     w, eps, conv = nxt
     h = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
     if conv is None:
@@ -308,14 +332,31 @@ def post_norm(x, y, w, eps, nxt=None):
     return _finish_row(x + v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w, nxt, y.dtype)[:2]
 
 
+def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=None, dtype=None):
+    """x + s1 * o + s2 * (combine(moe) + sigmoid(dense_gate) * dense), ``moe`` = (y, dest, wts); o, moe, dense may be None."""
+    dtype = dtype or next((t.dtype for t in (o, dense, moe[0] if moe is not None else None) if t is not None), x.dtype)
+    v = x
+    if o is not None:
+        v = v + s1 * o.float()
+    f = None
+    if moe is not None:
+        y, dest, wts = moe
+        f = (y.float()[dest.long()] * wts[..., None]).sum(1)
+    if dense is not None:
+        g = dense.float() if dense_gate is None else torch.sigmoid(dense_gate.float())[:, None] * dense.float()
+        f = g if f is None else f + g
+    return _finish_row(v if f is None else v + s2 * f, nxt, dtype)
+
+
 def rms_rows(x, rows, w, eps, dtype):
     v = x if rows is None else x[rows.long()]
     return (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
 
 
-def causal_conv(h, w, state, seq_slots, positions, q_start):
-    """h + causal convolution over time, w [taps, d]; ``state`` [n, taps - 1, d] holds each sequence's last inputs."""
-    out = torch.empty_like(h)
+def causal_conv(h, w, state, seq_slots, positions, q_start, bias=None):
+    """h + causal convolution over time, w [taps, d], or with ``bias`` silu(convolution + bias); ``state`` [n, taps - 1, d] holds each
+    sequence's last inputs."""
+    out = torch.empty(h.shape, dtype=h.dtype, device=h.device)
     taps = w.shape[0]
     qs = q_start.tolist()
     for b in range(len(qs) - 1):
@@ -327,10 +368,10 @@ def causal_conv(h, w, state, seq_slots, positions, q_start):
         if slot >= 0 and taps > 1 and int(positions[q0]) > 0:
             old = state[slot]
         ext = torch.cat([old, h[q0:q1]], 0)
-        acc = h[q0:q1].float()
+        acc = h[q0:q1].float() if bias is None else bias.expand(q1 - q0, -1)
         for j in range(taps):
             acc = acc + w[j].float() * ext[j:j + q1 - q0].float()
-        out[q0:q1] = acc.to(h.dtype)
+        out[q0:q1] = (acc if bias is None else F.silu(acc)).to(h.dtype)
         if slot >= 0 and taps > 1:
             state[slot] = ext[q1 - q0:].clone()
     return out
@@ -423,6 +464,29 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     return out
 
 
+# ---- selective scan (csrc/kernels/selective_scan.cu) ------------------------------------------------------------------------------------
+def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
+    """Runs the recurrence of ``m`` (``ops.specs.SelectiveScan``) over a batch; result columns go to ``out`` [T, channels]."""
+    N = m.state
+    qs = q_start.tolist()
+    for b in range(len(qs) - 1):
+        q0, q1 = qs[b], qs[b + 1]
+        if q1 <= q0:
+            continue
+        slot = int(seq_slots[b])
+        S = state[slot].clone() if slot >= 0 and int(positions[q0]) > 0 else torch.zeros_like(m.neg_a)
+        xs, BC, d = x[q0:q1].float(), bc[q0:q1].float(), _softplus(dt[q0:q1].float())
+        a, u = torch.exp(d[..., None] * m.neg_a), (d * xs)[..., None] * BC[:, None, :N]
+        y = torch.empty_like(xs)
+        for t in range(q1 - q0):
+            S = a[t] * S + u[t]
+            y[t] = S @ BC[t, N:2 * N]
+        if slot >= 0:
+            state[slot] = S
+        out[q0:q1] = ((y + m.skip * xs) * F.silu(z[q0:q1].float()) * m.out_scale).to(out.dtype)
+    return out
+
+
 # ---- grouped-query attention over paged rows (csrc/kernels/gqa_attention.cu) ------------------------------------------------------------
 def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
     """Norms and rotates q and k, stores the rows of the cache; returns q [T, H, D].  ``m``: ``ops.specs.Gqa``."""
@@ -431,7 +495,8 @@ def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
 
     def post(x, n, w):
         x = x.float().reshape(T, n, D)
-        x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + m.eps) * w
+        if w is not None:
+            x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + m.eps) * w
         return torch.cat([_rope(x[..., :m.rot], cs, True), x[..., m.rot:]], -1)
     qo = post(q, H, m.q_norm).to(q.dtype)
     rows = torch.cat([post(k, G, m.k_norm).reshape(T, G * D), v.float()], 1).to(cache.dtype)
@@ -463,8 +528,9 @@ def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size
         if m.softcap:
             s = m.softcap * torch.tanh(s / m.softcap)
         s = s.masked_fill(~see, float("-inf"))
-        if m.sink:                                                # a key of score 0 without a value
-            s = torch.cat([s, torch.zeros_like(s[..., :1])], -1)
+        if m.sink:                                                # a key without a value
+            k0 = torch.zeros_like(s[..., :1])
+            s = torch.cat([s, k0 if m.sink_w is None else k0 + m.sink_w[:, None, None]], -1)
         p = torch.softmax(s, -1)[..., :S]
         o = torch.einsum("hij,jhv->ihv", p, v)
         if gate is not None:

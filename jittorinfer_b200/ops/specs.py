@@ -41,8 +41,9 @@ class StateMix:
 
 @dataclass
 class Gqa:
-    """Grouped-query attention with normed q and k, rotate-half RoPE on the first ``rot`` dimensions, scores * scale, softcap (0: none), a
-    causal mask with a sliding window and / or chunks (0: none), and with ``sink`` one more key of score 0 without a value."""
+    """Grouped-query attention with normed q and k (norm weights None: no norm), rotate-half RoPE on the first ``rot`` dimensions, scores *
+    scale, softcap (0: none), a causal mask with a sliding window and / or chunks (0: none), and with ``sink`` one more key without a value,
+    of score 0 or ``sink_w[head]``."""
     heads: int
     kv_heads: int
     dim: int
@@ -57,7 +58,29 @@ class Gqa:
     sink: bool = False
     eps: float = 1e-6
     out_scale: float = 1.0
+    sink_w: Optional[torch.Tensor] = None       # [heads] fp32
 
     @property
     def kv_row(self) -> int:
         return self.kv_heads * (self.dim + self.vdim)
+
+
+@dataclass
+class SelectiveScan:
+    """A state-space recurrence with a decay per channel and state: S[c, n] <- exp(dt_c neg_a[c, n]) S[c, n] + dt_c x_c B_n,
+    y_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c) out_scale, dt = softplus(.).  ``channels`` and ``state`` are multiples of 8 (a model
+    pads with zero weights)."""
+    channels: int
+    state: int
+    neg_a: torch.Tensor                         # [channels, state] fp32
+    skip: torch.Tensor                          # [channels]
+    out_scale: float = 1.0
+
+
+@dataclass
+class RowNorms:
+    """What an updated residual row turns into: row / rms * w1, and with ``w2`` row / rms * w2 as well; ``w1`` None: the row itself in the
+    activation type."""
+    eps: float = 0.0
+    w1: Optional[torch.Tensor] = None
+    w2: Optional[torch.Tensor] = None

@@ -31,6 +31,9 @@ class SplitCache:
         for d, n in counts.items():
             self.by_dev[d] = torch.zeros(n, n_slots, row, dtype=dtype, device=d)
 
+    def __len__(self) -> int:
+        return len(self.index)
+
     def __getitem__(self, il: int) -> torch.Tensor:
         d, i = self.index[il]
         return self.by_dev[d][i]
@@ -47,7 +50,7 @@ class SplitCache:
 
 
 class HybridCache:
-    """``rows[i]``: width of layer i's paged rows, ``("layer", j)`` for a layer that reads layer j's, None for none.
+    """One entry per layer, or per layer run where a model runs a layer several times.  ``rows[i]``: width of layer i's paged rows, ``("layer", j)`` for a layer that reads layer j's, None for none.
     ``state[name][i]``: (shape, dtype) of what one sequence keeps for layer i under that name, or None.
 
     ``cache[i]`` is the [n_slots, width] tensor layer i reads; ``cache.state[name][i]`` the [n_seqs, *shape] tensor.  State rows are
@@ -69,6 +72,9 @@ class HybridCache:
                 self._rows.append(t)
         self.state = {k: [None if s is None else torch.zeros((n_seqs,) + tuple(s[0]), dtype=s[1], device=device) for s in v]
                       for k, v in state.items()}
+
+    def __len__(self) -> int:
+        return len(self._rows)
 
     def __getitem__(self, il: int) -> Optional[torch.Tensor]:
         return self._rows[il]

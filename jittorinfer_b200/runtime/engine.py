@@ -319,7 +319,7 @@ class LLMEngine:
         if blocks.size == 0:
             return
         bs = self.cfg.block_size
-        for il in range(self.hp.n_layer):
+        for il in range(len(self.kv_cache)):
             layer = self.kv_cache[il]
             if layer is None:            # a layer without paged rows
                 continue

@@ -93,7 +93,7 @@ def main(argv=None, world: int = 1, rank: int = 0, control_group=None) -> int:
     ap.add_argument("--config", "-c", default=None, help="YAML file with the reference's keys (configs/*.yaml)")
     ap.add_argument("--port", type=int, default=None)
     ap.add_argument("--host", default=None)
-    ap.add_argument("--random-init", default=None, help="serve a random-init preset (tiny | lite | v2 | nibalix-tiny | nibalix-lite | lugovik-tiny | lugovik-lite) instead of a model file")
+    ap.add_argument("--random-init", default=None, help="serve a random-init preset (tiny | lite | v2 | nibalix-tiny | nibalix-lite | lugovik-tiny | lugovik-lite | zomavik-tiny | zomavik-lite) instead of a model file")
     args = ap.parse_args(argv)
     logging.basicConfig(level=os.environ.get("JITTORINFER_LOG", "INFO"), format="%(asctime)s %(levelname)s %(name)s: %(message)s")
     from ..config import load_yaml

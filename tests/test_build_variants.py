@@ -65,7 +65,8 @@ def test_every_entry_point_is_exported():
                  "jib_kv_block_copy", "jib_gather_rows", "jib_allreduce_oneshot", "jib_allreduce_twoshot", "jib_ar_epoch_bump",
                  "jib_ep_plan", "jib_ep_push", "jib_ep_combine", "jib_symm_alloc", "jib_symm_open", "jib_allgather_rows",
                  "jib_moe_permute_multi", "jib_moe_route_fused", "jib_moe_combine_norm", "jib_moe_combine_allreduce", "jib_sample_topk",
-                 "jib_gemm_simt", "jib_embed_norm", "jib_block_update", "jib_rms_rows", "jib_causal_conv", "jib_mingru"):
+                 "jib_gemm_simt", "jib_embed_norm", "jib_block_update", "jib_rms_rows", "jib_causal_conv", "jib_mingru",
+                 "jib_scaled_update", "jib_selective_scan"):
         assert hasattr(L, name), name
 
 
@@ -88,9 +89,9 @@ int main() {
     F(jib_gemm_desc, seg); F(jib_gemm_desc, x_row_stride); F(jib_gemm_desc, x_rows_total); F(jib_gemm_desc, scratch_bytes);
     F(jib_gemm_desc, n_counters); F(jib_gemm_desc, T); F(jib_gemm_desc, splits); F(jib_gemm_desc, ar_site); F(jib_gemm_desc, ar);
     F(jib_gemm_desc, out_row_ptr); F(jib_gemm_desc, ag_flags); F(jib_gemm_desc, ag_epoch); F(jib_gemm_desc, ag_rows);
-    F(jib_gemm_desc, ag_world); F(jib_gemm_desc, ar_rs_rows);
+    F(jib_gemm_desc, ag_world); F(jib_gemm_desc, ar_rs_rows); F(jib_gemm_desc, unary); F(jib_gemm_desc, softcap);
     printf("jib_row_tail %zu\n", sizeof(jib_row_tail));
-    F(jib_row_tail, conv_w); F(jib_row_tail, status); F(jib_row_tail, eps); F(jib_row_tail, n_state);
+    F(jib_row_tail, conv_w); F(jib_row_tail, status); F(jib_row_tail, eps); F(jib_row_tail, n_state); F(jib_row_tail, h2_out);
     return 0;
 }
 """

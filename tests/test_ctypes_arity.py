@@ -69,7 +69,7 @@ def test_descriptors_have_the_fields_of_their_c_structs_in_order():
     from jittorinfer_b200.ops import native
     src = re.sub(r"//[^\n]*", "", open(os.path.join(PKG, "csrc", "kernels", "jib_kernels.h")).read())
     for name, cls in (("jib_gemm_desc", native.GemmDesc), ("jib_row_tail", native.RowTail), ("jib_state_mix", native.StateMixDesc),
-                      ("jib_gqa", native.GqaDesc)):
+                      ("jib_gqa", native.GqaDesc), ("jib_scan", native.ScanDesc)):
         body = re.search(r"typedef struct %s \{(.*?)\} %s;" % (name, name), src, re.S).group(1)
         fields = [re.sub(r"[^A-Za-z0-9_]", "", v.split()[-1]) for d in body.split(";") if d.strip() for v in d.split(",")]
         assert fields == [n for n, _ in cls._fields_], name
@@ -79,14 +79,15 @@ def test_descriptor_field_names_exist():
     """ctypes structures accept assignments to names that are not fields (they become plain attributes and never reach the
     library): every ``d.<name> = ...`` on a GEMM descriptor and every ``ctx.<name>`` write on the communicator / dispatcher
     contexts must name a declared field."""
-    from jittorinfer_b200.ops.native import GemmDesc, GqaDesc, StateMixDesc
+    from jittorinfer_b200.ops.native import GemmDesc, GqaDesc, ScanDesc, StateMixDesc
     from jittorinfer_b200.parallel.comm import ArCtx
     from jittorinfer_b200.parallel.ep import EpCtx
     checks = [(os.path.join(PKG, "ops", "native.py"), "d", {n for n, _ in GemmDesc._fields_}),
               (os.path.join(PKG, "parallel", "comm.py"), "ctx", {n for n, _ in ArCtx._fields_}),
               (os.path.join(PKG, "parallel", "ep.py"), "ctx", {n for n, _ in EpCtx._fields_})]
     checks += [(os.path.join(PKG, "ops", "native.py"), "sd", {n for n, _ in StateMixDesc._fields_}),
-               (os.path.join(PKG, "ops", "native.py"), "gd", {n for n, _ in GqaDesc._fields_})]
+               (os.path.join(PKG, "ops", "native.py"), "gd", {n for n, _ in GqaDesc._fields_}),
+               (os.path.join(PKG, "ops", "native.py"), "cd", {n for n, _ in ScanDesc._fields_})]
     bad = []
     for path, var, fields in checks:
         tree = ast.parse(open(path).read())
