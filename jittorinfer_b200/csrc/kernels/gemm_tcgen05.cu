@@ -70,7 +70,7 @@ struct GemmArgs {
     int w_evict_first;        // weight tiles are loaded with the L2 evict_first policy (each is read once: small batches)
     int act;                  // of a gated pair (JIB_ACT_*)
     int unary;                // of a single product (JIB_UNARY_*)
-    float scale, softcap;
+    float scale, softcap, cap2;      // cap2 = 2 scale / softcap
     int vec_store;            // bf16 result rows are written as 16-byte vectors through a shared-memory transpose
     const int * src_token;    // grouped, decode batches: x holds the T token rows unsorted, every expert multiplies all of
                               // them (one token tile) and sorted row i of the result is accumulator column src_token[i]
@@ -157,8 +157,8 @@ __device__ __forceinline__ float gated(float x, int act) {
 __device__ __forceinline__ float unary(float v, const GemmArgs & a) {
     if (a.unary == JIB_UNARY_NONE) return v;
     if (a.unary == JIB_UNARY_RELU2) return v > 0.f ? v * v : 0.f;
-    v *= a.scale;
-    return a.softcap > 0.f ? a.softcap * (1.f - 2.f / (1.f + __expf(2.f * fminf(v / a.softcap, 40.f)))) : v;
+    if (a.softcap <= 0.f) return v * a.scale;
+    return a.softcap * (1.f - __fdividef(2.f, 1.f + __expf(fminf(v * a.cap2, 80.f))));
 }
 
 // Cluster-wide barrier (all threads of all CTAs of the cluster) and a load from a peer CTA's shared memory.
@@ -1155,6 +1155,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream_)
     if (a.ar_rs_rows < 0) return JIB_E_ARG;
     if (a.row_ptr != nullptr && (dual || d->out_f32 || d->residual != nullptr || d->ar != nullptr)) return JIB_E_ARG;
     a.act = d->act; a.unary = dual ? JIB_UNARY_NONE : d->unary; a.scale = d->scale; a.softcap = d->softcap;
+    a.cap2 = d->softcap > 0.f ? 2.f * d->scale / d->softcap : 0.f;
     if (a.unary != JIB_UNARY_NONE && d->ar != nullptr) return JIB_E_ARG;
     memset(&a.ar, 0, sizeof(a.ar));
     if (d->ar != nullptr) {
@@ -1329,7 +1330,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16_noalloc(const void * x, const void * w, 
     a.expert_list = nullptr;
     a.list_tiles = 0;
     a.ag_flags = nullptr; a.ag_epoch = nullptr; a.ag_rows = 0; a.ag_world = 0; a.ar_rs_rows = 0; a.ag_spin_limit = 0;
-    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = 0.f;
+    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = a.cap2 = 0.f;
     memset(&a.ar, 0, sizeof(a.ar));
     dim3 grid(p.n_tiles, 1, p.splits);
     switch (p.bn) {

@@ -264,14 +264,13 @@ JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, v
 JIB_EXPORT long long jib_state_chunk_bytes(const jib_state_mix * m);
 
 // ---- selective scan: a diagonal state per channel (selective_scan.cu) -------------------------------------------------------------
-//   S[c][n] <- exp(dt_c a[c][n]) S[c][n] + dt_c x_c B_n;   y_c = (sum_n S[c][n] C_n + skip_c x_c) * silu(z_c) * out_scale,   dt = softplus(dt_c)
+//   S[c][n] <- exp(dt_c a[c][n]) S[c][n] + dt_c x_c B_n;   y_c = (sum_n S[c][n] C_n + skip_c x_c) * silu(z_c) * out_scale,   dt = softplus(dt_c + bias_c)
 // over ch channels (a multiple of 8) with N states each (a multiple of 8, at most 256).
 typedef struct jib_scan {
-    const void * x, * z, * bc; // activations: [T][ldx], [T][ldz], and [T][ldbc] = B | C
-    const float * dt;          // [T][lddt] pre-activations of the step sizes, bias included
+    const void * x, * z, * bc, * dt;       // activations: [T][ldx], [T][ldz], [T][ldbc] = B | C, [T][lddt]
     void * y;                  // [T][ldy]
     const float * neg_a;       // [ch][N]
-    const float * skip;        // [ch]
+    const float * skip, * dt_bias;         // [ch]
     float * state;             // [n_state][ch][N]
     const int * seq_slots, * positions, * q_start;
     int * status;

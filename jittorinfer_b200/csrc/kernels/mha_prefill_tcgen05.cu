@@ -93,7 +93,8 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     constexpr int NC = F::NC, Q_BYTES = F::Q_BYTES, K_BYTES = F::K_BYTES;
     extern __shared__ uint8_t smem_raw[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h = blockIdx.y;
+    // GQA: all heads' longest query tiles start first
+    const int h = GQA ? blockIdx.x : blockIdx.y;
     // columns of this head's keys and values in the gathered rows, and of its queries
     const int kcol = GQA ? h / (a.H / a.G) * DN : h * (DN + DV), vcol = GQA ? a.G * DN + h / (a.H / a.G) * DV : h * (DN + DV) + DN, qcol = h * NC * 64;
 
@@ -143,11 +144,11 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const uint32_t tmem = *tmem_slot;
     const uint32_t tm_S = tmem, tm_O = tmem + 2 * KT;
 
-    // ---- which (sequence, query tile) is this CTA?  blockIdx.x walks the tiles of all sequences, last tile of a
+    // ---- which (sequence, query tile) is this CTA?  blockIdx.x (GQA: .y) walks the tiles of all sequences, last tile of a
     // sequence first (it sees the most KV tiles) ----
     int b = -1, q0 = 0, q_len = 0, tile = 0;
     {
-        int x = blockIdx.x;
+        int x = GQA ? blockIdx.y : blockIdx.x;
         for (int s = 0; s < a.n_seqs; ++s) {
             const int qs = a.q_start[s], ql = a.q_start[s + 1] - qs;
             const int nt = (ql + QT - 1) / QT;
@@ -503,7 +504,7 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
     constexpr int SMEM = Form<true>::SMEM_BYTES;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(mha_prefill_kernel<true>, SMEM, attr_done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((mha_prefill_kernel<true>), dim3(n_q_tiles, m->H), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
+    JIB_LAUNCH((mha_prefill_kernel<true>), dim3(m->H, n_q_tiles), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 

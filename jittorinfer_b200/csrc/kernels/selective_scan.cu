@@ -2,14 +2,15 @@
 //
 //   S[c][n] <- exp(dt_c a[c][n]) S[c][n] + dt_c x_c B_n;   y_c = (sum_n S[c][n] C_n + skip_c x_c) * silu(z_c) * out_scale
 //
-// with dt = softplus(dt_c) and B, C shared by the channels.  L lanes of a warp share a channel, NS states each.
+// with dt = softplus(dt_c + bias_c) and B, C shared by the channels.  L lanes of a warp share a channel, NS states each.
 //
-//   scan_step      one token per sequence: the state is read and written once
+//   scan_step      one token per sequence: the state is read and written once, several sequences per thread in flight
 //   scan_portions  ranges of any length: a CTA owns 128 / L channels of one sequence, keeps their states in registers and walks the
 //                  tokens in tiles of TT, the next tile's inputs on their way while one is worked on
 //
-// The exponentials do not depend on the state, so a token costs its lane one multiply-add of latency.  The lanes' partial sums of
-// several tokens meet in one butterfly that leaves each lane with one token's sum.
+// The exponentials do not depend on the state, so a token costs its lane one multiply-add of latency.  Tokens go in groups of 8: the
+// lanes' partial sums of a group meet in one butterfly that leaves each lane with the sums of some of the tokens, and it runs
+// under the next group's exponentials.
 //
 // A sequence's state lives in row seq_slots[b] of [n_state][ch][N]; a range that starts at position 0 starts from zeros whatever the
 // row holds.  Sequence b owns token rows q_start[b] .. q_start[b + 1].  Activations bf16 or fp32, the rest fp32.
@@ -35,17 +36,69 @@ __device__ __forceinline__ void put(float * p, float v) { *p = v; }
 template <typename T> __device__ __forceinline__ float silu(float v);
 template <> __device__ __forceinline__ float silu<bf16>(float v) { return v * __fdividef(1.f, 1.f + __expf(-v)); }
 template <> __device__ __forceinline__ float silu<float>(float v) { return v / (1.f + expf(-v)); }
-template <typename T> __device__ __forceinline__ float rate(float neg_a);            // what decay() takes
+template <typename T> __device__ __forceinline__ float rate(float neg_a);            // what advance() takes, times dt
 template <> __device__ __forceinline__ float rate<bf16>(float neg_a) { return neg_a * 1.4426950408889634f; }
 template <> __device__ __forceinline__ float rate<float>(float neg_a) { return neg_a; }
-template <typename T> __device__ __forceinline__ float decay(float v);
-template <> __device__ __forceinline__ float decay<bf16>(float v) {
+// exp(v) s + u, v <= 0.  fp32: a decay close to 1 as s + s (exp(v) - 1), or its rounding to 24 bits would bias every step alike
+template <typename T> __device__ __forceinline__ float advance(float v, float s, float u);
+template <> __device__ __forceinline__ float advance<bf16>(float v, float s, float u) {
     float r;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r * s + u;
+}
+template <> __device__ __forceinline__ float advance<float>(float v, float s, float u) {
+    return (v > -0.5f ? fmaf(s, expm1f(v), s) : s * expf(v)) + u;
+}
+// log(1 + e^v) = max(v, 0) + log1p(e^-|v|).  bf16: log1p(e) = 2 atanh(r), r = e / (2 + e) <= 1/3, by atanh's series to r^13 (relative
+// error below 1e-7).
+template <typename T> __device__ __forceinline__ float softplus(float v);
+template <> __device__ __forceinline__ float softplus<float>(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+template <> __device__ __forceinline__ float softplus<bf16>(float v) {
+    const float e = __expf(-fabsf(v)), r = __fdividef(e, 2.f + e), q = r * r;
+    float p = q * (2.f / 13.f) + 2.f / 11.f;
+    p = p * q + 2.f / 9.f;
+    p = p * q + 2.f / 7.f;
+    p = p * q + 2.f / 5.f;
+    p = p * q + 2.f / 3.f;
+    p = p * q + 2.f;
+    return fmaxf(v, 0.f) + p * r;
+}
+// two fp32 operations per instruction
+struct F2 {
+    unsigned long long v;
+};
+__device__ __forceinline__ F2 pack(float a, float b) {
+    F2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(a), "f"(b));
     return r;
 }
-template <> __device__ __forceinline__ float decay<float>(float v) { return expf(v); }
-__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+__device__ __forceinline__ float2 unpack(F2 a) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+    return r;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+    F2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+    return r;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+    F2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+    return r;
+}
+// advance() of two states
+template <typename T> __device__ __forceinline__ F2 advance2(F2 v, F2 s, F2 u);
+template <> __device__ __forceinline__ F2 advance2<bf16>(F2 v, F2 s, F2 u) {
+    float2 e = unpack(v);
+    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.x));
+    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.y));
+    return fma2(pack(e.x, e.y), s, u);
+}
+template <> __device__ __forceinline__ F2 advance2<float>(F2 v, F2 s, F2 u) {
+    const float2 e = unpack(v), x = unpack(s), y = unpack(u);
+    return pack(advance<float>(e.x, x.x, y.x), advance<float>(e.y, x.y, y.y));
+}
 
 // 4 adjacent elements, kept as stored until they are needed (many loads in flight)
 template <typename T> struct Quad;
@@ -71,25 +124,17 @@ template <> struct Quad<bf16> {
         *(uint2 *) p = o;
     }
 };
-// NS adjacent floats
+// NS adjacent floats, NS a multiple of 4
 template <int NS> __device__ __forceinline__ void load_n(const float * p, float (&v)[NS]) {
 #pragma unroll
-    for (int i = 0; i < NS; i += (NS >= 4 ? 4 : 2)) {
-        if (NS >= 4) {
-            const float4 x = *(const float4 *) (p + i);
-            v[i] = x.x; v[i + 1] = x.y; v[(i + 2) % NS] = x.z; v[(i + 3) % NS] = x.w;
-        } else {
-            const float2 x = *(const float2 *) (p + i);
-            v[i] = x.x; v[i + 1] = x.y;
-        }
+    for (int i = 0; i < NS; i += 4) {
+        const float4 x = *(const float4 *) (p + i);
+        v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
     }
 }
 template <int NS> __device__ __forceinline__ void store_n(float * p, const float (&v)[NS]) {
 #pragma unroll
-    for (int i = 0; i < NS; i += (NS >= 4 ? 4 : 2)) {
-        if (NS >= 4) *(float4 *) (p + i) = make_float4(v[i], v[i + 1], v[(i + 2) % NS], v[(i + 3) % NS]);
-        else *(float2 *) (p + i) = make_float2(v[i], v[i + 1]);
-    }
+    for (int i = 0; i < NS; i += 4) *(float4 *) (p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
 }
 
 __device__ __forceinline__ int checked_slot(const jib_scan & a, int b, int site) {
@@ -101,43 +146,60 @@ __device__ __forceinline__ int checked_slot(const jib_scan & a, int b, int site)
     return slot;
 }
 
-// ---- single tokens: grid (ceil(ch / (NT / L)), T), row t belongs to sequence t -----------------------------------------------------
-template <typename T, int NS, int L>
+// ---- single tokens: grid (ceil(ch / (NT / L)), ceil(T / U)), row t belongs to sequence t ---------------------------------------------
+template <typename T, int NS, int L, int U>
 __global__ void __launch_bounds__(NT) scan_step_kernel(const __grid_constant__ jib_scan a) {
     PDL_TRIGGER_TOP();
-    const int lane = threadIdx.x % L, c = blockIdx.x * (NT / L) + threadIdx.x / L, t = blockIdx.y, n0 = lane * NS;
+    const int lane = threadIdx.x % L, c = blockIdx.x * (NT / L) + threadIdx.x / L, n0 = lane * NS;
     const bool mine = c < a.ch, live = mine && n0 < a.N;
     const int cc = mine ? c : a.ch - 1, nn = n0 < a.N ? n0 : 0;
-    float ra[NS], s[NS];
+    float ra[NS];
     load_n<NS>(a.neg_a + (size_t) cc * a.N + nn, ra);        // launch-invariant
-    const float skip = a.skip[cc];
+    const float skip = a.skip[cc], bias = a.dt_bias[cc];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int slot = checked_slot(a, t, 51);
-    float * st = a.state + ((size_t) (slot < 0 ? 0 : slot) * a.ch + cc) * a.N + nn;
-    const bool past = slot >= 0 && live && a.positions[t] > 0;
+    int slot[U];
+    float s[U][NS], dt[U], x[U], z[U];
+    Quad<T> B[U][NS / 4], C[U][NS / 4];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) s[i] = 0.f;
-    if (past) load_n<NS>(st, s);
-    const T * bc = (const T *) a.bc + (size_t) t * a.ldbc + nn;
-    float B[NS], C[NS];
+    for (int u = 0; u < U; ++u) {                            // everything the rows need is requested before any of it is used
+        const int t = blockIdx.y * U + u, tt = min(t, a.T - 1);
+        slot[u] = t < a.T ? checked_slot(a, t, 51) : -1;
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-        B[i] = to_f(bc[i]);
-        C[i] = to_f(bc[a.N + i]);
+        for (int i = 0; i < NS; ++i) s[u][i] = 0.f;
+        if (slot[u] >= 0 && live && a.positions[tt] > 0) load_n<NS>(a.state + ((size_t) slot[u] * a.ch + cc) * a.N + nn, s[u]);
+        const T * bc = (const T *) a.bc + (size_t) tt * a.ldbc + nn;
+#pragma unroll
+        for (int i = 0; i < NS / 4; ++i) {
+            B[u][i].load(bc + 4 * i);
+            C[u][i].load(bc + a.N + 4 * i);
+        }
+        x[u] = to_f(((const T *) a.x)[(size_t) tt * a.ldx + cc]);
+        z[u] = to_f(((const T *) a.z)[(size_t) tt * a.ldz + cc]);
+        dt[u] = to_f(((const T *) a.dt)[(size_t) tt * a.lddt + cc]);
     }
-    const float x = to_f(((const T *) a.x)[(size_t) t * a.ldx + cc]), z = to_f(((const T *) a.z)[(size_t) t * a.ldz + cc]);
-    const float dt = softplus(a.dt[(size_t) t * a.lddt + cc]), dx = dt * x;
-    float y = 0.f;
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-        s[i] = decay<T>(dt * rate<T>(ra[i])) * s[i] + dx * B[i];
-        y += s[i] * C[i];
+    for (int i = 0; i < NS; ++i) ra[i] = rate<T>(ra[i]);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int t = blockIdx.y * U + u;
+        const float d = softplus<T>(dt[u] + bias), dx = d * x[u];
+        float y = 0.f;
+#pragma unroll
+        for (int i = 0; i < NS / 4; ++i) {
+            const float4 b = B[u][i].get(), k = C[u][i].get();
+            const float bv[4] = {b.x, b.y, b.z, b.w}, kv[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[u][4 * i + e] = advance<T>(d * ra[4 * i + e], s[u][4 * i + e], dx * bv[e]);
+                y += s[u][4 * i + e] * kv[e];
+            }
+        }
+        if (!live) y = 0.f;
+        if (live && slot[u] >= 0) store_n<NS>(a.state + ((size_t) slot[u] * a.ch + cc) * a.N + nn, s[u]);
+#pragma unroll
+        for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+        if (lane == 0 && mine && t < a.T) put((T *) a.y + (size_t) t * a.ldy + c, (y + skip * x[u]) * silu<T>(z[u]) * a.out_scale);
     }
-    if (!live) y = 0.f;
-    if (live && slot >= 0) store_n<NS>(st, s);
-#pragma unroll
-    for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-    if (lane == 0 && mine) put((T *) a.y + (size_t) t * a.ldy + c, (y + skip * x) * silu<T>(z) * a.out_scale);
 }
 
 // ---- portions: grid (ceil(ch / CH), n_seqs) ----------------------------------------------------------------------------------------
@@ -145,12 +207,11 @@ template <typename T, int NS, int L>
 struct Scan {
     static constexpr int NP = NS * L, CH = NT / L;
     static constexpr int TT = NP <= 64 ? 32 : 8;             // tokens of a tile
-    static constexpr int GT = L < 8 ? L : 8;                 // tokens whose sums meet in one butterfly
+    static constexpr int G = 8;                              // tokens of a group
     static constexpr int QX = TT * CH / 4, QB = TT * 2 * NP / 4;                     // quads of a tile: per channel input, of B | C
     static constexpr int RX = (QX + NT - 1) / NT, RB = (QB + NT - 1) / NT;
-    static constexpr int SMEM = 4 * (TT * CH * 2 + TT * 2 * NP + TT * CH);
-    Quad<T> x[RX], z[RX], bc[RB];
-    Quad<float> dt[RX];
+    static constexpr int SMEM = 4 * (TT * CH * 4 + TT * 2 * NP + TT * CH);
+    Quad<T> x[RX], z[RX], dt[RX], bc[RB];
     // tokens t0 .. of the sequence's n, whose first row is q0
     __device__ __forceinline__ void load(const jib_scan & a, int q0, int n, int t0, int c0) {
 #pragma unroll
@@ -161,7 +222,7 @@ struct Scan {
                 const size_t r = q0 + t;
                 x[i].load((const T *) a.x + r * a.ldx + c);
                 z[i].load((const T *) a.z + r * a.ldz + c);
-                dt[i].load(a.dt + r * a.lddt + c);
+                dt[i].load((const T *) a.dt + r * a.lddt + c);
             }
         }
         const int n4 = a.N / 2;                              // quads of a row of B | C
@@ -174,22 +235,44 @@ struct Scan {
     }
 };
 
+// The L lanes' partial sums of 8 tokens -> lane j < W holds those of tokens j * 8 / W .. in p[0 .. 8 / W), W = min(L, 8).
+template <int L> __device__ __forceinline__ void meet(float (&p)[8], int lane) {
+    constexpr int W = L < 8 ? L : 8;
+    int n = 8;
+#pragma unroll
+    for (int o = W / 2; o > 0; o >>= 1) {
+        n >>= 1;
+        const bool up = (lane & o) != 0;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            if (k >= n) break;
+            const float keep = up ? p[k + n] : p[k], send = up ? p[k] : p[k + n];
+            p[k] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+#pragma unroll
+    for (int o = W; o < L; o <<= 1) p[0] += __shfl_xor_sync(0xffffffffu, p[0], o);
+}
+
 template <typename T, int NS, int L>
 __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant__ jib_scan a) {
     using S = Scan<T, NS, L>;
-    constexpr int NP = S::NP, CH = S::CH, TT = S::TT, GT = S::GT;
+    constexpr int NP = S::NP, CH = S::CH, TT = S::TT, G = S::G, W = L < 8 ? L : 8, H = NS / 2;
     extern __shared__ __align__(16) float smem[];
-    float2 * sdx = (float2 *) smem;                          // [TT][CH]: step size, step size * x
-    float * sb = smem + TT * CH * 2, * sc = sb + TT * NP, * sy = sc + TT * NP;       // [TT][NP], [TT][NP], [TT][CH]
+    float4 * sdx = (float4 *) smem;                          // [TT][CH]: step size twice, step size * x twice
+    float * sb = smem + TT * CH * 4, * sc = sb + TT * NP, * sy = sc + TT * NP;       // [TT][NP], [TT][NP], [TT][CH]
     PDL_TRIGGER_TOP();
     const int lane = threadIdx.x % L, cl = threadIdx.x / L, c0 = blockIdx.x * CH, c = c0 + cl, b = blockIdx.y, n0 = lane * NS;
     const bool live = c < a.ch && n0 < a.N;
-    float ra[NS], s[NS];
+    F2 ra[H], s[H];
+    {
+        float v[NS];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) ra[i] = s[i] = 0.f;
-    if (live) load_n<NS>(a.neg_a + (size_t) c * a.N + n0, ra);
+        for (int i = 0; i < NS; ++i) v[i] = 0.f;
+        if (live) load_n<NS>(a.neg_a + (size_t) c * a.N + n0, v);
 #pragma unroll
-    for (int i = 0; i < NS; ++i) ra[i] = rate<T>(ra[i]);
+        for (int i = 0; i < H; ++i) ra[i] = pack(rate<T>(v[2 * i]), rate<T>(v[2 * i + 1]));
+    }
     for (int i = threadIdx.x; i < TT * 2 * NP; i += NT) sb[i] = 0.f;                 // columns past N stay zero
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
@@ -198,7 +281,21 @@ __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant
     cur.load(a, q0, n, 0, c0);
     const int slot = checked_slot(a, b, 52);
     float * st = a.state + ((size_t) (slot < 0 ? 0 : slot) * a.ch + c) * a.N + n0;
-    if (live && slot >= 0 && a.positions[q0] > 0) load_n<NS>(st, s);
+    {
+        float v[NS];
+#pragma unroll
+        for (int i = 0; i < NS; ++i) v[i] = 0.f;
+        if (live && slot >= 0 && a.positions[q0] > 0) load_n<NS>(st, v);
+#pragma unroll
+        for (int i = 0; i < H; ++i) s[i] = pack(v[2 * i], v[2 * i + 1]);
+    }
+    const int cq = threadIdx.x % (CH / 4) * 4;               // this thread's quads: the same channels of different tokens
+    static_assert(NT % (CH / 4) == 0, "");
+    float4 skip = make_float4(0.f, 0.f, 0.f, 0.f), bias = skip;
+    if (c0 + cq < a.ch) {
+        skip = *(const float4 *) (a.skip + c0 + cq);
+        bias = *(const float4 *) (a.dt_bias + c0 + cq);
+    }
     __syncthreads();
     for (int t0 = 0; t0 < n; t0 += TT) {
 #pragma unroll
@@ -206,11 +303,12 @@ __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant
             const int q = threadIdx.x + i * NT, t = q / (CH / 4);
             if (q >= S::QX) continue;
             const float4 x = cur.x[i].get(), d = cur.dt[i].get();
-            const bool in = t0 + t < n;                      // past the end: the state passes through
-            const float dt[4] = {softplus(d.x), softplus(d.y), softplus(d.z), softplus(d.w)};
-            float4 * o = (float4 *) (sdx + t * CH + q % (CH / 4) * 4);
-            o[0] = in ? make_float4(dt[0], dt[0] * x.x, dt[1], dt[1] * x.y) : make_float4(0.f, 0.f, 0.f, 0.f);
-            o[1] = in ? make_float4(dt[2], dt[2] * x.z, dt[3], dt[3] * x.w) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float xv[4] = {x.x, x.y, x.z, x.w}, dv[4] = {d.x + bias.x, d.y + bias.y, d.z + bias.z, d.w + bias.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float k = t0 + t < n ? softplus<T>(dv[e]) : 0.f;               // past the end: the state passes through
+                sdx[t * CH + cq + e] = make_float4(k, k, k * xv[e], k * xv[e]);
+            }
         }
         const int n4 = a.N / 2;
 #pragma unroll
@@ -221,68 +319,80 @@ __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant
         __syncthreads();
         if (t0 + TT < n) nxt.load(a, q0, n, t0 + TT, c0);
         const int m = min(TT, n - t0);
+        float p[G], last[G];
+        auto out = [&](int g) {                              // the group whose sums are in last
+            meet<L>(last, lane);
+            if (lane < W) {
+#pragma unroll
+                for (int k = 0; k < G / W; ++k) sy[(g + lane * (G / W) + k) * CH + cl] = last[k];
+            }
+        };
 #pragma unroll 1
-        for (int g = 0; g < m; g += GT) {
-            float p[GT];
+        for (int g = 0; g < m; g += G) {
+            if (g > 0) out(g - G);
 #pragma unroll
-            for (int k = 0; k < GT; ++k) {
-                const float2 d = sdx[(g + k) * CH + cl];
-                float B[NS], C[NS];
-                load_n<NS>(sb + (g + k) * NP + n0, B);
-                load_n<NS>(sc + (g + k) * NP + n0, C);
-                p[k] = 0.f;
+            for (int k = 0; k < G; ++k) {
+                const ulonglong2 d = *(const ulonglong2 *) (sdx + (g + k) * CH + cl);
+                F2 acc;
 #pragma unroll
-                for (int i = 0; i < NS; ++i) {
-                    s[i] = decay<T>(d.x * ra[i]) * s[i] + d.y * B[i];
-                    p[k] += s[i] * C[i];
+                for (int i = 0; i < H; ++i) {
+                    const F2 B = {*(const unsigned long long *) (sb + (g + k) * NP + n0 + 2 * i)};
+                    const F2 C = {*(const unsigned long long *) (sc + (g + k) * NP + n0 + 2 * i)};
+                    s[i] = advance2<T>(mul2({d.x}, ra[i]), s[i], mul2({d.y}, B));
+                    acc = i == 0 ? mul2(s[i], C) : fma2(s[i], C, acc);
                 }
+                const float2 y = unpack(acc);
+                p[k] = y.x + y.y;
             }
 #pragma unroll
-            for (int o = GT / 2; o > 0; o >>= 1)
-#pragma unroll
-                for (int k = 0; k < o; ++k) {
-                    const bool up = (lane & o) != 0;
-                    const float keep = up ? p[k + o] : p[k], send = up ? p[k] : p[k + o];
-                    p[k] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                }
-#pragma unroll
-            for (int o = GT; o < L; o <<= 1) p[0] += __shfl_xor_sync(0xffffffffu, p[0], o);
-            if (lane < GT) sy[(g + lane) * CH + cl] = p[0];
+            for (int k = 0; k < G; ++k) last[k] = p[k];
         }
+        out((m - 1) / G * G);
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < S::RX; ++i) {
-            const int q = threadIdx.x + i * NT, t = q / (CH / 4), cq = q % (CH / 4) * 4;
+            const int q = threadIdx.x + i * NT, t = q / (CH / 4);
             if (q >= S::QX || t >= m || c0 + cq >= a.ch) continue;
-            const float4 y = *(const float4 *) (sy + t * CH + cq), x = cur.x[i].get(), z = cur.z[i].get(), k = *(const float4 *) (a.skip + c0 + cq);
+            const float4 y = *(const float4 *) (sy + t * CH + cq), x = cur.x[i].get(), z = cur.z[i].get();
             Quad<T>::store((T *) a.y + (size_t) (q0 + t0 + t) * a.ldy + c0 + cq,
-                           make_float4((y.x + k.x * x.x) * silu<T>(z.x) * a.out_scale, (y.y + k.y * x.y) * silu<T>(z.y) * a.out_scale,
-                                       (y.z + k.z * x.z) * silu<T>(z.z) * a.out_scale, (y.w + k.w * x.w) * silu<T>(z.w) * a.out_scale));
+                           make_float4((y.x + skip.x * x.x) * silu<T>(z.x) * a.out_scale, (y.y + skip.y * x.y) * silu<T>(z.y) * a.out_scale,
+                                       (y.z + skip.z * x.z) * silu<T>(z.z) * a.out_scale, (y.w + skip.w * x.w) * silu<T>(z.w) * a.out_scale));
         }
         cur = nxt;
     }
-    if (live && slot >= 0) store_n<NS>(st, s);
+    if (live && slot >= 0) {
+        float v[NS];
+#pragma unroll
+        for (int i = 0; i < H; ++i) {
+            const float2 x = unpack(s[i]);
+            v[2 * i] = x.x;
+            v[2 * i + 1] = x.y;
+        }
+        store_n<NS>(st, v);
+    }
 }
 
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
 template <typename T, int NS, int L>
 int run(const jib_scan & a, int single, cudaStream_t s) {
-    constexpr int CH = NT / L;
+    constexpr int CH = NT / L, U = sizeof(T) == 2 && NS == 4 ? 4 : 1;
+    const unsigned gx = (a.ch + CH - 1) / CH;
     if (single) {
-        JIB_LAUNCH((scan_step_kernel<T, NS, L>), dim3((a.ch + CH - 1) / CH, a.T), NT, 0, s, a);
+        if (U > 1 && a.T * gx > 148 * 8) JIB_LAUNCH((scan_step_kernel<T, NS, L, U>), dim3(gx, (a.T + U - 1) / U), NT, 0, s, a);
+        else JIB_LAUNCH((scan_step_kernel<T, NS, L, 1>), dim3(gx, a.T), NT, 0, s, a);
         return launched();
     }
     constexpr int SMEM = Scan<T, NS, L>::SMEM;
     static_assert(SMEM <= 48 * 1024, "fits without an attribute");
-    JIB_LAUNCH((scan_portions_kernel<T, NS, L>), dim3((a.ch + CH - 1) / CH, a.n_seqs), NT, SMEM, s, a);
+    JIB_LAUNCH((scan_portions_kernel<T, NS, L>), dim3(gx, a.n_seqs), NT, SMEM, s, a);
     return launched();
 }
 
 template <typename T>
 int dispatch(const jib_scan & a, int single, cudaStream_t s) {
-    if (a.N <= 8) return run<T, 2, 4>(a, single, s);
-    if (a.N <= 16) return run<T, 2, 8>(a, single, s);
+    if (a.N <= 8) return run<T, 4, 2>(a, single, s);
+    if (a.N <= 16) return run<T, 4, 4>(a, single, s);
     if (a.N <= 32) return run<T, 4, 8>(a, single, s);
     if (a.N <= 64) return run<T, 4, 16>(a, single, s);
     if (a.N <= 128) return run<T, 4, 32>(a, single, s);
@@ -296,8 +406,8 @@ extern "C" JIB_EXPORT int jib_selective_scan(const jib_scan * m, int single, int
     if (a.T <= 0 || a.n_seqs <= 0) return 0;
     if (a.ch < 8 || a.ch % 8 || a.N < 8 || a.N % 8 || a.N > 256 || a.T > 65535 || a.n_seqs > 65535 || (single && a.T != a.n_seqs)) return JIB_E_ARG;
     const uintptr_t mask = f32 ? 15 : 7;                     // quads of activations, 16 bytes of fp32
-    if ((((uintptr_t) a.x | (uintptr_t) a.z | (uintptr_t) a.bc | (uintptr_t) a.y) & mask) || ((a.ldx | a.ldz | a.ldbc | a.ldy | a.lddt) & 3) ||
-        (((uintptr_t) a.dt | (uintptr_t) a.neg_a | (uintptr_t) a.skip | (uintptr_t) a.state) & 15))
+    if ((((uintptr_t) a.x | (uintptr_t) a.z | (uintptr_t) a.bc | (uintptr_t) a.dt | (uintptr_t) a.y) & mask) || ((a.ldx | a.ldz | a.ldbc | a.ldy | a.lddt) & 3) ||
+        (((uintptr_t) a.dt_bias | (uintptr_t) a.neg_a | (uintptr_t) a.skip | (uintptr_t) a.state) & 15))
         return JIB_E_ALIGN;
     cudaStream_t s = (cudaStream_t) stream;
     return f32 ? dispatch<float>(a, single, s) : dispatch<bf16>(a, single, s);

@@ -295,7 +295,7 @@ def _padded(t: torch.Tensor, *shape: int) -> torch.Tensor:
 
 class _Layer:
     __slots__ = ("norm1", "norm2", "ls1", "ls2", "w_in", "b_in", "cols", "w_o", "y_col", "attn", "rope", "scan", "conv_w", "conv_b", "w_x", "w_dt",
-                 "b_dt", "w_up", "w_down", "router", "n_merged", "w_gate_exps", "w_up_exps", "w_down_exps", "w_gate_sh", "w_up_sh", "w_down_sh")
+                 "w_up", "w_down", "router", "n_merged", "w_gate_exps", "w_up_exps", "w_down_exps", "w_gate_sh", "w_up_sh", "w_down_sh")
 
     def __init__(self):
         for s in self.__slots__:
@@ -345,7 +345,7 @@ class ZomavikModel:
             if i >= 0 and base.startswith("mlp.") and isinstance(hp.layers[i].mlp, Experts) and base.count(".") == 2 and base[-3:] != ".sg":
                 self._take_expert(i, *base.split(".")[1:], t)          # straight into the stacked tensors: nothing is held twice
             else:
-                small = t.dim() == 1 or base.endswith((".conv", ".A_log", ".router", ".sg"))
+                small = t.dim() == 1 or base.endswith((".conv", ".A_log"))
                 pend[name] = t.to(device=dev, dtype=f32 if small else self.dtype).contiguous()
             if i >= 0:
                 todo[i].discard(name)
@@ -395,8 +395,9 @@ class ZomavikModel:
         w, rows = take("mix.right.x"), (0, r.dt_rank, r.dt_rank + r.state, r.dt_rank + 2 * r.state)
         w, _ = stack_rows([(str(k), w[rows[k]:rows[k + 1]]) for k in range(3)])                      # dt | B | C
         L.w_x = _padded(w, w.shape[0], ch)
-        L.w_dt, L.b_dt = _padded(take("mix.right.dt"), ch, R), _padded(take("mix.right.dt.b"), ch)
-        L.scan = SelectiveScan(ch, N, _padded(-torch.exp(take("mix.right.A_log")), ch, N), _padded(take("mix.right.D"), ch), s.mixer.right_scale)
+        L.w_dt = _padded(take("mix.right.dt"), ch, R)
+        L.scan = SelectiveScan(ch, N, _padded(-torch.exp(take("mix.right.A_log")), ch, N), _padded(take("mix.right.D"), ch),
+                               _padded(take("mix.right.dt.b"), ch), s.mixer.right_scale)
         wl, wr = take("mix.left.o"), take("mix.right.o")
         L.y_col = up(wl.shape[1])                             # the scan's first column
         L.w_o = torch.zeros(wl.shape[0], L.y_col + ch, dtype=wl.dtype, device=wl.device)
@@ -440,7 +441,7 @@ class ZomavikModel:
         xc = ops.causal_conv(x, L.conv_w, cache.state["conv"][r], b.seq_slots, b.positions, b.q_start, L.conv_b)
         low = ops.linear(xc, L.w_x)                           # dt | B | C
         R = L.w_dt.shape[1]
-        dt = ops.linear(low[:, :R], L.w_dt, residual=L.b_dt.expand(T, -1), out_dtype=torch.float32)
+        dt = ops.linear(low[:, :R], L.w_dt)
         ops.selective_scan(m, xc, z, low[:, R:], dt, cache.state["scan"][r], b.seq_slots, b.positions, b.q_start, single, y[:, L.y_col:])
         return ops.linear(y, L.w_o)
 

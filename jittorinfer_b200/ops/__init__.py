@@ -97,7 +97,7 @@ def mla_attention(q, cache, block_tables, seq_lens, q_start, scale, r, block_siz
 
 def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_shared=0, group_top2=False, route=None, pre_norm=None,
              logit_bias=None, shared_gate=False):
-    """``shared_gate``: the last row of ``w_router`` is the shared experts' gate, not an expert: their weight is its sigmoid (``n_shared``
+    """``w_router`` fp32, or bf16 with bf16 activations (products of exact operands on the tensor cores, fp32 sums).  ``shared_gate``: the last row of ``w_router`` is the shared experts' gate, not an expert: their weight is its sigmoid (``n_shared``
     columns), and the router outputs' last column is returned as well.
     ``route=(expert_base, E_local)`` tells the CUDA path which local expert sort follows (see ``native.moe_gate``).
     ``pre_norm=(weight, eps)``: ``g`` is the un-normalised block input; returns (ids, wts, rmsnorm(g) * weight) -- on the CUDA
@@ -183,7 +183,7 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
 
 
 def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
-    """``m``: ``specs.SelectiveScan``; ``bc`` = B | C, ``dt`` fp32 pre-activations of the step sizes; result columns go to ``out`` (a view)."""
+    """``m``: ``specs.SelectiveScan``; ``bc`` = B | C, ``dt`` the step sizes' projection; result columns go to ``out`` (a view)."""
     return (nat() if use_native(x) else ref).selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out)
 
 

@@ -91,7 +91,7 @@ class GqaDesc(C.Structure):
 
 
 class ScanDesc(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("x", "z", "bc", "dt", "y", "neg_a", "skip", "state", "seq_slots", "positions", "q_start", "status")] + \
+    _fields_ = [(n, C.c_void_p) for n in ("x", "z", "bc", "dt", "y", "neg_a", "skip", "dt_bias", "state", "seq_slots", "positions", "q_start", "status")] + \
                [(n, C.c_longlong) for n in ("ldx", "ldz", "ldbc", "lddt", "ldy")] + \
                [(n, C.c_int) for n in ("ch", "N", "n_state", "n_seqs", "T")] + [("out_scale", C.c_float)]
 
@@ -551,6 +551,8 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
     else:
         pre_norm_k = pre_norm
     E = w_router.shape[0]
+    by_gemm = w_router.dtype == torch.bfloat16          # a router kept in bf16: its outputs come from the tensor cores
+    fused = fused and not by_gemm
     ids = torch.empty(T, k + n_shared, dtype=torch.int32, device=g.device)
     wts = torch.empty(T, k + n_shared, dtype=torch.float32, device=g.device)
     logits = torch.empty(T, E, dtype=torch.float32, device=g.device)
@@ -571,8 +573,10 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
         _route_stash.clear()                       # at most one pending result: the sort that follows this gate
         _route_stash[(ids.data_ptr(), expert_base, E_local)] = (seg, src, dest, ids)
         return (ids, wts, g_out if g_out is not None else g_pre) if pre_norm is not None else (ids, wts)
-    own = g.dtype == torch.bfloat16 and d % 8 == 0 and d <= 8192          # the router kernel; else fp32 products of the library
-    if not own:
+    own = g.dtype == torch.bfloat16 and not by_gemm and d % 8 == 0 and d <= 8192      # the router kernel; else fp32 products of the library
+    if by_gemm:
+        gemm(g, w_router, out=logits)
+    elif not own:
         torch.matmul(g.float(), w_router.T, out=logits)
     _ck(load().jib_moe_gate(g.data_ptr() if own else None, w_router.data_ptr(), _p(bias), _p(logit_bias), logits.data_ptr(), ids.data_ptr(), wts.data_ptr(), T, d,
                             E, k, n_group, topk_group, float(scale), int(norm), int(sigmoid), n_shared, int(group_top2), int(shared_gate), _stream()),
@@ -832,13 +836,14 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
 
 def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
     T = x.shape[0]
-    assert x.dtype == z.dtype == bc.dtype == out.dtype and dt.dtype == state.dtype == torch.float32 and state.is_contiguous()
+    assert x.dtype == z.dtype == bc.dtype == dt.dtype == out.dtype and state.dtype == torch.float32 and state.is_contiguous()
     assert x.stride(1) == z.stride(1) == bc.stride(1) == dt.stride(1) == out.stride(1) == 1 and m.neg_a.is_contiguous()
     cd = ScanDesc()
     for name, t in (("x", x), ("z", z), ("bc", bc), ("dt", dt), ("y", out)):
         setattr(cd, name, t.data_ptr())
         setattr(cd, "ld" + name, t.stride(0))
     cd.neg_a, cd.skip, cd.state, cd.status = m.neg_a.data_ptr(), m.skip.data_ptr(), state.data_ptr(), workspace(x.device).status.data_ptr()
+    cd.dt_bias = m.dt_bias.data_ptr()
     cd.seq_slots, cd.positions, cd.q_start = seq_slots.data_ptr(), positions.data_ptr(), q_start.data_ptr()
     cd.ch, cd.N, cd.n_state, cd.n_seqs, cd.T, cd.out_scale = m.channels, m.state, state.shape[0], q_start.shape[0] - 1, T, m.out_scale
     _ck(load().jib_selective_scan(C.byref(cd), int(single), int(x.dtype == torch.float32), _stream()), "selective_scan")

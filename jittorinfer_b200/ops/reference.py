@@ -475,7 +475,7 @@ def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single
             continue
         slot = int(seq_slots[b])
         S = state[slot].clone() if slot >= 0 and int(positions[q0]) > 0 else torch.zeros_like(m.neg_a)
-        xs, BC, d = x[q0:q1].float(), bc[q0:q1].float(), _softplus(dt[q0:q1].float())
+        xs, BC, d = x[q0:q1].float(), bc[q0:q1].float(), _softplus(dt[q0:q1].float() + m.dt_bias)
         a, u = torch.exp(d[..., None] * m.neg_a), (d * xs)[..., None] * BC[:, None, :N]
         y = torch.empty_like(xs)
         for t in range(q1 - q0):

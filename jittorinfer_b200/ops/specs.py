@@ -68,12 +68,13 @@ class Gqa:
 @dataclass
 class SelectiveScan:
     """A state-space recurrence with a decay per channel and state: S[c, n] <- exp(dt_c neg_a[c, n]) S[c, n] + dt_c x_c B_n,
-    y_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c) out_scale, dt = softplus(.).  ``channels`` and ``state`` are multiples of 8 (a model
+    y_c = (sum_n S[c, n] C_n + skip_c x_c) silu(z_c) out_scale, dt = softplus(. + dt_bias).  ``channels`` and ``state`` are multiples of 8 (a model
     pads with zero weights)."""
     channels: int
     state: int
     neg_a: torch.Tensor                         # [channels, state] fp32
-    skip: torch.Tensor                          # [channels]
+    skip: torch.Tensor                          # [channels] fp32
+    dt_bias: torch.Tensor                       # [channels] fp32
     out_scale: float = 1.0
 
 

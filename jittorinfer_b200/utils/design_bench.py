@@ -23,8 +23,14 @@ def sizes(design: str):
         dense = lambda n, d, h, ff: DeepSeek2HParams(n_layer=n, n_layer_dense_lead=n, n_embd=d, n_head=h, n_ff=ff)       # noqa: E731
         return [("width 2048, 16 heads of 128, feed-forward 5632, 12 layers", preset("lugovik-lite"), dense(12, 2048, 16, 5632)),
                 ("width 4096, 32 heads of 128, feed-forward 11008, 8 layers", preset("lugovik-wide"), dense(8, 4096, 32, 11008))]
+    if design == "zomavik":
+        v2 = DeepSeek2HParams(n_layer=4, n_layer_dense_lead=0, n_embd=5120, n_head=128, n_ff_exp=1536, n_expert=160, expert_weights_scale=16.0,
+                              n_group=8, topk_group=3, q_lora_rank=1536)
+        return [("width 2048, 16 heads, 64 experts top-6 of 1408 + 2 shared, 12 layer runs", preset("zomavik-lite"),
+                 DeepSeek2HParams(n_layer=12, n_layer_dense_lead=0)),
+                ("width 5120, 40 heads (closest: 128), 160 experts top-6 of 1536 + 2 shared, 4 layer runs", preset("zomavik-v2"), v2)]
     if design != "nibalix":
-        raise SystemExit(f"unknown design {design!r} (known: nibalix, lugovik)")
+        raise SystemExit(f"unknown design {design!r} (known: nibalix, lugovik, zomavik)")
     lite = DeepSeek2HParams(n_layer=12, n_layer_dense_lead=0, n_expert_shared=0)
     v2 = DeepSeek2HParams(n_layer=4, n_layer_dense_lead=0, n_expert_shared=0, n_embd=5120, n_head=128, n_ff_exp=1536, n_expert=160,
                           expert_weights_scale=16.0, n_group=8, topk_group=3, q_lora_rank=1536)
@@ -112,7 +118,7 @@ def run(args, sampler=None) -> int:
     out = {"metric": f"{args.design}: decode output tokens/s at concurrency 8, first size", "value": head["tokens_per_s"], "unit": "tokens/s",
            "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup), "ms_per_step": head["ms_per_step"], "higher_is_better": True,
            "vs_baseline": None, "dtype": "bf16", "data": "synthetic (uniform-random token ids, random weights)", "impl": "ours",
-           "config": {"prompt_len": args.prompt_len, "closest": "DeepSeek-V2 layers of equal sizes" + (", dense feed-forwards" if args.design == "lugovik" else ", no shared experts"),
+           "config": {"prompt_len": args.prompt_len, "closest": "DeepSeek-V2 layers of equal sizes" + {"lugovik": ", dense feed-forwards", "nibalix": ", no shared experts"}.get(args.design, ""),
                       "l2": "weights exceed L2; no flush needed"},
            "gpu_launches": launches, "sizes": recs}
     if sampler is not None:
