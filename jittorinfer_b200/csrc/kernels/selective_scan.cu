@@ -8,9 +8,9 @@
 //   scan_portions  ranges of any length: a CTA owns 128 / L channels of one sequence, keeps their states in registers and walks the
 //                  tokens in tiles of TT, the next tile's inputs on their way while one is worked on
 //
-// The exponentials do not depend on the state, so a token costs its lane one multiply-add of latency.  Tokens go in groups of 8: the
-// lanes' partial sums of a group meet in one butterfly that leaves each lane with the sums of some of the tokens, and it runs
-// under the next group's exponentials.
+// The exponentials do not depend on the state, so a token costs its lane one multiply-add of latency.  Tokens go in groups of 8: while
+// a group's recurrence runs the next one's decays and inputs are computed, and the lanes' partial sums meet in one butterfly that
+// leaves each lane with the sums of some of the tokens.  A bf16 tile is one straight line of code.
 //
 // A sequence's state lives in row seq_slots[b] of [n_state][ch][N]; a range that starts at position 0 starts from zeros whatever the
 // row holds.  Sequence b owns token rows q_start[b] .. q_start[b + 1].  Activations bf16 or fp32, the rest fp32.
@@ -87,17 +87,20 @@ __device__ __forceinline__ F2 mul2(F2 a, F2 b) {
     asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
     return r;
 }
-// advance() of two states
-template <typename T> __device__ __forceinline__ F2 advance2(F2 v, F2 s, F2 u);
-template <> __device__ __forceinline__ F2 advance2<bf16>(F2 v, F2 s, F2 u) {
+// the decays of two states, and their next values; fp32 decays are kept as the exponent (see advance)
+template <typename T> __device__ __forceinline__ F2 decay2(F2 v);
+template <> __device__ __forceinline__ F2 decay2<bf16>(F2 v) {
     float2 e = unpack(v);
-    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.x));
-    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.y));
-    return fma2(pack(e.x, e.y), s, u);
+    asm volatile("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.x));        // stays where it is written, ahead of its use
+    asm volatile("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.y));
+    return pack(e.x, e.y);
 }
-template <> __device__ __forceinline__ F2 advance2<float>(F2 v, F2 s, F2 u) {
-    const float2 e = unpack(v), x = unpack(s), y = unpack(u);
-    return pack(advance<float>(e.x, x.x, y.x), advance<float>(e.y, x.y, y.y));
+template <> __device__ __forceinline__ F2 decay2<float>(F2 v) { return v; }
+template <typename T> __device__ __forceinline__ F2 next2(F2 e, F2 s, F2 u);
+template <> __device__ __forceinline__ F2 next2<bf16>(F2 e, F2 s, F2 u) { return fma2(e, s, u); }
+template <> __device__ __forceinline__ F2 next2<float>(F2 e, F2 s, F2 u) {
+    const float2 v = unpack(e), x = unpack(s), y = unpack(u);
+    return pack(advance<float>(v.x, x.x, y.x), advance<float>(v.y, x.y, y.y));
 }
 
 // 4 adjacent elements, kept as stored until they are needed (many loads in flight)
@@ -106,6 +109,10 @@ template <> struct Quad<float> {
     float4 r;
     __device__ __forceinline__ void zero() { r = make_float4(0.f, 0.f, 0.f, 0.f); }
     __device__ __forceinline__ void load(const float * p) { r = *(const float4 *) p; }
+    // not moved towards the use
+    __device__ __forceinline__ void request(const float * p) {
+        asm volatile("ld.global.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(r.x), "=f"(r.y), "=f"(r.z), "=f"(r.w) : "l"(p));
+    }
     __device__ __forceinline__ float4 get() const { return r; }
     __device__ __forceinline__ static void store(float * p, float4 v) { *(float4 *) p = v; }
 };
@@ -113,6 +120,7 @@ template <> struct Quad<bf16> {
     uint2 r;
     __device__ __forceinline__ void zero() { r = make_uint2(0, 0); }
     __device__ __forceinline__ void load(const bf16 * p) { r = *(const uint2 *) p; }
+    __device__ __forceinline__ void request(const bf16 * p) { asm volatile("ld.global.v2.u32 {%0, %1}, [%2];" : "=r"(r.x), "=r"(r.y) : "l"(p)); }
     __device__ __forceinline__ float4 get() const {
         const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &r.x), y = __bfloat1622float2(*(const __nv_bfloat162 *) &r.y);
         return make_float4(x.x, x.y, y.x, y.y);
@@ -124,17 +132,38 @@ template <> struct Quad<bf16> {
         *(uint2 *) p = o;
     }
 };
-// NS adjacent floats, NS a multiple of 4
+// NS adjacent floats, NS 2 or a multiple of 4
 template <int NS> __device__ __forceinline__ void load_n(const float * p, float (&v)[NS]) {
+    if constexpr (NS == 2) {
+        const float2 x = *(const float2 *) p;
+        v[0] = x.x; v[1] = x.y;
+    } else {
 #pragma unroll
-    for (int i = 0; i < NS; i += 4) {
-        const float4 x = *(const float4 *) (p + i);
-        v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
+        for (int i = 0; i < NS; i += 4) {
+            const float4 x = *(const float4 *) (p + i);
+            v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
+        }
     }
 }
 template <int NS> __device__ __forceinline__ void store_n(float * p, const float (&v)[NS]) {
+    if constexpr (NS == 2) {
+        *(float2 *) p = make_float2(v[0], v[1]);
+    } else {
 #pragma unroll
-    for (int i = 0; i < NS; i += 4) *(float4 *) (p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+        for (int i = 0; i < NS; i += 4) *(float4 *) (p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    }
+}
+template <int H> __device__ __forceinline__ void load_pairs(const float * p, F2 (&v)[H]) {
+    if constexpr (H == 1) {
+        v[0].v = *(const unsigned long long *) p;
+    } else {
+#pragma unroll
+        for (int i = 0; i < H; i += 2) {
+            const ulonglong2 x = *(const ulonglong2 *) (p + 2 * i);
+            v[i].v = x.x;
+            v[i + 1].v = x.y;
+        }
+    }
 }
 
 __device__ __forceinline__ int checked_slot(const jib_scan & a, int b, int site) {
@@ -220,9 +249,9 @@ struct Scan {
             x[i].zero(); z[i].zero(); dt[i].zero();
             if (q < QX && t < n && c < a.ch) {
                 const size_t r = q0 + t;
-                x[i].load((const T *) a.x + r * a.ldx + c);
-                z[i].load((const T *) a.z + r * a.ldz + c);
-                dt[i].load((const T *) a.dt + r * a.lddt + c);
+                x[i].request((const T *) a.x + r * a.ldx + c);
+                z[i].request((const T *) a.z + r * a.ldz + c);
+                dt[i].request((const T *) a.dt + r * a.lddt + c);
             }
         }
         const int n4 = a.N / 2;                              // quads of a row of B | C
@@ -230,7 +259,7 @@ struct Scan {
         for (int i = 0; i < RB; ++i) {
             const int q = threadIdx.x + i * NT, k = q / n4, t = t0 + k;
             bc[i].zero();
-            if (k < TT && t < n) bc[i].load((const T *) a.bc + (size_t) (q0 + t) * a.ldbc + (q - k * n4) * 4);
+            if (k < TT && t < n) bc[i].request((const T *) a.bc + (size_t) (q0 + t) * a.ldbc + (q - k * n4) * 4);
         }
     }
 };
@@ -255,7 +284,7 @@ template <int L> __device__ __forceinline__ void meet(float (&p)[8], int lane) {
 }
 
 template <typename T, int NS, int L>
-__global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant__ jib_scan a) {
+__global__ void __launch_bounds__(NT, NS >= 8 ? 1 : 3) scan_portions_kernel(const __grid_constant__ jib_scan a) {
     using S = Scan<T, NS, L>;
     constexpr int NP = S::NP, CH = S::CH, TT = S::TT, G = S::G, W = L < 8 ? L : 8, H = NS / 2;
     extern __shared__ __align__(16) float smem[];
@@ -319,35 +348,56 @@ __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant
         __syncthreads();
         if (t0 + TT < n) nxt.load(a, q0, n, t0 + TT, c0);
         const int m = min(TT, n - t0);
-        float p[G], last[G];
-        auto out = [&](int g) {                              // the group whose sums are in last
-            meet<L>(last, lane);
-            if (lane < W) {
+        // decays and inputs of token t
+        auto prepare = [&](int t, F2 (&e)[H], F2 (&u)[H]) {
+            const ulonglong2 d = *(const ulonglong2 *) (sdx + t * CH + cl);
+            F2 B[H];
+            load_pairs<H>(sb + t * NP + n0, B);
 #pragma unroll
-                for (int k = 0; k < G / W; ++k) sy[(g + lane * (G / W) + k) * CH + cl] = last[k];
+            for (int i = 0; i < H; ++i) {
+                e[i] = decay2<T>(mul2({d.x}, ra[i]));
+                u[i] = mul2({d.y}, B[i]);
             }
         };
-#pragma unroll 1
-        for (int g = 0; g < m; g += G) {
-            if (g > 0) out(g - G);
+        constexpr int GROUPS = TT / G, UNROLL = sizeof(T) == 2 ? GROUPS : 1;
+        F2 e[G][H], u[G][H];
+        float sum[UNROLL][G / W];                            // this lane's tokens of every group
+        auto keep = [&](int g, const float * v) {
+            if (lane < W) {
+#pragma unroll
+                for (int k = 0; k < G / W; ++k) sy[(g * G + lane * (G / W) + k) * CH + cl] = v[k];
+            }
+        };
+#pragma unroll
+        for (int k = 0; k < G; ++k) prepare(k, e[k], u[k]);
+#pragma unroll UNROLL
+        for (int g = 0; g < GROUPS; ++g) {
+            float p[G];
 #pragma unroll
             for (int k = 0; k < G; ++k) {
-                const ulonglong2 d = *(const ulonglong2 *) (sdx + (g + k) * CH + cl);
-                F2 acc;
+                F2 acc, C[H];
+                load_pairs<H>(sc + (g * G + k) * NP + n0, C);
 #pragma unroll
                 for (int i = 0; i < H; ++i) {
-                    const F2 B = {*(const unsigned long long *) (sb + (g + k) * NP + n0 + 2 * i)};
-                    const F2 C = {*(const unsigned long long *) (sc + (g + k) * NP + n0 + 2 * i)};
-                    s[i] = advance2<T>(mul2({d.x}, ra[i]), s[i], mul2({d.y}, B));
-                    acc = i == 0 ? mul2(s[i], C) : fma2(s[i], C, acc);
+                    s[i] = next2<T>(e[k][i], s[i], u[k][i]);
+                    acc = i == 0 ? mul2(s[i], C[i]) : fma2(s[i], C[i], acc);
                 }
                 const float2 y = unpack(acc);
                 p[k] = y.x + y.y;
+                if (g + 1 < GROUPS) prepare((g + 1) * G + k, e[k], u[k]);
             }
+            meet<L>(p, lane);
+            if (UNROLL == 1) {
+                keep(g, p);
+            } else {                                         // stored at the end: no store between the loads of shared memory
 #pragma unroll
-            for (int k = 0; k < G; ++k) last[k] = p[k];
+                for (int k = 0; k < G / W; ++k) sum[g % UNROLL][k] = p[k];
+            }
         }
-        out((m - 1) / G * G);
+        if (UNROLL > 1) {
+#pragma unroll
+            for (int g = 0; g < UNROLL; ++g) keep(g, sum[g]);
+        }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < S::RX; ++i) {
@@ -375,28 +425,29 @@ __global__ void __launch_bounds__(NT) scan_portions_kernel(const __grid_constant
 inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH; }
 
 template <typename T, int NS, int L>
-int run(const jib_scan & a, int single, cudaStream_t s) {
+int step(const jib_scan & a, cudaStream_t s) {
     constexpr int CH = NT / L, U = sizeof(T) == 2 && NS == 4 ? 4 : 1;
     const unsigned gx = (a.ch + CH - 1) / CH;
-    if (single) {
-        if (U > 1 && a.T * gx > 148 * 8) JIB_LAUNCH((scan_step_kernel<T, NS, L, U>), dim3(gx, (a.T + U - 1) / U), NT, 0, s, a);
-        else JIB_LAUNCH((scan_step_kernel<T, NS, L, 1>), dim3(gx, a.T), NT, 0, s, a);
-        return launched();
-    }
-    constexpr int SMEM = Scan<T, NS, L>::SMEM;
+    if (U > 1 && a.T * gx > 148 * 8) JIB_LAUNCH((scan_step_kernel<T, NS, L, U>), dim3(gx, (a.T + U - 1) / U), NT, 0, s, a);
+    else JIB_LAUNCH((scan_step_kernel<T, NS, L, 1>), dim3(gx, a.T), NT, 0, s, a);
+    return launched();
+}
+template <typename T, int NS, int L>
+int portions(const jib_scan & a, cudaStream_t s) {
+    constexpr int CH = NT / L, SMEM = Scan<T, NS, L>::SMEM;
     static_assert(SMEM <= 48 * 1024, "fits without an attribute");
-    JIB_LAUNCH((scan_portions_kernel<T, NS, L>), dim3(gx, a.n_seqs), NT, SMEM, s, a);
+    JIB_LAUNCH((scan_portions_kernel<T, NS, L>), dim3((a.ch + CH - 1) / CH, a.n_seqs), NT, SMEM, s, a);
     return launched();
 }
 
 template <typename T>
 int dispatch(const jib_scan & a, int single, cudaStream_t s) {
-    if (a.N <= 8) return run<T, 4, 2>(a, single, s);
-    if (a.N <= 16) return run<T, 4, 4>(a, single, s);
-    if (a.N <= 32) return run<T, 4, 8>(a, single, s);
-    if (a.N <= 64) return run<T, 4, 16>(a, single, s);
-    if (a.N <= 128) return run<T, 4, 32>(a, single, s);
-    return run<T, 8, 32>(a, single, s);
+    if (a.N <= 8) return single ? step<T, 4, 2>(a, s) : portions<T, 2, 4>(a, s);
+    if (a.N <= 16) return single ? step<T, 4, 4>(a, s) : portions<T, 2, 8>(a, s);
+    if (a.N <= 32) return single ? step<T, 4, 8>(a, s) : portions<T, 4, 8>(a, s);
+    if (a.N <= 64) return single ? step<T, 4, 16>(a, s) : portions<T, 4, 16>(a, s);
+    if (a.N <= 128) return single ? step<T, 4, 32>(a, s) : portions<T, 4, 32>(a, s);
+    return single ? step<T, 8, 32>(a, s) : portions<T, 8, 32>(a, s);
 }
 
 }  // namespace

@@ -3,6 +3,8 @@
 ``config`` is the parsed model configuration, ``w`` maps tensor names to tensors.  Nothing of the package is used here.
 Everything runs in the dtype of the weights handed in (the tests use float32 or float64).
 """
+import math
+
 import torch
 
 
@@ -53,13 +55,12 @@ def attend(q, k, v, scale, softcap, sink):
     n, H, _ = q.shape
     rep = H // k.shape[1]
     out = torch.zeros(n, H, v.shape[2], dtype=q.dtype)
+    future = torch.ones(n, n, dtype=torch.bool).triu(1)
     for h in range(H):
-        kk, vv = k[:, h // rep], v[:, h // rep]
-        for i in range(n):
-            s = capped((kk[:i + 1] @ q[i, h]) * scale, softcap)
-            top = torch.maximum(s.max(), sink[h])
-            e = torch.exp(s - top)
-            out[i, h] = (e @ vv[:i + 1]) / (torch.exp(sink[h] - top) + e.sum())
+        s = capped((q[:, h] @ k[:, h // rep].T) * scale, softcap).masked_fill(future, -math.inf)
+        top = torch.maximum(s.max(-1).values, sink[h])[:, None]
+        e = torch.exp(s - top)
+        out[:, h] = (e @ v[:, h // rep]) / (torch.exp(sink[h] - top) + e.sum(-1, keepdim=True))
     return out
 
 
