@@ -372,9 +372,13 @@ __global__ void gather_rows_kernel(const bf16 * __restrict__ x, const int * __re
     const int s = src_row[rrow];
     JIB_BC(s < n_src, 13, s);
     if (s < 0 || s >= n_src) return;   // unowned / out-of-range row: leave the destination untouched
-    const uint4 * src = (const uint4 *) (x + (size_t) s * d);
-    uint4 * dst = (uint4 *) (out + (size_t) rrow * d);
-    for (int i = threadIdx.x; i < d / 8; i += blockDim.x) dst[i] = src[i];
+    if (d % 8 == 0) {
+        const uint4 * src = (const uint4 *) (x + (size_t) s * d);
+        uint4 * dst = (uint4 *) (out + (size_t) rrow * d);
+        for (int i = threadIdx.x; i < d / 8; i += blockDim.x) dst[i] = src[i];
+    } else {                           // rows that 16-byte vectors do not divide
+        for (int i = threadIdx.x; i < d; i += blockDim.x) out[(size_t) rrow * d + i] = x[(size_t) s * d + i];
+    }
     JIB_KS(7, 9);
 }
 
@@ -467,7 +471,6 @@ int jib_kv_block_copy(void * cache, long long layer_stride_elems, int n_layers, 
 
 int jib_gather_rows(const void * x, const int * src_row, void * out, int rows, int d, int n_src, void * stream) {
     if (rows <= 0) return 0;
-    if (d % 8) return JIB_E_ARG;
     JIB_LAUNCH((gather_rows_kernel), rows, 128, 0, (cudaStream_t) stream, (const bf16 *) x, src_row, (bf16 *) out, d, n_src);
     return launched();
 }
