@@ -10,7 +10,8 @@
 //
 // The exponentials do not depend on the state, so a token costs its lane one multiply-add of latency.  Tokens go in groups of 8: while
 // a group's recurrence runs the next one's decays and inputs are computed, and the lanes' partial sums meet in one butterfly that
-// leaves each lane with the sums of some of the tokens.  A bf16 tile is one straight line of code.
+// leaves each lane with the sums of some of the tokens.  A bf16 tile is one straight line of code.  Shared memory's bandwidth is the
+// tightest resource (a load moves a warp's full width even where lanes share an address), so B and C stay bf16 there.
 //
 // A sequence's state lives in row seq_slots[b] of [n_state][ch][N]; a range that starts at position 0 starts from zeros whatever the
 // row holds.  Sequence b owns token rows q_start[b] .. q_start[b + 1].  Activations bf16 or fp32, the rest fp32.
@@ -91,8 +92,8 @@ __device__ __forceinline__ F2 mul2(F2 a, F2 b) {
 template <typename T> __device__ __forceinline__ F2 decay2(F2 v);
 template <> __device__ __forceinline__ F2 decay2<bf16>(F2 v) {
     float2 e = unpack(v);
-    asm volatile("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.x));        // stays where it is written, ahead of its use
-    asm volatile("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.y));
+    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.x));
+    asm("ex2.approx.ftz.f32 %0, %0;" : "+f"(e.y));
     return pack(e.x, e.y);
 }
 template <> __device__ __forceinline__ F2 decay2<float>(F2 v) { return v; }
@@ -165,6 +166,44 @@ template <int H> __device__ __forceinline__ void load_pairs(const float * p, F2 
         }
     }
 }
+
+// B and C of a tile in shared memory, a lane's NS states of both adjacent (row: L times NS of B, NS of C), as stored: bf16 halves the traffic
+template <typename T, int NS> struct Operands;
+template <int NS> struct Operands<float, NS> {
+    static __device__ __forceinline__ void put(float * row, int col, bool is_c, const Quad<float> & v) {
+        const float x[4] = {v.r.x, v.r.y, v.r.z, v.r.w};
+#pragma unroll
+        for (int i = 0; i < 4; i += 2) *(float2 *) (row + (col + i) / NS * 2 * NS + (is_c ? NS : 0) + (col + i) % NS) = make_float2(x[i], x[i + 1]);
+    }
+    static __device__ __forceinline__ void get(const float * p, F2 (&B)[NS / 2], F2 (&C)[NS / 2]) {
+        load_pairs<NS / 2>(p, B);
+        load_pairs<NS / 2>(p + NS, C);
+    }
+};
+template <int NS> struct Operands<bf16, NS> {
+    static __device__ __forceinline__ void put(bf16 * row, int col, bool is_c, const Quad<bf16> & v) {
+        *(uint32_t *) (row + col / NS * 2 * NS + (is_c ? NS : 0) + col % NS) = v.r.x;
+        *(uint32_t *) (row + (col + 2) / NS * 2 * NS + (is_c ? NS : 0) + (col + 2) % NS) = v.r.y;
+    }
+    static __device__ __forceinline__ void get(const bf16 * p, F2 (&B)[NS / 2], F2 (&C)[NS / 2]) {
+        uint32_t r[NS];
+        if constexpr (NS == 2) {
+            const uint2 x = *(const uint2 *) p;
+            r[0] = x.x; r[1] = x.y;
+        } else {
+#pragma unroll
+            for (int i = 0; i < NS; i += 4) {
+                const uint4 x = *(const uint4 *) (p + 2 * i);
+                r[i] = x.x; r[i + 1] = x.y; r[i + 2] = x.z; r[i + 3] = x.w;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NS / 2; ++i) {
+            B[i] = pack(__uint_as_float(r[i] << 16), __uint_as_float(r[i] & 0xffff0000u));
+            C[i] = pack(__uint_as_float(r[NS / 2 + i] << 16), __uint_as_float(r[NS / 2 + i] & 0xffff0000u));
+        }
+    }
+};
 
 __device__ __forceinline__ int checked_slot(const jib_scan & a, int b, int site) {
     const int slot = a.seq_slots[b];
@@ -239,7 +278,7 @@ struct Scan {
     static constexpr int G = 8;                              // tokens of a group
     static constexpr int QX = TT * CH / 4, QB = TT * 2 * NP / 4;                     // quads of a tile: per channel input, of B | C
     static constexpr int RX = (QX + NT - 1) / NT, RB = (QB + NT - 1) / NT;
-    static constexpr int SMEM = 4 * (TT * CH * 4 + TT * 2 * NP + TT * CH);
+    static constexpr int SMEM = TT * CH * 8 + TT * 2 * NP * (int) sizeof(T) + TT * CH * 4;
     Quad<T> x[RX], z[RX], dt[RX], bc[RB];
     // tokens t0 .. of the sequence's n, whose first row is q0
     __device__ __forceinline__ void load(const jib_scan & a, int q0, int n, int t0, int c0) {
@@ -288,8 +327,9 @@ __global__ void __launch_bounds__(NT, NS >= 8 ? 1 : 3) scan_portions_kernel(cons
     using S = Scan<T, NS, L>;
     constexpr int NP = S::NP, CH = S::CH, TT = S::TT, G = S::G, W = L < 8 ? L : 8, H = NS / 2;
     extern __shared__ __align__(16) float smem[];
-    float4 * sdx = (float4 *) smem;                          // [TT][CH]: step size twice, step size * x twice
-    float * sb = smem + TT * CH * 4, * sc = sb + TT * NP, * sy = sc + TT * NP;       // [TT][NP], [TT][NP], [TT][CH]
+    float2 * sdx = (float2 *) smem;                          // [TT][CH]: step size, step size * x
+    float * sy = smem + TT * CH * 2;                         // [TT][CH]
+    T * sbc = (T *) (sy + TT * CH);                          // [TT][2 NP], see Operands
     PDL_TRIGGER_TOP();
     const int lane = threadIdx.x % L, cl = threadIdx.x / L, c0 = blockIdx.x * CH, c = c0 + cl, b = blockIdx.y, n0 = lane * NS;
     const bool live = c < a.ch && n0 < a.N;
@@ -302,7 +342,7 @@ __global__ void __launch_bounds__(NT, NS >= 8 ? 1 : 3) scan_portions_kernel(cons
 #pragma unroll
         for (int i = 0; i < H; ++i) ra[i] = pack(rate<T>(v[2 * i]), rate<T>(v[2 * i + 1]));
     }
-    for (int i = threadIdx.x; i < TT * 2 * NP; i += NT) sb[i] = 0.f;                 // columns past N stay zero
+    for (int i = threadIdx.x; i < TT * 2 * NP; i += NT) put(sbc + i, 0.f);           // columns past N stay zero
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
     if (n <= 0) return;
@@ -333,34 +373,35 @@ __global__ void __launch_bounds__(NT, NS >= 8 ? 1 : 3) scan_portions_kernel(cons
             if (q >= S::QX) continue;
             const float4 x = cur.x[i].get(), d = cur.dt[i].get();
             const float xv[4] = {x.x, x.y, x.z, x.w}, dv[4] = {d.x + bias.x, d.y + bias.y, d.z + bias.z, d.w + bias.w};
+            float k[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float k = t0 + t < n ? softplus<T>(dv[e]) : 0.f;               // past the end: the state passes through
-                sdx[t * CH + cq + e] = make_float4(k, k, k * xv[e], k * xv[e]);
-            }
+            for (int e = 0; e < 4; ++e) k[e] = t0 + t < n ? softplus<T>(dv[e]) : 0.f;   // past the end: the state passes through
+            float4 * o = (float4 *) (sdx + t * CH + cq);
+            o[0] = make_float4(k[0], k[0] * xv[0], k[1], k[1] * xv[1]);
+            o[1] = make_float4(k[2], k[2] * xv[2], k[3], k[3] * xv[3]);
         }
         const int n4 = a.N / 2;
 #pragma unroll
         for (int i = 0; i < S::RB; ++i) {
             const int q = threadIdx.x + i * NT, t = q / n4, col = (q - t * n4) * 4;
-            if (t < TT) *(float4 *) ((col < a.N ? sb + col : sc + col - a.N) + t * NP) = cur.bc[i].get();
+            if (t < TT) Operands<T, NS>::put(sbc + t * 2 * NP, col < a.N ? col : col - a.N, col >= a.N, cur.bc[i]);
         }
         __syncthreads();
         if (t0 + TT < n) nxt.load(a, q0, n, t0 + TT, c0);
         const int m = min(TT, n - t0);
-        // decays and inputs of token t
-        auto prepare = [&](int t, F2 (&e)[H], F2 (&u)[H]) {
-            const ulonglong2 d = *(const ulonglong2 *) (sdx + t * CH + cl);
+        // decays, inputs and read-out weights of token t
+        auto prepare = [&](int t, F2 (&e)[H], F2 (&u)[H], F2 (&C)[H]) {
+            const float2 d = sdx[t * CH + cl];
             F2 B[H];
-            load_pairs<H>(sb + t * NP + n0, B);
+            Operands<T, NS>::get(sbc + t * 2 * NP + 2 * n0, B, C);
 #pragma unroll
             for (int i = 0; i < H; ++i) {
-                e[i] = decay2<T>(mul2({d.x}, ra[i]));
-                u[i] = mul2({d.y}, B[i]);
+                e[i] = decay2<T>(mul2(pack(d.x, d.x), ra[i]));
+                u[i] = mul2(pack(d.y, d.y), B[i]);
             }
         };
         constexpr int GROUPS = TT / G, UNROLL = sizeof(T) == 2 ? GROUPS : 1;
-        F2 e[G][H], u[G][H];
+        F2 e[G][H], u[G][H], C[G][H];
         float sum[UNROLL][G / W];                            // this lane's tokens of every group
         auto keep = [&](int g, const float * v) {
             if (lane < W) {
@@ -369,22 +410,21 @@ __global__ void __launch_bounds__(NT, NS >= 8 ? 1 : 3) scan_portions_kernel(cons
             }
         };
 #pragma unroll
-        for (int k = 0; k < G; ++k) prepare(k, e[k], u[k]);
+        for (int k = 0; k < G; ++k) prepare(k, e[k], u[k], C[k]);
 #pragma unroll UNROLL
         for (int g = 0; g < GROUPS; ++g) {
             float p[G];
 #pragma unroll
             for (int k = 0; k < G; ++k) {
-                F2 acc, C[H];
-                load_pairs<H>(sc + (g * G + k) * NP + n0, C);
+                F2 acc;
 #pragma unroll
                 for (int i = 0; i < H; ++i) {
                     s[i] = next2<T>(e[k][i], s[i], u[k][i]);
-                    acc = i == 0 ? mul2(s[i], C[i]) : fma2(s[i], C[i], acc);
+                    acc = i == 0 ? mul2(s[i], C[k][i]) : fma2(s[i], C[k][i], acc);
                 }
                 const float2 y = unpack(acc);
                 p[k] = y.x + y.y;
-                if (g + 1 < GROUPS) prepare((g + 1) * G + k, e[k], u[k]);
+                if (g + 1 < GROUPS) prepare((g + 1) * G + k, e[k], u[k], C[k]);
             }
             meet<L>(p, lane);
             if (UNROLL == 1) {
