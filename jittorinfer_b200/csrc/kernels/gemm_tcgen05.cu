@@ -153,9 +153,8 @@ __device__ __forceinline__ float gated(float x, int act) {
     return x / (1.0f + __expf(-z));
 }
 
-// JIB_UNARY_* of a single product; softcap y = c tanh(s v / c) with tanh(u) = 1 - 2 / (1 + e^{2u})
+// JIB_UNARY_* of a single product (FN instances: the plain kernels stay free of it); softcap y = c tanh(s v / c) with tanh(u) = 1 - 2 / (1 + e^{2u})
 __device__ __forceinline__ float unary(float v, const GemmArgs & a) {
-    if (a.unary == JIB_UNARY_NONE) return v;
     if (a.unary == JIB_UNARY_RELU2) return v > 0.f ? v * v : 0.f;
     if (a.softcap <= 0.f) return v * a.scale;
     return a.softcap * (1.f - __fdividef(2.f, 1.f + __expf(fminf(v * a.cap2, 80.f))));
@@ -173,7 +172,7 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t local_smem_addr, uint32_t
     return v;
 }
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool FN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA2,
             const __grid_constant__ CUtensorMap tmB, const GemmArgs args) {
@@ -395,7 +394,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         }
         // One finished element: feature n of row (row_base + t_rel); gv / uv are the summed accumulators.
         auto finish = [&](int t_rel, float gv, float uv) {
-            float y = DUAL ? gated(gv, args.act) * uv : unary(gv, args);
+            float y = DUAL ? gated(gv, args.act) * uv : FN ? unary(gv, args) : gv;
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
@@ -572,7 +571,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     const int ltid = (int) threadIdx.x - 64;
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : unary(g[j], args);
+                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : FN ? unary(g[j], args) : g[j];
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -729,7 +728,7 @@ __device__ __forceinline__ bool ptile_decode(const GemmArgs & args, int item, in
     return t.row0 < t.rows_valid;
 }
 
-template <int BN, bool DUAL>
+template <int BN, bool DUAL, bool FN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA2,
                        const __grid_constant__ CUtensorMap tmB, const GemmArgs args, const int n_x, const int n_y, const int n_items) {
@@ -861,7 +860,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
-                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : unary(g, args);
+                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : FN ? unary(g, args) : g;
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
@@ -1019,14 +1018,33 @@ int auto_splits(long long base_ctas, int num_kb, int bn, int sms) {
     return splits;
 }
 
-template <int BN, bool DUAL>
-int launch(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid,
+template <int BN, bool DUAL, bool FN>
+int launch_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid,
            cudaStream_t stream) {
     using C = Cfg<BN, DUAL>;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(gemm_kernel<BN, DUAL>, C::SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;
-    const cudaError_t e = jib::launch_pdl_cluster(gemm_kernel<BN, DUAL>, grid, dim3(NUM_THREADS), C::SMEM_BYTES, stream,
+    if (!jib::ensure_dyn_smem(gemm_kernel<BN, DUAL, FN>, C::SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;
+    const cudaError_t e = jib::launch_pdl_cluster(gemm_kernel<BN, DUAL, FN>, grid, dim3(NUM_THREADS), C::SMEM_BYTES, stream,
                                                   args.cluster_split ? args.splits : 1, a, a2, b, args);
+    if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
+    return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
+}
+
+template <int BN, bool DUAL>
+int launch(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid, cudaStream_t stream) {
+    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_as<BN, DUAL, !DUAL>(a, a2, b, args, grid, stream);
+    return launch_as<BN, DUAL, false>(a, a2, b, args, grid, stream);
+}
+
+template <int BN, bool DUAL, bool FN>
+int launch_persistent_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, int n_x, int n_y,
+                      long long n_items, int sms, cudaStream_t stream) {
+    using C = PCfg<BN, DUAL>;
+    static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
+    if (!jib::ensure_dyn_smem(gemm_persistent_kernel<BN, DUAL, FN>, C::SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;
+    const int grid = (int) (n_items < sms ? n_items : sms);
+    const cudaError_t e = jib::launch_pdl(gemm_persistent_kernel<BN, DUAL, FN>, dim3(grid), dim3(NUM_THREADS), C::SMEM_BYTES, stream, a, a2, b, args,
+                                          n_x, n_y, (int) n_items);
     if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
@@ -1034,14 +1052,8 @@ int launch(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b,
 template <int BN, bool DUAL>
 int launch_persistent(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, int n_x, int n_y,
                       long long n_items, int sms, cudaStream_t stream) {
-    using C = PCfg<BN, DUAL>;
-    static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(gemm_persistent_kernel<BN, DUAL>, C::SMEM_BYTES, attr_done)) return JIB_E_LAUNCH;
-    const int grid = (int) (n_items < sms ? n_items : sms);
-    const cudaError_t e = jib::launch_pdl(gemm_persistent_kernel<BN, DUAL>, dim3(grid), dim3(NUM_THREADS), C::SMEM_BYTES, stream, a, a2, b, args,
-                                          n_x, n_y, (int) n_items);
-    if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
-    return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
+    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_persistent_as<BN, DUAL, !DUAL>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
+    return launch_persistent_as<BN, DUAL, false>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
 }
 
 // JIB_GEMM_PERSIST=0: launches with several waves of tiles use the one-tile-per-CTA kernel as well (A/B measurements).

@@ -46,7 +46,7 @@ template <typename T> __device__ __forceinline__ float silu(float g) { return g 
 // of the channels.  Up to CONV_TAPS taps only a sequence's first run reaches back to the stored rows: it loads every row once,
 // slides over them in registers and then, as their only reader, replaces the stored rows by the range's last ones.  Longer
 // filters go token by token; there the first token's CTA computes the first taps - 1 tokens for the same reason.
-constexpr int CONV_RUN = 8, CONV_TAPS = 4, CONV_NT = 128;
+constexpr int CONV_RUN = 4, CONV_TAPS = 4, CONV_NT = 128;
 static_assert(CONV_RUN >= CONV_TAPS - 1, "only the first run may reach back to the stored rows");
 
 // Run c of the batch -> (sequence, run inside it): sequence b's runs start at index q_start[b] / CONV_RUN + b, which leaves room for
