@@ -23,6 +23,7 @@ class Rotation:
     dims: int
     base: float
     yarn: Optional[Yarn] = None
+    stretch: float = 1.0             # every frequency is divided by it
 
 
 def fits(shape: Sequence[int], want: Sequence[Optional[int]]) -> bool:
@@ -53,9 +54,9 @@ def checked_tensors(directory: str, table: Dict[str, Tuple[Optional[int], ...]],
 
 
 def rope_table(n_pos: int, rot: Rotation, device) -> torch.Tensor:
-    """[n_pos, dims / 2, 2] fp32 (cos, sin), with YaRN's blend of stretched and plain frequencies and its magnitude factor."""
+    """[n_pos, dims / 2, 2] fp32 (cos, sin), with linear stretching or YaRN's blend of stretched and plain frequencies and its magnitude factor."""
     i = torch.arange(rot.dims // 2, dtype=torch.float64)
-    f, mult = rot.base ** (-2.0 * i / rot.dims), 1.0
+    f, mult = rot.base ** (-2.0 * i / rot.dims) / rot.stretch, 1.0
     if rot.yarn is not None:
         y = rot.yarn
         at = lambda turns: rot.dims * math.log(y.original / (2 * math.pi * turns)) / (2 * math.log(rot.base))       # noqa: E731

@@ -10,7 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Any, Callable, Dict, Optional
 
-from . import lugovik, nibalix, zomavik
+from . import lugovik, nibalix, rupatar, zomavik
 from .deepseek2 import DeepSeek2Model
 from .hparams import ARCH as DEEPSEEK2, DeepSeek2HParams
 from .hparams import preset as _deepseek2_preset
@@ -37,6 +37,8 @@ ARCHITECTURES: Dict[str, Architecture] = {
                                lugovik.iter_checkpoint, lugovik.iter_random),
     zomavik.ARCH: Architecture(zomavik.ARCH, zomavik.ZomavikHParams, zomavik.ZomavikModel, zomavik.preset, zomavik.load_config,
                                zomavik.iter_checkpoint, zomavik.iter_random),
+    rupatar.ARCH: Architecture(rupatar.ARCH, rupatar.RupatarHParams, rupatar.RupatarModel, rupatar.preset, rupatar.load_config,
+                               rupatar.iter_checkpoint, rupatar.iter_random),
 }
 
 

@@ -57,7 +57,7 @@ def rmsnorm(x, w, eps, residual=None):
 
 
 def linear(x, w, residual=None, out_dtype=None, unary=None):
-    """f(x w^T) + residual (a bias: one row expanded over the tokens); ``unary``: None, ("relu2",) or ("cap", scale, softcap)."""
+    """f(x w^T) + residual (a bias: one row expanded over the tokens); ``unary``: None, ("relu2",), ("gelu",) or ("cap", scale, softcap)."""
     if use_native(x) and x.dtype == torch.bfloat16:
         return nat().linear(x, w, residual, out_dtype, unary)
     return ref.linear(x, w, residual, out_dtype, unary)
@@ -112,7 +112,8 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
 
 
 def moe_routed(x, ids, wts, wg, wu, wd):
-    """(expert outputs of the (token, choice) pairs, row of each pair); the weighted sum is the caller's (``block_update``)."""
+    """(expert outputs of the (token, choice) pairs, row of each pair); the weighted sum is the caller's (``block_update``).  ``wg`` None: experts
+    without a gate, gelu(w x up^T) down^T -- the weight multiplies their input, the sum of the outputs is the result."""
     return (nat() if use_native(x) else ref).moe_routed(x, ids, wts, wg, wu, wd)
 
 
@@ -158,13 +159,13 @@ def block_update(x, mult, o, gates, b1, b2, moe=None, nxt=None):
 
 def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=None, dtype=None):
     """(x + s1 * o + s2 * (combine(moe) + sigmoid(dense_gate) * dense), h, h2); ``o``, ``moe`` = (rows, row of each pair, weights) and
-    ``dense`` may be None, ``dense_gate`` [T] None is a factor of one; ``dtype``: activation type (default: that of the sublayers' rows); x may be
+    ``dense`` may be None, ``s1``, ``s2``, the weights or ``dense_gate`` [T] None is a factor of one; ``dtype``: activation type (default: that of the sublayers' rows); x may be
     overwritten."""
     return (nat() if use_native(x) else ref).scaled_update(x, o, s1, s2, moe, dense, dense_gate, nxt, dtype)
 
 
-def rms_rows(x, rows, w, eps, dtype):
-    return (nat() if use_native(x) else ref).rms_rows(x, rows, w, eps, dtype)
+def rms_rows(x, rows, w, eps, dtype, groups=1):
+    return (nat() if use_native(x) else ref).rms_rows(x, rows, w, eps, dtype, groups)
 
 
 def causal_conv(h, w, state, seq_slots, positions, q_start, bias=None):
@@ -177,9 +178,10 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 
 
 # ---- mixers described by a spec (ops/specs.py) ------------------------------------------------------------------------------------
-def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
-    """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view)."""
-    return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out)
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top=None):
+    """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view).  ``state`` [n, heads,
+    dim, m.cols] fp32.  "mlstm": ``dec_in`` [T, 2 heads] fp32 = input | forget gates' pre-activations, ``top`` [n, heads] fp32."""
+    return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top)
 
 
 def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):
@@ -187,13 +189,15 @@ def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single
     return (nat() if use_native(x) else ref).selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out)
 
 
-def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
-    return (nat() if use_native(q) else ref).gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache)
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache, v_first=None, pooled=None):
+    """``v_first``: the values that ``m.v_mix`` mixes in.  ``pooled`` (with ``m.pool``): (pooled rows, block tables, seq_lens, q_start, block size, one
+    token per sequence); the means of the blocks that are now complete are stored as well."""
+    return (nat() if use_native(q) else ref).gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache, v_first, pooled)
 
 
-def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
-    """Result columns go to ``out`` (a view)."""
-    return (nat() if use_native(q) else ref).gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out)
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out, pool=None):
+    """Result columns go to ``out`` (a view); ``pool``: the pooled rows of ``m.pool``."""
+    return (nat() if use_native(q) else ref).gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out, pool)
 
 
 def argmax(logits):

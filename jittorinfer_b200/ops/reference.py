@@ -31,9 +31,11 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, residual: Optional[tor
 
 
 def unary_of(y: torch.Tensor, unary) -> torch.Tensor:
-    """None, ("relu2",): max(y, 0)^2, or ("cap", s, c): c tanh(s y / c), s y with c = 0."""
+    """None, ("relu2",): max(y, 0)^2, ("gelu",): the exact gelu, or ("cap", s, c): c tanh(s y / c), s y with c = 0."""
     if unary is None:
         return y
+    if unary[0] == "gelu":
+        return F.gelu(y.float())
     if unary[0] == "relu2":
         return torch.relu(y).square()
     y = y.float() * unary[1]
@@ -278,18 +280,27 @@ def kv_block_copy(cache: torch.Tensor, src_blocks: torch.Tensor, dst_blocks: tor
 
 
 def moe_routed(x, ids, wts, wg, wu, wd):
-    """Expert outputs of every (token, choice) pair: (y [T*k, d], dest [T, k] row of each pair); here in pair order."""
+    """Expert outputs of every (token, choice) pair: (y [T*k, d], dest [T, k] row of each pair); here in pair order.  ``wg`` None: experts
+    gelu(w x up^T) down^T, the weight on their input."""
     T, k = ids.shape
     y = torch.zeros(T * k, x.shape[1], dtype=x.dtype, device=x.device)
     flat = ids.reshape(-1).long()
-    for e in range(wg.shape[0]):
+    for e in range(wu.shape[0]):
         rows = torch.nonzero(flat == e).reshape(-1)
-        if rows.numel():
+        if rows.numel() and wg is None:
+            u = linear(x[rows // k], wu[e], out_dtype=torch.float32) * wts.reshape(-1)[rows][:, None]
+            y[rows] = linear(F.gelu(u).to(x.dtype), wd[e])
+        elif rows.numel():
             y[rows] = linear(gateup_silu(x[rows // k], wg[e], wu[e]), wd[e])
     return y, torch.arange(T * k, dtype=torch.int32, device=x.device).view(T, k)
 
 
 # ---- blocks over an fp32 residual stream whose sublayers read one norm (csrc/kernels/parallel_block.cu) ------------------------
+def _group_rms(x, groups, eps):
+    v = x.reshape(x.shape[0], groups, -1)
+    return (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape)
+
+
 def _finish_row(x, nxt, dtype):
     """x fp32 -> (x, h, hc) for ``nxt`` = (norm weight, eps, conv) with conv = None or (w [taps, d], state, seq_slots, positions), or a
     ``RowNorms``."""
@@ -298,7 +309,7 @@ def _finish_row(x, nxt, dtype):
     if isinstance(nxt, RowNorms):
         if nxt.w1 is None:
             return x, x.to(dtype, copy=True), None
-        n = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + nxt.eps)
+        n = _group_rms(x, nxt.groups, nxt.eps)
         return x, (n * nxt.w1).to(dtype), None if nxt.w2 is None else (n * nxt.w2).to(dtype)
     w, eps, conv = nxt
     h = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
@@ -333,24 +344,24 @@ def post_norm(x, y, w, eps, nxt=None):
 
 
 def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=None, dtype=None):
-    """x + s1 * o + s2 * (combine(moe) + sigmoid(dense_gate) * dense), ``moe`` = (y, dest, wts); o, moe, dense may be None."""
+    """x + s1 * o + s2 * (combine(moe) + sigmoid(dense_gate) * dense), ``moe`` = (y, dest, wts); o, moe, dense may be None; s1, s2, wts None: one."""
     dtype = dtype or next((t.dtype for t in (o, dense, moe[0] if moe is not None else None) if t is not None), x.dtype)
     v = x
     if o is not None:
-        v = v + s1 * o.float()
+        v = v + (o.float() if s1 is None else s1 * o.float())
     f = None
     if moe is not None:
         y, dest, wts = moe
-        f = (y.float()[dest.long()] * wts[..., None]).sum(1)
+        f = y.float()[dest.long()]
+        f = (f if wts is None else f * wts[..., None]).sum(1)
     if dense is not None:
         g = dense.float() if dense_gate is None else torch.sigmoid(dense_gate.float())[:, None] * dense.float()
         f = g if f is None else f + g
-    return _finish_row(v if f is None else v + s2 * f, nxt, dtype)
+    return _finish_row(v if f is None else v + f if s2 is None else v + s2 * f, nxt, dtype)
 
 
-def rms_rows(x, rows, w, eps, dtype):
-    v = x if rows is None else x[rows.long()]
-    return (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w).to(dtype)
+def rms_rows(x, rows, w, eps, dtype, groups=1):
+    return (_group_rms(x if rows is None else x[rows.long()], groups, eps) * w).to(dtype)
 
 
 def causal_conv(h, w, state, seq_slots, positions, q_start, bias=None):
@@ -405,7 +416,7 @@ def _softplus(x):
     return F.softplus(x, threshold=1e9)
 
 
-def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top=None):
     """Runs the mixer described by ``m`` (``ops.specs.StateMix``) over a batch; result columns go to ``out`` [T, H * V]."""
     H, K, V, Hk = m.heads, m.dim, m.vdim, m.heads // m.rep
     qs = q_start.tolist()
@@ -432,19 +443,33 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
         cols = lambda off, h, w: x[:, off:off + h * w].view(n, h, w)          # noqa: B023,E731
         q, k, v = cols(m.q_off, Hk, K), cols(m.k_off, Hk, K), cols(m.v_off, H, V)
         s = torch.ones(n, H, device=proj.device)
+        if m.kind == "hgrn":
+            z = (dec_in[q0:q1].float() + m.bias).view(n, H, K)
+            low = m.lower.view(H, K)
+            dec, k, q = low + (1 - low) * torch.sigmoid(z), (1 - low) * torch.sigmoid(-z), F.silu(q)
+        if m.kind == "mlstm":
+            i, f = (m.gate_cap * torch.tanh(dec_in[q0:q1].float() / m.gate_cap)).view(n, 2, H).unbind(1)
+            f, t0 = F.logsigmoid(f), top[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, device=proj.device)
+            tops, dec = torch.empty(n, H, device=proj.device), torch.empty(n, H, 1, device=proj.device)
+            for t in range(n):
+                tops[t] = torch.maximum(f[t] + t0, i[t])
+                dec[t, :, 0], s[t], t0 = torch.exp(f[t] + t0 - tops[t]), torch.exp(i[t] - tops[t]), tops[t]
+            if slot >= 0:
+                top[slot] = t0
+            v = torch.cat([v, torch.ones(n, H, 1, device=proj.device), torch.zeros(n, H, m.cols - V - 1, device=proj.device)], 2)
         if m.kind == "delta":
             q, k = (y / torch.sqrt(y.pow(2).sum(-1, keepdim=True) + 1e-6) for y in (q, k))
             s = torch.sigmoid(x[:, m.s_off:m.s_off + H])
         if m.kind == "ssd":
             s = _softplus(x[:, m.s_off:m.s_off + H] + m.bias)
             dec = torch.exp(m.neg_a * s)[..., None]
-        else:
+        elif m.kind in ("delta", "linear"):
             z = dec_in[q0:q1].float() + m.bias
             dec = torch.exp(m.neg_a[:, None] * _softplus(z).view(n, H, K)) if m.kind == "delta" else \
                 torch.exp(-m.inv_tau * _softplus(-z)).view(n, H, K)
         q, k = (q * m.q_scale).repeat_interleave(m.rep, 1), k.repeat_interleave(m.rep, 1)
-        S = state[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, K, V, device=proj.device)
-        o = torch.empty(n, H, V, device=proj.device)
+        S = state[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, K, m.cols, device=proj.device)
+        o = torch.empty(n, H, m.cols, device=proj.device)
         for t in range(n):
             S = S * dec[t][..., None]
             u = v[t] - torch.einsum("hkv,hk->hv", S, k[t]) if m.kind == "delta" else v[t]
@@ -452,6 +477,15 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
             o[t] = torch.einsum("hkv,hk->hv", S, q[t])
         if slot >= 0:
             state[slot] = S
+        if m.kind == "mlstm":
+            o = o[..., :V] / (torch.maximum(o[..., V].abs(), torch.exp(-tops)) + 1e-6)[..., None]
+            o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + m.eps)).reshape(n, H * V)
+            out[q0:q1, :H * V] = (o * m.norm_w * torch.sigmoid(gate[q0:q1, :H * V].float()) * m.out_scale).to(out.dtype)
+            continue
+        if m.kind == "hgrn":
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + m.eps) * m.norm_w
+            out[q0:q1, :H * V] = (o * m.out_scale).reshape(n, H * V).to(out.dtype)
+            continue
         g = gate[q0:q1, :H * V].float()
         if m.kind == "ssd":
             y = (o + m.skip[:, None] * v).reshape(n, H * V) * F.silu(g)
@@ -488,7 +522,13 @@ def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single
 
 
 # ---- grouped-query attention over paged rows (csrc/kernels/gqa_attention.cu) ------------------------------------------------------------
-def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
+def pooled_row(table, b, pool: int, per_block: int, block_size: int):
+    """Rows of the pooled tensor that hold the means of blocks ``b`` of ``pool`` positions: they lie in the cache block of their last position."""
+    page = (b * pool + pool - 1) // block_size
+    return table.long()[page] * per_block + b - page * block_size // pool
+
+
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache, v_first=None, pooled=None):
     """Norms and rotates q and k, stores the rows of the cache; returns q [T, H, D].  ``m``: ``ops.specs.Gqa``."""
     T, H, G, D, V = q.shape[0], m.heads, m.kv_heads, m.dim, m.vdim
     cs = rope_table[positions.long()]
@@ -497,16 +537,28 @@ def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
         x = x.float().reshape(T, n, D)
         if w is not None:
             x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + m.eps) * w
-        return torch.cat([_rope(x[..., :m.rot], cs, True), x[..., m.rot:]], -1)
+        x = torch.cat([_rope(x[..., :m.rot], cs, not m.neighbours), x[..., m.rot:]], -1)
+        return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + m.eps) if m.unit else x
     qo = post(q, H, m.q_norm).to(q.dtype)
+    if m.v_mix is not None:
+        v = (1 - m.v_mix) * v.float() + m.v_mix * v_first.float()
     rows = torch.cat([post(k, G, m.k_norm).reshape(T, G * D), v.float()], 1).to(cache.dtype)
     ok = slot_mapping >= 0
     cache[slot_mapping[ok].long()] = rows[ok]
+    if m.pool:
+        pool, tables, seq_lens, q_start, bs, _ = pooled
+        P, qs, sl = m.pool, q_start.tolist(), seq_lens.tolist()
+        for s in range(len(qs) - 1):
+            n, S = qs[s + 1] - qs[s], sl[s]
+            for b in range((S - n) // P, S // P) if n > 0 and S > 0 else ():          # blocks that end among the new positions
+                pos = torch.arange(b * P, b * P + P, device=cache.device)
+                rows = cache[tables[s].long()[pos // bs] * bs + pos % bs].float()
+                pool[pooled_row(tables[s], torch.tensor(b, device=cache.device), P, m.pool_rows(bs), bs)] = rows.mean(0).to(pool.dtype)
     return qo
 
 
-def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
-    """Result columns go to ``out`` [T, H * V]; ``gate`` [T, H] pre-activations."""
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out, pool=None):
+    """Result columns go to ``out`` [T, H * V]; ``gate`` [T, H] pre-activations (``gate_each``: [T, H * V])."""
     T, H, D = q.shape
     G, V = m.kv_heads, m.vdim
     qs, sl = q_start.tolist(), seq_lens.tolist()
@@ -516,14 +568,18 @@ def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size
             continue
         pos = torch.arange(S, device=q.device)
         rows = cache[block_tables[b].long()[pos // block_size] * block_size + pos % block_size].float()
-        k = rows[:, :G * D].view(S, G, D).repeat_interleave(H // G, 1)
-        v = rows[:, G * D:].view(S, G, V).repeat_interleave(H // G, 1)
         i, j = torch.arange(S - (q1 - q0), S, device=q.device)[:, None], pos[None]
         see = j <= i
         if m.window:
             see = see & (i - j < m.window)
         if m.chunk:
             see = see & (i // m.chunk == j // m.chunk)
+        if m.pool and m.window and S // m.pool:
+            blocks = torch.arange(S // m.pool, device=q.device)
+            rows = torch.cat([rows, pool[pooled_row(block_tables[b], blocks, m.pool, m.pool_rows(block_size), block_size)].float()])
+            see = torch.cat([see, blocks[None] * m.pool + m.pool - 1 <= i - m.window], 1)
+        k = rows[:, :G * D].view(-1, G, D).repeat_interleave(H // G, 1)
+        v = rows[:, G * D:].view(-1, G, V).repeat_interleave(H // G, 1)
         s = torch.einsum("ihd,jhd->hij", q[q0:q1].float(), k) * m.scale
         if m.softcap:
             s = m.softcap * torch.tanh(s / m.softcap)
@@ -531,9 +587,10 @@ def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size
         if m.sink:                                                # a key without a value
             k0 = torch.zeros_like(s[..., :1])
             s = torch.cat([s, k0 if m.sink_w is None else k0 + m.sink_w[:, None, None]], -1)
-        p = torch.softmax(s, -1)[..., :S]
+        p = torch.softmax(s, -1)[..., :rows.shape[0]]
         o = torch.einsum("hij,jhv->ihv", p, v)
         if gate is not None:
-            o = o * torch.sigmoid(gate[q0:q1].float())[..., None]
+            g = torch.sigmoid(gate[q0:q1].float())
+            o = o * (g.view(q1 - q0, H, V) if m.gate_each else g[..., None])
         out[q0:q1, :H * V] = (o * m.out_scale).reshape(q1 - q0, H * V).to(out.dtype)
     return out

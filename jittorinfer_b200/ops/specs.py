@@ -13,7 +13,11 @@ class StateMix:
 
     ``kind``  "delta": q, k unit vectors, decay exp(neg_a softplus(. + bias)) per key channel, s = sigmoid(.), norm per head, sigmoid gate;
     "linear": decay sigmoid(. + bias)^inv_tau per key channel, s = 1, norm per head, silu gate;
-    "ssd": s = softplus(. + bias), decay exp(neg_a s) per head, silu gate, then a norm over ``norm_groups`` parts of the row.
+    "ssd": s = softplus(. + bias), decay exp(neg_a s) per head, silu gate, then a norm over ``norm_groups`` parts of the row;
+    "hgrn": decay f = lower + (1 - lower) sigmoid(. + bias) per key channel, k = 1 - f, silu on q, s = 1, norm per head, no gate;
+    "mlstm": decay and s per head from two log gates i = cap tanh(. / cap) and f = log sigmoid(cap tanh(. / cap)), relative to a running
+    maximum top <- max(f + top, i) that starts at 0: decay exp(f + top_old - top), s exp(i - top).  k decays and adds up like k v^T does (column
+    ``vdim`` of the state); o is divided by max(|that sum . q|, exp(-top)) + 1e-6, then a norm per head (``norm_w`` [heads * vdim]), sigmoid gate.
     ``*_off``: columns of the projection.  Columns conv0 .. conv0 + n of it pass a causal convolution of ``taps`` taps (0: none) and silu."""
     kind: str
     heads: int
@@ -37,13 +41,25 @@ class StateMix:
     inv_tau: float = 1.0
     eps: float = 1e-6
     out_scale: float = 1.0
+    lower: Optional[torch.Tensor] = None        # [heads * dim] fp32, "hgrn"
+    gate_cap: float = 0.0                       # "mlstm"
+
+    @property
+    def cols(self) -> int:
+        """Columns of a state row: the values', and for "mlstm" that of the keys' sum (padded to a multiple of 4)."""
+        return (self.vdim + 4) // 4 * 4 if self.kind == "mlstm" else self.vdim
 
 
 @dataclass
 class Gqa:
-    """Grouped-query attention with normed q and k (norm weights None: no norm), rotate-half RoPE on the first ``rot`` dimensions, scores *
-    scale, softcap (0: none), a causal mask with a sliding window and / or chunks (0: none), and with ``sink`` one more key without a value,
-    of score 0 or ``sink_w[head]``."""
+    """Grouped-query attention with normed q and k (norm weights None: no norm), RoPE on the first ``rot`` dimensions (pairs (i, i + rot / 2), or
+    with ``neighbours`` (2 i, 2 i + 1)), with ``unit`` q and k over their root mean square after it, scores * scale, softcap (0: none), a
+    causal mask with a sliding window and / or chunks (0: none), and with ``sink`` one more key without a value, of score 0 or
+    ``sink_w[head]``.
+
+    ``pool`` > 0: beside its window a query sees one key and value for every block of ``pool`` positions that lies wholly before the window,
+    the means of the block's cached rows.  ``v_mix`` is not None: the cached values are (1 - v_mix) v + v_mix v_first.  ``gate_each``: the
+    gate holds a column per head and value channel instead of one per head."""
     heads: int
     kv_heads: int
     dim: int
@@ -59,10 +75,22 @@ class Gqa:
     eps: float = 1e-6
     out_scale: float = 1.0
     sink_w: Optional[torch.Tensor] = None       # [heads] fp32
+    neighbours: bool = False
+    unit: bool = False
+    pool: int = 0
+    v_mix: Optional[float] = None
+    gate_each: bool = False
 
     @property
     def kv_row(self) -> int:
         return self.kv_heads * (self.dim + self.vdim)
+
+    def pool_rows(self, block_size: int) -> int:
+        """Pooled rows kept per cache block: those of the pooled blocks that end in it (padded so that cache blocks stay 16-byte multiples)."""
+        if not self.pool:
+            return 0
+        n = (block_size + self.pool - 1) // self.pool
+        return n if n * self.kv_row % 8 == 0 else (n + 7) // 8 * 8
 
 
 @dataclass
@@ -81,7 +109,8 @@ class SelectiveScan:
 @dataclass
 class RowNorms:
     """What an updated residual row turns into: row / rms * w1, and with ``w2`` row / rms * w2 as well; ``w1`` None: the row itself in the
-    activation type."""
+    activation type.  ``groups``: equal parts of the row, each over its own rms."""
     eps: float = 0.0
     w1: Optional[torch.Tensor] = None
     w2: Optional[torch.Tensor] = None
+    groups: int = 1

@@ -54,13 +54,16 @@ class HybridCache:
     ``state[name][i]``: (shape, dtype) of what one sequence keeps for layer i under that name, or None.
 
     ``cache[i]`` is the [n_slots, width] tensor layer i reads; ``cache.state[name][i]`` the [n_seqs, *shape] tensor.  State rows are
-    never cleared: kernels start a sequence's first token from zeros."""
+    never cleared: kernels start a sequence's first token from zeros.  ``pooled[i]`` > 0: layer i also keeps that many rows of the same
+    width per block, ``cache.pool[i]`` [blocks * rows, width], which go where the block goes."""
 
     def __init__(self, rows: Sequence[Any], state: Dict[str, Sequence[Optional[Tuple[Tuple[int, ...], torch.dtype]]]], n_slots: int,
-                 n_seqs: int, dtype: torch.dtype, device: torch.device, block_size: int):
+                 n_seqs: int, dtype: torch.dtype, device: torch.device, block_size: int, pooled: Optional[Sequence[int]] = None):
         self.block_size = block_size
         self.own: List[torch.Tensor] = []
         self._rows: List[Optional[torch.Tensor]] = []
+        self.pool_rows = list(pooled) if pooled is not None else [0] * len(rows)
+        self.pool = [torch.zeros(n_slots // block_size * n, r, dtype=dtype, device=device) if n else None for n, r in zip(self.pool_rows, rows)]
         for r in rows:
             if r is None:
                 self._rows.append(None)
@@ -87,3 +90,6 @@ class HybridCache:
         d = torch.from_numpy(np.ascontiguousarray(dst)).to(dev)
         for t in self.own:
             ops.kv_block_copy(t[None], s, d, self.block_size)
+        for t, n in zip(self.pool, self.pool_rows):
+            if t is not None:
+                ops.kv_block_copy(t[None], s, d, n)

@@ -326,6 +326,9 @@ class LLMEngine:
             rows = (torch.from_numpy(blocks.astype(np.int64)).to(layer.device)[:, None] * bs +
                     torch.arange(bs, device=layer.device)[None, :]).reshape(-1)
             layer[rows] = float("nan")
+            pool, n = (self.kv_cache.pool[il], self.kv_cache.pool_rows[il]) if hasattr(self.kv_cache, "pool") else (None, 0)
+            if pool is not None:
+                pool.view(-1, n, pool.shape[1])[torch.from_numpy(blocks.astype(np.int64)).to(pool.device)] = float("nan")
         self.stats["poisoned_blocks"] += int(blocks.size)
 
     def _graph_for(self, bucket: int, mode: str):
