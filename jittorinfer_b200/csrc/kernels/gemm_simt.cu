@@ -22,7 +22,11 @@ __device__ __forceinline__ float gate_arg(float z, int act) {
     return act == JIB_ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
 }
 
-__device__ __forceinline__ float unary(float v, const jib_gemm_desc & d) {
+__device__ __forceinline__ float unary(float v, const jib_gemm_desc & d, long long row) {
+    if (d.unary == JIB_UNARY_GELU) {
+        if (d.row_scale != nullptr) v *= d.row_scale[row];
+        return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+    }
     if (d.unary == JIB_UNARY_NONE) return v;
     if (d.unary == JIB_UNARY_RELU2) return v > 0.f ? v * v : 0.f;
     v *= d.scale;
@@ -87,7 +91,7 @@ __global__ void __launch_bounds__(NT) gemm_simt_kernel(const jib_gemm_desc d) {
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             if (n >= d.N) continue;
-            float y = DUAL ? acc[i][j] / (1.f + expf(-gate_arg(acc[i][j], d.act))) * acu[i][j] : unary(acc[i][j], d);
+            float y = DUAL ? acc[i][j] / (1.f + expf(-gate_arg(acc[i][j], d.act))) * acu[i][j] : unary(acc[i][j], d, row);
             if (d.residual != nullptr) {
                 const long long ri = (long long) batch * d.res_batch_stride + row * d.ldr + n;
                 y += d.res_f32 ? ((const float *) d.residual)[ri] : to_f(((const bf16 *) d.residual)[ri]);

@@ -71,6 +71,7 @@ struct GemmArgs {
     int act;                  // of a gated pair (JIB_ACT_*)
     int unary;                // of a single product (JIB_UNARY_*)
     float scale, softcap, cap2;      // cap2 = 2 scale / softcap
+    const float * row_scale;  // JIB_UNARY_GELU: null, or a factor of every result row's product
     int vec_store;            // bf16 result rows are written as 16-byte vectors through a shared-memory transpose
     const int * src_token;    // grouped, decode batches: x holds the T token rows unsorted, every expert multiplies all of
                               // them (one token tile) and sorted row i of the result is accumulator column src_token[i]
@@ -159,6 +160,14 @@ __device__ __forceinline__ float unary(float v, const GemmArgs & a) {
     if (a.softcap <= 0.f) return v * a.scale;
     return a.softcap * (1.f - __fdividef(2.f, 1.f + __expf(fminf(v * a.cap2, 80.f))));
 }
+// FN instances: 0 the product itself, 1 relu^2 and softcap, 2 gelu of the product times its row's factor.  A row past the tile's last has none.
+template <int FN>
+__device__ __forceinline__ float function_of(float v, const GemmArgs & a, long long row, bool valid) {
+    if (FN == 0) return v;
+    if (FN == 1) return unary(v, a);
+    if (a.row_scale != nullptr && valid) v *= __ldg(a.row_scale + row);
+    return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+}
 
 // Cluster-wide barrier (all threads of all CTAs of the cluster) and a load from a peer CTA's shared memory.
 __device__ __forceinline__ void cluster_sync_all() {
@@ -172,7 +181,7 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t local_smem_addr, uint32_t
     return v;
 }
 
-template <int BN, bool DUAL, bool FN>
+template <int BN, bool DUAL, int FN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA2,
             const __grid_constant__ CUtensorMap tmB, const GemmArgs args) {
@@ -394,9 +403,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         }
         // One finished element: feature n of row (row_base + t_rel); gv / uv are the summed accumulators.
         auto finish = [&](int t_rel, float gv, float uv) {
-            float y = DUAL ? gated(gv, args.act) * uv : FN ? unary(gv, args) : gv;
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
+            float y = DUAL ? gated(gv, args.act) * uv : function_of<FN>(gv, args, row, true);
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
                 args.ar.recv2[ar_owner][ar_par + ((size_t) args.ar.rank * args.ar.max_rows2 + row) * args.ar.d_max + n] = y;
                 return;
@@ -571,7 +580,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     const int ltid = (int) threadIdx.x - 64;
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : FN ? unary(g[j], args) : g[j];
+                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j]
+                                                                          : function_of<FN>(g[j], args, (long long) row_base + row0 + c + j, c + j < ncols);
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -728,7 +738,7 @@ __device__ __forceinline__ bool ptile_decode(const GemmArgs & args, int item, in
     return t.row0 < t.rows_valid;
 }
 
-template <int BN, bool DUAL, bool FN>
+template <int BN, bool DUAL, int FN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmA2,
                        const __grid_constant__ CUtensorMap tmB, const GemmArgs args, const int n_x, const int n_y, const int n_items) {
@@ -860,7 +870,8 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
 #pragma unroll
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
-                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k]) : FN ? unary(g, args) : g;
+                    sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k])
+                                          : function_of<FN>(g, args, (long long) t.row_base + t.row0 + c + k, c + k < ncols);
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
@@ -1018,7 +1029,7 @@ int auto_splits(long long base_ctas, int num_kb, int bn, int sms) {
     return splits;
 }
 
-template <int BN, bool DUAL, bool FN>
+template <int BN, bool DUAL, int FN>
 int launch_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid,
            cudaStream_t stream) {
     using C = Cfg<BN, DUAL>;
@@ -1032,11 +1043,12 @@ int launch_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap &
 
 template <int BN, bool DUAL>
 int launch(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid, cudaStream_t stream) {
-    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_as<BN, DUAL, !DUAL>(a, a2, b, args, grid, stream);
-    return launch_as<BN, DUAL, false>(a, a2, b, args, grid, stream);
+    if (!DUAL && args.unary == JIB_UNARY_GELU) return launch_as<BN, DUAL, DUAL ? 0 : 2>(a, a2, b, args, grid, stream);
+    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_as<BN, DUAL, DUAL ? 0 : 1>(a, a2, b, args, grid, stream);
+    return launch_as<BN, DUAL, 0>(a, a2, b, args, grid, stream);
 }
 
-template <int BN, bool DUAL, bool FN>
+template <int BN, bool DUAL, int FN>
 int launch_persistent_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, int n_x, int n_y,
                       long long n_items, int sms, cudaStream_t stream) {
     using C = PCfg<BN, DUAL>;
@@ -1052,8 +1064,9 @@ int launch_persistent_as(const CUtensorMap & a, const CUtensorMap & a2, const CU
 template <int BN, bool DUAL>
 int launch_persistent(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, int n_x, int n_y,
                       long long n_items, int sms, cudaStream_t stream) {
-    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_persistent_as<BN, DUAL, !DUAL>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
-    return launch_persistent_as<BN, DUAL, false>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
+    if (!DUAL && args.unary == JIB_UNARY_GELU) return launch_persistent_as<BN, DUAL, DUAL ? 0 : 2>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
+    if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_persistent_as<BN, DUAL, DUAL ? 0 : 1>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
+    return launch_persistent_as<BN, DUAL, 0>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
 }
 
 // JIB_GEMM_PERSIST=0: launches with several waves of tiles use the one-tile-per-CTA kernel as well (A/B measurements).
@@ -1166,7 +1179,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream_)
     if (a.ag_flags != nullptr && (a.ag_epoch == nullptr || a.ag_rows <= 0 || a.ag_world <= 0 || grouped || batch != 1)) return JIB_E_ARG;
     if (a.ar_rs_rows < 0) return JIB_E_ARG;
     if (a.row_ptr != nullptr && (dual || d->out_f32 || d->residual != nullptr || d->ar != nullptr)) return JIB_E_ARG;
-    a.act = d->act; a.unary = dual ? JIB_UNARY_NONE : d->unary; a.scale = d->scale; a.softcap = d->softcap;
+    a.act = d->act; a.unary = dual ? JIB_UNARY_NONE : d->unary; a.scale = d->scale; a.softcap = d->softcap; a.row_scale = d->row_scale;
     a.cap2 = d->softcap > 0.f ? 2.f * d->scale / d->softcap : 0.f;
     if (a.unary != JIB_UNARY_NONE && d->ar != nullptr) return JIB_E_ARG;
     memset(&a.ar, 0, sizeof(a.ar));
@@ -1342,7 +1355,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16_noalloc(const void * x, const void * w, 
     a.expert_list = nullptr;
     a.list_tiles = 0;
     a.ag_flags = nullptr; a.ag_epoch = nullptr; a.ag_rows = 0; a.ag_world = 0; a.ar_rs_rows = 0; a.ag_spin_limit = 0;
-    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = a.cap2 = 0.f;
+    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = a.cap2 = 0.f; a.row_scale = nullptr;
     memset(&a.ar, 0, sizeof(a.ar));
     dim3 grid(p.n_tiles, 1, p.splits);
     switch (p.bn) {

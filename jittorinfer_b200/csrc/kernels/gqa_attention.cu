@@ -1,9 +1,12 @@
 // Grouped-query attention over paged key / value rows: H query heads share G key / value heads (head h reads h / (H / G)).
 // A cached row holds the normed and rotated keys of a token (G * D columns), then its values (G * V columns).
 //
-//   gqa_qkv_post    per-head RMS norm of q and k (or none), rotate-half RoPE on the first rot dimensions, rows into the cache
-//   gqa_attention   scores * scale, softcap, causal mask with a sliding window and / or chunks counted from position 0, softmax
-//                   with or without a sink (a key without a value, of score 0 or of a number per head), a gate per head: any mix of portions and single
+//   gqa_qkv_post    per-head RMS norm of q and k (or none; with weights ahead of the rotation, without after it), RoPE on the first rot
+//                   dimensions, a blend of the values with another layer's, rows into the cache
+//   gqa_pool        means of the cached rows of complete blocks of positions (single tokens: part of gqa_qkv_post)
+//   gqa_attention   scores * scale, softcap, causal mask with a sliding window and / or chunks counted from position 0, one more key per
+//                   block of positions that has left the window, softmax with or without a sink (a key without a value, of score 0 or of a
+//                   number per head), a gate per head or channel: any mix of portions and single
 //                   tokens, keys split over a thread-block cluster.  bf16 heads whose sizes are multiples of 16: products on the
 //                   tensor cores (gqa_mma); fp32 and other sizes: CUDA cores (gqa_attention).  Prompts with heads of 128 have a
 //                   kernel of their own (mha_prefill_tcgen05.cu).
@@ -47,7 +50,7 @@ template <typename T, int N>
 __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ k,
                                                            const T * __restrict__ v, long long ld, const float * __restrict__ q_norm,
                                                            const float * __restrict__ k_norm, const float * __restrict__ rope,
-                                                           const int * __restrict__ slot_mapping, T * __restrict__ q_out) {
+                                                           const int * __restrict__ slot_mapping, T * __restrict__ q_out, int single) {
     extern __shared__ float heads[];                         // [8 warps][D]
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
@@ -64,11 +67,31 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
         if (slot < 0) return;                                // a padding row
         row = (T *) a.cache + (size_t) slot * a.row;
     }
+    // single tokens: one that completes a block of positions also stores the mean of its rows (the others' are in the cache)
+    const int * bt = nullptr;
+    T * pooled = nullptr;
+    int pos = a.positions[t];
+    if (row != nullptr && single && a.pool_size > 0 && pos >= 0 && (pos + 1) % a.pool_size == 0) {
+        bt = a.block_tables + (size_t) t * a.max_blocks;
+        pooled = (T *) a.pool + gqa_pool_row(bt, pos / a.pool_size, a.pool_size, a.pool_rows, a.block_size) * a.row;
+    }
+    auto earlier = [&](int col) {                            // sum over the block's earlier rows
+        float s = 0.f;
+#pragma unroll 4
+        for (int p = pos - a.pool_size + 1; p < pos; ++p)
+            s += to_f(((const T *) a.cache)[((long long) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row + col]);
+        return s;
+    };
     if (item >= H + G) {
         const int g = item - H - G;
-        const T * src = v + (size_t) t * ld + g * V;
+        const T * src = v + (size_t) t * ld + g * V, * first = (const T *) a.v_first + (size_t) t * a.ld_first + g * V;
         T * dst = row + G * D + g * V;
-        for (int c = lane; c < V; c += 32) dst[c] = src[c];
+        for (int c = lane; c < V; c += 32) {
+            T y = src[c];
+            if (a.mix_v) put(&y, (1.f - a.v_mix) * to_f(y) + a.v_mix * to_f(first[c]));
+            dst[c] = y;
+            if (pooled != nullptr) put(pooled + G * D + g * V + c, (earlier(G * D + g * V + c) + to_f(y)) / (float) a.pool_size);
+        }
         return;
     }
     const bool is_q = item < H;
@@ -83,20 +106,20 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
         e[i] = c < D ? to_f(src[c]) : 0.f;
         ss += e[i] * e[i];
     }
-    int pos = a.positions[t];
-    if (pos < 0 || pos >= a.max_pos) {
-        if (lane == 0) jib_report(a.status, JIB_ERR_BOUNDS, 49, pos);
-        pos = 0;
+    int at = pos;
+    if (at < 0 || at >= a.max_pos) {
+        if (lane == 0) jib_report(a.status, JIB_ERR_BOUNDS, 49, at);
+        at = 0;
     }
     const int half = a.rot / 2;
-    const float2 * cs = (const float2 *) rope + (size_t) pos * half;
+    const float2 * cs = (const float2 *) rope + (size_t) at * half;
     float wt[N];
     float2 r[N];
 #pragma unroll
     for (int i = 0; i < N; ++i) {                            // requested before the reduction
         const int c = lane + 32 * i;
         wt[i] = w != nullptr && c < D ? w[c] : 0.f;
-        r[i] = c < a.rot ? cs[c < half ? c : c - half] : make_float2(1.f, 0.f);
+        r[i] = c < a.rot ? cs[a.neighbours ? c >> 1 : c < half ? c : c - half] : make_float2(1.f, 0.f);
     }
     if (w != nullptr) {
         const float inv = rsqrtf(warp_sum(ss) / (float) D + a.eps);
@@ -108,14 +131,56 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
         if (lane + 32 * i < D) x[lane + 32 * i] = e[i];
     __syncwarp();
     T * dst = is_q ? q_out + ((size_t) t * H + head) * D : row + head * D;
+    ss = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i) {
         const int c = lane + 32 * i;
         if (c >= D) continue;
-        float y = e[i];
-        if (c < half) y = y * r[i].x - x[c + half] * r[i].y;
-        else if (c < a.rot) y = y * r[i].x + x[c - half] * r[i].y;
-        put(dst + c, y);
+        if (a.neighbours) {
+            if (c < a.rot) e[i] = e[i] * r[i].x + ((c & 1) ? x[c - 1] : -x[c + 1]) * r[i].y;
+        } else if (c < half) {
+            e[i] = e[i] * r[i].x - x[c + half] * r[i].y;
+        } else if (c < a.rot) {
+            e[i] = e[i] * r[i].x + x[c - half] * r[i].y;
+        }
+        ss += e[i] * e[i];
+    }
+    const float inv = a.unit ? rsqrtf(warp_sum(ss) / (float) D + a.eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const int c = lane + 32 * i;
+        if (c >= D) continue;
+        T y;
+        put(&y, e[i] * inv);
+        dst[c] = y;
+        if (pooled != nullptr) put(pooled + head * D + c, (earlier(head * D + c) + to_f(y)) / (float) a.pool_size);
+    }
+}
+
+// Means of complete blocks of pool_size positions, portions.  One CTA per block that can end in this batch: sequence b's begin at index
+// q_start[b] / pool_size + b, the first is the one its first new position lies in; indices in the gaps have none.
+template <typename T>
+__global__ void __launch_bounds__(256) gqa_pool_kernel(const __grid_constant__ jib_gqa a) {
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int P = a.pool_size;
+    int b = 0, hi = a.n_seqs;
+    while (hi - b > 1) {
+        const int mid = (b + hi) >> 1;
+        if (a.q_start[mid] / P + mid <= (int) blockIdx.x) b = mid; else hi = mid;
+    }
+    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0, S = a.seq_lens[b];
+    if (n <= 0 || S < n) return;
+    const int block = (S - n) / P + (int) blockIdx.x - (q0 / P + b), p0 = block * P;
+    if (block < (S - n) / P || p0 + P > S) return;
+    const int * bt = a.block_tables + (size_t) b * a.max_blocks;
+    T * dst = (T *) a.pool + gqa_pool_row(bt, block, P, a.pool_rows, a.block_size) * a.row;
+    const int cols = a.G * (a.D + a.V);
+    for (int c = threadIdx.x; c < cols; c += 256) {
+        float s = 0.f;
+#pragma unroll 8
+        for (int p = p0; p < p0 + P; ++p) s += to_f(((const T *) a.cache)[((long long) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row + c]);
+        put(dst + c, s / (float) P);
     }
 }
 
@@ -163,9 +228,10 @@ template <> struct Quad<bf16> {
     }
 };
 
-// What a CTA works on: rows (token i0 + r / nh of sequence b, head h0 + r % nh), r < rows, against the key tiles k_lo .. k_hi.
+// What a CTA works on: rows (token i0 + r / nh of sequence b, head h0 + r % nh), r < rows, against the tiles k_lo .. k_hi of its keys: first pt
+// tiles of pooled blocks (nb blocks), then the tiles of positions lo .. end, tile kt at positions (kt + t0) * KT.
 struct Work {
-    int b, q0, i0, g, h0, nh, rows, p0, lo, end, k_lo, k_hi;
+    int b, q0, i0, g, h0, nh, rows, p0, lo, end, k_lo, k_hi, nb, pt, t0;
 };
 // false: no work for this CTA nor for the others of its cluster
 __device__ __forceinline__ bool find_work(const jib_gqa & a, int run, int heads, int KT, Work & w) {
@@ -192,10 +258,13 @@ __device__ __forceinline__ bool find_work(const jib_gqa & a, int run, int heads,
     w.p0 = S - n + w.i0;                                     // position of the first token
     w.lo = max(0, gqa_first_key(w.p0, a.window, a.chunk));
     w.end = S > 0 ? w.p0 + nt : 0;
-    const int t_lo = w.lo / KT, tiles = w.end > w.lo ? (w.end - 1) / KT + 1 - t_lo : 0;
+    w.nb = gqa_blocks_seen(w.p0 + nt - 1, a.window, a.pool_size);
+    w.pt = (w.nb + KT - 1) / KT;
+    const int t_lo = w.lo / KT, tiles = w.pt + (w.end > w.lo ? (w.end - 1) / KT + 1 - t_lo : 0);
+    w.t0 = t_lo - w.pt;
     const int per = (tiles + (int) gridDim.z - 1) / (int) gridDim.z;
-    w.k_lo = t_lo + (int) blockIdx.z * per;
-    w.k_hi = min(t_lo + tiles, w.k_lo + per);
+    w.k_lo = (int) blockIdx.z * per;
+    w.k_hi = min(tiles, w.k_lo + per);
     return true;
 }
 
@@ -219,7 +288,7 @@ __device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, c
             ls[s] = n_splits > 1 ? ld_peer(l_s + r, s) : l_s[r];
             os[s] = n_splits > 1 ? ld_peer(part + r * V + col, s) : part[r * V + col];
         }
-        const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + h]) : 0.f;
+        const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + (a.gate_each ? h * V + col : h)]) : 0.f;
 #pragma unroll
         for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
         float l = a.sink ? exp_t<T>(sink - m) : 0.f, o = 0.f;
@@ -272,9 +341,14 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
     const int key = tid % KT, rg = tid / KT, rpt = ROWS * KT / NT;       // scores: this thread's key and its rpt rows
     for (int kt = w.k_lo; kt < w.k_hi; ++kt) {
         __syncthreads();
+        const bool pooled = kt < w.pt;
+        const int base = (pooled ? kt : kt + w.t0) * KT, first = pooled ? 0 : lo, last = pooled ? w.nb : end;      // keys first .. last - 1 exist
+        const T * src = pooled ? (const T *) a.pool : (const T *) a.cache;
         if (tid < KT) {                                      // where this tile's rows are
-            const int p = kt * KT + tid;
-            rows_s[tid] = p < end && p >= lo ? bt[p / a.block_size] * a.block_size + p % a.block_size : -1;
+            const int p = base + tid;
+            rows_s[tid] = p >= last || p < first ? -1
+                                                 : pooled ? (int) gqa_pool_row(bt, p, a.pool_size, a.pool_rows, a.block_size)
+                                                          : bt[p / a.block_size] * a.block_size + p % a.block_size;
         }
         __syncthreads();
         const int k4 = DP / 4 - 1, w4 = k4 + VP / 4;
@@ -287,7 +361,7 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
                 x[u].zero();
                 const int slot = e < KT * w4 ? rows_s[j] : -1;
                 if (slot < 0) continue;
-                const T * row = (const T *) a.cache + (size_t) slot * a.row;
+                const T * row = src + (size_t) slot * a.row;
                 if (c < k4) x[u].load(row + g * D, 4 * c, D, vec);
                 else x[u].load(row + a.G * D + g * V, 4 * (c - k4), V, vec);
             }
@@ -311,13 +385,13 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
                 s[r] += x.x * y.x + x.y * y.y + x.z * y.z + x.w * y.w;
             }
         }
-        const int p = kt * KT + key;
+        const int p = base + key;
 #pragma unroll
         for (int r = 0; r < 8; ++r) {
             if (r >= rpt) break;
             const int row = rg * rpt + r;
             const int pos = p0 + (row < rows ? row / nh : 0);
-            const bool see = row < rows && p <= pos && p >= gqa_first_key(pos, a.window, a.chunk);
+            const bool see = row < rows && (pooled ? p < gqa_blocks_seen(pos, a.window, a.pool_size) : p <= pos && p >= gqa_first_key(pos, a.window, a.chunk));
             const float v = a.softcap > 0.f ? capped<T>(s[r], a.softcap) : s[r];
             ps[key * ROWS + row] = see ? v : -INFINITY;
         }
@@ -350,8 +424,8 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
         for (int c = 0; c < NVC; ++c)
 #pragma unroll
             for (int r = 0; r < ROWS; ++r) acc[c][r] *= c_s[r];
-        const int jn = min(KT, end - kt * KT);
-        for (int j = max(0, lo - kt * KT); j < jn; ++j) {
+        const int jn = min(KT, last - base);
+        for (int j = max(0, first - base); j < jn; ++j) {
             float pr[ROWS];
 #pragma unroll
             for (int r = 0; r < ROWS; r += 4) {
@@ -421,9 +495,12 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
     // a thread copies half of one key's row: 2 threads per key
     auto stage = [&](int kt, int buf) {
         if (kt < w.k_hi) {
-            const int j = tid >> 1, p = kt * MK + j;
-            const bool in = p >= w.lo && p < w.end;
-            const bf16 * row = in ? cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row : cache;
+            const bool pooled = kt < w.pt;
+            const int j = tid >> 1, p = (pooled ? kt : kt + w.t0) * MK + j;
+            const bool in = pooled ? p < w.nb : p >= w.lo && p < w.end;
+            const bf16 * row = !in ? cache
+                               : pooled ? (const bf16 *) a.pool + gqa_pool_row(bt, p, a.pool_size, a.pool_rows, a.block_size) * a.row
+                                        : cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row;
             const uint32_t kd = kv_addr + buf * tile_bytes + j * LD * 2, vd = kv_addr + buf * tile_bytes + (MK * LD + j * LV) * 2;
             for (int c = tid & 1; c < d8; c += 2) cp16(kd + c * 16, row + w.g * D + c * 8, in);
             for (int c = tid & 1; c < v8; c += 2) cp16(vd + c * 16, row + a.G * D + w.g * V + c * 8, in);
@@ -436,13 +513,14 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
     }
     stage(w.k_lo, 0);
     const int fr = lane >> 2, fc = (lane & 3) * 2;
-    // positions and first keys of this thread's two rows
-    int pos[2], first[2];
+    // positions, first keys and pooled blocks of this thread's two rows
+    int pos[2], first[2], blocks[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
         const int r = fr + 8 * e;
         pos[e] = r < w.rows ? w.p0 + r / w.nh : -1;
         first[e] = r < w.rows ? gqa_first_key(pos[e], a.window, a.chunk) : 0;
+        blocks[e] = gqa_blocks_seen(pos[e], a.window, a.pool_size);
     }
     float o[2 * NV][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 #pragma unroll
@@ -470,7 +548,9 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
             mma(s[0], x, y[0], y[1]);
             mma(s[1], x, y[2], y[3]);
         }
-        const int key = kt * MK + warp * 16 + fc;            // this thread's keys: key, key + 1, key + 8, key + 9
+        const bool pooled = kt < w.pt;
+        const int key = (pooled ? kt : kt + w.t0) * MK + warp * 16 + fc;            // this thread's keys: key, key + 1, key + 8, key + 9
+        const int end[2] = {pooled ? blocks[0] : pos[0] + 1, pooled ? blocks[1] : pos[1] + 1}, from[2] = {pooled ? 0 : first[0], pooled ? 0 : first[1]};
         float mt[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < 2; ++n)
@@ -484,7 +564,7 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
                     y = cap - 2.f * cap * r;                 // 1 - 2 / (1 + e^{2 y}) = tanh(y)
                 }
                 const int p = key + n * 8 + (e & 1);
-                s[n][e] = p <= pos[e >> 1] && p >= first[e >> 1] ? y : -INFINITY;
+                s[n][e] = p < end[e >> 1] && p >= from[e >> 1] ? y : -INFINITY;
                 mt[e >> 1] = fmaxf(mt[e >> 1], s[n][e]);
             }
         float cf[2];
@@ -597,7 +677,7 @@ int launch_attention(const jib_gqa & a, const void * q, const void * gate, long 
 
 // bf16 rows that 16-byte copies can address
 bool mma_ok(const jib_gqa & a, const void * q) {
-    return a.D % 16 == 0 && a.V % 16 == 0 && a.V <= 256 && a.row % 8 == 0 && (((uintptr_t) a.cache | (uintptr_t) q) & 15) == 0;
+    return a.D % 16 == 0 && a.V % 16 == 0 && a.V <= 256 && a.row % 8 == 0 && (((uintptr_t) a.cache | (uintptr_t) a.pool | (uintptr_t) q) & 15) == 0;
 }
 
 template <int NV>
@@ -617,7 +697,9 @@ int launch_mma(const jib_gqa & a, const void * q, const void * gate, long long l
 
 bool ok(const jib_gqa & a) {
     return a.H >= 1 && a.G >= 1 && a.H % a.G == 0 && a.D >= 1 && a.D <= 32 * POST_D && a.V >= 1 && a.V <= 4 * NT && a.rot >= 0 && a.rot % 2 == 0 && a.rot <= a.D &&
-           a.row >= (long long) a.G * (a.D + a.V) && a.T <= 65535 && a.block_size > 0;
+           a.row >= (long long) a.G * (a.D + a.V) && a.T <= 65535 && a.block_size > 0 &&
+           (a.pool_size == 0 || (a.pool_size > 0 && a.window > 0 && a.pool != nullptr && a.block_tables != nullptr &&
+                                 a.pool_rows >= (a.block_size + a.pool_size - 1) / a.pool_size));
 }
 
 }  // namespace
@@ -625,16 +707,16 @@ bool ok(const jib_gqa & a) {
 extern "C" {
 
 JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * k, const void * v, long long ld, const float * q_norm,
-                                const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int f32, void * stream) {
+                                const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int single, int f32, void * stream) {
     const jib_gqa & a = *m;
     if (a.T <= 0) return 0;
-    if (!ok(a)) return JIB_E_ARG;
+    if (!ok(a) || (a.mix_v && a.v_first == nullptr) || (single && a.pool_size > 0 && a.n_seqs != a.T)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
     const dim3 grid((a.H + 2 * a.G + 7) / 8, a.T);
     const int smem = 8 * a.D * 4;
 #define POST(TT, N)                                                                                                                        \
     JIB_LAUNCH((gqa_qkv_post_kernel<TT, N>), grid, 256, smem, s, a, (const TT *) q, (const TT *) k, (const TT *) v, ld, q_norm, k_norm, rope, \
-               slot_mapping, (TT *) q_out)
+               slot_mapping, (TT *) q_out, single)
 #define CALL(N)                     \
     do {                            \
         if (f32) POST(float, N);    \
@@ -645,6 +727,11 @@ JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * 
     else CALL(POST_D);
 #undef CALL
 #undef POST
+    const int rc = launched();
+    if (rc || single || a.pool_size == 0) return rc;
+    if (a.q_start == nullptr || a.seq_lens == nullptr || a.n_seqs <= 0) return JIB_E_ARG;
+    if (f32) JIB_LAUNCH((gqa_pool_kernel<float>), a.T / a.pool_size + a.n_seqs, 256, 0, s, a);
+    else JIB_LAUNCH((gqa_pool_kernel<bf16>), a.T / a.pool_size + a.n_seqs, 256, 0, s, a);
     return launched();
 }
 

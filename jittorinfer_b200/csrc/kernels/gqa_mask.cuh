@@ -8,3 +8,15 @@ __host__ __device__ __forceinline__ int gqa_first_key(int p, int window, int chu
     if (chunk > 0 && p / chunk * chunk > lo) lo = p / chunk * chunk;
     return lo;
 }
+
+// Blocks of `pool` positions that a query at position p sees as one key each: blocks 0 .. n - 1, those that lie wholly before its window.
+// Non-decreasing in p.
+__host__ __device__ __forceinline__ int gqa_blocks_seen(int p, int window, int pool) {
+    return pool > 0 && p - window + 1 >= pool ? (p - window + 1) / pool : 0;
+}
+
+// Row of pooled block b: the pooled blocks that end in a cache block go with it, `rows` places for each.
+__device__ __forceinline__ long long gqa_pool_row(const int * block_table, int b, int pool, int rows, int block_size) {
+    const int page = ((b + 1) * pool - 1) / block_size;
+    return (long long) block_table[page] * rows + b - page * block_size / pool;
+}

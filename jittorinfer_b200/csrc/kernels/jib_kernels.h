@@ -17,8 +17,9 @@ enum {
 
 // Activation of a gated pair: z * sigmoid(z), or 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
 enum { JIB_ACT_SILU = 0, JIB_ACT_GELU_TANH = 1 };
-// Function of a single product (no w2): none, max(y, 0)^2, or s y with s = scale, capped to softcap tanh(s y / softcap) unless softcap is 0.
-enum { JIB_UNARY_NONE = 0, JIB_UNARY_RELU2 = 1, JIB_UNARY_CAP = 2 };
+// Function of a single product (no w2): none, max(y, 0)^2, s y with s = scale, capped to softcap tanh(s y / softcap) unless softcap is 0, or
+// gelu(r y) = r y (1 + erf(r y / sqrt 2)) / 2 with r = row_scale[row] (1 without).
+enum { JIB_UNARY_NONE = 0, JIB_UNARY_RELU2 = 1, JIB_UNARY_CAP = 2, JIB_UNARY_GELU = 3 };
 
 #ifdef __cplusplus
 extern "C" {
@@ -72,6 +73,7 @@ typedef struct jib_gemm_desc {
     int act;                   // with w2: JIB_ACT_*
     int unary;                // without w2: JIB_UNARY_*, applied before the residual (not with ar)
     float scale, softcap;     // of JIB_UNARY_CAP
+    const float * row_scale;  // of JIB_UNARY_GELU: NULL, or [rows of out], a factor of each (grouped: expert-sorted) row's product
 } jib_gemm_desc;
 
 JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream);
@@ -121,14 +123,14 @@ JIB_EXPORT int jib_moe_route_fused(const void * g, const float * w_router, const
 // Stable counting sort of the (token, k) pairs by local expert. dest[t*k+j] = sorted row or -1 (not local).
 // seg has room for 2 * E_local + 1 ints: the E_local + 1 segment offsets, then the list of the experts that have rows (in
 // order, -1 after the last): what jib_gemm_desc.expert_list takes.  (jib_moe_route_fused writes the same; the multi-CTA
-// sort for large batches writes the offsets only.)
+// sort for large batches writes the offsets only.)  wts NULL, or [T][k]: row_wts[row] receives the weight of the pair in sorted row `row`.
 JIB_EXPORT int jib_moe_permute(const int * ids, int T, int k, int expert_base, int E_local, int * seg, int * src_token, int * dest,
-                               void * stream);
+                               const float * wts, float * row_wts, void * stream);
 // (expert, token tile) work list of a grouped launch with token-tile width bn: out[i] = tile << 16 | expert for every tile of
 // every expert that has rows, in expert order, -1 up to cap.  cap >= rows / bn + E_local always suffices.
 JIB_EXPORT int jib_moe_tile_list(const int * seg, int E_local, int bn, int * out, int cap, void * stream);
 JIB_EXPORT int jib_moe_permute_multi(const int * ids, int T, int k, int expert_base, int E_local, int * seg, int * src_token, int * dest,
-                                     int * tmp, void * stream);
+                                     int * tmp, const float * wts, float * row_wts, void * stream);
 JIB_EXPORT int jib_moe_combine(const void * y, const int * dest, const float * wts, const void * shared, const void * residual,
                                void * out, int T, int k, int d, void * stream);
 // The same followed by RMSNorm(out) * norm_w (fp32 weights, as jib_rmsnorm) in one launch; bitwise the two-launch results.
@@ -151,10 +153,11 @@ JIB_EXPORT int jib_mla_flash(const void * q, const void * cache, long long n_slo
                              float * part_o, float * part_ml, void * o_lat, int * status, void * stream);
 
 // ---- prefill attention in the per-head form (mha_prefill_tcgen05.cu): head dims 128 + 64 (keys), 128 (values) ---------------
-// jib_kv_gather: lat [total_cap][row_elems] <- the cached latent rows of every sequence, in sequence order; kv_start [n_seqs].
+// jib_kv_gather: lat [total_cap][row_elems] <- the cached latent rows of every sequence, in sequence order; kv_start [n_seqs].  pool null, or pooled
+// rows (jib_gqa): those the sequence's last position sees come ahead of its own.
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, void * lat, int * kv_start,
-                             int total_cap, void * stream);
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, const void * pool, int pool_size,
+                             int pool_rows, void * lat, int * kv_start, int total_cap, void * stream);
 // q [T][H][192] (RoPE applied), kv [total][H][256] = k_nope | v, kpe [total][64] (row stride kpe_stride), out [T][H * 128].
 JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * kv, const void * kpe, long long kpe_stride, long long total,
                                const int * q_start, const int * seq_lens, const int * kv_start, int n_seqs, int T, int H, float scale,
@@ -179,6 +182,7 @@ typedef struct jib_row_tail {
     int taps, n_state;
     const float * norm2_w;     // null, or a second norm of the same row (not with conv_w)
     void * h2_out;
+    int groups;                // > 1: the norms are taken over that many equal parts of the row, each by itself (embed_norm, scaled_update)
 } jib_row_tail;
 // x_out = scale * table[ids[t]], RMS-normed and times w unless w is null.
 JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float * w, float eps, float scale, int T, int d, int n_vocab, int f32,
@@ -192,11 +196,11 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
                                 const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
                                 const jib_row_tail * tail, void * stream);
 // x_out = x + s1 * o + s2 * (sum_j wts[t][j] * y[dest[t][j]] + g * f), s1, s2 [d]; any of o, y, f may be null (absent).  f [T][d]: a dense
-// sublayer; g = sigmoid(f_gate[t * ld_gate]), 1 with f_gate null.  x_out may be x, or null: only the tail's norms.
+// sublayer; g = sigmoid(f_gate[t * ld_gate]), 1 with f_gate null; s1, s2 or wts null: ones.  x_out may be x, or null: only the tail's norms.
 JIB_EXPORT int jib_scaled_update(const float * x, const void * o, const float * s1, const void * y, const int * dest, const float * wts, int k,
                                  const void * f, const float * f_gate, long long ld_gate, const float * s2, int T, int d, int f32,
                                  const jib_row_tail * tail, void * stream);
-JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
+JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int groups, int f32, void * out,
                             void * stream);
 // out = h + causal convolution over time of h (w [taps][d] fp32), or with silu != 0 out = silu(bias + convolution); h [T][ldh], out
 // [T][d]; sequence b continues from, and advances, its stored rows (state [n_state][taps - 1][d]).
@@ -221,11 +225,24 @@ typedef struct jib_gqa {
     float scale, softcap;      // softcap 0: none
     float eps, out_scale;
     const float * sink_w;      // [H] or null
+    // pool_size > 0 (with a window): position i also sees one key and value per block b of pool_size positions with
+    // (b + 1) pool_size - 1 <= i - window, the mean of the block's cached rows.  It lies in row b - first of the pool_rows rows that go with the
+    // cache block of the pooled block's last position, first = the first pooled block that ends there.
+    void * pool;               // [blocks][pool_rows][row]
+    const void * v_first;      // mix_v: values [T][ld_first]; cached are (1 - v_mix) v + v_mix v_first
+    long long ld_first;
+    int pool_size, pool_rows;
+    int neighbours;            // rotated pairs are (2 i, 2 i + 1) instead of (i, i + rot / 2)
+    int unit;                  // q and k over their root mean square, after the rotation
+    int gate_each;             // the gate has a column per head and value channel instead of one per head
+    int mix_v;
+    float v_mix;
 } jib_gqa;
-// q, k, v: columns of the projection (row stride ld); q_norm, k_norm [D], or null: no norm.  rope [max_pos][rot / 2] pairs (cos, sin); pairs are (i, i + rot / 2).
+// q, k, v: columns of the projection (row stride ld); q_norm, k_norm [D], or null: no norm.  rope [max_pos][rot / 2] pairs (cos, sin).  With a pool
+// the pooled rows that are complete are stored as well; single: one token per sequence.
 JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * k, const void * v, long long ld, const float * q_norm,
-                                const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int f32, void * stream);
-// q [T][H][D]; gate null or [T][ld_gate] pre-activations of one sigmoid per head; out [T][ldo].  single: one token per sequence.
+                                const float * k_norm, const float * rope, const int * slot_mapping, void * q_out, int single, int f32, void * stream);
+// q [T][H][D]; gate null or [T][ld_gate] pre-activations of sigmoids; out [T][ldo].  single: one token per sequence.
 // splits (<= 8): CTAs that share a row's keys.
 JIB_EXPORT int jib_gqa_attention(const jib_gqa * m, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single,
                                  int splits, int f32, void * stream);
@@ -236,10 +253,11 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
                                long long ld_gate, int n_q_tiles, void * out, long long ldo, void * stream);
 
 // ---- mixers with a matrix state per head (state_mix.cu) ----------------------------------------------------------------------
-enum { JIB_STATE_DELTA = 0, JIB_STATE_LINEAR = 1, JIB_STATE_SSD = 2 };
+enum { JIB_STATE_DELTA = 0, JIB_STATE_LINEAR = 1, JIB_STATE_SSD = 2, JIB_STATE_HGRN = 3, JIB_STATE_MLSTM = 4 };
 typedef struct jib_state_mix {
     // activations (bf16 or fp32): proj [T][ld] holds q (H / rep heads x K), k, v (H x V) and the pre-activation of the per-head
-    // factor (s_off; H columns; not LINEAR) at these columns; dec_in [T][ld_dec] the decays' (H x K; not SSD); gate [T][ld_gate] H x V
+    // factor (s_off; H columns; DELTA, SSD) at these columns (HGRN has no k); dec_in [T][ld_dec] the decays' (H x K; not SSD), MLSTM: fp32
+    // input | forget gates' (2 H); gate [T][ld_gate] H x V (not HGRN)
     const void * proj, * dec_in, * gate;
     void * y;                  // [T][ldy] result, H x V columns
     // per-sequence state: [n_state][taps][n_conv] ring of convolution inputs (activation type), [n_state][H][K][V] fp32
@@ -250,14 +268,19 @@ typedef struct jib_state_mix {
     const float * bias;        // decays' (H x K) or SSD's factor's (H)
     const float * neg_a;       // [H], not LINEAR
     const float * skip;        // [H], SSD
-    const float * norm_w;      // [V], SSD [H x V]
+    const float * norm_w;      // [V], SSD, MLSTM [H x V]
     const int * seq_slots, * positions, * q_start;
     int * status;
-    float * qk, * v, * dec, * s, * o;      // scratch: [T][2][H / rep][K], [T][H][V], [T][H][K] (SSD [T][H]), [T][H], [T][H][V]
+    float * qk, * v, * dec, * s, * o;      // scratch: [T][2][H / rep][K], [T][H][V], [T][H][K] (SSD, MLSTM [T][H]), [T][H], [T][H][V]; MLSTM: V
+                                           // rounded up to the next multiple of 4 above it
     void * chunk;              // null, or chunk_bytes >= jib_state_chunk_bytes: portions of bf16 go through the tensor cores (then qk, dec unused)
     long long ld, ld_dec, ld_gate, ldy, chunk_bytes;
     int kind, H, K, V, rep, taps, conv0, n_conv, q_off, k_off, v_off, s_off, norm_groups, n_state, n_seqs, T;
     float q_scale, inv_tau, eps, out_scale;
+    const float * lower;       // [H x K], HGRN: lower bounds of the decays
+    float * extra;             // [n_state][H][K + 1], MLSTM: what the keys add up to, then the running maximum of the gates
+    float * tops;              // scratch [T][H], MLSTM: the running maximum at every token
+    float gate_cap;            // MLSTM
 } jib_state_mix;
 // single: one token per sequence (row t = sequence t; scratch only for SSD: o).  K <= 512.
 JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single, int f32, void * stream);

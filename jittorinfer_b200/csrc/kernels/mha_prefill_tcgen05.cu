@@ -22,7 +22,8 @@
 // expanded, and a CTA starts at the KV tile that holds the first row its first query sees.
 // A second form of the same kernel (GQA) serves grouped-query attention: keys of 128 dims and values of 128 per key / value head, shared
 // by H / G query heads and gathered as they are cached (no expansion, no RoPE part of their own), with softcap, a sink, chunks counted
-// from position 0 and a gate per head.
+// from position 0, a gate per head or channel, and one more key per block of positions that has left the window: the pooled rows are gathered
+// ahead of the sequence's own, and a CTA walks the tiles of those its last query sees, then the tiles of its window.
 // All waits are bounded (sm100.cuh); no multicast.
 #include "sm100.cuh"
 
@@ -70,6 +71,7 @@ struct MhaArgs {
     int G, chunk, sink;
     const float * sink_w;     // null: the sink's score is 0
     float cap_log2e, inv_cap2, out_scale;     // softcap * log2 e (0: none), 2 * scale * log2 e / softcap
+    int pool_size, gate_each;
 };
 
 // Rows of a sequence with S cached tokens that its last q_len tokens can see: the last ...
@@ -156,18 +158,29 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             x -= nt;
         }
     }
-    // n_tiles KV tiles from tile kt0 on, in gathered coordinates (row 0 = the first row the chunk can see)
-    int n_tiles = 0, kt0 = 0, ctx0 = 0, kv0 = 0, rows = 0, base_pos = 0;      // base_pos: position of gathered row 0
+    // n_tiles KV tiles in gathered coordinates (row 0 = the first row the chunk can see, pooled rows ahead of it): tiles 0 .. pt - 1, then from
+    // tile kt0 on
+    int n_tiles = 0, pt = 0, kt0 = 0, ctx0 = 0, kv0 = 0, rows = 0, base_pos = 0;      // base_pos: position of gathered row 0
     if (b >= 0) {
         const int S = visible_rows(a.seq_lens[b], q_len, a.window, a.chunk);
         base_pos = a.seq_lens[b] - S;
         ctx0 = S - q_len;                             // gathered rows before this chunk
+        if (GQA) {
+            const int np = gqa_blocks_seen(a.seq_lens[b] - 1, a.window, a.pool_size);
+            ctx0 += np;
+            base_pos -= np;
+        }
         kv0 = a.kv_start[b];
         rows = min(QT, q_len - tile * QT);            // valid query rows of the tile
         const int last_lim = ctx0 + tile * QT + rows; // kv rows visible to the last valid query row
         kt0 = max(0, gqa_first_key(base_pos + ctx0 + tile * QT, a.window, a.chunk) - base_pos) / KT;
-        n_tiles = rows > 0 && S > 0 ? (last_lim + KT - 1) / KT - kt0 : 0;
+        if (GQA) {
+            pt = (gqa_blocks_seen(base_pos + last_lim - 1, a.window, a.pool_size) + KT - 1) / KT;
+            kt0 = max(kt0, pt);
+        }
+        n_tiles = rows > 0 && S > 0 ? pt + (last_lim + KT - 1) / KT - kt0 : 0;
     }
+    auto tile_at = [&](int i) { return GQA && i < pt ? i : kt0 + i - pt; };
     const int row0 = q0 + tile * QT;                  // first query row (global)
 
     if (n_tiles > 0 && warp == 0) {
@@ -177,7 +190,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             for (int c = 0; c < NC; ++c) tma_load_2d(q_s + c * CHUNK, &tmQ, q_full, qcol + c * 64, row0);
             for (int kt = 0; kt < n_tiles; ++kt) {
                 const int s = kt & 1;
-                const int krow = kv0 + (kt0 + kt) * KT;
+                const int krow = kv0 + tile_at(kt) * KT;
                 if (!mbar_wait(&k_empty[s], ((kt >> 1) & 1) ^ 1)) { jib_report(a.status, JIB_ERR_WAIT_TIMEOUT, 31, kt); break; }
                 uint8_t * kd = k_s + s * K_BYTES;
                 mbar_expect_tx(&k_full[s], K_BYTES);
@@ -245,6 +258,9 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         // first visible gathered row of this query row, and of the tile's last one
         const int first = gqa_first_key(base_pos + ctx0 + tile * QT + r, a.window, a.chunk) - base_pos;
         const int first_last = gqa_first_key(base_pos + ctx0 + tile * QT + QT - 1, a.window, a.chunk) - base_pos;
+        // pooled rows this query row sees, and the tile's first one
+        const int blocks = GQA && r < rows ? gqa_blocks_seen(base_pos + ctx0 + tile * QT + r, a.window, a.pool_size) : 0;
+        const int blocks_first = GQA ? gqa_blocks_seen(base_pos + ctx0 + tile * QT, a.window, a.pool_size) : 0;
         float m_ref = -INFINITY;                      // exponent base, log2 domain (score * scale * log2 e)
         float l_sum = 0.f;
         bool ok = true;
@@ -255,11 +271,11 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             if (!ok) break;
             tc_fence_after();
             const uint32_t ts = tm_S + lane_addr + s * KT;
-            const int col0 = (kt0 + kt) * KT;
+            const int col0 = tile_at(kt) * KT;
             // the tile reaches the diagonal (or the sequence end), or begins before what the last row sees does
-            const bool need_mask = col0 + KT > lim_first || col0 < first_last;
+            const bool need_mask = (col0 + KT > lim_first || col0 < first_last) && (!GQA || col0 + KT > blocks_first);
             const int vis = lim - col0;               // columns [inv, vis) of this tile are visible to this row
-            const int inv = first - col0;
+            const int inv = first - col0, pooled = blocks - col0;
             // The row's 128 scores come out of tensor memory once, all loads in flight before one wait; the S buffer is
             // handed back to the tensor core right away (Q.K^T of the tile after the next may start).
             float x[KT];
@@ -275,13 +291,17 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
                 for (int c = 0; c < KT; ++c) x[c] = capped_log2(x[c], a);       // no branch around it: the 128 chains overlap
                 if (need_mask) {
 #pragma unroll
-                    for (int c = 0; c < KT; ++c) x[c] = (c < vis && c >= inv) ? x[c] : -INFINITY;
+                    for (int c = 0; c < KT; ++c) x[c] = (c < vis && c >= inv) || c < pooled ? x[c] : -INFINITY;
                 }
 #pragma unroll
                 for (int c = 0; c < KT; ++c) mt = fmaxf(mt, x[c]);
             } else if (need_mask) {
 #pragma unroll
-                for (int c = 0; c < KT; ++c) { x[c] = (c < vis && c >= inv) ? x[c] * a.scale_log2e : -INFINITY; mt = fmaxf(mt, x[c]); }
+                for (int c = 0; c < KT; ++c) {
+                    const bool see = (c < vis && c >= inv) || (GQA && c < pooled);
+                    x[c] = see ? x[c] * a.scale_log2e : -INFINITY;
+                    mt = fmaxf(mt, x[c]);
+                }
             } else {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) { x[c] *= a.scale_log2e; mt = fmaxf(mt, x[c]); }
@@ -352,7 +372,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
             if (GQA) {
                 inv *= a.out_scale;
-                if (a.gate != nullptr && valid)
+                if (a.gate != nullptr && !a.gate_each && valid)
                     inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(a.gate[(size_t) (row0 + r) * a.ld_gate + h])));
             }
             bf16 * dst = a.out + (size_t) (row0 + (valid ? r : 0)) * a.ldo + (size_t) h * DV;
@@ -362,6 +382,15 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
                 tmem_ld16(tm_O + lane_addr + c, v);
                 tmem_ld_wait();
                 uint32_t o[8];
+                if (GQA && a.gate_each && a.gate != nullptr && valid) {
+                    uint4 g[2];
+                    const uint4 * src = (const uint4 *) (a.gate + (size_t) (row0 + r) * a.ld_gate + (size_t) h * DV + c);
+                    g[0] = src[0];
+                    g[1] = src[1];
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        v[j] = __float_as_uint(__fdividef(__uint_as_float(v[j]), 1.f + __expf(-__bfloat162float(((const bf16 *) g)[j]))));
+                }
 #pragma unroll
                 for (int j = 0; j < 16; j += 2) {
                     const __nv_bfloat162 pk = __floats2bfloat162_rn(__uint_as_float(v[j]) * inv, __uint_as_float(v[j + 1]) * inv);
@@ -382,27 +411,28 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 
 // ---- latent rows of the sequences of a batch, gathered from the paged cache into one contiguous buffer ---------------------
 // lat [total][row] <- cache[block_tables[b][s / bs] * bs + s % bs][row] for s < seq_lens[b] (with a window: for the rows the
-// sequence's last q_len tokens can see); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
+// sequence's last q_len tokens can see, and ahead of them the pooled rows its last token sees); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
 __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict__ cache, const int * __restrict__ block_tables, int max_blocks,
                                                         const int * __restrict__ seq_lens, int n_seqs, int block_size, int row_elems,
                                                         long long n_slots, const int * __restrict__ q_start, int window, int chunk,
-                                                        bf16 * __restrict__ lat, int * __restrict__ kv_start, int total_cap) {
+                                                        const bf16 * __restrict__ pool, int pool_size, int pool_rows, bf16 * __restrict__ lat, int * __restrict__ kv_start, int total_cap) {
     PDL_TRIGGER_TOP();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = blockIdx.x * 8 + warp;              // global row of the gathered buffer this warp copies
-    int b = -1, s = 0, acc = 0;
+    int b = -1, s = 0, acc = 0;                       // s < 0: pooled row -1 - s
     for (int i = 0; i < n_seqs; ++i) {
         const int S = seq_lens[i], n = window > 0 || chunk > 0 ? visible_rows(S, q_start[i + 1] - q_start[i], window, chunk) : S;
+        const int np = gqa_blocks_seen(S - 1, window, pool_size);
         if (blockIdx.x == 0 && threadIdx.x == 0) kv_start[i] = acc;
-        if (b < 0 && g < acc + n) { b = i; s = S - n + g - acc; }
-        acc += n;
+        if (b < 0 && g < acc + np + n) { b = i; s = g < acc + np ? acc - g - 1 : S - n + g - acc - np; }
+        acc += np + n;
     }
     if (b < 0 || g >= total_cap) return;
-    const int blk = block_tables[(size_t) b * max_blocks + s / block_size];
-    const long long slot = (long long) blk * block_size + s % block_size;
-    if (slot < 0 || slot >= n_slots) return;
-    const uint4 * src = (const uint4 *) (cache + (size_t) slot * row_elems);
+    const int * bt = block_tables + (size_t) b * max_blocks;
+    const long long slot = s < 0 ? gqa_pool_row(bt, -1 - s, pool_size, pool_rows, block_size) : (long long) bt[s / block_size] * block_size + s % block_size;
+    if (slot < 0 || (s >= 0 && slot >= n_slots)) return;
+    const uint4 * src = (const uint4 *) ((s < 0 ? pool : cache) + (size_t) slot * row_elems);
     uint4 * dst = (uint4 *) (lat + (size_t) g * row_elems);
     for (int i = lane; i < row_elems / 8; i += 32) dst[i] = src[i];
 }
@@ -445,12 +475,13 @@ extern "C" {
 // Gathers the cached rows of all sequences of the batch (seq_lens[b] rows each, or with a window or chunks those the sequence's last
 // q_len[b] tokens can see, in sequence order) from the paged cache layer into lat [total_cap][row_elems] and writes the first row of every sequence to kv_start [n_seqs].
 JIB_EXPORT int jib_kv_gather(const void * cache, long long n_slots, const int * block_tables, int max_blocks, const int * seq_lens,
-                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, void * lat, int * kv_start,
-                             int total_cap, void * stream) {
+                             int n_seqs, int block_size, int row_elems, const int * q_start, int window, int chunk, const void * pool, int pool_size,
+                             int pool_rows, void * lat, int * kv_start, int total_cap, void * stream) {
     if (n_seqs <= 0 || total_cap <= 0) return 0;
-    if (row_elems % 8 || block_size <= 0 || ((window > 0 || chunk > 0) && q_start == nullptr)) return JIB_E_ARG;
+    if (row_elems % 8 || block_size <= 0 || ((window > 0 || chunk > 0) && q_start == nullptr) || (pool_size > 0 && pool == nullptr))
+        return JIB_E_ARG;
     JIB_LAUNCH((kv_gather_kernel), (total_cap + 7) / 8, 256, 0, (cudaStream_t) stream, (const bf16 *) cache, block_tables, max_blocks, seq_lens,
-               n_seqs, block_size, row_elems, n_slots, q_start, window, chunk, (bf16 *) lat, kv_start, total_cap);
+               n_seqs, block_size, row_elems, n_slots, q_start, window, chunk, (const bf16 *) pool, pool_size, pool_rows, (bf16 *) lat, kv_start, total_cap);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 
@@ -489,6 +520,7 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
     if (m->T <= 0 || m->n_seqs <= 0 || n_q_tiles <= 0) return 0;
     if (m->D != DN || m->V != DV || m->H < 1 || m->G < 1 || m->H % m->G || m->row < (long long) m->G * (DN + DV)) return JIB_E_ARG;
     if (ldo % 8 || ((uintptr_t) out & 15) || total <= 0) return JIB_E_ALIGN;
+    if (m->gate_each && gate != nullptr && (ld_gate % 8 || ((uintptr_t) gate & 15))) return JIB_E_ALIGN;
     CUtensorMap mq, mkv;
     int rc = map_2d(&mq, q, m->T, (long long) m->H * DN, (long long) m->H * DN);
     if (rc) return rc;
@@ -500,7 +532,7 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
     a.scale_log2e = m->scale * 1.4426950408889634f;
     a.cap_log2e = m->softcap * 1.4426950408889634f;
     a.inv_cap2 = m->softcap > 0.f ? 2.f * a.scale_log2e / m->softcap : 0.f;
-    a.gate = (const bf16 *) gate; a.ld_gate = ld_gate; a.out_scale = m->out_scale;
+    a.gate = (const bf16 *) gate; a.ld_gate = ld_gate; a.out_scale = m->out_scale; a.pool_size = m->pool_size; a.gate_each = m->gate_each;
     constexpr int SMEM = Form<true>::SMEM_BYTES;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(mha_prefill_kernel<true>, SMEM, attr_done)) return JIB_E_LAUNCH;

@@ -283,7 +283,8 @@ __global__ void __launch_bounds__(32) moe_gate_kernel(const float * __restrict__
 constexpr int SORT_SMEM_MAX = 4096;
 __device__ __noinline__ void sort_pairs(const int * __restrict__ ids, int n, int k, int expert_base, int E_local, int * __restrict__ seg,
                                            int * __restrict__ src_token, int * __restrict__ dest, int * count, int * offs,
-                                           bool dry = false, int * __restrict__ active = nullptr) {
+                                           bool dry = false, int * __restrict__ active = nullptr, const float * __restrict__ wts = nullptr,
+                                           float * __restrict__ row_wts = nullptr) {
     // dry: same instructions, no global stores (instruction-cache warm-up, see gate_token)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     for (int e = warp; e < E_local; e += nw) {
@@ -343,7 +344,10 @@ __device__ __noinline__ void sort_pairs(const int * __restrict__ ids, int n, int
             if (hit && !dry) {
                 const int row = base + __popc(m & ((1u << lane) - 1));
                 dest[i] = row;
-                if (row < n) src_token[row] = i / k;
+                if (row < n) {
+                    src_token[row] = i / k;
+                    if (row_wts != nullptr) row_wts[row] = wts[i];
+                }
             }
             base += __popc(m);
         }
@@ -352,7 +356,8 @@ __device__ __noinline__ void sort_pairs(const int * __restrict__ ids, int n, int
 
 __global__ void __launch_bounds__(1024) moe_permute_kernel(const int * __restrict__ ids, int n, int k, int expert_base, int E_local,
                                                           int * __restrict__ seg, int * __restrict__ src_token, int * __restrict__ dest,
-                                                          int warm, int * __restrict__ active) {
+                                                          int warm, int * __restrict__ active, const float * __restrict__ wts,
+                                                          float * __restrict__ row_wts) {
     JIB_KS(11, 0);
     PDL_TRIGGER_TOP();
     __shared__ int count[MAX_E + 1];
@@ -370,7 +375,7 @@ __global__ void __launch_bounds__(1024) moe_permute_kernel(const int * __restric
         for (int i = threadIdx.x; i < n; i += blockDim.x) ids_s[i] = ids[i];
         __syncthreads();
     }
-    sort_pairs(n <= SORT_SMEM_MAX ? ids_s : ids, n, k, expert_base, E_local, seg, src_token, dest, count, offs, false, active);
+    sort_pairs(n <= SORT_SMEM_MAX ? ids_s : ids, n, k, expert_base, E_local, seg, src_token, dest, count, offs, false, active, wts, row_wts);
     JIB_KS(11, 9);
 }
 
@@ -427,7 +432,8 @@ __global__ void __launch_bounds__(MAX_E) permute_scan_kernel(int * __restrict__ 
 
 __global__ void __launch_bounds__(PERM_CHUNK) permute_scatter_kernel(const int * __restrict__ ids, int n, int k, int expert_base, int E_local,
                                                                      const int * __restrict__ tmp, int * __restrict__ src_token,
-                                                                     int * __restrict__ dest) {
+                                                                     int * __restrict__ dest, const float * __restrict__ wts,
+                                                                     float * __restrict__ row_wts) {
     PDL_TRIGGER_TOP();
     pdl_wait();
     extern __shared__ int warp_cnt[];              // [32 warps][E_local]: pairs of expert e in warp w, then their prefix over w
@@ -456,7 +462,10 @@ __global__ void __launch_bounds__(PERM_CHUNK) permute_scatter_kernel(const int *
         } else {
             const int row = tmp[(size_t) blockIdx.x * E_local + le] + warp_cnt[warp * E_local + le] + rank;
             dest[i] = row;
-            if (row < n) src_token[row] = i / k;
+            if (row < n) {
+                src_token[row] = i / k;
+                if (row_wts != nullptr) row_wts[row] = wts[i];
+            }
         }
     }
 }
@@ -784,11 +793,12 @@ int jib_moe_route_fused(const void * g, const float * w_router, const float * bi
     return launched();
 }
 
-int jib_moe_permute(const int * ids, int T, int k, int expert_base, int E_local, int * seg, int * src_token, int * dest, void * stream) {
+int jib_moe_permute(const int * ids, int T, int k, int expert_base, int E_local, int * seg, int * src_token, int * dest, const float * wts,
+                    float * row_wts, void * stream) {
     if (T <= 0) return 0;
-    if (E_local > MAX_E) return JIB_E_ARG;
+    if (E_local > MAX_E || (row_wts != nullptr && wts == nullptr)) return JIB_E_ARG;
     JIB_LAUNCH((moe_permute_kernel), 1, 1024, 0, (cudaStream_t) stream, ids, T * k, k, expert_base, E_local, seg, src_token, dest,
-               jib::warm_for(T), seg + E_local + 1);
+               jib::warm_for(T), seg + E_local + 1, wts, row_wts);
     return launched();
 }
 
@@ -800,9 +810,9 @@ int jib_moe_tile_list(const int * seg, int E_local, int bn, int * out, int cap, 
 
 // Same contract as jib_moe_permute, for large n: three launches over ceil(n / 1024) CTAs.  tmp: device int[ceil(T*k/1024) * E_local].
 int jib_moe_permute_multi(const int * ids, int T, int k, int expert_base, int E_local, int * seg, int * src_token, int * dest, int * tmp,
-                          void * stream) {
+                          const float * wts, float * row_wts, void * stream) {
     if (T <= 0) return 0;
-    if (E_local > MAX_E || tmp == nullptr) return JIB_E_ARG;
+    if (E_local > MAX_E || tmp == nullptr || (row_wts != nullptr && wts == nullptr)) return JIB_E_ARG;
     const int n = T * k;
     const int n_chunks = (n + PERM_CHUNK - 1) / PERM_CHUNK;
     const size_t smem = (size_t) 32 * E_local * sizeof(int);
@@ -810,7 +820,7 @@ int jib_moe_permute_multi(const int * ids, int T, int k, int expert_base, int E_
     JIB_LAUNCH((permute_count_kernel), n_chunks, PERM_CHUNK, 0, (cudaStream_t) stream, ids, n, expert_base, E_local, tmp);
     JIB_LAUNCH((permute_scan_kernel), 1, MAX_E, 0, (cudaStream_t) stream, tmp, n_chunks, E_local, n, seg, src_token);
     JIB_LAUNCH((permute_scatter_kernel), n_chunks, PERM_CHUNK, smem, (cudaStream_t) stream, ids, n, k, expert_base, E_local,
-               (const int *) tmp, src_token, dest);
+               (const int *) tmp, src_token, dest, wts, row_wts);
     return launched();
 }
 

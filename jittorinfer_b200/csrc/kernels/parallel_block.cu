@@ -80,12 +80,36 @@ template <typename T> __device__ __forceinline__ float sigmoid(float v);
 template <> __device__ __forceinline__ float sigmoid<bf16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
 template <> __device__ __forceinline__ float sigmoid<float>(float v) { return 1.f / (1.f + expf(-v)); }
 
+constexpr int MAX_PARTS = 1024;      // equal parts of a row that a norm is taken over one by one
+
+// 1 / rms of the part that each of a thread's vectors belongs to, from the vectors' sums of squares.  gs: NT * MAXV + MAX_PARTS floats; parts
+// are whole vectors.
+template <int NT, int MAXV>
+__device__ __forceinline__ void part_inverses(const float (&ss)[MAXV], int d, int parts, float eps, float * gs, float (&inv)[MAXV]) {
+    const int nv = d / 8, per = nv / parts;
+    float * out = gs + NT * MAXV;
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it)
+        if (threadIdx.x + it * NT < nv) gs[threadIdx.x + it * NT] = ss[it];
+    __syncthreads();
+    for (int g = threadIdx.x >> 5; g < parts; g += NT / 32) {
+        float s = 0.f;
+        for (int i = threadIdx.x & 31; i < per; i += 32) s += gs[g * per + i];
+        s = warp_sum(s);
+        if ((threadIdx.x & 31) == 0) out[g] = rsqrtf(s / (float) (8 * per) + eps);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int it = 0; it < MAXV; ++it) inv[it] = out[min((int) (threadIdx.x + it * NT) / per, parts - 1)];
+}
+
 constexpr int FAST_TAPS = 4;         // up to this many taps the stored rows are requested before the row's reductions
 
 // x row -> residual store, norm, and (decode) the next block's input convolution.
-// CONV: the tail has the convolution (decode: registers for latency); else (prompts) occupancy matters.
-template <typename T, int NT, int MAXV, bool CONV>
-__device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, const jib_row_tail & a, float * red, bool dry) {
+// CONV: the tail has the convolution (decode: registers for latency); else (prompts) occupancy matters.  PARTS: the norm is taken part by
+// part (gs: see part_inverses).
+template <typename T, int NT, int MAXV, bool CONV, bool PARTS = false>
+__device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, const jib_row_tail & a, float * red, bool dry, float * gs = nullptr) {
     const int nv = d / 8;
     constexpr bool conv = CONV;
     int slot = -1;
@@ -109,16 +133,20 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
             if (past && j < n_old && threadIdx.x < nv) old[j].load(state + (size_t) j * d + 8 * threadIdx.x);
         }
     }
-    float ss = 0.f;
+    float ss = 0.f, sq[MAXV], invs[MAXV];
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
+        if (PARTS) sq[it] = 0.f;
         if (i < nv) {
             Pack8<float> k;
             k.set(v[it]);
             if (!dry && a.x_out != nullptr) k.store((float *) a.x_out + (size_t) t * d + 8 * i);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+            for (int e = 0; e < 8; ++e) {
+                if (PARTS) sq[it] += v[it][e] * v[it][e];
+                else ss += v[it][e] * v[it][e];
+            }
             if (a.norm_w == nullptr && a.h_out != nullptr && !dry) {
                 Pack8<T> hp;
                 hp.set(v[it]);
@@ -127,12 +155,18 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
         }
     }
     if (a.norm_w == nullptr) return;
-    ss = block_sum<NT>(ss, red);
-    const float inv = rsqrtf(ss / (float) d + a.eps);
+    float inv = 0.f;
+    if (PARTS) {
+        part_inverses<NT, MAXV>(sq, d, a.groups, a.eps, gs, invs);
+    } else {
+        ss = block_sum<NT>(ss, red);
+        inv = rsqrtf(ss / (float) d + a.eps);
+    }
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i >= nv) continue;
+        if (PARTS) inv = invs[it];
         float w[8], h[8];
         load8(a.norm_w + 8 * i, w);
 #pragma unroll
@@ -189,11 +223,12 @@ __device__ __forceinline__ void finish_row(float (&v)[MAXV][8], int t, int d, co
     }
 }
 
-template <typename T, int NT, int MAXV, bool CONV>
+template <typename T, int NT, int MAXV, bool CONV, bool PARTS>
 __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ table, const int * __restrict__ ids, const float * __restrict__ w,
                                                         float eps, float scale, int d, int n_vocab, const jib_row_tail tail) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
+    __shared__ float gs[PARTS ? NT * MAXV + MAX_PARTS : 1];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int t = blockIdx.x;
     int id = ids[t];
@@ -230,7 +265,7 @@ __global__ void __launch_bounds__(NT) embed_norm_kernel(const T * __restrict__ t
             }
         }
     }
-    finish_row<T, NT, MAXV, CONV>(v, t, d, tail, red, false);
+    finish_row<T, NT, MAXV, CONV, PARTS>(v, t, d, tail, red, false, gs);
 }
 
 struct UpdateArgs {
@@ -278,7 +313,7 @@ __device__ __forceinline__ void stage_pairs(const int * dest, const float * w, i
     if (threadIdx.x < k) {
         const int r = dry ? 0 : dest[(size_t) t * k + threadIdx.x];
         rows[threadIdx.x] = r < 0 ? 0 : r;
-        wts[threadIdx.x] = r < 0 ? 0.f : w[(size_t) t * k + threadIdx.x];
+        wts[threadIdx.x] = r < 0 ? 0.f : w == nullptr ? 1.f : w[(size_t) t * k + threadIdx.x];
     }
     __syncthreads();
 }
@@ -390,8 +425,15 @@ struct ScaledArgs {
     int k, d;
 };
 
-template <typename T, int NT, int MAXV>
-__device__ __noinline__ void scaled_update_row(const ScaledArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, bool dry) {
+// a scale per element, or one
+__device__ __forceinline__ void load_scale(Pack8<float> & p, const float * s, int c) {
+    if (s != nullptr) p.load(s + c);
+    else p.a = p.b = make_float4(1.f, 1.f, 1.f, 1.f);
+}
+
+template <typename T, int NT, int MAXV, bool PARTS>
+__device__ __noinline__ void scaled_update_row(const ScaledArgs & a, const jib_row_tail & tail, float * red, int * rows, float * wts, float * gs,
+                                               bool dry) {
     const int t = blockIdx.x, d = a.d, nv = d / 8;
     if (a.y != nullptr) stage_pairs(a.dest, a.wts, a.k, t, dry, rows, wts);
     const float g = a.f_gate != nullptr ? sigmoid<T>(a.f_gate[(size_t) t * a.ld_gate]) : 1.f;
@@ -406,9 +448,9 @@ __device__ __noinline__ void scaled_update_row(const ScaledArgs & a, const jib_r
         op.zero(); fp.zero(); s1p.zero(); s2p.zero();
         if (a.o != nullptr) {
             op.load((const T *) a.o + (size_t) t * d + 8 * i);
-            s1p.load(a.s1 + 8 * i);
+            load_scale(s1p, a.s1, 8 * i);
         }
-        if (a.y != nullptr || a.f != nullptr) s2p.load(a.s2 + 8 * i);
+        if (a.y != nullptr || a.f != nullptr) load_scale(s2p, a.s2, 8 * i);
         if (a.f != nullptr) fp.load((const T *) a.f + (size_t) t * d + 8 * i);
         float sum[8], p[8], q[8];
         if (a.y != nullptr) {
@@ -427,21 +469,22 @@ __device__ __noinline__ void scaled_update_row(const ScaledArgs & a, const jib_r
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[it][e] = p[e] + sum[e];
     }
-    finish_row<T, NT, MAXV, false>(v, t, d, tail, red, dry);
+    finish_row<T, NT, MAXV, false, PARTS>(v, t, d, tail, red, dry, gs);
 }
 
-template <typename T, int NT, int MAXV>
+template <typename T, int NT, int MAXV, bool PARTS>
 __global__ void __launch_bounds__(NT) scaled_update_kernel(const __grid_constant__ ScaledArgs a, const __grid_constant__ jib_row_tail tail, int warm) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
     __shared__ int rows[MAX_TOP];
     __shared__ float wts[MAX_TOP];
+    __shared__ float gs[PARTS ? NT * MAXV + MAX_PARTS : 1];
     if (warm) {
-        scaled_update_row<T, NT, MAXV>(a, tail, red, rows, wts, true);
+        scaled_update_row<T, NT, MAXV, PARTS>(a, tail, red, rows, wts, gs, true);
         __syncthreads();
     }
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    scaled_update_row<T, NT, MAXV>(a, tail, red, rows, wts, false);
+    scaled_update_row<T, NT, MAXV, PARTS>(a, tail, red, rows, wts, gs, false);
 }
 
 // The row kernels for widths that 8-element vectors do not divide: element by element, the row re-read from memory.
@@ -472,6 +515,7 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
     __shared__ float red[32];
     __shared__ int pair_rows[MAX_TOP];
     __shared__ float pair_wts[MAX_TOP];
+    __shared__ float part_inv[MAX_PARTS];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int t = blockIdx.x, d = a.d;
     const ScaledArgs & u = a.u;
@@ -506,23 +550,39 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
             float f = u.f != nullptr ? gate * as_f<T>(u.f, row * d + i) : 0.f;
             if (u.y != nullptr)
                 for (int j = 0; j < u.k; ++j) f += pair_wts[j] * as_f<T>(u.y, (size_t) pair_rows[j] * d + i);
-            v += u.s2[i] * f;
+            v += (u.s2 != nullptr ? u.s2[i] : 1.f) * f;
         }
-        if (u.o != nullptr) v += u.s1[i] * as_f<T>(u.o, row * d + i);
+        if (u.o != nullptr) v += (u.s1 != nullptr ? u.s1[i] : 1.f) * as_f<T>(u.o, row * d + i);
         return a.x != nullptr ? v + a.x[row * d + i] : v;
     };
     float * xo = (float *) tail.x_out;
     float ss = 0.f;
+    const int parts = tail.norm_w != nullptr && tail.groups > 1 ? tail.groups : 1, part = d / parts;
     for (int i = threadIdx.x; i < d; i += 256) {
+        if (parts > 1) break;
         const float v = value(i);
         ss += v * v;
         if (tail.norm_w == nullptr && tail.h_out != nullptr) put_f((T *) tail.h_out + (size_t) t * d + i, v);
         if (tail.norm_w == nullptr && xo != nullptr) xo[(size_t) t * d + i] = v;
     }
     if (tail.norm_w == nullptr) return;
-    const float ni = rsqrtf(block_sum<256>(ss, red) / (float) d + tail.eps);
+    if (parts > 1) {
+        for (int g = threadIdx.x >> 5; g < parts; g += 8) {
+            float s = 0.f;
+            for (int i = threadIdx.x & 31; i < part; i += 32) {
+                const float v = value(g * part + i);
+                s += v * v;
+            }
+            s = warp_sum(s);
+            if ((threadIdx.x & 31) == 0) part_inv[g] = rsqrtf(s / (float) part + tail.eps);
+        }
+        __syncthreads();
+    } else {
+        ss = block_sum<256>(ss, red);
+    }
+    const float all_inv = rsqrtf(ss / (float) d + tail.eps);
     for (int i = threadIdx.x; i < d; i += 256) {
-        const float v = value(i);
+        const float v = value(i), ni = parts > 1 ? part_inv[i / part] : all_inv;
         put_f((T *) tail.h_out + (size_t) t * d + i, v * ni * tail.norm_w[i]);
         if (tail.norm2_w != nullptr) put_f((T *) tail.h2_out + (size_t) t * d + i, v * ni * tail.norm2_w[i]);
         if (xo != nullptr) xo[(size_t) t * d + i] = v;            // last: x_out may be x
@@ -530,32 +590,41 @@ __global__ void __launch_bounds__(256) any_row_kernel(const AnyRow a, const jib_
 }
 
 // out[i] = x[rows[i]] / rms * w
-template <typename T, int NT, int MAXV>
+template <typename T, int NT, int MAXV, bool PARTS>
 __global__ void __launch_bounds__(NT) rms_rows_kernel(const float * __restrict__ x, const int * __restrict__ rows, const float * __restrict__ w,
-                                                      float eps, int d, int n_src, T * __restrict__ out) {
+                                                      float eps, int d, int n_src, int parts, T * __restrict__ out) {
     PDL_TRIGGER_TOP();
     __shared__ float red[32];
+    __shared__ float gs[PARTS ? NT * MAXV + MAX_PARTS : 1];
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     int r = rows != nullptr ? rows[blockIdx.x] : (int) blockIdx.x;
     r = r < 0 ? 0 : (r >= n_src ? n_src - 1 : r);
     const int nv = d / 8;
     float v[MAXV][8];
-    float ss = 0.f;
+    float ss = 0.f, sq[MAXV], invs[MAXV];
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
+        sq[it] = 0.f;
         if (i < nv) {
             load8(x + (size_t) r * d + 8 * i, v[it]);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss += v[it][e] * v[it][e];
+            for (int e = 0; e < 8; ++e) sq[it] += v[it][e] * v[it][e];
         }
+        ss += sq[it];
     }
-    ss = block_sum<NT>(ss, red);
-    const float inv = rsqrtf(ss / (float) d + eps);
+    float inv = 0.f;
+    if (PARTS) {
+        part_inverses<NT, MAXV>(sq, d, parts, eps, gs, invs);
+    } else {
+        ss = block_sum<NT>(ss, red);
+        inv = rsqrtf(ss / (float) d + eps);
+    }
 #pragma unroll
     for (int it = 0; it < MAXV; ++it) {
         const int i = threadIdx.x + it * NT;
         if (i < nv) {
+            if (PARTS) inv = invs[it];
             float k[8];
             load8(w + 8 * i, k);
 #pragma unroll
@@ -572,6 +641,7 @@ inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAU
 inline bool tail_ok(const jib_row_tail * t, int d) {
     if (t == nullptr || t->x_out == nullptr || d > 16384) return false;
     if (t->norm2_w != nullptr && (t->norm_w == nullptr || t->h2_out == nullptr || t->conv_w != nullptr)) return false;
+    if (t->groups > 1 && (t->groups > MAX_PARTS || d % t->groups || t->conv_w != nullptr)) return false;
     if (d % 8) return t->conv_w == nullptr && (t->norm_w == nullptr || t->h_out != nullptr);      // the element-wise kernel
     if (t->norm_w != nullptr && t->h_out == nullptr) return false;
     if (t->conv_w != nullptr)
@@ -579,6 +649,8 @@ inline bool tail_ok(const jib_row_tail * t, int d) {
                t->seq_slots != nullptr && t->positions != nullptr && t->n_state >= 0;
     return true;
 }
+// rows (or parts of rows) that 8-element vectors do not divide take the element-wise kernel
+inline bool by_element(int d, int parts) { return d % 8 || (parts > 1 && d / parts % 8); }
 
 }  // namespace
 
@@ -604,21 +676,24 @@ JIB_EXPORT int jib_embed_norm(const void * table, const int * ids, const float *
     if (T <= 0) return 0;
     if (!tail_ok(tail, d)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
-    if (d % 8) {
+    if (by_element(d, tail->groups)) {
         AnyRow a = {};
         a.src = table; a.ids = ids; a.w = w; a.eps = eps; a.scale = scale; a.d = d; a.n_src = n_vocab;
         return launch_any(a, *tail, T, f32, s);
     }
-#define EMBED(TT, NT, MAXV, CONV) \
-    JIB_LAUNCH((embed_norm_kernel<TT, NT, MAXV, CONV>), T, NT, 0, s, (const TT *) table, ids, w, eps, scale, d, n_vocab, *tail)
+#define EMBED(TT, NT, MAXV, CONV, PARTS) \
+    JIB_LAUNCH((embed_norm_kernel<TT, NT, MAXV, CONV, PARTS>), T, NT, 0, s, (const TT *) table, ids, w, eps, scale, d, n_vocab, *tail)
 #define CALL(NT, MAXV)                                                    \
     do {                                                                  \
         if (tail->conv_w != nullptr) {                                    \
-            if (f32) EMBED(float, NT, MAXV, true);                        \
-            else EMBED(bf16, NT, MAXV, true);                             \
+            if (f32) EMBED(float, NT, MAXV, true, false);                 \
+            else EMBED(bf16, NT, MAXV, true, false);                      \
+        } else if (tail->groups > 1) {                                    \
+            if (f32) EMBED(float, NT, MAXV, false, true);                 \
+            else EMBED(bf16, NT, MAXV, false, true);                      \
         } else {                                                          \
-            if (f32) EMBED(float, NT, MAXV, false);                       \
-            else EMBED(bf16, NT, MAXV, false);                            \
+            if (f32) EMBED(float, NT, MAXV, false, false);                \
+            else EMBED(bf16, NT, MAXV, false, false);                     \
         }                                                                 \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
@@ -631,7 +706,7 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
                                 const float * b2, const void * y, const int * dest, const float * wts, int k, int T, int d, int f32,
                                 const jib_row_tail * tail, void * stream) {
     if (T <= 0) return 0;
-    if (!tail_ok(tail, d) || d % 8 || gate_stride % 8 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1 || k > MAX_TOP))) return JIB_E_ARG;
+    if (!tail_ok(tail, d) || tail->groups > 1 || d % 8 || gate_stride % 8 || (y != nullptr && (dest == nullptr || wts == nullptr || b2 == nullptr || k < 1 || k > MAX_TOP))) return JIB_E_ARG;
     UpdateArgs a;
     a.x = x; a.o = o; a.gates = gates; a.b1 = b1; a.b2 = b2; a.y = y; a.dest = dest; a.wts = wts; a.gate_stride = gate_stride;
     a.k = k; a.d = d; a.mult = mult;
@@ -657,7 +732,7 @@ JIB_EXPORT int jib_block_update(const float * x, float mult, const void * o, con
 JIB_EXPORT int jib_post_norm(const float * x, const void * y, const float * w, float eps, int T, int d, int f32, const jib_row_tail * tail,
                              void * stream) {
     if (T <= 0) return 0;
-    if (!tail_ok(tail, d) || tail->conv_w != nullptr || w == nullptr) return JIB_E_ARG;
+    if (!tail_ok(tail, d) || tail->groups > 1 || tail->conv_w != nullptr || w == nullptr) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
     if (d % 8) {
         AnyRow a = {};
@@ -681,48 +756,61 @@ JIB_EXPORT int jib_scaled_update(const float * x, const void * o, const float * 
     if (T <= 0) return 0;
     jib_row_tail chk = *tail;
     if (chk.x_out == nullptr) chk.x_out = (void *) x;
-    if (!tail_ok(&chk, d) || tail->conv_w != nullptr || (o != nullptr && s1 == nullptr) || ((y != nullptr || f != nullptr) && s2 == nullptr) ||
-        (y != nullptr && (dest == nullptr || wts == nullptr || k < 1 || k > MAX_TOP)))
+    if (!tail_ok(&chk, d) || tail->conv_w != nullptr || (y != nullptr && (dest == nullptr || k < 1 || k > MAX_TOP)))
         return JIB_E_ARG;
     ScaledArgs a;
     a.x = x; a.o = o; a.y = y; a.f = f; a.s1 = s1; a.s2 = s2; a.dest = dest; a.wts = wts; a.f_gate = f_gate; a.ld_gate = ld_gate;
     a.k = k; a.d = d;
     cudaStream_t s = (cudaStream_t) stream;
-    if (d % 8) {
+    if (by_element(d, tail->groups)) {
         AnyRow r = {};
         r.x = x; r.d = d; r.n_src = T; r.scale = 1.f; r.u = a;
         return launch_any(r, *tail, T, f32, s);
     }
     const int warm = jib::warm_for(T);
-#define CALL(NT, MAXV)                                                                                    \
-    do {                                                                                                  \
-        if (f32) JIB_LAUNCH((scaled_update_kernel<float, NT, MAXV>), T, NT, 0, s, a, *tail, warm);        \
-        else JIB_LAUNCH((scaled_update_kernel<bf16, NT, MAXV>), T, NT, 0, s, a, *tail, warm);             \
+#define UPDATE(TT, NT, MAXV, PARTS) JIB_LAUNCH((scaled_update_kernel<TT, NT, MAXV, PARTS>), T, NT, 0, s, a, *tail, warm)
+#define CALL(NT, MAXV)                                                    \
+    do {                                                                  \
+        if (tail->norm_w != nullptr && tail->groups > 1) {                \
+            if (f32) UPDATE(float, NT, MAXV, true);                       \
+            else UPDATE(bf16, NT, MAXV, true);                            \
+        } else {                                                          \
+            if (f32) UPDATE(float, NT, MAXV, false);                      \
+            else UPDATE(bf16, NT, MAXV, false);                           \
+        }                                                                 \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
 #undef CALL
+#undef UPDATE
     return launched();
 }
 
-JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int f32, void * out,
+JIB_EXPORT int jib_rms_rows(const float * x, const int * rows, const float * w, float eps, int n, int d, int n_src, int groups, int f32, void * out,
                             void * stream) {
     if (n <= 0) return 0;
-    if (d > 16384 || n_src <= 0) return JIB_E_ARG;
+    if (d > 16384 || n_src <= 0 || groups < 1 || groups > MAX_PARTS || d % groups) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
-    if (d % 8) {
+    if (by_element(d, groups)) {
         AnyRow a = {};
         jib_row_tail t = {};
         a.x = x; a.rows = rows; a.d = d; a.n_src = n_src; a.scale = 1.f;
-        t.norm_w = w; t.eps = eps; t.h_out = out;
+        t.norm_w = w; t.eps = eps; t.h_out = out; t.groups = groups;
         return launch_any(a, t, n, f32, s);
     }
-#define CALL(NT, MAXV)                                                                                                       \
-    do {                                                                                                                     \
-        if (f32) JIB_LAUNCH((rms_rows_kernel<float, NT, MAXV>), n, NT, 0, s, x, rows, w, eps, d, n_src, (float *) out);      \
-        else JIB_LAUNCH((rms_rows_kernel<bf16, NT, MAXV>), n, NT, 0, s, x, rows, w, eps, d, n_src, (bf16 *) out);            \
+#define ROWS(TT, NT, MAXV, PARTS) JIB_LAUNCH((rms_rows_kernel<TT, NT, MAXV, PARTS>), n, NT, 0, s, x, rows, w, eps, d, n_src, groups, (TT *) out)
+#define CALL(NT, MAXV)                                                    \
+    do {                                                                  \
+        if (groups > 1) {                                                 \
+            if (f32) ROWS(float, NT, MAXV, true);                         \
+            else ROWS(bf16, NT, MAXV, true);                              \
+        } else {                                                          \
+            if (f32) ROWS(float, NT, MAXV, false);                        \
+            else ROWS(bf16, NT, MAXV, false);                             \
+        }                                                                 \
     } while (0)
     JIB_ROW_DISPATCH(d, CALL);
 #undef CALL
+#undef ROWS
     return launched();
 }
 

@@ -10,6 +10,8 @@
 // Every exponent that occurs is a difference G_t - G_s with s <= t and so at most 0, however fast the decay: nothing overflows and no
 // quotient of vanishing products is formed.
 //   prepare (one CTA per chunk and head; SSD: per chunk and group): convolution, unit norm, decays, A, W, U0.  Independent of S.
+//   HGRN is LINEAR with q, k and decays of its own; MLSTM is SSD without groups whose decays and factors mlstm_gates has written, with one more
+//   value column (v = 1): the state of that column is what the keys add up to.
 //   pass    (K / 32 warps per head and 16 value columns): walks the chunks, S in registers, everything else a product of small matrices.
 // State, decays, A, W, U0 are fp32; the tensor cores see each as a sum of two bf16 numbers and the products hi * hi + hi * lo + lo * hi
 // (about 16 bits of mantissa); q and k of SSD are bf16 to begin with.  Accumulation is fp32.
@@ -22,15 +24,16 @@ using namespace state_mix;
 
 constexpr int C = 32, NT = 256;                              // tokens of a chunk; threads of prepare
 constexpr float LOG2E = 1.4426950408889634f;
+__host__ __device__ constexpr bool per_head(int kind) { return !per_channel(kind); }       // SSD, MLSTM
 
 // A chunk's record: bf16 tiles of 32 rows x K columns in 16-byte units u of row r stored at u ^ (r & 7); A: 32 x 32, unit u ^ (r / 2 & 3).
 template <int KIND, int K> struct Rec {
     static constexpr int TILE = C * K * 2, ATILE = C * C * 2;
-    static constexpr int Q = 0, D = KIND == SSD ? TILE : 2 * TILE;                        // q e^G, k e^{G_C - G} (SSD: q, k)
-    static constexpr int A = KIND == SSD ? 2 * TILE : 4 * TILE;                           // hi, lo
+    static constexpr int Q = 0, D = per_head(KIND) ? TILE : 2 * TILE;                     // q e^G, k e^{G_C - G} (SSD: q, k)
+    static constexpr int A = per_head(KIND) ? 2 * TILE : 4 * TILE;                        // hi, lo
     static constexpr int W = A + 2 * ATILE;                                               // DELTA
     static constexpr int E = W + (KIND == DELTA ? 2 * TILE : 0);                          // e^{G_C}; SSD: e^{G_t}, then s_t e^{G_C - G_t}
-    static constexpr int BYTES = E + (KIND == SSD ? 2 * C : K) * 4;
+    static constexpr int BYTES = E + (per_head(KIND) ? 2 * C : K) * 4;
 };
 // SSD: q and k (the first A bytes) are shared by a group; the rest is per head and lies behind all groups' parts.
 template <int K> __device__ __forceinline__ uint8_t * ssd_group_part(const jib_state_mix & a, int ci, int group) {
@@ -187,6 +190,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         float x[8][4];
         float * dst;
         int ld, col, run;
+        if (KIND == HGRN && j >= jk && j < 2 * jk + jv) continue;              // k comes with the decays, the pass reads the values where they are
         if (j < 2 * jk + jv) {
             const int jj = j < jk ? j : j < 2 * jk ? j - jk : j - 2 * jk, w = j < 2 * jk ? K / 4 : V / 4;
             col = jj % w * 4;
@@ -194,6 +198,12 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
             ld = j < 2 * jk ? KS : VS;
             dst = j < jk ? q : j < 2 * jk ? k : v;
             conv_run(a, r0, p0, nr, t0 + run, (j < jk ? a.q_off + h / a.rep * K : j < 2 * jk ? a.k_off + h / a.rep * K : a.v_off + h * V) + col, slot, x);
+            if (KIND == HGRN) {
+#pragma unroll
+                for (int r = 0; r < 8; ++r)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) x[r][e] = silu<bf16>(x[r][e]);
+            }
             if (KIND == LINEAR && j >= 2 * jk) {             // values as they are
 #pragma unroll
                 for (int r = 0; r < 8; ++r) {
@@ -211,15 +221,33 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
             dst = G;
             const bf16 * z = (const bf16 *) a.dec_in + (size_t) (r0 + t0) * a.ld_dec + h * K + col;
             const float4 bias = *(const float4 *) (a.bias + h * K + col);
-            const float f = LOG2E * (KIND == DELTA ? a.neg_a[h] : -a.inv_tau);
+            const float f = KIND == HGRN ? 0.f : LOG2E * (KIND == DELTA ? a.neg_a[h] : -a.inv_tau);
 #pragma unroll
             for (int r = 0; r < 8; ++r) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) x[r][e] = 0.f;
                 if (run + r < n) load4(z + (size_t) (run + r) * a.ld_dec, x[r]);
             }
+            if (KIND == HGRN) {
+                const float4 l4 = *(const float4 *) (a.lower + h * K + col);
+                const float l[4] = {l4.x, l4.y, l4.z, l4.w}, bz[4] = {bias.x, bias.y, bias.z, bias.w};
+#pragma unroll
+                for (int r = 0; r < 8; ++r) {
+                    float y[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        float g, rest;
+                        bounded_gate(x[r][e] + bz[e], l[e], g, rest);
+                        const bool in = run + r < n;
+                        y[e] = in ? rest : 0.f;              // log f to a few ulp: near 1 from 1 - f
+                        x[r][e] = in ? LOG2E * (rest < 0.5f ? log1pf(-rest) : logf(fmaxf(g, 1e-37f))) : 0.f;
+                    }
+                    *(float4 *) (k + (run + r) * KS + col) = make_float4(y[0], y[1], y[2], y[3]);
+                }
+            }
 #pragma unroll
             for (int r = 0; r < 8; ++r) {
+                if (KIND == HGRN) break;
                 const float s = KIND == DELTA ? 1.f : -1.f;
                 x[r][0] = run + r < n ? f * softplus_series(s * (x[r][0] + bias.x)) : 0.f;
                 x[r][1] = run + r < n ? f * softplus_series(s * (x[r][1] + bias.y)) : 0.f;
@@ -334,7 +362,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
         put_tile4<K>(rec + R::D, t, c, make_float4(y.x * ex2(e.x - g.x), y.y * ex2(e.y - g.y), y.z * ex2(e.z - g.z), y.w * ex2(e.w - g.w)));
     }
     for (int c = tid; c < K; c += NT) ((float *) (rec + R::E))[c] = ex2(G[(C - 1) * KS + c]);
-    if (KIND == LINEAR) return;
+    if (KIND != DELTA) return;
     float * U = (float *) (rec + R::BYTES);
     __syncthreads();
     // forward substitution, one right-hand side per thread: columns of k e^G, then of v
@@ -373,7 +401,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
 // (A_ts also holds the factor s_s of the earlier token, and D on the diagonal).  Then runs of 256 value columns (bf16 into a.v).
 constexpr int HB = 16;
 
-template <int K>
+template <int KIND, int K>
 __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<SSD, K>;
     constexpr int KS = K + 4;
@@ -423,14 +451,21 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
         for (int i = tid >> 5; i < HB && block * HB + i < a.rep; i += NT / 32) {
             const int h = y * a.rep + block * HB + i;
             uint8_t * hr = ssd_head_part<K>(a, ci, h);
-            const float f = lane < n ? softplus_series(to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + lane) * a.ld + a.s_off + h]) + a.bias[h]) : 0.f;
-            float g = a.neg_a[h] * LOG2E * f;                // lane t: G_t
+            float f = 0.f, g;                                // lane t: s_t, G_t
+            if (KIND == MLSTM) {
+                const size_t at = (size_t) (r0 + t0 + min(lane, n - 1)) * a.H + h;
+                f = lane < n ? a.s[at] : 0.f;
+                g = lane < n ? a.dec[at] : 0.f;
+            } else {
+                if (lane < n) f = softplus_series(to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + lane) * a.ld + a.s_off + h]) + a.bias[h]);
+                g = a.neg_a[h] * LOG2E * f;
+            }
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const float x = __shfl_up_sync(0xffffffffu, g, o);
                 if (lane >= o) g += x;
             }
-            const float gC = __shfl_sync(0xffffffffu, g, 31), skip = a.skip[h];
+            const float gC = __shfl_sync(0xffffffffu, g, 31), skip = KIND == MLSTM ? 0.f : a.skip[h];
             float * e = (float *) (hr + R::E - R::A);
             e[lane] = ex2(g);
             e[C + lane] = f * ex2(gC - g);
@@ -475,7 +510,7 @@ __device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
 template <int KIND, int K> struct Pass {
     using R = Rec<KIND, K>;
     static constexpr int KS = K / 32;                        // warps that share a head's 16 value columns, 32 key channels each
-    static constexpr int NG = (KIND == SSD ? 8 : 4) / KS;    // groups of 16 columns
+    static constexpr int NG = (per_head(KIND) ? 8 : 4) / KS; // groups of 16 columns
     static constexpr int WARPS = KS * NG, PT = WARPS * 32, PV = NG * 16;
     static constexpr int STAGES = KIND == DELTA ? 3 : 4;
     static constexpr int XS = PV * 2 + 16;                   // bytes of a row of v: rows hit different banks
@@ -494,14 +529,19 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     using R = Rec<KIND, K>;
     using P = Pass<KIND, K>;
     constexpr int ST = P::STAGES, KS = P::KS, PT = P::PT, PV = P::PV;
+    constexpr bool HEAD = per_head(KIND);
     extern __shared__ __align__(16) uint8_t smem[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, V = a.V, H = a.H;
-    const int splits = (V + PV - 1) / PV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * PV, b = blockIdx.y;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, V = a.V, H = a.H, VS = scratch_cols(KIND, V);
+    const int NC = V + (KIND == MLSTM ? 16 : 0);             // value columns, those of the keys' sum last
+    // values: rows of proj, or (after a convolution) of a.v
+    const bf16 * val = KIND == HGRN || KIND == MLSTM ? (const bf16 *) a.proj + a.v_off : (const bf16 *) a.v;
+    const size_t ldv = KIND == HGRN || KIND == MLSTM ? (size_t) a.ld : (size_t) H * V;
+    const int splits = (NC + PV - 1) / PV, h = blockIdx.x / splits, v0 = blockIdx.x % splits * PV, b = blockIdx.y;
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int r0 = a.q_start[b], n = a.q_start[b + 1] - r0;
     if (n <= 0) return;
     const int slot = checked_slot(a, b, 46), chunks = (n + C - 1) / C;
-    const int units = min(PV, V - v0) / 8;                   // 8-column units that exist
+    const int units = min(PV, NC - v0) / 8;                  // 8-column units that exist
     const int grp = warp / KS, ks = warp % KS;               // this warp's columns and channels
     const bool active = grp * 2 < units;
     const size_t rec_bytes = R::BYTES + (KIND == DELTA ? C * 4 * V : 0);
@@ -509,10 +549,10 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     auto stage = [&](int i) {
         if (i < chunks) {
             uint8_t * dst = smem + i % ST * P::STAGE;
-            const uint8_t * src = KIND == SSD ? ssd_group_part<K>(a, c0 + i, h / a.rep) : (const uint8_t *) a.chunk + ((size_t) (c0 + i) * H + h) * rec_bytes;
+            const uint8_t * src = HEAD ? ssd_group_part<K>(a, c0 + i, h / a.rep) : (const uint8_t *) a.chunk + ((size_t) (c0 + i) * H + h) * rec_bytes;
 #pragma unroll 4
-            for (int o = tid * 16; o < (KIND == SSD ? R::A : R::BYTES); o += PT * 16) cp16(dst + o, src + o);
-            if (KIND == SSD) {
+            for (int o = tid * 16; o < (HEAD ? R::A : R::BYTES); o += PT * 16) cp16(dst + o, src + o);
+            if (HEAD) {
                 const uint8_t * hr = ssd_head_part<K>(a, c0 + i, h);
                 for (int o = tid * 16; o < R::BYTES - R::A; o += PT * 16) cp16(dst + R::A + o, hr + o);
             }
@@ -523,8 +563,10 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                 for (int j = tid; j < C * (PV / 8); j += PT) {
                     const int row = j / (PV / 8), u = j % (PV / 8);
                     if (row >= m) *(uint4 *) (dst + P::X + row * P::XS + (u << 4)) = make_uint4(0, 0, 0, 0);
+                    else if (KIND == MLSTM && v0 + u * 8 >= V)                 // 1, then zeros
+                        *(uint4 *) (dst + P::X + row * P::XS + (u << 4)) = make_uint4(v0 + u * 8 == V ? 0x3f80 : 0, 0, 0, 0);
                     else if (u < units)
-                        cp16(dst + P::X + row * P::XS + (u << 4), (const bf16 *) a.v + (size_t) (r0 + i * C + row) * H * V + h * V + v0 + u * 8);
+                        cp16(dst + P::X + row * P::XS + (u << 4), val + (size_t) (r0 + i * C + row) * ldv + h * V + v0 + u * 8);
                 }
             }
         }
@@ -537,12 +579,14 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
     const int fr = lane >> 2, fc = (lane & 3) * 2;           // accumulator element: rows fr, fr + 8 (values), columns fc, fc + 1
     const int tr = (lane & 7) + ((lane >> 4) << 3), tu = (lane >> 3) & 1;
     float st[4][4];                                          // 4 tiles of 8 channels
-    float * state = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K + ks * 32) * V + v0 + grp * 16 + fr;
+    const bool sum = KIND == MLSTM && v0 + grp * 16 >= V;    // the columns of the keys' sum, of which one exists
+    const size_t row_at = ((size_t) (slot < 0 ? 0 : slot) * H + h), lds = sum ? 1 : V;
+    float * state = sum ? a.extra + row_at * (K + 1) + ks * 32 : a.state + (row_at * K + ks * 32) * V + v0 + grp * 16 + fr;
     const bool past = slot >= 0 && a.positions[r0] > 0 && active;
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[i][e] = past ? state[(size_t) (i * 8 + fc + (e & 1)) * V + 8 * (e >> 1)] : 0.f;
+        for (int e = 0; e < 4; ++e) st[i][e] = past && (!sum || (fr == 0 && e < 2)) ? state[(i * 8 + fc + (e & 1)) * lds + 8 * (e >> 1)] : 0.f;
     for (int ch = 0; ch < chunks; ++ch) {
         asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
         __syncthreads();                                     // this chunk's record is there; the oldest is free
@@ -552,8 +596,8 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
         const uint32_t A_addr = rec_addr + R::A;
         float4 * part = (float4 *) (smem + P::O) + warp * 128 + lane;          // this warp's partial sums: [4 token tiles][32 lanes]
         uint32_t xh[2][4], xl[2][4], yh[2][4], yl[2][4];     // u^T, hi and lo, 16 tokens at a time (x: of the read-out, y: of the update)
-        const float * eg = (const float *) (rec + R::E), * wt = eg + C;        // SSD
-        const float dC = KIND == SSD ? eg[C - 1] : 0.f;
+        const float * eg = (const float *) (rec + R::E), * wt = eg + C;        // SSD, MLSTM
+        const float dC = HEAD ? eg[C - 1] : 0.f;
         if (active) {
             float o[4][4], w[4][4];
 #pragma unroll
@@ -589,7 +633,7 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                     mma(o[i], sl[j], y[i][2 * j], y[i][2 * j + 1]);
                 }
             }
-            if (KIND != SSD) {
+            if (!HEAD) {
                 if (KIND == DELTA) rows(z, R::W + R::TILE);
                 rows(y, R::Q + R::TILE);
 #pragma unroll
@@ -630,7 +674,7 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
 #pragma unroll
                 for (int e = 0; e < 2; ++e) ldm4t(xh[e], rec_addr + P::X + (e * 16 + tr) * P::XS + ((grp * 2 + tu) << 4));
             }
-            if (KIND == SSD) {
+            if (HEAD) {
 #pragma unroll
                 for (int e = 0; e < 2; ++e)
 #pragma unroll
@@ -649,20 +693,20 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
             for (int i = 0; i < 4; ++i) {
                 const uint32_t off = lane * (K * 2) + (((ks * 4 + i) ^ (lane & 7)) << 4);
                 ldm4t(y[i], rec_addr + R::D + off);
-                if (KIND != SSD) ldm4t(z[i], rec_addr + R::D + R::TILE + off);
+                if (!HEAD) ldm4t(z[i], rec_addr + R::D + R::TILE + off);
                 float2 d = make_float2(dC, dC);
-                if (KIND != SSD) d = *(const float2 *) (rec + R::E + (ks * 32 + i * 8 + fc) * 4);
+                if (!HEAD) d = *(const float2 *) (rec + R::E + (ks * 32 + i * 8 + fc) * 4);
                 st[i][0] *= d.x; st[i][1] *= d.y; st[i][2] *= d.x; st[i][3] *= d.y;
             }
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
 #pragma unroll
-                for (int i = 0; i < 4; ++i) mma(st[i], KIND == SSD ? yh[e] : xh[e], y[i][2 * e], y[i][2 * e + 1]);
-                if (KIND != LINEAR) {
+                for (int i = 0; i < 4; ++i) mma(st[i], HEAD ? yh[e] : xh[e], y[i][2 * e], y[i][2 * e + 1]);
+                if (KIND == DELTA || HEAD) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) mma(st[i], KIND == SSD ? yl[e] : xl[e], y[i][2 * e], y[i][2 * e + 1]);
+                    for (int i = 0; i < 4; ++i) mma(st[i], HEAD ? yl[e] : xl[e], y[i][2 * e], y[i][2 * e + 1]);
                 }
-                if (KIND != SSD) {
+                if (!HEAD) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) mma(st[i], xh[e], z[i][2 * e], z[i][2 * e + 1]);
                 }
@@ -680,7 +724,7 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
                     const float4 x = all[p * 128];
                     o[0] += x.x; o[1] += x.y; o[2] += x.z; o[3] += x.w;
                 }
-                if (KIND == SSD) {
+                if (HEAD) {
                     const float2 e = *(const float2 *) (eg + i * 8 + fc);
                     o[0] *= e.x; o[1] *= e.y; o[2] *= e.x; o[3] *= e.y;
                 }
@@ -697,7 +741,7 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int t = ch * C + i * 8 + fc + (e & 1);
-                    if (t < n) a.o[((size_t) (r0 + t) * H + h) * V + v0 + grp * 16 + fr + 8 * (e >> 1)] = o[e] + q[e];
+                    if (t < n && (!sum || (fr == 0 && e < 2))) a.o[((size_t) (r0 + t) * H + h) * VS + v0 + grp * 16 + fr + 8 * (e >> 1)] = o[e] + q[e];
                 }
             }
         }
@@ -707,7 +751,8 @@ __global__ void __launch_bounds__(Pass<KIND, K>::PT, 1) chunk_pass_kernel(const 
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) state[(size_t) (i * 8 + fc + (e & 1)) * V + 8 * (e >> 1)] = st[i][e];
+            for (int e = 0; e < 4; ++e)
+                if (!sum || (fr == 0 && e < 2)) state[(i * 8 + fc + (e & 1)) * lds + 8 * (e >> 1)] = st[i][e];
     }
 }
 
@@ -718,7 +763,7 @@ inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAU
 template <int KIND, int K> int launch_pass(const jib_state_mix & a, cudaStream_t s) {
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(chunk_pass_kernel<KIND, K>, Pass<KIND, K>::SMEM, done)) return JIB_E_LAUNCH;
-    chunk_pass_kernel<KIND, K><<<dim3(a.H * ((a.V + Pass<KIND, K>::PV - 1) / Pass<KIND, K>::PV), a.n_seqs), Pass<KIND, K>::PT, Pass<KIND, K>::SMEM, s>>>(a);
+    chunk_pass_kernel<KIND, K><<<dim3(a.H * ((a.V + (KIND == MLSTM ? 16 : 0) + Pass<KIND, K>::PV - 1) / Pass<KIND, K>::PV), a.n_seqs), Pass<KIND, K>::PT, Pass<KIND, K>::SMEM, s>>>(a);
     return launched();
 }
 template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t s) {
@@ -728,19 +773,20 @@ template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t 
     const int rc = launched();
     return rc ? rc : launch_pass<KIND, K>(a, s);
 }
-template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
+template <int KIND, int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     constexpr int smem = (2 * C * (K + 4) + C * (C + 1)) * 4;
-    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(a.T / C + a.n_seqs, a.H / a.rep * ((a.rep + HB - 1) / HB) + (a.H * a.V + 255) / 256), NT, smem, s, a);
+    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<KIND, K>, smem, done)) return JIB_E_LAUNCH;
+    const int values = KIND == MLSTM ? 0 : (a.H * a.V + 255) / 256;      // MLSTM: the pass reads them where they are
+    JIB_LAUNCH((chunk_prepare_ssd_kernel<KIND, K>), dim3(a.T / C + a.n_seqs, a.H / a.rep * ((a.rep + HB - 1) / HB) + values), NT, smem, s, a);
     const int rc = launched();
-    return rc ? rc : launch_pass<SSD, K>(a, s);
+    return rc ? rc : launch_pass<KIND, K>(a, s);
 }
 
 long long rec_bytes(const jib_state_mix & a) {
 #define REC(KIND, FIELD) (a.K == 64 ? Rec<KIND, 64>::FIELD : Rec<KIND, 128>::FIELD)
     const long long nch = a.T / C + a.n_seqs;
-    if (a.kind == SSD) return nch * (a.H / a.rep * REC(SSD, A) + a.H * (REC(SSD, BYTES) - REC(SSD, A)));
+    if (per_head(a.kind)) return nch * (a.H / a.rep * REC(SSD, A) + a.H * (REC(SSD, BYTES) - REC(SSD, A)));
     return nch * a.H * (a.kind == DELTA ? REC(DELTA, BYTES) + C * 4 * a.V : REC(LINEAR, BYTES));
 #undef REC
 }
@@ -748,9 +794,10 @@ long long rec_bytes(const jib_state_mix & a) {
 }  // namespace
 
 bool jib_state_chunk_ok(const jib_state_mix & a) {
-    const long long cols = a.ld | a.q_off | a.k_off | a.v_off | a.conv0 | a.n_conv | (a.kind == SSD ? 0 : a.ld_dec);
+    const long long cols = a.ld | a.q_off | a.k_off | a.v_off | a.conv0 | a.n_conv | (per_head(a.kind) ? 0 : a.ld_dec);
+    if ((a.kind == HGRN || a.kind == MLSTM) && (a.ld % 8 || a.v_off % 8 || a.taps != 0 || ((uintptr_t) a.proj & 15))) return false;
     return (a.K == 64 || a.K == 128) && a.V % 16 == 0 && a.V <= 256 && a.taps <= 4 && cols % 4 == 0 && ((uintptr_t) a.proj & 7) == 0 &&
-           (a.kind == SSD || ((uintptr_t) a.dec_in & 7) == 0) && a.H % a.rep == 0;
+           (per_head(a.kind) || ((uintptr_t) a.dec_in & 7) == 0) && a.H % a.rep == 0;
 }
 
 int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s) {
@@ -758,7 +805,9 @@ int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s) {
     switch (a.kind) {
         case DELTA: return a.K == 64 ? run_chunks<DELTA, 64>(a, s) : run_chunks<DELTA, 128>(a, s);
         case LINEAR: return a.K == 64 ? run_chunks<LINEAR, 64>(a, s) : run_chunks<LINEAR, 128>(a, s);
-        default: return a.K == 64 ? run_chunks_ssd<64>(a, s) : run_chunks_ssd<128>(a, s);
+        case HGRN: return a.K == 64 ? run_chunks<HGRN, 64>(a, s) : run_chunks<HGRN, 128>(a, s);
+        case MLSTM: return a.K == 64 ? run_chunks_ssd<MLSTM, 64>(a, s) : run_chunks_ssd<MLSTM, 128>(a, s);
+        default: return a.K == 64 ? run_chunks_ssd<SSD, 64>(a, s) : run_chunks_ssd<SSD, 128>(a, s);
     }
 }
 

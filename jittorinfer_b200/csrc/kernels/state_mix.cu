@@ -2,17 +2,20 @@
 //
 //   S <- diag(decay_t) S;   u = s_t (v_t - [delta] S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t + D v_t
 //
-// in three kinds that differ in where q, k, v, the decay and the factor s come from:
+// in kinds that differ in where q, k, v, the decay and the factor s come from:
 //   DELTA   q, k unit vectors, one decay per (head, key channel) = exp(-a_h softplus(. + bias)), s = sigmoid(.), the delta term
 //   LINEAR  one decay per (head, key channel) = sigmoid(. + bias)^(1/tau), s = 1
 //   SSD     one decay per head = exp(-a_h s), s = softplus(. + bias); q and k shared by a group of heads
+//   HGRN    one decay f per (head, key channel), bounded from below, k = 1 - f, silu on q, s = 1
+//   MLSTM   one decay per head = exp(f + m - m'), s = exp(i - m'), relative to a running maximum m' = max(f + m, i) of the log gates; a
+//           vector n of keys that decays and grows like the state; o is divided by max(|n . q|, exp(-m')) + 1e-6
 // A window of the projection's columns may pass a short causal convolution and silu first (DELTA: q, k, v; SSD: v, k, q).
-// What follows the read-out: DELTA / LINEAR a norm over each head's V channels times a gate; SSD a gate, then a norm over
-// parts of the row.
+// What follows the read-out: DELTA / LINEAR / MLSTM a norm over each head's V channels times a gate, HGRN the norm alone; SSD a gate, then a
+// norm over parts of the row.
 //
 // Single tokens (decode): state_step does all of it in one launch per layer (SSD: plus the gated norm of whole rows).
-// Portions: state_prep (convolution, unit norm, decays -> fp32), state_scan (the recurrence, token by token), state_finish (gate and
-// norm); bf16 portions of the head sizes it is built for take state_chunk.cu in place of the first two.
+// Portions: state_prep (convolution, unit norm, decays -> fp32; MLSTM: mlstm_gates ahead of it), state_scan (the recurrence, token by token),
+// state_finish (gate and norm); bf16 portions of the head sizes it is built for take state_chunk.cu in place of the first two.
 //
 // A sequence's state lives in row seq_slots[b] of [n_state][H][K][V]; its last convolution inputs in a ring [n_state][taps][channels]
 // whose row p % taps holds position p's.  A range that starts at position 0 starts from zeros whatever the rows hold, so slots are
@@ -33,6 +36,7 @@ using namespace state_mix;
 // ---- portions: inputs of the recurrence in fp32 ------------------------------------------------------------------------------
 // qk [T][2][Hk][K], v [T][H][V], dec [T][H][K] (SSD: [T][H]), s [T][H].  One warp per (token, item); items: q heads, k heads,
 // value heads, then one for the per-head factors and (DELTA, LINEAR) one per head's decays.
+// MLSTM: v and o have one more column, v = 1, whose state is n.
 constexpr int PREP_C = 16;                                   // channels of a q / k head per lane: K <= 32 * PREP_C
 
 template <typename T, int KIND>
@@ -52,10 +56,18 @@ __global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__
         for (int i = 0; i < PREP_C; ++i) {
             const int c = lane + 32 * i;
             v[i] = 0.f;
-            if (c < a.K) v[i] = column<T>(a, t, c0 + c, p, back, slot);
+            if (c >= a.K) continue;
+            if (KIND == HGRN && !is_q) {
+                const int g = (item - Hk) * a.K + c;
+                float f;
+                bounded_gate(to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + g]) + a.bias[g], a.lower[g], f, v[i]);
+            } else {
+                v[i] = column<T>(a, t, c0 + c, p, back, slot);
+                if (KIND == HGRN) v[i] = silu<T>(v[i]);
+            }
             if (KIND == DELTA) ss += v[i] * v[i];
         }
-        float scale = is_q ? a.q_scale : 1.f;
+        float scale = is_q && KIND != MLSTM ? a.q_scale : 1.f;
         if (KIND == DELTA) scale /= sqrtf(warp_sum(ss) + 1e-6f);
         float * out = a.qk + ((size_t) t * 2 * Hk + item) * a.K;
 #pragma unroll
@@ -65,12 +77,13 @@ __global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__
     }
     item -= 2 * Hk;
     if (item < a.H) {
-        for (int c = lane; c < a.V; c += 32)
-            a.v[((size_t) t * a.H + item) * a.V + c] = column<T>(a, t, a.v_off + item * a.V + c, p, back, slot);
+        const int VS = scratch_cols(KIND, a.V);
+        for (int c = lane; c < VS; c += 32)
+            a.v[((size_t) t * a.H + item) * VS + c] = c < a.V ? column<T>(a, t, a.v_off + item * a.V + c, p, back, slot) : c == a.V ? 1.f : 0.f;
         return;
     }
     item -= a.H;
-    if (KIND != LINEAR && item == 0) {
+    if ((KIND == DELTA || KIND == SSD) && item == 0) {
         for (int h = lane; h < a.H; h += 32) {
             const float s = head_factor<KIND>(a, to_f(((const T *) a.proj)[(size_t) t * a.ld + a.s_off + h]), h);
             a.s[(size_t) t * a.H + h] = s;
@@ -78,12 +91,91 @@ __global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__
         }
         return;
     }
-    if (KIND != LINEAR) --item;
-    if (KIND != SSD && item < a.H)
+    if (KIND == DELTA || KIND == SSD) --item;
+    if (per_channel(KIND) && item < a.H)
         for (int c = lane; c < a.K; c += 32) {
             const int i = item * a.K + c;
-            a.dec[(size_t) t * a.H * a.K + i] = channel_decay<KIND>(a, to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + i]) + a.bias[i], item);
+            const float z = to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + i]) + a.bias[i];
+            float f, rest;
+            if (KIND == HGRN) bounded_gate(z, a.lower[i], f, rest);
+            else f = channel_decay<KIND>(a, z, item);
+            a.dec[(size_t) t * a.H * a.K + i] = f;
         }
+}
+
+// ---- portions, MLSTM: gates relative to the running maximum --------------------------------------------------------------------
+// m_t = max(f_t + m_(t-1), i_t) is a composition of maps m -> max(m + A, B).  grid (H, n_seqs): a thread composes the maps of GATE_N tokens, the
+// CTA scans the compositions, then every thread runs its tokens from where it knows m.  Writes the decays (base-2 logarithms with log2), the
+// factors s, the maxima, and the sequence's new maximum.
+constexpr int GATE_NT = 256, GATE_N = 8;
+
+__global__ void __launch_bounds__(GATE_NT) mlstm_gates_kernel(const __grid_constant__ jib_state_mix a, int log2) {
+    __shared__ float wa[GATE_NT / 32], wb[GATE_NT / 32];
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int h = blockIdx.x, b = blockIdx.y, H = a.H, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
+    if (n <= 0) return;
+    const int slot = checked_slot(a, b, 50);
+    float * top = a.extra + ((size_t) (slot < 0 ? 0 : slot) * H + h) * (a.K + 1) + a.K;
+    float m0 = slot >= 0 && a.positions[q0] > 0 ? *top : 0.f;
+    __syncthreads();                                         // read before the last token's thread replaces it
+    for (int t0 = 0; t0 < n; t0 += GATE_NT * GATE_N) {
+        float gi[GATE_N], gf[GATE_N], A = 0.f, B = -INFINITY;
+        const int first = t0 + threadIdx.x * GATE_N;
+#pragma unroll
+        for (int i = 0; i < GATE_N; ++i) {
+            const float * z = (const float *) a.dec_in + (size_t) (q0 + min(first + i, n - 1)) * a.ld_dec + h;
+            gi[i] = z[0];
+            gf[i] = z[H];
+        }
+#pragma unroll
+        for (int i = 0; i < GATE_N; ++i) {
+            gi[i] = first + i < n ? log_input_gate(gi[i], a.gate_cap) : -INFINITY;
+            gf[i] = first + i < n ? log_forget_gate(gf[i], a.gate_cap) : 0.f;
+            A += gf[i];
+            B = fmaxf(B + gf[i], gi[i]);
+        }
+        // exclusive scan: x -> max(x + A, B) of all tokens before this thread's
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float pa = __shfl_up_sync(0xffffffffu, A, o), pb = __shfl_up_sync(0xffffffffu, B, o);
+            if (lane >= o) {
+                B = fmaxf(pb + A, B);
+                A += pa;
+            }
+        }
+        if (lane == 31) {
+            wa[warp] = A;
+            wb[warp] = B;
+        }
+        A = __shfl_up_sync(0xffffffffu, A, 1);
+        B = __shfl_up_sync(0xffffffffu, B, 1);
+        if (lane == 0) {
+            A = 0.f;
+            B = -INFINITY;
+        }
+        __syncthreads();
+        float m = m0, next = m0;
+        for (int w = 0; w < GATE_NT / 32; ++w) {
+            if (w < warp) m = fmaxf(m + wa[w], wb[w]);
+            next = fmaxf(next + wa[w], wb[w]);
+        }
+        m = fmaxf(m + A, B);
+#pragma unroll
+        for (int i = 0; i < GATE_N; ++i) {
+            if (first + i >= n) break;
+            const float x = gf[i] + m, mt = fmaxf(x, gi[i]);
+            const size_t at = (size_t) (q0 + first + i) * H + h;
+            a.dec[at] = log2 ? (x - mt) * 1.4426950408889634f : expf(x - mt);
+            a.s[at] = expf(gi[i] - mt);
+            a.tops[at] = mt;
+            m = mt;
+            if (slot >= 0 && first + i == n - 1) *top = mt;
+        }
+        m0 = next;
+        __syncthreads();                                     // wa, wb are free
+    }
 }
 
 // ---- portions: the recurrence --------------------------------------------------------------------------------------------------
@@ -95,36 +187,38 @@ constexpr int SCAN_NT = 128, SCAN_TT = 8;
 template <typename T, int KIND, int LK>
 __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_constant__ jib_state_mix a, int splits, int aligned) {
     constexpr int KP = LK * 16, VB = SCAN_NT / LK;
-    constexpr int ROW = (KIND == SSD ? 2 : 3) * KP;          // k | q | decay
+    constexpr bool CHANNELS = per_channel(KIND);
+    constexpr int ROW = (CHANNELS ? 3 : 2) * KP;             // k | q | decay
     constexpr int TILE = SCAN_TT * (ROW + VB + 2);
     extern __shared__ float smem[];
     PDL_TRIGGER_TOP();
     const int h = blockIdx.x / splits, v0 = (blockIdx.x % splits) * VB;
     const int b = blockIdx.y, lane = threadIdx.x % LK, col = threadIdx.x / LK;
-    const int K = a.K, V = a.V, H = a.H, Hk = H / a.rep, nv = min(VB, V - v0);
+    const int K = a.K, V = a.V, H = a.H, Hk = H / a.rep, VS = scratch_cols(KIND, V), nv = min(VB, V + (KIND == MLSTM) - v0);
     for (int i = threadIdx.x; i < 2 * TILE; i += SCAN_NT) smem[i] = 0.f;       // channels past K stay zero
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0;
     if (n <= 0) return;
     const int slot = checked_slot(a, b, 46);
     store_conv_tail<T>(a, slot, q0, n, blockIdx.x * SCAN_NT + threadIdx.x, gridDim.x * SCAN_NT);
-    const bool mine = col < nv;
-    float * st = a.state + (((size_t) (slot < 0 ? 0 : slot) * H + h) * K) * V + v0 + col;
+    const bool mine = col < nv, sum = KIND == MLSTM && v0 + col == V;
+    const size_t at = (size_t) (slot < 0 ? 0 : slot) * H + h, ld = sum ? 1 : V;
+    float * st = sum ? a.extra + at * (K + 1) : a.state + at * K * V + v0 + col;
     float s[16];
     const bool past = slot >= 0 && a.positions[q0] > 0;
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
         const int c = ((i >> 2) * LK + lane) * 4 + (i & 3);
-        s[i] = past && mine && c < K ? st[(size_t) c * V] : 0.f;
+        s[i] = past && mine && c < K ? st[c * ld] : 0.f;
     }
     const float * kp = a.qk + ((size_t) q0 * 2 * Hk + Hk + h / a.rep) * K;
     const float * qp = a.qk + ((size_t) q0 * 2 * Hk + h / a.rep) * K;
-    const float * vp = a.v + ((size_t) q0 * H + h) * V + v0;
-    const float * dp = a.dec + (KIND == SSD ? (size_t) q0 * H + h : ((size_t) q0 * H + h) * K);
+    const float * vp = a.v + ((size_t) q0 * H + h) * VS + v0;
+    const float * dp = a.dec + (CHANNELS ? ((size_t) q0 * H + h) * K : (size_t) q0 * H + h);
     const float * sp = a.s + (size_t) q0 * H + h;
     auto stage = [&](int t0, float * d) {
         const int m = min(SCAN_TT, n - t0);
-        constexpr int NR = KIND == SSD ? 2 : 3;
+        constexpr int NR = CHANNELS ? 3 : 2;
         if (aligned) {
             const int k4 = K / 4;
             for (int i = threadIdx.x; i < m * NR * k4; i += SCAN_NT) {
@@ -142,18 +236,18 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
             }
         }
         float * dv = d + SCAN_TT * ROW;
-        for (int i = threadIdx.x; i < m * nv; i += SCAN_NT) cp4(dv + (i / nv) * VB + i % nv, vp + (size_t) (t0 + i / nv) * H * V + i % nv);
+        for (int i = threadIdx.x; i < m * nv; i += SCAN_NT) cp4(dv + (i / nv) * VB + i % nv, vp + (size_t) (t0 + i / nv) * H * VS + i % nv);
         float * ds = dv + SCAN_TT * VB;
         if (threadIdx.x < m) {
-            if (KIND != LINEAR) cp4(ds + threadIdx.x, sp + (size_t) (t0 + threadIdx.x) * H);
-            if (KIND == SSD) cp4(ds + SCAN_TT + threadIdx.x, dp + (size_t) (t0 + threadIdx.x) * H);
+            if (KIND == DELTA || !CHANNELS) cp4(ds + threadIdx.x, sp + (size_t) (t0 + threadIdx.x) * H);
+            if (!CHANNELS) cp4(ds + SCAN_TT + threadIdx.x, dp + (size_t) (t0 + threadIdx.x) * H);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     __syncthreads();
     stage(0, smem);
     const float skip = KIND == SSD ? a.skip[h] : 0.f;
-    float * op = a.o + ((size_t) q0 * H + h) * V + v0 + col;
+    float * op = a.o + ((size_t) q0 * H + h) * VS + v0 + col;
     int buf = 0;
     for (int t0 = 0; t0 < n; t0 += SCAN_TT, buf ^= 1) {
         if (t0 + SCAN_TT < n) {
@@ -175,7 +269,7 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
                 k[4 * j] = x.x; k[4 * j + 1] = x.y; k[4 * j + 2] = x.z; k[4 * j + 3] = x.w;
                 q[4 * j] = y.x; q[4 * j + 1] = y.y; q[4 * j + 2] = y.z; q[4 * j + 3] = y.w;
             }
-            if (KIND == SSD) {
+            if (!CHANNELS) {
                 const float g = ds[SCAN_TT + i];
 #pragma unroll
                 for (int c = 0; c < 16; ++c) s[c] *= g;
@@ -197,7 +291,7 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
                 for (int o = LK / 2; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
                 u = v - r;
             }
-            if (KIND != LINEAR) u *= ds[i];
+            if (KIND == DELTA || !CHANNELS) u *= ds[i];
             float e[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int c = 0; c < 16; ++c) {
@@ -207,7 +301,7 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
             float r = (e[0] + e[1]) + (e[2] + e[3]);
 #pragma unroll
             for (int o = LK / 2; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
-            if (lane == 0 && mine) op[(size_t) (t0 + i) * H * V] = KIND == SSD ? r + skip * v : r;
+            if (lane == 0 && mine) op[(size_t) (t0 + i) * H * VS] = KIND == SSD ? r + skip * v : r;
         }
         __syncthreads();
     }
@@ -215,7 +309,7 @@ __global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_consta
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
             const int c = ((i >> 2) * LK + lane) * 4 + (i & 3);
-            if (c < K) st[(size_t) c * V] = s[i];
+            if (c < K) st[c * ld] = s[i];
         }
     }
 }
@@ -255,16 +349,17 @@ template <int E> __device__ __forceinline__ void store_vals(bf16 * p, const Vals
     }
 }
 
-// DELTA / LINEAR: one warp per (token, head): o / rms(o) * norm_w * gate.  V <= 32 * N * E.
+// All but SSD: one warp per (token, head): o / rms(o) * norm_w [* gate]; MLSTM: o is divided by its size first.  V <= 32 * N * E.
 template <typename T, int KIND, int E, int N>
 __global__ void __launch_bounds__(256) state_finish_kernel(const __grid_constant__ jib_state_mix a) {
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
     const int lane = threadIdx.x & 31, i = blockIdx.x * 8 + (threadIdx.x >> 5), t = i / a.H, h = i % a.H, V = a.V;
     if (t >= a.T) return;
-    const float * o = a.o + (size_t) i * V;
+    const float * o = a.o + (size_t) i * scratch_cols(KIND, V), * norm_w = a.norm_w + (KIND == MLSTM ? h * V : 0);
     const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * V;
     T * y = (T *) a.y + (size_t) t * a.ldy + h * V;
+    const float size = KIND == MLSTM ? a.q_scale / (fmaxf(fabsf(o[V] * a.q_scale), expf(-a.tops[i])) + 1e-6f) : 1.f;
     Vals<E> x[N], g[N], w[N];
     float ss = 0.f;
 #pragma unroll
@@ -272,21 +367,25 @@ __global__ void __launch_bounds__(256) state_finish_kernel(const __grid_constant
         const int c = (lane + 32 * k) * E;
         if (c >= V) continue;
         x[k] = load_vals<E>(o + c);
-        g[k] = load_vals<E>(gate + c);
-        w[k] = load_vals<E>(a.norm_w + c);
+        if (KIND != HGRN) g[k] = load_vals<E>(gate + c);
+        w[k] = load_vals<E>(norm_w + c);
     }
 #pragma unroll
     for (int k = 0; k < N; ++k)
         if ((lane + 32 * k) * E < V)
 #pragma unroll
-            for (int e = 0; e < E; ++e) ss += x[k].v[e] * x[k].v[e];
+            for (int e = 0; e < E; ++e) {
+                if (KIND == MLSTM) x[k].v[e] *= size;
+                ss += x[k].v[e] * x[k].v[e];
+            }
     const float inv = a.out_scale * rsqrtf(warp_sum(ss) / (float) V + a.eps);
 #pragma unroll
     for (int k = 0; k < N; ++k) {
         const int c = (lane + 32 * k) * E;
         if (c >= V) continue;
 #pragma unroll
-        for (int e = 0; e < E; ++e) x[k].v[e] *= inv * w[k].v[e] * (KIND == DELTA ? sigmoid<T>(g[k].v[e]) : silu<T>(g[k].v[e]));
+        for (int e = 0; e < E; ++e)
+            x[k].v[e] *= inv * w[k].v[e] * (KIND == HGRN ? 1.f : KIND == LINEAR ? silu<T>(g[k].v[e]) : sigmoid<T>(g[k].v[e]));
         store_vals<E>(y + c, x[k]);
     }
 }
@@ -394,17 +493,35 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const _
     };
     if (KEEP) load(0);                                       // in flight while the inputs are prepared
     const int hk = h / a.rep;
-    for (int i = tid; i < (KIND == SSD ? 2 : 3) * K + V; i += NT) {
-        if (i < K) sq[i] = column_single<T>(a, t, a.q_off + hk * K + i, p, slot);
+    float n_old[KIND == MLSTM ? 2 : 1];                      // MLSTM: what the keys add up to, K <= 512 on 256 threads or more
+    float * const extra = KIND == MLSTM ? a.extra + ((size_t) (slot < 0 ? 0 : slot) * H + h) * (K + 1) : nullptr;
+    float top = 0.f;
+    if (KIND == MLSTM) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) n_old[j % (KIND == MLSTM ? 2 : 1)] = past && tid + j * NT < K ? extra[tid + j * NT] : 0.f;
+        if (past) top = extra[K];
+    }
+    for (int i = tid; i < (per_channel(KIND) ? 3 : 2) * K + V; i += NT) {
+        if (i < K) sq[i] = KIND == HGRN ? silu<T>(column_single<T>(a, t, a.q_off + hk * K + i, p, slot)) : column_single<T>(a, t, a.q_off + hk * K + i, p, slot);
+        else if (i < 2 * K && KIND == HGRN) continue;        // comes with the decay
         else if (i < 2 * K) sk[i - K] = column_single<T>(a, t, a.k_off + hk * K + i - K, p, slot);
         else if (i < 2 * K + V) sv[i - 2 * K] = column_single<T>(a, t, a.v_off + h * V + i - 2 * K, p, slot);
         else {
             const int c = i - 2 * K - V, g = h * K + c;
-            sd[c] = channel_decay<KIND>(a, to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + g]) + a.bias[g], h);
+            const float z = to_f(((const T *) a.dec_in)[(size_t) t * a.ld_dec + g]) + a.bias[g];
+            if (KIND == HGRN) bounded_gate(z, a.lower[g], sd[c], sk[c]);
+            else sd[c] = channel_decay<KIND>(a, z, h);
         }
     }
     float factor = 1.f, decay = 1.f;
-    if (KIND != LINEAR) factor = head_factor<KIND>(a, to_f(((const T *) a.proj)[(size_t) t * a.ld + a.s_off + h]), h);
+    if (KIND == MLSTM) {
+        const float * z = (const float *) a.dec_in + (size_t) t * a.ld_dec + h;
+        const float gi = log_input_gate(z[0], a.gate_cap), x = log_forget_gate(z[H], a.gate_cap) + top;
+        top = fmaxf(x, gi);
+        decay = expf(x - top);
+        factor = expf(gi - top);
+    }
+    if (KIND == DELTA || KIND == SSD) factor = head_factor<KIND>(a, to_f(((const T *) a.proj)[(size_t) t * a.ld + a.s_off + h]), h);
     if (KIND == SSD) decay = expf(a.neg_a[h] * factor);
     __syncthreads();
     if (a.taps > 1 && slot >= 0) {                           // this position's convolution inputs; no reader of this launch needs the row
@@ -417,6 +534,20 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const _
         }
     }
     float qn = a.q_scale, kn = 1.f;
+    if (KIND == MLSTM) {                                     // n, and its product with q
+        float d = 0.f;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int c = tid + j * NT;
+            if (c >= K) continue;
+            const float x = n_old[j % (KIND == MLSTM ? 2 : 1)] * decay + factor * sk[c];
+            d += x * sq[c];
+            if (slot >= 0) extra[c] = x;
+        }
+        if (slot >= 0 && tid == 0) extra[K] = top;           // read by all threads ahead of the barrier above
+        d = warp_sum(d);
+        if ((tid & 31) == 0) sums[2 + NT / 32 + (tid >> 5)] = d;
+    }
     if (KIND == DELTA) {
         if (tid < 64) {
             const float * x = tid < 32 ? sq : sk;
@@ -466,7 +597,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const _
         for (int i = 0; i < R; ++i) {
             const int r = r0 + rg + i * nrg;
             if (r >= K || !live) continue;
-            const float g = KIND == SSD ? decay : sd[r], kk = sk[r], qq = sq[r];
+            const float g = per_channel(KIND) ? sd[r] : decay, kk = sk[r], qq = sq[r];
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
                 s[i].v[e] = s[i].v[e] * g + kk * u.v[e];
@@ -494,12 +625,19 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const _
     __syncthreads();
     ss = 0.f;
     for (int i = 0; i < NT / 32; ++i) ss += sums[2 + i];
-    const float inv = a.out_scale * rsqrtf(ss / (float) V + a.eps);
+    float size = 1.f;
+    if (KIND == MLSTM) {
+        float d = 0.f;
+        for (int i = 0; i < NT / 32; ++i) d += sums[2 + NT / 32 + i];
+        size = 1.f / (fmaxf(fabsf(d * qn), expf(-top)) + 1e-6f);
+    }
+    const float inv = a.out_scale * size * rsqrtf(ss * size * size / (float) V + a.eps);
     const T * gate = (const T *) a.gate + (size_t) t * a.ld_gate + h * V;
+    const float * norm_w = a.norm_w + (KIND == MLSTM ? h * V : 0);
     T * y = (T *) a.y + (size_t) t * a.ldy + h * V;
     for (int c = tid; c < V; c += NT) {
-        const float g = to_f(gate[c]);
-        put(y + c, sv[c] * inv * a.norm_w[c] * (KIND == DELTA ? sigmoid<T>(g) : silu<T>(g)));
+        const float g = KIND == HGRN ? 0.f : to_f(gate[c]);
+        put(y + c, sv[c] * inv * norm_w[c] * (KIND == HGRN ? 1.f : KIND == LINEAR ? silu<T>(g) : sigmoid<T>(g)));
     }
 }
 
@@ -507,10 +645,10 @@ inline int launched() { return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAU
 
 template <typename T, int KIND, int LK>
 int launch_scan(const jib_state_mix & a, cudaStream_t s) {
-    constexpr int VB = SCAN_NT / LK, SMEM = 2 * SCAN_TT * ((KIND == SSD ? 2 : 3) * LK * 16 + VB + 2) * 4;
+    constexpr int VB = SCAN_NT / LK, SMEM = 2 * SCAN_TT * ((per_channel(KIND) ? 3 : 2) * LK * 16 + VB + 2) * 4;
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     if (!jib::ensure_dyn_smem(state_scan_kernel<T, KIND, LK>, SMEM, done)) return JIB_E_LAUNCH;
-    const int splits = (a.V + VB - 1) / VB;
+    const int splits = (a.V + (KIND == MLSTM) + VB - 1) / VB;
     // a plain launch: as a programmatic dependent its CTAs would settle wherever the last CTAs of state_prep leave room, several to an SM
     state_scan_kernel<T, KIND, LK><<<dim3(a.H * splits, a.n_seqs), SCAN_NT, SMEM, s>>>(a, splits, a.K % 4 == 0);
     return launched();
@@ -537,7 +675,7 @@ int launch_finish(const jib_state_mix & a, cudaStream_t s) {
 template <typename T, int KIND, int VEC, int R, bool KEEP>
 int launch_step(const jib_state_mix & a, int nt, cudaStream_t s) {
     const int ncg = (a.V + VEC - 1) / VEC, nrg = nt / ncg;
-    const int smem = (3 * a.K + (a.V + 3) / 4 * 4 + nrg * ncg * VEC + 2 + 32) * 4;
+    const int smem = (3 * a.K + (a.V + 3) / 4 * 4 + nrg * ncg * VEC + 2 + 32) * 4;      // sums: 2 + at most 2 per warp
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     if (smem > 100 * 1024 || !jib::ensure_dyn_smem(state_step_kernel<T, KIND, VEC, R, KEEP>, 100 * 1024, done)) return JIB_E_ARG;
     JIB_LAUNCH((state_step_kernel<T, KIND, VEC, R, KEEP>), dim3(a.H, a.n_seqs), nt, smem, s, a);
@@ -559,11 +697,17 @@ int run(const jib_state_mix & a, int single, cudaStream_t s) {
     if (single) {
         return a.V % 4 == 0 && a.K % 4 == 0 ? step<T, KIND, 4>(a, s) : step<T, KIND, 1>(a, s);
     }
-    if (sizeof(T) == 2 && a.chunk != nullptr && jib_state_chunk_ok(a)) {
+    const bool chunks = sizeof(T) == 2 && a.chunk != nullptr && jib_state_chunk_ok(a);
+    if (KIND == MLSTM) {
+        JIB_LAUNCH((mlstm_gates_kernel), dim3(a.H, a.n_seqs), GATE_NT, 0, s, a, chunks ? 1 : 0);
+        const int rc = launched();
+        if (rc) return rc;
+    }
+    if (chunks) {
         const int rc = jib_state_chunk_run(a, s);
         return rc ? rc : launch_finish<T, KIND>(a, s);
     }
-    const int items = 2 * (a.H / a.rep) + a.H + (KIND == LINEAR ? 0 : 1) + (KIND == SSD ? 0 : a.H);
+    const int items = 2 * (a.H / a.rep) + a.H + (KIND == DELTA || KIND == SSD ? 1 : 0) + (per_channel(KIND) ? a.H : 0);
     JIB_LAUNCH((state_prep_kernel<T, KIND>), dim3((items + 7) / 8, a.T), 256, 0, s, a);
     int rc = launched();
     if (rc) return rc;
@@ -583,14 +727,18 @@ extern "C" JIB_EXPORT int jib_state_mix_run(const jib_state_mix * m, int single,
     if (a.T <= 0 || a.n_seqs <= 0) return 0;
     if (a.H < 1 || a.K < 1 || a.V < 1 || a.K > 32 * PREP_C || a.rep < 1 || a.H % a.rep || a.T > 65535 || a.n_seqs > 65535 ||
         (a.taps > 0 && (a.conv_state == nullptr || a.conv_w == nullptr)) || (a.kind == SSD && (a.norm_groups < 1 || (a.H * a.V) % a.norm_groups)) ||
-        (single && a.n_seqs != a.T) || (!single && a.chunk == nullptr && (a.qk == nullptr || a.v == nullptr || a.dec == nullptr)) || (a.kind != LINEAR && !single && a.chunk == nullptr && a.s == nullptr) ||
-        ((a.kind == SSD || !single) && a.o == nullptr))
+        (single && a.n_seqs != a.T) || (!single && a.chunk == nullptr && (a.qk == nullptr || a.v == nullptr || a.dec == nullptr)) ||
+        ((a.kind == DELTA || a.kind == SSD) && !single && a.chunk == nullptr && a.s == nullptr) || ((a.kind == SSD || !single) && a.o == nullptr) ||
+        (a.kind == HGRN && (a.lower == nullptr || a.rep != 1)) ||
+        (a.kind == MLSTM && (a.extra == nullptr || a.rep != 1 || a.gate_cap <= 0.f || (!single && (a.dec == nullptr || a.s == nullptr || a.tops == nullptr)))))
         return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
     switch (a.kind) {
         case DELTA: return f32 ? run<float, DELTA>(a, single, s) : run<bf16, DELTA>(a, single, s);
         case LINEAR: return f32 ? run<float, LINEAR>(a, single, s) : run<bf16, LINEAR>(a, single, s);
         case SSD: return f32 ? run<float, SSD>(a, single, s) : run<bf16, SSD>(a, single, s);
+        case HGRN: return f32 ? run<float, HGRN>(a, single, s) : run<bf16, HGRN>(a, single, s);
+        case MLSTM: return f32 ? run<float, MLSTM>(a, single, s) : run<bf16, MLSTM>(a, single, s);
     }
     return JIB_E_ARG;
 }

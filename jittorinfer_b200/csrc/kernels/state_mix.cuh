@@ -14,7 +14,12 @@ int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s);
 namespace state_mix {
 
 typedef __nv_bfloat16 bf16;
-enum { DELTA = JIB_STATE_DELTA, LINEAR = JIB_STATE_LINEAR, SSD = JIB_STATE_SSD };
+enum { DELTA = JIB_STATE_DELTA, LINEAR = JIB_STATE_LINEAR, SSD = JIB_STATE_SSD, HGRN = JIB_STATE_HGRN, MLSTM = JIB_STATE_MLSTM };
+__host__ __device__ constexpr bool per_channel(int kind) { return kind == DELTA || kind == LINEAR || kind == HGRN; }      // decays per key channel
+
+// Columns of the rows of v and o between the launches of a portion: MLSTM has one more, what the keys add up to (v = 1), padded to whole
+// vectors of 4.
+__host__ __device__ constexpr int scratch_cols(int kind, int V) { return kind == MLSTM ? (V + 4) / 4 * 4 : V; }
 
 __device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float to_f(float v) { return v; }
@@ -35,6 +40,16 @@ __device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1
 template <int KIND> __device__ __forceinline__ float channel_decay(const jib_state_mix & a, float z, int h) {
     return KIND == DELTA ? expf(a.neg_a[h] * softplus(z)) : expf(-a.inv_tau * softplus(-z));
 }
+// HGRN: decay f = l + (1 - l) sigmoid(z) and 1 - f, both without cancellation
+__device__ __forceinline__ void bounded_gate(float z, float l, float & f, float & rest) {
+    const float e = expf(-fabsf(z)), s = 1.f / (1.f + e), big = (1.f - l) * s, small = (1.f - l) * (e * s);      // sigmoid(|z|), sigmoid(-|z|)
+    f = l + (z >= 0.f ? big : small);
+    rest = z >= 0.f ? small : big;
+}
+// MLSTM: log gates from pre-activations
+__device__ __forceinline__ float log_input_gate(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ __forceinline__ float log_forget_gate(float z, float cap) { return -softplus(-cap * tanhf(z / cap)); }
+
 template <int KIND> __device__ __forceinline__ float head_factor(const jib_state_mix & a, float z, int h) {
     return KIND == DELTA ? 1.f / (1.f + expf(-z)) : softplus(z + a.bias[h]);
 }

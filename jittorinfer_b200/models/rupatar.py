@@ -196,7 +196,7 @@ def preset(name: str) -> RupatarHParams:
         # the layer sizes of DeepSeek-V2-Lite (64 experts of which 6 run) and DeepSeek-V2 (160 experts), two shared experts' width
         w, n, mlp = (2048, 12, Experts(1408, 64, 6, 2816)) if name == "rupatar-lite" else (5120, 4, Experts(1536, 160, 6, 3072))
         h = w // 128
-        attn = AttentionMixer(h, h // 4, 128, 128, 128 ** 0.5, 512, 16, Rotation(64, 500000.0, stretch=4.0), True)
+        attn = AttentionMixer(h, h // 4, 128, 128, 128 ** -0.5, 512, 16, Rotation(64, 500000.0, stretch=4.0), True)
         return RupatarHParams(n_vocab=102400, n_embd=w, eps=1e-6, groups=8, embed_scale=1.0,
                               layers=stack(n, attn, Hgrn2Mixer(h, 128, 128), MlstmMixer(h, 128, 128, 15.0), mlp))
     raise KeyError(name)
@@ -387,8 +387,8 @@ class RupatarModel:
         """Paged rows of ``n_slots`` tokens (and pooled rows beside them) for the attention, a state row per sequence slot for the recurrences."""
         from ..runtime.cache import HybridCache
         mixes = [L.mix for L in self.layers]
-        state = {"mix": [m and ((m.heads, m.dim, m.cols), torch.float32) for m in mixes],
-                 "top": [((m.heads,), torch.float32) if m is not None and m.kind == "mlstm" else None for m in mixes]}
+        state = {"mix": [m and ((m.heads, m.dim, m.vdim), torch.float32) for m in mixes],
+                 "extra": [((m.heads, m.dim + 1), torch.float32) if m is not None and m.kind == "mlstm" else None for m in mixes]}
         return HybridCache([L.attn and L.attn.kv_row for L in self.layers], state, n_slots, n_seqs, self.dtype, self.device, self.block_size,
                            [L.attn.pool_rows(self.block_size) if L.attn is not None else 0 for L in self.layers])
 
@@ -417,7 +417,7 @@ class RupatarModel:
         else:
             dec, gate = ops.linear(h, L.w_gates, residual=L.b_gates.expand(T, -1), out_dtype=torch.float32), proj[:, c["g"]:c["g"] + n]
         y = self._rows(h, L, n)
-        ops.state_mix(m, proj, dec, gate, None, cache.state["mix"][i], b.seq_slots, b.positions, b.q_start, single, y[:, :n], cache.state["top"][i])
+        ops.state_mix(m, proj, dec, gate, None, cache.state["mix"][i], b.seq_slots, b.positions, b.q_start, single, y[:, :n], cache.state["extra"][i])
         return ops.linear(y, L.w_o)
 
     @staticmethod

@@ -178,10 +178,11 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 
 
 # ---- mixers described by a spec (ops/specs.py) ------------------------------------------------------------------------------------
-def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top=None):
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra=None):
     """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view).  ``state`` [n, heads,
-    dim, m.cols] fp32.  "mlstm": ``dec_in`` [T, 2 heads] fp32 = input | forget gates' pre-activations, ``top`` [n, heads] fp32."""
-    return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top)
+    dim, vdim] fp32.  "mlstm": ``dec_in`` [T, 2 heads] fp32 = input | forget gates' pre-activations, ``extra`` [n, heads, dim + 1] fp32 = what the
+    keys add up to, the running maximum."""
+    return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra)
 
 
 def selective_scan(m, x, z, bc, dt, state, seq_slots, positions, q_start, single, out):

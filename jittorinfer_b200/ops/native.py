@@ -51,7 +51,7 @@ ERRORS = {-1: "unsupported shape/argument", -2: "pointer or stride not 16-byte a
 
 
 ACTS = {"silu": 0, "gelu_tanh": 1}     # activation of a gated pair (JIB_ACT_*)
-UNARIES = {"relu2": 1, "cap": 2}       # function of a single product (JIB_UNARY_*)
+UNARIES = {"relu2": 1, "cap": 2, "gelu": 3}       # function of a single product (JIB_UNARY_*)
 
 
 class GemmDesc(C.Structure):
@@ -66,12 +66,12 @@ class GemmDesc(C.Structure):
                                                                              ("src_token", C.c_void_p), ("src_rows", C.c_int), ("expert_list", C.c_void_p),
                                                                              ("n_slots", C.c_int), ("list_tiles", C.c_int), ("pdl_flags", C.c_int),
                                                                              ("act", C.c_int), ("unary", C.c_int), ("scale", C.c_float),
-                                                                             ("softcap", C.c_float)]
+                                                                             ("softcap", C.c_float), ("row_scale", C.c_void_p)]
 
 
 class RowTail(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("x_out", "norm_w", "h_out", "conv_w", "hc_out", "conv_state", "seq_slots", "positions", "status")] + \
-               [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int), ("norm2_w", C.c_void_p), ("h2_out", C.c_void_p)]
+               [("eps", C.c_float), ("taps", C.c_int), ("n_state", C.c_int), ("norm2_w", C.c_void_p), ("h2_out", C.c_void_p), ("groups", C.c_int)]
 
 
 class StateMixDesc(C.Structure):
@@ -80,14 +80,16 @@ class StateMixDesc(C.Structure):
                [(n, C.c_longlong) for n in ("ld", "ld_dec", "ld_gate", "ldy", "chunk_bytes")] + \
                [(n, C.c_int) for n in ("kind", "H", "K", "V", "rep", "taps", "conv0", "n_conv", "q_off", "k_off", "v_off", "s_off", "norm_groups",
                                        "n_state", "n_seqs", "T")] + \
-               [(n, C.c_float) for n in ("q_scale", "inv_tau", "eps", "out_scale")]
+               [(n, C.c_float) for n in ("q_scale", "inv_tau", "eps", "out_scale")] + [(n, C.c_void_p) for n in ("lower", "extra", "tops")] + \
+               [("gate_cap", C.c_float)]
 
 
 class GqaDesc(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("cache", "block_tables", "seq_lens", "q_start", "positions", "status")] + \
                [(n, C.c_longlong) for n in ("n_slots", "row")] + \
                [(n, C.c_int) for n in ("H", "G", "D", "V", "rot", "block_size", "max_blocks", "n_seqs", "T", "max_pos", "window", "chunk", "sink")] + \
-               [(n, C.c_float) for n in ("scale", "softcap", "eps", "out_scale")] + [("sink_w", C.c_void_p)]
+               [(n, C.c_float) for n in ("scale", "softcap", "eps", "out_scale")] + [(n, C.c_void_p) for n in ("sink_w", "pool", "v_first")] + \
+               [("ld_first", C.c_longlong)] + [(n, C.c_int) for n in ("pool_size", "pool_rows", "neighbours", "unit", "gate_each", "mix_v")] + [("v_mix", C.c_float)]
 
 
 class ScanDesc(C.Structure):
@@ -117,20 +119,20 @@ def load():
     sig("jib_embed_norm", vp, ip, fp, f, f, i, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_post_norm", fp, vp, fp, f, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_block_update", fp, f, vp, vp, ll, fp, fp, vp, ip, fp, i, i, i, i, C.POINTER(RowTail), vp)
-    sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, vp, vp)
+    sig("jib_rms_rows", fp, ip, fp, f, i, i, i, i, i, vp, vp)
     sig("jib_scaled_update", fp, vp, fp, vp, ip, fp, i, vp, fp, ll, fp, i, i, i, C.POINTER(RowTail), vp)
     sig("jib_causal_conv", vp, ll, fp, fp, i, i, vp, i, ip, ip, ip, i, i, i, i, vp, ip, vp)
     sig("jib_selective_scan", C.POINTER(ScanDesc), i, i, vp)
     sig("jib_mingru", vp, ll, fp, fp, fp, i, ip, ip, ip, i, i, i, i, i, vp, ip, vp)
     L.jib_state_chunk_bytes.restype, L.jib_state_chunk_bytes.argtypes = C.c_longlong, [C.POINTER(StateMixDesc)]
     sig("jib_state_mix_run", C.POINTER(StateMixDesc), i, i, vp)
-    sig("jib_gqa_qkv_post", C.POINTER(GqaDesc), vp, vp, vp, ll, fp, fp, fp, ip, vp, i, vp)
+    sig("jib_gqa_qkv_post", C.POINTER(GqaDesc), vp, vp, vp, ll, fp, fp, fp, ip, vp, i, i, vp)
     sig("jib_gqa_prefill", C.POINTER(GqaDesc), vp, vp, ll, ip, vp, ll, i, vp, ll, vp)
     sig("jib_gqa_attention", C.POINTER(GqaDesc), vp, vp, ll, vp, ll, i, i, i, vp)
     sig("jib_embed_gather", vp, ip, vp, i, i, i, vp)
     sig("jib_rmsnorm", vp, vp, fp, vp, vp, i, i, ll, f, vp)
     sig("jib_mla_qkv_post", vp, ll, vp, ll, fp, f, fp, ip, ip, vp, vp, ll, ll, i, i, i, i, i, i, ll, i, i, ip, vp)
-    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, ip, i, i, vp, ip, i, vp)
+    sig("jib_kv_gather", vp, ll, ip, i, ip, i, i, i, ip, i, i, vp, i, i, vp, ip, i, vp)
     sig("jib_mha_prefill", vp, ll, vp, vp, ll, ll, ip, ip, ip, i, i, i, f, i, i, vp, ll, ip, vp)
     sig("jib_argmax", fp, ip, i, i, vp)
     sig("jib_topk", fp, fp, ip, i, i, i, vp)
@@ -138,9 +140,9 @@ def load():
     sig("jib_kv_block_copy", vp, ll, i, ip, ip, i, i, vp)
     sig("jib_gather_rows", vp, ip, vp, i, i, i, vp)
     sig("jib_moe_gate", vp, fp, fp, fp, fp, ip, fp, i, i, i, i, i, i, f, i, i, i, i, i, vp)
-    sig("jib_moe_permute", ip, i, i, i, i, ip, ip, ip, vp)
+    sig("jib_moe_permute", ip, i, i, i, i, ip, ip, ip, fp, fp, vp)
     sig("jib_moe_route_fused", vp, fp, fp, fp, ip, fp, ip, ip, ip, ip, i, i, i, i, i, i, f, i, i, i, i, i, i, fp, f, vp, vp)
-    sig("jib_moe_permute_multi", ip, i, i, i, i, ip, ip, ip, ip, vp)
+    sig("jib_moe_permute_multi", ip, i, i, i, i, ip, ip, ip, ip, fp, fp, vp)
     sig("jib_moe_tile_list", ip, i, i, ip, i, vp)
     sig("jib_moe_combine", vp, ip, fp, vp, vp, vp, i, i, i, vp)
     sig("jib_moe_combine_norm", vp, ip, fp, vp, vp, fp, vp, vp, i, i, i, f, vp)
@@ -307,11 +309,12 @@ def _seg_has_list(seg: torch.Tensor, E: int) -> bool:
 def gemm_grouped_raw(x_ptr: int, x_rows_total: int, K: int, seg: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor],
                      max_rows: int, active_hint: int, splits: int = 0, bn: int = 0, device=None,
                      out_row_ptr: Optional[int] = None, src_token: Optional[torch.Tensor] = None, src_rows: int = 0,
-                     pdl_flags: int = 0, n_slots: int = 0, tile_list: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                     pdl_flags: int = 0, n_slots: int = 0, tile_list: Optional[torch.Tensor] = None,
+                     gelu_scale: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """Grouped GEMM over a raw row buffer (e.g. a peer-mapped receive buffer).  With ``out_row_ptr`` (device array of
     row addresses) every result row is stored through its pointer and nothing is returned.  With ``src_token`` the
     buffer holds the ``src_rows`` token rows unsorted and sorted result row i is computed from token ``src_token[i]``
-    (``x_rows_total`` stays the number of sorted rows, i.e. rows of the result)."""
+    (``x_rows_total`` stays the number of sorted rows, i.e. rows of the result).  ``gelu_scale``: the result is gelu(gelu_scale[row] * product)."""
     E, N, K2 = w.shape
     assert K2 == K
     device = device or w.device
@@ -330,6 +333,9 @@ def gemm_grouped_raw(x_ptr: int, x_rows_total: int, K: int, seg: torch.Tensor, w
     if src_token is not None:
         d.src_token, d.src_rows = src_token.data_ptr(), src_rows
     d.pdl_flags = pdl_flags
+    if gelu_scale is not None:
+        assert w2 is None and gelu_scale.dtype == torch.float32
+        d.unary, d.row_scale = UNARIES["gelu"], gelu_scale.data_ptr()
     f32 = w.dtype == torch.float32
     if f32 or not _tma_ok(x_ptr, d.w, d.w2 or 0, K * 2, N * K * 2):
         d.out_f32 = int(f32)
@@ -347,20 +353,20 @@ def gemm_grouped_raw(x_ptr: int, x_rows_total: int, K: int, seg: torch.Tensor, w
 
 def gemm_grouped(xp: torch.Tensor, seg: torch.Tensor, w: torch.Tensor, w2: Optional[torch.Tensor], max_rows: int,
                  active_hint: int, splits: int = 0, pdl_flags: int = 0, n_slots: int = 0, bn: int = 0,
-                 tile_list: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 tile_list: Optional[torch.Tensor] = None, gelu_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rows of xp are sorted by expert; expert e owns rows seg[e]:seg[e+1] and weight w[e] ([E,N,K])."""
     assert xp.stride(0) == xp.shape[1] and xp.stride(1) == 1
     return gemm_grouped_raw(xp.data_ptr(), xp.shape[0], xp.shape[1], seg, w, w2, max_rows, active_hint, splits, bn, device=xp.device,
-                            pdl_flags=pdl_flags, n_slots=n_slots, tile_list=tile_list)
+                            pdl_flags=pdl_flags, n_slots=n_slots, tile_list=tile_list, gelu_scale=gelu_scale)
 
 
 def linear(x, w, residual=None, out_dtype=None, unary=None):
     return gemm(x, w, residual=residual, out_dtype=out_dtype, unary=unary)
 
 
-def grouped_tma_ok(x: torch.Tensor, wg: torch.Tensor) -> bool:
+def grouped_tma_ok(x: torch.Tensor, wu: torch.Tensor) -> bool:
     """Whether the grouped expert products of these shapes run on the tensor cores."""
-    return x.dtype == torch.bfloat16 and wg.shape[1] % 8 == 0 and wg.shape[2] % 8 == 0
+    return x.dtype == torch.bfloat16 and wu.shape[1] % 8 == 0 and wu.shape[2] % 8 == 0
 
 
 def gateup_silu(x, wg, wu):
@@ -480,11 +486,12 @@ def visible_rows(q_len: int, s_len: int, window: int = 0, chunk: int = 0) -> int
     return s_len - max(0, p - window + 1 if window > 0 else 0, p // chunk * chunk if chunk > 0 else 0)
 
 
-def visible_total(meta, window: int, chunk: int = 0) -> int:
-    """Cached rows the queries of a step can see, over its sequences (what ``kv_gather`` writes)."""
+def visible_total(meta, window: int, chunk: int = 0, pool: int = 0) -> int:
+    """Cached rows the queries of a step can see, pooled ones included, over its sequences (what ``kv_gather`` writes)."""
     if window <= 0 and chunk <= 0:
         return int(meta["total_kv"])
-    return sum(visible_rows(int(q), int(s), window, chunk) for q, s in zip(meta["q_lens"], meta["s_lens"]))
+    pooled = sum(max(0, int(s) - window) // pool for s in meta["s_lens"]) if pool else 0
+    return pooled + sum(visible_rows(int(q), int(s), window, chunk) for q, s in zip(meta["q_lens"], meta["s_lens"]))
 
 
 def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, meta, window: int = 0) -> bool:
@@ -503,15 +510,17 @@ def mha_prefill_ok(T: int, dn: int, dr: int, dv: int, r: int, block_size: int, m
     return total > 0 and dec <= total - dec
 
 
-def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int, q_start=None, window: int = 0, chunk: int = 0):
-    """The cached rows of every sequence of the batch (with a window or chunks: those its query tokens can see), in sequence
-    order: ([total, row] bf16, first row of each sequence [n_seqs] int32)."""
+def kv_gather(cache, block_tables, seq_lens, total: int, block_size: int, q_start=None, window: int = 0, chunk: int = 0, pool=None,
+              pool_size: int = 0, pool_rows: int = 0):
+    """The cached rows of every sequence of the batch (with a window or chunks: those its query tokens can see, behind the pooled rows they
+    see), in sequence order: ([total, row] bf16, first row of each sequence [n_seqs] int32)."""
     n_seqs = seq_lens.shape[0]
     row = cache.shape[1]
     lat = torch.empty(total, row, dtype=torch.bfloat16, device=cache.device)
     kv_start = torch.empty(n_seqs, dtype=torch.int32, device=cache.device)
     _ck(load().jib_kv_gather(cache.data_ptr(), cache.shape[0], block_tables.data_ptr(), block_tables.stride(0), seq_lens.data_ptr(),
-                             n_seqs, block_size, row, _p(q_start), window, chunk, lat.data_ptr(), kv_start.data_ptr(), total, _stream()), "kv_gather")
+                             n_seqs, block_size, row, _p(q_start), window, chunk, _p(pool), pool_size, pool_rows, lat.data_ptr(), kv_start.data_ptr(),
+                             total, _stream()), "kv_gather")
     return lat, kv_start
 
 
@@ -586,11 +595,12 @@ def moe_gate(g, w_router, bias, k, n_group, topk_group, scale, norm, sigmoid, n_
     return (ids, wts) + ((g,) if pre_norm is not None else ()) + ((logits[:, E],) if shared_gate else ())
 
 
-def moe_permute(ids, expert_base, E_local):
+def moe_permute(ids, expert_base, E_local, wts=None, row_wts=None):
+    """``row_wts`` [T * k] fp32: receives the weights ``wts`` of the pairs in sorted order."""
     T, k = ids.shape
     dev = ids.device
     hit = _route_stash.pop((ids.data_ptr(), expert_base, E_local), None)
-    if hit is not None and hit[3] is ids:          # the fused router launch already sorted exactly these ids
+    if hit is not None and hit[3] is ids and row_wts is None:          # the fused router launch already sorted exactly these ids
         return hit[0], hit[1], hit[2]
     seg = torch.empty(2 * E_local + 1, dtype=torch.int32, device=dev)[:E_local + 1]       # + room for the list of experts hit
     src = torch.empty(T * k, dtype=torch.int32, device=dev)
@@ -599,10 +609,10 @@ def moe_permute(ids, expert_base, E_local):
         # large batches (prefill): histogram / scan / stable scatter over many CTAs instead of one CTA scanning every pair
         tmp = torch.empty(((T * k + 1023) // 1024) * E_local, dtype=torch.int32, device=dev)
         _ck(load().jib_moe_permute_multi(ids.data_ptr(), T, k, expert_base, E_local, seg.data_ptr(), src.data_ptr(), dest.data_ptr(),
-                                         tmp.data_ptr(), _stream()), "moe_permute_multi")
+                                         tmp.data_ptr(), _p(wts), _p(row_wts), _stream()), "moe_permute_multi")
         return seg, src, dest
     _ck(load().jib_moe_permute(ids.data_ptr(), T, k, expert_base, E_local, seg.data_ptr(), src.data_ptr(), dest.data_ptr(),
-                               _stream()), "moe_permute")
+                               _p(wts), _p(row_wts), _stream()), "moe_permute")
     return seg, src, dest
 
 
@@ -650,13 +660,16 @@ def expected_active_experts(T: int, k: int, E_local: int, n_expert: int) -> int:
 
 
 def moe_routed(x, ids, wts, wg, wu, wd, expert_base=0, n_expert=None):
-    """Expert-sorted rows -> grouped gate|up GEMM (SiLU*mul epilogue) -> grouped down GEMM.
-    Returns (y [T*k, d] in sorted order, dest [T,k])."""
+    """Expert-sorted rows -> grouped gate|up GEMM (SiLU*mul epilogue) -> grouped down GEMM.  ``wg`` None: the first product is wu's alone, its
+    epilogue gelu(weight of the row * product).  Returns (y [T*k, d] in sorted order, dest [T,k])."""
     T, k = ids.shape
-    E_local = wg.shape[0]
-    seg, src, dest = moe_permute(ids, expert_base, E_local)
+    E_local = wu.shape[0]
+    fn = None if wg is not None else torch.empty(T * k, dtype=torch.float32, device=x.device)
+    seg, src, dest = moe_permute(ids, expert_base, E_local, wts if fn is not None else None, fn)
+    if fn is not None:
+        wg, wu = wu, None
     if not grouped_tma_ok(x, wg):                  # fp32 operands, or rows TMA cannot address
-        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, 0)
+        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, 0, gelu_scale=fn)
         return gemm_grouped(h, seg, wd, None, T, 0), dest
     # the two grouped launches run back to back over one segment table: the second may start on its weights early
     pair = (1, 2) if GROUPED_PAIR else (0, 0)
@@ -669,15 +682,15 @@ def moe_routed(x, ids, wts, wg, wu, wd, expert_base=0, n_expert=None):
         # prompt chunks: an expert holds ~T*k/E rows, far fewer than the T the grid would have to be sized for; both grouped
         # launches walk a device-built list of the (expert, 128-token tile) pairs that exist
         tl = moe_tile_list(seg, E_local, 128, T * k)
-        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, active, pdl_flags=pair[0], bn=128, tile_list=tl)
+        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, active, pdl_flags=pair[0], bn=128, tile_list=tl, gelu_scale=fn)
         return gemm_grouped(h, seg, wd, None, T, active, pdl_flags=pair[1], bn=128, tile_list=tl), dest
     if GROUPED_SRC and T <= GROUPED_SRC_MAX_T and x.is_contiguous():
         # decode batches: every expert that has rows multiplies the whole (tiny) token tile and picks its tokens' columns in the
         # epilogue, so the token rows are never gathered into expert order
         h = gemm_grouped_raw(x.data_ptr(), T * k, x.shape[1], seg, wg, wu, T, active, device=x.device, src_token=src, src_rows=T,
-                             pdl_flags=pair[0], n_slots=slots)
+                             pdl_flags=pair[0], n_slots=slots, gelu_scale=fn)
     else:
-        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, active, pdl_flags=pair[0], n_slots=slots)
+        h = gemm_grouped(gather_rows(x, src), seg, wg, wu, T, active, pdl_flags=pair[0], n_slots=slots, gelu_scale=fn)
     y = gemm_grouped(h, seg, wd, None, T, active, pdl_flags=pair[1], n_slots=slots)
     return y, dest
 
@@ -705,7 +718,7 @@ def _row_tail(x_out, nxt, dtype):
     t.x_out, t.status = x_out.data_ptr(), workspace(x_out.device).status.data_ptr()
     if isinstance(nxt, RowNorms):
         h = torch.empty(x_out.shape, dtype=dtype, device=x_out.device)
-        t.h_out, t.norm_w, t.eps = h.data_ptr(), _p(nxt.w1), float(nxt.eps)
+        t.h_out, t.norm_w, t.eps, t.groups = h.data_ptr(), _p(nxt.w1), float(nxt.eps), nxt.groups
         if nxt.w2 is not None:
             hc = torch.empty_like(h)
             t.norm2_w, t.h2_out = nxt.w2.data_ptr(), hc.data_ptr()
@@ -765,10 +778,10 @@ def scaled_update(x, o, s1, s2=None, moe=None, dense=None, dense_gate=None, nxt=
     return x, h, h2
 
 
-def rms_rows(x, rows, w, eps, dtype):
+def rms_rows(x, rows, w, eps, dtype, groups=1):
     n, d = (rows.shape[0] if rows is not None else x.shape[0]), x.shape[1]
     out = torch.empty(n, d, dtype=dtype, device=x.device)
-    _ck(load().jib_rms_rows(x.data_ptr(), _p(rows), w.data_ptr(), float(eps), n, d, x.shape[0], int(dtype == torch.float32), out.data_ptr(),
+    _ck(load().jib_rms_rows(x.data_ptr(), _p(rows), w.data_ptr(), float(eps), n, d, x.shape[0], groups, int(dtype == torch.float32), out.data_ptr(),
                             _stream()), "rms_rows")
     return out
 
@@ -796,18 +809,22 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 
 # ---- mixers described by a spec: matrix state per head (state_mix.cu), grouped-query attention (gqa_attention.cu) ----------------
 STATE_CHUNKS = os.environ.get("JIB_STATE_CHUNKS", "1") == "1"      # "0": portions token by token on CUDA cores (A/B)
-STATE_KINDS = {"delta": 0, "linear": 1, "ssd": 2}
+STATE_KINDS = {"delta": 0, "linear": 1, "ssd": 2, "hgrn": 3, "mlstm": 4}
 
 
-def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out):
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra=None):
     T, H, K, V = proj.shape[0], m.heads, m.dim, m.vdim
-    assert proj.stride(1) == 1 and gate.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype == gate.dtype
+    mlstm = m.kind == "mlstm"
+    assert proj.stride(1) == 1 and out.stride(1) == 1 and out.dtype == proj.dtype and (gate is None or (gate.stride(1) == 1 and gate.dtype == proj.dtype))
+    assert (gate is None) == (m.kind == "hgrn") and mlstm == (extra is not None)
     assert state.dtype == torch.float32 and state.is_contiguous() and (m.taps == 0 or (conv_state.is_contiguous() and conv_state.dtype == proj.dtype))
     f32 = lambda *s: torch.empty(*s, dtype=torch.float32, device=proj.device)        # noqa: E731
     sd = StateMixDesc()
-    sd.proj, sd.ld, sd.gate, sd.ld_gate, sd.y, sd.ldy = proj.data_ptr(), proj.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
+    sd.proj, sd.ld, sd.y, sd.ldy = proj.data_ptr(), proj.stride(0), out.data_ptr(), out.stride(0)
+    if gate is not None:
+        sd.gate, sd.ld_gate = gate.data_ptr(), gate.stride(0)
     if dec_in is not None:
-        assert dec_in.stride(1) == 1 and dec_in.dtype == proj.dtype
+        assert dec_in.stride(1) == 1 and dec_in.dtype == (torch.float32 if mlstm else proj.dtype)
         sd.dec_in, sd.ld_dec = dec_in.data_ptr(), dec_in.stride(0)
     sd.conv_state, sd.state, sd.n_state = _p(conv_state), state.data_ptr(), state.shape[0]
     sd.conv_w, sd.conv_b, sd.bias, sd.neg_a, sd.skip, sd.norm_w = _p(m.conv_w), _p(m.conv_b), _p(m.bias), _p(m.neg_a), _p(m.skip), _p(m.norm_w)
@@ -818,19 +835,27 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     sd.q_off, sd.k_off, sd.v_off, sd.s_off, sd.norm_groups = m.q_off, m.k_off, m.v_off, m.s_off, m.norm_groups
     sd.n_seqs, sd.T = q_start.shape[0] - 1, T
     sd.q_scale, sd.inv_tau, sd.eps, sd.out_scale = m.q_scale, m.inv_tau, m.eps, m.out_scale
+    sd.lower, sd.gate_cap = _p(m.lower), m.gate_cap
+    if mlstm:
+        assert extra.dtype == torch.float32 and extra.is_contiguous() and extra.shape[1:] == (H, K + 1)
+        sd.extra = extra.data_ptr()
+    VS = (V + 4) // 4 * 4 if mlstm else V             # columns of v and o between a portion's launches
     scratch = []
     n = 0 if single or proj.dtype == torch.float32 or not STATE_CHUNKS else load().jib_state_chunk_bytes(C.byref(sd))
     if n > 0:                         # portions through the tensor cores
         scratch = [torch.empty(n, dtype=torch.uint8, device=proj.device)]
         sd.chunk, sd.chunk_bytes = scratch[0].data_ptr(), n
-        if m.kind != "delta":
+        if m.kind in ("linear", "ssd"):
             scratch.append(torch.empty(T, H * V, dtype=proj.dtype, device=proj.device))
             sd.v = scratch[1].data_ptr()
     elif not single:
-        scratch = [f32(T, 2 * (H // m.rep) * K), f32(T, H * V), f32(T, H * (1 if m.kind == "ssd" else K)), f32(T, H)]
+        scratch = [f32(T, 2 * (H // m.rep) * K), f32(T, H * VS), f32(T, H * (1 if m.kind in ("ssd", "mlstm") else K)), f32(T, H)]
         sd.qk, sd.v, sd.dec, sd.s = (x.data_ptr() for x in scratch)
+    if not single and mlstm:
+        gates = [f32(T, H), f32(T, H), f32(T, H)]
+        sd.dec, sd.s, sd.tops = (x.data_ptr() for x in gates)
     if not single or m.kind == "ssd":
-        scratch.append(f32(T, H * V))
+        scratch.append(f32(T, H * VS))
         sd.o = scratch[-1].data_ptr()
     _ck(load().jib_state_mix_run(C.byref(sd), int(single), int(proj.dtype == torch.float32), _stream()), "state_chunk" if n > 0 else "state_mix")
     return out
@@ -860,44 +885,65 @@ def _gqa_desc(m, cache, T, n_seqs):
     gd.window, gd.chunk, gd.sink = m.window, m.chunk, int(m.sink)
     gd.scale, gd.softcap, gd.eps, gd.out_scale = m.scale, m.softcap, m.eps, m.out_scale
     gd.sink_w = _p(m.sink_w)
+    gd.neighbours, gd.unit, gd.gate_each = int(m.neighbours), int(m.unit), int(m.gate_each)
     return gd
 
 
-def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache):
+def _gqa_pool(gd, m, pool, cache, block_tables, seq_lens, q_start, block_size):
+    assert pool.is_contiguous() and pool.dtype == cache.dtype and pool.shape[1] == cache.shape[1]
+    gd.pool, gd.pool_size, gd.pool_rows, gd.block_size = pool.data_ptr(), m.pool, m.pool_rows(block_size), block_size
+    gd.block_tables, gd.max_blocks, gd.seq_lens, gd.q_start = block_tables.data_ptr(), block_tables.stride(0), seq_lens.data_ptr(), q_start.data_ptr()
+
+
+def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache, v_first=None, pooled=None):
     T = q.shape[0]
     assert q.dtype == cache.dtype and q.stride(1) == 1 and k.stride(0) == q.stride(0) == v.stride(0) and rope_table.is_contiguous()
     out = torch.empty(T, m.heads, m.dim, dtype=q.dtype, device=q.device)
     gd = _gqa_desc(m, cache, T, 1)
     gd.positions, gd.max_pos = positions.data_ptr(), rope_table.shape[0]
+    single = False
+    if m.pool:
+        pool, tables, seq_lens, q_start, block_size, single = pooled
+        _gqa_pool(gd, m, pool, cache, tables, seq_lens, q_start, block_size)
+        gd.n_seqs = seq_lens.shape[0]
+    if m.v_mix is not None:
+        assert v_first.dtype == v.dtype and v_first.stride(1) == 1
+        gd.mix_v, gd.v_mix, gd.v_first, gd.ld_first = 1, m.v_mix, v_first.data_ptr(), v_first.stride(0)
     _ck(load().jib_gqa_qkv_post(C.byref(gd), q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _p(m.q_norm), _p(m.k_norm),
-                                rope_table.data_ptr(), slot_mapping.data_ptr(), out.data_ptr(), int(q.dtype == torch.float32), _stream()), "gqa_qkv_post")
+                                rope_table.data_ptr(), slot_mapping.data_ptr(), out.data_ptr(), int(single), int(q.dtype == torch.float32), _stream()),
+        "gqa_qkv_post")
     return out
 
 
 def gqa_splits(m, T, max_keys, sm_count=148):
     """CTAs that share one row's keys in a batch of single tokens: as many as fill the machine, at most one per 64 visible keys."""
-    keys = min([x for x in (m.window, m.chunk, max_keys) if x > 0])
+    keys = min([x for x in (m.window, m.chunk, max_keys) if x > 0]) + (max_keys // m.pool if m.pool else 0)
     fill = max(1, 4 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
     n = min(8, fill, (keys + 63) // 64)
     return 1 << (n.bit_length() - 1)
 
 
-def gqa_prefill_ok(m, q, cache, out, block_size: int, single: bool, meta) -> bool:
+def gqa_prefill_ok(m, q, cache, out, block_size: int, single: bool, meta, gate=None) -> bool:
     """Whether a batch of portions takes the tensor-core kernel (needs the host-side totals in ``meta``)."""
+    if m.gate_each and gate is not None and not _tma_ok(gate.data_ptr(), gate.stride(0) * 2):
+        return False
     return not single and MHA_PREFILL and meta is not None and "q_lens" in meta and q.dtype == torch.bfloat16 and q.shape[0] >= MHA_PREFILL_MIN_TOKENS and \
         m.dim == 128 and m.vdim == 128 and cache.shape[1] % 8 == 0 and block_size == 64 and _tma_ok(q.data_ptr(), out.data_ptr(), out.stride(0) * 2)
 
 
-def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out):
+def gqa_attention(m, q, cache, gate, block_tables, seq_lens, q_start, block_size, max_q_len, meta, out, pool=None):
     T, H, D = q.shape
     assert q.dtype == cache.dtype == out.dtype and q.is_contiguous() and out.stride(1) == 1
     single = max_q_len == 1 and seq_lens.shape[0] == T
     gd = _gqa_desc(m, cache, T, seq_lens.shape[0])
     gd.block_tables, gd.max_blocks, gd.block_size = block_tables.data_ptr(), block_tables.stride(0), block_size
     gd.seq_lens, gd.q_start = seq_lens.data_ptr(), q_start.data_ptr()
-    if gqa_prefill_ok(m, q, cache, out, block_size, single, meta):
-        total = visible_total(meta, m.window, m.chunk)
-        kv, kv_start = kv_gather(cache, block_tables, seq_lens, total, block_size, q_start, m.window, m.chunk)
+    if m.pool:
+        _gqa_pool(gd, m, pool, cache, block_tables, seq_lens, q_start, block_size)
+    if gqa_prefill_ok(m, q, cache, out, block_size, single, meta, gate):
+        total = visible_total(meta, m.window, m.chunk, m.pool)
+        kv, kv_start = kv_gather(cache, block_tables, seq_lens, total, block_size, q_start, m.window, m.chunk, pool if m.pool else None, m.pool,
+                                 m.pool_rows(block_size))
         _ck(load().jib_gqa_prefill(C.byref(gd), q.data_ptr(), kv.data_ptr(), total, kv_start.data_ptr(), _p(gate), gate.stride(0) if gate is not None else 0,
                                    int(meta["n_q_tiles"]), out.data_ptr(), out.stride(0), _stream()), "gqa_prefill")
         return out

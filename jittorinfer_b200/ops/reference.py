@@ -416,7 +416,7 @@ def _softplus(x):
     return F.softplus(x, threshold=1e9)
 
 
-def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, top=None):
+def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra=None):
     """Runs the mixer described by ``m`` (``ops.specs.StateMix``) over a batch; result columns go to ``out`` [T, H * V]."""
     H, K, V, Hk = m.heads, m.dim, m.vdim, m.heads // m.rep
     qs = q_start.tolist()
@@ -449,14 +449,12 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
             dec, k, q = low + (1 - low) * torch.sigmoid(z), (1 - low) * torch.sigmoid(-z), F.silu(q)
         if m.kind == "mlstm":
             i, f = (m.gate_cap * torch.tanh(dec_in[q0:q1].float() / m.gate_cap)).view(n, 2, H).unbind(1)
-            f, t0 = F.logsigmoid(f), top[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, device=proj.device)
+            f, t0 = F.logsigmoid(f), extra[slot, :, K].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, device=proj.device)
             tops, dec = torch.empty(n, H, device=proj.device), torch.empty(n, H, 1, device=proj.device)
             for t in range(n):
                 tops[t] = torch.maximum(f[t] + t0, i[t])
                 dec[t, :, 0], s[t], t0 = torch.exp(f[t] + t0 - tops[t]), torch.exp(i[t] - tops[t]), tops[t]
-            if slot >= 0:
-                top[slot] = t0
-            v = torch.cat([v, torch.ones(n, H, 1, device=proj.device), torch.zeros(n, H, m.cols - V - 1, device=proj.device)], 2)
+            v = torch.cat([v, torch.ones(n, H, 1, device=proj.device)], 2)                # one more column: what the keys add up to
         if m.kind == "delta":
             q, k = (y / torch.sqrt(y.pow(2).sum(-1, keepdim=True) + 1e-6) for y in (q, k))
             s = torch.sigmoid(x[:, m.s_off:m.s_off + H])
@@ -468,15 +466,21 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
             dec = torch.exp(m.neg_a[:, None] * _softplus(z).view(n, H, K)) if m.kind == "delta" else \
                 torch.exp(-m.inv_tau * _softplus(-z)).view(n, H, K)
         q, k = (q * m.q_scale).repeat_interleave(m.rep, 1), k.repeat_interleave(m.rep, 1)
-        S = state[slot].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, K, m.cols, device=proj.device)
-        o = torch.empty(n, H, m.cols, device=proj.device)
+        S = torch.zeros(H, K, v.shape[2], device=proj.device)
+        if slot >= 0 and p0 > 0:
+            S[..., :V] = state[slot]
+            if m.kind == "mlstm":
+                S[..., V] = extra[slot, :, :K]
+        o = torch.empty(n, H, v.shape[2], device=proj.device)
         for t in range(n):
             S = S * dec[t][..., None]
             u = v[t] - torch.einsum("hkv,hk->hv", S, k[t]) if m.kind == "delta" else v[t]
             S = S + k[t][..., None] * (s[t][:, None] * u)[:, None, :]
             o[t] = torch.einsum("hkv,hk->hv", S, q[t])
         if slot >= 0:
-            state[slot] = S
+            state[slot] = S[..., :V]
+            if m.kind == "mlstm":
+                extra[slot, :, :K], extra[slot, :, K] = S[..., V], t0
         if m.kind == "mlstm":
             o = o[..., :V] / (torch.maximum(o[..., V].abs(), torch.exp(-tops)) + 1e-6)[..., None]
             o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + m.eps)).reshape(n, H * V)

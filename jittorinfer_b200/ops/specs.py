@@ -16,8 +16,8 @@ class StateMix:
     "ssd": s = softplus(. + bias), decay exp(neg_a s) per head, silu gate, then a norm over ``norm_groups`` parts of the row;
     "hgrn": decay f = lower + (1 - lower) sigmoid(. + bias) per key channel, k = 1 - f, silu on q, s = 1, norm per head, no gate;
     "mlstm": decay and s per head from two log gates i = cap tanh(. / cap) and f = log sigmoid(cap tanh(. / cap)), relative to a running
-    maximum top <- max(f + top, i) that starts at 0: decay exp(f + top_old - top), s exp(i - top).  k decays and adds up like k v^T does (column
-    ``vdim`` of the state); o is divided by max(|that sum . q|, exp(-top)) + 1e-6, then a norm per head (``norm_w`` [heads * vdim]), sigmoid gate.
+    maximum top <- max(f + top, i) that starts at 0: decay exp(f + top_old - top), s exp(i - top).  What the k add up to decays and grows like the
+    state; o is divided by max(|that sum . q|, exp(-top)) + 1e-6, then a norm per head (``norm_w`` [heads * vdim]), sigmoid gate.
     ``*_off``: columns of the projection.  Columns conv0 .. conv0 + n of it pass a causal convolution of ``taps`` taps (0: none) and silu."""
     kind: str
     heads: int
@@ -43,11 +43,6 @@ class StateMix:
     out_scale: float = 1.0
     lower: Optional[torch.Tensor] = None        # [heads * dim] fp32, "hgrn"
     gate_cap: float = 0.0                       # "mlstm"
-
-    @property
-    def cols(self) -> int:
-        """Columns of a state row: the values', and for "mlstm" that of the keys' sum (padded to a multiple of 4)."""
-        return (self.vdim + 4) // 4 * 4 if self.kind == "mlstm" else self.vdim
 
 
 @dataclass
