@@ -124,7 +124,7 @@ def main():
                     help="diagnostic (needs JITTORINFER_KERNELS_SO = the timeline build): report how long the fused all-reduces "
                          "wait for their peers during the timed steps; the stamps cost time, so the tokens/s of such a run is not a result")
     ap.add_argument("--design", default=None,
-                    help="instead of the headline: prefill and decode throughput of this design (nibalix | lugovik | zomavik) at real layer sizes beside the "
+                    help="instead of the headline: prefill and decode throughput of this design (nibalix | lugovik | zomavik | rupatar) at real layer sizes beside the "
                          "closest other model at equal sizes (1 GPU)")
     args = ap.parse_args()
     if args.impl == "reference":

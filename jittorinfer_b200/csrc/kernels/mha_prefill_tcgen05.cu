@@ -87,7 +87,7 @@ __device__ __forceinline__ float capped_log2(float s, const MhaArgs & a) {
     return a.cap_log2e - 2.f * a.cap_log2e * r;               // 1 - 2 / (1 + e^{2 y}) = tanh(y), absolute error of a few 1e-7
 }
 
-template <bool GQA>
+template <bool GQA, bool POOL>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                    const __grid_constant__ CUtensorMap tmPE, const MhaArgs a) {
@@ -165,7 +165,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const int S = visible_rows(a.seq_lens[b], q_len, a.window, a.chunk);
         base_pos = a.seq_lens[b] - S;
         ctx0 = S - q_len;                             // gathered rows before this chunk
-        if (GQA) {
+        if (POOL) {
             const int np = gqa_blocks_seen(a.seq_lens[b] - 1, a.window, a.pool_size);
             ctx0 += np;
             base_pos -= np;
@@ -174,13 +174,13 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         rows = min(QT, q_len - tile * QT);            // valid query rows of the tile
         const int last_lim = ctx0 + tile * QT + rows; // kv rows visible to the last valid query row
         kt0 = max(0, gqa_first_key(base_pos + ctx0 + tile * QT, a.window, a.chunk) - base_pos) / KT;
-        if (GQA) {
+        if (POOL) {
             pt = (gqa_blocks_seen(base_pos + last_lim - 1, a.window, a.pool_size) + KT - 1) / KT;
             kt0 = max(kt0, pt);
         }
         n_tiles = rows > 0 && S > 0 ? pt + (last_lim + KT - 1) / KT - kt0 : 0;
     }
-    auto tile_at = [&](int i) { return GQA && i < pt ? i : kt0 + i - pt; };
+    auto tile_at = [&](int i) { return POOL && i < pt ? i : kt0 + i - pt; };
     const int row0 = q0 + tile * QT;                  // first query row (global)
 
     if (n_tiles > 0 && warp == 0) {
@@ -259,8 +259,8 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const int first = gqa_first_key(base_pos + ctx0 + tile * QT + r, a.window, a.chunk) - base_pos;
         const int first_last = gqa_first_key(base_pos + ctx0 + tile * QT + QT - 1, a.window, a.chunk) - base_pos;
         // pooled rows this query row sees, and the tile's first one
-        const int blocks = GQA && r < rows ? gqa_blocks_seen(base_pos + ctx0 + tile * QT + r, a.window, a.pool_size) : 0;
-        const int blocks_first = GQA ? gqa_blocks_seen(base_pos + ctx0 + tile * QT, a.window, a.pool_size) : 0;
+        const int blocks = POOL && r < rows ? gqa_blocks_seen(base_pos + ctx0 + tile * QT + r, a.window, a.pool_size) : 0;
+        const int blocks_first = POOL ? gqa_blocks_seen(base_pos + ctx0 + tile * QT, a.window, a.pool_size) : 0;
         float m_ref = -INFINITY;                      // exponent base, log2 domain (score * scale * log2 e)
         float l_sum = 0.f;
         bool ok = true;
@@ -273,9 +273,10 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             const uint32_t ts = tm_S + lane_addr + s * KT;
             const int col0 = tile_at(kt) * KT;
             // the tile reaches the diagonal (or the sequence end), or begins before what the last row sees does
-            const bool need_mask = (col0 + KT > lim_first || col0 < first_last) && (!GQA || col0 + KT > blocks_first);
+            const bool need_mask = (col0 + KT > lim_first || col0 < first_last) && (!POOL || col0 + KT > blocks_first);
             const int vis = lim - col0;               // columns [inv, vis) of this tile are visible to this row
             const int inv = first - col0, pooled = blocks - col0;
+            const unsigned span = (unsigned) max(vis - inv, 0);      // visible columns from inv on
             // The row's 128 scores come out of tensor memory once, all loads in flight before one wait; the S buffer is
             // handed back to the tensor core right away (Q.K^T of the tile after the next may start).
             float x[KT];
@@ -291,14 +292,14 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
                 for (int c = 0; c < KT; ++c) x[c] = capped_log2(x[c], a);       // no branch around it: the 128 chains overlap
                 if (need_mask) {
 #pragma unroll
-                    for (int c = 0; c < KT; ++c) x[c] = (c < vis && c >= inv) || c < pooled ? x[c] : -INFINITY;
+                    for (int c = 0; c < KT; ++c) x[c] = (POOL ? (unsigned) (c - inv) < span || c < pooled : c < vis && c >= inv) ? x[c] : -INFINITY;
                 }
 #pragma unroll
                 for (int c = 0; c < KT; ++c) mt = fmaxf(mt, x[c]);
             } else if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) {
-                    const bool see = (c < vis && c >= inv) || (GQA && c < pooled);
+                    const bool see = POOL ? (unsigned) (c - inv) < span || c < pooled : c < vis && c >= inv;
                     x[c] = see ? x[c] * a.scale_log2e : -INFINITY;
                     mt = fmaxf(mt, x[c]);
                 }
@@ -508,8 +509,8 @@ JIB_EXPORT int jib_mha_prefill(const void * q, long long q_stride, const void * 
     a.scale_log2e = scale * 1.4426950408889634f;
     constexpr int SMEM = Form<false>::SMEM_BYTES;
     static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(mha_prefill_kernel<false>, SMEM, attr_done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((mha_prefill_kernel<false>), dim3(n_q_tiles, H), NUM_THREADS, SMEM, stream, mq, mkv, mpe, a);
+    if (!jib::ensure_dyn_smem(mha_prefill_kernel<false, false>, SMEM, attr_done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((mha_prefill_kernel<false, false>), dim3(n_q_tiles, H), NUM_THREADS, SMEM, stream, mq, mkv, mpe, a);
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 
@@ -534,9 +535,14 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
     a.inv_cap2 = m->softcap > 0.f ? 2.f * a.scale_log2e / m->softcap : 0.f;
     a.gate = (const bf16 *) gate; a.ld_gate = ld_gate; a.out_scale = m->out_scale; a.pool_size = m->pool_size; a.gate_each = m->gate_each;
     constexpr int SMEM = Form<true>::SMEM_BYTES;
-    static std::atomic<unsigned char> attr_done[jib::MAX_DEVICES];
-    if (!jib::ensure_dyn_smem(mha_prefill_kernel<true>, SMEM, attr_done)) return JIB_E_LAUNCH;
-    JIB_LAUNCH((mha_prefill_kernel<true>), dim3(m->H, n_q_tiles), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
+    static std::atomic<unsigned char> attr_done[2][jib::MAX_DEVICES];
+    if (m->pool_size > 0) {
+        if (!jib::ensure_dyn_smem(mha_prefill_kernel<true, true>, SMEM, attr_done[1])) return JIB_E_LAUNCH;
+        JIB_LAUNCH((mha_prefill_kernel<true, true>), dim3(m->H, n_q_tiles), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
+    } else {
+        if (!jib::ensure_dyn_smem(mha_prefill_kernel<true, false>, SMEM, attr_done[0])) return JIB_E_LAUNCH;
+        JIB_LAUNCH((mha_prefill_kernel<true, false>), dim3(m->H, n_q_tiles), NUM_THREADS, SMEM, stream, mq, mkv, mq, a);
+    }
     return cudaGetLastError() == cudaSuccess ? 0 : JIB_E_LAUNCH;
 }
 

@@ -18,7 +18,7 @@ def main(argv=None) -> int:
     ap.add_argument("--config", "-c", default=None)
     ap.add_argument("--model", "-m", default=None, help="GGUF file, or a folder with config.json and safetensors files")
     ap.add_argument("--random-init", default=None,
-                    help="tiny | tiny-v2 | lite | v2 | nibalix-tiny | nibalix-lite | lugovik-tiny | lugovik-lite | zomavik-tiny | zomavik-lite: random weights instead of a model file")
+                    help="tiny | tiny-v2 | lite | v2 | nibalix-tiny | nibalix-lite | lugovik-tiny | lugovik-lite | zomavik-tiny | zomavik-lite | rupatar-tiny | rupatar-lite: random weights instead of a model file")
     ap.add_argument("--prompt", "-p", action="append", default=[], help="text prompt (repeatable)")
     ap.add_argument("--tokens", action="append", default=[], help="prompt as comma-separated token ids (repeatable)")
     ap.add_argument("--chat", action="store_true", help="wrap each text prompt in the chat template as a user turn")

@@ -37,7 +37,7 @@ import torch
 
 OPS = ("embed_gather", "select_rows", "rmsnorm", "linear", "gateup_silu", "mla_qkv_post", "q_absorb", "v_up", "mla_attention",
        "moe_gate", "moe_experts", "moe_ffn", "moe_routed", "embed_norm", "block_update", "rms_rows", "causal_conv", "mingru",
-       "gateup", "post_norm", "state_mix", "gqa_qkv_post", "gqa_attention", "argmax", "topk_logits", "sample_topk", "kv_block_copy")
+       "gateup", "post_norm", "scaled_update", "state_mix", "selective_scan", "gqa_qkv_post", "gqa_attention", "argmax", "topk_logits", "sample_topk", "kv_block_copy")
 
 
 def _sig(args, kwargs) -> str:
@@ -53,7 +53,7 @@ def _sig(args, kwargs) -> str:
 KERNEL_LEVEL = ("gemm", "gemm_batched", "gemm_grouped_raw", "moe_permute", "gather_rows", "moe_combine", "rmsnorm", "embed_gather",
                 "mla_qkv_post", "mla_attention", "moe_gate", "argmax", "topk_logits", "kv_block_copy", "mha_prefill", "kv_gather",
                 "mha_prefill_core", "embed_norm", "block_update", "rms_rows", "causal_conv", "mingru",
-                "post_norm", "state_mix", "gqa_qkv_post", "gqa_attention")
+                "post_norm", "scaled_update", "state_mix", "selective_scan", "gqa_qkv_post", "gqa_attention")
 
 
 class OpProfile:

@@ -23,14 +23,15 @@ def sizes(design: str):
         dense = lambda n, d, h, ff: DeepSeek2HParams(n_layer=n, n_layer_dense_lead=n, n_embd=d, n_head=h, n_ff=ff)       # noqa: E731
         return [("width 2048, 16 heads of 128, feed-forward 5632, 12 layers", preset("lugovik-lite"), dense(12, 2048, 16, 5632)),
                 ("width 4096, 32 heads of 128, feed-forward 11008, 8 layers", preset("lugovik-wide"), dense(8, 4096, 32, 11008))]
-    if design == "zomavik":
+    if design in ("zomavik", "rupatar"):
+        runs = "layer runs" if design == "zomavik" else "layers"
         v2 = DeepSeek2HParams(n_layer=4, n_layer_dense_lead=0, n_embd=5120, n_head=128, n_ff_exp=1536, n_expert=160, expert_weights_scale=16.0,
                               n_group=8, topk_group=3, q_lora_rank=1536)
-        return [("width 2048, 16 heads, 64 experts top-6 of 1408 + 2 shared, 12 layer runs", preset("zomavik-lite"),
+        return [(f"width 2048, 16 heads, 64 experts top-6 of 1408 + 2 shared, 12 {runs}", preset(f"{design}-lite"),
                  DeepSeek2HParams(n_layer=12, n_layer_dense_lead=0)),
-                ("width 5120, 40 heads (closest: 128), 160 experts top-6 of 1536 + 2 shared, 4 layer runs", preset("zomavik-v2"), v2)]
+                (f"width 5120, 40 heads (closest: 128), 160 experts top-6 of 1536 + 2 shared, 4 {runs}", preset(f"{design}-v2"), v2)]
     if design != "nibalix":
-        raise SystemExit(f"unknown design {design!r} (known: nibalix, lugovik, zomavik)")
+        raise SystemExit(f"unknown design {design!r} (known: nibalix, lugovik, zomavik, rupatar)")
     lite = DeepSeek2HParams(n_layer=12, n_layer_dense_lead=0, n_expert_shared=0)
     v2 = DeepSeek2HParams(n_layer=4, n_layer_dense_lead=0, n_expert_shared=0, n_embd=5120, n_head=128, n_ff_exp=1536, n_expert=160,
                           expert_weights_scale=16.0, n_group=8, topk_group=3, q_lora_rank=1536)

@@ -100,7 +100,7 @@ def write_model(directory, cfg, w):
         json.dump(cfg, f)
     head, blobs, off = {}, [], 0
     for name, t in w.items():
-        b = t.bfloat16().contiguous().view(torch.uint8).numpy().tobytes()
+        b = t.bfloat16().contiguous().reshape(-1).view(torch.uint8).numpy().tobytes()
         head[name] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [off, off + len(b)]}
         blobs.append(b)
         off += len(b)

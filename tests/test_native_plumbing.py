@@ -146,6 +146,27 @@ def test_zomavik_calls_fit_the_native_signatures(monkeypatch):
             "argmax"} <= set(calls), sorted(set(calls))
 
 
+def test_rupatar_calls_fit_the_native_signatures(monkeypatch):
+    from jittorinfer_b200.models import rupatar
+    hp = rupatar.preset("rupatar-tiny")
+    w = dict(rupatar.iter_random(hp, seed=0))
+    g = torch.Generator().manual_seed(1)
+    prompts = [torch.randint(0, hp.n_vocab, (n,), generator=g).tolist() for n in (9, 90)]
+
+    def run():
+        eng = LLMEngine(rupatar.RupatarModel(hp, w.items(), dtype=torch.bfloat16), EngineConfig(n_ctx=512, n_batch=32, n_parallel=2, n_ctx_slot=128))
+        return eng.generate(prompts, SamplingParams(temperature=0.0, ignore_eos=True), max_new_tokens=4)
+
+    want = run()
+    calls = []
+    fake, _ = _stand_in(calls, True)
+    monkeypatch.setattr(ops, "_native", fake)
+    monkeypatch.setattr(ops, "use_native", lambda t: True)
+    assert run() == want
+    assert {"embed_norm", "scaled_update", "rms_rows", "state_mix", "gqa_qkv_post", "gqa_attention", "moe_gate", "moe_routed", "linear",
+            "argmax"} <= set(calls), sorted(set(calls))
+
+
 def test_prompt_attention_form_is_chosen_by_what_would_be_expanded():
     """The per-head prompt attention expands the cached rows of every sequence of the step: it is taken for prompt chunks, not
     for small batches, other head sizes, or mixed steps whose rows are mostly the contexts of sequences that only decode."""
