@@ -72,6 +72,7 @@ struct GemmArgs {
     int unary;                // of a single product (JIB_UNARY_*)
     float scale, softcap, cap2;      // cap2 = 2 scale / softcap
     const float * row_scale;  // JIB_UNARY_GELU: null, or a factor of every result row's product
+    const float * bias;       // null, or [N]: a residual row that all rows share (then residual is null)
     int vec_store;            // bf16 result rows are written as 16-byte vectors through a shared-memory transpose
     const int * src_token;    // grouped, decode batches: x holds the T token rows unsorted, every expert multiplies all of
                               // them (one token tile) and sorted row i of the result is accumulator column src_token[i]
@@ -160,10 +161,12 @@ __device__ __forceinline__ float unary(float v, const GemmArgs & a) {
     if (a.softcap <= 0.f) return v * a.scale;
     return a.softcap * (1.f - __fdividef(2.f, 1.f + __expf(fminf(v * a.cap2, 80.f))));
 }
-// FN instances: 0 the product itself, 1 relu^2 and softcap, 2 gelu of the product times its row's factor.  A row past the tile's last has none.
+// FN instances: 0 the product itself, 1 relu^2 and softcap, 2 gelu of the product times its row's factor (a row past the tile's last has none),
+// 3 the product plus its feature's bias (an epilogue thread holds one feature: a register).
 template <int FN>
-__device__ __forceinline__ float function_of(float v, const GemmArgs & a, long long row, bool valid) {
+__device__ __forceinline__ float function_of(float v, const GemmArgs & a, long long row, bool valid, float bias) {
     if (FN == 0) return v;
+    if (FN == 3) return v + bias;
     if (FN == 1) return unary(v, a);
     if (a.row_scale != nullptr && valid) v *= __ldg(a.row_scale + row);
     return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
@@ -370,6 +373,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         const int q = warp & 3;                   // TMEM lane quarter this warp may access
         const int r = q * 32 + lane;              // feature row inside the tile
         const int n = n0 + r;
+        const float bias = FN == 3 && n < args.N ? args.bias[n] : 0.f;
         const bool acc_ok = mbar_wait(acc_ready, 0);
         if (!acc_ok) jib_report(args.status, JIB_ERR_WAIT_TIMEOUT, 3, 0);
         tc_fence_after();
@@ -405,7 +409,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         auto finish = [&](int t_rel, float gv, float uv) {
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
-            float y = DUAL ? gated(gv, args.act) * uv : function_of<FN>(gv, args, row, true);
+            float y = DUAL ? gated(gv, args.act) * uv : function_of<FN>(gv, args, row, true, bias);
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
                 args.ar.recv2[ar_owner][ar_par + ((size_t) args.ar.rank * args.ar.max_rows2 + row) * args.ar.d_max + n] = y;
                 return;
@@ -581,7 +585,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
 #pragma unroll
                     for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j]
-                                                                          : function_of<FN>(g[j], args, (long long) row_base + row0 + c + j, c + j < ncols);
+                                                                          : function_of<FN>(g[j], args, (long long) row_base + row0 + c + j, c + j < ncols, bias);
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -859,6 +863,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             const int ncols = min(BN, t.rows_valid - t.row0);
             const long long obase = (long long) t.batch * args.out_batch_stride;
             const long long rbase = (long long) t.batch * args.res_batch_stride;
+            const float bias = FN == 3 && t.n0 + r < args.N ? args.bias[t.n0 + r] : 0.f;
 #pragma unroll 1
             for (int c = 0; c < BN; c += 16) {
                 if (c >= ncols) break;
@@ -871,7 +876,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
                     sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k])
-                                          : function_of<FN>(g, args, (long long) t.row_base + t.row0 + c + k, c + k < ncols);
+                                          : function_of<FN>(g, args, (long long) t.row_base + t.row0 + c + k, c + k < ncols, bias);
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
@@ -1043,6 +1048,7 @@ int launch_as(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap &
 
 template <int BN, bool DUAL>
 int launch(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, dim3 grid, cudaStream_t stream) {
+    if (!DUAL && args.bias != nullptr) return launch_as<BN, DUAL, DUAL ? 0 : 3>(a, a2, b, args, grid, stream);
     if (!DUAL && args.unary == JIB_UNARY_GELU) return launch_as<BN, DUAL, DUAL ? 0 : 2>(a, a2, b, args, grid, stream);
     if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_as<BN, DUAL, DUAL ? 0 : 1>(a, a2, b, args, grid, stream);
     return launch_as<BN, DUAL, 0>(a, a2, b, args, grid, stream);
@@ -1064,6 +1070,7 @@ int launch_persistent_as(const CUtensorMap & a, const CUtensorMap & a2, const CU
 template <int BN, bool DUAL>
 int launch_persistent(const CUtensorMap & a, const CUtensorMap & a2, const CUtensorMap & b, const GemmArgs & args, int n_x, int n_y,
                       long long n_items, int sms, cudaStream_t stream) {
+    if (!DUAL && args.bias != nullptr) return launch_persistent_as<BN, DUAL, DUAL ? 0 : 3>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
     if (!DUAL && args.unary == JIB_UNARY_GELU) return launch_persistent_as<BN, DUAL, DUAL ? 0 : 2>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
     if (!DUAL && args.unary != JIB_UNARY_NONE) return launch_persistent_as<BN, DUAL, DUAL ? 0 : 1>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
     return launch_persistent_as<BN, DUAL, 0>(a, a2, b, args, n_x, n_y, n_items, sms, stream);
@@ -1180,6 +1187,11 @@ extern "C" JIB_EXPORT int jib_gemm_bf16(const jib_gemm_desc * d, void * stream_)
     if (a.ar_rs_rows < 0) return JIB_E_ARG;
     if (a.row_ptr != nullptr && (dual || d->out_f32 || d->residual != nullptr || d->ar != nullptr)) return JIB_E_ARG;
     a.act = d->act; a.unary = dual ? JIB_UNARY_NONE : d->unary; a.scale = d->scale; a.softcap = d->softcap; a.row_scale = d->row_scale;
+    a.bias = nullptr;
+    if (d->residual != nullptr && d->ldr == 0 && d->res_f32 && !dual && !grouped && batch == 1 && d->ar == nullptr && a.unary == JIB_UNARY_NONE) {
+        a.bias = (const float *) d->residual;
+        a.residual = nullptr;
+    }
     a.cap2 = d->softcap > 0.f ? 2.f * d->scale / d->softcap : 0.f;
     if (a.unary != JIB_UNARY_NONE && d->ar != nullptr) return JIB_E_ARG;
     memset(&a.ar, 0, sizeof(a.ar));
@@ -1355,7 +1367,7 @@ extern "C" JIB_EXPORT int jib_gemm_bf16_noalloc(const void * x, const void * w, 
     a.expert_list = nullptr;
     a.list_tiles = 0;
     a.ag_flags = nullptr; a.ag_epoch = nullptr; a.ag_rows = 0; a.ag_world = 0; a.ar_rs_rows = 0; a.ag_spin_limit = 0;
-    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = a.cap2 = 0.f; a.row_scale = nullptr;
+    a.act = JIB_ACT_SILU; a.unary = JIB_UNARY_NONE; a.scale = 1.f; a.softcap = a.cap2 = 0.f; a.row_scale = a.bias = nullptr;
     memset(&a.ar, 0, sizeof(a.ar));
     dim3 grid(p.n_tiles, 1, p.splits);
     switch (p.bn) {

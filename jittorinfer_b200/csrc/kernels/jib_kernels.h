@@ -256,8 +256,8 @@ JIB_EXPORT int jib_gqa_prefill(const jib_gqa * m, const void * q, const void * k
 enum { JIB_STATE_DELTA = 0, JIB_STATE_LINEAR = 1, JIB_STATE_SSD = 2, JIB_STATE_HGRN = 3, JIB_STATE_MLSTM = 4 };
 typedef struct jib_state_mix {
     // activations (bf16 or fp32): proj [T][ld] holds q (H / rep heads x K), k, v (H x V) and the pre-activation of the per-head
-    // factor (s_off; H columns; DELTA, SSD) at these columns (HGRN has no k); dec_in [T][ld_dec] the decays' (H x K; not SSD), MLSTM: fp32
-    // input | forget gates' (2 H); gate [T][ld_gate] H x V (not HGRN)
+    // factor (s_off; H columns; DELTA, SSD) at these columns (HGRN has no k); dec_in [T][ld_dec] the decays' (H x K; not SSD), MLSTM: input |
+    // forget gates' (2 H); gate [T][ld_gate] H x V (not HGRN)
     const void * proj, * dec_in, * gate;
     void * y;                  // [T][ldy] result, H x V columns
     // per-sequence state: [n_state][taps][n_conv] ring of convolution inputs (activation type), [n_state][H][K][V] fp32
@@ -265,7 +265,7 @@ typedef struct jib_state_mix {
     float * state;
     const float * conv_w;      // [taps][n_conv]: columns conv0 .. conv0 + n_conv of proj are convolved (taps 0: none), last tap = current
     const float * conv_b;      // [n_conv] or null
-    const float * bias;        // decays' (H x K) or SSD's factor's (H)
+    const float * bias;        // decays' (H x K), SSD's factor's (H), MLSTM's gates' (2 H)
     const float * neg_a;       // [H], not LINEAR
     const float * skip;        // [H], SSD
     const float * norm_w;      // [V], SSD, MLSTM [H x V]

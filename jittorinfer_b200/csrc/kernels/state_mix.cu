@@ -109,6 +109,7 @@ __global__ void __launch_bounds__(256) state_prep_kernel(const __grid_constant__
 // factors s, the maxima, and the sequence's new maximum.
 constexpr int GATE_NT = 256, GATE_N = 8;
 
+template <typename T>
 __global__ void __launch_bounds__(GATE_NT) mlstm_gates_kernel(const __grid_constant__ jib_state_mix a, int log2) {
     __shared__ float wa[GATE_NT / 32], wb[GATE_NT / 32];
     PDL_TRIGGER_TOP();
@@ -119,15 +120,16 @@ __global__ void __launch_bounds__(GATE_NT) mlstm_gates_kernel(const __grid_const
     const int slot = checked_slot(a, b, 50);
     float * top = a.extra + ((size_t) (slot < 0 ? 0 : slot) * H + h) * (a.K + 1) + a.K;
     float m0 = slot >= 0 && a.positions[q0] > 0 ? *top : 0.f;
+    const float bi = a.bias[h], bf = a.bias[H + h];
     __syncthreads();                                         // read before the last token's thread replaces it
     for (int t0 = 0; t0 < n; t0 += GATE_NT * GATE_N) {
         float gi[GATE_N], gf[GATE_N], A = 0.f, B = -INFINITY;
         const int first = t0 + threadIdx.x * GATE_N;
 #pragma unroll
         for (int i = 0; i < GATE_N; ++i) {
-            const float * z = (const float *) a.dec_in + (size_t) (q0 + min(first + i, n - 1)) * a.ld_dec + h;
-            gi[i] = z[0];
-            gf[i] = z[H];
+            const T * z = (const T *) a.dec_in + (size_t) (q0 + min(first + i, n - 1)) * a.ld_dec + h;
+            gi[i] = to_f(z[0]) + bi;
+            gf[i] = to_f(z[H]) + bf;
         }
 #pragma unroll
         for (int i = 0; i < GATE_N; ++i) {
@@ -515,8 +517,8 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) state_step_kernel(const _
     }
     float factor = 1.f, decay = 1.f;
     if (KIND == MLSTM) {
-        const float * z = (const float *) a.dec_in + (size_t) t * a.ld_dec + h;
-        const float gi = log_input_gate(z[0], a.gate_cap), x = log_forget_gate(z[H], a.gate_cap) + top;
+        const T * z = (const T *) a.dec_in + (size_t) t * a.ld_dec + h;
+        const float gi = log_input_gate(to_f(z[0]) + a.bias[h], a.gate_cap), x = log_forget_gate(to_f(z[H]) + a.bias[H + h], a.gate_cap) + top;
         top = fmaxf(x, gi);
         decay = expf(x - top);
         factor = expf(gi - top);
@@ -699,7 +701,7 @@ int run(const jib_state_mix & a, int single, cudaStream_t s) {
     }
     const bool chunks = sizeof(T) == 2 && a.chunk != nullptr && jib_state_chunk_ok(a);
     if (KIND == MLSTM) {
-        JIB_LAUNCH((mlstm_gates_kernel), dim3(a.H, a.n_seqs), GATE_NT, 0, s, a, chunks ? 1 : 0);
+        JIB_LAUNCH((mlstm_gates_kernel<T>), dim3(a.H, a.n_seqs), GATE_NT, 0, s, a, chunks ? 1 : 0);
         const int rc = launched();
         if (rc) return rc;
     }

@@ -14,9 +14,9 @@ Both sublayers of a layer read a norm in groups (equal parts of the row, each ov
 The recurrences are two kinds of ``ops.state_mix``.  Attention rows and the pooled rows are paged; states and the running maxima live in one
 row per sequence slot (``runtime/cache.py:HybridCache``), and a batch range that starts at position 0 starts from zeros.
 
-Every mixer reads one product of its input with its stacked projections (columns in multiples of 8, biases as its epilogue); the log gates of
-an mLSTM layer are a small product of their own with fp32 results.  A shared expert joins the grouped expert products when its width is a
-multiple of theirs.  On a GPU a decode step runs per layer: input GEMM [, gates], the mixer's launches, output GEMM, ``scaled_update``
+Every mixer reads one product of its input with its stacked projections (columns in multiples of 8, attention's biases as its epilogue).  A
+shared expert joins the grouped expert products when its width is a
+multiple of theirs.  On a GPU a decode step runs per layer: input GEMM, the mixer's launches, output GEMM, ``scaled_update``
 (residual, norm), router, gating, expert sort, two grouped GEMMs, ``scaled_update`` (combine, residual, next norm).  ``dtype`` float32 runs the
 same graph with fp32 kernels.
 """
@@ -268,7 +268,7 @@ def load_config(directory: str) -> RupatarHParams:
 
 
 class _Layer:
-    __slots__ = ("norm1", "norm2", "w_in", "b_in", "cols", "w_gates", "b_gates", "w_o", "b_o", "attn", "rope", "mix", "router", "n_merged", "w_up_exps",
+    __slots__ = ("norm1", "norm2", "w_in", "b_in", "cols", "w_o", "b_o", "attn", "rope", "mix", "router", "n_merged", "w_up_exps",
                  "w_down_exps", "w_up_sh", "w_down_sh")
 
     def __init__(self):
@@ -350,8 +350,11 @@ class RupatarModel:
         L.norm1 = take("norm1")
         if s.mlp is not None:
             L.norm2, L.router = take("norm2"), take("mlp.router")
-        parts = {AttentionMixer: "qkvg", Hgrn2Mixer: "qfv", MlstmMixer: "qkvg"}[type(x)]
-        L.w_in, c = stack_rows([(k, take("mix." + k)) for k in parts])
+        if isinstance(x, MlstmMixer):
+            parts = [(k, take("mix." + k)) for k in "qkvg"] + [("gates", torch.cat([take("mix.i"), take("mix.f")]))]
+        else:
+            parts = [(k, take("mix." + k)) for k in ("qfv" if isinstance(x, Hgrn2Mixer) else "qkvg")]
+        L.w_in, c = stack_rows(parts)
         L.cols, w = c, take("mix.o")
         L.w_o = torch.zeros(w.shape[0], up(w.shape[1]), dtype=w.dtype, device=w.device)      # its input's rows are 16-byte multiples
         L.w_o[:, :w.shape[1]] = w
@@ -367,9 +370,7 @@ class RupatarModel:
             L.mix = StateMix("hgrn", x.heads, x.dim, x.vdim, q_off=c["q"], v_off=c["v"], bias=take("mix.f.b"), lower=take("mix.lower"),
                              norm_w=take("mix.norm"), eps=eps)
         else:
-            L.w_gates = torch.cat([take("mix.i"), take("mix.f")]).contiguous()
-            L.b_gates = torch.cat([take("mix.i.b"), take("mix.f.b")])
-            L.mix = StateMix("mlstm", x.heads, x.dim, x.vdim, q_off=c["q"], k_off=c["k"], v_off=c["v"], norm_w=take("mix.norm"), q_scale=x.dim ** -0.5,
+            L.mix = StateMix("mlstm", x.heads, x.dim, x.vdim, q_off=c["q"], k_off=c["k"], v_off=c["v"], bias=torch.cat([take("mix.i.b"), take("mix.f.b")]), norm_w=take("mix.norm"), q_scale=x.dim ** -0.5,
                              gate_cap=x.gate_cap, eps=eps)
 
     def weight_bytes(self) -> int:
@@ -409,13 +410,13 @@ class RupatarModel:
         return ops.linear(y, L.w_o, residual=L.b_o.expand(T, -1)), v_first
 
     def _recurrence(self, i: int, L: _Layer, h: torch.Tensor, b: ForwardBatch, cache, single: bool) -> torch.Tensor:
-        T, c, m = h.shape[0], L.cols, L.mix
+        c, m = L.cols, L.mix
         n = m.heads * m.vdim
         proj = ops.linear(h, L.w_in)
         if m.kind == "hgrn":
             dec, gate = proj[:, c["f"]:c["f"] + m.heads * m.dim], None
         else:
-            dec, gate = ops.linear(h, L.w_gates, residual=L.b_gates.expand(T, -1), out_dtype=torch.float32), proj[:, c["g"]:c["g"] + n]
+            dec, gate = proj[:, c["gates"]:c["gates"] + 2 * m.heads], proj[:, c["g"]:c["g"] + n]
         y = self._rows(h, L, n)
         ops.state_mix(m, proj, dec, gate, None, cache.state["mix"][i], b.seq_slots, b.positions, b.q_start, single, y[:, :n], cache.state["extra"][i])
         return ops.linear(y, L.w_o)

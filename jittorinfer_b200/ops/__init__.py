@@ -180,7 +180,7 @@ def mingru(zxg, zb, xb, state, seq_slots, positions, q_start, single=False):
 # ---- mixers described by a spec (ops/specs.py) ------------------------------------------------------------------------------------
 def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra=None):
     """A mixer with a matrix state per head over a batch, convolution to gated norm; result columns go to ``out`` (a view).  ``state`` [n, heads,
-    dim, vdim] fp32.  "mlstm": ``dec_in`` [T, 2 heads] fp32 = input | forget gates' pre-activations, ``extra`` [n, heads, dim + 1] fp32 = what the
+    dim, vdim] fp32.  "mlstm": ``dec_in`` [T, 2 heads] = input | forget gates' pre-activations, ``extra`` [n, heads, dim + 1] fp32 = what the
     keys add up to, the running maximum."""
     return (nat() if use_native(proj) else ref).state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_start, single, out, extra)
 

@@ -824,7 +824,7 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
     if gate is not None:
         sd.gate, sd.ld_gate = gate.data_ptr(), gate.stride(0)
     if dec_in is not None:
-        assert dec_in.stride(1) == 1 and dec_in.dtype == (torch.float32 if mlstm else proj.dtype)
+        assert dec_in.stride(1) == 1 and dec_in.dtype == proj.dtype
         sd.dec_in, sd.ld_dec = dec_in.data_ptr(), dec_in.stride(0)
     sd.conv_state, sd.state, sd.n_state = _p(conv_state), state.data_ptr(), state.shape[0]
     sd.conv_w, sd.conv_b, sd.bias, sd.neg_a, sd.skip, sd.norm_w = _p(m.conv_w), _p(m.conv_b), _p(m.bias), _p(m.neg_a), _p(m.skip), _p(m.norm_w)

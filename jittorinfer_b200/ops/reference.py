@@ -448,7 +448,7 @@ def state_mix(m, proj, dec_in, gate, conv_state, state, seq_slots, positions, q_
             low = m.lower.view(H, K)
             dec, k, q = low + (1 - low) * torch.sigmoid(z), (1 - low) * torch.sigmoid(-z), F.silu(q)
         if m.kind == "mlstm":
-            i, f = (m.gate_cap * torch.tanh(dec_in[q0:q1].float() / m.gate_cap)).view(n, 2, H).unbind(1)
+            i, f = (m.gate_cap * torch.tanh((dec_in[q0:q1].float() + m.bias) / m.gate_cap)).view(n, 2, H).unbind(1)
             f, t0 = F.logsigmoid(f), extra[slot, :, K].clone() if slot >= 0 and p0 > 0 else torch.zeros(H, device=proj.device)
             tops, dec = torch.empty(n, H, device=proj.device), torch.empty(n, H, 1, device=proj.device)
             for t in range(n):

@@ -15,7 +15,7 @@ class StateMix:
     "linear": decay sigmoid(. + bias)^inv_tau per key channel, s = 1, norm per head, silu gate;
     "ssd": s = softplus(. + bias), decay exp(neg_a s) per head, silu gate, then a norm over ``norm_groups`` parts of the row;
     "hgrn": decay f = lower + (1 - lower) sigmoid(. + bias) per key channel, k = 1 - f, silu on q, s = 1, norm per head, no gate;
-    "mlstm": decay and s per head from two log gates i = cap tanh(. / cap) and f = log sigmoid(cap tanh(. / cap)), relative to a running
+    "mlstm": decay and s per head from two log gates i = cap tanh((. + bias) / cap) and f = log sigmoid(cap tanh((. + bias) / cap)) (``bias``: i, f), relative to a running
     maximum top <- max(f + top, i) that starts at 0: decay exp(f + top_old - top), s exp(i - top).  What the k add up to decays and grows like the
     state; o is divided by max(|that sum . q|, exp(-top)) + 1e-6, then a norm per head (``norm_w`` [heads * vdim]), sigmoid gate.
     ``*_off``: columns of the projection.  Columns conv0 .. conv0 + n of it pass a causal convolution of ``taps`` taps (0: none) and silu."""

@@ -54,12 +54,11 @@ def run_state(kind, dev, dtype, H, K, V, cuts, lens, seed=0, forget=0.0, write=0
         m.lower[::2] = 0
     else:
         m.norm_w, m.q_scale, m.gate_cap = rnd(H * V, seed=seed + 3, scale=0.2, mean=1.0), K ** -0.5, cap
+        m.bias = torch.tensor([write + 0.013 * h for h in range(H)] + [forget - 0.017 * h for h in range(H)])
     data, want = [], []
     for j, n in enumerate(lens):
         proj, gate = rnd(n, cols, seed=50 + 9 * j + seed), rnd(n, H * V, seed=51 + 9 * j + seed)
         dec = rnd(n, dec_w, seed=52 + 9 * j + seed, scale=1.5)
-        if kind == "mlstm":
-            dec += torch.tensor([write] * H + [forget] * H)
         if mark is not None and mark[0] < n:
             proj[mark[0], v_off:] *= mark[1]
         data.append((proj, dec, gate))
@@ -71,6 +70,7 @@ def run_state(kind, dev, dtype, H, K, V, cuts, lens, seed=0, forget=0.0, write=0
             o, S = O.hgrn2_scan(q * O.sigmoid(q), f.view(n, H, K), part(v_off, V))
             want.append((1.3 * (O.rms(o, m.eps) * m.norm_w.double()).reshape(n, -1), (S,)))
         else:
+            z = z + m.bias.double()
             i, f = cap * torch.tanh(z[:, :H] / cap), O.log_sigmoid(cap * torch.tanh(z[:, H:] / cap))
             o, S = O.mlstm_scan(part(q_off, K) * K ** -0.5, part(q_off + H * K, K), part(v_off, V), i, f)
             want.append((1.3 * O.rms(o, m.eps).reshape(n, -1) * m.norm_w.double() * O.sigmoid(gate.double()), S))
@@ -81,10 +81,10 @@ def run_state(kind, dev, dtype, H, K, V, cuts, lens, seed=0, forget=0.0, write=0
     for cut in cuts:
         part = [(j, at[j], n) for j, n in enumerate(cut) if n]
         proj, dec, gate = (torch.cat([data[j][k][p:p + n] for j, p, n in part]).to(dev) for k in range(3))
-        proj, gate = proj.to(dtype), gate.to(dtype)
+        proj, dec, gate = proj.to(dtype), dec.to(dtype), gate.to(dtype)
         out = torch.full((proj.shape[0], H * V + 8), 9.0, dtype=dtype, device=dev)
         single = single_ok and all(n == 1 for *_, n in part)
-        ops.state_mix(md, proj, dec.to(dtype) if kind == "hgrn" else dec, None if kind == "hgrn" else gate, None, state, i32([slots[j] for j, *_ in part], dev),
+        ops.state_mix(md, proj, dec, None if kind == "hgrn" else gate, None, state, i32([slots[j] for j, *_ in part], dev),
                       i32([p + k for _, p, n in part for k in range(n)], dev), starts([n for *_, n in part], dev), single, out[:, :H * V], extra)
         close(out[:, :H * V], torch.cat([want[j][0][p:p + n] for j, p, n in part]), dtype, f"cut {cut} at {at}")
         assert bool((out[:, H * V:] == 9).all())
@@ -161,11 +161,11 @@ def test_recurrence_keeps_a_mark_among_a_thousand_tokens(kind):
 @pytest.mark.parametrize("kind", ["hgrn", "mlstm"])
 def test_padding_rows_leave_every_state_alone(kind, K, dev, dtype):
     H, V = 2, 16
-    m = moved(StateMix(kind, H, K, V, q_off=0, k_off=H * K, v_off=2 * H * K, bias=rnd(H * K), lower=torch.zeros(H * K), norm_w=rnd(V if kind == "hgrn" else H * V), gate_cap=5.0), dev)
+    m = moved(StateMix(kind, H, K, V, q_off=0, k_off=H * K, v_off=2 * H * K, bias=rnd(H * K if kind == "hgrn" else 2 * H), lower=torch.zeros(H * K), norm_w=rnd(V if kind == "hgrn" else H * V), gate_cap=5.0), dev)
     st, ex = torch.full((2, H, K, V), 5.0, device=dev), torch.full((2, H, K + 1), 5.0, device=dev)
     for single in (True, False):
         out = torch.empty(2, H * V, dtype=dtype, device=dev)
-        dec = rnd(2, H * K).to(dev, dtype) if kind == "hgrn" else rnd(2, 2 * H).to(dev)
+        dec = rnd(2, H * K if kind == "hgrn" else 2 * H).to(dev, dtype)
         ops.state_mix(m, rnd(2, 2 * H * K + H * V).to(dev, dtype), dec, rnd(2, H * V).to(dev, dtype) if kind == "mlstm" else None, None, st, i32([-1, -1], dev), i32([0, 9], dev),
                       i32([0, 1, 2], dev), single, out, ex if kind == "mlstm" else None)
     assert bool((st == 5).all()) and bool((ex == 5).all())
@@ -334,7 +334,7 @@ def test_norms_in_parts(d, groups, dev, dtype):
     w, table = rnd(d, seed=1, scale=0.3, mean=1.0), rnd(20, d, seed=2)
     x, o, y, f = rnd(T, d, seed=3, scale=2.0), rnd(T, d, seed=4), rnd(T * k, d, seed=5), rnd(T, d, seed=6)
     for t in (table, x):                                             # parts of very different sizes
-        t *= (1 + torch.arange(groups)).repeat_interleave(d // groups) / groups
+        t.copy_((t * (1 + torch.arange(groups)).repeat_interleave(d // groups) / groups).bfloat16())
     put, put32 = (lambda t: t.to(dev, dtype)), (lambda t: t.to(dev))          # noqa: E731
     nxt = RowNorms(eps, w.to(dev), groups=groups)
     norm = lambda v: O.group_norm(v.double(), w.double(), groups, eps)          # noqa: E731
