@@ -43,6 +43,45 @@ template <> __device__ __forceinline__ float capped<bf16>(float s, float cap) {
 }
 template <> __device__ __forceinline__ float capped<float>(float s, float cap) { return cap * tanhf(s / cap); }
 
+// 4 adjacent elements of aligned rows, kept as stored until they are needed
+template <typename T> struct Vec4;
+template <> struct Vec4<float> {
+    float4 r;
+    __device__ __forceinline__ void load(const float * p) { r = *(const float4 *) p; }
+    __device__ __forceinline__ float4 get() const { return r; }
+    static __device__ __forceinline__ void store(float * p, float4 v) { *(float4 *) p = v; }
+};
+template <> struct Vec4<bf16> {
+    uint2 r;
+    __device__ __forceinline__ void load(const bf16 * p) { r = *(const uint2 *) p; }
+    __device__ __forceinline__ float4 get() const {
+        const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *) &r.x), y = __bfloat1622float2(*(const __nv_bfloat162 *) &r.y);
+        return make_float4(x.x, x.y, y.x, y.y);
+    }
+    static __device__ __forceinline__ void store(bf16 * p, float4 v) {
+        uint2 x;
+        *(__nv_bfloat162 *) &x.x = __floats2bfloat162_rn(v.x, v.y);
+        *(__nv_bfloat162 *) &x.y = __floats2bfloat162_rn(v.z, v.w);
+        *(uint2 *) p = x;
+    }
+};
+
+// The pooled block a CTA of a portion works on: one CTA (blockIdx.x) per block that can end in this batch.  Sequence b's begin at index
+// q_start[b] / pool_size + b, the first is the one its first new position lies in; indices in the gaps have none.
+__device__ __forceinline__ bool pool_block(const jib_gqa & a, int & b, int & block) {
+    const int P = a.pool_size;
+    int hi = a.n_seqs;
+    b = 0;
+    while (hi - b > 1) {
+        const int mid = (b + hi) >> 1;
+        if (a.q_start[mid] / P + mid <= (int) blockIdx.x) b = mid; else hi = mid;
+    }
+    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0, S = a.seq_lens[b];
+    if (n <= 0 || S < n) return false;
+    block = (S - n) / P + (int) blockIdx.x - (q0 / P + b);
+    return block >= (S - n) / P && (block + 1) * P <= S;
+}
+
 // ---- norm, rotation, cache rows: one warp per (token, head of q / k / v) ------------------------------------------------------
 constexpr int POST_D = 16;                                   // elements of a head per lane (N): D <= 32 * POST_D
 
@@ -157,22 +196,138 @@ __global__ void __launch_bounds__(256) gqa_qkv_post_kernel(const __grid_constant
     }
 }
 
-// Means of complete blocks of pool_size positions, portions.  One CTA per block that can end in this batch: sequence b's begin at index
-// q_start[b] / pool_size + b, the first is the one its first new position lies in; indices in the gaps have none.
+// The same for rotated neighbours (and no norm weights) where whole vectors of 4 can be read: a lane holds 4 adjacent elements, two pairs, and
+// the warp takes TOK tokens at a time.  D, V <= 128 * N.
+template <typename T, int N, int TOK>
+__global__ void __launch_bounds__(256) gqa_pairs_post_kernel(const __grid_constant__ jib_gqa a, const T * __restrict__ q, const T * __restrict__ k,
+                                                             const T * __restrict__ v, long long ld, const float * __restrict__ rope,
+                                                             const int * __restrict__ slot_mapping, T * __restrict__ q_out) {
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int lane = threadIdx.x & 31, item = blockIdx.x * 8 + (threadIdx.x >> 5), t0 = blockIdx.y * TOK;
+    const int D = a.D, V = a.V, H = a.H, G = a.G;
+    if (item >= H + 2 * G) return;
+    const bool is_q = item < H, is_v = item >= H + G;
+    const int head = is_q ? item : is_v ? item - H - G : item - H, n = is_v ? V : D;
+    Vec4<T> x[TOK][N], y[TOK][N];
+    T * dst[TOK];
+    float4 cs[TOK][N];                                       // cos, sin of the two pairs
+#pragma unroll
+    for (int j = 0; j < TOK; ++j) {                          // everything is requested before any of it is used
+        const int t = min(t0 + j, a.T - 1);
+        dst[j] = nullptr;
+        if (t0 + j < a.T) {
+            if (is_q) {
+                dst[j] = q_out + ((size_t) t * H + head) * D;
+            } else {
+                const long long slot = slot_mapping[t];
+                if (slot >= a.n_slots) {
+                    if (lane == 0) jib_report(a.status, JIB_ERR_BOUNDS, 48, (int) slot);
+                } else if (slot >= 0) {
+                    dst[j] = (T *) a.cache + (size_t) slot * a.row + (is_v ? G * D : 0) + head * n;
+                }
+            }
+        }
+        int at = a.positions[t];
+        if (!is_v && (at < 0 || at >= a.max_pos)) {
+            if (lane == 0) jib_report(a.status, JIB_ERR_BOUNDS, 49, at);
+            at = 0;
+        }
+        const T * src = (is_q ? q : is_v ? v : k) + (size_t) t * ld + head * n, * first = (const T *) a.v_first + (size_t) t * a.ld_first + head * n;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = 4 * (lane + 32 * i);
+            if (c >= n) continue;
+            x[j][i].load(src + c);
+            if (is_v && a.mix_v) y[j][i].load(first + c);
+            cs[j][i] = make_float4(1.f, 0.f, 1.f, 0.f);
+            if (!is_v && c < a.rot) {
+                const float2 * r = (const float2 *) rope + (size_t) at * (a.rot / 2) + c / 2;
+                const float2 r0 = r[0], r1 = c + 2 < a.rot ? r[1] : make_float2(1.f, 0.f);
+                cs[j][i] = make_float4(r0.x, r0.y, r1.x, r1.y);
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < TOK; ++j) {
+        float4 e[N];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            if (4 * (lane + 32 * i) >= n) continue;
+            const float4 z = x[j][i].get(), r = cs[j][i];
+            if (is_v) {
+                e[i] = z;
+                if (a.mix_v) {
+                    const float4 w = y[j][i].get();
+                    const float m = a.v_mix, o = 1.f - m;
+                    e[i] = make_float4(o * z.x + m * w.x, o * z.y + m * w.y, o * z.z + m * w.z, o * z.w + m * w.w);
+                }
+            } else {
+                e[i] = make_float4(z.x * r.x - z.y * r.y, z.y * r.x + z.x * r.y, z.z * r.z - z.w * r.w, z.w * r.z + z.z * r.w);
+                ss += e[i].x * e[i].x + e[i].y * e[i].y + e[i].z * e[i].z + e[i].w * e[i].w;
+            }
+        }
+        const float inv = a.unit && !is_v ? rsqrtf(warp_sum(ss) / (float) D + a.eps) : 1.f;
+        if (dst[j] == nullptr) continue;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = 4 * (lane + 32 * i);
+            if (c < n) Vec4<T>::store(dst[j] + c, make_float4(e[i].x * inv, e[i].y * inv, e[i].z * inv, e[i].w * inv));
+        }
+    }
+}
+
+// Means of complete blocks of pool_size positions, portions, where whole 16-byte vectors can be read: see gqa_pool_kernel; blockIdx.y takes 32
+// vectors of the row, 8 threads share one's rows.
+template <typename T>
+__global__ void __launch_bounds__(256) gqa_pool_vec_kernel(const __grid_constant__ jib_gqa a) {
+    constexpr int E = 16 / sizeof(T);
+    __shared__ float part[8][32][E + 1];
+    PDL_TRIGGER_TOP();
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    int b, block;
+    if (!pool_block(a, b, block)) return;
+    const int P = a.pool_size, lane = threadIdx.x & 31, g = threadIdx.x >> 5, c = (blockIdx.y * 32 + lane) * E;
+    const bool in = c < a.G * (a.D + a.V);
+    const int * bt = a.block_tables + (size_t) b * a.max_blocks;
+    float s[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) s[e] = 0.f;
+    if (in) {
+#pragma unroll 4
+        for (int p = block * P + g; p < block * P + P; p += 8) {
+            const uint4 r = *(const uint4 *) ((const T *) a.cache + ((long long) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row + c);
+#pragma unroll
+            for (int e = 0; e < E; ++e) s[e] += to_f(((const T *) &r)[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < E; ++e) part[g][lane][e] = s[e];
+    __syncthreads();
+    if (g > 0 || !in) return;
+    T out[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+        float x = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) x += part[k][lane][e];
+        put(out + e, x / (float) P);
+    }
+    T * dst = (T *) a.pool + gqa_pool_row(bt, block, P, a.pool_rows, a.block_size) * a.row + c;
+    uint4 r;
+    memcpy(&r, out, 16);
+    *(uint4 *) dst = r;
+}
+
+// Any sizes.
 template <typename T>
 __global__ void __launch_bounds__(256) gqa_pool_kernel(const __grid_constant__ jib_gqa a) {
     PDL_TRIGGER_TOP();
     pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
-    const int P = a.pool_size;
-    int b = 0, hi = a.n_seqs;
-    while (hi - b > 1) {
-        const int mid = (b + hi) >> 1;
-        if (a.q_start[mid] / P + mid <= (int) blockIdx.x) b = mid; else hi = mid;
-    }
-    const int q0 = a.q_start[b], n = a.q_start[b + 1] - q0, S = a.seq_lens[b];
-    if (n <= 0 || S < n) return;
-    const int block = (S - n) / P + (int) blockIdx.x - (q0 / P + b), p0 = block * P;
-    if (block < (S - n) / P || p0 + P > S) return;
+    int b, block;
+    if (!pool_block(a, b, block)) return;
+    const int P = a.pool_size, p0 = block * P;
     const int * bt = a.block_tables + (size_t) b * a.max_blocks;
     T * dst = (T *) a.pool + gqa_pool_row(bt, block, P, a.pool_rows, a.block_size) * a.row;
     const int cols = a.G * (a.D + a.V);
@@ -278,6 +433,15 @@ __device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, c
         const int r = i / V, col = i % V;
         const int t = w.q0 + w.i0 + r / w.nh, h = w.h0 + r % w.nh;
         const float sink = !a.sink ? -INFINITY : a.sink_w != nullptr ? a.sink_w[h] : 0.f;
+        const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + (a.gate_each ? h * V + col : h)]) : 0.f;
+        if (n_splits == 1) {
+            const float m1 = m_s[r], m = fmaxf(sink, m1), e = m1 == -INFINITY ? 0.f : exp_t<T>(m1 - m);
+            const float l = e * l_s[r] + (a.sink ? exp_t<T>(sink - m) : 0.f);
+            float y = l > 0.f ? e * part[r * V + col] / l * a.out_scale : 0.f;
+            if (gate != nullptr) y /= 1.f + exp_t<T>(-gt);
+            put(out + (size_t) t * ldo + h * V + col, y);
+            continue;
+        }
         float ms[8], ls[8], os[8], m = sink;
 #pragma unroll
         for (int s = 0; s < 8; ++s) {                        // every peer's value requested before any is used
@@ -288,7 +452,6 @@ __device__ __forceinline__ void finish_rows(const jib_gqa & a, const Work & w, c
             ls[s] = n_splits > 1 ? ld_peer(l_s + r, s) : l_s[r];
             os[s] = n_splits > 1 ? ld_peer(part + r * V + col, s) : part[r * V + col];
         }
-        const float gt = gate != nullptr ? to_f(gate[(size_t) t * ld_gate + (a.gate_each ? h * V + col : h)]) : 0.f;
 #pragma unroll
         for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
         float l = a.sink ? exp_t<T>(sink - m) : 0.f, o = 0.f;
@@ -457,8 +620,9 @@ __global__ void __launch_bounds__(NT) gqa_attention_kernel(const __grid_constant
 }
 
 // ---- attention on tensor cores: bf16, D and V multiples of 16 ---------------------------------------------------------------------
-// The same decomposition; the 16 rows are the M of m16n8k16 products.  Tiles of 64 keys arrive by asynchronous copies, one ahead; each
-// of the 4 warps takes 16 keys of a tile and keeps its own running maximum, sum and output (NV x 8 columns), which meet at the end.
+// The same decomposition; the 16 rows are the M of m16n8k16 products.  Tiles of 64 keys arrive by asynchronous copies, ST - 1 ahead; each
+// of the 4 warps takes 16 keys of a tile, copies them itself (no barrier in the loop) and keeps its own running maximum, sum and output
+// (NV x 8 columns), which meet at the end.
 constexpr int MK = 64, PADC = 8;                             // keys per tile; padding of the shared rows (16 bytes: rows hit different banks)
 
 __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&x)[4], uint32_t y0, uint32_t y1) {
@@ -472,11 +636,16 @@ __device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
 __device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ void cp16(uint32_t dst, const void * src, bool valid) {       // zeros if not valid (src is not read)
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
 }
 
-template <int NV>                                            // columns of V per 16: V <= 16 NV
+template <int NV, int ST>                                    // columns of V per 16: V <= 16 NV; tiles in shared memory
 __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib_gqa a, const bf16 * __restrict__ q, const bf16 * __restrict__ gate,
                                                      long long ld_gate, bf16 * __restrict__ out, long long ldo, int run, int heads) {
     extern __shared__ __align__(16) uint8_t smem_mma[];
@@ -492,18 +661,46 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
     const int * bt = a.block_tables + (size_t) w.b * a.max_blocks;
     const bf16 * cache = (const bf16 *) a.cache;
     const int d8 = D / 8, v8 = V / 8;
-    // a thread copies half of one key's row: 2 threads per key
+    // the warp's 16 keys, as 16-byte units that go round the lanes, row after row (several at a time if they are short).  16 adjacent positions
+    // of a cache block follow one another; else lane l knows where key l & 15 is
+    const int units = d8 + v8, at_once = units <= 32 ? 32 / units : 1, sub = units <= 32 ? lane / units : 0, unit = units <= 32 ? lane % units : lane;
+    const bool whole = a.block_size % 16 == 0 && units == 32;
     auto stage = [&](int kt, int buf) {
-        if (kt < w.k_hi) {
+        if (kt < w.k_hi && kt >= w.pt && whole) {
+            const int p = (kt + w.t0) * MK + warp * 16;
+            const bool any = p + 15 >= w.lo && p < w.end;    // else there may be no block
+            const bool is_k = lane < d8;
+            const int col = is_k ? w.g * D + lane * 8 : a.G * D + w.g * V + (lane - d8) * 8;
+            const bf16 * src = any ? cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row + col : cache;
+            uint32_t dst = kv_addr + buf * tile_bytes + (is_k ? warp * 16 * LD + lane * 8 : MK * LD + warp * 16 * LV + (lane - d8) * 8) * 2;
+            const uint32_t step = (is_k ? LD : LV) * 2;
+            const size_t row = any ? (size_t) a.row : 0;
+#pragma unroll
+            for (int r = 0; r < 16; ++r) {
+                cp16(dst, src, p + r >= w.lo && p + r < w.end);
+                dst += step;
+                src += row;
+            }
+        } else if (kt < w.k_hi) {
             const bool pooled = kt < w.pt;
-            const int j = tid >> 1, p = (pooled ? kt : kt + w.t0) * MK + j;
+            const int p = (pooled ? kt : kt + w.t0) * MK + warp * 16 + (lane & 15);
             const bool in = pooled ? p < w.nb : p >= w.lo && p < w.end;
             const bf16 * row = !in ? cache
                                : pooled ? (const bf16 *) a.pool + gqa_pool_row(bt, p, a.pool_size, a.pool_rows, a.block_size) * a.row
                                         : cache + ((size_t) bt[p / a.block_size] * a.block_size + p % a.block_size) * a.row;
-            const uint32_t kd = kv_addr + buf * tile_bytes + j * LD * 2, vd = kv_addr + buf * tile_bytes + (MK * LD + j * LV) * 2;
-            for (int c = tid & 1; c < d8; c += 2) cp16(kd + c * 16, row + w.g * D + c * 8, in);
-            for (int c = tid & 1; c < v8; c += 2) cp16(vd + c * 16, row + a.G * D + w.g * V + c * 8, in);
+            const uint32_t kd = kv_addr + buf * tile_bytes + warp * 16 * LD * 2, vd = kv_addr + buf * tile_bytes + (MK * LD + warp * 16 * LV) * 2;
+#pragma unroll 4
+            for (int r0 = 0; r0 < 16; r0 += at_once) {
+                const int r = r0 + sub;
+                const bf16 * src = (const bf16 *) __shfl_sync(0xffffffffu, (unsigned long long) row, r & 15);
+                const bool ok = __shfl_sync(0xffffffffu, in, r & 15);
+                if (sub >= at_once || r >= 16) continue;
+                for (int c = unit; c < units; c += 32) {
+                    if (c < d8) cp16(kd + (r * LD + c * 8) * 2, src + w.g * D + c * 8, ok);
+                    else cp16(vd + (r * LV + (c - d8) * 8) * 2, src + a.G * D + w.g * V + (c - d8) * 8, ok);
+                    if (units <= 32) break;
+                }
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -511,7 +708,9 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
         const int r = i / d8, c = i % d8;
         cp16(q_addr + (r * LD + c * 8) * 2, q + (r < w.rows ? ((size_t) (w.q0 + w.i0 + r / w.nh) * a.H + w.h0 + r % w.nh) * D + c * 8 : 0), r < w.rows);
     }
-    stage(w.k_lo, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < ST - 1; ++i) stage(w.k_lo + i, i);
     const int fr = lane >> 2, fc = (lane & 3) * 2;
     // positions, first keys and pooled blocks of this thread's two rows
     int pos[2], first[2], blocks[2];
@@ -529,11 +728,13 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
         for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
     constexpr float LOG2E = 1.4426950408889634f;
     const float sc = a.softcap > 0.f ? 2.f * LOG2E * a.scale / a.softcap : a.scale * LOG2E, cap = a.softcap * LOG2E;
+    asm volatile("cp.async.wait_group %0;" ::"n"(ST - 1) : "memory");
+    __syncthreads();                                         // the queries are there
     for (int kt = w.k_lo; kt < w.k_hi; ++kt) {
-        const int buf = (kt - w.k_lo) & 1;
-        stage(kt + 1, buf ^ 1);
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
+        const int buf = (kt - w.k_lo) % ST;
+        stage(kt + ST - 1, (buf + ST - 1) % ST);
+        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 1) : "memory");
+        __syncwarp();
         const uint32_t k_addr = kv_addr + buf * tile_bytes + warp * 16 * LD * 2, v_addr = kv_addr + buf * tile_bytes + (MK * LD + warp * 16 * LV) * 2;
         float s[2][4];
 #pragma unroll
@@ -567,13 +768,14 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
                 s[n][e] = p < end[e >> 1] && p >= from[e >> 1] ? y : -INFINITY;
                 mt[e >> 1] = fmaxf(mt[e >> 1], s[n][e]);
             }
-        float cf[2];
+        float cf[2], base[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             mt[e] = fmaxf(mt[e], __shfl_xor_sync(0xffffffffu, mt[e], 1));
             mt[e] = fmaxf(mt[e], __shfl_xor_sync(0xffffffffu, mt[e], 2));
             const float mn = fmaxf(m[e], mt[e]);
-            cf[e] = mn == -INFINITY ? 1.f : exp2f(m[e] - mn);
+            base[e] = mn == -INFINITY ? 0.f : mn;            // every score is -inf then
+            cf[e] = ex2(m[e] - base[e]);
             m[e] = mn;
             l[e] *= cf[e];
         }
@@ -582,7 +784,7 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
         for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const float p0 = s[n][2 * e] == -INFINITY ? 0.f : exp2f(s[n][2 * e] - m[e]), p1 = s[n][2 * e + 1] == -INFINITY ? 0.f : exp2f(s[n][2 * e + 1] - m[e]);
+                const float p0 = ex2(s[n][2 * e] - base[e]), p1 = ex2(s[n][2 * e + 1] - base[e]);
                 l[e] += p0 + p1;
                 const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
                 x[n * 2 + e] = *(const uint32_t *) &pk;
@@ -600,7 +802,7 @@ __global__ void __launch_bounds__(NT) gqa_mma_kernel(const __grid_constant__ jib
             mma(o[n], x, y[0], y[1]);
             mma(o[n + 1], x, y[2], y[3]);
         }
-        __syncthreads();                                     // the buffer is free
+        __syncwarp();                                        // the buffer is free
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
@@ -680,18 +882,48 @@ bool mma_ok(const jib_gqa & a, const void * q) {
     return a.D % 16 == 0 && a.V % 16 == 0 && a.V <= 256 && a.row % 8 == 0 && (((uintptr_t) a.cache | (uintptr_t) a.pool | (uintptr_t) q) & 15) == 0;
 }
 
+template <int NV, int ST>
+int launch_mma_as(const jib_gqa & a, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single, int splits,
+                  cudaStream_t s) {
+    const int tile = MK * (a.D + a.V + 2 * PADC) * 2, smem = ROWS * (a.D + PADC) * 2 + ST * tile;       // >= the [ROWS][V] partial results
+    constexpr int CAP = 220 * 1024;
+    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
+    if (smem > CAP || !jib::ensure_dyn_smem(gqa_mma_kernel<NV, ST>, CAP, done)) return JIB_E_ARG;
+    const int rep = a.H / a.G, heads = rep < ROWS ? rep : ROWS, run = single ? 0 : ROWS / heads;
+    const dim3 grid(single ? a.T : a.T / run + a.n_seqs, a.G * ((rep + heads - 1) / heads), splits);
+    const cudaError_t e = jib::launch_pdl_cluster(gqa_mma_kernel<NV, ST>, grid, dim3(NT), (size_t) smem, s, splits, a, (const bf16 *) q, (const bf16 *) gate,
+                                                  ld_gate, (bf16 *) out, ldo, run, heads);
+    if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
+    return launched();
+}
+
+// Three tiles in shared memory while two CTAs fit on an SM
 template <int NV>
 int launch_mma(const jib_gqa & a, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single, int splits,
                cudaStream_t s) {
-    const int tile = MK * (a.D + a.V + 2 * PADC) * 2, smem = ROWS * (a.D + PADC) * 2 + 2 * tile;       // >= the [ROWS][V] partial results
-    constexpr int CAP = 220 * 1024;
-    static std::atomic<unsigned char> done[jib::MAX_DEVICES];
-    if (smem > CAP || !jib::ensure_dyn_smem(gqa_mma_kernel<NV>, CAP, done)) return JIB_E_ARG;
-    const int rep = a.H / a.G, heads = rep < ROWS ? rep : ROWS, run = single ? 0 : ROWS / heads;
-    const dim3 grid(single ? a.T : a.T / run + a.n_seqs, a.G * ((rep + heads - 1) / heads), splits);
-    const cudaError_t e = jib::launch_pdl_cluster(gqa_mma_kernel<NV>, grid, dim3(NT), (size_t) smem, s, splits, a, (const bf16 *) q, (const bf16 *) gate,
-                                                  ld_gate, (bf16 *) out, ldo, run, heads);
-    if (e != cudaSuccess) { (void) cudaGetLastError(); return JIB_E_LAUNCH; }
+    const int smem = ROWS * (a.D + PADC) * 2 + 3 * MK * (a.D + a.V + 2 * PADC) * 2;
+    return smem <= 112 * 1024 ? launch_mma_as<NV, 3>(a, q, gate, ld_gate, out, ldo, single, splits, s)
+                              : launch_mma_as<NV, 2>(a, q, gate, ld_gate, out, ldo, single, splits, s);
+}
+
+// Whole vectors of 4 in every row that gqa_pairs_post reads and writes
+bool pairs_ok(const jib_gqa & a, const void * q, const void * k, const void * v, long long ld, const void * q_out, int el) {
+    const uintptr_t at = (uintptr_t) q | (uintptr_t) k | (uintptr_t) v | (uintptr_t) q_out | (uintptr_t) a.cache | (uintptr_t) a.v_first;
+    const long long n = a.D | a.V | ld | a.row | (a.mix_v ? a.ld_first : 0);
+    return at % (4 * el) == 0 && n % 4 == 0 && a.D <= 512 && a.V <= 512;
+}
+
+int launch_pool(const jib_gqa & a, int f32, cudaStream_t s) {
+    if (a.q_start == nullptr || a.seq_lens == nullptr || a.n_seqs <= 0) return JIB_E_ARG;
+    const int e = f32 ? 4 : 8, cols = a.G * (a.D + a.V), n = a.T / a.pool_size + a.n_seqs;
+    if (cols % e == 0 && a.row % e == 0 && (((uintptr_t) a.cache | (uintptr_t) a.pool) & 15) == 0) {
+        const dim3 grid(n, (cols / e + 31) / 32);
+        if (f32) JIB_LAUNCH((gqa_pool_vec_kernel<float>), grid, 256, 0, s, a);
+        else JIB_LAUNCH((gqa_pool_vec_kernel<bf16>), grid, 256, 0, s, a);
+        return launched();
+    }
+    if (f32) JIB_LAUNCH((gqa_pool_kernel<float>), n, 256, 0, s, a);
+    else JIB_LAUNCH((gqa_pool_kernel<bf16>), n, 256, 0, s, a);
     return launched();
 }
 
@@ -712,6 +944,28 @@ JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * 
     if (a.T <= 0) return 0;
     if (!ok(a) || (a.mix_v && a.v_first == nullptr) || (single && a.pool_size > 0 && a.n_seqs != a.T)) return JIB_E_ARG;
     cudaStream_t s = (cudaStream_t) stream;
+    const int el = f32 ? 4 : 2;
+    const bool pool = a.pool_size > 0;
+    if (a.neighbours && q_norm == nullptr && k_norm == nullptr && !(single && pool) && pairs_ok(a, q, k, v, ld, q_out, el)) {
+        const int n = a.D > a.V ? a.D : a.V, tok = a.T >= 256 && n <= 256 ? 2 : 1;
+        const dim3 grid((a.H + 2 * a.G + 7) / 8, (a.T + tok - 1) / tok);
+#define PAIRS(TT, N, TOK) \
+    JIB_LAUNCH((gqa_pairs_post_kernel<TT, N, TOK>), grid, 256, 0, s, a, (const TT *) q, (const TT *) k, (const TT *) v, ld, rope, slot_mapping, (TT *) q_out)
+#define CALL(N, TOK)                    \
+    do {                                \
+        if (f32) PAIRS(float, N, TOK);  \
+        else PAIRS(bf16, N, TOK);       \
+    } while (0)
+        if (n <= 128 && tok == 2) CALL(1, 2);
+        else if (n <= 128) CALL(1, 1);
+        else if (n <= 256 && tok == 2) CALL(2, 2);
+        else if (n <= 256) CALL(2, 1);
+        else CALL(4, 1);
+#undef CALL
+#undef PAIRS
+        const int rc = launched();
+        return rc || !pool ? rc : launch_pool(a, f32, s);
+    }
     const dim3 grid((a.H + 2 * a.G + 7) / 8, a.T);
     const int smem = 8 * a.D * 4;
 #define POST(TT, N)                                                                                                                        \
@@ -728,11 +982,7 @@ JIB_EXPORT int jib_gqa_qkv_post(const jib_gqa * m, const void * q, const void * 
 #undef CALL
 #undef POST
     const int rc = launched();
-    if (rc || single || a.pool_size == 0) return rc;
-    if (a.q_start == nullptr || a.seq_lens == nullptr || a.n_seqs <= 0) return JIB_E_ARG;
-    if (f32) JIB_LAUNCH((gqa_pool_kernel<float>), a.T / a.pool_size + a.n_seqs, 256, 0, s, a);
-    else JIB_LAUNCH((gqa_pool_kernel<bf16>), a.T / a.pool_size + a.n_seqs, 256, 0, s, a);
-    return launched();
+    return rc || single || !pool ? rc : launch_pool(a, f32, s);
 }
 
 JIB_EXPORT int jib_gqa_attention(const jib_gqa * m, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single,

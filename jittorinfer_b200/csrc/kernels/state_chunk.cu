@@ -167,6 +167,18 @@ template <int K> __device__ __forceinline__ void put_tile4(uint8_t * hi, int r, 
     *(uint2 *) (hi + C * K * 2 + tile_off<K>(r, c)) = l;
 }
 
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&x)[4], uint32_t y0, uint32_t y1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(x[0]), "r"(x[1]), "r"(x[2]), "r"(x[3]), "r"(y0), "r"(y1));
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
 // ---- prepare: DELTA, LINEAR ------------------------------------------------------------------------------------------------------
 template <int K> constexpr int prep_smem(int V) { return 4 * (3 * C * (K + 4) + C * (V + 4) + C * 36 + 3 * C); }
 
@@ -401,7 +413,7 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_kernel(const __grid_const
 // (A_ts also holds the factor s_s of the earlier token, and D on the diagonal).  Then runs of 256 value columns (bf16 into a.v).
 constexpr int HB = 16;
 
-template <int KIND, int K>
+template <int K>
 __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_constant__ jib_state_mix a) {
     using R = Rec<SSD, K>;
     constexpr int KS = K + 4;
@@ -451,21 +463,14 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
         for (int i = tid >> 5; i < HB && block * HB + i < a.rep; i += NT / 32) {
             const int h = y * a.rep + block * HB + i;
             uint8_t * hr = ssd_head_part<K>(a, ci, h);
-            float f = 0.f, g;                                // lane t: s_t, G_t
-            if (KIND == MLSTM) {
-                const size_t at = (size_t) (r0 + t0 + min(lane, n - 1)) * a.H + h;
-                f = lane < n ? a.s[at] : 0.f;
-                g = lane < n ? a.dec[at] : 0.f;
-            } else {
-                if (lane < n) f = softplus_series(to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + lane) * a.ld + a.s_off + h]) + a.bias[h]);
-                g = a.neg_a[h] * LOG2E * f;
-            }
+            const float f = lane < n ? softplus_series(to_f(((const bf16 *) a.proj)[(size_t) (r0 + t0 + lane) * a.ld + a.s_off + h]) + a.bias[h]) : 0.f;
+            float g = a.neg_a[h] * LOG2E * f;                // lane t: G_t
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const float x = __shfl_up_sync(0xffffffffu, g, o);
                 if (lane >= o) g += x;
             }
-            const float gC = __shfl_sync(0xffffffffu, g, 31), skip = KIND == MLSTM ? 0.f : a.skip[h];
+            const float gC = __shfl_sync(0xffffffffu, g, 31), skip = a.skip[h];
             float * e = (float *) (hr + R::E - R::A);
             e[lane] = ex2(g);
             e[C + lane] = f * ex2(gC - g);
@@ -494,23 +499,87 @@ __global__ void __launch_bounds__(NT, 3) chunk_prepare_ssd_kernel(const __grid_c
     }
 }
 
-// ---- pass --------------------------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&x)[4], uint32_t y0, uint32_t y1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(x[0]), "r"(x[1]), "r"(x[2]), "r"(x[3]), "r"(y0), "r"(y1));
-}
-__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+// ---- prepare: MLSTM ----------------------------------------------------------------------------------------------------------------
+// One CTA per chunk and head: q and k as they are, their products on the tensor cores (a warp per 16 x 8 of them), times decays and factors.
+template <int K>
+__global__ void __launch_bounds__(NT) chunk_prepare_mlstm_kernel(const __grid_constant__ jib_state_mix a) {
+    using R = Rec<MLSTM, K>;
+    __shared__ __align__(16) uint8_t tiles[2 * R::TILE];
+    PDL_TRIGGER_TOP();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    pdl_wait();      // inputs come from earlier kernels; nothing is written before this point
+    const int ci = blockIdx.x, h = blockIdx.y, b = chunk_seq(a, ci);
+    const int r0 = a.q_start[b], nr = a.q_start[b + 1] - r0, t0 = (ci - chunk_key(a.q_start, b)) * C;
+    if (t0 < 0 || t0 >= nr) return;
+    const int n = min(C, nr - t0);
+    uint8_t * rec = ssd_group_part<K>(a, ci, h), * hr = ssd_head_part<K>(a, ci, h);
+    const bf16 * x = (const bf16 *) a.proj + (size_t) (r0 + t0) * a.ld + h * K;
+    constexpr int U = K / 8;                                 // 16-byte units of a row
+    uint4 v[2 * C * U / NT];
+#pragma unroll
+    for (int i = 0; i < 2 * C * U / NT; ++i) {
+        const int j = tid + i * NT, r = j / U % C, u = j % U;
+        v[i] = make_uint4(0, 0, 0, 0);
+        if (r < n) v[i] = *(const uint4 *) (x + (size_t) r * a.ld + (j < C * U ? a.q_off : a.k_off) + u * 8);
+    }
+    float f = 0.f, g = 0.f;                                  // lane t: s_t, G_t
+    if (lane < n) {
+        const size_t at = (size_t) (r0 + t0 + lane) * a.H + h;
+        f = a.s[at];
+        g = a.dec[at];
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float y = __shfl_up_sync(0xffffffffu, g, o);
+        if (lane >= o) g += y;
+    }
+    const float gC = __shfl_sync(0xffffffffu, g, 31);
+    if (warp == 0) {
+        float * e = (float *) (hr + R::E - R::A);
+        e[lane] = ex2(g);
+        e[C + lane] = f * ex2(gC - g);
+    }
+#pragma unroll
+    for (int i = 0; i < 2 * C * U / NT; ++i) {
+        const int j = tid + i * NT, r = j / U % C, u = j % U, off = (j < C * U ? R::Q : R::D) + tile_off<K>(r, u * 8);
+        *(uint4 *) (tiles + off) = v[i];
+        *(uint4 *) (rec + off) = v[i];
+    }
+    __syncthreads();
+    const int mt = warp >> 2, nt = warp & 3;                 // rows (later tokens) 16 mt .., columns (earlier ones) 8 nt ..
+    const uint32_t base = sm100::smem_u32(tiles);
+    float c[4] = {0.f, 0.f, 0.f, 0.f};
+    if (8 * nt <= 16 * mt + 15) {
+#pragma unroll
+        for (int kk = 0; kk < K; kk += 32) {
+            uint32_t p[4], q[4], y[4];
+            const int r = mt * 16 + (lane & 15), s = nt * 8 + (lane & 7);
+            ldm4(p, base + R::Q + tile_off<K>(r, kk + (lane >> 4) * 8));
+            ldm4(q, base + R::Q + tile_off<K>(r, kk + 16 + (lane >> 4) * 8));
+            ldm4(y, base + R::D + tile_off<K>(s, kk + (lane >> 3) * 8));
+            mma(c, p, y[0], y[1]);
+            mma(c, q, y[2], y[3]);
+        }
+    }
+    const int s0 = nt * 8 + (lane & 3) * 2;
+    const float g0 = __shfl_sync(0xffffffffu, g, s0), g1 = __shfl_sync(0xffffffffu, g, s0 + 1);
+    const float f0 = __shfl_sync(0xffffffffu, f, s0), f1 = __shfl_sync(0xffffffffu, f, s0 + 1);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int t = mt * 16 + (lane >> 2) + 8 * e;
+        const float gt = __shfl_sync(0xffffffffu, g, t);
+        uint32_t hi, lo;
+        split2(s0 <= t ? c[2 * e] * (ex2(gt - g0) * f0) : 0.f, s0 + 1 <= t ? c[2 * e + 1] * (ex2(gt - g1) * f1) : 0.f, hi, lo);
+        *(uint32_t *) (hr + a_off(t, s0)) = hi;
+        *(uint32_t *) (hr + R::ATILE + a_off(t, s0)) = lo;
+    }
 }
 
+// ---- pass --------------------------------------------------------------------------------------------------------------------------
 template <int KIND, int K> struct Pass {
     using R = Rec<KIND, K>;
     static constexpr int KS = K / 32;                        // warps that share a head's 16 value columns, 32 key channels each
-    static constexpr int NG = (per_head(KIND) ? 8 : 4) / KS; // groups of 16 columns
+    static constexpr int NG = (KIND == SSD ? 8 : 4) / KS;    // groups of 16 columns
     static constexpr int WARPS = KS * NG, PT = WARPS * 32, PV = NG * 16;
     static constexpr int STAGES = KIND == DELTA ? 3 : 4;
     static constexpr int XS = PV * 2 + 16;                   // bytes of a row of v: rows hit different banks
@@ -773,14 +842,18 @@ template <int KIND, int K> int run_chunks(const jib_state_mix & a, cudaStream_t 
     const int rc = launched();
     return rc ? rc : launch_pass<KIND, K>(a, s);
 }
-template <int KIND, int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
+template <int K> int run_chunks_mlstm(const jib_state_mix & a, cudaStream_t s) {
+    JIB_LAUNCH((chunk_prepare_mlstm_kernel<K>), dim3(a.T / C + a.n_seqs, a.H), NT, 0, s, a);
+    const int rc = launched();
+    return rc ? rc : launch_pass<MLSTM, K>(a, s);
+}
+template <int K> int run_chunks_ssd(const jib_state_mix & a, cudaStream_t s) {
     static std::atomic<unsigned char> done[jib::MAX_DEVICES];
     constexpr int smem = (2 * C * (K + 4) + C * (C + 1)) * 4;
-    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<KIND, K>, smem, done)) return JIB_E_LAUNCH;
-    const int values = KIND == MLSTM ? 0 : (a.H * a.V + 255) / 256;      // MLSTM: the pass reads them where they are
-    JIB_LAUNCH((chunk_prepare_ssd_kernel<KIND, K>), dim3(a.T / C + a.n_seqs, a.H / a.rep * ((a.rep + HB - 1) / HB) + values), NT, smem, s, a);
+    if (!jib::ensure_dyn_smem(chunk_prepare_ssd_kernel<K>, smem, done)) return JIB_E_LAUNCH;
+    JIB_LAUNCH((chunk_prepare_ssd_kernel<K>), dim3(a.T / C + a.n_seqs, a.H / a.rep * ((a.rep + HB - 1) / HB) + (a.H * a.V + 255) / 256), NT, smem, s, a);
     const int rc = launched();
-    return rc ? rc : launch_pass<KIND, K>(a, s);
+    return rc ? rc : launch_pass<SSD, K>(a, s);
 }
 
 long long rec_bytes(const jib_state_mix & a) {
@@ -795,6 +868,7 @@ long long rec_bytes(const jib_state_mix & a) {
 
 bool jib_state_chunk_ok(const jib_state_mix & a) {
     const long long cols = a.ld | a.q_off | a.k_off | a.v_off | a.conv0 | a.n_conv | (per_head(a.kind) ? 0 : a.ld_dec);
+    if (a.kind == MLSTM && (a.q_off | a.k_off) % 8) return false;
     if ((a.kind == HGRN || a.kind == MLSTM) && (a.ld % 8 || a.v_off % 8 || a.taps != 0 || ((uintptr_t) a.proj & 15))) return false;
     return (a.K == 64 || a.K == 128) && a.V % 16 == 0 && a.V <= 256 && a.taps <= 4 && cols % 4 == 0 && ((uintptr_t) a.proj & 7) == 0 &&
            (per_head(a.kind) || ((uintptr_t) a.dec_in & 7) == 0) && a.H % a.rep == 0;
@@ -806,8 +880,8 @@ int jib_state_chunk_run(const jib_state_mix & a, cudaStream_t s) {
         case DELTA: return a.K == 64 ? run_chunks<DELTA, 64>(a, s) : run_chunks<DELTA, 128>(a, s);
         case LINEAR: return a.K == 64 ? run_chunks<LINEAR, 64>(a, s) : run_chunks<LINEAR, 128>(a, s);
         case HGRN: return a.K == 64 ? run_chunks<HGRN, 64>(a, s) : run_chunks<HGRN, 128>(a, s);
-        case MLSTM: return a.K == 64 ? run_chunks_ssd<MLSTM, 64>(a, s) : run_chunks_ssd<MLSTM, 128>(a, s);
-        default: return a.K == 64 ? run_chunks_ssd<SSD, 64>(a, s) : run_chunks_ssd<SSD, 128>(a, s);
+        case MLSTM: return a.K == 64 ? run_chunks_mlstm<64>(a, s) : run_chunks_mlstm<128>(a, s);
+        default: return a.K == 64 ? run_chunks_ssd<64>(a, s) : run_chunks_ssd<128>(a, s);
     }
 }
 

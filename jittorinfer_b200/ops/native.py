@@ -916,9 +916,10 @@ def gqa_qkv_post(m, q, k, v, rope_table, positions, slot_mapping, cache, v_first
 
 
 def gqa_splits(m, T, max_keys, sm_count=148):
-    """CTAs that share one row's keys in a batch of single tokens: as many as fill the machine, at most one per 64 visible keys."""
+    """CTAs that share one row's keys in a batch of single tokens: as many as the machine holds at a time (three on an SM), at most one per 64
+    visible keys."""
     keys = min([x for x in (m.window, m.chunk, max_keys) if x > 0]) + (max_keys // m.pool if m.pool else 0)
-    fill = max(1, 4 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
+    fill = max(1, 3 * sm_count // max(1, T * m.kv_heads * ((m.heads // m.kv_heads + 15) // 16)))
     n = min(8, fill, (keys + 63) // 64)
     return 1 << (n.bit_length() - 1)
 
