@@ -163,13 +163,26 @@ __device__ __forceinline__ float unary(float v, const GemmArgs & a) {
 }
 // FN instances: 0 the product itself, 1 relu^2 and softcap, 2 gelu of the product times its row's factor (a row past the tile's last has none),
 // 3 the product plus its feature's bias (an epilogue thread holds one feature: a register).
+// erfc(|z|) by Abramowitz and Stegun's formula 7.1.26 (absolute error 1.5e-7): a polynomial in 1 / (1 + p |z|) times e^{-z^2}.
+__device__ __forceinline__ float gelu(float v) {
+    const float z = fabsf(v) * 0.70710678118654752f;
+    float t, e;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(1.f + 0.3275911f * z));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * z * z));
+    const float p = t * (0.254829592f + t * (-0.284496736f + t * (1.421413741f + t * (-1.453152027f + t * 1.061405429f))));
+    const float half = 0.5f * v * (p * e);                   // v erfc(|z|) / 2
+    return v > 0.f ? v - half : half;
+}
+__device__ __forceinline__ float row_factor(const GemmArgs & a, long long row, bool valid) {
+    return a.row_scale != nullptr && valid ? __ldg(a.row_scale + row) : 1.f;
+}
+// by: the row's factor (FN 2) or the feature's bias (FN 3)
 template <int FN>
-__device__ __forceinline__ float function_of(float v, const GemmArgs & a, long long row, bool valid, float bias) {
+__device__ __forceinline__ float function_of(float v, const GemmArgs & a, float by) {
     if (FN == 0) return v;
-    if (FN == 3) return v + bias;
+    if (FN == 3) return v + by;
     if (FN == 1) return unary(v, a);
-    if (a.row_scale != nullptr && valid) v *= __ldg(a.row_scale + row);
-    return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+    return gelu(v * by);
 }
 
 // Cluster-wide barrier (all threads of all CTAs of the cluster) and a load from a peer CTA's shared memory.
@@ -409,7 +422,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
         auto finish = [&](int t_rel, float gv, float uv) {
             const long long row = row_base + t_rel;
             if (row >= args.rows_total) { jib_report(args.status, JIB_ERR_BOUNDS, 5, (int) row); return; }
-            float y = DUAL ? gated(gv, args.act) * uv : function_of<FN>(gv, args, row, true, bias);
+            float y = DUAL ? gated(gv, args.act) * uv : function_of<FN>(gv, args, FN == 2 ? row_factor(args, row, true) : bias);
             if (args.ar_on == 2) {      // two-shot: the partial goes to the tile's owner only
                 args.ar.recv2[ar_owner][ar_par + ((size_t) args.ar.rank * args.ar.max_rows2 + row) * args.ar.d_max + n] = y;
                 return;
@@ -583,9 +596,14 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                     // adjacent features of one token row as one 16-byte vector (residual added in fp32 before rounding).
                     const int ltid = (int) threadIdx.x - 64;
                     float * sb = stage + ((c >> 4) & 1) * (16 * BM);
+                    float by[FN == 2 ? 16 : 1];
+                    if (FN == 2) {
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j]
-                                                                          : function_of<FN>(g[j], args, (long long) row_base + row0 + c + j, c + j < ncols, bias);
+                        for (int j = 0; j < 16; ++j) by[FN == 2 ? j : 0] = row_factor(args, (long long) row_base + row0 + c + j, c + j < ncols);
+                    }
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        sb[j * BM + r] = DUAL ? gated(g[j], args.act) * u[j] : function_of<FN>(g[j], args, FN == 2 ? by[FN == 2 ? j : 0] : bias);
                     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1
                     for (int it = 0; it < 2; ++it) {
@@ -868,6 +886,11 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
             for (int c = 0; c < BN; c += 16) {
                 if (c >= ncols) break;
                 uint32_t gv[16], uv[16];
+                float by[FN == 2 ? 16 : 1];
+                if (FN == 2) {
+#pragma unroll
+                    for (int k = 0; k < 16; ++k) by[FN == 2 ? k : 0] = row_factor(args, (long long) t.row_base + t.row0 + c + k, c + k < ncols);
+                }
                 tmem_ld16(tbase + c, gv);
                 if (DUAL) tmem_ld16(tbase + BN + c, uv);
                 tmem_ld_wait();
@@ -876,7 +899,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_con
                 for (int k = 0; k < 16; ++k) {
                     const float g = __uint_as_float(gv[k]);
                     sb[k * BM + r] = DUAL ? gated(g, args.act) * __uint_as_float(uv[k])
-                                          : function_of<FN>(g, args, (long long) t.row_base + t.row0 + c + k, c + k < ncols, bias);
+                                          : function_of<FN>(g, args, FN == 2 ? by[FN == 2 ? k : 0] : bias);
                 }
                 asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll 1

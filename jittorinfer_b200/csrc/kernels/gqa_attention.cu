@@ -897,12 +897,12 @@ int launch_mma_as(const jib_gqa & a, const void * q, const void * gate, long lon
     return launched();
 }
 
-// Three tiles in shared memory while two CTAs fit on an SM
+// Three tiles in shared memory while two CTAs fit on an SM; two where the keys are split over CTAs that have one or two tiles each
 template <int NV>
 int launch_mma(const jib_gqa & a, const void * q, const void * gate, long long ld_gate, void * out, long long ldo, int single, int splits,
                cudaStream_t s) {
     const int smem = ROWS * (a.D + PADC) * 2 + 3 * MK * (a.D + a.V + 2 * PADC) * 2;
-    return smem <= 112 * 1024 ? launch_mma_as<NV, 3>(a, q, gate, ld_gate, out, ldo, single, splits, s)
+    return smem <= 112 * 1024 && splits == 1 ? launch_mma_as<NV, 3>(a, q, gate, ld_gate, out, ldo, single, splits, s)
                               : launch_mma_as<NV, 2>(a, q, gate, ld_gate, out, ldo, single, splits, s);
 }
 

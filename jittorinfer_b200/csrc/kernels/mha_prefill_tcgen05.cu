@@ -79,6 +79,12 @@ __host__ __device__ __forceinline__ int visible_rows(int S, int q_len, int windo
     return S <= 0 ? S : S - gqa_first_key(S > q_len ? S - q_len : 0, window, chunk);
 }
 
+__device__ __forceinline__ float ex2(float x) {                // 2^x; results below the smallest normal number are 0
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // softcap * tanh(score * scale / softcap) * log2 e from the raw product
 __device__ __forceinline__ float capped_log2(float s, const MhaArgs & a) {
     float e, r;
@@ -294,19 +300,19 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
                     for (int c = 0; c < KT; ++c) x[c] = (POOL ? (unsigned) (c - inv) < span || c < pooled : c < vis && c >= inv) ? x[c] : -INFINITY;
                 }
-#pragma unroll
-                for (int c = 0; c < KT; ++c) mt = fmaxf(mt, x[c]);
             } else if (need_mask) {
 #pragma unroll
                 for (int c = 0; c < KT; ++c) {
                     const bool see = POOL ? (unsigned) (c - inv) < span || c < pooled : c < vis && c >= inv;
                     x[c] = see ? x[c] * a.scale_log2e : -INFINITY;
-                    mt = fmaxf(mt, x[c]);
                 }
             } else {
 #pragma unroll
-                for (int c = 0; c < KT; ++c) { x[c] *= a.scale_log2e; mt = fmaxf(mt, x[c]); }
+                for (int c = 0; c < KT; ++c) x[c] *= a.scale_log2e;
             }
+            // one warp per scheduler: maxima and sums of four keep the chains short
+#pragma unroll
+            for (int c = 0; c < KT; c += 4) mt = fmaxf(mt, fmaxf(fmaxf(x[c], x[c + 1]), fmaxf(x[c + 2], x[c + 3])));
             // the exponent base follows the maximum only when it has fallen behind by more than RESCALE_LAG
             const bool grow = mt > m_ref + RESCALE_LAG || m_ref == -INFINITY;
             const float m_new = grow ? mt : m_ref;
@@ -338,11 +344,12 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             const float base_l2 = m_ref == -INFINITY ? 0.f : m_ref;   // every x is -inf then: p = 0
             uint32_t packed[KT / 2];
 #pragma unroll
-            for (int c = 0; c < KT; c += 2) {
-                const float p0 = exp2f(x[c] - base_l2), p1 = exp2f(x[c + 1] - base_l2);
-                l_sum += p0 + p1;
-                const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
+            for (int c = 0; c < KT; c += 4) {
+                const float p0 = ex2(x[c] - base_l2), p1 = ex2(x[c + 1] - base_l2), p2 = ex2(x[c + 2] - base_l2), p3 = ex2(x[c + 3] - base_l2);
+                l_sum += (p0 + p1) + (p2 + p3);
+                const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1), pl = __floats2bfloat162_rn(p2, p3);
                 packed[c >> 1] = *(const uint32_t *) &pk;
+                packed[(c >> 1) + 1] = *(const uint32_t *) &pl;
             }
             // the previous P.V must have read P before it is overwritten
             if (kt > 0 && !mbar_wait(p_empty, (kt - 1) & 1)) { jib_report(a.status, JIB_ERR_WAIT_TIMEOUT, 38, kt); ok = false; }
