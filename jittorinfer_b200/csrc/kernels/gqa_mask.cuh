@@ -15,6 +15,9 @@ __host__ __device__ __forceinline__ int gqa_blocks_seen(int p, int window, int p
     return pool > 0 && p - window + 1 >= pool ? (p - window + 1) / pool : 0;
 }
 
+// Gathered for a prompt, the pooled rows fill whole tiles of 128 rows (the last is padded with zeros), so that a window of whole tiles stays so.
+__host__ __device__ __forceinline__ int gqa_pool_gathered(int blocks) { return (blocks + 127) / 128 * 128; }
+
 // Row of pooled block b: the pooled blocks that end in a cache block go with it, `rows` places for each.
 __device__ __forceinline__ long long gqa_pool_row(const int * block_table, int b, int pool, int rows, int block_size) {
     const int page = ((b + 1) * pool - 1) / block_size;

@@ -172,7 +172,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         base_pos = a.seq_lens[b] - S;
         ctx0 = S - q_len;                             // gathered rows before this chunk
         if (POOL) {
-            const int np = gqa_blocks_seen(a.seq_lens[b] - 1, a.window, a.pool_size);
+            const int np = gqa_pool_gathered(gqa_blocks_seen(a.seq_lens[b] - 1, a.window, a.pool_size));
             ctx0 += np;
             base_pos -= np;
         }
@@ -419,7 +419,7 @@ mha_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 
 // ---- latent rows of the sequences of a batch, gathered from the paged cache into one contiguous buffer ---------------------
 // lat [total][row] <- cache[block_tables[b][s / bs] * bs + s % bs][row] for s < seq_lens[b] (with a window: for the rows the
-// sequence's last q_len tokens can see, and ahead of them the pooled rows its last token sees); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
+// sequence's last q_len tokens can see, and ahead of them the pooled rows its last token sees, see gqa_pool_gathered); kv_start[b] = first row of sequence b (exclusive prefix of the row counts).  grid (ceil(max rows / 8), 1): every CTA walks the sequence table itself.
 __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict__ cache, const int * __restrict__ block_tables, int max_blocks,
                                                         const int * __restrict__ seq_lens, int n_seqs, int block_size, int row_elems,
                                                         long long n_slots, const int * __restrict__ q_start, int window, int chunk,
@@ -429,19 +429,28 @@ __global__ void __launch_bounds__(256) kv_gather_kernel(const bf16 * __restrict_
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = blockIdx.x * 8 + warp;              // global row of the gathered buffer this warp copies
     int b = -1, s = 0, acc = 0;                       // s < 0: pooled row -1 - s
+    bool padding = false;
     for (int i = 0; i < n_seqs; ++i) {
         const int S = seq_lens[i], n = window > 0 || chunk > 0 ? visible_rows(S, q_start[i + 1] - q_start[i], window, chunk) : S;
-        const int np = gqa_blocks_seen(S - 1, window, pool_size);
+        const int seen = gqa_blocks_seen(S - 1, window, pool_size), np = gqa_pool_gathered(seen);
         if (blockIdx.x == 0 && threadIdx.x == 0) kv_start[i] = acc;
-        if (b < 0 && g < acc + np + n) { b = i; s = g < acc + np ? acc - g - 1 : S - n + g - acc - np; }
+        if (b < 0 && g < acc + np + n) {
+            b = i;
+            s = g < acc + np ? acc - g - 1 : S - n + g - acc - np;
+            padding = s < 0 && -1 - s >= seen;
+        }
         acc += np + n;
     }
     if (b < 0 || g >= total_cap) return;
+    uint4 * dst = (uint4 *) (lat + (size_t) g * row_elems);
+    if (padding) {
+        for (int i = lane; i < row_elems / 8; i += 32) dst[i] = make_uint4(0, 0, 0, 0);
+        return;
+    }
     const int * bt = block_tables + (size_t) b * max_blocks;
     const long long slot = s < 0 ? gqa_pool_row(bt, -1 - s, pool_size, pool_rows, block_size) : (long long) bt[s / block_size] * block_size + s % block_size;
     if (slot < 0 || (s >= 0 && slot >= n_slots)) return;
     const uint4 * src = (const uint4 *) ((s < 0 ? pool : cache) + (size_t) slot * row_elems);
-    uint4 * dst = (uint4 *) (lat + (size_t) g * row_elems);
     for (int i = lane; i < row_elems / 8; i += 32) dst[i] = src[i];
 }
 

@@ -490,7 +490,7 @@ def visible_total(meta, window: int, chunk: int = 0, pool: int = 0) -> int:
     """Cached rows the queries of a step can see, pooled ones included, over its sequences (what ``kv_gather`` writes)."""
     if window <= 0 and chunk <= 0:
         return int(meta["total_kv"])
-    pooled = sum(max(0, int(s) - window) // pool for s in meta["s_lens"]) if pool else 0
+    pooled = sum((max(0, int(s) - window) // pool + 127) // 128 * 128 for s in meta["s_lens"]) if pool else 0       # in whole tiles of 128 rows
     return pooled + sum(visible_rows(int(q), int(s), window, chunk) for q, s in zip(meta["q_lens"], meta["s_lens"]))
 
 

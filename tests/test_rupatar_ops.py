@@ -394,3 +394,11 @@ def test_sigmoid_router_keeps_its_scores(dev, dtype):
     got = torch.zeros(T, E + 2, dtype=torch.float64).scatter_(1, ids.long().cpu(), wts.double().cpu())
     close(got[:, :E], O.route(x.double() @ w.double().T, top), F32, scale=10)
     assert bool((got[:, E:] == 1).all()) and math.isclose(float(O.gelu(torch.tensor(1.0, dtype=torch.float64))), 0.8413447460685429)
+
+
+def test_gathered_rows_count_whole_tiles_of_pooled_rows():
+    from jittorinfer_b200.ops import native
+    meta = {"total_kv": 5000, "q_lens": [500, 1, 30], "s_lens": [2000, 3000, 90]}
+    seen = [len(O.seen_blocks(s - 1, 100, 16)) for s in meta["s_lens"]]
+    assert seen == [118, 181, 0]
+    assert native.visible_total(meta, 100, 0, 16) == 128 + 599 + 256 + 100 + 0 + 90 and native.visible_total(meta, 100) == 599 + 100 + 90
